@@ -1,6 +1,8 @@
 """Build the native libraries in-tree with nvcc / g++ (no JIT cache, no torch headers):
 
   xfastertransformer_b200/lib/libxft_b200_kernels.so   all sm_100a CUDA kernels, C ABI
+  xfastertransformer_b200/lib/libxft_b200_layered.so   the subset of them that a layered bf16 / fp32 model calls; built by
+                                                        bin/trace_run when the full library is not there
   xfastertransformer_b200/lib/libxft_b200_core.so      C++ runtime (INI, loader, sequences, paged KV, samplers,
                                                         xft::Model C++ API)
 
@@ -22,6 +24,12 @@ NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
 NVFLAGS = ARCH + ["-lineinfo", "-O3", "-std=c++17", "-Xcompiler", "-fPIC", "--use_fast_math", "-Xptxas", "-v"]
 
+# sources that need the accurate division, expf and tanhf
+ACCURATE = {"plain.cu"}
+# what a layered model calls: GEMMs, attention, norms, rotary + cache append, arg-max, and what these link against
+LAYERED = ["attention.cu", "attention_prefill_sm100.cu", "elementwise.cu", "gemm_decode_sm100.cu",
+           "gemm_prefill_sm100.cu", "gemm_sm100.cu", "plain.cu", "residual_norm.cu"]
+
 
 def _newer(src, dst, deps=()):
     if not os.path.exists(dst):
@@ -40,23 +48,42 @@ def _run(cmd, verbose):
     return r.stderr
 
 
-def build(force=False, verbose=False):
+def build_kernels(cus, name, force=False, verbose=False):
+    """Compile the kernel sources `cus` (those that changed) and link them into lib/<name>."""
     os.makedirs(OUT, exist_ok=True)
     os.makedirs(OBJ, exist_ok=True)
     kdir = os.path.join(HERE, "kernels")
     headers = tuple(os.path.join(kdir, f) for f in os.listdir(kdir) if f.endswith((".cuh", ".h")))
-    cus = sorted(f for f in os.listdir(kdir) if f.endswith(".cu"))
     objs, jobs = [], []
     for f in cus:
         src, obj = os.path.join(kdir, f), os.path.join(OBJ, f[:-3] + ".o")
         objs.append(obj)
         if force or _newer(src, obj, headers):
-            jobs.append([NVCC] + NVFLAGS + ["-c", src, "-o", obj])
+            flags = [x for x in NVFLAGS if f not in ACCURATE or x != "--use_fast_math"]
+            jobs.append([NVCC] + flags + ["-c", src, "-o", obj])
     with ThreadPoolExecutor(max_workers=8) as ex:
         logs = list(ex.map(lambda c: _run(c, verbose), jobs))
-    lib = os.path.join(OUT, "libxft_b200_kernels.so")
-    if jobs or not os.path.exists(lib):
-        _run([NVCC] + ARCH + ["-shared", "-o", lib] + objs + ["-lcudart"], verbose)
+    lib = os.path.join(OUT, name)
+    if jobs or not os.path.exists(lib) or any(_newer(o, lib) for o in objs):
+        part = lib + ".part"
+        _run([NVCC] + ARCH + ["-shared", "-o", part] + objs + ["-lcudart"], verbose)
+        os.replace(part, lib)
+    return lib, jobs, logs
+
+
+def build_layered(verbose=False):
+    """The kernels of a layered model, unless the full library is there and no older than its sources."""
+    full = os.path.join(OUT, "libxft_b200_kernels.so")
+    kdir = os.path.join(HERE, "kernels")
+    if os.path.exists(full) and not any(_newer(os.path.join(kdir, f), full) for f in os.listdir(kdir)):
+        return full
+    return build_kernels(LAYERED, "libxft_b200_layered.so", False, verbose)[0]
+
+
+def build(force=False, verbose=False):
+    kdir = os.path.join(HERE, "kernels")
+    cus = sorted(f for f in os.listdir(kdir) if f.endswith(".cu"))
+    lib, jobs, logs = build_kernels(cus, "libxft_b200_kernels.so", force, verbose)
     # C++ runtime (links the kernel library; $ORIGIN rpath keeps the pair relocatable) and the example CLI
     cdir = os.path.join(HERE, "core")
     api = os.path.join(HERE, "api")

@@ -17,6 +17,10 @@
 // last merges all slices.  bf16 caches are fed by TMA into a CTA-wide ring (attn_decode_tma_kernel); int8 caches
 // keep the cp.async path, which converts to bf16 on the way into shared memory.  Prefill gives each warp 16 query rows of one head and shares K/V tiles
 // across the CTA.
+//
+// The EXT instantiations add, with their constants as launch parameters: a sliding window with kept first keys (position
+// i sees j <= i when i - j < window or j < keep; only tiles that hold a visible key are visited), a tanh cap on the
+// scores, and one sink per query head (a term of the softmax denominator that has no key and no value).
 #include "ptx.cuh"
 
 namespace xft {
@@ -43,6 +47,31 @@ struct AttnParams {
   int nsplit; float* part_o; float* part_ml;   // [B, hq, nsplit, HD], [B, hq, nsplit, 2]
   int* split_counters;      // [B * gridDim.y] arrival counters (zero between launches)
   int* status;
+  // EXT only
+  float softcap, inv_cap2;  // cap and 2 / cap (softcap 0: none)
+  int window, keep;         // window 2^30: every earlier key is visible
+  const float* sinks;       // [hq] or null
+};
+
+// softcap * tanh(x / softcap) with tanh(y) = 1 - 2 / (1 + exp(2y))
+__device__ __forceinline__ float cap_score(const AttnParams& p, float x) {
+  return p.softcap > 0.f ? p.softcap - __fdividef(2.f * p.softcap, 1.f + __expf(fminf(x * p.inv_cap2, 80.f))) : x;
+}
+
+// The key tiles (KT keys each) that hold a key visible to a query at position >= qlo, in visiting order: tiles of the
+// kept first keys, then the tiles from the window's first key up to `end`.
+template <bool EXT>
+struct TileList {
+  int n_keep, lo, n;
+  __device__ __forceinline__ TileList(const AttnParams& p, int qlo, int end, int KT) {
+    n_keep = lo = 0;
+    if (EXT) {
+      lo = min(max(0, qlo - p.window + 1) / KT, end);
+      n_keep = min((p.keep + KT - 1) / KT, lo);
+    }
+    n = n_keep + end - lo;
+  }
+  __device__ __forceinline__ int at(int i) const { return EXT ? (i < n_keep ? i : i - n_keep + lo) : i; }
 };
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
@@ -113,7 +142,7 @@ __device__ __forceinline__ void load_tile_int8(bf16* tile, const int8_t* g, int 
 
 // One warp: 16 query rows (A fragments re-read from the swizzled Q tile) against a KT-key tile.
 // Updates the running max m[2], sum l[2] and O accumulator (two rows per thread: lane/4 and lane/4+8).
-template <int HD, int KT, bool KV_TMA = false, int TROWS = KT>
+template <int HD, int KT, bool KV_TMA = false, int TROWS = KT, bool EXT = false>
 struct WarpAttn {
   float m[2], l[2];
   float o[HD / 8][4];
@@ -130,14 +159,22 @@ struct WarpAttn {
     for (int i = 0; i < HD / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
   }
 
+  // EXT: the two rows start from their sinks (row sums are per-lane partials, so one lane of the quad counts it)
+  __device__ __forceinline__ void init_sinks(float s0, float s1, int lane) {
+    m[0] = s0;
+    m[1] = s1;
+    l[0] = (lane & 3) == 0 && s0 != -INFINITY ? 1.f : 0.f;
+    l[1] = (lane & 3) == 0 && s1 != -INFINITY ? 1.f : 0.f;
+  }
+
   // qtile: [16][HD] rows of this warp; kt/vt: [KT][HD]; key0: global index of key 0 of the tile.
   // qpos0/qpos1: positions of this thread's two query rows (-1 => row unused); kv_len bounds the keys.
   // kscale/vscale: per-key fp32 (smem) or null.
   __device__ __forceinline__ void step(const bf16* qtile, const bf16* kt, const bf16* vt, int key0, int kv_len, int qpos0,
                                        int qpos1, float scale, float slope0, float slope1, bool use_alibi, int prefix_len,
-                                       const float* kscale, const float* vscale, int lane) {
+                                       const float* kscale, const float* vscale, int lane, const AttnParams& p) {
     float s[KT / 8][4];
-    scores(s, qtile, kt, key0, kv_len, qpos0, qpos1, scale, slope0, slope1, use_alibi, prefix_len, kscale, vscale, lane);
+    scores(s, qtile, kt, key0, kv_len, qpos0, qpos1, scale, slope0, slope1, use_alibi, prefix_len, kscale, vscale, lane, p);
     pv(s, vt, lane);
   }
 
@@ -179,7 +216,7 @@ struct WarpAttn {
   // scale, bias, mask; thread holds rows r0 = lane/4 (c0,c1) and r0+8 (c2,c3), key cols j*8 + 2*(lane%4) + {0,1}
   __device__ __forceinline__ void mask(float (&s)[KT / 8][4], int key0, int kv_len, int qpos0, int qpos1, float scale,
                                        float slope0, float slope1, bool use_alibi, int prefix_len, const float* kscale,
-                                       int lane) {
+                                       int lane, const AttnParams& p) {
 #pragma unroll
     for (int j = 0; j < KT / 8; ++j) {
 #pragma unroll
@@ -189,8 +226,10 @@ struct WarpAttn {
         const int qp = (e < 2) ? qpos0 : qpos1;
         float v = s[j][e] * scale;
         if (kscale) v *= kscale[kl];
+        if (EXT) v = cap_score(p, v);
         if (use_alibi) v += ((e < 2) ? slope0 : slope1) * (float)(key - qp);
-        const bool vis = key < kv_len && qp >= 0 && (key <= qp || key < prefix_len);
+        bool vis = key < kv_len && qp >= 0 && (key <= qp || key < prefix_len);
+        if (EXT) vis = vis && (qp - key < p.window || key < p.keep);
         s[j][e] = vis ? v : -INFINITY;
       }
     }
@@ -235,9 +274,10 @@ struct WarpAttn {
   // phase 1: S = Q K^T, mask, online-softmax update; leaves P (scaled by vscale) in s and rescales O
   __device__ __forceinline__ void scores(float (&s)[KT / 8][4], const bf16* qtile, const bf16* kt, int key0, int kv_len,
                                          int qpos0, int qpos1, float scale, float slope0, float slope1, bool use_alibi,
-                                         int prefix_len, const float* kscale, const float* vscale, int lane) {
+                                         int prefix_len, const float* kscale, const float* vscale, int lane,
+                                         const AttnParams& p) {
     qk(s, qtile, kt, lane);
-    mask(s, key0, kv_len, qpos0, qpos1, scale, slope0, slope1, use_alibi, prefix_len, kscale, lane);
+    mask(s, key0, kv_len, qpos0, qpos1, scale, slope0, slope1, use_alibi, prefix_len, kscale, lane, p);
     softmax_update(s, vscale, lane);
   }
 
@@ -271,7 +311,7 @@ struct WarpAttn {
 
 // ------------------------------------------------------------------------------------------ prefill
 // grid (q tiles of 64 rows, hq, B); 128 threads; K/V tiles of KT keys double-buffered.
-template <int HD, int KT, bool INT8>
+template <int HD, int KT, bool INT8, bool EXT>
 __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
   extern __shared__ __align__(128) uint8_t smem_raw[];
   bf16* qs = reinterpret_cast<bf16*>(smem_raw);                 // [64][HD]
@@ -290,7 +330,8 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
   const int prefix_len = p.prefix_lens ? p.prefix_lens[b] : 0;
   // keys needed by this tile: up to the position of its last row (or the prefix)
   int k_end = min(kv_len, max(pos_base + r0 + rows, prefix_len));
-  const int ntiles = (k_end + KT - 1) / KT;
+  const TileList<EXT> tiles(p, pos_base + r0, (k_end + KT - 1) / KT, KT);
+  const int ntiles = tiles.n;
   const int* bt = p.block_table + (size_t)b * p.bt_stride;
   const int tiles_per_block = p.bs / KT;
 
@@ -315,8 +356,9 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
     }
   };
 
-  WarpAttn<HD, KT> wa;
+  WarpAttn<HD, KT, false, KT, EXT> wa;
   wa.init();
+  if (EXT && p.sinks) wa.init_sinks(p.sinks[h], p.sinks[h], lane);
   const int rq0 = r0 + warp * 16 + (lane >> 2), rq1 = rq0 + 8;
   const int qpos0 = rq0 < q_len ? pos_base + rq0 : -1;
   const int qpos1 = rq1 < q_len ? pos_base + rq1 : -1;
@@ -324,18 +366,18 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
   const float slope = use_alibi ? p.slopes[h] : 0.f;
   const int warp_last_pos = pos_base + min(r0 + warp * 16 + 15, q_len - 1);
 
-  if (ntiles > 0) issue(0, 0);
+  if (ntiles > 0) issue(tiles.at(0), 0);
   cp_async_commit();
-  for (int ti = 0; ti < ntiles; ++ti) {
-    const int buf = ti & 1;
-    if (ti + 1 < ntiles) issue(ti + 1, buf ^ 1);
+  for (int n = 0; n < ntiles; ++n) {
+    const int buf = n & 1, ti = tiles.at(n);
+    if (n + 1 < ntiles) issue(tiles.at(n + 1), buf ^ 1);
     cp_async_commit();
     cp_async_wait<1>();
     __syncthreads();
     // skip tiles entirely above this warp's causal frontier (still take part in the barriers)
     if (ti * KT <= max(warp_last_pos, prefix_len - 1) && r0 + warp * 16 < q_len)
       wa.step(qs + warp * 16 * HD, kbuf + buf * KT * HD, vbuf + buf * KT * HD, ti * KT, kv_len, qpos0, qpos1, p.scale, slope,
-              slope, use_alibi, prefix_len, INT8 ? sc + (buf * 2 + 0) * KT : nullptr, INT8 ? sc + (buf * 2 + 1) * KT : nullptr, lane);
+              slope, use_alibi, prefix_len, INT8 ? sc + (buf * 2 + 0) * KT : nullptr, INT8 ? sc + (buf * 2 + 1) * KT : nullptr, lane, p);
     __syncthreads();
   }
   wa.reduce_l();
@@ -432,7 +474,7 @@ __device__ __forceinline__ void decode_finish(const AttnParams& p, WA& wa, float
 // ------------------------------------------------------------------------------------------ decode
 // grid (B, hkv * qchunks, nsplit); 128 threads; each warp walks its own tiles with private buffers.
 // Requires q_len == 1 for every sequence.
-template <int HD, int KT, bool INT8>
+template <int HD, int KT, bool INT8, bool EXT>
 __global__ void __launch_bounds__(128) attn_decode_kernel(const AttnParams p) {
   extern __shared__ __align__(128) uint8_t smem_raw[];
   bf16* qs = reinterpret_cast<bf16*>(smem_raw);                 // [16][HD]
@@ -452,7 +494,8 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const AttnParams p) {
   const int h_hi = min(min(p.hq, (kvh + 1) * p.group - p.q_off), h_lo + 16);
   const int nq = h_hi - h_lo;
   if (nq <= 0) return;
-  const int ntiles = (kv_len + KT - 1) / KT;
+  const TileList<EXT> tiles(p, kv_len - 1, (kv_len + KT - 1) / KT, KT);
+  const int ntiles = tiles.n;
   const int per = (ntiles + p.nsplit - 1) / p.nsplit;
   const int t_begin = split * per, t_end = min(ntiles, t_begin + per);
   const int* bt = p.block_table + (size_t)b * p.bt_stride;
@@ -469,8 +512,9 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const AttnParams p) {
   float* ksc = scb + warp * 2 * KT;
   float* vsc = ksc + KT;
 
-  auto issue_k = [&](int ti) {
-    if (ti < t_end) {
+  auto issue_k = [&](int n) {
+    if (n < t_end) {
+      const int ti = tiles.at(n);
       int blk = bt[ti / tiles_per_block];
       if (blk < 0 || blk >= p.num_blocks) { if (lane == 0 && p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); blk = 0; }
       const size_t row0 = ((size_t)blk * p.hkv + kvh) * p.bs + (ti % tiles_per_block) * KT;
@@ -484,8 +528,9 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const AttnParams p) {
     }
     cp_async_commit();
   };
-  auto issue_v = [&](int ti) {
-    if (ti < t_end) {
+  auto issue_v = [&](int n) {
+    if (n < t_end) {
+      const int ti = tiles.at(n);
       int blk = bt[ti / tiles_per_block];
       if (blk < 0 || blk >= p.num_blocks) blk = 0;
       const size_t row0 = ((size_t)blk * p.hkv + kvh) * p.bs + (ti % tiles_per_block) * KT;
@@ -502,9 +547,11 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const AttnParams p) {
 
   // Each warp runs its tiles as one "row block" of 16 rows where row r = head h_lo + r; all rows share
   // the query position kv_len-1.  S and P V are computed for all 16 rows (unused rows are zero queries).
-  WarpAttn<HD, KT> wa;
+  WarpAttn<HD, KT, false, KT, EXT> wa;
   wa.init();
   const int r0 = lane >> 2, r1 = r0 + 8;
+  if (EXT && p.sinks && split == 0 && warp == 0)       // the sink counts once per row: the first warp of the first slice
+    wa.init_sinks(r0 < nq ? p.sinks[h_lo + r0] : -INFINITY, r1 < nq ? p.sinks[h_lo + r1] : -INFINITY, lane);
   const int qpos = kv_len - 1;
   const int qpos0 = r0 < nq ? qpos : -1, qpos1 = r1 < nq ? qpos : -1;
   const bool use_alibi = p.slopes != nullptr;
@@ -520,8 +567,8 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const AttnParams p) {
     float s[KT / 8][4];
     cp_async_wait<1>();          // K(ti) landed (V(ti) may still be in flight)
     __syncwarp();
-    wa.scores(s, qs, kt, ti * KT, kv_len, qpos0, qpos1, p.scale, slope0, slope1, use_alibi, 0, INT8 ? ksc : nullptr,
-              INT8 ? vsc : nullptr, lane);
+    wa.scores(s, qs, kt, tiles.at(ti) * KT, kv_len, qpos0, qpos1, p.scale, slope0, slope1, use_alibi, 0,
+              INT8 ? ksc : nullptr, INT8 ? vsc : nullptr, lane, p);
     __syncwarp();
     issue_k(ti + 4);             // K buffer is free again
     cp_async_wait<1>();          // V(ti) landed
@@ -545,14 +592,14 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const AttnParams p) {
 // any warp waiting on its own request.
 // Rows of a block past kv_len hold finite stale data (the pool starts zeroed), so P = 0 masks them exactly.
 constexpr int kDecTile = 64;            // keys per ring stage (= the cache block size granule)
-constexpr int kDecMaxBlocks = 512;      // block ids of this CTA's slice cached in shared memory
+constexpr int kDecMaxBlocks = 512;      // block ids of this CTA's tiles cached in shared memory
 template <int HD>
 struct DecCfg {
   static constexpr int STAGE_BYTES = 2 * kDecTile * HD * 2;
   static constexpr int STAGES = (96 * 1024) / STAGE_BYTES >= 3 ? (96 * 1024) / STAGE_BYTES : 3;
 };
 
-template <int HD>
+template <int HD, bool EXT>
 __global__ void __launch_bounds__(160, (HD <= 128 ? 2 : 1)) attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK,
                                                                                   const __grid_constant__ CUtensorMap tmV,
                                                                                   const AttnParams p) {
@@ -588,34 +635,31 @@ __global__ void __launch_bounds__(160, (HD <= 128 ? 2 : 1)) attn_decode_tma_kern
   const int h_hi = min(min(p.hq, (kvh + 1) * p.group - p.q_off), h_lo + 16);
   const int nq = h_hi - h_lo;
   if (nq <= 0) return;
-  const int ntiles = (kv_len + KT - 1) / KT;
+  const TileList<EXT> tiles(p, kv_len - 1, (kv_len + KT - 1) / KT, KT);
+  const int ntiles = tiles.n;
   const int per = (ntiles + p.nsplit - 1) / p.nsplit;
   const int t_begin = split * per, t_end = min(ntiles, t_begin + per);
   const int nloc = max(t_end - t_begin, 0);
   const int* bt = p.block_table + (size_t)b * p.bt_stride;
   const int tiles_per_block = p.bs / KT;
 
-  const int blk_first = t_begin / tiles_per_block;
-  const int nblk = nloc > 0 ? (t_end - 1) / tiles_per_block - blk_first + 1 : 0;
-  for (int i = tid; i < min(nblk, kDecMaxBlocks); i += 160) {
-    int blk = bt[blk_first + i];
+  for (int i = tid; i < min(nloc, kDecMaxBlocks); i += 160) {
+    int blk = bt[tiles.at(t_begin + i) / tiles_per_block];
     if (blk < 0 || blk >= p.num_blocks) { if (p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); blk = 0; }
     s_blk[i] = blk;
   }
   __syncthreads();
   // tiles of this slice that cannot hold the token appended in this step: their loads start before the kernel in
   // front has finished (the first STAGES tiles find their stage free without a wait)
-  const int newest_tile = (kv_len - 1) / KT;
-  const int npre = max(0, min(min(STAGES, nloc), newest_tile - t_begin));
+  const int npre = max(0, min(min(STAGES, nloc), ntiles - 1 - t_begin));      // the newest token's tile is the last one
   auto issue_tile = [&](int n) {
     const int st = n % STAGES;
-    const int ti = t_begin + n;
-    const int bi = ti / tiles_per_block - blk_first;
+    const int ti = tiles.at(t_begin + n);
     int blk;
-    if (bi < kDecMaxBlocks) {
-      blk = s_blk[bi];
+    if (n < kDecMaxBlocks) {
+      blk = s_blk[n];
     } else {
-      blk = bt[blk_first + bi];
+      blk = bt[ti / tiles_per_block];
       if (blk < 0 || blk >= p.num_blocks) { if (p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); blk = 0; }
     }
     const int row = (blk * p.hkv + kvh) * p.bs + (ti % tiles_per_block) * KT;
@@ -635,7 +679,7 @@ __global__ void __launch_bounds__(160, (HD <= 128 ? 2 : 1)) attn_decode_tma_kern
   cp_async_wait<0>();
   __syncthreads();
 
-  WarpAttn<HD, KW, true, KT> wa;
+  WarpAttn<HD, KW, true, KT, EXT> wa;
   wa.init();
   if (warp == 4) {
     if (lane == 0) {
@@ -647,6 +691,8 @@ __global__ void __launch_bounds__(160, (HD <= 128 ? 2 : 1)) attn_decode_tma_kern
     }
   } else {
     const int r0 = lane >> 2, r1 = r0 + 8;
+    if (EXT && p.sinks && split == 0 && warp == 0)
+      wa.init_sinks(r0 < nq ? p.sinks[h_lo + r0] : -INFINITY, r1 < nq ? p.sinks[h_lo + r1] : -INFINITY, lane);
     const int qpos = kv_len - 1;
     const int qpos0 = r0 < nq ? qpos : -1, qpos1 = r1 < nq ? qpos : -1;
     const bool use_alibi = p.slopes != nullptr;
@@ -664,13 +710,13 @@ __global__ void __launch_bounds__(160, (HD <= 128 ? 2 : 1)) attn_decode_tma_kern
       if (!mbar_wait(&full_bar[st], (n / STAGES) & 1, p.status, XFT_ERR_WAIT_FULL)) { s_abort = 1; break; }
       // this warp's 16 keys of the tile: rows warp*16 .. +15 of both halves (the row offset keeps row & 7)
       const bf16* kt = ring + (size_t)st * 2 * TILE + warp * KW * 64;
-      const int key0 = (t_begin + n) * KT + warp * KW;
+      const int key0 = tiles.at(t_begin + n) * KT + warp * KW;
       if (key0 < kv_len) {
         float s[KW / 8][4];
         if constexpr (QREG) wa.qk_frag(s, reinterpret_cast<const uint32_t (&)[HD / 16][4]>(qa), kt, lane);
         else wa.qk(s, qs, kt, lane);
-        if (use_alibi || key0 + KW > kv_len) {
-          wa.mask(s, key0, kv_len, qpos0, qpos1, p.scale, slope0, slope1, use_alibi, 0, nullptr, lane);
+        if (EXT || use_alibi || key0 + KW > kv_len) {
+          wa.mask(s, key0, kv_len, qpos0, qpos1, p.scale, slope0, slope1, use_alibi, 0, nullptr, lane, p);
         } else {
           // every key is visible; rows past nq carry a zero query and are never stored
 #pragma unroll
@@ -716,21 +762,21 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
 
 using namespace xft;
 
-template <int HD, int KT>
+template <int HD, int KT, bool EXT>
 static int launch_prefill(const AttnParams& p, int B, int max_q, bool int8, cudaStream_t st) {
   size_t smem = (size_t)(64 * HD + 4 * KT * HD) * 2 + 4 * KT * sizeof(float);
   dim3 grid((max_q + 63) / 64, p.hq, B);
   if (int8) {
-    cudaFuncSetAttribute(attn_prefill_kernel<HD, KT, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    attn_prefill_kernel<HD, KT, true><<<grid, 128, smem, st>>>(p);
+    cudaFuncSetAttribute(attn_prefill_kernel<HD, KT, true, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    attn_prefill_kernel<HD, KT, true, EXT><<<grid, 128, smem, st>>>(p);
   } else {
-    cudaFuncSetAttribute(attn_prefill_kernel<HD, KT, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    attn_prefill_kernel<HD, KT, false><<<grid, 128, smem, st>>>(p);
+    cudaFuncSetAttribute(attn_prefill_kernel<HD, KT, false, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    attn_prefill_kernel<HD, KT, false, EXT><<<grid, 128, smem, st>>>(p);
   }
   return (int)cudaGetLastError();
 }
 
-template <int HD, int KT>
+template <int HD, int KT, bool EXT>
 static int launch_decode(const AttnParams& p, int B, bool int8, cudaStream_t st) {
   size_t kvbytes = (size_t)4 * 2 * KT * HD * 2;
   size_t merge = (size_t)4 * 16 * (HD + 2) * sizeof(float);
@@ -738,18 +784,18 @@ static int launch_decode(const AttnParams& p, int B, bool int8, cudaStream_t st)
   const int qchunks = (p.group + 15) / 16;
   dim3 grid(B, p.hkv * qchunks, p.nsplit);
   if (int8) {
-    cudaFuncSetAttribute(attn_decode_kernel<HD, KT, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    cudaError_t e = launch_pdl(attn_decode_kernel<HD, KT, true>, grid, dim3(128), smem, st, p);
+    cudaFuncSetAttribute(attn_decode_kernel<HD, KT, true, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = launch_pdl(attn_decode_kernel<HD, KT, true, EXT>, grid, dim3(128), smem, st, p);
     if (e != cudaSuccess) return (int)e;
   } else {
-    cudaFuncSetAttribute(attn_decode_kernel<HD, KT, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    cudaError_t e = launch_pdl(attn_decode_kernel<HD, KT, false>, grid, dim3(128), smem, st, p);
+    cudaFuncSetAttribute(attn_decode_kernel<HD, KT, false, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = launch_pdl(attn_decode_kernel<HD, KT, false, EXT>, grid, dim3(128), smem, st, p);
     if (e != cudaSuccess) return (int)e;
   }
   return (int)cudaGetLastError();
 }
 
-template <int HD>
+template <int HD, bool EXT>
 static int launch_decode_tma(const AttnParams& p, int B, cudaStream_t st) {
   CUtensorMap tmK, tmV;
   const uint64_t rows = (uint64_t)p.num_blocks * p.hkv * p.bs;
@@ -757,47 +803,72 @@ static int launch_decode_tma(const AttnParams& p, int B, cudaStream_t st) {
   const size_t smem = (size_t)DecCfg<HD>::STAGES * DecCfg<HD>::STAGE_BYTES + 16 * HD * 2 + 1024;
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(attn_decode_tma_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+    if (cudaFuncSetAttribute(attn_decode_tma_kernel<HD, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
       return -5;
     attr_set = true;
   }
   const int qchunks = (p.group + 15) / 16;
   dim3 grid(B, p.hkv * qchunks, p.nsplit);
-  cudaError_t e = launch_pdl(attn_decode_tma_kernel<HD>, grid, dim3(160), smem, st, tmK, tmV, p);
+  cudaError_t e = launch_pdl(attn_decode_tma_kernel<HD, EXT>, grid, dim3(160), smem, st, tmK, tmV, p);
   if (e != cudaSuccess) return (int)e;
   return (int)cudaGetLastError();
 }
 
-// decode != 0: every sequence has exactly one query row (2 forces the cp.async kernel for bf16 caches too).  nsplit/part_*: split-KV scratch (decode only).
-extern "C" int xft_paged_attention(const void* q, void* out, const void* kc, const void* vc, const float* ks, const float* vs,
-                                   const int* block_table, int bt_stride, const int* cu_q, const int* kv_lens, int B,
-                                   int max_q, int hq, int hkv, int group, int q_off, int HD, int bs, int num_blocks,
-                                   float scale, const float* slopes, const int* prefix_lens, int decode, int nsplit,
-                                   float* part_o, float* part_ml, int* split_counters, int* status, cudaStream_t st) {
+template <bool EXT>
+static int launch_attention(const AttnParams& p, int B, int max_q, int HD, int decode, cudaStream_t st) {
+  const bool int8 = p.ks != nullptr;
+  if (decode) {
+    if (p.nsplit > 1 && (!p.part_o || !p.part_ml || !p.split_counters)) return -3;
+    if (!int8 && decode != 2) {
+      if (HD == 64) return launch_decode_tma<64, EXT>(p, B, st);
+      if (HD == 128) return launch_decode_tma<128, EXT>(p, B, st);
+      if (HD == 256) return launch_decode_tma<256, EXT>(p, B, st);
+      return -1;
+    }
+    // per-warp K+V tiles of 16 KB: a CTA stays at ~64 KB so three CTAs (12 warps) overlap loads and math per SM
+    if (HD == 64) return launch_decode<64, 64, EXT>(p, B, int8, st);
+    if (HD == 128) return launch_decode<128, 32, EXT>(p, B, int8, st);
+    if (HD == 256) return launch_decode<256, 16, EXT>(p, B, int8, st);
+    return -1;
+  }
+  if (HD == 64) return launch_prefill<64, 64, EXT>(p, B, max_q, int8, st);
+  if (HD == 128) return launch_prefill<128, 64, EXT>(p, B, max_q, int8, st);
+  if (HD == 256) return launch_prefill<256, 32, EXT>(p, B, max_q, int8, st);
+  return -1;
+}
+
+// decode != 0: every sequence has exactly one query row (2 forces the cp.async kernel for bf16 caches too).
+// nsplit/part_*: split-KV scratch (decode only).  softcap > 0: scores become softcap * tanh(score / softcap).
+// window > 0: position i sees the keys j <= i with i - j < window or j < keep.  sinks [hq]: exp(sinks[h]) joins the
+// softmax denominator of head h.
+extern "C" int xft_paged_attention_ext(const void* q, void* out, const void* kc, const void* vc, const float* ks,
+                                       const float* vs, const int* block_table, int bt_stride, const int* cu_q,
+                                       const int* kv_lens, int B, int max_q, int hq, int hkv, int group, int q_off, int HD,
+                                       int bs, int num_blocks, float scale, const float* slopes, const int* prefix_lens,
+                                       int decode, int nsplit, float* part_o, float* part_ml, int* split_counters,
+                                       int* status, float softcap, int window, int keep, const float* sinks,
+                                       cudaStream_t st) {
   if (B <= 0) return 0;
   AttnParams p{};
   p.q = (const bf16*)q; p.out = (bf16*)out; p.kc = kc; p.vc = vc; p.ks = ks; p.vs = vs;
   p.block_table = block_table; p.bt_stride = bt_stride; p.cu_q = cu_q; p.kv_lens = kv_lens; p.slopes = slopes;
   p.prefix_lens = prefix_lens; p.hq = hq; p.hkv = hkv; p.group = group; p.q_off = q_off; p.bs = bs; p.scale = scale;
   p.num_blocks = num_blocks; p.nsplit = nsplit < 1 ? 1 : nsplit; p.part_o = part_o; p.part_ml = part_ml; p.split_counters = split_counters; p.status = status;
-  const bool int8 = ks != nullptr;
   if (bs % 64) return -2;
-  if (decode) {
-    if (p.nsplit > 1 && (!part_o || !part_ml || !split_counters)) return -3;
-    if (!int8 && decode != 2) {
-      if (HD == 64) return launch_decode_tma<64>(p, B, st);
-      if (HD == 128) return launch_decode_tma<128>(p, B, st);
-      if (HD == 256) return launch_decode_tma<256>(p, B, st);
-      return -1;
-    }
-    // per-warp K+V tiles of 16 KB: a CTA stays at ~64 KB so three CTAs (12 warps) overlap loads and math per SM
-    if (HD == 64) return launch_decode<64, 64>(p, B, int8, st);
-    if (HD == 128) return launch_decode<128, 32>(p, B, int8, st);
-    if (HD == 256) return launch_decode<256, 16>(p, B, int8, st);
-    return -1;
-  }
-  if (HD == 64) return launch_prefill<64, 64>(p, B, max_q, int8, st);
-  if (HD == 128) return launch_prefill<128, 64>(p, B, max_q, int8, st);
-  if (HD == 256) return launch_prefill<256, 32>(p, B, max_q, int8, st);
-  return -1;
+  if (softcap < 0.f || window < 0 || keep < 0) return -1;
+  if (softcap == 0.f && window == 0 && !sinks) return launch_attention<false>(p, B, max_q, HD, decode, st);
+  if (prefix_lens) return -1;                  // the prefix mask and the window do not combine
+  p.softcap = softcap; p.inv_cap2 = softcap > 0.f ? 2.f / softcap : 0.f;
+  p.window = window > 0 ? min(window, 1 << 30) : 1 << 30; p.keep = window > 0 ? keep : 0; p.sinks = sinks;
+  return launch_attention<true>(p, B, max_q, HD, decode, st);
+}
+
+extern "C" int xft_paged_attention(const void* q, void* out, const void* kc, const void* vc, const float* ks, const float* vs,
+                                   const int* block_table, int bt_stride, const int* cu_q, const int* kv_lens, int B,
+                                   int max_q, int hq, int hkv, int group, int q_off, int HD, int bs, int num_blocks,
+                                   float scale, const float* slopes, const int* prefix_lens, int decode, int nsplit,
+                                   float* part_o, float* part_ml, int* split_counters, int* status, cudaStream_t st) {
+  return xft_paged_attention_ext(q, out, kc, vc, ks, vs, block_table, bt_stride, cu_q, kv_lens, B, max_q, hq, hkv, group,
+                                 q_off, HD, bs, num_blocks, scale, slopes, prefix_lens, decode, nsplit, part_o, part_ml,
+                                 split_counters, status, 0.f, 0, 0, nullptr, st);
 }

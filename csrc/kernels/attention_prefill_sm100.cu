@@ -20,6 +20,10 @@
 // softmax of tile j overlaps the QK^T of tile j + 1, and CTAs with the most keys to visit (the last query rows of a
 // causal prompt) are scheduled first.
 //
+// The EXT instantiation adds, each with its constants as launch parameters: a sliding window with kept first keys (only
+// the key tiles that hold a visible key are visited: first those of the kept keys, then those of the window), a tanh cap
+// on the scores, and one sink per query head (a term of the softmax denominator without key or value).
+//
 // Warp roles (192 threads): warp 0 = TMA producer, warp 1 = TMEM owner + MMA issuer, warps 2-5 = softmax / output.
 // Every wait is bounded and reports through the status word.
 #include "ptx.cuh"
@@ -36,6 +40,10 @@ struct PrefillAttnParams {
   int hq, hkv, group, q_off;  // kv head of query head h = (h + q_off) / group
   int bs;                     // tokens per cache block (64)
   float scale_log2;           // softmax scale * log2(e)
+  // EXT only
+  float cap_log2, inv_cap2;   // softcap * log2(e), 2 log2(e) * scale / softcap (cap_log2 0: no cap)
+  int window, keep;           // keys within `window` positions and the first `keep` are visible (window 2^30: all)
+  const float* sinks;         // [hq] or null
   int num_blocks;
   int* status;
 };
@@ -69,6 +77,12 @@ constexpr int kPfHalf = kPfTile * 128;       // bytes of one 64-feature half of 
 constexpr int kPfTileBytes = 2 * kPfHalf;    // 32 KB: Q, P, and each K / V stage
 constexpr int kPfSmem = kPfTileBytes * 6 + 1024;   // Q, P, K x 2, V x 2
 
+// Capped score in log2 units: cap * tanh(raw * scale / cap) with tanh(x) = 1 - 2 / (1 + exp(2x)).
+__device__ __forceinline__ float capped_log2(const PrefillAttnParams& p, float raw) {
+  return p.cap_log2 - __fdividef(2.f * p.cap_log2, 1.f + exp2f(fminf(raw * p.inv_cap2, 120.f)));
+}
+
+template <bool EXT>
 __global__ void __launch_bounds__(192, 1) attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ,
                                                                  const __grid_constant__ CUtensorMap tmK,
                                                                  const __grid_constant__ CUtensorMap tmV,
@@ -91,7 +105,15 @@ __global__ void __launch_bounds__(192, 1) attn_prefill_tc_kernel(const __grid_co
   const int row0 = (n_qt - 1 - (int)blockIdx.x) * kPfQ;
   const int past = kv_len - q_len;            // keys before this call's first query
   const int last_row = min(row0 + kPfQ, q_len) - 1;
-  const int n_tiles = (min(kv_len, past + last_row + 1) + kPfTile - 1) / kPfTile;
+  const int end_tile = (min(kv_len, past + last_row + 1) + kPfTile - 1) / kPfTile;
+  // the tiles to visit: [0, keep_tiles) and [lo_tile, end_tile)
+  int lo_tile = 0, keep_tiles = 0;
+  if (EXT) {
+    lo_tile = min(max(0, past + row0 - p.window + 1) / kPfTile, end_tile);
+    keep_tiles = min((p.keep + kPfTile - 1) / kPfTile, lo_tile);
+  }
+  const int n_tiles = keep_tiles + end_tile - lo_tile;
+  auto tile_of = [&](int j) { return EXT ? (j < keep_tiles ? j : j - keep_tiles + lo_tile) : j; };
   const int kvh = (h + p.q_off) / p.group;
 
   if (threadIdx.x == 0) {
@@ -137,7 +159,7 @@ __global__ void __launch_bounds__(192, 1) attn_prefill_tc_kernel(const __grid_co
         int rowk[2];
         bool bad = false;
         for (int i = 0; i < 2; ++i) {
-          int blk = bt[min(2 * j + i, n_blocks - 1)];
+          int blk = bt[min(2 * tile_of(j) + i, n_blocks - 1)];
           if (blk < 0 || blk >= p.num_blocks) { bad = true; blk = 0; }
           rowk[i] = (blk * p.hkv + kvh) * p.bs;
         }
@@ -210,16 +232,20 @@ __global__ void __launch_bounds__(192, 1) attn_prefill_tc_kernel(const __grid_co
 #pragma unroll
     for (int i = 0; i < 128; ++i) o[i] = 0.f;
     float m = -INFINITY, l = 0.f;
+    if (EXT && p.sinks) { m = p.sinks[h] * 1.4426950408889634f; l = 1.f; }
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
       const int s = j & 1;
       if (!mbar_wait(&s_full[s], (j >> 1) & 1, p.status, XFT_ERR_WAIT_TMEM)) { ok = false; break; }
       tcgen05_fence_after();
       const uint32_t sa = lane_addr + (uint32_t)(s * 128);
-      const int k0 = j * kPfTile;
+      const int k0 = tile_of(j) * kPfTile;
       const int nvalid = min(qpos, kv_len - 1) - k0 + 1;    // keys [k0, k0 + nvalid) are visible to this row
+      // EXT: of these, the ones from k0 + first on and the ones below k0 + kept
+      const int first = EXT ? qpos - p.window + 1 - k0 : 0, kept = EXT ? p.keep - k0 : 0;
+      auto visible = [&](int i) { return i < nvalid && (!EXT || i >= first || i < kept); };
       // pass 1: row maximum of the visible scores
-      float mx = m;
+      float mx = EXT ? -INFINITY : m;
 #pragma unroll 1
       for (int c = 0; c < 128; c += 32) {
         uint32_t v[32];
@@ -227,9 +253,12 @@ __global__ void __launch_bounds__(192, 1) attn_prefill_tc_kernel(const __grid_co
         tmem_ld_wait();
 #pragma unroll
         for (int i = 0; i < 32; ++i)
-          if (c + i < nvalid) mx = fmaxf(mx, __uint_as_float(v[i]) * p.scale_log2);
+          if (visible(c + i)) mx = fmaxf(mx, EXT ? __uint_as_float(v[i]) : __uint_as_float(v[i]) * p.scale_log2);
       }
-      const float alpha = exp2f(m - mx);                    // m = -inf on the first tile: alpha = 0, o and l are 0
+      // EXT: the maximum was taken over the raw scores (the cap is increasing); m = -inf: nothing visible so far
+      if (EXT) mx = fmaxf(m, mx == -INFINITY ? -INFINITY : p.cap_log2 > 0.f ? capped_log2(p, mx) : mx * p.scale_log2);
+      // m = -inf on the first tile: alpha = 0, o and l are 0
+      const float alpha = (EXT && mx == -INFINITY) ? 1.f : exp2f(m - mx);
       m = mx;
       // pass 2: P = exp2(s - m) as bf16 into the swizzled K-major tile, row sum
       float sum = 0.f;
@@ -245,8 +274,11 @@ __global__ void __launch_bounds__(192, 1) attn_prefill_tc_kernel(const __grid_co
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
             const int e = g8 * 8 + 2 * i;
-            const float p0 = (c + e < nvalid) ? exp2f(__uint_as_float(v[e]) * p.scale_log2 - m) : 0.f;
-            const float p1 = (c + e + 1 < nvalid) ? exp2f(__uint_as_float(v[e + 1]) * p.scale_log2 - m) : 0.f;
+            float s0 = __uint_as_float(v[e]), s1 = __uint_as_float(v[e + 1]);
+            if (EXT && p.cap_log2 > 0.f) { s0 = capped_log2(p, s0); s1 = capped_log2(p, s1); }
+            else { s0 *= p.scale_log2; s1 *= p.scale_log2; }
+            const float p0 = visible(c + e) ? exp2f(s0 - m) : 0.f;
+            const float p1 = visible(c + e + 1) ? exp2f(s1 - m) : 0.f;
             const __nv_bfloat162 pb = __floats2bfloat162_rn(p0, p1);
             // the sum uses the rounded values, as the product does
             sum += __low2float(pb) + __high2float(pb);
@@ -304,17 +336,23 @@ using namespace xft;
 
 // Causal prefill attention over the paged bf16 cache, head_dim 128 (see the file comment).  q, out: [T, hq, 128];
 // caches [num_blocks, hkv, bs, 128] with bs = 64; cu_q [B + 1], kv_lens [B] (keys visible after this call's append).
+// softcap > 0: scores become softcap * tanh(score / softcap).  window > 0: position i sees the keys j <= i with
+// i - j < window or j < keep.  sinks [hq]: exp(sinks[h]) joins the softmax denominator of head h.
 // Returns 0, -1 for an unsupported shape, or a CUDA / tensor-map error.
 extern "C" int xft_attn_prefill_tc(const void* q, void* out, const void* kc, const void* vc, const int* block_table,
                                    int bt_stride, const int* cu_q, const int* kv_lens, int B, int T, int max_q, int hq,
-                                   int hkv, int group, int q_off, int bs, int num_blocks, float scale, int* status,
-                                   cudaStream_t st) {
+                                   int hkv, int group, int q_off, int bs, int num_blocks, float scale, float softcap,
+                                   int window, int keep, const float* sinks, int* status, cudaStream_t st) {
   if (B <= 0 || T <= 0 || max_q <= 0) return 0;
-  if (bs != 64 || hq <= 0 || hkv <= 0) return -1;
+  if (bs != 64 || hq <= 0 || hkv <= 0 || softcap < 0.f || window < 0 || keep < 0) return -1;
   PrefillAttnParams p{};
   p.out = (__nv_bfloat16*)out; p.block_table = block_table; p.bt_stride = bt_stride; p.cu_q = cu_q; p.kv_lens = kv_lens;
   p.hq = hq; p.hkv = hkv; p.group = group; p.q_off = q_off; p.bs = bs; p.scale_log2 = scale * 1.4426950408889634f;
   p.num_blocks = num_blocks; p.status = status;
+  const bool ext = softcap > 0.f || window > 0 || sinks;
+  p.window = window > 0 ? min(window, 1 << 30) : 1 << 30; p.keep = window > 0 ? keep : 0; p.sinks = sinks;
+  p.cap_log2 = softcap * 1.4426950408889634f;
+  p.inv_cap2 = softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f;
   CUtensorMap tmQ, tmK, tmV;
   const uint64_t rows = (uint64_t)num_blocks * hkv * bs;
   int r = make_tensor_map(&tmQ, q, (uint64_t)T, (uint64_t)hq * 128, (uint64_t)hq * 128, 128, 2);
@@ -322,11 +360,13 @@ extern "C" int xft_attn_prefill_tc(const void* q, void* out, const void* kc, con
   if (make_tensor_map(&tmK, kc, rows, 128, 128, 64, 2) || make_tensor_map(&tmV, vc, rows, 128, 128, 64, 2)) return -4;
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(attn_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kPfSmem) != cudaSuccess)
+    if (cudaFuncSetAttribute(attn_prefill_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPfSmem) != cudaSuccess ||
+        cudaFuncSetAttribute(attn_prefill_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPfSmem) != cudaSuccess)
       return 3000 + (int)cudaGetLastError();
     attr_set = true;
   }
   dim3 grid((max_q + kPfQ - 1) / kPfQ, hq, B);
-  cudaError_t e = launch_pdl(attn_prefill_tc_kernel, grid, dim3(192), (size_t)kPfSmem, st, tmQ, tmK, tmV, p);
+  cudaError_t e = launch_pdl(ext ? attn_prefill_tc_kernel<true> : attn_prefill_tc_kernel<false>, grid, dim3(192),
+                             (size_t)kPfSmem, st, tmQ, tmK, tmV, p);
   return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }

@@ -1,0 +1,262 @@
+// Plain kernels for any size: the 32-bit path of the layered decoder (fp32 weights, activations and cache), and what a
+// bf16 model needs when its heads are larger than the tensor-core kernels take.
+//
+//   xft_gemm_f32        Y[T, N] = X[T, K] W[N, K]^T in fp32 (no reduced-precision mode)
+//   xft_gated_act_f32   act(gate) * up
+//   xft_rope_cache      split q | k | v rows, rotate q and k, append k and v to the paged cache; key and value heads may
+//                       have different sizes
+//   xft_attention_plain one warp per (query, head): sliding window with kept first keys, capped scores, sinks
+//
+// This file is compiled without fast-math: tanhf, expf and the divisions are the accurate ones.
+#include "ptx.cuh"
+
+namespace xft {
+
+typedef __nv_bfloat16 bf16;
+
+template <typename T> __device__ __forceinline__ float to_f32(T v);
+template <> __device__ __forceinline__ float to_f32<float>(float v) { return v; }
+template <> __device__ __forceinline__ float to_f32<bf16>(bf16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T from_f32(float v);
+template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
+template <> __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16(v); }
+
+// ------------------------------------------------------------------------------------------ GEMM
+// 64 x 64 tile of Y per CTA, 256 threads with 4 x 4 values each, 16 columns of the reduction per step.
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ X, int ldx, const float* __restrict__ W, int ldw,
+                                                       float* __restrict__ Y, int ldo, int T, int N, int K) {
+  __shared__ float xs[16][68], ws[16][68];
+  const int t0 = blockIdx.y * 64, n0 = blockIdx.x * 64, tid = threadIdx.x;
+  const int lr = tid >> 2, lk = (tid & 3) * 4;             // this thread loads row lr, columns lk .. lk + 3
+  const int tx = tid & 15, ty = tid >> 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += 16) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int k = k0 + lk + j;
+      xs[lk + j][lr] = (t0 + lr < T && k < K) ? X[(size_t)(t0 + lr) * ldx + k] : 0.f;
+      ws[lk + j][lr] = (n0 + lr < N && k < K) ? W[(size_t)(n0 + lr) * ldw + k] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 16; ++k) {
+      float a[4], b[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) { a[j] = xs[k][ty * 4 + j]; b[j] = ws[k][tx * 4 + j]; }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int t = t0 + ty * 4 + i, n = n0 + tx * 4 + j;
+      if (t < T && n < N) Y[(size_t)t * ldo + n] = acc[i][j];
+    }
+}
+
+__global__ void gated_act_f32_kernel(const float* __restrict__ gu, int ld, float* __restrict__ out, int T, int I, int act) {
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= (size_t)T * I) return;
+  const int t = (int)(i / I), c = (int)(i % I);
+  const float g = gu[(size_t)t * ld + c], u = gu[(size_t)t * ld + I + c];
+  float a = g;
+  if (act == 1) a = fmaxf(g, 0.f);
+  else if (act == 2) a = g / (1.f + expf(-g));
+  else if (act == 3) a = 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+  out[i] = a * u;
+}
+
+// ------------------------------------------------------------------------------------------ rotary + cache append
+// One warp per (token, head); rows are hq query heads of kd, hkv key heads of kd, hkv value heads of vd.
+template <typename T>
+__global__ void __launch_bounds__(128) rope_cache_kernel(const T* __restrict__ qkv, int ldq, int n_tok, int hq, int hkv, int kd,
+                                                         int vd, const int* __restrict__ positions,
+                                                         const float* __restrict__ table, int rot, int style, int max_pos,
+                                                         T* __restrict__ q_out, T* __restrict__ kc, T* __restrict__ vc, int bs,
+                                                         long long nslots, const int* __restrict__ slots, int* status) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int nheads = hq + 2 * hkv;
+  const long long gw = (long long)blockIdx.x * 4 + warp;
+  if (gw >= (long long)n_tok * nheads) return;
+  const int t = (int)(gw / nheads), h = (int)(gw % nheads);
+  const bool is_v = h >= hq + hkv;
+  const T* src = qkv + (size_t)t * ldq + (is_v ? (hq + hkv) * kd + (h - hq - hkv) * vd : h * kd);
+  const int D = is_v ? vd : kd;
+  T* dst;
+  if (h < hq) {
+    dst = q_out + ((size_t)t * hq + h) * kd;
+  } else {
+    const long long slot = slots[t];
+    if (slot < 0 || slot >= nslots) { if (lane == 0 && status) atomicCAS(status, 0, XFT_ERR_BOUNDS); return; }
+    const int kh = is_v ? h - hq - hkv : h - hq;
+    dst = (is_v ? vc : kc) + ((size_t)((slot / bs) * hkv + kh) * bs + slot % bs) * D;
+  }
+  int pos = positions[t];
+  if (table && (pos < 0 || pos >= max_pos)) { if (lane == 0 && status) atomicCAS(status, 0, XFT_ERR_BOUNDS); pos = 0; }
+  const int half = rot >> 1;
+  for (int d = lane; d < D; d += 32) {
+    float x = to_f32<T>(src[d]);
+    if (!is_v && table && d < rot) {
+      const float* cs = table + (size_t)pos * rot;
+      const int i = style == 0 ? (d < half ? d : d - half) : d >> 1;
+      const bool second = style == 0 ? d >= half : (d & 1) != 0;
+      const int partner = style == 0 ? (second ? d - half : d + half) : d ^ 1;
+      const float y = to_f32<T>(src[partner]);
+      x = x * cs[i] + (second ? y : -y) * cs[half + i];
+    }
+    dst[d] = from_f32<T>(x);
+  }
+}
+
+// ------------------------------------------------------------------------------------------ attention
+// One warp per (query token, head).  A lane owns one of 32 keys while scores are computed and every 32nd output feature
+// while values are added up.
+template <typename T>
+__global__ void __launch_bounds__(128) attention_plain_kernel(const T* __restrict__ q, T* __restrict__ out,
+                                                              const T* __restrict__ kc, const T* __restrict__ vc,
+                                                              const int* __restrict__ block_table, int bt_stride,
+                                                              const int* __restrict__ cu_q, const int* __restrict__ kv_lens,
+                                                              int B, int n_tok, int hq, int hkv, int group, int q_off, int kd,
+                                                              int vd, int bs, int num_blocks, float scale, float softcap,
+                                                              int window, int keep, const float* __restrict__ sinks,
+                                                              int* status) {
+  extern __shared__ float sm[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* qs = sm + warp * (kd + vd + 64);
+  float* acc = qs + kd;
+  float* ps = acc + vd;                                   // 32 weights
+  int* rs = reinterpret_cast<int*>(ps + 32);              // 32 cache rows
+  const long long gw = (long long)blockIdx.x * 4 + warp;
+  if (gw >= (long long)n_tok * hq) return;
+  const int t = (int)(gw / hq), h = (int)(gw % hq);
+  int lo_b = 0, hi_b = B - 1;                             // the sequence that owns token t
+  while (lo_b < hi_b) {
+    const int mid = (lo_b + hi_b + 1) >> 1;
+    if (cu_q[mid] <= t) lo_b = mid; else hi_b = mid - 1;
+  }
+  const int b = lo_b, kv_len = kv_lens[b];
+  const int qpos = kv_len - (cu_q[b + 1] - cu_q[b]) + (t - cu_q[b]);
+  const int kvh = min((h + q_off) / group, hkv - 1);
+  for (int d = lane; d < kd; d += 32) qs[d] = to_f32<T>(q[((size_t)t * hq + h) * kd + d]);
+  for (int d = lane; d < vd; d += 32) acc[d] = 0.f;
+  __syncwarp();
+  // visible keys: [0, nk) and [lo, qpos]
+  const int lo = max(0, qpos - window + 1);
+  const int nk = min(keep, lo);
+  const int total = nk + qpos + 1 - lo;
+  const int* bt = block_table + (size_t)b * bt_stride;
+  float m = -INFINITY, l = 0.f;
+  if (sinks) { m = sinks[h]; l = 1.f; }
+  for (int n0 = 0; n0 < total; n0 += 32) {
+    const int n = n0 + lane;
+    float s = -INFINITY;
+    int row = 0;
+    if (n < total) {
+      const int key = n < nk ? n : n - nk + lo;
+      int blk = bt[key / bs];
+      if (blk < 0 || blk >= num_blocks) { if (status) atomicCAS(status, 0, XFT_ERR_BOUNDS); blk = 0; }
+      row = (blk * hkv + kvh) * bs + key % bs;
+      const T* kp = kc + (size_t)row * kd;
+      float dot = 0.f;
+      for (int d = 0; d < kd; ++d) dot = fmaf(qs[d], to_f32<T>(kp[d]), dot);
+      s = dot * scale;
+      if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+    }
+    float mx = s;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    const float mn = fmaxf(m, mx);
+    const float c = m == -INFINITY ? 0.f : expf(m - mn);
+    const float pr = n < total ? expf(s - mn) : 0.f;
+    float sum = pr;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    m = mn;
+    l = l * c + sum;
+    ps[lane] = pr;
+    rs[lane] = row;
+    __syncwarp();
+    const int cnt = min(32, total - n0);
+    for (int d = lane; d < vd; d += 32) {
+      float a = acc[d] * c;
+      for (int i = 0; i < cnt; ++i) a = fmaf(ps[i], to_f32<T>(vc[(size_t)rs[i] * vd + d]), a);
+      acc[d] = a;
+    }
+    __syncwarp();
+  }
+  for (int d = lane; d < vd; d += 32) out[((size_t)t * hq + h) * vd + d] = from_f32<T>(l > 0.f ? acc[d] / l : 0.f);
+}
+
+}  // namespace xft
+
+using namespace xft;
+
+extern "C" int xft_gemm_f32(const float* X, int ldx, const float* W, int ldw, float* Y, int ldo, int T, int N, int K,
+                            cudaStream_t st) {
+  if (T <= 0 || N <= 0) return 0;
+  if (K <= 0 || ldx < K || ldw < K || ldo < N) return -1;
+  const int ty = (T + 63) / 64;
+  if (ty > 65535) return -2;
+  gemm_f32_kernel<<<dim3((N + 63) / 64, ty), 256, 0, st>>>(X, ldx, W, ldw, Y, ldo, T, N, K);
+  return (int)cudaGetLastError();
+}
+
+extern "C" int xft_gated_act_f32(const float* gu, int ld, float* out, int T, int I, int act, cudaStream_t st) {
+  const size_t n = (size_t)T * I;
+  if (!n) return 0;
+  if (ld < 2 * I) return -1;
+  gated_act_f32_kernel<<<(unsigned)((n + 255) / 256), 256, 0, st>>>(gu, ld, out, T, I, act);
+  return (int)cudaGetLastError();
+}
+
+// f32: 1 = fp32 rows and cache, 0 = bf16.  hkv = 0: query heads only (a layer that reads another layer's cache).
+extern "C" int xft_rope_cache(const void* qkv, int ldq, int T, int hq, int hkv, int kd, int vd, const int* positions,
+                              const float* table, int rot, int style, int max_pos, void* q_out, void* kc, void* vc, int bs,
+                              long long nslots, const int* slots, int f32, int* status, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (hq <= 0 || hkv < 0 || kd <= 0 || vd <= 0 || bs <= 0 || rot < 0 || rot > kd || (rot & 1) ||
+      ldq < (hq + hkv) * kd + hkv * vd || (rot > 0 && !table)) return -1;
+  if (rot == 0) table = nullptr;
+  const long long warps = (long long)T * (hq + 2 * hkv);
+  const unsigned grid = (unsigned)((warps + 3) / 4);
+  if (f32)
+    rope_cache_kernel<float><<<grid, 128, 0, st>>>((const float*)qkv, ldq, T, hq, hkv, kd, vd, positions, table, rot, style,
+                                                   max_pos, (float*)q_out, (float*)kc, (float*)vc, bs, nslots, slots, status);
+  else
+    rope_cache_kernel<bf16><<<grid, 128, 0, st>>>((const bf16*)qkv, ldq, T, hq, hkv, kd, vd, positions, table, rot, style,
+                                                  max_pos, (bf16*)q_out, (bf16*)kc, (bf16*)vc, bs, nslots, slots, status);
+  return (int)cudaGetLastError();
+}
+
+// q [T, hq, kd], caches [num_blocks, hkv, bs, kd] and [num_blocks, hkv, bs, vd], out [T, hq, vd], all fp32 (f32 = 1) or
+// bf16.  window 0: every earlier key; softcap 0: none; sinks null: none.
+extern "C" int xft_attention_plain(const void* q, void* out, const void* kc, const void* vc, const int* block_table,
+                                   int bt_stride, const int* cu_q, const int* kv_lens, int B, int T, int hq, int hkv, int group,
+                                   int q_off, int kd, int vd, int bs, int num_blocks, float scale, float softcap, int window,
+                                   int keep, const float* sinks, int f32, int* status, cudaStream_t st) {
+  if (B <= 0 || T <= 0) return 0;
+  if (hq <= 0 || hkv <= 0 || group <= 0 || kd <= 0 || vd <= 0 || bs <= 0 || softcap < 0.f || window < 0 || keep < 0) return -1;
+  if ((long long)num_blocks * hkv * bs >= (1ll << 31)) return -2;
+  const size_t smem = (size_t)4 * (kd + vd + 64) * sizeof(float);
+  if (smem > 200 * 1024) return -3;
+  const int win = window > 0 ? (window < (1 << 30) ? window : 1 << 30) : 1 << 30;
+  const int kp = window > 0 ? keep : 0;
+  const unsigned grid = (unsigned)(((long long)T * hq + 3) / 4);
+  if (f32) {
+    if (smem > 48 * 1024) cudaFuncSetAttribute(attention_plain_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    attention_plain_kernel<float><<<grid, 128, smem, st>>>((const float*)q, (float*)out, (const float*)kc, (const float*)vc,
+                                                           block_table, bt_stride, cu_q, kv_lens, B, T, hq, hkv, group, q_off,
+                                                           kd, vd, bs, num_blocks, scale, softcap, win, kp, sinks, status);
+  } else {
+    if (smem > 48 * 1024) cudaFuncSetAttribute(attention_plain_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    attention_plain_kernel<bf16><<<grid, 128, smem, st>>>((const bf16*)q, (bf16*)out, (const bf16*)kc, (const bf16*)vc,
+                                                          block_table, bt_stride, cu_q, kv_lens, B, T, hq, hkv, group, q_off,
+                                                          kd, vd, bs, num_blocks, scale, softcap, win, kp, sinks, status);
+  }
+  return (int)cudaGetLastError();
+}

@@ -18,16 +18,17 @@ from .runtime.engine import Model
 
 
 class AutoModel:
-    def __init__(self, path, dtype: str = "fp16", kv_cache_dtype: str = "fp16"):
+    def __init__(self, path, dtype: str = "fp16", kv_cache_dtype: str = "fp16", max_cache_tokens: int = 0):
         if dtype not in WEIGHT_DTYPES:
             raise Exception(f"{self.__class__.__name__} don't support {dtype}.")
         if kv_cache_dtype not in KV_DTYPES:
             raise Exception(f"{self.__class__.__name__} don't support KV cache data type: {kv_cache_dtype}.")
-        self.model = Model(path, dtype, kv_cache_dtype)
+        self.model = Model(path, dtype, kv_cache_dtype, max_cache_tokens=max_cache_tokens)
 
     @classmethod
-    def from_pretrained(cls, path, dtype: str = "fp16", kv_cache_dtype: str = "fp16"):
-        return cls(path, dtype, kv_cache_dtype)
+    def from_pretrained(cls, path, dtype: str = "fp16", kv_cache_dtype: str = "fp16", max_cache_tokens: int = 0):
+        """``max_cache_tokens`` > 0 (extension): the KV pools are made for that many tokens and never grow."""
+        return cls(path, dtype, kv_cache_dtype, max_cache_tokens)
 
     def __call__(self, inputs, **kwargs):
         """All-position logits [bs, seq, vocab] (torch binding ``forward``, auto_model.h:160-190)."""
@@ -41,17 +42,18 @@ class AutoModel:
     def set_input_cb(self, input_ids: Optional[Union[List[int], List[List[int]], torch.Tensor]] = None,
                      seq_ids: Optional[Union[List[int], torch.Tensor]] = None,
                      max_length: Optional[Union[int, List[int], torch.Tensor]] = None, greedy: bool = False,
-                     append: bool = False, hold: bool = False, extend: bool = False):
+                     append: bool = False, hold: bool = False, extend: bool = False, rows=None, on_demand: bool = False):
         """``append`` / ``hold`` build one forward out of new prompts and running sequences, ``extend`` feeds further
         pieces of the prompts of known sequences (chunked prefill; ``input_ids`` = one list per sequence id); see
-        ``runtime.engine.Model.set_input_cb``.  All three are extensions of the reference's call."""
+        ``runtime.engine.Model.set_input_cb``, also for ``rows`` (whose logits are returned) and ``on_demand``.  All are
+        extensions of the reference's call."""
         seq_lens = None
         if extend:
             if seq_ids is None or not isinstance(input_ids, list) or not input_ids or not isinstance(input_ids[0], list):
                 raise ValueError("extend=True takes seq_ids and one list of tokens per sequence")
             seq_lens = [len(r) for r in input_ids]
             input_ids = [t for r in input_ids for t in r]
-            return self.model.set_input_cb(input_ids, seq_lens, seq_ids, max_length, greedy, append, hold, True)
+            return self.model.set_input_cb(input_ids, seq_lens, seq_ids, max_length, greedy, append, hold, True, rows)
         if isinstance(input_ids, list):
             if seq_ids is None:
                 if input_ids and isinstance(input_ids[0], list):
@@ -61,7 +63,8 @@ class AutoModel:
                     raise ValueError("For prompts, input_ids should not be List[int].")
             elif input_ids and isinstance(input_ids[0], list):
                 input_ids = [t for r in input_ids for t in r]
-        return self.model.set_input_cb(input_ids, seq_lens, seq_ids, max_length, greedy, append, hold)
+        return self.model.set_input_cb(input_ids, seq_lens, seq_ids, max_length, greedy, append, hold, False, rows,
+                                       on_demand)
 
     def follow(self):
         """Follower ranks: run rank 0's calls (generate, continuous batching, all-position logits) until shutdown."""

@@ -1,4 +1,4 @@
-"""Model configuration: ``config.ini`` parsing and dtype-string handling.
+"""Model configuration: ``config.ini`` / ``config.json`` parsing and dtype-string handling.
 
 The checkpoint directory contract is the reference's: one ``config.ini`` whose single
 section name selects the model family, plus raw ``.bin`` tensors.  The keys and their
@@ -8,20 +8,25 @@ vocabulary follows ``include/dtype.h:18-36`` and
 
 Unlike the reference, where every (family, weight type, kv type) triple is a C++ template
 instantiation, here all of this is *data*: one `ModelConfig` drives one generic decoder.
+
+Designs that describe themselves layer by layer come as ``config.json`` (plus ``model.safetensors``) instead: its
+``layers`` list becomes `ModelConfig.layers`, one `LayerConfig` per layer, and every size and constant is per layer.
 """
 from __future__ import annotations
 
 import configparser
+import json
 import math
 import os
 from dataclasses import dataclass, field
-from typing import Dict, Optional, Tuple
+from typing import Dict, List, Optional, Tuple
 
 # dtype strings accepted by AutoModel (reference automodel.py:20-37)
 WEIGHT_DTYPES = (
     "fp16", "bf16", "int8", "w8a8", "int4", "nf4",
     "bf16_fp16", "bf16_int8", "bf16_w8a8", "bf16_int4", "bf16_nf4",
     "w8a8_int8", "w8a8_int4", "w8a8_nf4", "fp8_e4m3",
+    "fp32",                           # everything in 32 bits: layered designs on a GPU, any family on CPU
 )
 KV_DTYPES = ("fp16", "bf16", "int8")
 
@@ -31,6 +36,9 @@ MODEL_TYPES = (
     "deepseek_moe", "baichuan", "chatglm", "chatglm2", "chatglm3", "chatglm4", "gpt",
     "telechat",
 )
+
+# config.json "architecture" -> model type
+ARCHITECTURES = {"Kafipel": "kafipel"}
 
 
 def split_hybrid_dtype(dtype: str) -> Tuple[str, str]:
@@ -68,6 +76,42 @@ class RopeConfig:
     beta_slow: float = 1.0
     mscale: float = 1.0
     mscale_all_dim: float = 1.0
+
+
+@dataclass(frozen=True)
+class RotaryConfig:
+    """Rotary positions of one layer: the first `dims` dimensions of each head, base, optional YaRN scaling."""
+    dims: int
+    base: float
+    factor: float = 0.0               # 0: no scaling
+    original: float = 0.0
+    fast: float = 32.0
+    slow: float = 1.0
+
+
+@dataclass(frozen=True)
+class MixerConfig:
+    """Token mixer of one layer.  `window` 0: every earlier position is visible; otherwise position i sees j <= i when
+    i - j < window or j < keep_first.  `softcap` 0: scores are not capped.  `kv_from` >= 0: this layer has queries only
+    and reads the keys and values of that layer."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    kind: str = "attention"
+    softcap: float = 0.0
+    window: int = 0
+    keep_first: int = 0
+    rot: Optional[RotaryConfig] = None
+    kv_from: int = -1
+
+
+@dataclass(frozen=True)
+class LayerConfig:
+    mixer: MixerConfig
+    ff: int = 0                       # 0: no feed-forward
+    ff_kind: str = "dense"
 
 
 @dataclass
@@ -116,6 +160,8 @@ class ModelConfig:
     v_head_dim: int = 0
     # Qwen3
     do_qk_norm: bool = False
+    # layered designs (config.json): one entry per layer; the scalar sizes above then hold the first layer's
+    layers: List[LayerConfig] = field(default_factory=list)
     # raw key/value pairs (for family-specific look-ups, like DecoderContext::GetAttr)
     raw: Dict[str, str] = field(default_factory=dict)
 
@@ -149,6 +195,36 @@ class ModelConfig:
         return self.raw.get(key, default)
 
     # ---- io ---------------------------------------------------------------------------
+    @classmethod
+    def load(cls, path: str) -> "ModelConfig":
+        """The configuration of a model directory: ``config.json`` of a layered design, else ``config.ini``."""
+        js = os.path.join(path, "config.json")
+        if os.path.isfile(js) and not os.path.exists(os.path.join(path, "config.ini")):
+            return cls.from_json(path)
+        return cls.from_ini(path)
+
+    @classmethod
+    def from_json(cls, path: str) -> "ModelConfig":
+        with open(path if path.endswith(".json") else os.path.join(path, "config.json")) as f:
+            d = json.load(f)
+        arch = d.get("architecture")
+        if arch not in ARCHITECTURES:
+            raise ValueError(f"unsupported architecture {arch!r} in {path}; known: {sorted(ARCHITECTURES)}")
+        layers = [_layer_config(i, e) for i, e in enumerate(d["layers"])]
+        for i, l in enumerate(layers):
+            j = l.mixer.kv_from
+            if j >= 0:
+                src = layers[j].mixer if j < i else None
+                if src is None or src.kv_from >= 0:
+                    raise ValueError(f"layer {i}: kv_from {j} is not an earlier layer with keys and values of its own")
+                if (src.kv_heads, src.dim, src.vdim) != (l.mixer.kv_heads, l.mixer.dim, l.mixer.vdim):
+                    raise ValueError(f"layer {i}: heads differ from those of layer {j}, whose keys it reads")
+        m = layers[0].mixer
+        return cls(model_type=ARCHITECTURES[arch], head_num=m.heads, kv_head_num=m.kv_heads, size_per_head=m.dim,
+                   v_head_dim=m.vdim, hidden_size=int(d["width"]), inter_size=layers[0].ff, num_layer=len(layers),
+                   vocab_size=int(d["vocab"]), layernorm_eps=float(d["norm"]["eps"]), start_id=-1, end_id=-1,
+                   weight_data_type="bf16", layers=layers, raw=d)
+
     @classmethod
     def from_ini(cls, path: str) -> "ModelConfig":
         ini = path if path.endswith(".ini") else os.path.join(path, "config.ini")
@@ -247,7 +323,12 @@ class ModelConfig:
         return c
 
     def to_ini(self, path: str, extra: Optional[Dict[str, str]] = None) -> None:
-        """Write a config.ini the way the converters do (one section = model type)."""
+        """Write a config.ini the way the converters do (one section = model type); config.json for a layered design."""
+        if self.layers:
+            os.makedirs(path, exist_ok=True)
+            with open(os.path.join(path, "config.json"), "w") as f:
+                json.dump(self.raw, f, indent=1)
+            return
         cp = configparser.ConfigParser()
         d: Dict[str, str] = dict(self.raw)
         d.update({
@@ -309,3 +390,30 @@ class ModelConfig:
         os.makedirs(path, exist_ok=True)
         with open(os.path.join(path, "config.ini"), "w") as f:
             cp.write(f)
+
+
+def _layer_config(i: int, e: dict) -> LayerConfig:
+    """One entry of config.json's ``layers``."""
+    if e.get("type") != "attention":
+        raise ValueError(f"layer {i}: unsupported mixer type {e.get('type')!r}")
+    m = e["mixer"]
+    rot = None
+    if m.get("rot"):
+        r, sc = m["rot"], m["rot"].get("scaling") or {}
+        rot = RotaryConfig(int(r["dims"]), float(r["base"]), float(sc.get("factor", 0.0)), float(sc.get("original", 0.0)),
+                           float(sc.get("fast", 32.0)), float(sc.get("slow", 1.0)))
+        if rot.dims % 2 or rot.dims > int(m["dim"]):
+            raise ValueError(f"layer {i}: rotary dims {rot.dims} do not fit heads of {m['dim']}")
+    mask = m.get("mask") or {}
+    mixer = MixerConfig(heads=int(m["heads"]), kv_heads=int(m.get("kv_heads", m["heads"])), dim=int(m["dim"]),
+                        vdim=int(m.get("vdim", m["dim"])), scale=float(m["scale"]), softcap=float(m.get("softcap") or 0.0),
+                        window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0), rot=rot,
+                        kv_from=-1 if m.get("kv_from") is None else int(m["kv_from"]))
+    if mixer.heads % mixer.kv_heads:
+        raise ValueError(f"layer {i}: {mixer.heads} query heads over {mixer.kv_heads} key/value heads")
+    f = e.get("mlp")
+    if not f:
+        return LayerConfig(mixer)
+    if f.get("kind") != "dense":
+        raise ValueError(f"layer {i}: unsupported feed-forward {f.get('kind')!r}")
+    return LayerConfig(mixer, int(f["ff"]), "dense")

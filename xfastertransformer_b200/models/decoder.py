@@ -70,26 +70,11 @@ class Layer:
 class Decoder:
     def __init__(self, cfg: ModelConfig, ctx: DistContext, path: str, weight_dtype: str,
                  act_dtype: Optional[torch.dtype] = None, embed_from: Optional["Decoder"] = None):
-        self.cfg = cfg
-        self.ctx = ctx
-        self.spec: FamilySpec = family_for(cfg)
-        self.device = ctx.device
-        self.kind = WEIGHT_KIND[weight_dtype]
-        if self.device.type == "cuda" and self.kind in ("fp16", "fp32"):
-            # activations on B200 are bf16 end to end; 16-bit float weights are kept in bf16 so
-            # both tcgen05 operands share a type
-            self.kind = "bf16"
-        if self.kind == "fp8" and cfg.weight_data_type != "fp8_e4m3" and not Env.get().fake_model:
-            pass  # a bf16 DeepSeek checkpoint quantised to fp8 at load
-        self.act_dtype = act_dtype or (torch.bfloat16 if self.device.type == "cuda" else torch.float32)
-        self.tp, self.tpr = ctx.tp_size, ctx.tp_rank
+        self._setup(cfg, ctx, weight_dtype, act_dtype)
         self.src = WeightSource(path, cfg.weight_data_type, self.device)
         # DeepSeek checkpoints keep embedding, lm_head, norms and the router in bf16 whatever the projection type
         # (deepseek_moe_convert.py:117-180)
         self.aux_dtype = "bf16" if cfg.model_type == "deepseek_moe" else None
-        self.l0, self.l1 = P.pp_layer_range(cfg.num_layer, ctx.pp_size, ctx.pp_rank)
-        self.first_stage = ctx.pp_rank == 0
-        self.last_stage = ctx.pp_rank == ctx.pp_size - 1
         c = cfg
         (self.qs, self.qe), (self.ks, self.ke) = P.head_range(c.head_num, c.kv_head_num, self.tp, self.tpr)
         self.hq, self.hkv = self.qe - self.qs, self.ke - self.ks
@@ -110,6 +95,26 @@ class Decoder:
             self._load_head(embed_from)
             self._fold_norms()
         self.has_moe = any(L.mlp_kind not in ("llama", "gpt") for L in self.layers)
+
+    def _setup(self, cfg: ModelConfig, ctx: DistContext, weight_dtype: str, act_dtype: Optional[torch.dtype]) -> None:
+        """Everything that does not depend on how the family stores or shapes its weights."""
+        self.cfg = cfg
+        self.ctx = ctx
+        self.spec: FamilySpec = family_for(cfg)
+        self.device = ctx.device
+        self.kind = WEIGHT_KIND[weight_dtype]
+        cuda = self.device.type == "cuda"
+        if cuda and (self.kind == "fp16" or self.kind == "fp32" and not self.spec.layered):
+            # activations on B200 are bf16 end to end; 16-bit float weights are kept in bf16 so
+            # both tcgen05 operands share a type
+            self.kind = "bf16"
+        self.act_dtype = act_dtype or (torch.bfloat16 if cuda and self.kind != "fp32" else torch.float32)
+        self.hidden_dtype = self.act_dtype          # type of the hidden state between pipeline stages
+        self.hidden_width = cfg.hidden_size
+        self.tp, self.tpr = ctx.tp_size, ctx.tp_rank
+        self.l0, self.l1 = P.pp_layer_range(cfg.num_layer, ctx.pp_size, ctx.pp_rank)
+        self.first_stage = ctx.pp_rank == 0
+        self.last_stage = ctx.pp_rank == ctx.pp_size - 1
         self.pairs_run = 0          # forward_pair calls
         self._overlap = False       # True while forward_pair interleaves two batches (all-reduces are started, not awaited)
         self._work = None
@@ -770,6 +775,8 @@ class Decoder:
         """Final norm on the rows that need logits + vocab-split lm_head -> fp32 [rows, vocab/tp]."""
         if b.logit_rows is not None:
             x = x.index_select(0, b.logit_rows)
+            if x.shape[0] == 0:
+                return torch.empty(0, self.v1 - self.v0, dtype=torch.float32, device=x.device)
         if self.head_fold:
             with TimeLine("DistLinear.forward"):
                 return ops.linear_rms(x, self.lm_head, self.eps, out_dtype=torch.float32)
@@ -788,6 +795,11 @@ class Decoder:
             return x
 
     # -- sizes ------------------------------------------------------------------------------
+    def plan_splits(self, B: int, max_kv: int, int8: bool) -> Optional[int]:
+        """Split-KV factor of a captured decode step, or None when every layer plans its own."""
+        from ..ops import native as N
+        return N.plan_attn_splits(B, max(self.hkv, 1), self.group, self.D, max_kv, int8)[0]
+
     def kv_geometry(self):
         c = self.cfg
         if self.spec.attention == "mla":

@@ -1,0 +1,264 @@
+"""Decoder for designs described layer by layer (``ModelConfig.layers``), first of them Kafipel.
+
+It is the generic decoder with sizes, rotation, mask and cache pool taken from each layer's own entry, served by the same
+engine, paged cache, decode runner, sampler and kernels.  What these designs add to it, each as an op with its constants
+as arguments:
+
+* a 32-bit residual stream with a norm before and after every sublayer, one launch between two products
+  (`ops.residual_norm`): x += norm_b(y) and h = norm(x) for the product that follows;
+* attention with a sliding window that keeps the first tokens, a tanh cap on the scores and a sink per head
+  (`ops.paged_attention(window=, keep_first=, softcap=, sinks=)`);
+* layers without keys and values of their own, which read the pool of an earlier layer (`kv_from`);
+* query/key and value heads of different sizes.
+
+Widths that the 16-byte rows of the tensor-core kernels do not allow are padded with zeros at load: the hidden and the
+feed-forward width to a multiple of 8, heads to the next size the attention kernels have.  A zero dimension adds nothing
+to a score or a sum.  The 32-bit path (dtype "fp32") and CPU tensors keep the heads as they are.
+"""
+from __future__ import annotations
+
+import math
+from typing import Dict, List, Optional
+
+import torch
+
+from .. import ops
+from ..config import LayerConfig, ModelConfig, RotaryConfig
+from ..ops import reference as R
+from ..parallel import partition as P
+from ..parallel.dist import DistContext
+from ..runtime.kv_cache import PagedKVCache
+from ..runtime.loader import SafetensorsSource, make_linear
+from ..utils import debugger
+from ..utils.progress import ProgressBar
+from ..utils.trace import TimeLine
+from .decoder import Batch, Decoder, Layer
+
+ATTENTION_HEADS = (64, 128, 256)          # head sizes of the tensor-core attention kernels
+
+
+def _up(n: int, m: int) -> int:
+    return (n + m - 1) // m * m
+
+
+def _pad(t: torch.Tensor, *shape: int) -> torch.Tensor:
+    """`t` in the corner of a zero tensor of `shape`."""
+    if tuple(t.shape) == shape:
+        return t
+    out = torch.zeros(shape, dtype=t.dtype, device=t.device)
+    out[tuple(slice(n) for n in t.shape)] = t
+    return out
+
+
+class LayeredDecoder(Decoder):
+    def __init__(self, cfg: ModelConfig, ctx: DistContext, path: str, weight_dtype: str,
+                 act_dtype: Optional[torch.dtype] = None, embed_from: Optional["LayeredDecoder"] = None):
+        self._setup(cfg, ctx, weight_dtype, act_dtype)
+        self.hidden_dtype = torch.float32
+        self.exact = self.kind == "fp32"
+        self.eps = cfg.layernorm_eps
+        self.W = cfg.hidden_size
+        gpu = self.device.type == "cuda"
+        self.hidden_width = self.WP = _up(self.W, 8) if gpu else self.W
+        self.pad_heads = gpu and not self.exact
+        self.src = SafetensorsSource(path, self.device)
+        self._ropes: Dict[RotaryConfig, torch.Tensor] = {}
+        self._old_ropes: List[torch.Tensor] = []
+        self.slopes = None
+        self.has_moe = False
+        with TimeLine("Decoder.loadWeights"):
+            self._load_ends(embed_from)
+            self.layers: List[Layer] = [self._load_layer(i)
+                                        for i in ProgressBar.wrap(range(self.l0, self.l1), "Loading layers")]
+        # cache pools: one per layer with keys and values of its own
+        self.pools: Dict[int, int] = {}
+        for L in self.layers:
+            if L.own_kv:
+                self.pools[L.idx] = len(self.pools)
+        for L in self.layers:
+            if L.kv_layer not in self.pools:
+                raise ValueError(f"layer {L.idx} reads the keys of layer {L.kv_layer}, which is on another pipeline stage")
+            L.pool = self.pools[L.kv_layer]
+        L = self.layers[0]
+        self.D, self.hq, self.hkv, self.group, self.scale = L.kd, L.hq, L.hkv, L.group, L.mix.scale
+        for L in self.layers:
+            self._rope(L.mix.rot, 2048)
+
+    # ------------------------------------------------------------------------------------
+    # rotary tables: one per distinct rotation, grown when a longer context comes up
+    # ------------------------------------------------------------------------------------
+    def _rope(self, rot: Optional[RotaryConfig], positions: int) -> Optional[torch.Tensor]:
+        if rot is None or rot.dims == 0:
+            return None
+        tab = self._ropes.get(rot)
+        if tab is None or tab.shape[0] < positions:
+            n = max(_up(positions, 2048), 2 * tab.shape[0] if tab is not None else 0)
+            if rot.factor > 0:
+                new = R.rope_table(n, rot.dims, rot.base, "yarn", rot.factor, rot.original, rot.fast, rot.slow,
+                                   table_scale=0.1 * math.log(rot.factor) + 1.0)
+            else:
+                new = R.rope_table(n, rot.dims, rot.base)
+            if tab is not None:
+                self._old_ropes.append(tab)       # captured decode graphs keep reading it (their positions fit it)
+            tab = self._ropes[rot] = new.to(self.device)
+        return tab
+
+    def _ensure_positions(self, b: Batch, cache: PagedKVCache) -> None:
+        need = max(b.max_kv, b.block_table.shape[1] * cache.block)     # a captured step may run to the table's width
+        for rot in list(self._ropes):
+            self._rope(rot, need)
+
+    # ------------------------------------------------------------------------------------
+    # weights
+    # ------------------------------------------------------------------------------------
+    def _gain(self, name: str):
+        return self.src.vector(name, self.W, fake_ones=True), None      # (gain, bias)
+
+    def _load_ends(self, share: Optional["LayeredDecoder"]) -> None:
+        c = self.cfg
+        self.v0, self.v1 = P.vocab_range(c.vocab_size, self.tp, self.tpr)
+        if share is not None:
+            self.wte, self.final, self.lm_head = share.wte, share.final, share.lm_head
+            return
+        self.wte = self.final = self.lm_head = None
+        if self.first_stage:
+            self.wte = _pad(self.src.matrix("embed", (c.vocab_size, self.W)).to(torch.bfloat16), c.vocab_size, self.WP)
+        if self.last_stage:
+            self.final = self._gain("final.norm")
+            w = self.src.matrix("head", (c.vocab_size, self.W), rows=(self.v0, self.v1))
+            kind = "fp32" if self.exact or self.device.type == "cpu" else "bf16"
+            self.lm_head = make_linear(_pad(w, w.shape[0], self.WP), kind)
+
+    def _head_size(self, n: int) -> int:
+        if not self.pad_heads:
+            return n
+        return next((d for d in ATTENTION_HEADS if n <= d), _up(n, 8))
+
+    def _head_rows(self, name: str, heads: int, rng, dim: int, padded: int) -> torch.Tensor:
+        """Rows of heads rng[0] .. rng[1] of a [heads * dim, width] projection, each head padded to `padded` rows."""
+        w = self.src.matrix(name, (heads * dim, self.W), rows=(rng[0] * dim, rng[1] * dim))
+        n = rng[1] - rng[0]
+        return _pad(w.view(n, dim, self.W), n, padded, self.WP).reshape(n * padded, self.WP)
+
+    def _load_layer(self, i: int) -> Layer:
+        lc: LayerConfig = self.cfg.layers[i]
+        m = lc.mixer
+        L = Layer()
+        L.idx, L.mix, L.ff = i, m, lc.ff
+        p = f"l{i}."
+        # this rank's heads; query head h reads key/value head h // (heads / kv_heads)
+        (qs, qe), (ks, ke) = P.head_range(m.heads, m.kv_heads, self.tp, self.tpr)
+        L.hq, L.hkv, L.group = qe - qs, ke - ks, m.heads // m.kv_heads
+        L.q_off = qs - ks * L.group
+        if L.hq <= 0:
+            raise ValueError(f"layer {i}: {m.heads} heads cannot be split over {self.tp} ranks")
+        L.kd, L.vd = self._head_size(m.dim), self._head_size(m.vdim)
+        if self.pad_heads:
+            L.kd = L.vd = max(L.kd, L.vd)         # the tensor-core kernels have one size for keys and values
+        L.own_kv = m.kv_from < 0
+        L.kv_layer = i if L.own_kv else m.kv_from
+        L.norm1, L.norm1b = self._gain(p + "norm1"), self._gain(p + "norm1b")
+        parts = [self._head_rows(p + "mix.q", m.heads, (qs, qe), m.dim, L.kd)]
+        if L.own_kv:
+            parts.append(self._head_rows(p + "mix.k", m.kv_heads, (ks, ke), m.dim, L.kd))
+            parts.append(self._head_rows(p + "mix.v", m.kv_heads, (ks, ke), m.vdim, L.vd))
+        L.qkv = make_linear(torch.cat(parts), self.kind)
+        L.sinks = None
+        if self.src.exists(p + "mix.sink") or self.src.fake:
+            L.sinks = self.src.vector(p + "mix.sink", m.heads, rng=(qs, qe)).contiguous()
+        w = self.src.matrix(p + "mix.o", (self.W, m.heads * m.vdim), cols=(qs * m.vdim, qe * m.vdim))
+        w = _pad(w.reshape(self.W, L.hq, m.vdim), self.WP, L.hq, L.vd)
+        L.o = make_linear(w.reshape(self.WP, L.hq * L.vd), self.kind)
+        L.mlp_kind = "none"
+        if lc.ff:
+            L.mlp_kind = "llama"
+            L.norm2, L.norm2b = self._gain(p + "norm2"), self._gain(p + "norm2b")
+            r = self._ffn_range(lc.ff)
+            n = r[1] - r[0]
+            np_ = _up(n, 8) if self.device.type == "cuda" else n
+            gate, up = (_pad(self.src.matrix(p + "mlp." + x, (lc.ff, self.W), rows=r), np_, self.WP) for x in ("gate", "up"))
+            L.gate_up = make_linear(torch.cat([gate, up]), self.kind)
+            L.down = make_linear(_pad(self.src.matrix(p + "mlp.down", (self.W, lc.ff), cols=r), self.WP, np_), self.kind)
+            L.act = "silu"
+        return L
+
+    # ------------------------------------------------------------------------------------
+    # forward
+    # ------------------------------------------------------------------------------------
+    def _mixer(self, L: Layer, h: torch.Tensor, b: Batch, cache: PagedKVCache) -> torch.Tensor:
+        """Attention sublayer: normalised input -> output projection (summed over tensor-parallel ranks)."""
+        m, li = L.mix, L.pool
+        kc, vc, ks, vs = cache.k[li], cache.v[li], cache.ks[li], cache.vs[li]
+        table, rot = self._rope(m.rot, 0), m.rot.dims if m.rot is not None else 0
+        new_kv = L.hkv if L.own_kv else 0
+        if h.is_cuda and not self.exact and ops.can_fuse_qkv_rope(L.qkv, h.shape[0], L.kd, kc, ks, None, None, "half"):
+            with TimeLine("QKV.linear+QKPO"):
+                q = ops.qkv_linear_rope_cache(h, L.qkv, None, None, L.hq, new_kv, b.positions, table, rot, "half", kc, vc,
+                                              b.slots)
+        else:
+            with TimeLine("QKV.linear"):
+                qkv = ops.linear(h, L.qkv)
+            with TimeLine("QKPO"):
+                q = ops.qkv_rope_cache(qkv, L.hq, new_kv, L.kd, b.positions, table, rot, "half", kc, vc, ks, vs, b.slots,
+                                       dv=L.vd)
+        with TimeLine("MHA"):
+            a = ops.paged_attention(q, kc, vc, b.block_table, b.cu_q, b.kv_lens, m.scale, ks, vs, group=L.group,
+                                    q_off=L.q_off, meta=b, softcap=m.softcap, window=m.window, keep_first=m.keep_first,
+                                    sinks=L.sinks)
+        with TimeLine("Output"):
+            return self._row_parallel(a.reshape(a.shape[0], -1), L.o, None, None)
+
+    def _ff(self, L: Layer, h: torch.Tensor) -> torch.Tensor:
+        with TimeLine("LlamaMLP"):
+            return self._row_parallel(ops.linear_gated(h, L.gate_up, L.act), L.down, None, None)
+
+    def _add_norm(self, x, y, post, nxt, **kw):
+        return ops.residual_norm(x, y, post, nxt, self.eps, self.spec.norm, h_dtype=self.act_dtype, **kw)
+
+    def forward(self, b: Batch, cache: PagedKVCache, hidden: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """Local logits on the last stage, the residual stream otherwise.  The norm of each sublayer's output, the
+        residual sum and the norm in front of the next sublayer are one launch; so are the embedding and the first norm,
+        and on the last stage the last sum and the final norm, on the rows whose logits are wanted."""
+        self._ensure_positions(b, cache)
+        dbg = debugger.enabled()
+        step = debugger.next_step() if dbg else 0
+        with TimeLine("Decoder.forward"):
+            first = self.layers[0].norm1
+            if self.first_stage:
+                x, h = self._add_norm(None, None, None, first, ids=b.ids, table=self.wte)
+            else:
+                x, h = self._add_norm(hidden, None, None, first)
+            if dbg:
+                debugger.dump("embedding", x[:, :self.W], self.ctx.rank, step)
+            for n, L in enumerate(self.layers):
+                last = n + 1 == len(self.layers)
+                after = None if last else self.layers[n + 1].norm1
+                y, post = self._mixer(L, h, b, cache), L.norm1b
+                if L.ff:
+                    x, h = self._add_norm(x, y, post, L.norm2)
+                    if dbg:
+                        debugger.dump(f"layer{L.idx}_attn_out", x[:, :self.W], self.ctx.rank, step)
+                    y, post = self._ff(L, h), L.norm2b
+                if not last:
+                    x, h = self._add_norm(x, y, post, after)
+                elif dbg or not self.last_stage:
+                    x, _ = self._add_norm(x, y, post, None)
+                    y = post = None
+                if dbg:
+                    debugger.dump(f"layer{L.idx}_ffn_out", x[:, :self.W], self.ctx.rank, step)
+            if not self.last_stage:
+                return x
+            if b.logit_rows is not None and b.logit_rows.numel() == 0:
+                return torch.empty(0, self.v1 - self.v0, dtype=torch.float32, device=x.device)
+            _, h = self._add_norm(x, y, post, self.final, rows=b.logit_rows, keep_x=False)
+            with TimeLine("DistLinear.forward"):
+                return ops.linear(h, self.lm_head, out_dtype=torch.float32)
+
+    # -- sizes ------------------------------------------------------------------------------
+    def plan_splits(self, B: int, max_kv: int, int8: bool) -> Optional[int]:
+        return None                               # windows differ from layer to layer: each launch plans its own split
+
+    def kv_geometry(self):
+        own = [L for L in self.layers if L.own_kv]
+        return dict(kv_heads=own[0].hkv, k_dim=own[0].kd, v_dim=own[0].vd, latent=False,
+                    layers=[(L.hkv, L.kd, L.vd) for L in own])

@@ -1,4 +1,4 @@
-"""Family registry: ``config.ini`` section name -> `FamilySpec`.
+"""Family registry: ``config.ini`` section name (``config.json`` architecture) -> `FamilySpec`.
 
 The reference instantiates one C++ class per family through a string-keyed factory
 (``src/models/model_factory.h:57-114``, table of families ``src/models/*.cpp``).  Here a family is
@@ -30,6 +30,8 @@ class FamilySpec:
     prefix_lm: bool = False         # chatglm-1 bidirectional prompt
     final_norm: bool = True
     embed_dtype: str = "same"
+    layered: bool = False           # sizes and mixers per layer (`ModelConfig.layers`), safetensors weights
+    post_norm: bool = False         # a second norm after each sublayer, before the residual sum
 
 
 FAMILIES: Dict[str, FamilySpec] = {
@@ -50,6 +52,7 @@ FAMILIES: Dict[str, FamilySpec] = {
     "chatglm4": FamilySpec("chatglm4", rope="interleaved", rot_frac=0.5, qkv_bias=True, mlp="chatglm2"),
     "gpt": FamilySpec("gpt", norm="layer", rope="none", qkv_bias=True, dense_bias=True, mlp="gpt", embedding="opt"),
     "telechat": FamilySpec("telechat", dense_bias=True, telechat_ntk=True),
+    "kafipel": FamilySpec("kafipel", norm="layer", layered=True, post_norm=True),
 }
 
 
@@ -61,6 +64,15 @@ def family_for(cfg: ModelConfig) -> FamilySpec:
         # Baichuan-13B has no rotary table: ALiBi (src/layers/attn_baichuan.h:33-47)
         spec = replace(spec, alibi=True, rope="none")
     return spec
+
+
+def decoder_class(cfg: ModelConfig):
+    """The class that runs a family: the generic decoder, or the layered one for designs described layer by layer."""
+    if family_for(cfg).layered:
+        from .layered import LayeredDecoder
+        return LayeredDecoder
+    from .decoder import Decoder
+    return Decoder
 
 
 def model_key(cfg: ModelConfig, weight_dtype: str, kv_dtype: str) -> str:

@@ -46,6 +46,15 @@ def layernorm(x, w, b, eps):
     return R.layernorm(x, w, b, eps)
 
 
+def residual_norm(x, y, post, nxt, eps, kind="layer", rows=None, h_dtype=torch.bfloat16, ids=None, table=None, keep_x=True):
+    """One step of a 32-bit residual stream in one launch: x (or table[ids]) += norm(y) with `post` = (gain, bias or
+    None) (plain y without it), then h = norm(x) with `nxt` for the next product.  Returns (x, h); on a GPU x is updated
+    in place unless `rows` selects rows, and buffers are as wide as x (a multiple of 8, padding zero)."""
+    if _cuda(x if x is not None else table):
+        return _nat().residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids, table, keep_x)
+    return R.residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids, table, keep_x)
+
+
 # -- GEMMs ---------------------------------------------------------------------------------
 def _verbose() -> bool:
     from ..utils.flags import Env
@@ -113,18 +122,18 @@ def gated_act(gu, act="silu"):
 
 # -- attention -----------------------------------------------------------------------------
 def qkv_rope_cache(qkv, hq, hkv, d, positions, table, rot_dim, style, kc, vc, ks, vs, slots,
-                   q_scale=None, q_norm_w=None, k_norm_w=None, eps=1e-6, rot_offset=0):
-    """Split packed qkv [T,(hq+2hkv)*d], optional per-head q/k RMSNorm (Qwen3), RoPE on q and k,
+                   q_scale=None, q_norm_w=None, k_norm_w=None, eps=1e-6, rot_offset=0, dv=None):
+    """Split packed qkv [T,(hq+2hkv)*d] (value heads of size `dv` when given; hkv = 0: query heads only), optional per-head q/k RMSNorm (Qwen3), RoPE on q and k,
     append k/v to the paged cache at `slots` (int8-quantising when scales are given); returns
     q [T,hq,d].  One kernel on the GPU (reference: QKPO + storeKVCache,
     src/layers/attention.h:560-640, src/kernels/attention_kernels.h:45-69)."""
     if _cuda(qkv):
         return _nat().qkv_rope_cache(qkv, hq, hkv, d, positions, table, rot_dim, style, kc, vc, ks, vs, slots,
-                                       q_scale, q_norm_w, k_norm_w, eps, rot_offset)
+                                       q_scale, q_norm_w, k_norm_w, eps, rot_offset, dv)
     T = qkv.shape[0]
     q = qkv[:, : hq * d].reshape(T, hq, d)
     k = qkv[:, hq * d:(hq + hkv) * d].reshape(T, hkv, d)
-    v = qkv[:, (hq + hkv) * d:].reshape(T, hkv, d)
+    v = qkv[:, (hq + hkv) * d:].reshape(T, hkv, dv or d)
     if q_norm_w is not None:
         q = R.rmsnorm(q, q_norm_w, eps)
         k = R.rmsnorm(k, k_norm_w, eps)
@@ -132,7 +141,8 @@ def qkv_rope_cache(qkv, hq, hkv, d, positions, table, rot_dim, style, kc, vc, ks
         q, k = R.rope_apply(q, k, positions, table, rot_dim, style, rot_offset, q_scale)
     elif q_scale is not None:
         q = (q.float() * q_scale[:, None, None]).to(q.dtype)
-    R.kv_cache_write(k, v, kc, vc, slots, ks, vs)
+    if hkv > 0:
+        R.kv_cache_write(k, v, kc, vc, slots, ks, vs)
     return q.contiguous()
 
 
@@ -167,12 +177,15 @@ def qkv_linear_rope_cache(x, W, bias, rms_eps, hq, hkv, positions, table, rot_di
 
 
 def paged_attention(q, kc, vc, block_table, cu_q, kv_lens, scale, ks=None, vs=None, slopes=None,
-                    causal=True, prefix_lm_lens=None, group=None, q_off=0, meta=None):
+                    causal=True, prefix_lm_lens=None, group=None, q_off=0, meta=None, softcap=0.0, window=0, keep_first=0,
+                    sinks=None):
+    """Attention of a ragged batch over the paged cache; `softcap`, `window` with `keep_first`, and `sinks` as in
+    `reference.paged_attention`."""
     if _cuda(q):
         return _nat().paged_attention(q, kc, vc, block_table, cu_q, kv_lens, scale, ks, vs, slopes,
-                                        causal, prefix_lm_lens, group, q_off, meta)
+                                        causal, prefix_lm_lens, group, q_off, meta, softcap, window, keep_first, sinks)
     return R.paged_attention(q, kc, vc, block_table, cu_q, kv_lens, scale, ks, vs, slopes, causal,
-                             prefix_lm_lens, group, q_off)
+                             prefix_lm_lens, group, q_off, softcap, window, keep_first, sinks)
 
 
 def mla_attention(q_nope, q_rope, latent_cache, block_table, cu_q, kv_lens, w_uk, w_uv, scale, absorbed=True,

@@ -35,7 +35,10 @@ def _ENV():
 
 
 def lib_path() -> str:
-    return os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "lib", "libxft_b200_kernels.so")
+    """The kernel library: the full one, or (when only that was built) the part that layered models call."""
+    d = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "lib")
+    full, part = os.path.join(d, "libxft_b200_kernels.so"), os.path.join(d, "libxft_b200_layered.so")
+    return part if os.path.exists(part) and not os.path.exists(full) else full
 
 
 def lib():
@@ -46,7 +49,8 @@ def lib():
             raise KernelError(f"{p} is missing: run `python csrc/build.py` (or __graft_entry__.build())")
         _LIB = C.CDLL(p)
         for fn in ("xft_gemm_bf16", "xft_embedding", "xft_rmsnorm", "xft_layernorm", "xft_gated_act",
-                   "xft_qkv_rope_cache", "xft_rope", "xft_latent_write", "xft_argmax", "xft_paged_attention"):
+                   "xft_qkv_rope_cache", "xft_rope", "xft_latent_write", "xft_argmax", "xft_paged_attention",
+                   "xft_paged_attention_ext"):
             getattr(_LIB, fn).restype = C.c_int
         # XFT_PDL=0: plain stream order instead of programmatic dependent launch between the kernels
         _LIB.xft_set_pdl(int(os.environ.get("XFT_PDL", "1") != "0"))
@@ -164,6 +168,58 @@ def layernorm(x, w, b, eps):
     return y.view(*x.shape[:-1], H)
 
 
+def residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids=None, table=None, keep_x=True):
+    """csrc/kernels/residual_norm.cu.  x fp32 [T, HP]; y bf16 or fp32 rows; gains fp32 [H]."""
+    dev = (x if x is not None else table).device
+    gain = nxt[0] if nxt is not None else post[0] if post is not None else None
+    H = gain.numel() if gain is not None else x.shape[1] if x is not None else table.shape[1]
+    HP = (H + 7) // 8 * 8
+    n_in = ids.numel() if ids is not None else x.shape[0]
+    n_out = rows.numel() if rows is not None else n_in
+    if ids is not None:
+        assert table.dtype == torch.bfloat16 and table.stride(1) == 1
+    else:
+        assert x.dtype == torch.float32 and x.stride(1) == 1
+    if y is not None:
+        y = y.reshape(-1, y.shape[-1])
+        assert y.shape[0] == n_in and y.stride(1) == 1 and y.dtype in (torch.float32, torch.bfloat16)
+    x_out = None
+    if keep_x:
+        x_out = x if ids is None and rows is None else torch.empty(n_out, HP, dtype=torch.float32, device=dev)
+    h = torch.empty(n_out, HP, dtype=h_dtype, device=dev) if nxt is not None else None
+    rows32 = None if rows is None else rows if rows.dtype == torch.int32 else rows.int()
+    ids32 = None if ids is None else ids if ids.dtype == torch.int32 else ids.int()
+    ws = Workspace.get(dev)
+    pw, pb = post if post is not None else (None, None)
+    nw, nb = nxt if nxt is not None else (None, None)
+    fn = lib().xft_residual_norm
+    fn.restype = C.c_int
+    _check(fn(_p(ids32), _p(table if ids is not None else None), 0 if ids is None else table.shape[0],
+              C.c_longlong(0 if ids is None else table.stride(0)), _p(x if ids is None else None),
+              0 if ids is not None else x.stride(0), _p(x_out), 0 if x_out is None else x_out.stride(0), _p(y),
+              0 if y is None else y.stride(0), int(y is not None and y.dtype == torch.float32), _p(pw), _p(pb), _p(nw), _p(nb),
+              _p(h), HP, int(h_dtype == torch.float32), _p(rows32), n_in, n_out, H, 0 if kind == "layer" else 1,
+              C.c_float(eps), _p(ws.status), _stream()), "residual_norm")
+    ws.launches += 1
+    return x_out, h
+
+
+def gemm_f32(x, w, N):
+    """Y[T,N] = X[T,K] W[N,K]^T, everything in 32 bits."""
+    x2 = x.reshape(-1, x.shape[-1])
+    if x2.stride(1) != 1:
+        x2 = x2.contiguous()
+    T, K = x2.shape
+    assert x2.dtype == torch.float32 and w.dtype == torch.float32 and w.stride(1) == 1 and w.shape[1] == K
+    y = torch.empty(T, N, dtype=torch.float32, device=x.device)
+    fn = lib().xft_gemm_f32
+    fn.restype = C.c_int
+    _check(fn(_p(x2), x2.stride(0) if T > 1 else max(x2.stride(0), K), _p(w), w.stride(0), _p(y), N, T, N, K, _stream()),
+           "gemm_f32")
+    Workspace.get(x.device).launches += 1
+    return y
+
+
 def gemm_bf16(x, w, N, gated=False, dual_off=0, bias=None, act=None, residual=None, res_scale=1.0, out_dtype=None,
               out=None, row_scale=None, force_splits=0):
     """Y[T,N] = epi(X[T,K] · W[rows,K]^T) on tcgen05.  `w`: bf16 [rows, K] (rows = N, or 2 blocks for gated)."""
@@ -274,7 +330,7 @@ def can_fuse_qkv_rope(W, T, D, kc, ks, q_norm_w, k_norm_w, style) -> bool:
     """The QKV product can end in RoPE + paged cache append (one kernel instead of two): bf16 weights, head_dim 128,
     a bf16 cache, no per-head q/k norm, at most SK_MAX_TOKENS rows."""
     e = _ENV()
-    return (e.gemm_streamk and e.fuse_qkv_rope and W.kind == "bf16" and T <= SK_MAX_TOKENS and D == 128 and ks is None
+    return (e.gemm_streamk and e.fuse_qkv_rope and W.kind == "bf16" and 0 < T <= SK_MAX_TOKENS and D == 128 and ks is None
             and kc.dtype == torch.bfloat16 and q_norm_w is None and k_norm_w is None and style in ("half", "interleaved"))
 
 
@@ -347,6 +403,10 @@ def linear(x, W, bias=None, act=None, residual=None, res_scale=1.0, out_dtype=No
     if W.kind == "bf16":
         y = gemm_bf16(x, W.w, W.out_features, bias=bias, act=act, residual=residual, res_scale=res_scale,
                       out_dtype=out_dtype)
+    elif W.kind == "fp32":
+        if bias is not None or act is not None or residual is not None or out_dtype not in (None, torch.float32):
+            raise KernelError("fp32 products have no epilogue")
+        y = gemm_f32(x, W.w, W.out_features)
     else:
         from . import native_quant
         y = native_quant.linear(x, W, bias, act, residual, res_scale, out_dtype)
@@ -358,6 +418,15 @@ def linear_gated(x, W, act="silu", bias=None):
     I = W.out_features // 2
     if W.kind == "bf16":
         y = gemm_bf16(x, W.w, I, gated=True, dual_off=I, bias=bias, act=act)
+    elif W.kind == "fp32":
+        if bias is not None:
+            raise KernelError("fp32 products have no epilogue")
+        gu = gemm_f32(x, W.w, 2 * I)
+        y = torch.empty(gu.shape[0], I, dtype=torch.float32, device=x.device)
+        fn = lib().xft_gated_act_f32
+        fn.restype = C.c_int
+        _check(fn(_p(gu), 2 * I, _p(y), gu.shape[0], I, _ACT[act], _stream()), "gated_act_f32")
+        Workspace.get(x.device).launches += 1
     else:
         from . import native_quant
         y = native_quant.linear_gated(x, W, act, bias)
@@ -375,7 +444,10 @@ def gated_act(gu, act="silu"):
 
 # ------------------------------------------------------------------------------------------
 def qkv_rope_cache(qkv, hq, hkv, d, positions, table, rot_dim, style, kc, vc, ks, vs, slots,
-                   q_scale=None, q_norm_w=None, k_norm_w=None, eps=1e-6, rot_offset=0):
+                   q_scale=None, q_norm_w=None, k_norm_w=None, eps=1e-6, rot_offset=0, dv=None):
+    if qkv.dtype == torch.float32 or d > 256 or (dv or d) != d:
+        return _rope_cache_plain(qkv, hq, hkv, d, dv or d, positions, table, rot_dim, style, kc, vc, ks, slots, q_scale,
+                                 q_norm_w, rot_offset)
     qkv2, ldq = _rows2d(qkv)
     T = qkv2.shape[0]
     q = torch.empty(T, hq, d, dtype=torch.bfloat16, device=qkv.device)
@@ -387,6 +459,28 @@ def qkv_rope_cache(qkv, hq, hkv, d, positions, table, rot_dim, style, kc, vc, ks
                                   C.c_float(eps), _p(q), _p(kc), _p(vc), _p(ks), _p(vs), int(ks is not None), bs,
                                   C.c_longlong(nb * bs), _p(slots), _p(ws.status), _stream())
     _check(rc, "qkv_rope_cache")
+    ws.launches += 1
+    return q
+
+
+def _rope_cache_plain(qkv, hq, hkv, kd, vd, positions, table, rot_dim, style, kc, vc, ks, slots, q_scale, q_norm_w,
+                      rot_offset):
+    """Head sizes and types the vectorised kernel does not take (csrc/kernels/plain.cu)."""
+    if ks is not None or q_scale is not None or q_norm_w is not None or rot_offset:
+        raise KernelError("fp32 rows or large heads: no int8 cache, q/k norm, query scaling or rotary offset")
+    if kc.dtype != qkv.dtype or vc.dtype != qkv.dtype:
+        raise KernelError(f"the cache ({kc.dtype}) must have the type of the rows ({qkv.dtype})")
+    T = qkv.shape[0]
+    qkv = qkv if qkv.stride(1) == 1 else qkv.contiguous()
+    q = torch.empty(T, hq, kd, dtype=qkv.dtype, device=qkv.device)
+    ws = Workspace.get(qkv.device)
+    nb, _, bs, _ = kc.shape
+    fn = lib().xft_rope_cache
+    fn.restype = C.c_int
+    rot = rot_dim if table is not None else 0
+    _check(fn(_p(qkv), max(qkv.stride(0), qkv.shape[1]), T, hq, hkv, kd, vd, _p(positions), _p(table), rot,
+              0 if style == "half" else 1, 0 if table is None else table.shape[0], _p(q), _p(kc), _p(vc), bs,
+              C.c_longlong(nb * bs), _p(slots), int(qkv.dtype == torch.float32), _p(ws.status), _stream()), "rope_cache")
     ws.launches += 1
     return q
 
@@ -475,10 +569,11 @@ def plan_attn_splits(B, hkv, group, D, max_kv, int8=False):
 
 
 def paged_attention(q, kc, vc, block_table, cu_q, kv_lens, scale, ks=None, vs=None, slopes=None, causal=True,
-                    prefix_lm_lens=None, group=None, q_off=0, meta=None):
+                    prefix_lm_lens=None, group=None, q_off=0, meta=None, softcap=0.0, window=0, keep_first=0, sinks=None):
     assert causal
     T, hq, D = q.shape
     nb, hkv, bs, _ = kc.shape
+    vd = vc.shape[3]
     dev = q.device
     ws = Workspace.get(dev)
     B = len(kv_lens)
@@ -495,10 +590,26 @@ def paged_attention(q, kc, vc, block_table, cu_q, kv_lens, scale, ks=None, vs=No
     if prefix_lm_lens is not None:
         pl = torch.tensor(list(prefix_lm_lens), dtype=torch.int32, device=dev)
     g = group or max(hq // hkv, 1)
+    if sinks is not None:
+        assert sinks.dtype == torch.float32 and sinks.numel() == hq and sinks.is_contiguous()
+    if q.dtype == torch.float32 or D not in (64, 128, 256) or vd != D:
+        if ks is not None or slopes is not None or pl is not None or kc.dtype != q.dtype or vc.dtype != q.dtype:
+            raise KernelError(f"head size {D} / {vd} in {q.dtype}: no int8 cache, ALiBi or prefix mask")
+        q = q.contiguous()
+        out = torch.empty(T, hq, vd, dtype=q.dtype, device=dev)
+        fn = lib().xft_attention_plain
+        fn.restype = C.c_int
+        _check(fn(_p(q), _p(out), _p(kc), _p(vc), _p(block_table), block_table.stride(0), _p(cu_dev), _p(kv_dev), B, T, hq,
+                  hkv, g, q_off, D, vd, bs, nb, C.c_float(scale), C.c_float(softcap), window, keep_first, _p(sinks),
+                  int(q.dtype == torch.float32), _p(ws.status), _stream()), "attention_plain")
+        ws.launches += 1
+        return out
     out = torch.empty_like(q)
     nsplit, po, pm = 1, None, None
     if decode:
-        nsplit, ntiles = plan_attn_splits(B, hkv, g, D, max_kv, ks is not None)
+        # a window bounds the keys a step can visit, whatever the context length
+        seen = min(max_kv, window + keep_first + 128) if window > 0 else max_kv
+        nsplit, ntiles = plan_attn_splits(B, hkv, g, D, seen, ks is not None)
         if meta is not None and getattr(meta, "meta", None) is not None and "nsplit" in meta.meta:
             nsplit = meta.meta["nsplit"]
         if B * hkv * ((g + 15) // 16) > ws.attn_counters.numel():
@@ -514,15 +625,17 @@ def paged_attention(q, kc, vc, block_table, cu_q, kv_lens, scale, ks=None, vs=No
         L = lib()
         L.xft_attn_prefill_tc.restype = C.c_int
         rc = L.xft_attn_prefill_tc(_p(q), _p(out), _p(kc), _p(vc), _p(block_table), block_table.stride(0), _p(cu_dev),
-                                   _p(kv_dev), B, T, max_q, hq, hkv, g, q_off, bs, nb, C.c_float(scale), _p(ws.status),
-                                   _stream())
+                                   _p(kv_dev), B, T, max_q, hq, hkv, g, q_off, bs, nb, C.c_float(scale),
+                                   C.c_float(softcap), window, keep_first, _p(sinks), _p(ws.status), _stream())
         _check(rc, "attn_prefill_tc")
         ws.launches += 1
         return out
-    rc = lib().xft_paged_attention(_p(q), _p(out), _p(kc), _p(vc), _p(ks), _p(vs), _p(block_table),
-                                   block_table.stride(0), _p(cu_dev), _p(kv_dev), B, max_q, hq, hkv, g, q_off, D, bs,
-                                   nb, C.c_float(scale), _p(slopes), _p(pl), (1 if _ENV().attn_tma else 2) if decode else 0, nsplit, _p(po), _p(pm),
-                                   _p(ws.attn_counters), _p(ws.status), _stream())
+    rc = lib().xft_paged_attention_ext(_p(q), _p(out), _p(kc), _p(vc), _p(ks), _p(vs), _p(block_table),
+                                       block_table.stride(0), _p(cu_dev), _p(kv_dev), B, max_q, hq, hkv, g, q_off, D, bs,
+                                       nb, C.c_float(scale), _p(slopes), _p(pl),
+                                       (1 if _ENV().attn_tma else 2) if decode else 0, nsplit, _p(po), _p(pm),
+                                       _p(ws.attn_counters), _p(ws.status), C.c_float(softcap), window, keep_first,
+                                       _p(sinks), _stream())
     _check(rc, "paged_attention")
     ws.launches += 1
     return out

@@ -65,6 +65,28 @@ def layernorm(x: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor], eps: 
     return y.to(x.dtype)
 
 
+def _norm(xf: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor], eps: float, kind: str) -> torch.Tensor:
+    d = xf - xf.mean(-1, keepdim=True) if kind == "layer" else xf
+    y = d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+    return y if b is None else y + b.float()
+
+
+def residual_norm(x, y, post, nxt, eps: float, kind: str = "layer", rows: Optional[torch.Tensor] = None,
+                  h_dtype: torch.dtype = torch.float32, ids=None, table=None, keep_x: bool = True):
+    """One step of a 32-bit residual stream: x (or table[ids]) plus y — normalised with `post` = (gain, bias) first, when
+    given — and the input of the next sublayer, h = norm(x) with `nxt` = (gain, bias).  `rows` selects rows.  Returns
+    (x or None, h or None)."""
+    xf = table[ids.long()].float() if ids is not None else x.float()
+    yf = None if y is None else y.float()
+    if rows is not None:
+        xf = xf[rows.long()]
+        yf = None if yf is None else yf[rows.long()]
+    if yf is not None:
+        xf = xf + (_norm(yf, post[0], post[1], eps, kind) if post is not None else yf)
+    h = None if nxt is None else _norm(xf, nxt[0], nxt[1], eps, kind).to(h_dtype)
+    return (xf if keep_x else None), h
+
+
 # ----------------------------------------------------------------------------------------
 # quantisation helpers (load time) and dequantisation (oracle)
 # ----------------------------------------------------------------------------------------
@@ -230,15 +252,15 @@ def yarn_mscale(scale: float = 1.0, mscale: float = 1.0) -> float:
 
 def rope_inv_freq(rot_dim: int, theta: float, scaling_type: str = "", factor: float = 1.0,
                   original_max_pos: int = 2048, beta_fast: float = 32, beta_slow: float = 1) -> torch.Tensor:
+    """Frequency of each rotated pair.  YaRN divides the slow ones by `factor`: none of the pairs up to `low`, all from
+    `high` on, a linear ramp between (a step when the two coincide)."""
     inv = 1.0 / (theta ** (torch.arange(0, rot_dim, 2, dtype=torch.float64) / rot_dim))
     if scaling_type == "linear" and factor != 1.0:
         inv = inv / factor
     elif scaling_type == "yarn" and factor != 1.0:
         low = max(math.floor(_yarn_find_dim(beta_fast, rot_dim, theta, original_max_pos)), 0)
         high = min(math.ceil(_yarn_find_dim(beta_slow, rot_dim, theta, original_max_pos)), rot_dim - 1)
-        if low == high:
-            high += 0.001
-        ramp = ((torch.arange(rot_dim // 2, dtype=torch.float64) - low) / (high - low)).clamp(0, 1)
+        ramp = ((torch.arange(rot_dim // 2, dtype=torch.float64) - low) / max(high - low, 0.001)).clamp(0, 1)
         mask = 1.0 - ramp                      # 1 -> extrapolate (keep), 0 -> interpolate
         inv = inv / factor * (1 - mask) + inv * mask
     return inv.float()
@@ -374,7 +396,8 @@ def paged_attention(q: torch.Tensor, kc: torch.Tensor, vc: torch.Tensor, block_t
                     ks: Optional[torch.Tensor] = None, vs: Optional[torch.Tensor] = None,
                     slopes: Optional[torch.Tensor] = None, causal: bool = True,
                     prefix_lm_lens: Optional[Sequence[int]] = None, group: Optional[int] = None,
-                    q_off: int = 0) -> torch.Tensor:
+                    q_off: int = 0, softcap: float = 0.0, window: int = 0, keep_first: int = 0,
+                    sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Ragged-batch attention over a paged cache that already holds the new tokens.
 
     q [T,Hq,D]; sequence b owns query rows cu_q[b]:cu_q[b+1]; its keys are cache positions
@@ -386,6 +409,9 @@ def paged_attention(q: torch.Tensor, kc: torch.Tensor, vc: torch.Tensor, block_t
     Local query head i reads local kv head (i + q_off) // group; the defaults (group = Hq/Hkv,
     q_off = 0) are plain GQA, other values appear with uneven TP head ranges
     (split_util.h:61-99: the kv range is the covering range of the q range).
+
+    `softcap` > 0: scores become softcap * tanh(score / softcap).  `window` > 0: position i sees the keys j <= i with
+    i - j < window or j < keep_first.  `sinks` [Hq]: exp(sinks[h]) joins the softmax denominator of head h.
     """
     T, Hq, D = q.shape
     Hkv = kc.shape[1]
@@ -404,6 +430,8 @@ def paged_attention(q: torch.Tensor, kc: torch.Tensor, vc: torch.Tensor, block_t
         Kx = K[hmap]
         Vx = V[hmap]
         s = torch.matmul(Q, Kx.transpose(1, 2)) * scale  # [Hq,ql,n]
+        if softcap > 0:
+            s = softcap * torch.tanh(s / softcap)
         qpos = torch.arange(n - ql, n, device=q.device)
         kpos = torch.arange(n, device=q.device)
         if slopes is not None:
@@ -413,8 +441,12 @@ def paged_attention(q: torch.Tensor, kc: torch.Tensor, vc: torch.Tensor, block_t
             mask = kpos[None, :] > qpos[:, None]
             if prefix_lm_lens is not None:
                 mask = mask & (kpos[None, :] >= int(prefix_lm_lens[b]))
+            if window > 0:
+                mask = mask | ((qpos[:, None] - kpos[None, :] >= window) & (kpos[None, :] >= keep_first))
             s = s.masked_fill(mask[None], float("-inf"))
-        p = torch.softmax(s, dim=-1)
+        if sinks is not None:                            # one more column that carries no value
+            s = torch.cat([s, sinks.to(s.device).float()[:, None, None].expand(Hq, ql, 1)], dim=-1)
+        p = torch.softmax(s, dim=-1)[..., :n]
         out[q0:q1] = torch.matmul(p, Vx).permute(1, 0, 2)
     return out.to(q.dtype)
 

@@ -139,14 +139,14 @@ class CudaRunner:
         g.host[o_cu:o_cu + B + 1] = torch.arange(B + 1, dtype=torch.int32)
         d = g.dev
         dec = m.decoder
-        from ..ops import native as N
-        g.nsplit, _ = N.plan_attn_splits(B, max(dec.hkv, 1), dec.group, dec.D, max_kv_hint, m.cache.int8)
+        g.nsplit = dec.plan_splits(B, max_kv_hint, m.cache.int8)
         b = Batch(ids=d[o_ids:o_ids + B], positions=d[o_pos:o_pos + B], slots=d[o_slot:o_slot + B],
                   cu_q=list(range(B + 1)), kv_lens=[max_kv_hint] * B, block_table=d[o_bt:o_bt + B * W].view(B, W),
                   logit_rows=None, is_decode=True, max_q=1, max_kv=max_kv_hint)
         b.cu_q_dev = d[o_cu:o_cu + B + 1]
         b.kv_lens_dev = d[o_kv:o_kv + B]
-        b.meta["nsplit"] = g.nsplit
+        if g.nsplit is not None:
+            b.meta["nsplit"] = g.nsplit
         g.batch = b
         g.version = m.cache.version
         g.graph = None

@@ -26,7 +26,8 @@ import torch
 
 from .. import ops
 from ..config import KV_DTYPES, ModelConfig, split_hybrid_dtype
-from ..models.decoder import Batch, Decoder
+from ..models.decoder import Batch, Decoder  # noqa: F401  (Decoder is re-exported)
+from ..models.registry import decoder_class, family_for
 from ..parallel.dist import CommError, DistContext
 from ..utils import log, trace
 from ..utils.flags import Env
@@ -54,27 +55,45 @@ def _to_lists(ids) -> List[List[int]]:
 
 class Model:
     def __init__(self, path: str, dtype: str = "bf16", kv_cache_dtype: str = "fp16",
-                 ctx: Optional[DistContext] = None):
+                 ctx: Optional[DistContext] = None, max_cache_tokens: int = 0):
+        """`max_cache_tokens` > 0 fixes the size of the KV pools (rounded up to whole blocks): they are made once and
+        never grow, and a request that does not fit raises MemoryError."""
         if kv_cache_dtype not in KV_DTYPES:
             raise ValueError(f"don't support KV cache data type: {kv_cache_dtype}.")
         self.ctx = ctx or DistContext.get()
-        self.cfg = ModelConfig.from_ini(path)
+        self.cfg = ModelConfig.load(path)
         self.env = Env.get()
         d_prefill, d_decode = split_hybrid_dtype(dtype)
+        layered = family_for(self.cfg).layered
+        if d_decode == "fp32":
+            if self.ctx.device.type == "cuda" and not layered:
+                raise ValueError(f"fp32 on a GPU is for layered designs; {self.cfg.model_type} runs in bf16 there")
+            if kv_cache_dtype == "int8" and layered:
+                raise ValueError("the 32-bit path keeps its KV cache in fp32")
+            kv_cache_dtype = "fp32" if kv_cache_dtype != "int8" else "int8"
+        if layered and self.ctx.dp_size > 1:
+            raise ValueError("XFT_ATTENTION_DP=1 is for mixture-of-experts models")
         if self.cfg.model_type == "deepseek_moe" and d_prefill not in ("bf16", "fp8_e4m3"):
             raise ValueError("deepseek_moe supports bf16 and fp8_e4m3 only")      # model_factory.h:105-114
         if d_prefill == "fp8_e4m3" and self.cfg.model_type != "deepseek_moe":
             raise ValueError("fp8_e4m3 is supported for deepseek_moe only")
         with TimeLine("Model.load"):
-            self.decoder = Decoder(self.cfg, self.ctx, path, d_decode)
+            make = decoder_class(self.cfg)
+            self.decoder = make(self.cfg, self.ctx, path, d_decode)
             # hybrid A_B: model A serves the first token, B the next ones; they share embedding,
             # head, KV cache and buffers (src/models/hybrid_model.h:23-105)
             self.prefill_decoder = self.decoder if d_prefill == d_decode else \
-                Decoder(self.cfg, self.ctx, path, d_prefill, embed_from=self.decoder)
+                make(self.cfg, self.ctx, path, d_prefill, embed_from=self.decoder)
         geo = self.decoder.kv_geometry()
+        blk = self.env.kv_block_size
+        # one block more for the padding rows of captured decode steps
+        spare = 1 if self.ctx.device.type == "cuda" and self.env.cuda_graph else 0
+        max_blocks = (max_cache_tokens + blk - 1) // blk + spare if max_cache_tokens > 0 else 0
         self.cache = PagedKVCache(len(self.decoder.layers), geo["kv_heads"], geo["k_dim"], geo["v_dim"],
-                                  kv_cache_dtype, self.ctx.device, self.env.kv_block_size,
-                                  self.decoder.act_dtype, geo["latent"])
+                                  kv_cache_dtype, self.ctx.device, blk, self.decoder.act_dtype, geo["latent"],
+                                  geo.get("layers"), max_blocks)
+        if max_blocks:
+            self.cache.ensure_blocks(max_blocks)
         if self.env.prefix_cache and self.ctx.dp_size == 1:
             # data-parallel attention keeps each sequence's cache on one rank only, while all ranks must agree on how
             # many tokens a prompt still has to run: automatic reuse stays off there
@@ -96,7 +115,7 @@ class Model:
         if self.ctx.device.type == "cuda" and self.ctx.tp_size > 1 and self.env.fused_comm and self.ctx.peer is None \
                 and self.ctx.tp_size <= 8:
             from ..parallel.fused_comm import PeerComm
-            self.ctx.peer = PeerComm(self.ctx, n_max=self.cfg.hidden_size)
+            self.ctx.peer = PeerComm(self.ctx, n_max=self.decoder.hidden_width)
         if self.ctx.device.type == "cuda" and self.ctx.dp_size > 1 and self.env.moe_fused_a2a and self.decoder.has_moe \
                 and self.ctx.epcomm is None and self.ctx.dp_size <= 8:
             from ..parallel.fused_comm import EpComm
@@ -104,7 +123,7 @@ class Model:
         if self.ctx.device.type == "cuda":
             from .cuda_runner import CudaRunner
             self.runner = CudaRunner(self)
-        if self.env.kv_cache_gb > 0:
+        if self.env.kv_cache_gb > 0 and not self.cache.max_blocks:
             # size the KV pools once: pools that never grow never move, so captured decode graphs stay valid
             per = max(self.cache.bytes_per_block(), 1)
             self.cache.ensure_blocks(max(int(self.env.kv_cache_gb * (1 << 30)) // per, 1))
@@ -457,7 +476,7 @@ class Model:
         else:
             rows = [s.all_tokens() for s in self.working]
             w = max(len(r) for r in rows) if rows else 0
-            pad = cfg.pad_token_id if cfg.pad_token_id >= 0 else cfg.eos_token_id
+            pad = max(cfg.pad_token_id if cfg.pad_token_id >= 0 else cfg.eos_token_id, 0)
             rows = [r + [pad] * (w - len(r)) for r in rows]
         self._release_working()
         if trace.enabled():
@@ -477,7 +496,8 @@ class Model:
     # continuous-batching API
     # ------------------------------------------------------------------------------------
     def set_input_cb(self, input_ids=None, seq_lens=None, seq_ids=None, max_length=None, greedy: bool = False,
-                     append: bool = False, hold: bool = False, extend: bool = False) -> torch.Tensor:
+                     append: bool = False, hold: bool = False, extend: bool = False, rows=None,
+                     on_demand: bool = False) -> torch.Tensor:
         """Prefill: ``input_ids`` = flattened prompts + ``seq_lens``; decode: ``input_ids`` [bs,1] +
         ``seq_ids``.  Returns the sequence ids (models.cpp:586-674).  ``greedy=True`` announces that the step will be
         run with ``forward_cb_greedy`` (followers need to know which forward follows).
@@ -489,7 +509,11 @@ class Model:
         Chunked prefill (``extend=True``, with ``seq_ids`` and ``seq_lens``): the tokens continue the PROMPTS of known
         sequences that have not generated anything yet, so a long prompt can be fed in pieces between the decode steps
         of the other sequences.  Create the sequence with its first piece and the ``max_length`` of the whole request;
-        the logits of every piece but the last are of no use to the caller."""
+        the logits of every piece but the last are of no use to the caller.
+
+        ``rows``: for each sequence of this call the places among its new tokens whose logits ``forward_cb`` returns
+        (default: the last one; may be empty).  ``on_demand``: new sequences take cache blocks as they grow instead of
+        reserving ``max_length`` tokens now."""
         def tl(x):
             if x is None:
                 return None
@@ -505,10 +529,13 @@ class Model:
                 isinstance(input_ids[0], (list, tuple)):
             seq_lens = [len(r) for r in input_ids]
         return self._call(OP_SET_INPUT_CB, (ids, tl(seq_lens), tl(seq_ids), tl(max_length), bool(greedy), bool(append),
-                                            bool(hold), bool(extend)))
+                                            bool(hold), bool(extend), None if rows is None else [list(r) for r in rows],
+                                            bool(on_demand)))
 
     def _do_set_input_cb(self, ids, seq_lens, seq_ids, max_len, greedy: bool = False, append: bool = False,
-                         hold: bool = False, extend: bool = False) -> torch.Tensor:
+                         hold: bool = False, extend: bool = False, rows=None, on_demand: bool = False) -> torch.Tensor:
+        if rows is not None and (self.ctx.dp_size > 1 or greedy):
+            raise ValueError("set_input_cb(rows=...): not with data-parallel attention or greedy=True")
         active = []
         self._cb_greedy = bool(greedy)
         self._cb_hold = bool(hold)
@@ -528,8 +555,9 @@ class Model:
                 self.cache.add_sequence(s.seq_id)
                 self._attach_prefix(s)            # before the reservation: adopted blocks must not be evicted for it
             # data-parallel attention: a rank caches only the sequences it owns
-            self.cache.reserve(sum(self.cache.blocks_for(s.max_len + 1) - len(self.cache.tables[s.seq_id])
-                                   for s in active if s.owner == self.ctx.dp_rank))
+            if not on_demand:
+                self.cache.reserve(sum(self.cache.blocks_for(s.max_len + 1) - len(self.cache.tables[s.seq_id])
+                                       for s in active if s.owner == self.ctx.dp_rank))
         elif extend:                                      # further prompt pieces of known sequences
             if not seq_lens or len(seq_lens) != len(seq_ids) or sum(seq_lens) != len(ids):
                 raise ValueError("set_input_cb(extend=True): one piece per sequence id, seq_lens adding up to the ids")
@@ -554,6 +582,12 @@ class Model:
                     raise RuntimeError(f"sequence {sid} has not been prefilled")
                 s.step_forward(int(t))
                 active.append(s)
+        if rows is not None and len(rows) != len(active):
+            raise ValueError("set_input_cb: one list of rows per sequence expected")
+        for i, s in enumerate(active):
+            s.rows = None if rows is None else rows[i]
+            if s.rows is not None and any(r < 0 or r >= len(s.pending) for r in s.rows):
+                raise ValueError(f"sequence {s.seq_id}: rows {s.rows} outside its {len(s.pending)} new tokens")
         self.cb_active = (self.cb_active + active) if append else active
         return torch.tensor([s.seq_id for s in active], dtype=torch.int64)
 
@@ -567,6 +601,9 @@ class Model:
             for s in seqs:                      # inputs are now in the cache
                 s.past_len += len(s.pending)
                 s.pending = []
+                s.rows = None
+            if local.shape[0] == 0:
+                return torch.empty(0, self.cfg.vocab_size, dtype=torch.float32, device=local.device)
             return S.gather_logits(local, self.ctx, self.vocab_sizes).float()
 
     def forward_cb_greedy(self) -> torch.Tensor:
@@ -703,12 +740,14 @@ class Model:
             slots.extend(sl)
             cu.append(cu[-1] + n)
             kvl.append(start + n)
-            rows.extend(range(cu[-2], cu[-1]) if logits_all else [cu[-1] - 1])
+            rows.extend(range(cu[-2], cu[-1]) if logits_all else [cu[-1] - 1] if s.rows is None else
+                        [cu[-2] + r for r in s.rows])
         decode = all(cu[i + 1] - cu[i] == 1 for i in range(len(seqs)))
+        every = rows == list(range(cu[-1]))              # each token's logits, in order: nothing to gather
         bt = self.cache.block_table([s.seq_id for s in seqs])
         i32 = lambda x: torch.tensor(x, dtype=torch.int32).to(dev, non_blocking=True)
         b = Batch(ids=i32(ids), positions=i32(pos), slots=i32(slots), cu_q=cu, kv_lens=kvl, block_table=bt.to(dev),
-                  logit_rows=None if (logits_all or decode) else i32(rows).long() if dev.type == "cpu" else i32(rows),
+                  logit_rows=None if every else i32(rows).long() if dev.type == "cpu" else i32(rows),
                   is_decode=decode, max_q=max(cu[i + 1] - cu[i] for i in range(len(seqs))), max_kv=max(kvl))
         b.cu_q_dev, b.kv_lens_dev = i32(cu), i32(kvl)
         if self.decoder.spec.rope == "2d":
@@ -768,7 +807,7 @@ class Model:
         groups = self._groups(seqs)
         if self.ctx.pp_size > 1:
             return self._pp_forward(groups, logits_all)
-        if self.env.prefill_overlap and self.ctx.tp_size > 1 and len(seqs) > 1 and all(len(s.pending) > 1 for s in seqs):
+        if self.env.prefill_overlap and not self.decoder.spec.layered and self.ctx.tp_size > 1 and len(seqs) > 1 and all(len(s.pending) > 1 for s in seqs):
             return self._run_overlapped(seqs, groups, logits_all)
         if len(groups) > 1:
             return torch.cat([self._run(g, logits_all) for g in groups], dim=0)
@@ -870,7 +909,7 @@ class Model:
         recvs = []
         if not first:
             for b, dec in zip(batches, decs):
-                h = torch.empty(b.ids.shape[0], self.cfg.hidden_size, dtype=dec.act_dtype, device=ctx.device)
+                h = torch.empty(b.ids.shape[0], dec.hidden_width, dtype=dec.hidden_dtype, device=ctx.device)
                 recvs.append((ctx.recv(h, ctx.rank - ctx.tp_size), h))
         outs, sends = [], []
         with torch.no_grad():
@@ -894,7 +933,7 @@ class Model:
         grp = self._pp_column_group()
         res = []
         for b, dec, out in zip(batches, decs, outs):
-            rows = b.num_seqs if b.logit_rows is not None or b.is_decode else b.ids.shape[0]
+            rows = b.logit_rows.numel() if b.logit_rows is not None else b.ids.shape[0]
             logits = out if last else torch.empty(rows, dec.v1 - dec.v0, dtype=torch.float32, device=ctx.device)
             dist.broadcast(logits, src, group=grp)
             res.append(logits)

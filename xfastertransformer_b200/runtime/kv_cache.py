@@ -10,6 +10,8 @@ reorder and prefix sharing physically copy rows (``kvcache_tensor.h:146-289``,
   parallel fp32 scale ``[num_blocks, kv_heads, block]`` — one scale per token·head exactly like
   the reference's int8 cache, ``kvcache_tensor.h:100-104``); MLA models keep a single latent pool
   ``[num_blocks, 1, block, kv_lora+rope]``.
+* layered designs give every pool its own ``(kv_heads, k_dim, v_dim)``; a layer that reads another layer's keys and
+  values has no pool at all (the decoder maps it to the pool it reads);
 * a sequence is a list of block ids; blocks are reference-counted so a shared prefix or a beam
   fork is a table copy, and beam reorder is a permutation of tables (no data moves unless the
   partially filled tail block must be split — copy-on-write).
@@ -19,7 +21,7 @@ implementation below is the same algorithm and the fallback.
 """
 from __future__ import annotations
 
-from typing import Dict, List, Optional, Sequence
+from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
@@ -131,14 +133,20 @@ class PrefixIndex:
 
 class PagedKVCache:
     def __init__(self, num_layers: int, kv_heads: int, k_dim: int, v_dim: int, dtype: str, device: torch.device,
-                 block_size: int = 64, act_dtype: torch.dtype = torch.bfloat16, latent: bool = False):
-        self.L, self.H, self.kd, self.vd = num_layers, kv_heads, k_dim, v_dim
+                 block_size: int = 64, act_dtype: torch.dtype = torch.bfloat16, latent: bool = False,
+                 geometry: Optional[Sequence[Tuple[int, int, int]]] = None, max_blocks: int = 0):
+        # (kv heads, key size, value size) of every pool
+        self.geometry = list(geometry) if geometry is not None else [(kv_heads, k_dim, v_dim)] * num_layers
+        self.L = len(self.geometry)
+        self.max_blocks = max_blocks             # > 0: the pools never grow past this many blocks
         self.block = block_size
         self.device = device
         self.latent = latent                     # MLA: single pool, no V
         self.int8 = dtype == "int8"
         if self.int8:
             self.dtype = torch.int8
+        elif dtype == "fp32":
+            self.dtype = torch.float32           # the 32-bit path
         elif dtype == "fp16" and act_dtype == torch.float16:
             self.dtype = torch.float16
         else:
@@ -159,21 +167,24 @@ class PagedKVCache:
     # -- capacity -------------------------------------------------------------------
     def bytes_per_block(self) -> int:
         e = torch.empty((), dtype=self.dtype).element_size()
-        per = self.H * self.block * self.kd * e + (0 if self.latent else self.H * self.block * self.vd * e)
-        if self.int8:
-            per += 2 * self.H * self.block * 4
-        return per * self.L
+        n = 0
+        for H, kd, vd in self.geometry:
+            n += H * self.block * (kd + (0 if self.latent else vd)) * e + (2 * H * self.block * 4 if self.int8 else 0)
+        return n
 
     def ensure_blocks(self, total: int) -> None:
         """Grow pools to hold `total` blocks (existing contents preserved)."""
         if total <= self.alloc.num_blocks:
             return
+        if self.max_blocks and total > self.max_blocks:
+            raise MemoryError(f"KV cache: {total} blocks needed, the pools are limited to {self.max_blocks}")
         old = self.alloc.num_blocks
-        mk = lambda d, dt=None: torch.zeros(total, self.H, self.block, d, dtype=dt or self.dtype, device=self.device)
+        mk = lambda H, d: torch.zeros(total, H, self.block, d, dtype=self.dtype, device=self.device)
         nk, nv, nks, nvs = [], [], [], []
         for l in range(self.L):
-            k = mk(self.kd)
-            v = None if self.latent else mk(self.vd)
+            H, kd, vd = self.geometry[l]
+            k = mk(H, kd)
+            v = None if self.latent else mk(H, vd)
             if old:
                 k[:old] = self.k[l]
                 if v is not None:
@@ -181,7 +192,7 @@ class PagedKVCache:
             nk.append(k)
             nv.append(v)
             if self.int8:
-                s1 = torch.zeros(total, self.H, self.block, dtype=torch.float32, device=self.device)
+                s1 = torch.zeros(total, H, self.block, dtype=torch.float32, device=self.device)
                 s2 = torch.zeros_like(s1)
                 if old:
                     s1[:old] = self.ks[l]
@@ -211,7 +222,8 @@ class PagedKVCache:
             if self.alloc.num_free >= extra_blocks:
                 return
         need = self.alloc.num_blocks - self.alloc.num_free + extra_blocks
-        self.ensure_blocks(max(need, int(self.alloc.num_blocks * 1.5)))
+        grow = int(self.alloc.num_blocks * 1.5)
+        self.ensure_blocks(max(need, min(grow, self.max_blocks) if self.max_blocks else grow))
 
     # -- sequences ------------------------------------------------------------------
     def add_sequence(self, seq_id: int, max_len: int = 0) -> None:

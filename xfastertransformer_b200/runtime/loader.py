@@ -15,7 +15,9 @@ N(0, 0.02) on the device (synthetic benchmarks: no files needed beyond config.in
 """
 from __future__ import annotations
 
+import json
 import os
+import struct
 import zlib
 from dataclasses import dataclass, field
 from typing import Optional, Sequence, Tuple
@@ -312,3 +314,81 @@ class WeightSource:
             return make_linear(R.pack_nibbles(q), kind, scale=s, zero=z)
         dense = q.float() * s[:, None] + z[:, None]
         return make_linear(dense, kind)
+
+
+_ST = {"BF16": (np.uint16, torch.bfloat16), "F32": (np.float32, None), "F16": (np.float16, None),
+       "I32": (np.int32, None), "I64": (np.int64, None), "I8": (np.int8, None), "U8": (np.uint8, None)}
+
+
+class SafetensorsFile:
+    """A memory-mapped ``.safetensors`` file: 8-byte little-endian header length, a JSON header (name -> dtype, shape,
+    data_offsets), then the data.  Shapes and extents are checked before anything is read."""
+
+    def __init__(self, path: str):
+        self.path = path
+        size = os.path.getsize(path)
+        with open(path, "rb") as f:
+            raw = f.read(8)
+            n = struct.unpack("<Q", raw)[0] if len(raw) == 8 else size
+            if 8 + n > size:
+                raise ValueError(f"{path}: truncated header")
+            head = json.loads(f.read(n))
+        self.base = 8 + n
+        self.entries = {k: v for k, v in head.items() if k != "__metadata__"}
+        self.mm = np.memmap(path, dtype=np.uint8, mode="r")
+        for k, e in self.entries.items():
+            if e["dtype"] not in _ST:
+                raise ValueError(f"{path}: tensor {k} has unsupported type {e['dtype']}")
+            a, b = e["data_offsets"]
+            want = int(np.prod(e["shape"], dtype=np.int64)) * np.dtype(_ST[e["dtype"]][0]).itemsize
+            if b - a != want or a < 0 or self.base + b > size:
+                raise ValueError(f"{path}: tensor {k} does not fit its extent")
+
+    def __contains__(self, name: str) -> bool:
+        return name in self.entries
+
+    def read(self, name: str, shape: Sequence[int], rows: Optional[Tuple[int, int]] = None,
+             cols: Optional[Tuple[int, int]] = None) -> torch.Tensor:
+        """The [rows, cols] slice of a tensor that must have `shape`."""
+        if name not in self.entries:
+            raise KeyError(f"{self.path}: no tensor {name}")
+        e = self.entries[name]
+        if tuple(e["shape"]) != tuple(shape):
+            raise ValueError(f"{self.path}: {name} has shape {tuple(e['shape'])}, expected {tuple(shape)}")
+        np_dt, view = _ST[e["dtype"]]
+        a, b = e["data_offsets"]
+        x = np.frombuffer(self.mm[self.base + a:self.base + b].tobytes(), dtype=np_dt).reshape(shape) \
+            if (self.base + a) % np.dtype(np_dt).itemsize else \
+            self.mm[self.base + a:self.base + b].view(np_dt).reshape(shape)
+        if rows is not None:
+            x = x[rows[0]:rows[1]]
+        if cols is not None:
+            x = x[..., cols[0]:cols[1]]
+        t = torch.from_numpy(np.array(x))
+        return t.view(view) if view is not None else t
+
+
+class SafetensorsSource(WeightSource):
+    """`WeightSource` over ``model.safetensors`` (linear weights stored [out, in]); fake mode works as there."""
+
+    def __init__(self, path: str, device: torch.device, fake: Optional[int] = None, seed: int = 0):
+        super().__init__(path, "bf16", device, fake, seed)
+        self.file = None if self.fake else SafetensorsFile(os.path.join(path, "model.safetensors"))
+
+    def exists(self, name: str) -> bool:
+        return False if self.fake else name in self.file
+
+    def _take(self, name, shape, rows=None, cols=None) -> torch.Tensor:
+        t = self.file.read(name, shape, rows, cols)
+        self.loaded_bytes += t.numel() * t.element_size()
+        return t.to(self.device)
+
+    def vector(self, name, n, dtype=None, out_dtype=torch.float32, rng=None, fake_ones=False):
+        if self.fake:
+            return super().vector(name, n, dtype, out_dtype, rng, fake_ones)
+        return self._take(name, (n,), rows=rng).to(out_dtype)
+
+    def matrix(self, name, shape, dtype=None, rows=None, cols=None):
+        if self.fake:
+            return super().matrix(name, shape, dtype, rows, cols)
+        return self._take(name, shape, rows, cols)

@@ -68,6 +68,7 @@ class SequenceMeta:
     group: int = -1                   # request index for beams
     prefix_len: int = 0               # tokens inherited from a shared prefix
     owner: int = 0                    # data-parallel attention: the rank that holds this sequence's KV cache
+    rows: Optional[List[int]] = None  # which of the pending tokens' logits the next forward returns (None: the last one)
 
     @property
     def total_len(self) -> int:
