@@ -1,0 +1,214 @@
+"""Scenarios of the layered decoder, run on CPU by test_layered_cpu.py and on a GPU by test_layered_gpu.py: the engine
+against tests/oracle_layered.py.  Every function takes the dtype it runs the engine in; `tolerance` says how far logits
+may be from the fp64 result (root mean square over the vocabulary, mean taken off, relative to the logits' spread)."""
+import random
+
+import torch
+
+import oracle_layered as O
+import xfastertransformer_b200 as xft
+from xfastertransformer_b200.tools.trace_run import TraceRunner
+
+YARN = {"factor": 3.0, "original": 96, "fast": 12.0, "slow": 1.0}
+
+# name -> config; none of the sizes repeat within a config unless that is the point
+CONFIGS = {
+    # unequal layers: heads, sizes, windows, rotation, a layer without feed-forward, one that reads another's keys
+    "unequal": O.config([
+        O.attention_layer(heads=6, kv_heads=3, dim=20, vdim=36, size=17, keep=3, rot_dims=12, scaling=YARN, softcap=9.0,
+                          ff=70),
+        O.attention_layer(heads=4, kv_heads=4, dim=48, vdim=24, size=70, keep=1, rot_dims=48, base=500.0, softcap=25.0,
+                          ff=None),
+        O.attention_layer(heads=6, kv_heads=3, dim=20, vdim=36, size=33, keep=6, rot_dims=12, scaling=YARN, softcap=4.0,
+                          scale=0.31, kv_from=0, ff=104)], width=90, vocab=131, eps=3e-4),
+    # head size 128: the tensor-core prompt kernel and the fused QKV epilogue; windows off the 64-token pages
+    "heads128": O.config([
+        O.attention_layer(heads=6, kv_heads=2, dim=128, vdim=128, size=100, keep=5, rot_dims=64, scaling=YARN,
+                          softcap=20.0, ff=200),
+        O.attention_layer(heads=6, kv_heads=2, dim=128, vdim=128, size=65, keep=2, rot_dims=64, scaling=YARN,
+                          softcap=20.0, kv_from=0, ff=136)], width=160, vocab=300),
+    # sizes between the kernels' head sizes, keys longer than values
+    "padded": O.config([
+        O.attention_layer(heads=5, kv_heads=1, dim=112, vdim=80, size=64, keep=64, rot_dims=16, softcap=15.0, ff=88),
+        O.attention_layer(heads=2, kv_heads=2, dim=160, vdim=200, size=1, keep=4, rot_dims=160, base=77.0, softcap=8.0,
+                          ff=64)], width=104, vocab=97),
+    # larger than any tensor-core attention kernel takes
+    "large_heads": O.config([
+        O.attention_layer(heads=2, kv_heads=1, dim=264, vdim=304, size=30, keep=2, rot_dims=32, softcap=12.0, ff=72)],
+        width=64, vocab=83),
+    # mechanisms left out one by one: no cap, no window, no rotation, no scaling, nothing kept, a window past the end
+    "bare": O.config([
+        O.attention_layer(heads=4, kv_heads=2, dim=32, vdim=32, softcap=None, mask=False, rot=False, ff=48),
+        O.attention_layer(heads=3, kv_heads=1, dim=64, vdim=64, softcap=None, size=21, keep=0, rot_dims=64, ff=40),
+        O.attention_layer(heads=3, kv_heads=3, dim=16, vdim=8, size=5000, keep=2, rot_dims=2, softcap=2.0, ff=24),
+        O.attention_layer(heads=4, kv_heads=2, dim=32, vdim=32, softcap=6.0, mask=False, rot=False, kv_from=0, ff=56)],
+        width=72, vocab=150),
+    # two layers that read the same keys, each with a window of its own, wider and narrower than the owner's
+    "shared": O.config([
+        O.attention_layer(heads=4, kv_heads=2, dim=64, vdim=64, size=24, keep=4, rot_dims=20, softcap=11.0, ff=96),
+        O.attention_layer(heads=8, kv_heads=1, dim=64, vdim=64, size=40, keep=0, rot_dims=64, softcap=13.0, ff=96),
+        O.attention_layer(heads=4, kv_heads=2, dim=64, vdim=64, size=90, keep=9, rot_dims=20, softcap=11.0, kv_from=0,
+                          ff=None),
+        O.attention_layer(heads=8, kv_heads=1, dim=64, vdim=64, size=7, keep=1, rot_dims=64, softcap=13.0, kv_from=1,
+                          ff=32)], width=128, vocab=220),
+}
+
+TOLERANCE = {"fp32": 3e-5, "bf16": 0.05}
+
+
+def tolerance(dtype):
+    return TOLERANCE[dtype]
+
+
+class Case:
+    """A checkpoint on disk, its weights, and the oracle's logits of prompts (computed once)."""
+
+    def __init__(self, root, name):
+        self.name, self.cfg = name, CONFIGS[name]
+        self.W = O.random_weights(self.cfg, seed=sum(map(ord, name)))
+        self.path = O.write_checkpoint(str(root / name), self.cfg, self.W)
+        self._want = {}
+
+    def tokens(self, n, seed=0):
+        r = random.Random(seed * 1000 + n)
+        return [r.randrange(self.cfg["vocab"]) for _ in range(n)]
+
+    def want(self, tokens):
+        key = tuple(tokens)
+        if key not in self._want:
+            self._want[key] = O.forward(self.cfg, self.W, list(tokens))
+        return self._want[key]
+
+
+def error(got, want):
+    """Per row: rms difference over the vocabulary (means taken off) over the spread of the wanted logits."""
+    d = got.double().cpu() - want
+    d = d - d.mean(-1, keepdim=True)
+    return d.pow(2).mean(-1).sqrt() / float((want - want.mean(-1, keepdim=True)).pow(2).mean().sqrt())
+
+
+def check(got, want, dtype, what=""):
+    assert got.shape == want.shape, (got.shape, want.shape)
+    e = error(got, want)
+    bad = int(e.argmax())
+    assert bool((e <= tolerance(dtype)).all()), f"{what}: row {bad} of {len(e)} is off by {float(e[bad]):.3g}"
+
+
+def cuts(n, sizes):
+    """Portions of a prompt of n tokens, cycling through `sizes`."""
+    out, at, i = [], 0, 0
+    while at < n:
+        s = min(sizes[i % len(sizes)], n - at)
+        out.append((at, at + s))
+        at += s
+        i += 1
+    return out
+
+
+def run_portions(runner, rid, tokens, portions):
+    """All positions' logits of one request fed in portions."""
+    rows = []
+    for k, (a, b) in enumerate(portions):
+        last = k + 1 == len(portions)
+        rows.append(runner.step([{"id": rid, "tokens": tokens[a:b], "want": list(range(b - a))}], [rid] if last else []))
+    return torch.cat(rows)
+
+
+# ------------------------------------------------------------------------------------------ scenarios
+def whole_prompt(case, dtype, n):
+    toks = case.tokens(n)
+    m = xft.AutoModel.from_pretrained(case.path, dtype=dtype)
+    check(m([toks])[0], case.want(toks), dtype, f"{case.name}: whole prompt of {n}")
+
+
+def first_tokens(case, dtype):
+    """Prompts of 1, 2, 3 ... tokens in one ragged batch."""
+    prompts = [case.tokens(n, 5) for n in (1, 2, 3, 5, 9)]
+    m = xft.AutoModel.from_pretrained(case.path, dtype=dtype)
+    got = m(prompts)
+    check(got, torch.cat([case.want(p) for p in prompts]), dtype, f"{case.name}: first tokens")
+
+
+def token_by_token(case, dtype, n, start=1):
+    """A prompt, then single tokens through the cache, against the prompt in one piece."""
+    toks = case.tokens(n, 1)
+    r = TraceRunner(case.path, dtype, n)
+    got = run_portions(r, "a", toks, [(0, start)] + [(i, i + 1) for i in range(start, n)])
+    check(got, case.want(toks), dtype, f"{case.name}: token by token")
+
+
+def portions(case, dtype, n, sizes):
+    toks = case.tokens(n, 2)
+    r = TraceRunner(case.path, dtype, n)
+    check(run_portions(r, "a", toks, cuts(n, sizes)), case.want(toks), dtype, f"{case.name}: portions {sizes}")
+
+
+def mixed_batches(case, dtype, seed=0, lengths=(150, 97, 64, 30, 1, 129), live=3):
+    """Requests of unequal lengths in random portions — prompts' portions beside single tokens, some left out of a step —
+    over pools just large enough for those alive, so that freed blocks are used again (and are filled with large values
+    in between: a masked key must not leak)."""
+    r = random.Random(seed)
+    toks = {str(i): case.tokens(n, 10 + i) for i, n in enumerate(lengths)}
+    pages = lambda n: (n + 63) // 64 * 64
+    run = TraceRunner(case.path, dtype, sum(sorted((pages(n) for n in lengths), reverse=True)[:live]))
+    cache = run.model.model.cache
+    size = cache.alloc.num_blocks
+    at, got = {k: 0 for k in toks}, {k: [] for k in toks}
+    waiting, alive = list(toks), []
+    steps = 0
+    while waiting or alive:
+        while waiting and len(alive) < live:
+            alive.append(waiting.pop(0))
+        entries, end = [], []
+        for k in r.sample(alive, r.randint(1, len(alive))):
+            left = len(toks[k]) - at[k]
+            n = min(left, r.choice([1, 1, 2, 3, 7, 29, 64, 90]))
+            entries.append({"id": k, "tokens": toks[k][at[k]:at[k] + n], "want": list(range(n))})
+            at[k] += n
+            if n == left:
+                end.append(k)
+        rows = run.step(entries, end)
+        for e in entries:
+            n = len(e["tokens"])
+            got[e["id"]].append(rows[:n])
+            rows = rows[n:]
+        for k in end:
+            alive.remove(k)
+        for b in cache.alloc.free:                       # what freed pages hold must not matter
+            for pool in (cache.k, cache.v):
+                for t in pool:
+                    t[b].fill_(30.0)
+        steps += 1
+    assert cache.alloc.num_blocks == size and not cache.tables, "pools grew or requests were left behind"
+    for k, rows in got.items():
+        check(torch.cat(rows), case.want(toks[k]), dtype, f"{case.name}: request {k} of {len(toks[k])} tokens")
+    return steps
+
+
+def greedy(case, dtype, n_prompt, n_new):
+    """generate() on a batch of unequal prompts (through the engine's batching, decode runner and sampler): each emitted
+    token is the best one, up to rounding, given everything before it."""
+    prompts = [case.tokens(n_prompt, 30), case.tokens(n_prompt, 31)]
+    m = xft.AutoModel.from_pretrained(case.path, dtype=dtype)
+    out = m.generate(torch.tensor(prompts), max_length=n_prompt + n_new).tolist()
+    for p, row in zip(prompts, out):
+        assert row[:n_prompt] == p and len(row) == n_prompt + n_new
+        w = case.want(row[:-1])[n_prompt - 1:]
+        spread = float((w - w.mean(-1, keepdim=True)).pow(2).mean().sqrt())
+        picked = w.gather(1, torch.tensor(row[n_prompt:])[:, None])[:, 0]
+        short = (w.max(-1).values - picked) / spread
+        assert float(short.max()) <= (1e-4 if dtype == "fp32" else 6 * tolerance(dtype)), f"a worse token by {float(short.max())}"
+    return out
+
+
+def rows_and_order(case, dtype):
+    """`want` may be empty, partial or out of order; a step in which nothing is wanted still fills the cache."""
+    a, b = case.tokens(40, 3), case.tokens(25, 4)
+    r = TraceRunner(case.path, dtype, 192)
+    assert r.step([{"id": "a", "tokens": a[:17], "want": []}]).shape == (0, case.cfg["vocab"])
+    got = r.step([{"id": "b", "tokens": b, "want": [24, 0, 7]}, {"id": "a", "tokens": a[17:30], "want": [12]}], ["b"])
+    wa, wb = case.want(a), case.want(b)
+    check(got, torch.stack([wb[24], wb[0], wb[7], wa[29]]), dtype, "rows")
+    got = r.step([{"id": "a", "tokens": a[30:], "want": [3, 9]}], ["a"])
+    check(got, torch.stack([wa[33], wa[39]]), dtype, "rows of a later portion")
+    assert not r.model.model.cache.tables

@@ -48,13 +48,13 @@ def rotate(x, positions, rot):
     f, m = rotary_frequencies(rot)
     half = rot["dims"] // 2
     y = x.clone()
-    for t, p in enumerate(positions):
-        for i in range(half):
-            a = p * f[i]
-            c, s = math.cos(a) * m, math.sin(a) * m
-            u, v = x[t, :, i].clone(), x[t, :, i + half].clone()
-            y[t, :, i] = u * c - v * s
-            y[t, :, i + half] = v * c + u * s
+    for i in range(half):
+        a = [p * f[i] for p in positions]
+        c = torch.tensor([math.cos(t) * m for t in a], dtype=x.dtype)[:, None]
+        s = torch.tensor([math.sin(t) * m for t in a], dtype=x.dtype)[:, None]
+        u, v = x[:, :, i], x[:, :, i + half]
+        y[:, :, i] = u * c - v * s
+        y[:, :, i + half] = v * c + u * s
     return y
 
 
@@ -67,11 +67,22 @@ def sees(i, j, mask):
     return i - j < mask["size"] or j < mask["keep_first"]
 
 
+_VISIBLE = {}
+
+
+def visible(T, mask):
+    """The table of `sees` for one sequence."""
+    key = (T, tuple(sorted(mask.items())) if mask else None)
+    if key not in _VISIBLE:
+        _VISIBLE[key] = torch.tensor([[sees(i, j, mask) for j in range(T)] for i in range(T)])
+    return _VISIBLE[key]
+
+
 def attention(q, k, v, scale, softcap, mask, sink):
     """q [T, H, d], k [T, G, d], v [T, G, dv] (already rotated) -> [T, H, dv]."""
     T, H, _ = q.shape
     G = k.shape[1]
-    vis = torch.tensor([[sees(i, j, mask) for j in range(T)] for i in range(T)])
+    vis = visible(T, mask)
     out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
     for h in range(H):
         g = h // (H // G)
