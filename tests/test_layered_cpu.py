@@ -1,7 +1,5 @@
 """Layered designs (Kafipel) on the CPU path: the engine, cache, batching and command-line tool against a plain
-implementation of the equations, and each mechanism of the op set alone."""
-import json
-import math
+implementation of the equations."""
 import os
 import subprocess
 import sys
@@ -15,11 +13,7 @@ sys.path.insert(0, os.path.join(ROOT, "tests"))
 import layered_cases as C  # noqa: E402
 import oracle_layered as O  # noqa: E402
 import xfastertransformer_b200 as xft  # noqa: E402
-from xfastertransformer_b200 import ops  # noqa: E402
 from xfastertransformer_b200.config import ModelConfig  # noqa: E402
-from xfastertransformer_b200.models.registry import decoder_class, family_for  # noqa: E402
-from xfastertransformer_b200.ops import reference as R  # noqa: E402
-from xfastertransformer_b200.runtime.loader import SafetensorsFile  # noqa: E402
 
 
 @pytest.fixture(autouse=True)

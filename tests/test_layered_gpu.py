@@ -1,0 +1,230 @@
+"""Layered designs (Kafipel) on a GPU: every kernel of the path alone, and whole models in bf16 and in 32 bits, against a
+plain implementation of the equations."""
+import os
+import sys
+
+import pytest
+import torch
+
+pytestmark = pytest.mark.gpu
+
+ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+sys.path.insert(0, os.path.join(ROOT, "tests"))
+
+import layered_cases as C  # noqa: E402
+import layered_ops_cases as M  # noqa: E402
+import oracle_layered as O  # noqa: E402
+import xfastertransformer_b200 as xft  # noqa: E402
+
+BF16_TOL = 1.2e-2                # a product of bf16 operands against fp64 on the same operands
+
+
+def _dev():
+    return torch.device("cuda", 0)
+
+
+@pytest.fixture(scope="module")
+def cases(tmp_path_factory):
+    root, made = tmp_path_factory.mktemp("layered"), {}
+
+    def get(name):
+        if name not in made:
+            made[name] = C.Case(root, name)
+        return made[name]
+    return get
+
+
+# ------------------------------------------------------------------------------------------ attention kernels
+@pytest.mark.parametrize("window,keep", [(40, 5), (64, 64), (1, 3), (129, 2), (33, 70)])
+@pytest.mark.parametrize("d,decode", [(64, False), (64, True), (128, False), (128, True), (256, False), (256, True)])
+def test_window_edges_bf16(d, decode, window, keep):
+    """mma.sync prompt kernels (64, 256), the tcgen05 prompt kernel (128), the TMA-ring decode kernel."""
+    M.window_edges(_dev(), torch.bfloat16, d, d, window, keep, decode, BF16_TOL)
+
+
+@pytest.mark.parametrize("window,keep", [(40, 5), (129, 2), (1, 0)])
+@pytest.mark.parametrize("d", [64, 128])
+def test_window_edges_cp_async_decode(d, window, keep, monkeypatch):
+    from xfastertransformer_b200.utils.flags import Env
+    monkeypatch.setenv("XFT_ATTN_TMA", "0")
+    Env.get().reload()
+    M.window_edges(_dev(), torch.bfloat16, d, d, window, keep, True, BF16_TOL)
+
+
+@pytest.mark.parametrize("splits", [2, 5])
+def test_window_edges_split_decode(splits, monkeypatch):
+    """Several CTAs per (sequence, head): the sink counts in one of them, the kept tiles may be another's."""
+    from xfastertransformer_b200.utils.flags import Env
+    monkeypatch.setenv("XFT_ATTN_SPLITS", str(splits))
+    Env.get().reload()
+    M.window_edges(_dev(), torch.bfloat16, 128, 128, 129, 2, True, BF16_TOL)
+    M.sink_counts_once(_dev(), torch.bfloat16, 128, BF16_TOL, T=330)
+
+
+def test_tc_prompt_kernel_off(monkeypatch):
+    from xfastertransformer_b200.utils.flags import Env
+    monkeypatch.setenv("XFT_ATTN_TC_MIN_Q", "1000000")
+    Env.get().reload()
+    M.window_edges(_dev(), torch.bfloat16, 128, 128, 40, 5, False, BF16_TOL)
+
+
+@pytest.mark.parametrize("window,keep", [(40, 5), (64, 64), (1, 0), (129, 2)])
+@pytest.mark.parametrize("decode", [False, True])
+@pytest.mark.parametrize("dtype,tol", [(torch.float32, 2e-6), (torch.bfloat16, 6e-3)])
+def test_window_edges_plain_kernel(dtype, tol, decode, window, keep):
+    M.window_edges(_dev(), dtype, 40, 24, window, keep, decode, tol)
+
+
+@pytest.mark.parametrize("d", [64, 128, 256])
+def test_sinks_and_cap_bf16(d):
+    M.sink_counts_once(_dev(), torch.bfloat16, d, BF16_TOL)
+    M.softcap(_dev(), torch.bfloat16, d, BF16_TOL)
+
+
+def test_sinks_and_cap_fp32():
+    M.sink_counts_once(_dev(), torch.float32, 36, 3e-6)
+    M.softcap(_dev(), torch.float32, 36, 3e-6)
+
+
+@pytest.mark.parametrize("d,pad", [(20, 64), (80, 128), (136, 256)])
+def test_padded_heads(d, pad):
+    for decode in (False, True):
+        M.window_edges(_dev(), torch.bfloat16, d, d - 4, 40, 5, decode, BF16_TOL, pad=pad)
+
+
+@pytest.mark.parametrize("group", [1, 6, 20])
+def test_group_sizes(group):
+    """More query heads per key/value head than one CTA's 16 rows."""
+    for decode in (False, True):
+        M.window_edges(_dev(), torch.bfloat16, 128, 128, 70, 3, decode, BF16_TOL, H=group * 2, G=2)
+
+
+def test_far_keys_among_many():
+    """One key thousands of positions back, inside a wide window or kept, found by prompt portions and decode steps."""
+    T = 2100
+    for window, keep, j in ((1900, 2, 250), (64, 130, 129), (64, 130, 130), (2000, 0, 99), (2000, 0, 101)):
+        q, k, v = M._inputs(T, 2, 1, 128, 128, torch.bfloat16, j)
+        q[..., 0], k[..., 0] = 3.0, 0.0
+        k[j, :, 0] = 8.0
+        sink = torch.tensor([0.5, -2.0])
+        want = O.attention(q.double(), k.double(), v.double(), 1.0, 50.0, {"size": window, "keep_first": keep}, sink.double())
+        for decode in (False, True):
+            got = M.attend(_dev(), torch.bfloat16, q, k, v, decode, T - 60, scale=1.0, softcap=50.0, window=window,
+                           keep_first=keep, sinks=sink.cuda())
+            M._close(got, want[T - 60:].float(), BF16_TOL, f"window {window}, kept {keep}, key {j}, decode {decode}")
+
+
+# ------------------------------------------------------------------------------------------ other kernels
+@pytest.mark.parametrize("H", [72, 100, 256, 1021, 1536, 3000, 5120, 12288, 20000])
+@pytest.mark.parametrize("kind", ["layer", "rms"])
+def test_residual_norm(H, kind):
+    M.residual_norm(_dev(), H, kind, torch.bfloat16, torch.bfloat16, 4e-6)
+    M.residual_norm(_dev(), H, kind, torch.float32, torch.float32, 4e-6)
+
+
+@pytest.mark.parametrize("T,N,K", [(1, 130, 77), (65, 64, 16), (200, 333, 1000)])
+def test_gemm_f32(T, N, K):
+    """True 32-bit products: a reduced-precision mode would be off by 1e-3."""
+    from xfastertransformer_b200.ops import native as N_
+    from xfastertransformer_b200.runtime.loader import make_linear
+    g = torch.Generator().manual_seed(N)
+    x, w = torch.randn(T, K, generator=g), torch.randn(2 * N, K, generator=g)
+    want = x.double() @ w.double().T
+    W = make_linear(w.cuda(), "fp32")
+    got = N_.linear(x.cuda(), W)
+    assert float((got.double().cpu() - want).abs().max() / want.abs().max()) < 2e-6
+    gate, up = want[:, :N], want[:, N:]
+    got = N_.linear_gated(x.cuda(), W, "silu")
+    ref = gate * torch.sigmoid(gate) * up
+    assert float((got.double().cpu() - ref).abs().max() / ref.abs().max()) < 2e-6
+
+
+@pytest.mark.parametrize("dtype,d,dv,tol", [(torch.float32, 40, 24, 2e-5), (torch.bfloat16, 264, 272, 8e-3), (torch.bfloat16, 64, 64, 8e-3)])
+def test_rotation(dtype, d, dv, tol):
+    M.rotation(_dev(), dtype, {"dims": 24, "base": 900.0, "scaling": {"factor": 3.0, "original": 50, "fast": 5.0, "slow": 0.5}},
+               d, dv, tol)
+
+
+# ------------------------------------------------------------------------------------------ whole models
+BOTH = pytest.mark.parametrize("dtype", ["fp32", "bf16"])
+
+
+@BOTH
+@pytest.mark.parametrize("name", sorted(C.CONFIGS))
+def test_whole_prompt(cases, name, dtype):
+    C.whole_prompt(cases(name), dtype, 140)
+
+
+@BOTH
+@pytest.mark.parametrize("name", ["unequal", "heads128"])
+def test_first_tokens(cases, name, dtype):
+    C.first_tokens(cases(name), dtype)
+
+
+@BOTH
+@pytest.mark.parametrize("name,start", [("unequal", 1), ("heads128", 40), ("padded", 70), ("shared", 1), ("bare", 100)])
+def test_token_by_token(cases, name, start, dtype):
+    C.token_by_token(cases(name), dtype, 140, start)
+
+
+@BOTH
+@pytest.mark.parametrize("sizes", [(2,), (3, 64, 1), (17, 29)])
+@pytest.mark.parametrize("name", ["unequal", "heads128"])
+def test_portions(cases, name, sizes, dtype):
+    C.portions(cases(name), dtype, 140, sizes)
+
+
+@BOTH
+@pytest.mark.parametrize("name", ["unequal", "heads128", "shared", "large_heads"])
+def test_mixed_batches_reuse_pages(cases, name, dtype):
+    assert C.mixed_batches(cases(name), dtype) > 8
+
+
+@BOTH
+@pytest.mark.parametrize("name", ["unequal", "heads128"])
+def test_rows_and_order(cases, name, dtype):
+    C.rows_and_order(cases(name), dtype)
+
+
+@BOTH
+@pytest.mark.parametrize("name", ["unequal", "heads128", "padded"])
+def test_greedy_generation(cases, name, dtype):
+    """generate(): the captured decode step (CUDA graph) included."""
+    C.greedy(cases(name), dtype, 20, 130)
+
+
+def test_graph_and_eager_steps_agree(cases, monkeypatch):
+    c = cases("heads128")
+    a = C.greedy(c, "bf16", 30, 60)
+    monkeypatch.setenv("XFT_CUDA_GRAPH", "0")
+    from xfastertransformer_b200.utils.flags import Env
+    Env.get().reload()
+    assert C.greedy(c, "bf16", 30, 60) == a
+
+
+@pytest.mark.parametrize("dtype,kv", [("int8", "bf16"), ("bf16", "int8")])
+def test_quantised_weights_and_cache(tmp_path, dtype, kv):
+    cfg = O.config([O.attention_layer(heads=4, kv_heads=2, dim=64, vdim=64, ff=128, size=30),
+                    O.attention_layer(heads=4, kv_heads=2, dim=64, vdim=64, ff=128, size=50, kv_from=0)], width=128, vocab=256)
+    W = O.random_weights(cfg)
+    p = O.write_checkpoint(str(tmp_path / "q"), cfg, W)
+    toks = [(7 * i) % 256 for i in range(90)]
+    want = O.forward(cfg, W, toks)
+    m = xft.AutoModel.from_pretrained(p, dtype=dtype, kv_cache_dtype=kv)
+    assert float((m([toks])[0].double().cpu() - want).pow(2).mean().sqrt() / want.std()) < 0.1
+    assert m.generate(torch.tensor([toks]), max_length=100).shape == (1, 100)
+
+
+def test_long_context_and_table_growth(tmp_path):
+    """A prompt past the first rotary table, and generation across its end."""
+    cfg = O.config([O.attention_layer(heads=2, kv_heads=1, dim=128, vdim=128, size=300, keep=3, rot_dims=32, ff=64)], width=64,
+                   vocab=90)
+    W = O.random_weights(cfg)
+    p = O.write_checkpoint(str(tmp_path / "long"), cfg, W)
+    toks = [(11 * i * i + i) % 90 for i in range(2300)]
+    m = xft.AutoModel.from_pretrained(p, dtype="bf16")
+    sid = m.set_input_cb([toks], max_length=2400, rows=[[0, 299, 2047, 2048, 2299]])
+    got = m.forward_cb()
+    m.free_seqs(sid)
+    C.check(got, O.forward(cfg, W, toks)[[0, 299, 2047, 2048, 2299]], "bf16", "long prompt")
+    assert m.generate(torch.tensor([toks[:2040]]), max_length=2060).shape == (1, 2060)

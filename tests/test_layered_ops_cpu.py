@@ -1,0 +1,216 @@
+"""Mechanisms of layered designs one by one, on the CPU path, with inputs in which a fault stands out; and the files such
+a model is read from."""
+import json
+import math
+import os
+import struct
+import subprocess
+import sys
+
+import pytest
+import torch
+
+ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+sys.path.insert(0, os.path.join(ROOT, "tests"))
+
+import layered_ops_cases as M  # noqa: E402
+import oracle_layered as O  # noqa: E402
+import xfastertransformer_b200 as xft  # noqa: E402
+from xfastertransformer_b200.config import ModelConfig  # noqa: E402
+from xfastertransformer_b200.models.registry import decoder_class, family_for  # noqa: E402
+from xfastertransformer_b200.ops import reference as R  # noqa: E402
+from xfastertransformer_b200.runtime.loader import SafetensorsFile, SafetensorsSource  # noqa: E402
+
+CPU = torch.device("cpu")
+
+
+@pytest.fixture(autouse=True)
+def _cpu(monkeypatch):
+    monkeypatch.setenv("XFT_ENGINE", "CPU")
+
+
+@pytest.mark.parametrize("window,keep", [(40, 5), (64, 64), (1, 0), (1, 3), (129, 2), (300, 1), (33, 70)])
+@pytest.mark.parametrize("decode", [False, True])
+def test_window_edges(window, keep, decode):
+    M.window_edges(CPU, torch.float32, 32, 32, window, keep, decode, 1e-5)
+
+
+def test_sink_counts_once():
+    M.sink_counts_once(CPU, torch.float32, 32, 1e-5)
+
+
+def test_softcap():
+    M.softcap(CPU, torch.float32, 32, 1e-5)
+
+
+@pytest.mark.parametrize("kind", ["layer", "rms"])
+def test_residual_norm(kind):
+    M.residual_norm(CPU, 77, kind, torch.float32, torch.float32, 2e-6)
+
+
+@pytest.mark.parametrize("rot", [{"dims": 24, "base": 1000.0},
+                                 {"dims": 16, "base": 50.0, "scaling": {"factor": 5.0, "original": 64, "fast": 6.0, "slow": 0.5}},
+                                 {"dims": 40, "base": 1e5, "scaling": {"factor": 2.5, "original": 4096, "fast": 40.0, "slow": 2.0}},
+                                 # the two ends of the ramp fall on one pair
+                                 {"dims": 8, "base": 1e6, "scaling": {"factor": 3.0, "original": 32, "fast": 4.0, "slow": 3.9}},
+                                 {"dims": 2, "base": 10.0, "scaling": {"factor": 7.0, "original": 10, "fast": 1.0, "slow": 1.0}}])
+def test_rotation(rot):
+    M.rotation(CPU, torch.float32, rot, 40, 24, 2e-5)
+
+
+def test_rotation_table_grows(tmp_path):
+    """Positions past the first table: it is made anew, longer, and the early rows stay what they were."""
+    cfg = O.config([O.attention_layer(size=9, rot_dims=8, base=31.0)], width=64, vocab=50)
+    p = O.write_checkpoint(str(tmp_path / "m"), cfg, O.random_weights(cfg))
+    d = xft.AutoModel.from_pretrained(p, dtype="fp32").model.decoder
+    rot = d.cfg.layers[0].mixer.rot
+    a = d._rope(rot, 0)
+    b = d._rope(rot, a.shape[0] + 1)
+    assert b.shape[0] >= 2 * a.shape[0] and torch.equal(b[:a.shape[0]], a)
+    f, _ = O.rotary_frequencies({"dims": 8, "base": 31.0})
+    assert abs(float(b[-1, 1]) - math.cos((b.shape[0] - 1) * f[1])) < 2e-4
+
+
+# ------------------------------------------------------------------------------------------ configuration
+def _write(tmp_path, cfg, name="m"):
+    return O.write_checkpoint(str(tmp_path / name), cfg, O.random_weights(cfg))
+
+
+def test_config_is_read_per_layer(tmp_path):
+    sc = {"factor": 2.5, "original": 77, "fast": 9.0, "slow": 0.7}
+    cfg = O.config([O.attention_layer(heads=6, kv_heads=3, dim=20, vdim=28, size=11, keep=2, rot_dims=10, scaling=sc, scale=0.3,
+                                      softcap=7.0, ff=44),
+                    O.attention_layer(heads=2, kv_heads=2, mask=False, rot=False, softcap=None, ff=None)], eps=2e-3)
+    c = ModelConfig.load(_write(tmp_path, cfg))
+    a, b = c.layers
+    assert (c.model_type, c.num_layer, c.hidden_size, c.vocab_size, c.layernorm_eps) == ("kafipel", 2, 96, 210, 2e-3)
+    assert (a.mixer.heads, a.mixer.kv_heads, a.mixer.dim, a.mixer.vdim, a.ff) == (6, 3, 20, 28, 44)
+    assert (a.mixer.window, a.mixer.keep_first, a.mixer.softcap, a.mixer.scale, a.mixer.kv_from) == (11, 2, 7.0, 0.3, -1)
+    r = a.mixer.rot
+    assert (r.dims, r.base, r.factor, r.original, r.fast, r.slow) == (10, 10000.0, 2.5, 77, 9.0, 0.7)
+    assert (b.mixer.window, b.mixer.softcap, b.mixer.rot, b.ff) == (0, 0.0, None, 0)
+    assert family_for(c).layered and decoder_class(c).__name__ == "LayeredDecoder"
+    c.to_ini(str(tmp_path / "again"))
+    assert ModelConfig.load(str(tmp_path / "again")).layers == c.layers
+
+
+@pytest.mark.parametrize("change,match", [
+    (lambda d: d.update(architecture="Other"), "unsupported architecture"),
+    (lambda d: d["layers"][1].update(type="convolution"), "unsupported mixer"),
+    (lambda d: d["layers"][1]["mlp"].update(kind="experts"), "unsupported feed-forward"),
+    (lambda d: d["layers"][1]["mixer"].update(kv_heads=3), "query heads over"),
+    (lambda d: d["layers"][1]["mixer"].update(kv_from=1), "not an earlier layer"),
+    (lambda d: d["layers"][1]["mixer"].update(kv_from=0, dim=16), "heads differ"),
+    (lambda d: d["layers"][1]["mixer"]["rot"].update(dims=34), "do not fit")])
+def test_config_faults(tmp_path, change, match):
+    cfg = O.config([O.attention_layer(), O.attention_layer()])
+    change(cfg)
+    os.makedirs(tmp_path / "m")
+    (tmp_path / "m" / "config.json").write_text(json.dumps(cfg))
+    with pytest.raises(ValueError, match=match):
+        ModelConfig.load(str(tmp_path / "m"))
+
+
+# ------------------------------------------------------------------------------------------ weights
+def test_safetensors_faults(tmp_path):
+    cfg = O.config([O.attention_layer()])
+    p = _write(tmp_path, cfg)
+    f = os.path.join(p, "model.safetensors")
+    st = SafetensorsFile(f)
+    W = O.random_weights(cfg)
+    assert torch.equal(st.read("l0.mix.q", (128, 96)), W["l0.mix.q"])
+    assert torch.equal(st.read("l0.mix.q", (128, 96), rows=(32, 64), cols=(3, 7)), W["l0.mix.q"][32:64, 3:7])
+    with pytest.raises(ValueError, match="expected"):
+        st.read("l0.mix.q", (96, 128))
+    with pytest.raises(KeyError):
+        st.read("l0.mix.z", (1,))
+    raw = open(f, "rb").read()
+    open(f, "wb").write(raw[:-2])
+    with pytest.raises(ValueError, match="extent"):
+        SafetensorsFile(f)
+    open(f, "wb").write(raw[:5])
+    with pytest.raises(ValueError, match="truncated"):
+        SafetensorsFile(f)
+    with pytest.raises(FileNotFoundError):
+        SafetensorsSource(str(tmp_path), CPU)
+
+
+def test_safetensors_types_and_odd_offsets(tmp_path):
+    """fp32, int32 and bf16 tensors, one of them at an odd offset."""
+    a = torch.arange(6, dtype=torch.int32).view(2, 3)
+    b = torch.randn(3)
+    c = torch.randn(5).bfloat16()
+    parts = [("u", "U8", [1], b"\x07"), ("a", "I32", [2, 3], a.numpy().tobytes()), ("b", "F32", [3], b.numpy().tobytes()),
+             ("c", "BF16", [5], c.view(torch.int16).numpy().tobytes())]
+    head, off = {"__metadata__": {"x": "y"}}, 0
+    for n, dt, sh, raw in parts:
+        head[n] = {"dtype": dt, "shape": sh, "data_offsets": [off, off + len(raw)]}
+        off += len(raw)
+    h = json.dumps(head).encode()
+    f = tmp_path / "t.safetensors"
+    f.write_bytes(struct.pack("<Q", len(h)) + h + b"".join(x[3] for x in parts))
+    st = SafetensorsFile(str(f))
+    assert torch.equal(st.read("a", (2, 3)), a) and torch.equal(st.read("b", (3,)), b) and torch.equal(st.read("c", (5,)), c)
+
+
+# ------------------------------------------------------------------------------------------ limits and refusals
+def test_fixed_pools_refuse_what_does_not_fit(tmp_path):
+    cfg = O.config([O.attention_layer(), O.attention_layer(kv_from=0, size=5)])
+    m = xft.AutoModel.from_pretrained(_write(tmp_path, cfg), dtype="fp32", max_cache_tokens=130)
+    cache = m.model.cache
+    assert cache.alloc.num_blocks == 3 and len(cache.k) == 1              # two layers, one pool
+    m.set_input_cb([[1] * 100], max_length=1 << 30, on_demand=True)
+    m.forward_cb()
+    m.set_input_cb([[1] * 100], max_length=1 << 30, on_demand=True)
+    with pytest.raises(MemoryError, match="limited to 3"):
+        m.forward_cb()
+    with pytest.raises(MemoryError):
+        m.set_input_cb([[1] * 10], max_length=500)
+
+
+def test_refusals(tmp_path):
+    cfg = O.config([O.attention_layer()])
+    p = _write(tmp_path, cfg)
+    with pytest.raises(ValueError, match="fp32"):
+        xft.AutoModel.from_pretrained(p, dtype="fp32", kv_cache_dtype="int8")
+    m = xft.AutoModel.from_pretrained(p, dtype="fp32")
+    with pytest.raises(ValueError, match="outside"):
+        m.set_input_cb([[1, 2, 3]], max_length=8, rows=[[3]])
+    with pytest.raises(ValueError, match="one list of rows"):
+        m.set_input_cb([[1, 2, 3]], max_length=8, rows=[[0], [1]])
+
+
+@pytest.mark.parametrize("dtype,kv,tol", [("int8", "bf16", 0.1), ("bf16_int8", "fp16", 0.1), ("bf16", "int8", 0.1)])
+def test_other_weight_and_cache_types(tmp_path, dtype, kv, tol):
+    """Quantised weights, hybrid types and an int8 cache go the way they go for the other families."""
+    cfg = O.config([O.attention_layer(), O.attention_layer(kv_from=0, size=7)])
+    W = O.random_weights(cfg)
+    p = O.write_checkpoint(str(tmp_path / "q"), cfg, W)
+    toks = list(range(3, 43))
+    m = xft.AutoModel.from_pretrained(p, dtype=dtype, kv_cache_dtype=kv)
+    want = O.forward(cfg, W, toks)
+    got = m([toks])[0].double()
+    assert float((got - want).pow(2).mean().sqrt() / want.std()) < tol
+    assert m.generate(torch.tensor([toks]), max_length=50).shape == (1, 50)
+
+
+def test_command_line(tmp_path):
+    """bin/trace_run as a program: JSON lines in, files of fp32 logits and a line per step out."""
+    cfg = O.config([O.attention_layer(), O.attention_layer(kv_from=0, size=7)], vocab=61)
+    W = O.random_weights(cfg)
+    p, out = O.write_checkpoint(str(tmp_path / "m"), cfg, W), tmp_path / "out"
+    out.mkdir()
+    a, b = list(range(40)), list(range(60, 40, -1))
+    steps = [{"step": 0, "entries": [{"id": "x", "tokens": a[:30], "want": []}], "end": []},
+             {"step": 1, "entries": [{"id": "y", "tokens": b, "want": [19, 2]}, {"id": "x", "tokens": a[30:31], "want": [0]}], "end": ["y"]},
+             {"step": 2, "entries": [{"id": "x", "tokens": a[31:], "want": [8]}], "end": ["x"]}]
+    r = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", p, "--dtype", "float32", "--out", str(out),
+                        "--max-tokens", "128"], input="\n".join(map(json.dumps, steps)) + "\n", text=True, capture_output=True,
+                       env=dict(os.environ, XFT_ENGINE="CPU"), timeout=240)
+    assert r.returncode == 0, r.stderr[-2000:]
+    assert [x for x in r.stdout.splitlines() if x.startswith("done")] == ["done 0", "done 1", "done 2"]
+    assert sorted(os.listdir(out)) == ["1.f32", "2.f32"]
+    wa, wb = O.forward(cfg, W, a), O.forward(cfg, W, b)
+    for name, want in (("1.f32", torch.stack([wb[19], wb[2], wa[30]])), ("2.f32", wa[39:40])):
+        got = torch.frombuffer(bytearray((out / name).read_bytes()), dtype=torch.float32).view(-1, 61)
+        assert torch.allclose(got.double(), want, atol=2e-4)
