@@ -128,10 +128,16 @@ def main():
     ap.add_argument("--input-len", type=int, default=2048)
     ap.add_argument("--dtype", default="bf16")
     ap.add_argument("--kv-dtype", default="bf16")
+    ap.add_argument("--design", default="", choices=["", "kafipel"],
+                    help="instead of the headline workload: this layered design beside Llama at equal sizes (one GPU)")
+    ap.add_argument("--size", default="all", choices=["all", "1b", "8b", "70b-layers"], help="with --design")
     ap.add_argument("--layers", type=int, default=0, help="debug only: fewer layers (result is flagged invalid)")
     args = ap.parse_args()
     if args.impl == "reference":
         return run_reference(args)
+    if args.design:
+        from benchmarks.bench_layered import run
+        return run(args, _clock_sampler, _clock_summary, ROOT)
     if args.warmup < 3:
         args.warmup = 3
 
