@@ -175,6 +175,7 @@ def kernels(s, peaks):
     attention(L, L, 4, 0, False)
     attention(L, L, 4, 0, True)
     attention(L, L, 4, 1024, True)
+    attention(1, 1088, B, 0, False)          # as many keys as a decode step sees through the window
     for ctx in (L, 8192):
         attention(1, ctx, B, 0, False)
         attention(1, ctx, B, 0, True)

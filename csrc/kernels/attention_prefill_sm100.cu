@@ -41,7 +41,7 @@ struct PrefillAttnParams {
   int bs;                     // tokens per cache block (64)
   float scale_log2;           // softmax scale * log2(e)
   // EXT only
-  float cap_log2, inv_cap2;   // softcap * log2(e), 2 log2(e) * scale / softcap (cap_log2 0: no cap)
+  float cap_log2, inv_cap;    // softcap * log2(e), scale / softcap (cap_log2 0: no cap)
   int window, keep;           // keys within `window` positions and the first `keep` are visible (window 2^30: all)
   const float* sinks;         // [hq] or null
   int num_blocks;
@@ -77,9 +77,22 @@ constexpr int kPfHalf = kPfTile * 128;       // bytes of one 64-feature half of 
 constexpr int kPfTileBytes = 2 * kPfHalf;    // 32 KB: Q, P, and each K / V stage
 constexpr int kPfSmem = kPfTileBytes * 6 + 1024;   // Q, P, K x 2, V x 2
 
-// Capped score in log2 units: cap * tanh(raw * scale / cap) with tanh(x) = 1 - 2 / (1 + exp(2x)).
+// Capped score in log2 units, cap * tanh(z) with z = raw * scale / cap: tanh(z) = 1 - 2 / (1 + exp(2z)).
 __device__ __forceinline__ float capped_log2(const PrefillAttnParams& p, float raw) {
-  return p.cap_log2 - __fdividef(2.f * p.cap_log2, 1.f + exp2f(fminf(raw * p.inv_cap2, 120.f)));
+  return p.cap_log2 - __fdividef(2.f * p.cap_log2, 1.f + exp2f(fminf(raw * p.inv_cap * 2.8853900817779268f, 120.f)));
+}
+// The same for |z| <= 1 without the special-function unit: tanh(z) / z as a polynomial in z^2, fitted with minimax
+// weights on [0, 1] (relative error below 2e-7, the size of the rounding).
+__device__ __forceinline__ float capped_log2_small(const PrefillAttnParams& p, float raw) {
+  const float z = raw * p.inv_cap, t = z * z;
+  float q = 0.0010410224785f;
+  q = fmaf(q, t, -0.0062033790164f);
+  q = fmaf(q, t, 0.020289981738f);
+  q = fmaf(q, t, -0.053457029164f);
+  q = fmaf(q, t, 0.13325203957f);
+  q = fmaf(q, t, -0.33332839608f);
+  q = fmaf(q, t, 0.99999994040f);
+  return z * p.cap_log2 * q;
 }
 
 template <bool EXT>
@@ -246,14 +259,35 @@ __global__ void __launch_bounds__(192, 1) attn_prefill_tc_kernel(const __grid_co
       auto visible = [&](int i) { return i < nvalid && (!EXT || i >= first || i < kept); };
       // pass 1: row maximum of the visible scores
       float mx = EXT ? -INFINITY : m;
+      float big = 0.f;                                       // EXT: largest |raw score| of the row
+      // EXT: which of the four 32-key chunks hold no key visible to any row of this warp, and which only visible ones
+      uint32_t none = 0, whole = 0;
+      if (EXT) {
+#pragma unroll
+        for (int c = 0; c < 128; c += 32) {
+          if (__all_sync(0xffffffffu, nvalid <= c || (first >= c + 32 && kept <= c))) none |= 1u << (c >> 5);
+          if (__all_sync(0xffffffffu, nvalid >= c + 32 && (first <= c || kept >= c + 32))) whole |= 1u << (c >> 5);
+        }
+      }
 #pragma unroll 1
       for (int c = 0; c < 128; c += 32) {
+        if (EXT && (none >> (c >> 5) & 1)) continue;
         uint32_t v[32];
         tmem_ld32(sa + c, v);
         tmem_ld_wait();
+        if (EXT && (whole >> (c >> 5) & 1)) {
 #pragma unroll
-        for (int i = 0; i < 32; ++i)
-          if (visible(c + i)) mx = fmaxf(mx, EXT ? __uint_as_float(v[i]) : __uint_as_float(v[i]) * p.scale_log2);
+          for (int i = 0; i < 32; ++i) {
+            mx = fmaxf(mx, __uint_as_float(v[i]));
+            big = fmaxf(big, fabsf(__uint_as_float(v[i])));
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            if (visible(c + i)) mx = fmaxf(mx, EXT ? __uint_as_float(v[i]) : __uint_as_float(v[i]) * p.scale_log2);
+            if (EXT) big = fmaxf(big, fabsf(__uint_as_float(v[i])));
+          }
+        }
       }
       // EXT: the maximum was taken over the raw scores (the cap is increasing); m = -inf: nothing visible so far
       if (EXT) mx = fmaxf(m, mx == -INFINITY ? -INFINITY : p.cap_log2 > 0.f ? capped_log2(p, mx) : mx * p.scale_log2);
@@ -262,31 +296,49 @@ __global__ void __launch_bounds__(192, 1) attn_prefill_tc_kernel(const __grid_co
       m = mx;
       // pass 2: P = exp2(s - m) as bf16 into the swizzled K-major tile, row sum
       float sum = 0.f;
+      auto weights = [&](auto score) {
 #pragma unroll 1
-      for (int c = 0; c < 128; c += 32) {
-        uint32_t v[32];
-        tmem_ld32(sa + c, v);
-        tmem_ld_wait();
-        uint8_t* prow = sP + (c >> 6) * kPfHalf + r * 128;
+        for (int c = 0; c < 128; c += 32) {
+          uint8_t* prow = sP + (c >> 6) * kPfHalf + r * 128;
+          const int chunk0 = (c & 63) >> 3;                  // 16-byte chunk of the 128-byte row
+          if (EXT && (none >> (c >> 5) & 1)) {
 #pragma unroll
-        for (int g8 = 0; g8 < 4; ++g8) {
-          uint32_t w[4];
-#pragma unroll
-          for (int i = 0; i < 4; ++i) {
-            const int e = g8 * 8 + 2 * i;
-            float s0 = __uint_as_float(v[e]), s1 = __uint_as_float(v[e + 1]);
-            if (EXT && p.cap_log2 > 0.f) { s0 = capped_log2(p, s0); s1 = capped_log2(p, s1); }
-            else { s0 *= p.scale_log2; s1 *= p.scale_log2; }
-            const float p0 = visible(c + e) ? exp2f(s0 - m) : 0.f;
-            const float p1 = visible(c + e + 1) ? exp2f(s1 - m) : 0.f;
-            const __nv_bfloat162 pb = __floats2bfloat162_rn(p0, p1);
-            // the sum uses the rounded values, as the product does
-            sum += __low2float(pb) + __high2float(pb);
-            w[i] = *reinterpret_cast<const uint32_t*>(&pb);
+            for (int g8 = 0; g8 < 4; ++g8)
+              *reinterpret_cast<uint4*>(prow + (((chunk0 + g8) ^ (r & 7)) << 4)) = make_uint4(0, 0, 0, 0);
+            continue;
           }
-          const int chunk = ((c & 63) >> 3) + g8;            // 16-byte chunk of the 128-byte row
-          *reinterpret_cast<uint4*>(prow + ((chunk ^ (r & 7)) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
+          uint32_t v[32];
+          tmem_ld32(sa + c, v);
+          tmem_ld_wait();
+          auto store = [&](auto seen) {
+#pragma unroll
+            for (int g8 = 0; g8 < 4; ++g8) {
+              uint32_t w[4];
+#pragma unroll
+              for (int i = 0; i < 4; ++i) {
+                const int e = g8 * 8 + 2 * i;
+                const float p0 = seen(c + e) ? exp2f(score(__uint_as_float(v[e])) - m) : 0.f;
+                const float p1 = seen(c + e + 1) ? exp2f(score(__uint_as_float(v[e + 1])) - m) : 0.f;
+                const __nv_bfloat162 pb = __floats2bfloat162_rn(p0, p1);
+                // the sum uses the rounded values, as the product does
+                sum += __low2float(pb) + __high2float(pb);
+                w[i] = *reinterpret_cast<const uint32_t*>(&pb);
+              }
+              *reinterpret_cast<uint4*>(prow + (((chunk0 + g8) ^ (r & 7)) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
+            }
+          };
+          if (EXT && (whole >> (c >> 5) & 1)) store([](int) { return true; });
+          else store(visible);
         }
+      };
+      auto plain = [&](float x) { return x * p.scale_log2; };
+      if (EXT && p.cap_log2 > 0.f) {
+        if (__all_sync(0xffffffffu, big * fabsf(p.inv_cap) <= 1.f))
+          weights([&](float x) { return capped_log2_small(p, x); });
+        else
+          weights([&](float x) { return capped_log2(p, x); });
+      } else {
+        weights(plain);
       }
       l = l * alpha + sum;
       // P is complete: make the generic-proxy stores visible to the tensor core, then tell the MMA warp
@@ -352,7 +404,7 @@ extern "C" int xft_attn_prefill_tc(const void* q, void* out, const void* kc, con
   const bool ext = softcap > 0.f || window > 0 || sinks;
   p.window = window > 0 ? min(window, 1 << 30) : 1 << 30; p.keep = window > 0 ? keep : 0; p.sinks = sinks;
   p.cap_log2 = softcap * 1.4426950408889634f;
-  p.inv_cap2 = softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f;
+  p.inv_cap = softcap > 0.f ? scale / softcap : 0.f;
   CUtensorMap tmQ, tmK, tmV;
   const uint64_t rows = (uint64_t)num_blocks * hkv * bs;
   int r = make_tensor_map(&tmQ, q, (uint64_t)T, (uint64_t)hq * 128, (uint64_t)hq * 128, 128, 2);

@@ -79,9 +79,9 @@ __device__ __forceinline__ void store8(bf16* p, const float (&v)[8]) {
 }
 
 // in-place norm of the CTA's row; columns from H on become zero
-template <int NT, int CH>
+template <int NT, int CH, bool PRE>
 __device__ __forceinline__ void norm_row(float (&v)[CH][8], const ResidualNormParams& p, const float* w, const float* b,
-                                         float* sh) {
+                                         const float (&pre)[PRE ? CH : 1][8], float* sh) {
   float mean = 0.f;
   if (!p.rms) {
     float s = 0.f;
@@ -107,9 +107,9 @@ __device__ __forceinline__ void norm_row(float (&v)[CH][8], const ResidualNormPa
     const int i = (threadIdx.x + c * NT) * 8;
     if (i < p.H) {
       float g[8];
-      load8(w + i, p.H - i, g);
+      if (!PRE) load8(w + i, p.H - i, g);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) v[c][j] *= inv * g[j];
+      for (int j = 0; j < 8; ++j) v[c][j] *= inv * (PRE ? pre[PRE ? c : 0][j] : g[j]);
       if (b) {
         load8(b + i, p.H - i, g);
 #pragma unroll
@@ -119,10 +119,20 @@ __device__ __forceinline__ void norm_row(float (&v)[CH][8], const ResidualNormPa
   }
 }
 
-template <int NT, int CH>
+// PRE: the gains, which are weights, are read before the kernel in front has finished (few rows: latency counts)
+template <int NT, int CH, bool PRE>
 __global__ void __launch_bounds__(NT) residual_norm_kernel(const ResidualNormParams p) {
   __shared__ float sh[4][NT / 32 > 0 ? NT / 32 : 1];
   grid_dep_launch();
+  float g1[PRE ? CH : 1][8], g2[PRE ? CH : 1][8];
+  if (PRE) {
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+      const int i = (threadIdx.x + c * NT) * 8, left = p.H - i;
+      if (p.post_w) load8(p.post_w + (left > 0 ? i : 0), left, g1[PRE ? c : 0]);
+      if (p.next_w) load8(p.next_w + (left > 0 ? i : 0), left, g2[PRE ? c : 0]);
+    }
+  }
   grid_dep_wait();
   const int r = blockIdx.x;
   int src = r;
@@ -148,7 +158,7 @@ __global__ void __launch_bounds__(NT) residual_norm_kernel(const ResidualNormPar
     }
   }
   if (p.y) {
-    if (p.post_w) norm_row<NT, CH>(y, p, p.post_w, p.post_b, sh[0]);
+    if (p.post_w) norm_row<NT, CH, PRE>(y, p, p.post_w, p.post_b, g1, sh[0]);
 #pragma unroll
     for (int c = 0; c < CH; ++c)
 #pragma unroll
@@ -162,7 +172,7 @@ __global__ void __launch_bounds__(NT) residual_norm_kernel(const ResidualNormPar
     }
   }
   if (p.h) {
-    norm_row<NT, CH>(x, p, p.next_w, p.next_b, sh[2]);
+    norm_row<NT, CH, PRE>(x, p, p.next_w, p.next_b, g2, sh[2]);
 #pragma unroll
     for (int c = 0; c < CH; ++c) {
       const int i = (threadIdx.x + c * NT) * 8;
@@ -196,14 +206,19 @@ extern "C" int xft_residual_norm(const int* ids, const void* table, int vocab, l
   ResidualNormParams p{ids, (const bf16*)table, vocab, ldt, x, ldx, x_out, ldxo, y, ldy, y_f32, post_w, post_b, next_w,
                        next_b, h, ldh, h_f32, rows, n_in, H, HP, kind, eps, status};
   cudaError_t e;
-#define XFT_RN(NT, CH) e = launch_pdl(residual_norm_kernel<NT, CH>, dim3(n_out), dim3(NT), 0, st, p)
-  if (HP <= 256) XFT_RN(32, 1);
-  else if (HP <= 1024) XFT_RN(128, 1);
-  else if (HP <= 2048) XFT_RN(256, 1);
-  else if (HP <= 4096) XFT_RN(256, 2);
-  else if (HP <= 8192) XFT_RN(512, 2);
-  else if (HP <= 16384) XFT_RN(512, 4);
-  else XFT_RN(1024, 4);
+#define XFT_RN(NT, CH, PRE) e = launch_pdl(residual_norm_kernel<NT, CH, PRE>, dim3(n_out), dim3(NT), 0, st, p)
+  const bool few = n_out <= 296;                           // decode: a wide CTA per row, everything in one round of loads
+  if (HP <= 256) XFT_RN(32, 1, true);
+  else if (few && HP <= 1024) XFT_RN(128, 1, true);
+  else if (few && HP <= 2048) XFT_RN(256, 1, true);
+  else if (few && HP <= 4096) XFT_RN(512, 1, true);
+  else if (few && HP <= 8192) XFT_RN(1024, 1, true);
+  else if (HP <= 1024) XFT_RN(128, 1, false);
+  else if (HP <= 2048) XFT_RN(128, 2, false);
+  else if (HP <= 4096) XFT_RN(256, 2, false);
+  else if (HP <= 8192) XFT_RN(512, 2, false);
+  else if (HP <= 16384) XFT_RN(512, 4, false);
+  else XFT_RN(1024, 4, false);
 #undef XFT_RN
   return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }

@@ -553,16 +553,16 @@ def mla_prep(q, kv, Hl, nope, rope, kvl, positions, table, kv_norm_w, eps, cache
     return q_nope.transpose(0, 1), q_rope
 
 
-def plan_attn_splits(B, hkv, group, D, max_kv, int8=False):
+def plan_attn_splits(B, hkv, group, D, max_kv, int8=False, least=8):
     """Split-KV factor of a decode launch and the tile count it was planned on: fill the resident CTA slots (two
     CTAs per SM for the TMA-ring kernel of bf16 caches, three for the cp.async kernel of int8 caches) while leaving
-    every slice at least eight tiles."""
+    every slice at least `least` tiles."""
     tma = not int8 and _ENV().attn_tma
     kt = 64 if tma else {64: 64, 128: 32, 256: 16}[D]
     slots = (296 if D <= 128 else 148) if tma else 444
     ntiles = (max_kv + kt - 1) // kt
     ctas = B * max(hkv, 1) * ((group + 15) // 16)
-    nsplit = max(1, min(slots // max(ctas, 1), ntiles // 8 if ntiles >= 16 else 1, 32))
+    nsplit = max(1, min(slots // max(ctas, 1), ntiles // least if ntiles >= 16 else 1, 32))
     if _ENV().attn_splits > 0:
         nsplit = max(1, min(_ENV().attn_splits, ntiles, 32))
     return nsplit, ntiles
@@ -607,9 +607,9 @@ def paged_attention(q, kc, vc, block_table, cu_q, kv_lens, scale, ks=None, vs=No
     out = torch.empty_like(q)
     nsplit, po, pm = 1, None, None
     if decode:
-        # a window bounds the keys a step can visit, whatever the context length
+        # a window bounds the keys a step can visit, whatever the context length (short slices then pay: measured)
         seen = min(max_kv, window + keep_first + 128) if window > 0 else max_kv
-        nsplit, ntiles = plan_attn_splits(B, hkv, g, D, seen, ks is not None)
+        nsplit, ntiles = plan_attn_splits(B, hkv, g, D, seen, ks is not None, 4 if window > 0 else 8)
         if meta is not None and getattr(meta, "meta", None) is not None and "nsplit" in meta.meta:
             nsplit = meta.meta["nsplit"]
         if B * hkv * ((g + 15) // 16) > ws.attn_counters.numel():
