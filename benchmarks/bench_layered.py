@@ -21,31 +21,19 @@ SIZES = {
 VOCAB = 32000
 
 
-def kafipel_config(s, window=1024, keep=4, share=True):
-    """The second half of the layers reads the keys of the last layer of the first half."""
-    layers = []
-    for i in range(s["layers"]):
-        m = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0,
-             "rot": {"dims": 64, "base": 500000.0, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}},
-             "mask": {"size": window, "keep_first": keep}}
-        if share and i >= s["layers"] // 2:
-            m["kv_from"] = s["layers"] // 2 - 1
-        layers.append({"type": "attention", "mixer": m, "mlp": {"kind": "dense", "ff": s["ff"]}})
-    return {"architecture": "Kafipel", "width": s["width"], "vocab": VOCAB, "norm": {"eps": 1e-5}, "layers": layers}
-
-
 def _model(kind, s, tmp):
     import xfastertransformer_b200 as xft
-    from xfastertransformer_b200.tools.synthetic import config_only, preset
+    from xfastertransformer_b200.config import ModelConfig
+    from xfastertransformer_b200.tools.synthetic import config_only, kafipel_config, preset
     d = os.path.join(tmp, kind)
     if kind == "llama":
         config_only(d, preset("llama-2-7b", num_layer=s["layers"], hidden_size=s["width"], head_num=s["heads"],
                               kv_head_num=s["kv_heads"], size_per_head=128, inter_size=s["ff"], vocab_size=VOCAB,
                               max_pos_seq_len=8192))
     else:
-        os.makedirs(d)
-        with open(os.path.join(d, "config.json"), "w") as f:
-            json.dump(kafipel_config(s, **({"window": 1 << 20, "share": False} if kind == "kafipel_full" else {})), f)
+        kw = {k: s[k] for k in ("width", "heads", "kv_heads", "ff", "layers")}
+        full = {"window": 1 << 20, "share": False} if kind == "kafipel_full" else {}
+        config_only(d, ModelConfig.from_dict(kafipel_config(vocab=VOCAB, **kw, **full)))
     return xft.AutoModel.from_pretrained(d, dtype="bf16", kv_cache_dtype="bf16")
 
 

@@ -206,10 +206,14 @@ class ModelConfig:
     @classmethod
     def from_json(cls, path: str) -> "ModelConfig":
         with open(path if path.endswith(".json") else os.path.join(path, "config.json")) as f:
-            d = json.load(f)
+            return cls.from_dict(json.load(f), path)
+
+    @classmethod
+    def from_dict(cls, d: dict, where: str = "config.json") -> "ModelConfig":
+        """A layered design from the contents of its ``config.json``."""
         arch = d.get("architecture")
         if arch not in ARCHITECTURES:
-            raise ValueError(f"unsupported architecture {arch!r} in {path}; known: {sorted(ARCHITECTURES)}")
+            raise ValueError(f"unsupported architecture {arch!r} in {where}; known: {sorted(ARCHITECTURES)}")
         layers = [_layer_config(i, e) for i, e in enumerate(d["layers"])]
         for i, l in enumerate(layers):
             j = l.mixer.kv_from

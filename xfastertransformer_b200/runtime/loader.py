@@ -368,6 +368,23 @@ class SafetensorsFile:
         return t.view(view) if view is not None else t
 
 
+def write_safetensors(path: str, tensors: dict) -> None:
+    """Write bf16 / fp32 / int32 tensors in the layout `SafetensorsFile` reads."""
+    names = {torch.bfloat16: "BF16", torch.float32: "F32", torch.int32: "I32"}
+    head, off = {}, 0
+    for n, t in tensors.items():
+        size = t.numel() * t.element_size()
+        head[n] = {"dtype": names[t.dtype], "shape": list(t.shape), "data_offsets": [off, off + size]}
+        off += size
+    h = json.dumps(head).encode()
+    h += b" " * (-len(h) % 8)
+    with open(path, "wb") as f:
+        f.write(struct.pack("<Q", len(h)) + h)
+        for t in tensors.values():
+            t = t.detach().cpu().contiguous()
+            (t.view(torch.int16) if t.dtype == torch.bfloat16 else t).numpy().tofile(f)
+
+
 class SafetensorsSource(WeightSource):
     """`WeightSource` over ``model.safetensors`` (linear weights stored [out, in]); fake mode works as there."""
 

@@ -16,7 +16,7 @@ import torch
 
 from ..config import ModelConfig, RopeConfig
 from ..ops import reference as R
-from ..runtime.loader import write_bin
+from ..runtime.loader import write_bin, write_safetensors
 
 PRESETS: Dict[str, dict] = {
     # BASELINE configs
@@ -45,11 +45,66 @@ PRESETS: Dict[str, dict] = {
 }
 
 
+def kafipel_config(width: int, heads: int, kv_heads: int, ff: int, layers: int, vocab: int = 32000, dim: int = 128,
+                   window: int = 1024, keep_first: int = 4, share: bool = True, eps: float = 1e-5) -> dict:
+    """config.json of a Kafipel model with equal layers; with `share`, the second half of them reads the keys and values of
+    the last layer of the first half."""
+    out = []
+    for i in range(layers):
+        m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "softcap": 50.0,
+             "rot": {"dims": dim // 2, "base": 500000.0,
+                     "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}},
+             "mask": {"size": window, "keep_first": keep_first}}
+        if share and i >= max(layers // 2, 1):
+            m["kv_from"] = max(layers // 2, 1) - 1
+        out.append({"type": "attention", "mixer": m, "mlp": {"kind": "dense", "ff": ff}})
+    return {"architecture": "Kafipel", "width": width, "vocab": vocab, "norm": {"eps": eps}, "layers": out}
+
+
+LAYERED_PRESETS: Dict[str, dict] = {
+    "tiny-kafipel": dict(width=192, heads=6, kv_heads=2, ff=512, layers=3, vocab=1000, dim=64, window=48),
+    "kafipel-1b": dict(width=2048, heads=16, kv_heads=4, ff=5632, layers=16),
+    "kafipel-8b": dict(width=4096, heads=32, kv_heads=8, ff=14336, layers=32),
+}
+
+
+def _write_layered(path: str, cfg: ModelConfig, seed: int, std: float) -> str:
+    """config.json and model.safetensors of a layered design, every tensor N(0, std) (norm gains around one)."""
+    cfg.to_ini(path)
+    g = torch.Generator().manual_seed(seed)
+    W, t = cfg.hidden_size, {}
+
+    def put(name, *shape, around=0.0, s=std):
+        t[name] = (around + torch.randn(*shape, generator=g) * s).bfloat16()
+
+    put("embed", cfg.vocab_size, W)
+    put("final.norm", W, around=1.0, s=0.05)
+    put("head", cfg.vocab_size, W)
+    for i, lc in enumerate(cfg.layers):
+        p, m = f"l{i}.", lc.mixer
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if lc.ff else ()):
+            put(p + n, W, around=1.0, s=0.05)
+        put(p + "mix.q", m.heads * m.dim, W)
+        if m.kv_from < 0:
+            put(p + "mix.k", m.kv_heads * m.dim, W)
+            put(p + "mix.v", m.kv_heads * m.vdim, W)
+        put(p + "mix.sink", m.heads, s=1.0)
+        put(p + "mix.o", W, m.heads * m.vdim)
+        if lc.ff:
+            put(p + "mlp.gate", lc.ff, W)
+            put(p + "mlp.up", lc.ff, W)
+            put(p + "mlp.down", W, lc.ff)
+    write_safetensors(os.path.join(path, "model.safetensors"), t)
+    return path
+
+
 def preset(name: str, **over) -> ModelConfig:
+    if name in LAYERED_PRESETS:
+        return ModelConfig.from_dict(kafipel_config(**dict(LAYERED_PRESETS[name], **over)))
     if name not in PRESETS:
         from .model_zoo import ZOO          # public model architectures (examples/model_config)
         if name not in ZOO:
-            raise KeyError(f"unknown model preset '{name}'; known: {sorted(set(PRESETS) | set(ZOO))}")
+            raise KeyError(f"unknown model preset '{name}'; known: {sorted(set(PRESETS) | set(LAYERED_PRESETS) | set(ZOO))}")
         d = dict(ZOO[name])
     else:
         d = dict(PRESETS[name])
@@ -70,6 +125,8 @@ def write_synthetic_checkpoint(path: str, cfg: ModelConfig, seed: int = 0, std: 
                                dtype: Optional[str] = None) -> str:
     """Write config.ini and every tensor.  Linear weights are drawn in HF orientation [out,in]
     in fp32, rounded to `dtype`, and stored transposed ([in,out]) like the converters do."""
+    if cfg.layers:
+        return _write_layered(path, cfg, seed, std)
     dtype = dtype or cfg.weight_data_type
     os.makedirs(path, exist_ok=True)
     cfg.weight_data_type = dtype
