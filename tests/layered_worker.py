@@ -29,3 +29,4 @@ if model.rank == 0:
     torch.save({"rows": rows, "tokens": tokens, "prompts": prompts, "heads": heads}, out)
 m._closed = True
 dist.barrier()
+dist.destroy_process_group()

@@ -31,3 +31,4 @@ if model.rank == 0:
     torch.save({"logits": logits, "logits2": logits2, "held": held}, out)
 m._closed = True
 dist.barrier()
+dist.destroy_process_group()

@@ -135,7 +135,7 @@ def _ranks(case, tmp_path, port, n=2, **env):
 def test_tensor_parallel_two_ranks(cases, tmp_path):
     """Heads (also a key/value head that both ranks read), sinks, feed-forward rows and the head split over two ranks."""
     c = cases("shared")
-    r, out = _ranks(c, tmp_path, 29731)
+    r, out = _ranks(c, tmp_path, 29831)
     assert r.returncode == 0, r.stdout[-2000:] + r.stderr[-2000:]
     got = torch.load(out)
     C.check(got["rows"], torch.cat([c.want(got["prompts"][0])[[3, 49]], c.want(got["prompts"][1])[-1:]]), "fp32", "two ranks")
@@ -151,7 +151,7 @@ def test_pipeline_stages(cases, tmp_path):
     c = C.Case.__new__(C.Case)
     c.name, c.cfg, c.W, c._want = "stages", cfg, O.random_weights(cfg, 4), {}
     c.path = O.write_checkpoint(str(tmp_path / "stages"), cfg, c.W)
-    r, out = _ranks(c, tmp_path, 29741, XFT_PIPELINE_STAGE="2")
+    r, out = _ranks(c, tmp_path, 29841, XFT_PIPELINE_STAGE="2")
     assert r.returncode == 0, r.stdout[-2000:] + r.stderr[-2000:]
     got = torch.load(out)
     C.check(got["rows"], torch.cat([c.want(got["prompts"][0])[[3, 49]], c.want(got["prompts"][1])[-1:]]), "fp32", "stages")
