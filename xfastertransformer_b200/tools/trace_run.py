@@ -2,14 +2,13 @@
 
     bin/trace_run --model DIR --dtype bfloat16|float32 --out DIR --max-tokens N < steps.jsonl
 
-Each line of standard input is one step, a JSON object
+A line of standard input describes one step of the engine:
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 7, "entries": [{"id": "q1", "tokens": [812], "want": [0]}, {"id": "q2", "tokens": [4, 4, 90], "want": []}], "end": ["q1"]}
 
-whose entries (the next tokens of each request) run as ONE batch of the engine, portions of prompts beside single decoded
-tokens.  ``want`` are the places among an entry's tokens whose logits go to OUT/<step>.f32 (little-endian fp32, in the
-order of the entries and of ``want``; no file when nothing is wanted); ``end`` names requests whose cache blocks are given
-back after the step.  After every step a line ``done <step>`` is printed.
+All entries go through the model in one batch, prompt portions of any length next to single tokens.  ``want`` lists places
+in an entry's tokens; their logits are stored in OUT/<step>.f32 as fp32 rows, entry by entry (a step that wants none leaves
+no file).  The cache blocks of the requests in ``end`` are freed once the step has run, and ``done <step>`` is printed.
 
 The tool is a thin client of the continuous-batching API: a request's first entry is admitted with `set_input_cb`, later
 ones continue it (`extend=True`), `forward_cb` runs the step, `free_seqs` ends requests.  Nothing is sampled.  The KV pools
@@ -32,7 +31,6 @@ class TraceRunner:
 
         from ..automodel import AutoModel
         from ..utils.flags import Env
-        self.torch = torch
         if not torch.cuda.is_available() and not Env.get().engine.upper().startswith("CPU"):
             raise RuntimeError("no CUDA device (XFT_ENGINE=CPU runs the PyTorch path)")
         self.model = AutoModel.from_pretrained(path, dtype=dtype, kv_cache_dtype="bf16", max_cache_tokens=max_tokens)
