@@ -95,9 +95,9 @@ class LayeredDecoder(Decoder):
             n = max(_up(positions, 2048), 2 * tab.shape[0] if tab is not None else 0)
             if rot.factor > 0:
                 new = R.rope_table(n, rot.dims, rot.base, "yarn", rot.factor, rot.original, rot.fast, rot.slow,
-                                   table_scale=0.1 * math.log(rot.factor) + 1.0)
+                                   table_scale=0.1 * math.log(rot.factor) + 1.0, angle_dtype=torch.float64)
             else:
-                new = R.rope_table(n, rot.dims, rot.base)
+                new = R.rope_table(n, rot.dims, rot.base, angle_dtype=torch.float64)
             if tab is not None:
                 self._old_ropes.append(tab)       # captured decode graphs keep reading it (their positions fit it)
             tab = self._ropes[rot] = new.to(self.device)

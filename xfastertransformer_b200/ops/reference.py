@@ -251,7 +251,8 @@ def yarn_mscale(scale: float = 1.0, mscale: float = 1.0) -> float:
 
 
 def rope_inv_freq(rot_dim: int, theta: float, scaling_type: str = "", factor: float = 1.0,
-                  original_max_pos: int = 2048, beta_fast: float = 32, beta_slow: float = 1) -> torch.Tensor:
+                  original_max_pos: int = 2048, beta_fast: float = 32, beta_slow: float = 1,
+                  dtype: torch.dtype = torch.float32) -> torch.Tensor:
     """Frequency of each rotated pair.  YaRN divides the slow ones by `factor`: none of the pairs up to `low`, all from
     `high` on, a linear ramp between (a step when the two coincide)."""
     inv = 1.0 / (theta ** (torch.arange(0, rot_dim, 2, dtype=torch.float64) / rot_dim))
@@ -263,27 +264,27 @@ def rope_inv_freq(rot_dim: int, theta: float, scaling_type: str = "", factor: fl
         ramp = ((torch.arange(rot_dim // 2, dtype=torch.float64) - low) / max(high - low, 0.001)).clamp(0, 1)
         mask = 1.0 - ramp                      # 1 -> extrapolate (keep), 0 -> interpolate
         inv = inv / factor * (1 - mask) + inv * mask
-    return inv.float()
+    return inv.to(dtype)
 
 
 def rope_table(max_pos: int, rot_dim: int, theta: float = 10000.0, scaling_type: str = "",
                factor: float = 1.0, original_max_pos: int = 2048, beta_fast: float = 32,
                beta_slow: float = 1, mscale: float = 1.0, mscale_all_dim: float = 0.0,
-               table_scale: Optional[float] = None) -> torch.Tensor:
+               table_scale: Optional[float] = None, angle_dtype: torch.dtype = torch.float32) -> torch.Tensor:
     """-> fp32 [max_pos, rot_dim] = cat(cos, sin) of pos*inv_freq (rot_dim/2 each).
 
     YaRN multiplies the table by yarn_mscale(factor, mscale)/yarn_mscale(factor, mscale_all_dim)
     (rotary_embedding_deepseekv2.cpp:62-85; yarn_scaled_rotary_embedding.cpp:26-84 uses
-    0.1*ln(factor)+1)."""
-    inv = rope_inv_freq(rot_dim, theta, scaling_type, factor, original_max_pos, beta_fast, beta_slow)
-    t = torch.arange(max_pos, dtype=torch.float32)
+    0.1*ln(factor)+1).  `angle_dtype` float64 keeps the rounding of large angles out of the table."""
+    inv = rope_inv_freq(rot_dim, theta, scaling_type, factor, original_max_pos, beta_fast, beta_slow, angle_dtype)
+    t = torch.arange(max_pos, dtype=angle_dtype)
     fr = torch.outer(t, inv)
     s = 1.0
     if table_scale is not None:
         s = table_scale
     elif scaling_type == "yarn" and factor > 1.0:
         s = yarn_mscale(factor, mscale) / (yarn_mscale(factor, mscale_all_dim) if mscale_all_dim else 1.0)
-    return torch.cat([fr.cos() * s, fr.sin() * s], dim=-1)
+    return torch.cat([fr.cos() * s, fr.sin() * s], dim=-1).float()
 
 
 def telechat_ntk_alpha(true_seq_len: int) -> float:
