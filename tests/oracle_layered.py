@@ -1,4 +1,5 @@
-"""A plain, slow implementation of the Kafipel design, one function per mechanism, for the tests to compare against.
+"""A plain, slow implementation of the layered designs (Kafipel, Vepivik), one function per mechanism, for the tests to
+compare against.
 
 It works on one whole sequence at a time, without a cache, in the precision of the tensors it is given (tests use fp64
 or fp32), straight from the equations; nothing here is shared with the package.
@@ -18,6 +19,10 @@ def layer_norm(x, w, eps):
     d = x - mu
     var = (d * d).sum(-1, keepdim=True) / x.shape[-1]
     return d / torch.sqrt(var + eps) * w
+
+
+def rms_norm(x, w, eps):
+    return x / torch.sqrt((x * x).sum(-1, keepdim=True) / x.shape[-1] + eps) * w
 
 
 def rotary_frequencies(rot):
@@ -41,8 +46,9 @@ def rotary_frequencies(rot):
     return out, 0.1 * math.log(sc["factor"]) + 1.0
 
 
-def rotate(x, positions, rot):
-    """x [T, heads, dim]: dimension i < dims/2 turns together with dimension i + dims/2."""
+def rotate(x, positions, rot, interleaved=False):
+    """x [T, heads, dim]: dimension i < dims/2 turns together with dimension i + dims/2, or, interleaved, dimension 2i with
+    dimension 2i + 1."""
     if not rot:
         return x
     f, m = rotary_frequencies(rot)
@@ -52,9 +58,10 @@ def rotate(x, positions, rot):
         a = [p * f[i] for p in positions]
         c = torch.tensor([math.cos(t) * m for t in a], dtype=x.dtype)[:, None]
         s = torch.tensor([math.sin(t) * m for t in a], dtype=x.dtype)[:, None]
-        u, v = x[:, :, i], x[:, :, i + half]
-        y[:, :, i] = u * c - v * s
-        y[:, :, i + half] = v * c + u * s
+        iu, iv = (2 * i, 2 * i + 1) if interleaved else (i, i + half)
+        u, v = x[:, :, iu], x[:, :, iv]
+        y[:, :, iu] = u * c - v * s
+        y[:, :, iv] = v * c + u * s
     return y
 
 
@@ -64,7 +71,7 @@ def sees(i, j, mask):
         return False
     if not mask:
         return True
-    return i - j < mask["size"] or j < mask["keep_first"]
+    return i - j < mask["size"] or j < mask.get("keep_first", 0)
 
 
 _VISIBLE = {}
@@ -117,6 +124,78 @@ def mixer(h, m, W, prefix, positions, kept):
     return a.reshape(T, -1) @ W[prefix + ".mix.o"].T
 
 
+def latent_scores_and_values(q, c, kr, uk, uv, scale, rot_dim):
+    """Scores [H, T, T] (no mask) and values [T, H, vdim] from latents c [T, rank], shared rotated keys kr [T, rot_dim],
+    queries q [T, H, dim + rot_dim] and the per-head matrices uk [H, dim, rank], uv [H, vdim, rank]."""
+    H, d = uk.shape[:2]
+    s = torch.stack([(q[:, h, :d] @ (c @ uk[h].T).T + q[:, h, d:] @ kr.T) * scale for h in range(H)])
+    v = torch.stack([c @ uv[h].T for h in range(H)], 1)
+    return s, v
+
+
+def masked_softmax(s, mask):
+    """Weights of the visible keys; s [..., T, T]."""
+    vis = visible(s.shape[-1], mask)
+    e = torch.where(vis, torch.exp(s - torch.where(vis, s, torch.full_like(s, -math.inf)).max(-1, keepdim=True).values), 0.0)
+    return e / e.sum(-1, keepdim=True)
+
+
+def latent_attention(q, c, kr, uk, uv, scale, mask):
+    """-> [T, H, vdim]"""
+    s, v = latent_scores_and_values(q, c, kr, uk, uv, scale, kr.shape[1])
+    return torch.stack([masked_softmax(s[h], mask) @ v[:, h] for h in range(s.shape[0])], 1)
+
+
+def latent_mixer(h, m, W, prefix, positions, kept, eps):
+    """Latent attention sublayer.  `kept` maps a layer index to its (latents after the norm, shared key part after rotation)."""
+    T, H, d, rd, R = h.shape[0], m["heads"], m["dim"], m["rot_dim"], m["kv_rank"]
+    P = prefix + ".mix."
+    q = (h @ W[P + "q"].T).view(T, H, d + rd).clone()
+    q[:, :, d:] = rotate(q[:, :, d:], positions, m["rot"], interleaved=True)
+    if m.get("kv_from") is None:
+        kv = h @ W[P + "dkv"].T
+        c = rms_norm(kv[:, :R], W[P + "dkv.norm"], eps)
+        kr = rotate(kv[:, None, R:], positions, m["rot"], interleaved=True)[:, 0]
+    else:
+        c, kr = kept[m["kv_from"]]
+    kept[int(prefix[1:])] = (c, kr)
+    a = latent_attention(q, c, kr, W[P + "uk"].view(H, d, R), W[P + "uv"].view(H, m["vdim"], R), m["scale"], m.get("mask"))
+    a = a.reshape(T, -1) * output_gate(h, W[P + "g"])
+    return a @ W[P + "o"].T
+
+
+def output_gate(h, wg):
+    return 1 / (1 + torch.exp(-(h @ wg.T)))
+
+
+def router(z, top):
+    """Chosen experts [T, top] (best first) and their weights."""
+    e = torch.exp(z - z.max(-1, keepdim=True).values)
+    s = e / e.sum(-1, keepdim=True)
+    idx = torch.argsort(s, -1, descending=True)[:, :top]
+    w = torch.gather(s, 1, idx)
+    return idx, w / (w.sum(-1, keepdim=True) + 1e-20)
+
+
+def expert(h, up, down):
+    u = h @ up.T
+    u = torch.where(u > 0, u, torch.zeros_like(u))
+    return (u * u) @ down.T
+
+
+def experts(h, f, W, prefix):
+    """Mixture of experts: the chosen experts' weighted outputs plus the shared expert's."""
+    P = prefix + ".mlp."
+    idx, w = router(h @ W[P + "router"].T, f["router"]["top"])
+    out = torch.zeros(h.shape[0], W["embed"].shape[1], dtype=h.dtype)
+    for t in range(h.shape[0]):
+        for e, we in zip(idx[t].tolist(), w[t]):
+            out[t] += we * expert(h[t:t + 1], W[P + f"e{e}.up"], W[P + f"e{e}.down"])[0]
+    if f.get("shared"):
+        out = out + expert(h, W[P + "shared.up"], W[P + "shared.down"])
+    return out
+
+
 def feed_forward(h, W, prefix):
     g, u = h @ W[prefix + ".mlp.gate"].T, h @ W[prefix + ".mlp.up"].T
     return (g / (1 + torch.exp(-g)) * u) @ W[prefix + ".mlp.down"].T
@@ -125,6 +204,11 @@ def feed_forward(h, W, prefix):
 def forward(cfg, W, tokens, layers_out=None, dtype=torch.float64):
     """Logits [T, vocab] of one sequence; `layers_out` (a list) collects the residual stream after every layer."""
     W = {n: (t.to(dtype) if t.is_floating_point() else t) for n, t in W.items()}
+    run = {"Kafipel": _kafipel, "Vepivik": _vepivik}[cfg["architecture"]]
+    return run(cfg, W, tokens, [] if layers_out is None else layers_out)
+
+
+def _kafipel(cfg, W, tokens, layers_out):
     eps = cfg["norm"]["eps"]
     positions = list(range(len(tokens)))
     x = W["embed"][torch.tensor(tokens)]
@@ -136,9 +220,26 @@ def forward(cfg, W, tokens, layers_out=None, dtype=torch.float64):
         if layer.get("mlp"):
             y = feed_forward(layer_norm(x, W[p + ".norm2"], eps), W, p)
             x = x + layer_norm(y, W[p + ".norm2b"], eps)
-        if layers_out is not None:
-            layers_out.append(x.clone())
+        layers_out.append(x.clone())
     return layer_norm(x, W["final.norm"], eps) @ W["head"].T
+
+
+def _vepivik(cfg, W, tokens, layers_out):
+    eps = cfg["norm"]["eps"]
+    positions = list(range(len(tokens)))
+    x = W["embed"][torch.tensor(tokens)] * cfg["embedding"]["scale"]
+    kept = {}
+    for i, layer in enumerate(cfg["layers"]):
+        p = f"l{i}"
+        h = rms_norm(x, W[p + ".norm1"], eps)
+        if layer["type"] == "latent_attention":
+            x = x + latent_mixer(h, layer["mixer"], W, p, positions, kept, eps)
+        else:
+            x = x + mixer(h, layer["mixer"], W, p, positions, kept)
+        if layer.get("mlp"):
+            x = x + experts(rms_norm(x, W[p + ".norm2"], eps), layer["mlp"], W, p)
+        layers_out.append(x.clone())
+    return rms_norm(x, W["final.norm"], eps) @ W["embed"].T
 
 
 # ------------------------------------------------------------------------------------------ small checkpoints
@@ -162,6 +263,37 @@ def config(layers, width=96, vocab=210, eps=1e-5):
     return {"architecture": "Kafipel", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width}
 
 
+def moe(ff=40, experts=6, top=2, shared=56):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top},
+            "shared": {"ff": shared} if shared else None}
+
+
+def window_layer(heads=4, kv_heads=2, dim=32, vdim=24, size=24, scale=None, mlp=None, mask=True):
+    """Attention without rotation."""
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale if scale else dim ** -0.5}
+    if mask:
+        m["mask"] = {"size": size}
+    return {"type": "attention", "mixer": m, "mlp": mlp}
+
+
+def latent_layer(heads=4, dim=32, rot_dim=16, vdim=24, kv_rank=40, size=24, base=10000.0, scaling=None, scale=None, kv_from=None,
+                 mlp=None, mask=True):
+    m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank,
+         "scale": scale if scale else (dim + rot_dim) ** -0.5, "rot": {"dims": rot_dim, "base": base}}
+    if scaling:
+        m["rot"]["scaling"] = scaling
+    if mask:
+        m["mask"] = {"size": size}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "latent_attention", "mixer": m, "mlp": mlp}
+
+
+def vepivik(layers, width=96, vocab=210, eps=1e-5, scale=2.0):
+    return {"architecture": "Vepivik", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width,
+            "embedding": {"scale": scale}}
+
+
 def random_weights(cfg, seed=0, gain=1.0):
     """bf16-representable weights, scaled so that scores spread over several units and every mechanism matters."""
     g = torch.Generator().manual_seed(seed)
@@ -173,21 +305,45 @@ def random_weights(cfg, seed=0, gain=1.0):
         return (around + s * torch.randn(n, generator=g)).bfloat16()
 
     D = cfg["width"]
-    W = {"embed": torch.randn(cfg["vocab"], D, generator=g).bfloat16(), "final.norm": vec(D),
-         "head": mat(cfg["vocab"], D)}
+    kafipel = cfg["architecture"] == "Kafipel"
+    W = {"embed": torch.randn(cfg["vocab"], D, generator=g).bfloat16(), "final.norm": vec(D)}
+    if kafipel:
+        W["head"] = mat(cfg["vocab"], D)
+    else:
+        W["embed"] = (W["embed"].float() / math.sqrt(D)).bfloat16()
     for i, layer in enumerate(cfg["layers"]):
         p, m = f"l{i}", layer["mixer"]
-        W[p + ".norm1"], W[p + ".norm1b"] = vec(D), vec(D, 0.7)
-        W[p + ".mix.q"] = mat(m["heads"] * m["dim"], D, 1.6)
-        if m.get("kv_from") is None:
-            W[p + ".mix.k"] = mat(m["kv_heads"] * m["dim"], D, 1.6)
-            W[p + ".mix.v"] = mat(m["kv_heads"] * m["vdim"], D)
-        W[p + ".mix.sink"] = vec(m["heads"], 1.0, 1.0)
+        W[p + ".norm1"] = vec(D)
+        if kafipel:
+            W[p + ".norm1b"] = vec(D, 0.7)
+        if layer["type"] == "latent_attention":
+            W[p + ".mix.q"] = mat(m["heads"] * (m["dim"] + m["rot_dim"]), D, 1.6)
+            if m.get("kv_from") is None:
+                W[p + ".mix.dkv"] = mat(m["kv_rank"] + m["rot_dim"], D, 1.3)
+                W[p + ".mix.dkv.norm"] = vec(m["kv_rank"])
+            W[p + ".mix.uk"] = mat(m["heads"] * m["dim"], m["kv_rank"], 1.6)
+            W[p + ".mix.uv"] = mat(m["heads"] * m["vdim"], m["kv_rank"])
+            W[p + ".mix.g"] = mat(m["heads"] * m["vdim"], D, 2.0)
+        else:
+            W[p + ".mix.q"] = mat(m["heads"] * m["dim"], D, 1.6)
+            if m.get("kv_from") is None:
+                W[p + ".mix.k"] = mat(m["kv_heads"] * m["dim"], D, 1.6)
+                W[p + ".mix.v"] = mat(m["kv_heads"] * m["vdim"], D)
+            if kafipel:
+                W[p + ".mix.sink"] = vec(m["heads"], 1.0, 1.0)
         W[p + ".mix.o"] = mat(D, m["heads"] * m["vdim"])
-        if layer.get("mlp"):
-            f = layer["mlp"]["ff"]
-            W[p + ".norm2"], W[p + ".norm2b"] = vec(D), vec(D, 0.7)
-            W[p + ".mlp.gate"], W[p + ".mlp.up"], W[p + ".mlp.down"] = mat(f, D), mat(f, D), mat(D, f)
+        f = layer.get("mlp")
+        if not f:
+            continue
+        W[p + ".norm2"] = vec(D)
+        if f["kind"] == "moe":
+            W[p + ".mlp.router"] = mat(f["router"]["experts"], D, 2.0)
+            for n, ff in [(f"e{e}", f["expert"]["ff"]) for e in range(f["router"]["experts"])] + \
+                    ([("shared", f["shared"]["ff"])] if f.get("shared") else []):
+                W[p + f".mlp.{n}.up"], W[p + f".mlp.{n}.down"] = mat(ff, D), mat(D, ff, 0.8)
+        else:
+            W[p + ".norm2b"] = vec(D, 0.7)
+            W[p + ".mlp.gate"], W[p + ".mlp.up"], W[p + ".mlp.down"] = mat(f["ff"], D), mat(f["ff"], D), mat(D, f["ff"])
     return W
 
 

@@ -38,7 +38,7 @@ MODEL_TYPES = (
 )
 
 # config.json "architecture" -> model type
-ARCHITECTURES = {"Kafipel": "kafipel"}
+ARCHITECTURES = {"Kafipel": "kafipel", "Vepivik": "vepivik"}
 
 
 def split_hybrid_dtype(dtype: str) -> Tuple[str, str]:
@@ -80,20 +80,26 @@ class RopeConfig:
 
 @dataclass(frozen=True)
 class RotaryConfig:
-    """Rotary positions of one layer: the first `dims` dimensions of each head, base, optional YaRN scaling."""
+    """Rotary positions of one layer: the first `dims` dimensions of each head (of the rotated part, in latent attention),
+    base, optional YaRN scaling; `style` "half" pairs dimension i with i + dims/2, "interleaved" 2i with 2i + 1."""
     dims: int
     base: float
     factor: float = 0.0               # 0: no scaling
     original: float = 0.0
     fast: float = 32.0
     slow: float = 1.0
+    style: str = "half"
 
 
 @dataclass(frozen=True)
 class MixerConfig:
     """Token mixer of one layer.  `window` 0: every earlier position is visible; otherwise position i sees j <= i when
     i - j < window or j < keep_first.  `softcap` 0: scores are not capped.  `kv_from` >= 0: this layer has queries only
-    and reads the keys and values of that layer."""
+    and reads the keys and values of that layer.
+
+    `kind` "latent": keys and values come from one latent of `kv_rank` values per token, expanded per head to `dim` key and
+    `vdim` value dimensions, plus `rot_dim` rotated key dimensions that all heads share (kv_heads is 1: one cache row per
+    token).  `gate`: the concatenated heads are multiplied with sigmoid(W_g h)."""
     heads: int
     kv_heads: int
     dim: int
@@ -105,13 +111,34 @@ class MixerConfig:
     keep_first: int = 0
     rot: Optional[RotaryConfig] = None
     kv_from: int = -1
+    kv_rank: int = 0
+    rot_dim: int = 0
+    gate: bool = False
+
+    def kv_shape(self) -> tuple:
+        """What two layers must agree on for one to read the other's cache."""
+        if self.kind == "latent":
+            return self.kind, self.kv_rank, self.rot_dim, self.rot
+        return self.kind, self.kv_heads, self.dim, self.vdim
+
+
+@dataclass(frozen=True)
+class MoeConfig:
+    """Mixture of experts of one layer: softmax over `experts` router logits, the `top` best with their scores divided by
+    their sum, and (`shared` > 0) one more expert that every token uses.  An expert is down(act(up x))."""
+    experts: int
+    top: int
+    ff: int
+    shared: int = 0
+    act: str = "relu2"
 
 
 @dataclass(frozen=True)
 class LayerConfig:
     mixer: MixerConfig
-    ff: int = 0                       # 0: no feed-forward
+    ff: int = 0                       # width of a dense feed-forward; 0: none
     ff_kind: str = "dense"
+    moe: Optional[MoeConfig] = None
 
 
 @dataclass
@@ -162,6 +189,7 @@ class ModelConfig:
     do_qk_norm: bool = False
     # layered designs (config.json): one entry per layer; the scalar sizes above then hold the first layer's
     layers: List[LayerConfig] = field(default_factory=list)
+    embed_scale: float = 1.0
     # raw key/value pairs (for family-specific look-ups, like DecoderContext::GetAttr)
     raw: Dict[str, str] = field(default_factory=dict)
 
@@ -221,13 +249,14 @@ class ModelConfig:
                 src = layers[j].mixer if j < i else None
                 if src is None or src.kv_from >= 0:
                     raise ValueError(f"layer {i}: kv_from {j} is not an earlier layer with keys and values of its own")
-                if (src.kv_heads, src.dim, src.vdim) != (l.mixer.kv_heads, l.mixer.dim, l.mixer.vdim):
+                if src.kv_shape() != l.mixer.kv_shape():
                     raise ValueError(f"layer {i}: heads differ from those of layer {j}, whose keys it reads")
         m = layers[0].mixer
         return cls(model_type=ARCHITECTURES[arch], head_num=m.heads, kv_head_num=m.kv_heads, size_per_head=m.dim,
                    v_head_dim=m.vdim, hidden_size=int(d["width"]), inter_size=layers[0].ff, num_layer=len(layers),
                    vocab_size=int(d["vocab"]), layernorm_eps=float(d["norm"]["eps"]), start_id=-1, end_id=-1,
-                   weight_data_type="bf16", layers=layers, raw=d)
+                   weight_data_type="bf16", layers=layers, raw=d,
+                   embed_scale=float((d.get("embedding") or {}).get("scale", 1.0)))
 
     @classmethod
     def from_ini(cls, path: str) -> "ModelConfig":
@@ -396,28 +425,45 @@ class ModelConfig:
             cp.write(f)
 
 
+def _rotary(i: int, m: dict, width: int, style: str) -> Optional[RotaryConfig]:
+    if not m.get("rot"):
+        return None
+    r, sc = m["rot"], m["rot"].get("scaling") or {}
+    rot = RotaryConfig(int(r["dims"]), float(r["base"]), float(sc.get("factor", 0.0)), float(sc.get("original", 0.0)),
+                       float(sc.get("fast", 32.0)), float(sc.get("slow", 1.0)), style)
+    if rot.dims % 2 or rot.dims > width:
+        raise ValueError(f"layer {i}: rotary dims {rot.dims} do not fit heads of {width}")
+    return rot
+
+
 def _layer_config(i: int, e: dict) -> LayerConfig:
     """One entry of config.json's ``layers``."""
-    if e.get("type") != "attention":
-        raise ValueError(f"layer {i}: unsupported mixer type {e.get('type')!r}")
-    m = e["mixer"]
-    rot = None
-    if m.get("rot"):
-        r, sc = m["rot"], m["rot"].get("scaling") or {}
-        rot = RotaryConfig(int(r["dims"]), float(r["base"]), float(sc.get("factor", 0.0)), float(sc.get("original", 0.0)),
-                           float(sc.get("fast", 32.0)), float(sc.get("slow", 1.0)))
-        if rot.dims % 2 or rot.dims > int(m["dim"]):
-            raise ValueError(f"layer {i}: rotary dims {rot.dims} do not fit heads of {m['dim']}")
+    kind, m = e.get("type"), e["mixer"]
     mask = m.get("mask") or {}
-    mixer = MixerConfig(heads=int(m["heads"]), kv_heads=int(m.get("kv_heads", m["heads"])), dim=int(m["dim"]),
-                        vdim=int(m.get("vdim", m["dim"])), scale=float(m["scale"]), softcap=float(m.get("softcap") or 0.0),
-                        window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0), rot=rot,
-                        kv_from=-1 if m.get("kv_from") is None else int(m["kv_from"]))
+    common = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m.get("vdim", m["dim"])), scale=float(m["scale"]),
+                  window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0),
+                  softcap=float(m.get("softcap") or 0.0), kv_from=-1 if m.get("kv_from") is None else int(m["kv_from"]))
+    if kind == "attention":
+        mixer = MixerConfig(kv_heads=int(m.get("kv_heads", m["heads"])), rot=_rotary(i, m, int(m["dim"]), "half"), **common)
+    elif kind == "latent_attention":
+        rd = int(m["rot_dim"])
+        mixer = MixerConfig(kind="latent", kv_heads=1, rot=_rotary(i, m, rd, "interleaved"), kv_rank=int(m["kv_rank"]), rot_dim=rd,
+                            gate=True, **common)
+        if mixer.keep_first or mixer.softcap:
+            raise ValueError(f"layer {i}: latent attention has no kept first keys and no cap on the scores")
+    else:
+        raise ValueError(f"layer {i}: unsupported mixer type {kind!r}")
     if mixer.heads % mixer.kv_heads:
         raise ValueError(f"layer {i}: {mixer.heads} query heads over {mixer.kv_heads} key/value heads")
     f = e.get("mlp")
     if not f:
         return LayerConfig(mixer)
-    if f.get("kind") != "dense":
+    if f.get("kind") == "dense":
+        return LayerConfig(mixer, int(f["ff"]), "dense")
+    if f.get("kind") != "moe":
         raise ValueError(f"layer {i}: unsupported feed-forward {f.get('kind')!r}")
-    return LayerConfig(mixer, int(f["ff"]), "dense")
+    moe = MoeConfig(experts=int(f["router"]["experts"]), top=int(f["router"]["top"]), ff=int(f["expert"]["ff"]),
+                    shared=int((f.get("shared") or {}).get("ff", 0)))
+    if not 0 < moe.top <= moe.experts:
+        raise ValueError(f"layer {i}: {moe.top} of {moe.experts} experts")
+    return LayerConfig(mixer, 0, "moe", moe)

@@ -814,8 +814,7 @@ class Decoder:
                     n += v.nbytes
                 elif isinstance(v, (list, tuple)):
                     for e in v:
-                        if isinstance(e, tuple):
-                            n += sum(w.nbytes for w in e if isinstance(w, LinearWeight))
+                        n += sum(w.nbytes for w in (e if isinstance(e, tuple) else (e,)) if isinstance(w, LinearWeight))
         if self.lm_head is not None:
             n += self.lm_head.nbytes
         return n

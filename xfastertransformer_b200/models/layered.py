@@ -1,18 +1,23 @@
-"""Decoder for designs described layer by layer (``ModelConfig.layers``), first of them Kafipel.
+"""Decoder for designs described layer by layer (``ModelConfig.layers``): Kafipel, Vepivik.
 
 It is the generic decoder with sizes, rotation, mask and cache pool taken from each layer's own entry, served by the same
 engine, paged cache, decode runner, sampler and kernels.  What these designs add to it, each as an op with its constants
 as arguments:
 
-* a 32-bit residual stream with a norm before and after every sublayer, one launch between two products
+* a 32-bit residual stream with a norm before and (per design) after every sublayer, one launch between two products
   (`ops.residual_norm`): x += norm_b(y) and h = norm(x) for the product that follows;
 * attention with a sliding window that keeps the first tokens, a tanh cap on the scores and a sink per head
   (`ops.paged_attention(window=, keep_first=, softcap=, sinks=)`);
 * layers without keys and values of their own, which read the pool of an earlier layer (`kv_from`);
-* query/key and value heads of different sizes.
+* query/key and value heads of different sizes;
+* latent attention with a window, an output gate and layers that read another layer's latents
+  (`ops.latent_prep`, `ops.latent_attention`); its pools have one row per token and no values;
+* mixtures of experts without a gate product (`ops.route`, `ops.moe_experts`), next to a shared expert;
+* a scaled embedding, and logits from the embedding table.
 
 Widths that the 16-byte rows of the tensor-core kernels do not allow are padded with zeros at load: the hidden and the
-feed-forward width to a multiple of 8, heads to the next size the attention kernels have.  A zero dimension adds nothing
+feed-forward width to a multiple of 8, heads to the next size the attention kernels have, each part of a latent head to a
+multiple of 64.  A zero dimension adds nothing
 to a score or a sum.  The 32-bit path (dtype "fp32") and CPU tensors keep the heads as they are.
 """
 from __future__ import annotations
@@ -23,7 +28,7 @@ from typing import Dict, List, Optional
 import torch
 
 from .. import ops
-from ..config import LayerConfig, ModelConfig, RotaryConfig
+from ..config import LayerConfig, ModelConfig, MoeConfig, RotaryConfig
 from ..ops import reference as R
 from ..parallel import partition as P
 from ..parallel.dist import DistContext
@@ -125,8 +130,10 @@ class LayeredDecoder(Decoder):
             self.wte = _pad(self.src.matrix("embed", (c.vocab_size, self.W)).to(torch.bfloat16), c.vocab_size, self.WP)
         if self.last_stage:
             self.final = self._gain("final.norm")
-            w = self.src.matrix("head", (c.vocab_size, self.W), rows=(self.v0, self.v1))
+            w = self.src.matrix("embed" if self.spec.tied_head else "head", (c.vocab_size, self.W), rows=(self.v0, self.v1))
             kind = "fp32" if self.exact or self.device.type == "cpu" else "bf16"
+            if self.spec.tied_head and self.wte is not None and kind == "bf16":
+                w = self.wte[self.v0:self.v1]                  # one copy serves both ends
             self.lm_head = make_linear(_pad(w, w.shape[0], self.WP), kind)
 
     def _head_size(self, n: int) -> int:
@@ -134,11 +141,23 @@ class LayeredDecoder(Decoder):
             return n
         return next((d for d in ATTENTION_HEADS if n <= d), _up(n, 8))
 
-    def _head_rows(self, name: str, heads: int, rng, dim: int, padded: int) -> torch.Tensor:
-        """Rows of heads rng[0] .. rng[1] of a [heads * dim, width] projection, each head padded to `padded` rows."""
+    def _rows(self, name: str, heads: int, rng, *parts) -> torch.Tensor:
+        """Rows of heads rng[0] .. rng[1] of a [heads * size, width] projection.  `parts` lists (rows, padded rows) of a
+        head, in order."""
+        dim, padded = sum(a for a, _ in parts), sum(b for _, b in parts)
         w = self.src.matrix(name, (heads * dim, self.W), rows=(rng[0] * dim, rng[1] * dim))
         n = rng[1] - rng[0]
-        return _pad(w.view(n, dim, self.W), n, padded, self.WP).reshape(n * padded, self.WP)
+        w, out, at = w.view(n, dim, self.W), [], 0
+        for a, b in parts:
+            out.append(_pad(w[:, at:at + a], n, b, self.WP))
+            at += a
+        return torch.cat(out, 1).reshape(n * padded, self.WP)
+
+    def _out_rows(self, L: Layer, p: str, heads: int, rng, vdim: int) -> None:
+        """The output projection: its columns are heads of `vdim`, padded to L.vd."""
+        w = self.src.matrix(p + "mix.o", (self.W, heads * vdim), cols=(rng[0] * vdim, rng[1] * vdim))
+        w = _pad(w.reshape(self.W, L.hq, vdim), self.WP, L.hq, L.vd)
+        L.o = make_linear(w.reshape(self.WP, L.hq * L.vd), self.kind)
 
     def _load_layer(self, i: int) -> Layer:
         lc: LayerConfig = self.cfg.layers[i]
@@ -152,65 +171,147 @@ class LayeredDecoder(Decoder):
         L.q_off = qs - ks * L.group
         if L.hq <= 0:
             raise ValueError(f"layer {i}: {m.heads} heads cannot be split over {self.tp} ranks")
-        L.kd, L.vd = self._head_size(m.dim), self._head_size(m.vdim)
-        if self.pad_heads:
-            L.kd = L.vd = max(L.kd, L.vd)         # the tensor-core kernels have one size for keys and values
         L.own_kv = m.kv_from < 0
         L.kv_layer = i if L.own_kv else m.kv_from
-        L.norm1, L.norm1b = self._gain(p + "norm1"), self._gain(p + "norm1b")
-        parts = [self._head_rows(p + "mix.q", m.heads, (qs, qe), m.dim, L.kd)]
-        if L.own_kv:
-            parts.append(self._head_rows(p + "mix.k", m.kv_heads, (ks, ke), m.dim, L.kd))
-            parts.append(self._head_rows(p + "mix.v", m.kv_heads, (ks, ke), m.vdim, L.vd))
-        L.qkv = make_linear(torch.cat(parts), self.kind)
-        L.sinks = None
-        if self.src.exists(p + "mix.sink") or self.src.fake:
-            L.sinks = self.src.vector(p + "mix.sink", m.heads, rng=(qs, qe)).contiguous()
-        w = self.src.matrix(p + "mix.o", (self.W, m.heads * m.vdim), cols=(qs * m.vdim, qe * m.vdim))
-        w = _pad(w.reshape(self.W, L.hq, m.vdim), self.WP, L.hq, L.vd)
-        L.o = make_linear(w.reshape(self.WP, L.hq * L.vd), self.kind)
+        second = self._gain if self.spec.post_norm else lambda name: None
+        L.norm1, L.norm1b = self._gain(p + "norm1"), second(p + "norm1b")
+        if m.kind == "latent":
+            self._load_latent(L, p, (qs, qe))
+        else:
+            self._load_attention(L, p, (qs, qe), (ks, ke))
         L.mlp_kind = "none"
-        if lc.ff:
+        if lc.ff_kind == "moe" or lc.ff:
+            L.norm2, L.norm2b = self._gain(p + "norm2"), second(p + "norm2b")
+        if lc.ff_kind == "moe":
+            self._load_experts(L, p, lc.moe)
+        elif lc.ff:
             L.mlp_kind = "llama"
-            L.norm2, L.norm2b = self._gain(p + "norm2"), self._gain(p + "norm2b")
             r = self._ffn_range(lc.ff)
             n = r[1] - r[0]
-            np_ = _up(n, 8) if self.device.type == "cuda" else n
+            np_ = self._ff_size(n)
             gate, up = (_pad(self.src.matrix(p + "mlp." + x, (lc.ff, self.W), rows=r), np_, self.WP) for x in ("gate", "up"))
             L.gate_up = make_linear(torch.cat([gate, up]), self.kind)
             L.down = make_linear(_pad(self.src.matrix(p + "mlp.down", (self.W, lc.ff), cols=r), self.WP, np_), self.kind)
             L.act = "silu"
         return L
 
+    def _ff_size(self, n: int) -> int:
+        return _up(n, 8) if self.device.type == "cuda" else n
+
+    def _load_attention(self, L: Layer, p: str, q, kv) -> None:
+        m = L.mix
+        L.kd, L.vd = self._head_size(m.dim), self._head_size(m.vdim)
+        if self.pad_heads:
+            L.kd = L.vd = max(L.kd, L.vd)         # the tensor-core kernels have one size for keys and values
+        parts = [self._rows(p + "mix.q", m.heads, q, (m.dim, L.kd))]
+        if L.own_kv:
+            parts.append(self._rows(p + "mix.k", m.kv_heads, kv, (m.dim, L.kd)))
+            parts.append(self._rows(p + "mix.v", m.kv_heads, kv, (m.vdim, L.vd)))
+        L.qkv = make_linear(torch.cat(parts), self.kind)
+        L.sinks = None
+        if self.spec.sinks and (self.src.exists(p + "mix.sink") or self.src.fake):
+            L.sinks = self.src.vector(p + "mix.sink", m.heads, rng=q).contiguous()
+        self._out_rows(L, p, m.heads, q, m.vdim)
+
+    def _load_latent(self, L: Layer, p: str, q) -> None:
+        """Latent attention: heads are split over ranks, the latents (one row per token) are on every rank."""
+        m = L.mix
+        size = (lambda n: _up(n, 64)) if self.pad_heads else (lambda n: n)
+        d = L.dims = ops.LatentDims(L.hq, size(m.dim), size(m.rot_dim), size(m.kv_rank), size(m.vdim), L.own_kv, m.gate, m.kv_rank)
+        L.kd, L.vd = d.rank + d.rot, d.vdim
+        parts = [self._rows(p + "mix.q", m.heads, q, (m.dim, d.dim), (m.rot_dim, d.rot))]
+        L.latent_norm = None
+        if L.own_kv:
+            parts.append(self._rows(p + "mix.dkv", 1, (0, 1), (m.kv_rank, d.rank), (m.rot_dim, d.rot)))
+            L.latent_norm = _pad(self.src.vector(p + "mix.dkv.norm", m.kv_rank, fake_ones=True), d.rank)
+        if d.gate:
+            parts.append(self._rows(p + "mix.g", m.heads, q, (m.vdim, d.vdim)))
+        L.qkv = make_linear(torch.cat(parts), self.kind)
+
+        def per_head(name, n, padded):
+            w = self.src.matrix(p + name, (m.heads * n, m.kv_rank), rows=(q[0] * n, q[1] * n))
+            return _pad(w.view(L.hq, n, m.kv_rank), L.hq, padded, d.rank).to(self.act_dtype)
+        L.up = ops.LatentWeights(per_head("mix.uk", m.dim, d.dim), per_head("mix.uv", m.vdim, d.vdim))
+        self._out_rows(L, p, m.heads, q, m.vdim)
+
+    def _load_experts(self, L: Layer, p: str, f: MoeConfig) -> None:
+        """Router and experts; an expert's width is split over tensor-parallel ranks (whole experts with XFT_EXPERT_PARALLEL)."""
+        L.mlp_kind, L.moe, L.act = "moe", f, f.act
+        kind = "fp32" if self.exact or self.device.type == "cpu" else "bf16"
+        L.router = make_linear(_pad(self.src.matrix(p + "mlp.router", (f.experts, self.W)), f.experts, self.WP), kind)
+
+        def pair(name, ff, r):
+            n = self._ff_size(r[1] - r[0])
+            return (make_linear(_pad(self.src.matrix(p + name + ".up", (ff, self.W), rows=r), n, self.WP), self.kind),
+                    make_linear(_pad(self.src.matrix(p + name + ".down", (self.W, ff), cols=r), self.WP, n), self.kind))
+        L.e0, L.e1 = self._local_experts(f.experts)
+        r = (0, f.ff) if self.ctx.ep_size > 1 else self._ffn_range(f.ff)
+        L.experts = [pair(f"mlp.e{e}", f.ff, r) for e in range(L.e0, L.e1)]
+        L.shared = pair("mlp.shared", f.shared, self._ffn_range(f.shared)) if f.shared else None
+
     # ------------------------------------------------------------------------------------
     # forward
     # ------------------------------------------------------------------------------------
     def _mixer(self, L: Layer, h: torch.Tensor, b: Batch, cache: PagedKVCache) -> torch.Tensor:
-        """Attention sublayer: normalised input -> output projection (summed over tensor-parallel ranks)."""
+        """Token-mixing sublayer: normalised input -> output projection (summed over tensor-parallel ranks)."""
+        a = (self._latent if L.mix.kind == "latent" else self._attend)(L, h, b, cache)
+        with TimeLine("Output"):
+            return self._row_parallel(a, L.o, None, None)
+
+    def _latent(self, L: Layer, h: torch.Tensor, b: Batch, cache: PagedKVCache) -> torch.Tensor:
+        m, pool = L.mix, cache.k[L.pool]
+        with TimeLine("QKV.linear"):
+            x = ops.linear(h, L.qkv)
+        with TimeLine("QKPO"):
+            ops.latent_prep(x, L.dims, b.positions, self._rope(m.rot, 0), m.rot.dims if m.rot is not None else 0, L.latent_norm,
+                            self.eps, pool, b.slots)
+        with TimeLine("MHA"):
+            return ops.latent_attention(x, L.dims, pool, b.block_table, b.cu_q, b.kv_lens, L.up, m.scale, m.window, meta=b)
+
+    def _attend(self, L: Layer, h: torch.Tensor, b: Batch, cache: PagedKVCache) -> torch.Tensor:
         m, li = L.mix, L.pool
         kc, vc, ks, vs = cache.k[li], cache.v[li], cache.ks[li], cache.vs[li]
         table, rot = self._rope(m.rot, 0), m.rot.dims if m.rot is not None else 0
+        style = m.rot.style if m.rot is not None else "half"
         new_kv = L.hkv if L.own_kv else 0
-        if h.is_cuda and not self.exact and ops.can_fuse_qkv_rope(L.qkv, h.shape[0], L.kd, kc, ks, None, None, "half"):
+        if h.is_cuda and not self.exact and ops.can_fuse_qkv_rope(L.qkv, h.shape[0], L.kd, kc, ks, None, None, style):
             with TimeLine("QKV.linear+QKPO"):
-                q = ops.qkv_linear_rope_cache(h, L.qkv, None, None, L.hq, new_kv, b.positions, table, rot, "half", kc, vc,
+                q = ops.qkv_linear_rope_cache(h, L.qkv, None, None, L.hq, new_kv, b.positions, table, rot, style, kc, vc,
                                               b.slots)
         else:
             with TimeLine("QKV.linear"):
                 qkv = ops.linear(h, L.qkv)
             with TimeLine("QKPO"):
-                q = ops.qkv_rope_cache(qkv, L.hq, new_kv, L.kd, b.positions, table, rot, "half", kc, vc, ks, vs, b.slots,
+                q = ops.qkv_rope_cache(qkv, L.hq, new_kv, L.kd, b.positions, table, rot, style, kc, vc, ks, vs, b.slots,
                                        dv=L.vd)
         with TimeLine("MHA"):
             a = ops.paged_attention(q, kc, vc, b.block_table, b.cu_q, b.kv_lens, m.scale, ks, vs, group=L.group,
                                     q_off=L.q_off, meta=b, softcap=m.softcap, window=m.window, keep_first=m.keep_first,
                                     sinks=L.sinks)
-        with TimeLine("Output"):
-            return self._row_parallel(a.reshape(a.shape[0], -1), L.o, None, None)
+        return a.reshape(a.shape[0], -1)
 
     def _ff(self, L: Layer, h: torch.Tensor) -> torch.Tensor:
+        if L.mlp_kind == "moe":
+            with TimeLine("MoE"):
+                return self._experts(L, h)
         with TimeLine("LlamaMLP"):
             return self._row_parallel(ops.linear_gated(h, L.gate_up, L.act), L.down, None, None)
+
+    def _experts(self, L: Layer, h: torch.Tensor) -> torch.Tensor:
+        """Mixture of experts -> fp32 rows (summed over tensor-parallel ranks)."""
+        f = L.moe
+        logits = ops.linear(h, L.router, out_dtype=torch.float32)
+        idx, w = ops.route(logits, "deepseek", f.top, norm_topk=True, scoring="softmax")
+        shared = None
+        if L.shared is not None:
+            shared = ops.linear(ops.linear(h, L.shared[0], act=L.act), L.shared[1], out_dtype=torch.float32)
+        out = ops.moe_experts(h, idx, w, L.experts, L.act, L.e0, gated=False, add=shared)
+        if self.tp > 1:
+            peer = getattr(self.ctx, "peer", None)
+            if peer is not None and out.is_cuda and out.numel() <= peer.slot:
+                return peer.all_reduce(out.contiguous())
+            return self.ctx.all_reduce(out)
+        return out
 
     def _add_norm(self, x, y, post, nxt, **kw):
         return ops.residual_norm(x, y, post, nxt, self.eps, self.spec.norm, h_dtype=self.act_dtype, **kw)
@@ -225,7 +326,7 @@ class LayeredDecoder(Decoder):
         with TimeLine("Decoder.forward"):
             first = self.layers[0].norm1
             if self.first_stage:
-                x, h = self._add_norm(None, None, None, first, ids=b.ids, table=self.wte)
+                x, h = self._add_norm(None, None, None, first, ids=b.ids, table=self.wte, embed_scale=self.cfg.embed_scale)
             else:
                 x, h = self._add_norm(hidden, None, None, first)
             if dbg:
@@ -234,7 +335,7 @@ class LayeredDecoder(Decoder):
                 last = n + 1 == len(self.layers)
                 after = None if last else self.layers[n + 1].norm1
                 y, post = self._mixer(L, h, b, cache), L.norm1b
-                if L.ff:
+                if L.mlp_kind != "none":
                     x, h = self._add_norm(x, y, post, L.norm2)
                     if dbg:
                         debugger.dump(f"layer{L.idx}_attn_out", x[:, :self.W], self.ctx.rank, step)
@@ -260,5 +361,5 @@ class LayeredDecoder(Decoder):
 
     def kv_geometry(self):
         own = [L for L in self.layers if L.own_kv]
-        return dict(kv_heads=own[0].hkv, k_dim=own[0].kd, v_dim=own[0].vd, latent=False,
-                    layers=[(L.hkv, L.kd, L.vd) for L in own])
+        pools = [(1, L.kd, 0) if L.mix.kind == "latent" else (L.hkv, L.kd, L.vd) for L in own]
+        return dict(kv_heads=pools[0][0], k_dim=pools[0][1], v_dim=pools[0][2], latent=False, layers=pools)

@@ -32,6 +32,8 @@ class FamilySpec:
     embed_dtype: str = "same"
     layered: bool = False           # sizes and mixers per layer (`ModelConfig.layers`), safetensors weights
     post_norm: bool = False         # a second norm after each sublayer, before the residual sum
+    sinks: bool = False             # one softmax sink per attention head
+    tied_head: bool = False         # logits are products with the embedding table
 
 
 FAMILIES: Dict[str, FamilySpec] = {
@@ -52,7 +54,8 @@ FAMILIES: Dict[str, FamilySpec] = {
     "chatglm4": FamilySpec("chatglm4", rope="interleaved", rot_frac=0.5, qkv_bias=True, mlp="chatglm2"),
     "gpt": FamilySpec("gpt", norm="layer", rope="none", qkv_bias=True, dense_bias=True, mlp="gpt", embedding="opt"),
     "telechat": FamilySpec("telechat", dense_bias=True, telechat_ntk=True),
-    "kafipel": FamilySpec("kafipel", norm="layer", layered=True, post_norm=True),
+    "kafipel": FamilySpec("kafipel", norm="layer", layered=True, post_norm=True, sinks=True),
+    "vepivik": FamilySpec("vepivik", layered=True, tied_head=True),
 }
 
 

@@ -6,6 +6,7 @@ kernel for the requested variant, the call raises.
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Optional, Sequence
 
 import torch
@@ -21,6 +22,11 @@ def _nat():
         import importlib
         _native = importlib.import_module(__name__ + ".native")
     return _native
+
+
+def _nat_latent():
+    from . import native_latent
+    return native_latent
 
 
 def _cuda(t: torch.Tensor) -> bool:
@@ -46,13 +52,14 @@ def layernorm(x, w, b, eps):
     return R.layernorm(x, w, b, eps)
 
 
-def residual_norm(x, y, post, nxt, eps, kind="layer", rows=None, h_dtype=torch.bfloat16, ids=None, table=None, keep_x=True):
-    """One step of a 32-bit residual stream in one launch: x (or table[ids]) += norm(y) with `post` = (gain, bias or
+def residual_norm(x, y, post, nxt, eps, kind="layer", rows=None, h_dtype=torch.bfloat16, ids=None, table=None, keep_x=True,
+                  embed_scale=1.0):
+    """One step of a 32-bit residual stream in one launch: x (or table[ids] * embed_scale) += norm(y) with `post` = (gain, bias or
     None) (plain y without it), then h = norm(x) with `nxt` for the next product.  Returns (x, h); on a GPU x is updated
     in place unless `rows` selects rows, and buffers are as wide as x (a multiple of 8, padding zero)."""
     if _cuda(x if x is not None else table):
-        return _nat().residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids, table, keep_x)
-    return R.residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids, table, keep_x)
+        return _nat().residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids, table, keep_x, embed_scale)
+    return R.residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids, table, keep_x, embed_scale)
 
 
 # -- GEMMs ---------------------------------------------------------------------------------
@@ -225,6 +232,72 @@ def mla_prep(q, kv, Hl, nope, rope, kvl, positions, table, kv_norm_w, eps, cache
     return q3[..., :nope].contiguous(), q_rope.contiguous()
 
 
+@dataclass(frozen=True)
+class LatentDims:
+    """Sizes of a latent-attention layer as its kernels see them (heads of this rank; sizes possibly padded with zeros).
+    A packed row is [q: heads x (dim + rot) | latent: rank + rot (unless the layer reads another's) | gate: heads x vdim]."""
+    heads: int
+    dim: int                    # unrotated query/key dimensions per head
+    rot: int                    # rotated dimensions per head
+    rank: int                   # latent
+    vdim: int
+    own_kv: bool
+    gate: bool
+    rank_real: int              # values of the latent that are not padding (the norm's count)
+
+    @property
+    def q_width(self) -> int:
+        return self.heads * (self.dim + self.rot)
+
+    @property
+    def gate_at(self) -> int:
+        return self.q_width + (self.rank + self.rot if self.own_kv else 0)
+
+    @property
+    def row(self) -> int:
+        return self.gate_at + (self.heads * self.vdim if self.gate else 0)
+
+
+def latent_prep(x, dims: LatentDims, positions, table, rot_dims, norm_w, eps, cache, slots):
+    """What sits between the packed projection x [T, dims.row] of a latent-attention layer and its attention: rotates the
+    rotated part of every query in place (interleaved pairs, the first `rot_dims`), and, for a layer with a cache of its
+    own, appends [RMS-normed latent | rotated key part] to `cache` [blocks, 1, block, rank + rot] at `slots`."""
+    if _cuda(x):
+        return _nat_latent().latent_prep(x, dims, positions, table, rot_dims, norm_w, eps, cache, slots)
+    d, T = dims, x.shape[0]
+    q = x[:, :d.q_width].view(T, d.heads, d.dim + d.rot)
+    kr = x[:, d.q_width + d.rank:d.q_width + d.rank + d.rot].reshape(T, 1, d.rot) if d.own_kv else None
+    if table is not None and rot_dims > 0:
+        qr, kr = R.rope_apply(q[..., d.dim:], kr, positions, table, rot_dims, "interleaved")
+        q[..., d.dim:] = qr
+    if d.own_kv:
+        c = x[:, d.q_width:d.q_width + d.rank].float()
+        n = c * torch.rsqrt(c.pow(2).sum(-1, keepdim=True) / d.rank_real + eps) * norm_w
+        latent_cache_write(torch.cat([n.to(x.dtype), kr.reshape(T, d.rot)], -1), cache, slots)
+
+
+def latent_attention(x, dims: LatentDims, cache, block_table, cu_q, kv_lens, weights, scale, window=0, meta=None):
+    """Attention of the packed rows x (after `latent_prep`) over a latent cache -> [T, heads * vdim], multiplied with the
+    sigmoid of the rows' gate.  `weights`: `LatentWeights`.  `window` as in `paged_attention`."""
+    if _cuda(x):
+        return _nat_latent().latent_attention(x, dims, cache, block_table, cu_q, kv_lens, weights, scale, window, meta)
+    d, T = dims, x.shape[0]
+    q = x[:, :d.q_width].view(T, d.heads, d.dim + d.rot)
+    a = R.mla_attention(q[..., :d.dim], q[..., d.dim:], cache, block_table, cu_q, kv_lens, weights.uk, weights.uv, scale,
+                        max(cu_q[i + 1] - cu_q[i] for i in range(len(kv_lens))) == 1, window).reshape(T, -1)
+    if d.gate:
+        a = (a.float() * torch.sigmoid(x[:, d.gate_at:d.gate_at + d.heads * d.vdim].float())).to(a.dtype)
+    return a
+
+
+class LatentWeights:
+    """The per-head matrices of a latent-attention layer: uk [heads, dim, rank], uv [heads, vdim, rank]."""
+
+    def __init__(self, uk, uv):
+        self.uk, self.uv = uk.contiguous(), uv.contiguous()
+        self.cache: dict = {}               # layouts the kernels want, made once
+
+
 # -- MoE -----------------------------------------------------------------------------------
 def route(logits, kind, top_k, bias=None, n_group=1, topk_group=1, routed_scaling=1.0, norm_topk=True,
           scoring="sigmoid"):
@@ -239,10 +312,12 @@ def route(logits, kind, top_k, bias=None, n_group=1, topk_group=1, routed_scalin
     raise ValueError(kind)
 
 
-def moe_experts(x, idx, w, experts, act="silu", expert_offset=0, packed=None, expected_pairs=None):
+def moe_experts(x, idx, w, experts, act="silu", expert_offset=0, packed=None, expected_pairs=None, gated=True, add=None):
+    """Weighted sum of the chosen experts' outputs (see `reference.moe_experts`) in fp32, plus `add` [T, H] fp32."""
     if _cuda(x):
-        return _nat().moe_experts(x, idx, w, experts, act, expert_offset, packed, expected_pairs)
-    return R.moe_experts(x, idx, w, experts, act, expert_offset)
+        return _nat().moe_experts(x, idx, w, experts, act, expert_offset, packed, expected_pairs, gated, add)
+    out = R.moe_experts(x, idx, w, experts, act, expert_offset, gated)
+    return out if add is None else out + add
 
 
 # -- sampling ------------------------------------------------------------------------------

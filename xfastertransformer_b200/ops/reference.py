@@ -72,11 +72,11 @@ def _norm(xf: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor], eps: flo
 
 
 def residual_norm(x, y, post, nxt, eps: float, kind: str = "layer", rows: Optional[torch.Tensor] = None,
-                  h_dtype: torch.dtype = torch.float32, ids=None, table=None, keep_x: bool = True):
-    """One step of a 32-bit residual stream: x (or table[ids]) plus y — normalised with `post` = (gain, bias) first, when
+                  h_dtype: torch.dtype = torch.float32, ids=None, table=None, keep_x: bool = True, embed_scale: float = 1.0):
+    """One step of a 32-bit residual stream: x (or table[ids] * embed_scale) plus y — normalised with `post` = (gain, bias) first, when
     given — and the input of the next sublayer, h = norm(x) with `nxt` = (gain, bias).  `rows` selects rows.  Returns
     (x or None, h or None)."""
-    xf = table[ids.long()].float() if ids is not None else x.float()
+    xf = table[ids.long()].float() * embed_scale if ids is not None else x.float()
     yf = None if y is None else y.float()
     if rows is not None:
         xf = xf[rows.long()]
@@ -192,6 +192,8 @@ def _act(y: torch.Tensor, act: Optional[str]) -> torch.Tensor:
         return F.silu(y)
     if act in ("gelu", "gelu_tanh", "gelu_new", "gelu_pytorch_tanh"):
         return F.gelu(y, approximate="tanh")
+    if act == "relu2":
+        return F.relu(y).square()
     if act == "gelu_erf":
         return F.gelu(y)
     raise ValueError(act)
@@ -457,12 +459,13 @@ def paged_attention(q: torch.Tensor, kc: torch.Tensor, vc: torch.Tensor, block_t
 # ----------------------------------------------------------------------------------------
 def mla_attention(q_nope: torch.Tensor, q_rope: torch.Tensor, latent_cache: torch.Tensor,
                   block_table: torch.Tensor, cu_q, kv_lens, w_uk: torch.Tensor, w_uv: torch.Tensor,
-                  scale: float, absorbed: bool = True) -> torch.Tensor:
+                  scale: float, absorbed: bool = True, window: int = 0) -> torch.Tensor:
     """DeepSeek MLA over the latent cache (c_kv[kv_lora] ‖ k_rope[rope] per token).
 
     q_nope [T,H,nope], q_rope [T,H,rope]; w_uk [H,nope,kv_lora], w_uv [H,v,kv_lora].
     absorbed:   S = (q_nope·W_uk)·c_kvᵀ + q_rope·k_ropeᵀ ; O = (softmax(S)·c_kv)·W_uvᵀ
     otherwise:  K_nope = c_kv·W_ukᵀ, V = c_kv·W_uvᵀ are materialised (prefill form).
+    `window` > 0: position i sees the keys j <= i with i - j < window.
     Reference: crossAttnByHead_DS (attention_kernels.h:1132-1281), selfAttention_MLA (:569-766).
     """
     T, H, nope = q_nope.shape
@@ -487,7 +490,10 @@ def mla_attention(q_nope: torch.Tensor, q_rope: torch.Tensor, latent_cache: torc
         s = s * scale
         qpos = torch.arange(n - ql, n, device=s.device)
         kpos = torch.arange(n, device=s.device)
-        s = s.masked_fill((kpos[None, :] > qpos[:, None])[None], float("-inf"))
+        mask = kpos[None, :] > qpos[:, None]
+        if window > 0:
+            mask = mask | (qpos[:, None] - kpos[None, :] >= window)
+        s = s.masked_fill(mask[None], float("-inf"))
         p = torch.softmax(s, -1)
         if absorbed:
             o = torch.matmul(torch.matmul(p, ckv), w_uv.float().transpose(1, 2))   # [H,ql,v]
@@ -542,9 +548,10 @@ def route_deepseek(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: in
 
 
 def moe_experts(x: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, experts, act: str = "silu",
-                expert_offset: int = 0) -> torch.Tensor:
+                expert_offset: int = 0, gated: bool = True) -> torch.Tensor:
     """sum_k w[t,k] * down_e(act(gate_e x) * up_e x) over the experts in `experts`
-    (list of (gate_up LinearWeight, down LinearWeight), global id = expert_offset+i).
+    (list of (gate_up LinearWeight, down LinearWeight), global id = expert_offset+i); without `gated`,
+    down_e(act(up_e x)) and the first weight of a pair is up alone.
     Experts with no token are skipped (gather -> MLP -> weighted scatter-add:
     moe_deepseek.h:380-398, mlp_mixtral.h:204-219).  Returns fp32 [T, hidden]."""
     T = x.shape[0]
@@ -554,7 +561,7 @@ def moe_experts(x: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, experts, ac
         tok, slot = (idx == e).nonzero(as_tuple=True)
         if tok.numel() == 0:
             continue
-        h = linear_gated(x[tok], gu, act)
+        h = linear_gated(x[tok], gu, act) if gated else linear(x[tok], gu, act=act)
         y = linear(h, dn, out_dtype=torch.float32)
         if out is None:
             out = torch.zeros(T, y.shape[-1], dtype=torch.float32, device=x.device)

@@ -72,7 +72,9 @@ class Model:
                 raise ValueError("the 32-bit path keeps its KV cache in fp32")
             kv_cache_dtype = "fp32" if kv_cache_dtype != "int8" else "int8"
         if layered and self.ctx.dp_size > 1:
-            raise ValueError("XFT_ATTENTION_DP=1 is for mixture-of-experts models")
+            raise ValueError("XFT_ATTENTION_DP=1 does not run layered designs")
+        if layered and kv_cache_dtype == "int8" and any(l.mixer.kind == "latent" for l in self.cfg.layers):
+            raise ValueError("latent attention keeps its cache in the activation type: kv_cache_dtype int8 is not for it")
         if self.cfg.model_type == "deepseek_moe" and d_prefill not in ("bf16", "fp8_e4m3"):
             raise ValueError("deepseek_moe supports bf16 and fp8_e4m3 only")      # model_factory.h:105-114
         if d_prefill == "fp8_e4m3" and self.cfg.model_type != "deepseek_moe":

@@ -10,7 +10,7 @@ reorder and prefix sharing physically copy rows (``kvcache_tensor.h:146-289``,
   parallel fp32 scale ``[num_blocks, kv_heads, block]`` — one scale per token·head exactly like
   the reference's int8 cache, ``kvcache_tensor.h:100-104``); MLA models keep a single latent pool
   ``[num_blocks, 1, block, kv_lora+rope]``.
-* layered designs give every pool its own ``(kv_heads, k_dim, v_dim)``; a layer that reads another layer's keys and
+* layered designs give every pool its own ``(kv_heads, k_dim, v_dim)``, ``v_dim`` 0 for a latent pool; a layer that reads another layer's keys and
   values has no pool at all (the decoder maps it to the pool it reads);
 * a sequence is a list of block ids; blocks are reference-counted so a shared prefix or a beam
   fork is a table copy, and beam reorder is a permutation of tables (no data moves unless the
@@ -141,7 +141,7 @@ class PagedKVCache:
         self.max_blocks = max_blocks             # > 0: the pools never grow past this many blocks
         self.block = block_size
         self.device = device
-        self.latent = latent                     # MLA: single pool, no V
+        self.latent = latent                     # MLA: every pool is a latent one (v_dim 0: no V)
         self.int8 = dtype == "int8"
         if self.int8:
             self.dtype = torch.int8
@@ -169,7 +169,7 @@ class PagedKVCache:
         e = torch.empty((), dtype=self.dtype).element_size()
         n = 0
         for H, kd, vd in self.geometry:
-            n += H * self.block * (kd + (0 if self.latent else vd)) * e + (2 * H * self.block * 4 if self.int8 else 0)
+            n += H * self.block * (kd + vd) * e + (2 * H * self.block * 4 if self.int8 else 0)
         return n
 
     def ensure_blocks(self, total: int) -> None:
@@ -184,7 +184,7 @@ class PagedKVCache:
         for l in range(self.L):
             H, kd, vd = self.geometry[l]
             k = mk(H, kd)
-            v = None if self.latent else mk(H, vd)
+            v = mk(H, vd) if vd else None
             if old:
                 k[:old] = self.k[l]
                 if v is not None:
