@@ -189,6 +189,7 @@ __global__ void __launch_bounds__(NT) layernorm_kernel(const bf16* __restrict__ 
 // ------------------------------------------------------------------------------ gated activation (unfused fallback)
 __device__ __forceinline__ float act_fn(float x, int act) {
   if (act == 1) return fmaxf(x, 0.f);
+  if (act == 4) { const float r = fmaxf(x, 0.f); return r * r; }
   if (act == 2) return x / (1.f + __expf(-x));
   if (act == 3) { float u = 0.7978845608028654f * (x + 0.044715f * x * x * x); return 0.5f * x * (1.f + tanhf(u)); }
   return x;

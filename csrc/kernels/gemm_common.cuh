@@ -45,6 +45,7 @@ __device__ __forceinline__ void ll_unpack2(unsigned w, float& lo, float& hi) {
 __device__ __forceinline__ float apply_act(float x, int act) {
   switch (act) {
     case 1: return fmaxf(x, 0.f);
+    case 4: { const float r = fmaxf(x, 0.f); return r * r; }
     case 2: return x / (1.f + __expf(-x));
     case 3: {
       const float c = 0.7978845608028654f;

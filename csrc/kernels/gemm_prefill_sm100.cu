@@ -65,6 +65,7 @@ struct PrefillParams {
 __device__ __forceinline__ float prefill_act(float x, int act) {
   switch (act) {
     case 1: return fmaxf(x, 0.f);
+    case 4: { const float r = fmaxf(x, 0.f); return r * r; }
     case 2: return x / (1.f + __expf(-x));
     case 3: {
       const float c = 0.7978845608028654f;

@@ -41,7 +41,7 @@ struct GemmParams {
   const __nv_bfloat16* residual;
   int ldr;
   float res_scale;
-  int act;                 // 0 none, 1 relu, 2 silu, 3 gelu(tanh)
+  int act;                 // 0 none, 1 relu, 2 silu, 3 gelu(tanh), 4 relu squared
   int splits, kb_per_split, num_kb;
   float* ws;               // split-K partials
   int* counters;           // one per output tile, zero between launches
@@ -55,6 +55,12 @@ struct GemmParams {
   const int* num_group_tiles;
   int group_w_rows;
   const float* col_scale;  // optional per-token factor applied to the result (routing weight)
+  // Head mode (batch_tiles > 0): tile_t = group * batch_tiles + j covers rows j * BN .. of group's operand, which is the
+  // column range starting at group * x_col_stride of X; the group's weight rows start at group * group_w_rows and its
+  // results go to columns group * y_col_stride ...  `gate` (same column layout): results are multiplied with its sigmoid.
+  int batch_tiles, x_col_stride, y_col_stride;
+  const __nv_bfloat16* gate;
+  int ldg;
   // pair != 0 (DUAL instantiation, no gating): the two accumulators are two independent 128-feature tiles
   // (rows n and n + 128 of W) sharing one token tile — 256 x BN of output per CTA, which halves the
   // operand bytes per FLOP of the compute-bound (prefill) shapes.
@@ -142,9 +148,12 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
     }
     __syncthreads();
   }
-  const int w_row0 = grouped ? s_group[0] * p.group_w_rows : 0;      // first weight row of this tile's group
-  const int x_row0 = grouped ? s_group[1] : tile_t * BN;            // first token row of this tile
-  const int x_rows = grouped ? s_group[2] : BN;                     // valid token rows in this tile
+  const int head = p.batch_tiles > 0 ? tile_t / p.batch_tiles : 0;
+  // first weight row of this tile's group, first token row of this tile, valid token rows in it, column offsets of its group
+  const int w_row0 = (grouped ? s_group[0] : head) * p.group_w_rows;
+  const int x_row0 = grouped ? s_group[1] : (tile_t - head * p.batch_tiles) * BN;
+  const int x_rows = grouped ? s_group[2] : BN;
+  const int x_col0 = head * p.x_col_stride, y_col0 = head * p.y_col_stride;
   const bool active = !grouped || x_rows > 0;
   const int tn_stride = (DUAL && p.pair) ? 256 : 128;      // output features covered per CTA
 
@@ -166,7 +175,7 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
       }
       grid_dep_wait();
       for (int i = 0; i < pre; ++i)
-        tma_load_2d(smem + i * STAGE_BYTES + A_BYTES * NACC, &tmX, &full_bar[i], (kb0 + i) * 64, x_row0, hint_x);
+        tma_load_2d(smem + i * STAGE_BYTES + A_BYTES * NACC, &tmX, &full_bar[i], x_col0 + (kb0 + i) * 64, x_row0, hint_x);
       int it = pre;
       for (int kb = kb0 + pre; kb < kend; ++kb, ++it) {
         const int s = it % stages;
@@ -176,7 +185,7 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
         uint8_t* a = smem + s * STAGE_BYTES;
         tma_load_2d(a, &tmW, &full_bar[s], kb * 64, w_row0 + tile_n * tn_stride, hint_w);
         if (DUAL) tma_load_2d(a + A_BYTES, &tmW, &full_bar[s], kb * 64, w_row0 + p.dual_off + tile_n * tn_stride, hint_w);
-        tma_load_2d(a + A_BYTES * NACC, &tmX, &full_bar[s], kb * 64, x_row0, hint_x);
+        tma_load_2d(a + A_BYTES * NACC, &tmX, &full_bar[s], x_col0 + kb * 64, x_row0, hint_x);
       }
     }
   } else if (warp == 1) {
@@ -413,11 +422,12 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
                   x = apply_act(x, p.act);
                   if (DUAL && !pair) x *= (u[j] * (rs * ts) + bias_u);
                   if (p.col_scale) x *= p.col_scale[t];
+                  if (p.gate) x = __fdividef(x, 1.f + __expf(-__bfloat162float(p.gate[(size_t)t * p.ldg + y_col0 + n])));
                   if (p.residual) x += p.res_scale * __bfloat162float(p.residual[(size_t)t * p.ldr + n]);
                   g[j] = x;                     // kept for the two-shot broadcast below
                 }
-                if (p.out_fp32) reinterpret_cast<float*>(p.out)[(size_t)t * p.ldo + n] = x;
-                else reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)t * p.ldo + n] = __float2bfloat16(x);
+                if (p.out_fp32) reinterpret_cast<float*>(p.out)[(size_t)t * p.ldo + y_col0 + n] = x;
+                else reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)t * p.ldo + y_col0 + n] = __float2bfloat16(x);
               }
             }
             if (two_shot && i_reduce) {
@@ -735,6 +745,37 @@ extern "C" int xft_gemm_bf16_grouped(const void* X, int ldx, int x_rows, const v
     XFT_LAUNCH(128)
   }
 #undef XFT_LAUNCH
+  return -1;
+}
+
+// One product per head: Y[:, h * ys + n] = sum_k X[:, h * xs + k] W[h * N + n, k] for h < heads, n < N, k < K; W is
+// [heads * N, K].  gate (bf16 [T, ldg], columns laid out as Y's) or null: results are multiplied with sigmoid(gate).
+// xs and K multiples of 8; columns of X from h * xs + K up to the next multiple of 64 are read (times zero).
+extern "C" int xft_gemm_bf16_heads(const void* X, int ldx, int x_cols, int xs, const void* W, int ldw, void* Y, int ldo, int ys,
+                                   int heads, int T, int N, int K, const void* gate, int ldg, int* status, cudaStream_t st) {
+  if (T <= 0 || N <= 0 || K <= 0 || heads <= 0) return 0;
+  if ((xs & 7) || (K & 7) || (heads - 1) * xs + K > x_cols || x_cols > ldx || (heads - 1) * ys + N > ldo) return -1;
+  GemmParams p{};
+  p.N = N; p.T = T; p.K = K; p.out = Y; p.ldo = ldo; p.res_scale = 1.f; p.status = status;
+  p.group_w_rows = N; p.x_col_stride = xs; p.y_col_stride = ys;
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate); p.ldg = ldg;
+  const int bn = min(pick_bn(T), 128);
+  p.batch_tiles = (T + bn - 1) / bn;
+  p.n_tiles = (N + 127) / 128;
+  p.t_tiles = heads * p.batch_tiles;
+  p.num_kb = (K + 63) / 64;
+  p.splits = 1; p.kb_per_split = p.num_kb;
+  CUtensorMap tmW, tmX;
+  int r = make_tensor_map(&tmW, W, (uint64_t)heads * N, (uint64_t)K, (uint64_t)ldw, 128, 2);
+  if (r) return 1000 - r;
+  r = make_tensor_map(&tmX, X, (uint64_t)T, (uint64_t)x_cols, (uint64_t)ldx, (uint32_t)bn, 2);
+  if (r) return 2000 - r;
+  switch (bn) {
+    case 16: return launch_gemm<16, false>(tmW, tmX, p, st);
+    case 32: return launch_gemm<32, false>(tmW, tmX, p, st);
+    case 64: return launch_gemm<64, false>(tmW, tmX, p, st);
+    case 128: return launch_gemm<128, false>(tmW, tmX, p, st);
+  }
   return -1;
 }
 

@@ -1,8 +1,10 @@
 // Plain kernels for any size: the 32-bit path of the layered decoder (fp32 weights, activations and cache), and what a
 // bf16 model needs when its heads are larger than the tensor-core kernels take.
 //
-//   xft_gemm_f32        Y[T, N] = X[T, K] W[N, K]^T in fp32 (no reduced-precision mode)
+//   xft_gemm_f32        Y[T, N] = act(X[T, K] W[N, K]^T) in fp32 (no reduced-precision mode); also one product per head,
+//                       and products of rows grouped by expert
 //   xft_gated_act_f32   act(gate) * up
+//   xft_sigmoid_gate    x * sigmoid(gate)
 //   xft_rope_cache      split q | k | v rows, rotate q and k, append k and v to the paged cache; key and value heads may
 //                       have different sizes
 //   xft_attention_plain one warp per (query, head): sliding window with kept first keys, capped scores, sinks
@@ -22,20 +24,45 @@ template <> __device__ __forceinline__ float from_f32<float>(float v) { return v
 template <> __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16(v); }
 
 // ------------------------------------------------------------------------------------------ GEMM
+struct GemmF32 {
+  const float* X; int ldx; const float* W; int ldw; float* Y; int ldo; int T, N, K, act;
+  long long sx, sw, sy;                        // blockIdx.z steps through a batch with these strides
+  // grouped form: blockIdx.y is a tile {group, first row, rows, -} of 64 rows; X row r comes from src[r] when given
+  const int4* tiles; const int* num_tiles; const int* src; const float* row_w; int group_w_rows;
+};
+
+__device__ __forceinline__ float act_f32(float x, int act) {
+  if (act == 1) return fmaxf(x, 0.f);
+  if (act == 2) return x / (1.f + expf(-x));
+  if (act == 3) return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+  if (act == 4) { const float r = fmaxf(x, 0.f); return r * r; }
+  return x;
+}
+
 // 64 x 64 tile of Y per CTA, 256 threads with 4 x 4 values each, 16 columns of the reduction per step.
-__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ X, int ldx, const float* __restrict__ W, int ldw,
-                                                       float* __restrict__ Y, int ldo, int T, int N, int K) {
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32 p) {
   __shared__ float xs[16][68], ws[16][68];
-  const int t0 = blockIdx.y * 64, n0 = blockIdx.x * 64, tid = threadIdx.x;
+  const float* W = p.W + blockIdx.z * p.sw;
+  int t0 = blockIdx.y * 64, rows = min(64, p.T - t0);
+  if (p.tiles) {
+    if ((int)blockIdx.y >= *p.num_tiles) return;
+    const int4 e = p.tiles[blockIdx.y];
+    t0 = e.y;
+    rows = e.z;
+    W += (size_t)e.x * p.group_w_rows * p.ldw;
+  }
+  const int n0 = blockIdx.x * 64, tid = threadIdx.x;
   const int lr = tid >> 2, lk = (tid & 3) * 4;             // this thread loads row lr, columns lk .. lk + 3
   const int tx = tid & 15, ty = tid >> 4;
+  const float* xrow = p.X + blockIdx.z * p.sx + (size_t)(lr < rows ? (p.src ? p.src[t0 + lr] : t0 + lr) : 0) * p.ldx;
+  const float* wrow = W + (size_t)(n0 + lr < p.N ? n0 + lr : 0) * p.ldw;
   float acc[4][4] = {};
-  for (int k0 = 0; k0 < K; k0 += 16) {
+  for (int k0 = 0; k0 < p.K; k0 += 16) {
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int k = k0 + lk + j;
-      xs[lk + j][lr] = (t0 + lr < T && k < K) ? X[(size_t)(t0 + lr) * ldx + k] : 0.f;
-      ws[lk + j][lr] = (n0 + lr < N && k < K) ? W[(size_t)(n0 + lr) * ldw + k] : 0.f;
+      xs[lk + j][lr] = (lr < rows && k < p.K) ? xrow[k] : 0.f;
+      ws[lk + j][lr] = (n0 + lr < p.N && k < p.K) ? wrow[k] : 0.f;
     }
     __syncthreads();
 #pragma unroll
@@ -50,12 +77,17 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
     }
     __syncthreads();
   }
+  float* Y = p.Y + blockIdx.z * p.sy;
 #pragma unroll
   for (int i = 0; i < 4; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      const int t = t0 + ty * 4 + i, n = n0 + tx * 4 + j;
-      if (t < T && n < N) Y[(size_t)t * ldo + n] = acc[i][j];
+      const int r = ty * 4 + i, n = n0 + tx * 4 + j;
+      if (r < rows && n < p.N) {
+        float v = act_f32(acc[i][j], p.act);
+        if (p.row_w) v *= p.row_w[t0 + r];
+        Y[(size_t)(t0 + r) * p.ldo + n] = v;
+      }
     }
 }
 
@@ -64,11 +96,18 @@ __global__ void gated_act_f32_kernel(const float* __restrict__ gu, int ld, float
   if (i >= (size_t)T * I) return;
   const int t = (int)(i / I), c = (int)(i % I);
   const float g = gu[(size_t)t * ld + c], u = gu[(size_t)t * ld + I + c];
-  float a = g;
-  if (act == 1) a = fmaxf(g, 0.f);
-  else if (act == 2) a = g / (1.f + expf(-g));
-  else if (act == 3) a = 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
-  out[i] = a * u;
+  out[i] = act_f32(g, act) * u;
+}
+
+// out[t, c] = x[t, c] * sigmoid(gate[t, c])
+template <typename T>
+__global__ void sigmoid_gate_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ gate, int ldg, T* __restrict__ out,
+                                    int ldo, int n_tok, int n) {
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= (size_t)n_tok * n) return;
+  const int t = (int)(i / n), c = (int)(i % n);
+  const float g = to_f32<T>(gate[(size_t)t * ldg + c]);
+  out[(size_t)t * ldo + c] = from_f32<T>(to_f32<T>(x[(size_t)t * ldx + c]) / (1.f + expf(-g)));
 }
 
 // ------------------------------------------------------------------------------------------ rotary + cache append
@@ -122,7 +161,7 @@ __global__ void __launch_bounds__(128) attention_plain_kernel(const T* __restric
                                                               const int* __restrict__ block_table, int bt_stride,
                                                               const int* __restrict__ cu_q, const int* __restrict__ kv_lens,
                                                               int B, int n_tok, int hq, int hkv, int group, int q_off, int kd,
-                                                              int vd, int bs, int num_blocks, float scale, float softcap,
+                                                              int vd, int vld, int bs, int num_blocks, float scale, float softcap,
                                                               int window, int keep, const float* __restrict__ sinks,
                                                               int* status) {
   extern __shared__ float sm[];
@@ -184,7 +223,7 @@ __global__ void __launch_bounds__(128) attention_plain_kernel(const T* __restric
     const int cnt = min(32, total - n0);
     for (int d = lane; d < vd; d += 32) {
       float a = acc[d] * c;
-      for (int i = 0; i < cnt; ++i) a = fmaf(ps[i], to_f32<T>(vc[(size_t)rs[i] * vd + d]), a);
+      for (int i = 0; i < cnt; ++i) a = fmaf(ps[i], to_f32<T>(vc[(size_t)rs[i] * vld + d]), a);
       acc[d] = a;
     }
     __syncwarp();
@@ -196,13 +235,50 @@ __global__ void __launch_bounds__(128) attention_plain_kernel(const T* __restric
 
 using namespace xft;
 
-extern "C" int xft_gemm_f32(const float* X, int ldx, const float* W, int ldw, float* Y, int ldo, int T, int N, int K,
+// act: 0 none, 1 relu, 2 silu, 3 gelu (tanh), 4 relu squared
+extern "C" int xft_gemm_f32(const float* X, int ldx, const float* W, int ldw, float* Y, int ldo, int T, int N, int K, int act,
                             cudaStream_t st) {
   if (T <= 0 || N <= 0) return 0;
   if (K <= 0 || ldx < K || ldw < K || ldo < N) return -1;
   const int ty = (T + 63) / 64;
   if (ty > 65535) return -2;
-  gemm_f32_kernel<<<dim3((N + 63) / 64, ty), 256, 0, st>>>(X, ldx, W, ldw, Y, ldo, T, N, K);
+  GemmF32 p{X, ldx, W, ldw, Y, ldo, T, N, K, act};
+  gemm_f32_kernel<<<dim3((N + 63) / 64, ty), 256, 0, st>>>(p);
+  return (int)cudaGetLastError();
+}
+
+// One product per head: Y[:, h * ys + n] = sum_k X[:, h * xs + k] W[h * N + n, k]; W [heads * N, K].
+extern "C" int xft_gemm_f32_heads(const float* X, int ldx, int xs, const float* W, float* Y, int ldo, int ys, int heads, int T,
+                                  int N, int K, cudaStream_t st) {
+  if (T <= 0 || N <= 0 || heads <= 0) return 0;
+  if (K <= 0 || ldx < (heads - 1) * xs + K || ldo < (heads - 1) * ys + N || heads > 65535) return -1;
+  const int ty = (T + 63) / 64;
+  if (ty > 65535) return -2;
+  GemmF32 p{X, ldx, W, K, Y, ldo, T, N, K, 0, xs, (long long)N * K, ys};
+  gemm_f32_kernel<<<dim3((N + 63) / 64, ty, heads), 256, 0, st>>>(p);
+  return (int)cudaGetLastError();
+}
+
+// Products of rows sorted by group (experts): tiles of 64 rows from xft_moe_plan; src: row r is X[src[r]] (null: X[r]);
+// row_w: factor of a row's result (null: none).  W [groups * group_w_rows, K].
+extern "C" int xft_gemm_f32_grouped(const float* X, int ldx, const float* W, int ldw, float* Y, int ldo, int N, int K,
+                                    int group_w_rows, const void* tiles, const int* num_tiles, int max_tiles, const int* src,
+                                    const float* row_w, int act, cudaStream_t st) {
+  if (max_tiles <= 0 || N <= 0) return 0;
+  if (K <= 0 || ldx < K || ldw < K || ldo < N || max_tiles > 65535) return -1;
+  GemmF32 p{X, ldx, W, ldw, Y, ldo, 0, N, K, act, 0, 0, 0, (const int4*)tiles, num_tiles, src, row_w, group_w_rows};
+  gemm_f32_kernel<<<dim3((N + 63) / 64, max_tiles), 256, 0, st>>>(p);
+  return (int)cudaGetLastError();
+}
+
+extern "C" int xft_sigmoid_gate(const void* x, int ldx, const void* gate, int ldg, void* out, int ldo, int T, int n, int f32,
+                                cudaStream_t st) {
+  const size_t m = (size_t)T * n;
+  if (!m) return 0;
+  if (ldx < n || ldg < n || ldo < n) return -1;
+  const unsigned grid = (unsigned)((m + 255) / 256);
+  if (f32) sigmoid_gate_kernel<float><<<grid, 256, 0, st>>>((const float*)x, ldx, (const float*)gate, ldg, (float*)out, ldo, T, n);
+  else sigmoid_gate_kernel<bf16><<<grid, 256, 0, st>>>((const bf16*)x, ldx, (const bf16*)gate, ldg, (bf16*)out, ldo, T, n);
   return (int)cudaGetLastError();
 }
 
@@ -233,14 +309,14 @@ extern "C" int xft_rope_cache(const void* qkv, int ldq, int T, int hq, int hkv, 
   return (int)cudaGetLastError();
 }
 
-// q [T, hq, kd], caches [num_blocks, hkv, bs, kd] and [num_blocks, hkv, bs, vd], out [T, hq, vd], all fp32 (f32 = 1) or
-// bf16.  window 0: every earlier key; softcap 0: none; sinks null: none.
+// q [T, hq, kd], caches [num_blocks, hkv, bs, kd] and [num_blocks, hkv, bs, vld], out [T, hq, vd], all fp32 (f32 = 1) or
+// bf16; values are the first vd of vld columns (latent attention: vc = kc, vld = kd).  window 0: every earlier key; softcap 0: none; sinks null: none.
 extern "C" int xft_attention_plain(const void* q, void* out, const void* kc, const void* vc, const int* block_table,
                                    int bt_stride, const int* cu_q, const int* kv_lens, int B, int T, int hq, int hkv, int group,
-                                   int q_off, int kd, int vd, int bs, int num_blocks, float scale, float softcap, int window,
-                                   int keep, const float* sinks, int f32, int* status, cudaStream_t st) {
+                                   int q_off, int kd, int vd, int vld, int bs, int num_blocks, float scale, float softcap,
+                                   int window, int keep, const float* sinks, int f32, int* status, cudaStream_t st) {
   if (B <= 0 || T <= 0) return 0;
-  if (hq <= 0 || hkv <= 0 || group <= 0 || kd <= 0 || vd <= 0 || bs <= 0 || softcap < 0.f || window < 0 || keep < 0) return -1;
+  if (hq <= 0 || hkv <= 0 || group <= 0 || kd <= 0 || vd <= 0 || vld < vd || bs <= 0 || softcap < 0.f || window < 0 || keep < 0) return -1;
   if ((long long)num_blocks * hkv * bs >= (1ll << 31)) return -2;
   const size_t smem = (size_t)4 * (kd + vd + 64) * sizeof(float);
   if (smem > 200 * 1024) return -3;
@@ -251,12 +327,12 @@ extern "C" int xft_attention_plain(const void* q, void* out, const void* kc, con
     if (smem > 48 * 1024) cudaFuncSetAttribute(attention_plain_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     attention_plain_kernel<float><<<grid, 128, smem, st>>>((const float*)q, (float*)out, (const float*)kc, (const float*)vc,
                                                            block_table, bt_stride, cu_q, kv_lens, B, T, hq, hkv, group, q_off,
-                                                           kd, vd, bs, num_blocks, scale, softcap, win, kp, sinks, status);
+                                                           kd, vd, vld, bs, num_blocks, scale, softcap, win, kp, sinks, status);
   } else {
     if (smem > 48 * 1024) cudaFuncSetAttribute(attention_plain_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     attention_plain_kernel<bf16><<<grid, 128, smem, st>>>((const bf16*)q, (bf16*)out, (const bf16*)kc, (const bf16*)vc,
                                                           block_table, bt_stride, cu_q, kv_lens, B, T, hq, hkv, group, q_off,
-                                                          kd, vd, bs, num_blocks, scale, softcap, win, kp, sinks, status);
+                                                          kd, vd, vld, bs, num_blocks, scale, softcap, win, kp, sinks, status);
   }
   return (int)cudaGetLastError();
 }

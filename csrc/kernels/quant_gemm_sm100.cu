@@ -55,6 +55,7 @@ struct QGemmParams {
 
 __device__ __forceinline__ float q_act(float x, int act) {
   if (act == 1) return fmaxf(x, 0.f);
+  if (act == 4) { const float r = fmaxf(x, 0.f); return r * r; }
   if (act == 2) return x / (1.f + __expf(-x));
   if (act == 3) { float u = 0.7978845608028654f * (x + 0.044715f * x * x * x); return 0.5f * x * (1.f + tanhf(u)); }
   return x;

@@ -3,7 +3,7 @@
 //   x <- x + post(y)        y = output of the sublayer just finished; post = a norm with its own gain, or nothing
 //   h <- next(x)            input of the sublayer that follows, for the next product (bf16 or fp32)
 //
-// and, for the first layer, x <- table[id] instead of the first line.  The norm is LayerNorm (mean and variance) or
+// and, for the first layer, x <- table[id] * scale instead of the first line.  The norm is LayerNorm (mean and variance) or
 // RMSNorm, with a gain and an optional bias.  Either half can be left out; `rows` restricts the work to some rows of
 // the batch (the ones whose logits are wanted).  One CTA per row: the row stays in registers between the reductions,
 // so x and y are read once and x and h written once.  Row buffers may be wider than H (`HP`, a multiple of 8, so that
@@ -28,7 +28,7 @@ struct ResidualNormParams {
   const int* rows;                                                  // row r of the outputs comes from rows[r], or null
   int n_in;                                                         // rows of x and y
   int H, HP, rms;
-  float eps;
+  float eps, embed_scale;
   int* status;
 };
 
@@ -150,8 +150,11 @@ __global__ void __launch_bounds__(NT) residual_norm_kernel(const ResidualNormPar
   for (int c = 0; c < CH; ++c) {
     const int i = (threadIdx.x + c * NT) * 8;
     const int left = p.H - i;                              // <= 0: nothing of the row here
-    if (p.ids) load8(p.table + (size_t)id * p.ldt + (left > 0 ? i : 0), left, x[c]);
-    else load8(p.x + (size_t)src * p.ldx + (left > 0 ? i : 0), left, x[c]);
+    if (p.ids) {
+      load8(p.table + (size_t)id * p.ldt + (left > 0 ? i : 0), left, x[c]);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) x[c][j] *= p.embed_scale;
+    } else load8(p.x + (size_t)src * p.ldx + (left > 0 ? i : 0), left, x[c]);
     if (p.y) {
       if (p.y_f32) load8(reinterpret_cast<const float*>(p.y) + (size_t)src * p.ldy + (left > 0 ? i : 0), left, y[c]);
       else load8(reinterpret_cast<const bf16*>(p.y) + (size_t)src * p.ldy + (left > 0 ? i : 0), left, y[c]);
@@ -193,8 +196,8 @@ using namespace xft;
 extern "C" int xft_residual_norm(const int* ids, const void* table, int vocab, long long ldt, const float* x, int ldx,
                                  float* x_out, int ldxo, const void* y, int ldy, int y_f32, const float* post_w,
                                  const float* post_b, const float* next_w, const float* next_b, void* h, int ldh, int h_f32,
-                                 const int* rows, int n_in, int n_out, int H, int kind, float eps, int* status,
-                                 cudaStream_t st) {
+                                 const int* rows, int n_in, int n_out, int H, int kind, float eps, float embed_scale,
+                                 int* status, cudaStream_t st) {
   if (n_out <= 0) return 0;
   const int HP = (H + 7) / 8 * 8;
   if (H <= 0 || H > 32768 || (!ids && !x) || (h && !next_w) || (!rows && n_out > n_in)) return -1;
@@ -204,7 +207,7 @@ extern "C" int xft_residual_norm(const int* ids, const void* table, int vocab, l
        (uintptr_t)next_w | (uintptr_t)next_b | (uintptr_t)h) & 15) return -3;
   if (rows && x_out == x && x_out) return -4;              // gathered rows cannot be written back in place
   ResidualNormParams p{ids, (const bf16*)table, vocab, ldt, x, ldx, x_out, ldxo, y, ldy, y_f32, post_w, post_b, next_w,
-                       next_b, h, ldh, h_f32, rows, n_in, H, HP, kind, eps, status};
+                       next_b, h, ldh, h_f32, rows, n_in, H, HP, kind, eps, embed_scale, status};
   cudaError_t e;
 #define XFT_RN(NT, CH, PRE) e = launch_pdl(residual_norm_kernel<NT, CH, PRE>, dim3(n_out), dim3(NT), 0, st, p)
   const bool few = n_out <= 296;                           // decode: a wide CTA per row, everything in one round of loads

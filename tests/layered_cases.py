@@ -51,7 +51,34 @@ CONFIGS = {
                           ff=None),
         O.attention_layer(heads=8, kv_heads=1, dim=64, vdim=64, size=7, keep=1, rot_dims=64, softcap=13.0, kv_from=1,
                           ff=32)], width=128, vocab=220),
+    # Vepivik: both mixers, unequal sizes, a reader with other heads and another window than the layer whose latents it
+    # reads, a layer without feed-forward, one expert per token
+    "latent": O.vepivik([
+        O.window_layer(heads=6, kv_heads=3, dim=20, vdim=36, size=17, mlp=O.moe(ff=36, experts=5, top=3, shared=20)),
+        O.latent_layer(heads=3, dim=24, rot_dim=12, vdim=20, kv_rank=28, size=33, scaling=YARN, mlp=O.moe(ff=44, experts=7, top=1,
+                                                                                                        shared=12)),
+        O.latent_layer(heads=5, dim=40, rot_dim=12, vdim=12, kv_rank=28, size=70, scaling=YARN, scale=0.2, kv_from=1),
+        O.window_layer(heads=4, kv_heads=1, dim=56, vdim=16, size=70, mlp=O.moe(ff=24, experts=3, top=2, shared=60))],
+        width=90, vocab=131, eps=3e-4, scale=1.7),
+    # sizes of the kernels without padding; the expanded form's two head chunks, a window off the 64-token pages
+    "latent128": O.vepivik([
+        O.latent_layer(heads=18, dim=128, rot_dim=64, vdim=128, kv_rank=128, size=100, scaling=YARN,
+                       mlp=O.moe(ff=64, experts=6, top=2, shared=128)),
+        O.window_layer(heads=6, kv_heads=2, dim=128, vdim=128, size=65, mlp=O.moe(ff=64, experts=4, top=4, shared=64)),
+        O.latent_layer(heads=2, dim=64, rot_dim=64, vdim=64, kv_rank=256, size=64, base=500.0,
+                       mlp=O.moe(ff=128, experts=2, top=1, shared=32))], width=160, vocab=300),
+    # mechanisms left out one by one: no window, no scaling, no shared expert, every expert chosen, one head, no feed-forward
+    "latent_bare": O.vepivik([
+        O.latent_layer(heads=1, dim=16, rot_dim=2, vdim=8, kv_rank=12, mask=False, mlp=O.moe(ff=16, experts=3, top=3, shared=None)),
+        O.window_layer(heads=2, kv_heads=2, dim=32, vdim=32, mask=False, mlp=None),
+        O.latent_layer(heads=2, dim=8, rot_dim=2, vdim=64, kv_rank=12, size=1, kv_from=0, mlp=O.moe(ff=8, experts=1, top=1, shared=8)),
+        O.latent_layer(heads=2, dim=72, rot_dim=70, vdim=24, kv_rank=20, size=5000, mlp=None)], width=72, vocab=150, scale=0.5),
+    # larger than any tensor-core latent kernel takes; three key chunks of the expanded form
+    "latent_large": O.vepivik([
+        O.latent_layer(heads=2, dim=208, rot_dim=80, vdim=144, kv_rank=520, size=30, scaling=YARN, mlp=O.moe()),
+        O.latent_layer(heads=3, dim=136, rot_dim=24, vdim=72, kv_rank=300, size=41, mlp=O.moe(top=3))], width=64, vocab=83),
 }
+LATENT = ["latent", "latent128", "latent_bare", "latent_large"]
 
 TOLERANCE = {"fp32": 3e-5, "bf16": 0.05}
 
@@ -177,7 +204,8 @@ def mixed_batches(case, dtype, seed=0, lengths=(150, 97, 64, 30, 1, 129), live=3
         for b in cache.alloc.free:                       # what freed pages hold must not matter
             for pool in (cache.k, cache.v):
                 for t in pool:
-                    t[b].fill_(30.0)
+                    if t is not None:
+                        t[b].fill_(30.0)
         steps += 1
     assert cache.alloc.num_blocks == size and not cache.tables, "pools grew or requests were left behind"
     for k, rows in got.items():

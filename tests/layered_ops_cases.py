@@ -91,6 +91,145 @@ def sink_counts_once(dev, dtype, d, tol, T=150, H=3, G=1, **kw):
                     assert float(got[:, h].abs().max()) < 1e-6
 
 
+def _latent_layer(H, d, rd, R, dv, T, seed, quiet=1 / 16):
+    g = torch.Generator().manual_seed(seed)
+    r = lambda *s: torch.randn(*s, generator=g).bfloat16().float()
+    q = r(T, H, d + rd) * quiet
+    return q, r(T, R), r(T, rd), r(H, d, R) / R ** 0.5, r(H, dv, R) / R ** 0.5, r(T, H * dv)
+
+
+def latent_run(dev, dtype, q, c, kr, uk, uv, gate, scale, window, decode, start, extra=0):
+    """ops.latent_attention of queries start .. T - 1, as one portion or as decode steps that share the pages; with `extra`,
+    the portion's batch also holds `extra` short portions of two tokens (the last ones, over the same pages)."""
+    T, H, _ = q.shape
+    d, R, dv = uk.shape[1], uk.shape[2], uv.shape[1]
+    rd = kr.shape[1]
+    up = (lambda n: (n + 63) // 64 * 64) if dev.type == "cuda" and dtype == torch.bfloat16 else (lambda n: n)
+    rank = next((x for x in (64, 128, 256, 512) if R <= x), up(R)) if up(1) > 1 else R
+    dims = ops.LatentDims(H, up(d), up(rd), rank, up(dv), False, True, R)
+
+    def pad(t, *shape):
+        out = torch.zeros(*shape, dtype=t.dtype)
+        out[tuple(slice(n) for n in t.shape)] = t
+        return out
+    qp = torch.cat([pad(q[..., :d], T, H, dims.dim), pad(q[..., d:], T, H, dims.rot)], -1).reshape(T, -1)
+    x = torch.cat([qp, pad(gate.view(T, H, dv), T, H, dims.vdim).reshape(T, -1)], -1)
+    rows = torch.cat([pad(c, T, dims.rank), pad(kr, T, dims.rot)], -1)
+    pool, bt = paged(rows[:, None].to(dtype))
+    w = ops.LatentWeights(pad(uk, H, dims.dim, dims.rank).to(dtype).to(dev), pad(uv, H, dims.vdim, dims.rank).to(dtype).to(dev))
+    n = T - start
+    xs, cu, lens = x[start:], [0, n], [T]
+    if decode:
+        cu, lens = list(range(n + 1)), [i + 1 for i in range(start, T)]
+    for i in range(extra):
+        xs, cu, lens = torch.cat([xs, x[T - 2 - i:T - i]]), cu + [cu[-1] + 2], lens + [T - i]
+    xs = xs.to(dtype).to(dev).contiguous()
+    out = ops.latent_attention(xs, dims, pool.to(dev), bt.repeat(len(lens), 1).to(dev), cu, lens, w, scale, window)
+    if dev.type == "cuda":
+        from xfastertransformer_b200.ops import native
+        native.Workspace.get(dev).check_status()
+    return out.float().cpu().view(-1, H, dims.vdim)[..., :dv]
+
+
+def latent_want(q, c, kr, uk, uv, gate, scale, window):
+    a = O.latent_attention(q.double(), c.double(), kr.double(), uk.double(), uv.double(), scale, {"size": window} if window else None)
+    return (a * torch.sigmoid(gate.double()).view(a.shape)).float()
+
+
+def latent_window_edges(dev, dtype, window, decode, tol, T=200, H=3, d=24, rd=12, R=40, dv=20, extra=0):
+    """One key stands out at every distance that is special, once through the shared rotated part and once through the
+    latent: a query that sees it returns its value almost alone."""
+    q, c, kr, uk, uv, gate = _latent_layer(H, d, rd, R, dv, T, window)
+    q[..., d], kr[:, 0] = 2.0, 0.0
+    start, i = 100, T - 30
+    for j in sorted({i - window - 1, i - window, i - window + 1, 63, 64, 127, 128, 0, i}):
+        if not 0 <= j < T:
+            continue
+        k2 = kr.clone()
+        k2[j, 0] = 10.0
+        want = latent_want(q, c, k2, uk, uv, gate, 1.0, window)
+        got = latent_run(dev, dtype, q, c, k2, uk, uv, gate, 1.0, window, decode, start, extra)
+        rows = list(range(start, T)) + [t for e in range(extra) for t in (T - 2 - e, T - 1 - e)]
+        _close(got, want[rows], tol, f"window {window}, key {j}")
+
+
+def latent_heads_differ(dev, dtype, tol, decode, T=150, H=20, d=32, rd=16, R=64, dv=48, window=60, extra=0):
+    """Scores spread over several units, every head with matrices of its own: a head that uses another's is far off."""
+    q, c, kr, uk, uv, gate = _latent_layer(H, d, rd, R, dv, T, 3, quiet=0.7)
+    want = latent_want(q, c, kr, uk, uv, gate, 0.5, window)
+    got = latent_run(dev, dtype, q, c, kr, uk, uv, gate, 0.5, window, decode, 40, extra)
+    rows = list(range(40, T)) + [t for e in range(extra) for t in (T - 2 - e, T - 1 - e)]
+    e = (got - want[rows]).pow(2).mean().sqrt() / want.pow(2).mean().sqrt()
+    assert float(e) <= tol, f"off by {float(e):.3g}"
+
+
+def latent_prep(dev, dtype, tol, T=70, H=5, d=24, rd=12, R=40, spare=4):
+    """Rotation of the queries' rotated part in place (columns past the rotated ones pass), norm over the real latent only,
+    append in scrambled slots; a layer that reads another's rows only rotates."""
+    from xfastertransformer_b200.ops import reference as Rf
+    g = torch.Generator().manual_seed(8)
+    r = lambda *s: torch.randn(*s, generator=g).to(dtype)
+    rot = {"dims": rd, "base": 700.0, "scaling": {"factor": 3.0, "original": 50, "fast": 5.0, "slow": 0.5}}
+    tab = Rf.rope_table(256, rd, 700.0, "yarn", 3.0, 50, 5.0, 0.5, table_scale=O.rotary_frequencies(rot)[1], angle_dtype=torch.float64)
+    rp, rk = rd + spare, R + spare
+    dims = ops.LatentDims(H, d, rp, rk, 8, True, True, R)
+    x = r(T, dims.row)
+    x[:, dims.q_width + R:dims.q_width + rk] = 0
+    w = torch.cat([torch.rand(R, generator=g) + 0.5, torch.zeros(spare)])
+    pos = list(range(31, 31 + T))
+    pool = torch.zeros(3, 1, 64, rk + rp, dtype=dtype).to(dev)
+    slots = torch.randperm(3 * 64, generator=g)[:T].int()
+    y = x.clone().to(dev)
+    p = torch.tensor(pos, dtype=torch.int32).to(dev)
+    ops.latent_prep(y, dims, p, tab.to(dev), rd, w.to(dev), 1e-3, pool, slots.to(dev))
+    xd = x.double()
+    q = xd[:, :dims.q_width].view(T, H, d + rp).clone()
+    q[..., d:] = O.rotate(q[..., d:], pos, rot, True)
+    c = torch.cat([O.rms_norm(xd[:, dims.q_width:dims.q_width + R], w[:R].double(), 1e-3), torch.zeros(T, spare)], -1)
+    k = O.rotate(xd[:, None, dims.q_width + rk:dims.gate_at], pos, rot, True)[:, 0]
+    got = pool.cpu()[(slots // 64).long(), 0, (slots % 64).long()]
+    for a, b, what in ((y[:, :dims.q_width].view(T, H, -1), q, "queries"), (got[:, :rk], c, "latents"), (got[:, rk:], k, "shared keys"),
+                       (y[:, dims.gate_at:], xd[:, dims.gate_at:], "gate")):
+        e = float((a.double().cpu() - b).abs().max() / b.abs().max())
+        assert e <= tol, f"{what}: {e:.3g}"
+    reader = ops.LatentDims(H, d, rp, rk, 8, False, True, R)
+    z = torch.cat([x[:, :dims.q_width], x[:, dims.gate_at:]], -1).contiguous().to(dev)
+    before = pool.clone()
+    ops.latent_prep(z, reader, p, tab.to(dev), rd, None, 1e-3, pool, slots.to(dev))
+    assert torch.equal(z[:, :dims.q_width], y[:, :dims.q_width]) and torch.equal(pool, before)
+
+
+def experts(dev, dtype, tol, T, E, top, ff, shared, width=72, spread=2.0):
+    """Router and gate-free experts against the plain form; unused experts and experts that get every token included."""
+    from xfastertransformer_b200.runtime.loader import make_linear
+    g = torch.Generator().manual_seed(T * 31 + E)
+    r = lambda *s: torch.randn(*s, generator=g).bfloat16().float()
+    h = r(T, width)
+    W = {"embed": torch.zeros(1, width), "l0.mlp.router": r(E, width) * (spread / width ** 0.5)}
+    W["l0.mlp.router"] = W["l0.mlp.router"].bfloat16().float()
+    sizes = [(f"e{e}", ff) for e in range(E)] + ([("shared", shared)] if shared else [])
+    for n, f in sizes:
+        W[f"l0.mlp.{n}.up"], W[f"l0.mlp.{n}.down"] = (r(f, width) / width ** 0.5).bfloat16().float(), (r(width, f) / f ** 0.5).bfloat16().float()
+    W = {k: v.double() for k, v in W.items()}
+    want = O.experts(h.double(), {"router": {"top": top}, "shared": bool(shared)}, W, "l0")
+    kind = "bf16" if dtype == torch.bfloat16 else "fp32"
+    lin = lambda n: make_linear(W["l0.mlp." + n].float().to(dev), kind)
+    x = h.to(dtype).to(dev)
+    idx, w = ops.route(ops.linear(x, lin("router"), out_dtype=torch.float32), "deepseek", top, norm_topk=True, scoring="softmax")
+    pair = lambda n: (lin(n + ".up"), lin(n + ".down"))
+    add = None
+    if shared:
+        up, down = pair("shared")
+        add = ops.linear(ops.linear(x, up, act="relu2"), down, out_dtype=torch.float32)
+    got = ops.moe_experts(x, idx, w, [pair(f"e{e}") for e in range(E)], "relu2", 0, gated=False, add=add)
+    assert got.dtype == torch.float32
+    wi, ww = O.router(h.double() @ W["l0.mlp.router"].T, top)
+    assert torch.equal(torch.sort(idx.cpu().long(), -1).values, torch.sort(wi, -1).values), "other experts"
+    assert float((w.cpu().double().sum(-1) - 1).abs().max()) < 1e-5
+    e = float((got.double().cpu() - want).abs().max() / want.abs().max())
+    assert e <= tol, f"{T} tokens, {top} of {E}: {e:.3g}"
+
+
 def softcap(dev, dtype, d, tol, T=140, H=2, G=2, **kw):
     """Scores far above and far below the cap."""
     g = torch.Generator().manual_seed(9)
@@ -156,6 +295,10 @@ def residual_norm(dev, H, kind, y_dtype, h_dtype, tol, T=9):
     close(h, norm(xs, w2)[rows.long()], ht, "selected rows")
     a, h = run(None, None, None, (w2, None), ids=ids.to(dev), table=wide(table))
     close(a, table[ids.long()].double(), 0.0, "embedding")
+    a, h = run(None, None, None, (w2, None), ids=ids.to(dev), table=wide(table), embed_scale=2.75)
+    close(a, table[ids.long()].double() * 2.75, 0.0, "scaled embedding")
+    close(h, norm(table[ids.long()].double() * 2.75, w2), ht, "scaled embedding's norm")
+    a, h = run(None, None, None, (w2, None), ids=ids.to(dev), table=wide(table))
     close(h, norm(table[ids.long()], w2), ht, "embedding's norm")
 
 

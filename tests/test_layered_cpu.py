@@ -1,4 +1,4 @@
-"""Layered designs (Kafipel) on the CPU path: the engine, cache, batching and command-line tool against a plain
+"""Layered designs (Kafipel, Vepivik) on the CPU path: the engine, cache, batching and command-line tool against a plain
 implementation of the equations."""
 import os
 import subprocess
@@ -38,32 +38,35 @@ def test_whole_prompt(cases, name):
     C.whole_prompt(cases(name), "fp32", 75)
 
 
-@pytest.mark.parametrize("name", ["unequal", "bare"])
+@pytest.mark.parametrize("name", ["unequal", "bare", "latent", "latent_bare"])
 def test_first_tokens(cases, name):
     C.first_tokens(cases(name), "fp32")
 
 
-@pytest.mark.parametrize("name,n,start", [("unequal", 75, 1), ("shared", 75, 60)])
+@pytest.mark.parametrize("name,n,start", [("unequal", 75, 1), ("shared", 75, 60), ("latent", 75, 1)])
 def test_token_by_token(cases, name, n, start):
     C.token_by_token(cases(name), "fp32", n, start)
 
 
 @pytest.mark.parametrize("sizes", [(2,), (3, 64, 1), (17, 29)])
-def test_portions(cases, sizes):
-    C.portions(cases("unequal"), "fp32", 75, sizes)
+@pytest.mark.parametrize("name", ["unequal", "latent"])
+def test_portions(cases, name, sizes):
+    C.portions(cases(name), "fp32", 75, sizes)
 
 
-@pytest.mark.parametrize("name", ["unequal", "shared"])
+@pytest.mark.parametrize("name", ["unequal", "shared", "latent"])
 def test_mixed_batches_reuse_pages(cases, name):
     assert C.mixed_batches(cases(name), "fp32", lengths=(75, 50, 20, 1, 66), live=2) > 5
 
 
-def test_greedy_generation(cases):
-    C.greedy(cases("unequal"), "fp32", 20, 40)
+@pytest.mark.parametrize("name", ["unequal", "latent"])
+def test_greedy_generation(cases, name):
+    C.greedy(cases(name), "fp32", 20, 40)
 
 
-def test_rows_and_order(cases):
-    C.rows_and_order(cases("unequal"), "fp32")
+@pytest.mark.parametrize("name", ["unequal", "latent"])
+def test_rows_and_order(cases, name):
+    C.rows_and_order(cases(name), "fp32")
 
 
 def test_long_decoding(cases):
@@ -71,10 +74,11 @@ def test_long_decoding(cases):
     C.greedy(cases("large_heads"), "fp32", 5, 140)
 
 
-def test_scheduler_serves_it(cases):
+@pytest.mark.parametrize("name", ["shared", "latent"])
+def test_scheduler_serves_it(cases, name):
     """The serving scheduler (chunked prefill, mixed steps) emits generate()'s tokens."""
     from serving import openai_server as oai
-    c = cases("shared")
+    c = cases(name)
     m = xft.AutoModel.from_pretrained(c.path, dtype="fp32")
     prompts = [c.tokens(n, 40 + n) for n in (33, 7, 70)]
     want = [m.generate(torch.tensor([p]), max_length=len(p) + 12)[0, len(p):].tolist() for p in prompts]
@@ -97,9 +101,10 @@ def test_scheduler_serves_it(cases):
         s.join(timeout=30)
 
 
-def test_beams_sampling_and_prefix_reuse(cases, monkeypatch):
+@pytest.mark.parametrize("name", ["unequal", "latent"])
+def test_beams_sampling_and_prefix_reuse(cases, monkeypatch, name):
     """The parts of the engine above the step function work on a layered model as on any other."""
-    c = cases("unequal")
+    c = cases(name)
     p = c.tokens(70, 50)
     m = xft.AutoModel.from_pretrained(c.path, dtype="fp32")
     g = m.generate(torch.tensor([p]), max_length=80)
@@ -132,14 +137,17 @@ def _ranks(case, tmp_path, port, n=2, **env):
     return r, out
 
 
-def test_tensor_parallel_two_ranks(cases, tmp_path):
-    """Heads (also a key/value head that both ranks read), sinks, feed-forward rows and the head split over two ranks."""
-    c = cases("shared")
-    r, out = _ranks(c, tmp_path, 29831)
+@pytest.mark.parametrize("name,heads,env", [("shared", [2, 4], {}), ("latent", [3, 2], {}),
+                                            ("latent", [3, 2], {"XFT_EXPERT_PARALLEL": "1"})])
+def test_tensor_parallel_two_ranks(cases, tmp_path, name, heads, env):
+    """Heads (also a key/value head or latents that both ranks read), sinks, feed-forward rows or experts and the logits
+    split over two ranks."""
+    c = cases(name)
+    r, out = _ranks(c, tmp_path, 29831, **env)
     assert r.returncode == 0, r.stdout[-2000:] + r.stderr[-2000:]
     got = torch.load(out)
     C.check(got["rows"], torch.cat([c.want(got["prompts"][0])[[3, 49]], c.want(got["prompts"][1])[-1:]]), "fp32", "two ranks")
-    assert got["heads"] == [[2, 4], [2, 4]]
+    assert got["heads"][0] == heads
     m = xft.AutoModel.from_pretrained(c.path, dtype="fp32")
     assert torch.equal(got["tokens"], m.generate(torch.tensor([got["prompts"][0]]), max_length=60))
 

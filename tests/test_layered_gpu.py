@@ -1,4 +1,4 @@
-"""Layered designs (Kafipel) on a GPU: every kernel of the path alone, and whole models in bf16 and in 32 bits, against a
+"""Layered designs (Kafipel, Vepivik) on a GPU: every kernel of the path alone, and whole models in bf16 and in 32 bits, against a
 plain implementation of the equations."""
 import os
 import sys
@@ -145,6 +145,79 @@ def test_rotation(dtype, d, dv, tol):
                d, dv, tol)
 
 
+# ------------------------------------------------------------------------------------------ latent attention, experts
+FORMS = pytest.mark.parametrize("form", ["decode", "portion", "short portion", "mixed"])
+
+
+def _form(monkeypatch, form):
+    """(decode steps?, extra short portions) of a form; "short portion" keeps a long portion in the absorbed form."""
+    from xfastertransformer_b200.utils.flags import Env
+    monkeypatch.setenv("XFT_LATENT_EXPAND_MIN_Q", "100000" if form == "short portion" else "16")
+    Env.get().reload()
+    return form == "decode", 2 if form == "mixed" else 0
+
+
+@FORMS
+@pytest.mark.parametrize("window", [40, 64, 1, 129, 0])
+def test_latent_window_edges(monkeypatch, form, window):
+    decode, extra = _form(monkeypatch, form)
+    M.latent_window_edges(_dev(), torch.bfloat16, window, decode, BF16_TOL, extra=extra)
+    M.latent_window_edges(_dev(), torch.bfloat16, window, decode, BF16_TOL, H=17, d=128, rd=64, R=200, dv=128, extra=extra)
+
+
+@FORMS
+@pytest.mark.parametrize("sizes", [dict(H=2, d=208, rd=80, R=520, dv=144), dict(H=3, d=136, rd=24, R=300, dv=72),
+                                   dict(H=33, d=64, rd=64, R=512, dv=64), dict(H=4, d=16, rd=2, R=12, dv=8)])
+def test_latent_sizes(monkeypatch, form, sizes):
+    """Sizes without a tensor-core kernel, three key chunks, more than 16 heads per token twice over, very small ones."""
+    decode, extra = _form(monkeypatch, form)
+    M.latent_window_edges(_dev(), torch.bfloat16, 70, decode, BF16_TOL, extra=extra, **sizes)
+    M.latent_heads_differ(_dev(), torch.bfloat16, BF16_TOL, decode, extra=extra, **sizes)
+
+
+@pytest.mark.parametrize("window", [40, 129, 0])
+@pytest.mark.parametrize("decode", [False, True])
+def test_latent_fp32(window, decode):
+    M.latent_window_edges(_dev(), torch.float32, window, decode, 5e-6)
+    M.latent_heads_differ(_dev(), torch.float32, 5e-6, decode)
+
+
+def test_latent_far_keys(monkeypatch):
+    """A key thousands of positions back, just inside and just outside a wide window, in split decode steps and in portions
+    of several key tiles whose maxima grow from tile to tile."""
+    T = 2100
+    q, c, kr, uk, uv, gate = M._latent_layer(2, 64, 32, 100, 64, T, 1)
+    q[..., 64], kr[:, 0] = 3.0, 0.0
+    kr[:, 1], q[..., 65] = torch.arange(T) / 300.0, 2.0            # later keys weigh more: the running maximum rises
+    for window, j in ((1900, 250), (1900, 180), (2000, 99), (2000, 101), (0, 5)):
+        k2 = kr.clone()
+        k2[j, 0] = 12.0
+        want = M.latent_want(q, c, k2, uk, uv, gate, 1.0, window)
+        for form in ("decode", "portion", "short portion"):
+            decode, _ = _form(monkeypatch, form)
+            for start in (T - 60,) if form != "portion" else (T - 60, T - 700):
+                got = M.latent_run(_dev(), torch.bfloat16, q, c, k2, uk, uv, gate, 1.0, window, decode, start)
+                M._close(got, want[start:], BF16_TOL, f"window {window}, key {j}, {form}")
+
+
+def test_latent_expanded_by_head_groups(monkeypatch):
+    from xfastertransformer_b200.ops import native_latent
+    monkeypatch.setattr(native_latent, "EXPAND_BYTES", 7 * 2 * 150 * (64 + 64))
+    M.latent_heads_differ(_dev(), torch.bfloat16, BF16_TOL, False, window=0)
+
+
+@pytest.mark.parametrize("dtype,tol", [(torch.float32, 2e-6), (torch.bfloat16, 8e-3)])
+def test_latent_prep(dtype, tol):
+    M.latent_prep(_dev(), dtype, tol)
+    M.latent_prep(_dev(), dtype, tol, T=3, H=33, d=64, rd=64, R=512, spare=0)
+
+
+@pytest.mark.parametrize("T,E,top,ff,shared", [(9, 5, 2, 24, 40), (1, 7, 7, 8, 0), (300, 33, 3, 64, 128), (200, 1, 1, 136, 8)])
+@pytest.mark.parametrize("dtype,tol", [(torch.float32, 3e-6), (torch.bfloat16, 1e-2)])
+def test_experts(dtype, tol, T, E, top, ff, shared):
+    M.experts(_dev(), dtype, tol, T, E, top, ff, shared)
+
+
 # ------------------------------------------------------------------------------------------ whole models
 BOTH = pytest.mark.parametrize("dtype", ["fp32", "bf16"])
 
@@ -156,45 +229,47 @@ def test_whole_prompt(cases, name, dtype):
 
 
 @BOTH
-@pytest.mark.parametrize("name", ["unequal", "heads128"])
+@pytest.mark.parametrize("name", ["unequal", "heads128", "latent", "latent128"])
 def test_first_tokens(cases, name, dtype):
     C.first_tokens(cases(name), dtype)
 
 
 @BOTH
-@pytest.mark.parametrize("name,start", [("unequal", 1), ("heads128", 40), ("padded", 70), ("shared", 1), ("bare", 100)])
+@pytest.mark.parametrize("name,start", [("unequal", 1), ("heads128", 40), ("padded", 70), ("shared", 1), ("bare", 100),
+                                        ("latent", 1), ("latent128", 40), ("latent_bare", 30), ("latent_large", 100)])
 def test_token_by_token(cases, name, start, dtype):
     C.token_by_token(cases(name), dtype, 140, start)
 
 
 @BOTH
 @pytest.mark.parametrize("sizes", [(2,), (3, 64, 1), (17, 29)])
-@pytest.mark.parametrize("name", ["unequal", "heads128"])
+@pytest.mark.parametrize("name", ["unequal", "heads128", "latent", "latent128"])
 def test_portions(cases, name, sizes, dtype):
     C.portions(cases(name), dtype, 140, sizes)
 
 
 @BOTH
-@pytest.mark.parametrize("name", ["unequal", "heads128", "shared", "large_heads"])
+@pytest.mark.parametrize("name", ["unequal", "heads128", "shared", "large_heads"] + C.LATENT)
 def test_mixed_batches_reuse_pages(cases, name, dtype):
     assert C.mixed_batches(cases(name), dtype) > 8
 
 
 @BOTH
-@pytest.mark.parametrize("name", ["unequal", "heads128"])
+@pytest.mark.parametrize("name", ["unequal", "heads128", "latent"])
 def test_rows_and_order(cases, name, dtype):
     C.rows_and_order(cases(name), dtype)
 
 
 @BOTH
-@pytest.mark.parametrize("name", ["unequal", "heads128", "padded"])
+@pytest.mark.parametrize("name", ["unequal", "heads128", "padded", "latent", "latent128"])
 def test_greedy_generation(cases, name, dtype):
     """generate(): the captured decode step (CUDA graph) included."""
     C.greedy(cases(name), dtype, 20, 130)
 
 
-def test_graph_and_eager_steps_agree(cases, monkeypatch):
-    c = cases("heads128")
+@pytest.mark.parametrize("name", ["heads128", "latent128"])
+def test_graph_and_eager_steps_agree(cases, monkeypatch, name):
+    c = cases(name)
     a = C.greedy(c, "bf16", 30, 60)
     monkeypatch.setenv("XFT_CUDA_GRAPH", "0")
     from xfastertransformer_b200.utils.flags import Env

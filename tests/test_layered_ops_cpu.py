@@ -71,6 +71,22 @@ def test_rotation_table_grows(tmp_path):
     assert abs(float(b[-1, 1]) - math.cos((b.shape[0] - 1) * f[1])) < 2e-4
 
 
+@pytest.mark.parametrize("window", [40, 64, 1, 129, 0])
+@pytest.mark.parametrize("decode", [False, True])
+def test_latent_window_edges(window, decode):
+    M.latent_window_edges(CPU, torch.float32, window, decode, 1e-5)
+
+
+def test_latent_heads_and_prep():
+    M.latent_heads_differ(CPU, torch.float32, 1e-5, False)
+    M.latent_prep(CPU, torch.float32, 2e-5)
+
+
+@pytest.mark.parametrize("T,E,top,ff,shared", [(9, 5, 2, 24, 40), (1, 7, 7, 8, 0), (30, 1, 1, 16, 16), (40, 33, 3, 20, 8)])
+def test_experts(T, E, top, ff, shared):
+    M.experts(CPU, torch.float32, 1e-5, T, E, top, ff, shared)
+
+
 # ------------------------------------------------------------------------------------------ configuration
 def _write(tmp_path, cfg, name="m"):
     return O.write_checkpoint(str(tmp_path / name), cfg, O.random_weights(cfg))
@@ -92,6 +108,44 @@ def test_config_is_read_per_layer(tmp_path):
     assert family_for(c).layered and decoder_class(c).__name__ == "LayeredDecoder"
     c.to_ini(str(tmp_path / "again"))
     assert ModelConfig.load(str(tmp_path / "again")).layers == c.layers
+
+
+def test_latent_config_is_read_per_layer(tmp_path):
+    sc = {"factor": 2.5, "original": 77, "fast": 9.0, "slow": 0.7}
+    cfg = O.vepivik([O.window_layer(heads=6, kv_heads=2, dim=20, vdim=28, size=11, scale=0.3, mlp=O.moe(ff=44, experts=9, top=4, shared=52)),
+                     O.latent_layer(heads=5, dim=14, rot_dim=6, vdim=18, kv_rank=22, size=31, base=77.0, scaling=sc, scale=0.4),
+                     O.latent_layer(heads=2, dim=30, rot_dim=6, vdim=4, kv_rank=22, base=77.0, scaling=sc, kv_from=1, mask=False,
+                                    mlp=O.moe(shared=None))], eps=2e-3, scale=4.5)
+    c = ModelConfig.load(_write(tmp_path, cfg))
+    a, b, r = c.layers
+    assert (c.model_type, c.embed_scale, c.layernorm_eps, c.num_layer) == ("vepivik", 4.5, 2e-3, 3)
+    assert (a.mixer.kind, a.mixer.window, a.mixer.keep_first, a.mixer.rot, a.mixer.gate, a.ff) == ("attention", 11, 0, None, False, 0)
+    assert (a.moe.experts, a.moe.top, a.moe.ff, a.moe.shared, a.ff_kind) == (9, 4, 44, 52, "moe")
+    m = b.mixer
+    assert (m.kind, m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank, m.window, m.scale) == ("latent", 5, 14, 6, 18, 22, 31, 0.4)
+    assert (m.rot.dims, m.rot.base, m.rot.factor, m.rot.style, m.gate, b.moe, b.ff) == (6, 77.0, 2.5, "interleaved", True, None, 0)
+    assert (r.mixer.kv_from, r.mixer.window, r.moe.shared) == (1, 0, 0)
+    f = family_for(c)
+    assert f.layered and f.tied_head and not f.post_norm and not f.sinks and f.norm == "rms"
+    c.to_ini(str(tmp_path / "again"))
+    assert ModelConfig.load(str(tmp_path / "again")).layers == c.layers
+
+
+@pytest.mark.parametrize("change,match", [
+    (lambda d: d["layers"][1]["mixer"].update(kv_rank=24), "heads differ"),
+    (lambda d: d["layers"][1]["mixer"]["rot"].update(base=5.0), "heads differ"),
+    (lambda d: d["layers"][1]["mixer"].update(kv_from=2), "not an earlier layer"),
+    (lambda d: d["layers"][2]["mixer"].update(kv_from=0), "heads differ"),
+    (lambda d: d["layers"][0]["mlp"]["router"].update(top=7), "of 6 experts"),
+    (lambda d: d["layers"][0]["mlp"].update(kind="mixture"), "unsupported feed-forward"),
+    (lambda d: d["layers"][0]["mixer"]["rot"].update(dims=18), "do not fit")])
+def test_latent_config_faults(tmp_path, change, match):
+    cfg = O.vepivik([O.latent_layer(mlp=O.moe()), O.latent_layer(kv_from=0), O.window_layer()])
+    change(cfg)
+    os.makedirs(tmp_path / "m")
+    (tmp_path / "m" / "config.json").write_text(json.dumps(cfg))
+    with pytest.raises(ValueError, match=match):
+        ModelConfig.load(str(tmp_path / "m"))
 
 
 @pytest.mark.parametrize("change,match", [
@@ -166,6 +220,19 @@ def test_fixed_pools_refuse_what_does_not_fit(tmp_path):
         m.forward_cb()
     with pytest.raises(MemoryError):
         m.set_input_cb([[1] * 10], max_length=500)
+
+
+def test_latent_pools(tmp_path):
+    """A latent layer's pool has one row per token and no values; its reader has none; an int8 cache is refused."""
+    cfg = O.vepivik([O.window_layer(), O.latent_layer(), O.latent_layer(kv_from=1)])
+    p = _write(tmp_path, cfg)
+    m = xft.AutoModel.from_pretrained(p, dtype="fp32", max_cache_tokens=130)
+    cache = m.model.cache
+    assert [tuple(k.shape) for k in cache.k] == [(3, 2, 64, 32), (3, 1, 64, 56)]
+    assert cache.v[0].shape[3] == 24 and cache.v[1] is None
+    assert cache.bytes_per_block() == 64 * 4 * (2 * 56 + 56)
+    with pytest.raises(ValueError, match="int8"):
+        xft.AutoModel.from_pretrained(p, dtype="bf16", kv_cache_dtype="int8")
 
 
 def test_refusals(tmp_path):

@@ -40,6 +40,7 @@ from ..utils.trace import TimeLine
 from .decoder import Batch, Decoder, Layer
 
 ATTENTION_HEADS = (64, 128, 256)          # head sizes of the tensor-core attention kernels
+LATENTS = (64, 128, 256, 512)             # latent sizes of the tensor-core latent attention
 
 
 def _up(n: int, m: int) -> int:
@@ -217,7 +218,8 @@ class LayeredDecoder(Decoder):
         """Latent attention: heads are split over ranks, the latents (one row per token) are on every rank."""
         m = L.mix
         size = (lambda n: _up(n, 64)) if self.pad_heads else (lambda n: n)
-        d = L.dims = ops.LatentDims(L.hq, size(m.dim), size(m.rot_dim), size(m.kv_rank), size(m.vdim), L.own_kv, m.gate, m.kv_rank)
+        rank = next((r for r in LATENTS if m.kv_rank <= r), size(m.kv_rank)) if self.pad_heads else m.kv_rank
+        d = L.dims = ops.LatentDims(L.hq, size(m.dim), size(m.rot_dim), rank, size(m.vdim), L.own_kv, m.gate, m.kv_rank)
         L.kd, L.vd = d.rank + d.rot, d.vdim
         parts = [self._rows(p + "mix.q", m.heads, q, (m.dim, d.dim), (m.rot_dim, d.rot))]
         L.latent_norm = None

@@ -18,7 +18,7 @@ import torch
 
 _LIB = None
 _ACT = {None: 0, "none": 0, "relu": 1, "silu": 2, "gelu": 3, "gelu_tanh": 3, "gelu_new": 3, "gelu_pytorch_tanh": 3,
-        "swiglu": 2}
+        "swiglu": 2, "relu2": 4}
 
 STATUS_TEXT = {0: "ok", 1: "producer timed out waiting for a free stage", 2: "MMA warp timed out waiting for TMA data",
                3: "epilogue timed out waiting for the accumulator", 4: "timed out waiting for a peer flag",
@@ -168,7 +168,8 @@ def layernorm(x, w, b, eps):
     return y.view(*x.shape[:-1], H)
 
 
-def residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids=None, table=None, keep_x=True):
+def residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids=None, table=None, keep_x=True,
+                  embed_scale=1.0):
     """csrc/kernels/residual_norm.cu.  x fp32 [T, HP]; y bf16 or fp32 rows; gains fp32 [H]."""
     dev = (x if x is not None else table).device
     gain = nxt[0] if nxt is not None else post[0] if post is not None else None
@@ -199,13 +200,13 @@ def residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids=None, table=Non
               0 if ids is not None else x.stride(0), _p(x_out), 0 if x_out is None else x_out.stride(0), _p(y),
               0 if y is None else y.stride(0), int(y is not None and y.dtype == torch.float32), _p(pw), _p(pb), _p(nw), _p(nb),
               _p(h), HP, int(h_dtype == torch.float32), _p(rows32), n_in, n_out, H, 0 if kind == "layer" else 1,
-              C.c_float(eps), _p(ws.status), _stream()), "residual_norm")
+              C.c_float(eps), C.c_float(embed_scale), _p(ws.status), _stream()), "residual_norm")
     ws.launches += 1
     return x_out, h
 
 
-def gemm_f32(x, w, N):
-    """Y[T,N] = X[T,K] W[N,K]^T, everything in 32 bits."""
+def gemm_f32(x, w, N, act=None):
+    """Y[T,N] = act(X[T,K] W[N,K]^T), everything in 32 bits."""
     x2 = x.reshape(-1, x.shape[-1])
     if x2.stride(1) != 1:
         x2 = x2.contiguous()
@@ -214,8 +215,8 @@ def gemm_f32(x, w, N):
     y = torch.empty(T, N, dtype=torch.float32, device=x.device)
     fn = lib().xft_gemm_f32
     fn.restype = C.c_int
-    _check(fn(_p(x2), x2.stride(0) if T > 1 else max(x2.stride(0), K), _p(w), w.stride(0), _p(y), N, T, N, K, _stream()),
-           "gemm_f32")
+    _check(fn(_p(x2), x2.stride(0) if T > 1 else max(x2.stride(0), K), _p(w), w.stride(0), _p(y), N, T, N, K, _ACT[act],
+              _stream()), "gemm_f32")
     Workspace.get(x.device).launches += 1
     return y
 
@@ -404,9 +405,9 @@ def linear(x, W, bias=None, act=None, residual=None, res_scale=1.0, out_dtype=No
         y = gemm_bf16(x, W.w, W.out_features, bias=bias, act=act, residual=residual, res_scale=res_scale,
                       out_dtype=out_dtype)
     elif W.kind == "fp32":
-        if bias is not None or act is not None or residual is not None or out_dtype not in (None, torch.float32):
-            raise KernelError("fp32 products have no epilogue")
-        y = gemm_f32(x, W.w, W.out_features)
+        if bias is not None or residual is not None or out_dtype not in (None, torch.float32):
+            raise KernelError("fp32 products have no bias or residual")
+        y = gemm_f32(x, W.w, W.out_features, act)
     else:
         from . import native_quant
         y = native_quant.linear(x, W, bias, act, residual, res_scale, out_dtype)
@@ -596,14 +597,7 @@ def paged_attention(q, kc, vc, block_table, cu_q, kv_lens, scale, ks=None, vs=No
         if ks is not None or slopes is not None or pl is not None or kc.dtype != q.dtype or vc.dtype != q.dtype:
             raise KernelError(f"head size {D} / {vd} in {q.dtype}: no int8 cache, ALiBi or prefix mask")
         q = q.contiguous()
-        out = torch.empty(T, hq, vd, dtype=q.dtype, device=dev)
-        fn = lib().xft_attention_plain
-        fn.restype = C.c_int
-        _check(fn(_p(q), _p(out), _p(kc), _p(vc), _p(block_table), block_table.stride(0), _p(cu_dev), _p(kv_dev), B, T, hq,
-                  hkv, g, q_off, D, vd, bs, nb, C.c_float(scale), C.c_float(softcap), window, keep_first, _p(sinks),
-                  int(q.dtype == torch.float32), _p(ws.status), _stream()), "attention_plain")
-        ws.launches += 1
-        return out
+        return attention_plain(q, kc, vc, vd, block_table, cu_dev, kv_dev, B, scale, g, q_off, softcap, window, keep_first, sinks)
     out = torch.empty_like(q)
     nsplit, po, pm = 1, None, None
     if decode:
@@ -641,6 +635,31 @@ def paged_attention(q, kc, vc, block_table, cu_q, kv_lens, scale, ks=None, vs=No
     return out
 
 
+def attention_plain(q, kc, vc, vd, block_table, cu_dev, kv_dev, B, scale, group, q_off=0, softcap=0.0, window=0, keep_first=0,
+                    sinks=None):
+    """Attention for any head size in fp32 or bf16 (csrc/kernels/plain.cu); values are the first `vd` columns of vc's rows."""
+    T, hq, D = q.shape
+    nb, hkv, bs, _ = kc.shape
+    out = torch.empty(T, hq, vd, dtype=q.dtype, device=q.device)
+    ws = Workspace.get(q.device)
+    fn = lib().xft_attention_plain
+    fn.restype = C.c_int
+    _check(fn(_p(q), _p(out), _p(kc), _p(vc), _p(block_table), block_table.stride(0), _p(cu_dev), _p(kv_dev), B, T, hq,
+              hkv, group, q_off, D, vd, vc.shape[3], bs, nb, C.c_float(scale), C.c_float(softcap), window, keep_first, _p(sinks),
+              int(q.dtype == torch.float32), _p(ws.status), _stream()), "attention_plain")
+    ws.launches += 1
+    return out
+
+
+def batch_arrays(cu_q, kv_lens, meta, dev):
+    """(cu_q, kv_lens) on the device, number of sequences, every sequence has one query, longest context of a batch."""
+    B = len(kv_lens)
+    if meta is not None and getattr(meta, "cu_q_dev", None) is not None:
+        return meta.cu_q_dev, meta.kv_lens_dev, B, meta.is_decode, meta.max_kv
+    return (torch.tensor(list(cu_q), dtype=torch.int32, device=dev), torch.tensor(list(kv_lens), dtype=torch.int32, device=dev), B,
+            all(cu_q[i + 1] - cu_q[i] == 1 for i in range(B)), max(kv_lens))
+
+
 def mla_attention(q_nope, q_rope, latent_cache, block_table, cu_q, kv_lens, w_uk, w_uv, scale, absorbed=True,
                   meta=None):
     from . import native_mla
@@ -654,9 +673,9 @@ def route(logits, kind, top_k, bias=None, n_group=1, topk_group=1, routed_scalin
     return native_moe.route(logits, kind, top_k, bias, n_group, topk_group, routed_scaling, norm_topk, scoring)
 
 
-def moe_experts(x, idx, w, experts, act="silu", expert_offset=0, packed=None, expected_pairs=None):
+def moe_experts(x, idx, w, experts, act="silu", expert_offset=0, packed=None, expected_pairs=None, gated=True, add=None):
     from . import native_moe
-    return native_moe.moe_experts(x, idx, w, experts, act, expert_offset, packed, expected_pairs)
+    return native_moe.moe_experts(x, idx, w, experts, act, expert_offset, packed, expected_pairs, gated, add)
 
 
 # ------------------------------------------------------------------------------------------

@@ -40,8 +40,8 @@ def route(logits, kind, top_k, bias=None, n_group=1, topk_group=1, routed_scalin
 
 
 def pack_experts(experts) -> dict:
-    """Stack the local experts' weights: gate‖up [E*2I, H] and down [E*H, I] (bf16; other kinds are expanded
-    once here).  The per-expert LinearWeights are re-pointed at views of the stacks so nothing is held twice."""
+    """Stack the local experts' weights: gate‖up [E*2I, H] (or up [E*I, H]) and down [E*H, I] (bf16, or fp32 when all of
+    them are; other kinds are expanded once here).  The per-expert LinearWeights are re-pointed at views of the stacks so nothing is held twice."""
     # the pack lives in the first expert's weight object (an id()-keyed table would hand a dead list's pack to a
     # new list that happens to reuse its address)
     gu0, dn0 = experts[0]
@@ -53,15 +53,18 @@ def pack_experts(experts) -> dict:
     I, H = dn0.in_features, dn0.out_features
     E = len(experts)
     dev = gu0.w.device
-    gu = torch.empty(E * 2 * I, H, dtype=torch.bfloat16, device=dev)
-    dn = torch.empty(E * H, I, dtype=torch.bfloat16, device=dev)
+    kind = "fp32" if all(w.kind == "fp32" for e in experts for w in e) else "bf16"
+    dt = torch.float32 if kind == "fp32" else torch.bfloat16
+    up = gu0.out_features
+    gu = torch.empty(E * up, H, dtype=dt, device=dev)
+    dn = torch.empty(E * H, I, dtype=dt, device=dev)
     for e, (g, d) in enumerate(experts):
-        gv, dv = gu[e * 2 * I:(e + 1) * 2 * I], dn[e * H:(e + 1) * H]
-        gv.copy_(g.w if g.kind == "bf16" else R.dequant_weight(g))
-        dv.copy_(d.w if d.kind == "bf16" else R.dequant_weight(d))
-        if g.kind == "bf16":
+        gv, dv = gu[e * up:(e + 1) * up], dn[e * H:(e + 1) * H]
+        gv.copy_(g.w if g.kind == kind else R.dequant_weight(g))
+        dv.copy_(d.w if d.kind == kind else R.dequant_weight(d))
+        if g.kind == kind:
             g.w = gv
-        if d.kind == "bf16":
+        if d.kind == kind:
             d.w = dv
     pk = dict(gu=gu, dn=dn, I=I, H=H, E=E, last=experts[-1][0])
     gu0.cache["moe_pack"] = pk
@@ -97,15 +100,47 @@ def _pack_fp8(experts) -> dict:
     return pk
 
 
-def moe_experts(x, idx, w, experts, act="silu", expert_offset=0, packed=None, expected_pairs=None):
-    """sum_k w[t,k] * down_e(act(gate_e x) * up_e x) over the local experts -> fp32 [T, H].  `expected_pairs`: about how
+def _experts_f32(x, idx32, w, pk, act, expert_offset, gated, add):
+    """The 32-bit path: rows stay where they are, the first product reads them through the plan."""
+    if gated:
+        raise N.KernelError("fp32 experts have no gate product")
+    T, H = x.shape
+    k, E, I, dev = idx32.shape[1], pk["E"], pk["I"], x.device
+    lib, ws, n = _lib(), N.Workspace.get(dev), T * idx32.shape[1]
+    i32 = lambda *s: torch.empty(*s, dtype=torch.int32, device=dev)
+    f32 = lambda *s: torch.empty(*s, dtype=torch.float32, device=dev)
+    tiles_n = (n + 63) // 64 + E
+    pos, src, row_w, tiles, meta = i32(n), i32(n), f32(n), i32(tiles_n, 4), i32(2)
+    N._check(lib.xft_moe_plan(N._p(idx32), N._p(w), T, k, expert_offset, expert_offset + E, 64, N._p(pos), N._p(src), N._p(row_w),
+                              N._p(tiles), N._p(meta), tiles_n, n, N._stream()), "moe_plan")
+    h1, ys, out = f32(n, I), f32(n, H), f32(T, H)
+    fn = lib.xft_gemm_f32_grouped
+    fn.restype = C.c_int
+    N._check(fn(N._p(x), x.stride(0) if T > 1 else max(x.stride(0), H), N._p(pk["gu"]), H, N._p(h1), I, I, H, I, N._p(tiles),
+                N._p(meta), tiles_n, N._p(src), N._p(None), N._ACT[act], N._stream()), "grouped fp32 up")
+    N._check(fn(N._p(h1), I, N._p(pk["dn"]), I, N._p(ys), H, H, I, H, N._p(tiles), N._p(meta), tiles_n, N._p(None), N._p(row_w), 0,
+                N._stream()), "grouped fp32 down")
+    N._check(lib.xft_moe_combine(N._p(ys), N._p(pos), k, N._p(add), N._p(None), 0, N._p(None), N._p(out), T, H, N._stream()),
+             "moe_combine")
+    ws.launches += 4
+    return out
+
+
+def moe_experts(x, idx, w, experts, act="silu", expert_offset=0, packed=None, expected_pairs=None, gated=True, add=None):
+    """sum_k w[t,k] * down_e(act(gate_e x) * up_e x) over the local experts (+ `add`, fp32) -> fp32 [T, H]; without `gated`
+    down_e(act(up_e x)).  `expected_pairs`: about how
     many (token, expert) pairs are real when most rows of `idx` are padding (-1), e.g. the receive area of the expert
     exchange; it only picks the token tile of the grouped GEMMs."""
     pk = packed or pack_experts(experts)
+    if add is not None:
+        assert add.dtype == torch.float32 and add.is_contiguous()
+    if x.dtype == torch.float32:
+        return _experts_f32(x.reshape(-1, x.shape[-1]), idx.int(), w.contiguous(), pk, act, expert_offset, gated, add)
     x2, ldx = N._rows2d(x)
     T, H = x2.shape
     k = idx.shape[1]
     E, I = pk["E"], pk["I"]
+    up = 2 * I if gated else I                       # weight rows of one expert's first product
     dev = x.device
     ws = N.Workspace.get(dev)
     lib = _lib()
@@ -134,19 +169,19 @@ def moe_experts(x, idx, w, experts, act="silu", expert_offset=0, packed=None, ex
                                        N._p(pk["dns"]), pk["dns"].shape[1], N._p(tiles), N._p(meta), max_tiles, min(bn, 128),
                                        N._p(row_w), 0, N._p(ws.status), N._stream()), "grouped fp8 down")
         out = torch.empty(T, H, dtype=torch.float32, device=dev)
-        N._check(lib.xft_moe_combine(N._p(ys), N._p(pos), k, N._p(None), N._p(None), 0, N._p(None), N._p(out), T, H,
+        N._check(lib.xft_moe_combine(N._p(ys), N._p(pos), k, N._p(add), N._p(None), 0, N._p(None), N._p(out), T, H,
                                      N._stream()), "moe_combine")
         ws.launches += 5
         return out
-    N._check(lib.xft_gemm_bf16_grouped(N._p(xs), H, max_rows, N._p(pk["gu"]), E * 2 * I, H, N._p(h1), I, 0, I, H, 1, I,
-                                       2 * I, N._p(tiles), N._p(meta), max_tiles, bn, N._p(None), N._ACT[act],
+    N._check(lib.xft_gemm_bf16_grouped(N._p(xs), H, max_rows, N._p(pk["gu"]), E * up, H, N._p(h1), I, 0, I, H, int(gated), I,
+                                       up, N._p(tiles), N._p(meta), max_tiles, bn, N._p(None), N._ACT[act],
                                        N._p(ws.status), N._stream()), "grouped gate_up")
     ys = torch.empty(max_rows, H, dtype=torch.float32, device=dev)
     N._check(lib.xft_gemm_bf16_grouped(N._p(h1), I, max_rows, N._p(pk["dn"]), E * H, I, N._p(ys), H, 1, H, I, 0, 0, H,
                                        N._p(tiles), N._p(meta), max_tiles, bn, N._p(row_w), 0, N._p(ws.status),
                                        N._stream()), "grouped down")
     out = torch.empty(T, H, dtype=torch.float32, device=dev)
-    N._check(lib.xft_moe_combine(N._p(ys), N._p(pos), k, N._p(None), N._p(None), 0, N._p(None), N._p(out), T, H,
+    N._check(lib.xft_moe_combine(N._p(ys), N._p(pos), k, N._p(add), N._p(None), 0, N._p(None), N._p(out), T, H,
                                  N._stream()), "moe_combine")
     ws.launches += 5
     return out

@@ -77,6 +77,7 @@ class Env:
         # prompt attention through the tcgen05 kernel from this many query rows on (head_dim 128, bf16 cache, no ALiBi);
         # a very large value switches it off
         self.attn_tc_min_q = _int("XFT_ATTN_TC_MIN_Q", 2)
+        self.latent_expand_min_q = _int("XFT_LATENT_EXPAND_MIN_Q", 16)   # prompt portions from this size on expand their latents
         self.gemm_streamk = _int("XFT_GEMM_STREAMK", 1) != 0
         self.fuse_qkv_rope = _int("XFT_FUSE_QKV_ROPE", 1) != 0
         # tensor-parallel prefill: two groups of prompts are interleaved block by block, so that the all-reduce of one
