@@ -69,10 +69,10 @@ CONFIGS = {
                        mlp=O.moe(ff=128, experts=2, top=1, shared=32))], width=160, vocab=300),
     # mechanisms left out one by one: no window, no scaling, no shared expert, every expert chosen, one head, no feed-forward
     "latent_bare": O.vepivik([
-        O.latent_layer(heads=1, dim=16, rot_dim=2, vdim=8, kv_rank=12, mask=False, mlp=O.moe(ff=16, experts=3, top=3, shared=None)),
+        O.latent_layer(heads=1, dim=16, rot_dim=2, vdim=8, kv_rank=12, mask=False, scale=0.11, mlp=O.moe(ff=16, experts=3, top=3, shared=None)),
         O.window_layer(heads=2, kv_heads=2, dim=32, vdim=32, mask=False, mlp=None),
         O.latent_layer(heads=2, dim=8, rot_dim=2, vdim=64, kv_rank=12, size=1, kv_from=0, mlp=O.moe(ff=8, experts=1, top=1, shared=8)),
-        O.latent_layer(heads=2, dim=72, rot_dim=70, vdim=24, kv_rank=20, size=5000, mlp=None)], width=72, vocab=150, scale=0.5),
+        O.latent_layer(heads=2, dim=72, rot_dim=70, vdim=24, kv_rank=20, size=5000, scale=0.04, mlp=None)], width=72, vocab=150, scale=0.5),
     # larger than any tensor-core latent kernel takes; three key chunks of the expanded form
     "latent_large": O.vepivik([
         O.latent_layer(heads=2, dim=208, rot_dim=80, vdim=144, kv_rank=520, size=30, scaling=YARN, mlp=O.moe()),

@@ -295,7 +295,11 @@ def vepivik(layers, width=96, vocab=210, eps=1e-5, scale=2.0):
 
 
 def random_weights(cfg, seed=0, gain=1.0):
-    """bf16-representable weights, scaled so that scores spread over several units and every mechanism matters."""
+    """bf16-representable weights, scaled so that scores spread over several units and every mechanism matters.
+
+    Experts: the first columns of the residual stream hold a code that the embedding alone writes, a permutation of equally
+    spaced levels per token, and each router reads little else.  So every token has experts of its own, other ones in every
+    layer, and no choice is close enough for rounding to turn it."""
     g = torch.Generator().manual_seed(seed)
 
     def mat(o, i, s=1.0):
@@ -311,6 +315,10 @@ def random_weights(cfg, seed=0, gain=1.0):
         W["head"] = mat(cfg["vocab"], D)
     else:
         W["embed"] = (W["embed"].float() / math.sqrt(D)).bfloat16()
+    E = max([l["mlp"]["router"]["experts"] for l in cfg["layers"] if (l.get("mlp") or {}).get("kind") == "moe"], default=0)
+    if E:
+        levels = (torch.arange(E) - (E - 1) / 2) * 3.0 / math.sqrt(D)
+        W["embed"][:, :E] = torch.stack([levels[torch.randperm(E, generator=g)] for _ in range(cfg["vocab"])]).bfloat16()
     for i, layer in enumerate(cfg["layers"]):
         p, m = f"l{i}", layer["mixer"]
         W[p + ".norm1"] = vec(D)
@@ -337,13 +345,20 @@ def random_weights(cfg, seed=0, gain=1.0):
             continue
         W[p + ".norm2"] = vec(D)
         if f["kind"] == "moe":
-            W[p + ".mlp.router"] = mat(f["router"]["experts"], D, 2.0)
+            n = f["router"]["experts"]
+            r = 0.001 * torch.randn(n, D, generator=g)
+            r[:, :E] = torch.eye(E)[torch.randperm(E, generator=g)[:n]]
+            W[p + ".mlp.router"] = r.bfloat16()
+            W[p + ".norm2"][:E] = 1.0
             for n, ff in [(f"e{e}", f["expert"]["ff"]) for e in range(f["router"]["experts"])] + \
                     ([("shared", f["shared"]["ff"])] if f.get("shared") else []):
                 W[p + f".mlp.{n}.up"], W[p + f".mlp.{n}.down"] = mat(ff, D), mat(D, ff, 0.8)
         else:
             W[p + ".norm2b"] = vec(D, 0.7)
             W[p + ".mlp.gate"], W[p + ".mlp.up"], W[p + ".mlp.down"] = mat(f["ff"], D), mat(f["ff"], D), mat(D, f["ff"])
+    for n, t in W.items():
+        if E and (n.endswith(".mix.o") or n.endswith(".down")):
+            t[:E] = 0
     return W
 
 

@@ -283,17 +283,18 @@ def test_command_line(tmp_path):
         assert torch.allclose(got.double(), want, atol=2e-4)
 
 
-def test_synthetic_checkpoint_and_benchmark_tool(tmp_path, monkeypatch):
+@pytest.mark.parametrize("name", ["tiny-kafipel", "tiny-vepivik"])
+def test_synthetic_checkpoint_and_benchmark_tool(tmp_path, monkeypatch, name):
     """The presets write checkpoints that load, and the benchmark tool runs one by name with fake weights."""
     from xfastertransformer_b200.tools.synthetic import preset, write_synthetic_checkpoint
-    c = preset("tiny-kafipel")
+    c = preset(name)
     p = write_synthetic_checkpoint(str(tmp_path / "k"), c, seed=3, std=0.05)
     W = {n: SafetensorsFile(os.path.join(p, "model.safetensors")).read(n, e["shape"])
          for n, e in SafetensorsFile(os.path.join(p, "model.safetensors")).entries.items()}
     toks = list(range(60))
     got = xft.AutoModel.from_pretrained(p, dtype="fp32")([toks])[0].double()
     assert torch.allclose(got, O.forward(c.raw, W, toks), atol=1e-4)
-    r = subprocess.run([sys.executable, os.path.join(ROOT, "benchmarks", "benchmark.py"), "--model_name", "tiny-kafipel", "-in", "20",
+    r = subprocess.run([sys.executable, os.path.join(ROOT, "benchmarks", "benchmark.py"), "--model_name", name, "-in", "20",
                         "-out", "4", "-i", "1"], env=dict(os.environ, XFT_ENGINE="CPU", PYTHONPATH=ROOT), capture_output=True,
                        text=True, timeout=240)
     assert r.returncode == 0, r.stderr[-2000:]

@@ -61,46 +61,97 @@ def kafipel_config(width: int, heads: int, kv_heads: int, ff: int, layers: int, 
     return {"architecture": "Kafipel", "width": width, "vocab": vocab, "norm": {"eps": eps}, "layers": out}
 
 
-LAYERED_PRESETS: Dict[str, dict] = {
-    "tiny-kafipel": dict(width=192, heads=6, kv_heads=2, ff=512, layers=3, vocab=1000, dim=64, window=48),
-    "kafipel-1b": dict(width=2048, heads=16, kv_heads=4, ff=5632, layers=16),
-    "kafipel-8b": dict(width=4096, heads=32, kv_heads=8, ff=14336, layers=32),
+def vepivik_config(width: int, heads: int, kv_heads: int, layers: int, experts: int, top: int, ff: int, shared: int,
+                   vocab: int = 32000, dim: int = 128, rot_dim: int = 64, vdim: int = 128, kv_rank: int = 512, window: int = 1024,
+                   latent_window: int = 4096, latent_only: bool = False, share: bool = True, eps: float = 1e-5,
+                   scale: float = 4.0) -> dict:
+    """config.json of a Vepivik model: attention and latent-attention layers in turn (`latent_only`: the latter alone); with
+    `share`, every second latent layer reads the latents of the one before it."""
+    out, owner, n = [], None, 0
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": shared}}
+    for i in range(layers):
+        if i % 2 == 0 and not latent_only:
+            m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "mask": {"size": window}}
+            out.append({"type": "attention", "mixer": m, "mlp": mlp})
+            continue
+        m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "scale": (dim + rot_dim) ** -0.5,
+             "mask": {"size": latent_window},
+             "rot": {"dims": rot_dim, "base": 10000.0, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+        if share and n % 2 == 1:
+            m["kv_from"] = owner
+        else:
+            owner = i
+        n += 1
+        out.append({"type": "latent_attention", "mixer": m, "mlp": mlp})
+    return {"architecture": "Vepivik", "width": width, "vocab": vocab, "norm": {"eps": eps}, "embedding": {"scale": scale}, "layers": out}
+
+
+LAYERED_PRESETS: Dict[str, tuple] = {
+    "tiny-kafipel": (kafipel_config, dict(width=192, heads=6, kv_heads=2, ff=512, layers=3, vocab=1000, dim=64, window=48)),
+    "kafipel-1b": (kafipel_config, dict(width=2048, heads=16, kv_heads=4, ff=5632, layers=16)),
+    "kafipel-8b": (kafipel_config, dict(width=4096, heads=32, kv_heads=8, ff=14336, layers=32)),
+    "tiny-vepivik": (vepivik_config, dict(width=192, heads=5, kv_heads=1, layers=4, experts=6, top=2, ff=56, shared=72, vocab=1000, dim=40,
+                                          rot_dim=24, vdim=32, kv_rank=72, window=48, latent_window=90)),
+    "vepivik-lite": (vepivik_config, dict(width=2048, heads=16, kv_heads=4, layers=26, experts=64, top=6, ff=1408, shared=2816)),
 }
 
 
 def _write_layered(path: str, cfg: ModelConfig, seed: int, std: float) -> str:
     """config.json and model.safetensors of a layered design, every tensor N(0, std) (norm gains around one)."""
+    from ..models.registry import family_for
     cfg.to_ini(path)
+    spec = family_for(cfg)
     g = torch.Generator().manual_seed(seed)
     W, t = cfg.hidden_size, {}
 
     def put(name, *shape, around=0.0, s=std):
         t[name] = (around + torch.randn(*shape, generator=g) * s).bfloat16()
 
+    def gain(name, n=W):
+        put(name, n, around=1.0, s=0.05)
+
     put("embed", cfg.vocab_size, W)
-    put("final.norm", W, around=1.0, s=0.05)
-    put("head", cfg.vocab_size, W)
+    gain("final.norm")
+    if not spec.tied_head:
+        put("head", cfg.vocab_size, W)
     for i, lc in enumerate(cfg.layers):
-        p, m = f"l{i}.", lc.mixer
-        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if lc.ff else ()):
-            put(p + n, W, around=1.0, s=0.05)
-        put(p + "mix.q", m.heads * m.dim, W)
-        if m.kv_from < 0:
+        p, m, f = f"l{i}.", lc.mixer, lc.moe
+        for n in ("norm1",) + (("norm2",) if lc.ff or f else ()):
+            gain(p + n)
+            if spec.post_norm:
+                gain(p + n + "b")
+        put(p + "mix.q", m.heads * (m.dim + m.rot_dim), W)
+        if m.kind == "latent":
+            if m.kv_from < 0:
+                put(p + "mix.dkv", m.kv_rank + m.rot_dim, W)
+                gain(p + "mix.dkv.norm", m.kv_rank)
+            put(p + "mix.uk", m.heads * m.dim, m.kv_rank)
+            put(p + "mix.uv", m.heads * m.vdim, m.kv_rank)
+            if m.gate:
+                put(p + "mix.g", m.heads * m.vdim, W)
+        elif m.kv_from < 0:
             put(p + "mix.k", m.kv_heads * m.dim, W)
             put(p + "mix.v", m.kv_heads * m.vdim, W)
-        put(p + "mix.sink", m.heads, s=1.0)
+        if spec.sinks:
+            put(p + "mix.sink", m.heads, s=1.0)
         put(p + "mix.o", W, m.heads * m.vdim)
         if lc.ff:
             put(p + "mlp.gate", lc.ff, W)
             put(p + "mlp.up", lc.ff, W)
             put(p + "mlp.down", W, lc.ff)
+        if f:
+            put(p + "mlp.router", f.experts, W)
+            for n, ff in [(f"e{e}", f.ff) for e in range(f.experts)] + ([("shared", f.shared)] if f.shared else []):
+                put(p + f"mlp.{n}.up", ff, W)
+                put(p + f"mlp.{n}.down", W, ff)
     write_safetensors(os.path.join(path, "model.safetensors"), t)
     return path
 
 
 def preset(name: str, **over) -> ModelConfig:
     if name in LAYERED_PRESETS:
-        return ModelConfig.from_dict(kafipel_config(**dict(LAYERED_PRESETS[name], **over)))
+        make, sizes = LAYERED_PRESETS[name]
+        return ModelConfig.from_dict(make(**dict(sizes, **over)))
     if name not in PRESETS:
         from .model_zoo import ZOO          # public model architectures (examples/model_config)
         if name not in ZOO:
