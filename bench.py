@@ -128,9 +128,9 @@ def main():
     ap.add_argument("--input-len", type=int, default=2048)
     ap.add_argument("--dtype", default="bf16")
     ap.add_argument("--kv-dtype", default="bf16")
-    ap.add_argument("--design", default="", choices=["", "kafipel"],
-                    help="instead of the headline workload: this layered design beside Llama at equal sizes (one GPU)")
-    ap.add_argument("--size", default="all", choices=["all", "1b", "8b", "70b-layers"], help="with --design")
+    ap.add_argument("--design", default="", choices=["", "kafipel", "vepivik"],
+                    help="instead of the headline workload: this layered design beside the closest other family (one GPU)")
+    ap.add_argument("--size", default="all", help="with --design: one of its sizes (see benchmarks/bench_layered.py)")
     ap.add_argument("--layers", type=int, default=0, help="debug only: fewer layers (result is flagged invalid)")
     args = ap.parse_args()
     if args.impl == "reference":

@@ -1,6 +1,6 @@
-"""Prefill and decode of a layered design (Kafipel) beside the closest other family (Llama) at equal width, heads,
-feed-forward and depth, and the kernels of both one by one.  Run through ``bench.py --design kafipel [--size NAME]``; one
-GPU, random weights, one JSON line.
+"""Prefill and decode of a layered design beside the closest other family at equal sizes and depth, and the kernels of both
+one by one: Kafipel beside Llama here, Vepivik beside DeepSeek in bench_vepivik.py.  Run through ``bench.py --design NAME
+[--size NAME]``; one GPU, random weights, one JSON line.
 
 Throughput: prompts of `input_len` tokens through `forward()` (prefill and first token), then `steps` decode steps of the
 whole batch (the captured step), both timed with CUDA events.  Kernels: each launched over several sets of inputs that
@@ -37,10 +37,9 @@ def _model(kind, s, tmp):
     return xft.AutoModel.from_pretrained(d, dtype="bf16", kv_cache_dtype="bf16")
 
 
-def throughput(kind, s, steps, warmup, tmp):
+def throughput(model, s, steps, warmup):
     import torch
     from xfastertransformer_b200.ops import native as N
-    model = _model(kind, s, tmp)
     m = model.model
     B, L = s["batch"], s["input_len"]
     ids = torch.randint(0, VOCAB, (B, L), generator=torch.Generator().manual_seed(1)).pin_memory()
@@ -67,8 +66,6 @@ def throughput(kind, s, steps, warmup, tmp):
     out = {"prefill_tokens_per_s": round(B * L / min(pre[1:]) * 1e3), "prefill_ms": round(min(pre[1:]), 2),
            "decode_tokens_per_s": round(B / ms * 1e3, 1), "decode_ms": round(ms, 4), "kernels_per_step": launches[-1],
            "weights_gb": round(m.decoder.weight_bytes() / 1e9, 2)}
-    del model, m
-    torch.cuda.empty_cache()
     return out
 
 
@@ -202,23 +199,36 @@ def kernels(s, peaks):
 
 def run(args, clock_sampler, clock_summary, root):
     os.environ["XFT_FAKE_MODEL"] = "2"
+    import gc
+
     import torch
+
+    from . import bench_vepivik
     peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
     try:
         with open(os.path.join(root, "MEASURED_PEAKS.json")) as f:
             peaks = json.load(f)
     except OSError:
         pass
-    out = {"metric": "layered_design_tokens_per_s", "design": "kafipel", "data": "synthetic token ids; random-init weights",
+    here = globals() if args.design == "kafipel" else vars(bench_vepivik)
+    kinds = {"kafipel": ("kafipel", "kafipel_full", "llama"), "vepivik": ("vepivik", "vepivik_latent", "deepseek")}[args.design]
+    sizes = here["SIZES"]
+    if args.size != "all" and args.size not in sizes:
+        raise SystemExit(f"--size {args.size}: {args.design} has {sorted(sizes)}")
+    out = {"metric": "layered_design_tokens_per_s", "design": args.design, "data": "synthetic token ids; random-init weights",
            "dtype": "bf16", "n_gpus": 1, "steps": args.steps, "warmup": max(args.warmup, 3), "sizes": {}}
     sampler, path = clock_sampler()
-    for name in (SIZES if args.size == "all" else [args.size]):
-        s = SIZES[name]
+    for name in (sizes if args.size == "all" else [args.size]):
+        s = sizes[name]
         r = {"config": s}
-        for kind in ("kafipel", "kafipel_full", "llama"):
+        for kind in kinds:
             with tempfile.TemporaryDirectory() as tmp:
-                r[kind] = throughput(kind, s, args.steps, max(args.warmup, 3), tmp)
-        r["kernels"] = kernels(s, peaks)
+                model = here["_model"](kind, s, tmp)
+                r[kind] = throughput(model, s, args.steps, max(args.warmup, 3))
+                del model
+                gc.collect()
+                torch.cuda.empty_cache()
+        r["kernels"] = here["kernels"](s, peaks)
         torch.cuda.empty_cache()
         out["sizes"][name] = r
     out["clocks"] = clock_summary(sampler, path, 0)

@@ -83,25 +83,6 @@ __device__ __forceinline__ unsigned long long sk_now() {
   asm volatile("mov.u64 %0, %%globaltimer;" : "=l"(t));
   return t;
 }
-// thread-block cluster: rank of this CTA, the cluster-wide barrier in its two halves, shared memory of a peer CTA
-__device__ __forceinline__ uint32_t cluster_ctarank() {
-  uint32_t r;
-  asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r));
-  return r;
-}
-__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
-__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
-__device__ __forceinline__ uint32_t dsmem_addr(uint32_t smem_addr, uint32_t cta_rank) {
-  uint32_t a;
-  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(a) : "r"(smem_addr), "r"(cta_rank));
-  return a;
-}
-__device__ __forceinline__ float ld_dsmem(uint32_t addr) {
-  float v;
-  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
-  return v;
-}
-
 #define SK_STAMP(ev) do { if (p.trace) p.trace[(size_t)blockIdx.x * 8 + (ev)] = sk_now(); } while (0)
 
 // CTA that holds unit u when `units` units are dealt to `G` CTAs as [i * units / G, (i + 1) * units / G).  32-bit

@@ -131,8 +131,6 @@ def _expanded(x, d, cache, block_table, sp, weights, scale, window, out):
                                       N._p(sp.row), len(sp.long), sp.rows, N._p(flat), N._p(ws.status), N._stream()), "latent_gather")
     ws.launches += 1
     per = max(1, min(H, EXPAND_BYTES // (2 * sp.rows * (d.dim + d.vdim))))
-    ldx = max(x.stride(0), x.shape[1])
-    gate = x[:, d.gate_at:] if d.gate else None
     w = _stacked(weights, "ukv", lambda: torch.cat([weights.uk.reshape(H * d.dim, d.rank), weights.uv.reshape(H * d.vdim, d.rank)]))
     for h0 in range(0, H, per):
         n = min(per, H - h0)
@@ -142,12 +140,30 @@ def _expanded(x, d, cache, block_table, sp, weights, scale, window, out):
             kv = torch.empty(sp.rows, n * (d.dim + d.vdim), dtype=x.dtype, device=x.device)
             N.gemm_bf16(flat[:, :d.rank], w[h0 * d.dim:(h0 + n) * d.dim], n * d.dim, out=kv[:, :n * d.dim])
             N.gemm_bf16(flat[:, :d.rank], w[H * d.dim + h0 * d.vdim:H * d.dim + (h0 + n) * d.vdim], n * d.vdim, out=kv[:, n * d.dim:])
-        N._check(_fn("xft_attn_flat_tc")(
-            N._p(x), ldx, d.q_width, d.dim + d.rot, N._p(kv), kv.shape[1], n * d.dim, N._p(flat), W, d.rank, sp.rows, N._p(out),
-            out.stride(0), N._p(gate), ldx if d.gate else 0, N._p(sp.q_start), N._p(sp.q_len), N._p(sp.kv_len), N._p(sp.lo),
-            N._p(sp.row), len(sp.long), x.shape[0], sp.max_q, h0, n, d.dim // 64, d.rot // 64, d.vdim // 64, C.c_float(scale), window,
-            N._p(ws.status), N._stream()), "attn_flat_tc")
-        ws.launches += 1
+        flat_attention(x, d, kv, flat, sp, h0, n, scale, window, out)
+
+
+def flat_attention(x, d, kv, flat, sp, h0, n, scale, window, out):
+    """Heads h0 .. h0 + n - 1 of the packed rows x over expanded keys and values `kv` [rows, n * (dim + vdim)] and the gathered
+    cache rows `flat`, which hold the shared key part (csrc/kernels/latent_prefill_sm100.cu)."""
+    ws = N.Workspace.get(x.device)
+    ldx = max(x.stride(0), x.shape[1])
+    gate = x[:, d.gate_at:] if d.gate else None
+    N._check(_fn("xft_attn_flat_tc")(
+        N._p(x), ldx, d.q_width, d.dim + d.rot, N._p(kv), kv.shape[1], n * d.dim, N._p(flat), flat.shape[1], d.rank, sp.rows,
+        N._p(out), out.stride(0), N._p(gate), ldx if d.gate else 0, N._p(sp.q_start), N._p(sp.q_len), N._p(sp.kv_len), N._p(sp.lo),
+        N._p(sp.row), len(sp.long), x.shape[0], sp.max_q, h0, n, d.dim // 64, d.rot // 64, d.vdim // 64, C.c_float(scale), window,
+        N._p(ws.status), N._stream()), "attn_flat_tc")
+    ws.launches += 1
+
+
+def mla_splits(units: int, keys: int) -> int:
+    """CTAs per (token, 16 heads) of the absorbed kernel: as many as there are SMs, at least two
+    64-key tiles for every one, a power of two up to the portable cluster size."""
+    room, tiles, n = 148, (keys + 63) // 64, 1
+    while n < 8 and units * n * 2 <= room and tiles >= 4 * n:
+        n *= 2
+    return n
 
 
 def _absorbed(x, d, cache, block_table, cu_dev, kv_dev, B, max_kv, weights, scale, window, out):
@@ -173,20 +189,13 @@ def _absorbed(x, d, cache, block_table, cu_dev, kv_dev, B, max_kv, weights, scal
     ws = N.Workspace.get(x.device)
     qa, ol = new(T, H * d.rank), new(T, H * d.rank)
     _heads(x, ldx, d.q_width, hd, wk, H, d.rank, d.dim, qa, H * d.rank, d.rank)
-    nsplit, po, pm = 1, None, None
-    ctas = T * ((H + 15) // 16)
-    if ctas <= ws.attn_counters.numel():
-        seen = min(max_kv, window + 32) if window > 0 else max_kv
-        tiles, least = (seen + 31) // 32, 4 if window > 0 else 8
-        nsplit = max(1, min(296 // ctas, tiles // least if tiles >= 2 * least else 1, 16, ws.PART_O_FLOATS // (ctas * 16 * d.rank)))
-        if nsplit > 1:
-            po, pm = ws.attn_partials(ctas * nsplit * 16 * d.rank, ctas * nsplit * 32)
+    nsplit = mla_splits(T * ((H + 15) // 16), min(max_kv, window) if window > 0 else max_kv)
     nb, _, bs, _ = cache.shape
     LL = C.c_longlong
     qr = x[:, d.dim:]
     N._check(_fn("xft_mla_attention_ext")(
         N._p(qa), LL(d.rank), LL(H * d.rank), N._p(qr), LL(hd), LL(ldx), N._p(ol), LL(d.rank), LL(H * d.rank), N._p(cache),
         N._p(block_table), block_table.stride(0), N._p(cu_dev), N._p(kv_dev), B, T, H, d.rank, bs, nb, C.c_float(scale), window,
-        nsplit, N._p(po), N._p(pm), N._p(ws.attn_counters), N._p(ws.status), N._stream()), "mla_attention")
+        nsplit, N._p(ws.status), N._stream()), "mla_attention")
     ws.launches += 1
     return _heads(ol, H * d.rank, H * d.rank, d.rank, wv, H, d.vdim, d.rank, out, H * d.vdim, d.vdim, gate, ldx)

@@ -71,30 +71,21 @@ def mla_attention(q_nope, q_rope, latent_cache, block_table, cu_q, kv_lens, w_uk
     q_abs = _per_head_gemm(q_ht, wk, Hl, T, L, nope)                 # [Hl*T, L]
     if meta is not None and getattr(meta, "cu_q_dev", None) is not None:
         cu_dev, kv_dev, max_kv, B = meta.cu_q_dev, meta.kv_lens_dev, meta.max_kv, len(kv_lens)
-        decode = meta.is_decode
     else:
         cu_dev = torch.tensor(list(cu_q), dtype=torch.int32, device=dev)
         kv_dev = torch.tensor(list(kv_lens), dtype=torch.int32, device=dev)
         max_kv, B = max(kv_lens), len(kv_lens)
-        decode = all(cu_q[i + 1] - cu_q[i] == 1 for i in range(B))
     o_lat = torch.empty(Hl * T, L, dtype=torch.bfloat16, device=dev)
     nb, _, bs, W = latent_cache.shape
     chunks = (Hl + 15) // 16
-    nsplit, po, pm = 1, None, None
-    if decode:
-        ntiles = (max_kv + 31) // 32
-        ctas = T * chunks
-        nsplit = max(1, min(296 // max(ctas, 1), ntiles // 8 if ntiles >= 16 else 1, 16))
-        if nsplit > 1 and ctas <= ws.attn_counters.numel():
-            po, pm = ws.attn_partials(ctas * nsplit * 16 * L, ctas * nsplit * 32)
-        else:
-            nsplit = 1
+    from .native_latent import mla_splits
+    nsplit = mla_splits(T * chunks, max_kv)
     q_rope = q_rope.contiguous()
     rc = _lib().xft_mla_attention(N._p(q_abs), C.c_longlong(T * L), C.c_longlong(L), N._p(q_rope), C.c_longlong(rope),
                                   C.c_longlong(Hl * rope), N._p(o_lat), C.c_longlong(T * L), C.c_longlong(L),
                                   N._p(latent_cache), N._p(block_table), block_table.stride(0), N._p(cu_dev),
-                                  N._p(kv_dev), B, T, Hl, bs, nb, C.c_float(scale), nsplit, N._p(po), N._p(pm),
-                                  N._p(ws.attn_counters), N._p(ws.status), N._stream())
+                                  N._p(kv_dev), B, T, Hl, bs, nb, C.c_float(scale), nsplit, N._p(None), N._p(None),
+                                  N._p(None), N._p(ws.status), N._stream())
     N._check(rc, "mla_attention")
     ws.launches += 1
     o = _per_head_gemm(o_lat, wv, Hl, T, vd, L)                      # [Hl*T, vd]
