@@ -59,6 +59,11 @@ struct PrefillParams {
   const int* order;           // optional: i-th visited token block (a permutation of 0..t_tiles-1)
   int wide;                   // != 0: bf16 rows leave through shared memory as 256-byte runs (full 128-feature tiles)
   int* status;
+  // token-major kernel only: fp32 rows out, and the grouped form (experts): token tile i is group_tiles[i] = {group, first
+  // row, rows, -} of num_group_tiles[0] tiles, and a group's weight rows start at group * group_w_rows
+  int out_fp32;
+  const int4* group_tiles; const int* num_group_tiles;
+  int group_w_rows;
   BulkArParams ar;
 };
 
@@ -452,7 +457,24 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_tm_kernel(const __grid_co
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int stages = p.stages;
-  const int total = p.n_tiles * p.t_tiles;               // n_tiles: feature tiles of BNF, t_tiles: token blocks of 128
+  // n_tiles: feature tiles of BNF, t_tiles: token blocks of 128 (grouped: at most so many)
+  const int total = p.n_tiles * (p.group_tiles ? min(*p.num_group_tiles, p.t_tiles) : p.t_tiles);
+  // an item's feature tile, first token row, number of rows and first weight row of its group
+  struct Item { int nt, row0, rows, w0; };
+  auto item_of = [&](int item) {
+    Item r;
+    if (p.group_tiles) {
+      const int4 e = p.group_tiles[item / p.n_tiles];
+      r = {item % p.n_tiles, e.y, e.z, e.x * p.group_w_rows};
+    } else {
+      int blk;
+      decode_item(p, item, r.nt, blk);
+      r.row0 = blk * 128;
+      r.rows = p.T - r.row0;
+      r.w0 = 0;
+    }
+    return r;
+  };
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < stages; ++s) {
@@ -484,8 +506,7 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_tm_kernel(const __grid_co
       int it = 0;
       bool ok = true;
       for (int item = blockIdx.x; item < total && ok; item += gridDim.x) {
-        int nt, blk;
-        decode_item(p, item, nt, blk);
+        const Item im = item_of(item);
         for (int kb = 0; kb < p.num_kb; ++kb, ++it) {
           const int s = it % stages;
           const uint32_t ph = (it / stages) & 1;
@@ -495,9 +516,9 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_tm_kernel(const __grid_co
           }
           mbar_expect_tx(&full_bar[s], STAGE_BYTES);
           uint8_t* a = smem + s * STAGE_BYTES;
-          tma_load_2d(a, &tmX, &full_bar[s], kb * 64, blk * 128, hint);
-          tma_load_2d(a + A_BYTES, &tmW, &full_bar[s], kb * 64, nt * BNF, hint);
-          if (DUAL) tma_load_2d(a + A_BYTES + B_BYTES, &tmW, &full_bar[s], kb * 64, p.dual_off + nt * BNF, hint);
+          tma_load_2d(a, &tmX, &full_bar[s], kb * 64, im.row0, hint);
+          tma_load_2d(a + A_BYTES, &tmW, &full_bar[s], kb * 64, im.w0 + im.nt * BNF, hint);
+          if (DUAL) tma_load_2d(a + A_BYTES + B_BYTES, &tmW, &full_bar[s], kb * 64, im.w0 + p.dual_off + im.nt * BNF, hint);
         }
       }
       if (!ok) {
@@ -546,16 +567,15 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_tm_kernel(const __grid_co
     const bool vec = (p.N % 8 == 0) && (p.ldo % 8 == 0) && (!p.residual || p.ldr % 8 == 0);
     int lt = 0;
     for (int item = blockIdx.x; item < total; item += gridDim.x, ++lt) {
-      int nt, blk;
-      decode_item(p, item, nt, blk);
+      const Item im = item_of(item);
       const int a = lt & 1;
       const uint32_t aph = (lt >> 1) & 1;
       mbar_wait_or_abort(&tmem_full[a], aph, p.status, XFT_ERR_WAIT_TMEM, s_abort);
       if (named_bar_or(1, 128, *s_abort != 0)) break;
       tcgen05_fence_after();
       const uint32_t taddr = tmem_base + (uint32_t(q * 32) << 16) + (uint32_t)(a * BNF * NACC);
-      const int t = blk * 128 + row;
-      const bool t_ok = t < p.T;
+      const int t = im.row0 + row;
+      const bool t_ok = row < im.rows;
       __nv_bfloat16* orow = p.out + (size_t)t * p.ldo;
       const __nv_bfloat16* rrow = p.residual ? p.residual + (size_t)t * p.ldr : nullptr;
 #pragma unroll 1
@@ -570,7 +590,7 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_tm_kernel(const __grid_co
           __syncwarp();
           if (lane == 0) mbar_arrive(&tmem_empty[a]);
         }
-        const int n0 = nt * BNF + c;
+        const int n0 = im.nt * BNF + c;
         if (!t_ok || n0 >= p.N) continue;
         float x[16];
 #pragma unroll
@@ -590,7 +610,17 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_tm_kernel(const __grid_co
             x[j] *= u;
           }
         }
-        if (full) {
+        if (p.out_fp32) {
+          float* frow = reinterpret_cast<float*>(p.out) + (size_t)t * p.ldo + n0;
+          if (full) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+              reinterpret_cast<float4*>(frow)[j] = make_float4(x[4 * j], x[4 * j + 1], x[4 * j + 2], x[4 * j + 3]);
+          } else {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) if (n0 + j < p.N) frow[j] = x[j];
+          }
+        } else if (full) {
           if (rrow) {
             const uint4 r0 = *reinterpret_cast<const uint4*>(rrow + n0), r1 = *reinterpret_cast<const uint4*>(rrow + n0 + 8);
             const __nv_bfloat162* h0 = reinterpret_cast<const __nv_bfloat162*>(&r0);
@@ -778,6 +808,26 @@ extern "C" int xft_bulk_ar_layout(long long* out, int n) {
 
 // Token-major persistent GEMM (see gemm_prefill_tm_kernel): Y[T, N] = act(X W^T + bias) [* (X Wu^T + bias_u)] +
 // res_scale * residual, bf16.  gated != 0: gate rows [0, N) and up rows [dual_off, dual_off + N) of W.
+static int prefill_tm(const void* X, int ldx, const void* W, int w_rows, int ldw, PrefillParams& p, int gated, int num_ctas,
+                      cudaStream_t st) {
+  const int bnf = gated ? 128 : 256;
+  p.n_tiles = (p.N + bnf - 1) / bnf;
+  p.num_kb = (p.K + 63) / 64;
+  p.gn = 8;
+  if (num_ctas <= 0) {
+    int dev = 0, sms = 0;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+    num_ctas = sms > 0 ? sms : 148;
+  }
+  CUtensorMap tmW, tmX;
+  int r = make_tensor_map(&tmW, W, (uint64_t)w_rows, (uint64_t)p.K, (uint64_t)ldw, (uint32_t)bnf, 2);
+  if (r) return 1000 - r;
+  r = make_tensor_map(&tmX, X, (uint64_t)p.T, (uint64_t)p.K, (uint64_t)ldx, 128, 2);
+  if (r) return 2000 - r;
+  return gated ? launch_prefill_tm<128, true>(tmX, tmW, p, num_ctas, st) : launch_prefill_tm<256, false>(tmX, tmW, p, num_ctas, st);
+}
+
 extern "C" int xft_gemm_bf16_prefill_tm(const void* X, int ldx, const void* W, int w_rows, int ldw, void* Y, int ldo, int T,
                                         int N, int K, int gated, int dual_off, const float* bias, const void* residual,
                                         int ldr, float res_scale, int act, int* status, int num_ctas, cudaStream_t st) {
@@ -787,21 +837,33 @@ extern "C" int xft_gemm_bf16_prefill_tm(const void* X, int ldx, const void* W, i
   p.N = N; p.T = T; p.K = K; p.out = reinterpret_cast<__nv_bfloat16*>(Y); p.ldo = ldo; p.bias = bias;
   p.residual = reinterpret_cast<const __nv_bfloat16*>(residual); p.ldr = ldr; p.res_scale = res_scale; p.act = act;
   p.status = status; p.dual_off = dual_off;
-  const int bnf = gated ? 128 : 256;
-  p.n_tiles = (N + bnf - 1) / bnf;
   p.t_tiles = (T + 127) / 128;
-  p.num_kb = (K + 63) / 64;
-  p.gn = 8;
-  if (num_ctas <= 0) {
-    int dev = 0, sms = 0;
-    cudaGetDevice(&dev);
-    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-    num_ctas = sms > 0 ? sms : 148;
-  }
-  CUtensorMap tmW, tmX;
-  int r = make_tensor_map(&tmW, W, (uint64_t)w_rows, (uint64_t)K, (uint64_t)ldw, (uint32_t)bnf, 2);
-  if (r) return 1000 - r;
-  r = make_tensor_map(&tmX, X, (uint64_t)T, (uint64_t)K, (uint64_t)ldx, 128, 2);
-  if (r) return 2000 - r;
-  return gated ? launch_prefill_tm<128, true>(tmX, tmW, p, num_ctas, st) : launch_prefill_tm<256, false>(tmX, tmW, p, num_ctas, st);
+  return prefill_tm(X, ldx, W, w_rows, ldw, p, gated, num_ctas, st);
+}
+
+// The same with fp32 rows: Y[T, N] = act(X W^T + bias).
+extern "C" int xft_gemm_bf16_prefill_tm_f32(const void* X, int ldx, const void* W, int w_rows, int ldw, float* Y, int ldo, int T,
+                                            int N, int K, const float* bias, int act, int* status, cudaStream_t st) {
+  if (T <= 0 || N <= 0 || K <= 0) return 0;
+  if ((K & 7) || (ldx & 7) || (ldw & 7)) return -2;
+  PrefillParams p{};
+  p.N = N; p.T = T; p.K = K; p.out = reinterpret_cast<__nv_bfloat16*>(Y); p.ldo = ldo; p.bias = bias; p.res_scale = 1.f; p.act = act;
+  p.status = status; p.out_fp32 = 1;
+  p.t_tiles = (T + 127) / 128;
+  return prefill_tm(X, ldx, W, w_rows, ldw, p, 0, 0, st);
+}
+
+// Rows sorted by group (experts at prompt sizes): token tiles of 128 rows from xft_moe_plan, W [groups * group_w_rows, K];
+// gated: a group's rows are gate [0, N), up [dual_off, dual_off + N).  bf16 rows out.
+extern "C" int xft_gemm_bf16_grouped_tm(const void* X, int ldx, int x_rows, const void* W, int w_rows, int ldw, void* Y, int ldo,
+                                        int N, int K, int gated, int dual_off, int group_w_rows, const void* group_tiles,
+                                        const int* num_group_tiles, int max_tiles, int act, int* status, cudaStream_t st) {
+  if (x_rows <= 0 || N <= 0 || K <= 0 || max_tiles <= 0) return 0;
+  if ((K & 7) || (ldx & 7) || (ldw & 7) || !group_tiles || !num_group_tiles) return -2;
+  PrefillParams p{};
+  p.N = N; p.T = x_rows; p.K = K; p.out = reinterpret_cast<__nv_bfloat16*>(Y); p.ldo = ldo; p.res_scale = 1.f; p.act = act;
+  p.status = status; p.dual_off = dual_off;
+  p.group_tiles = reinterpret_cast<const int4*>(group_tiles); p.num_group_tiles = num_group_tiles; p.group_w_rows = group_w_rows;
+  p.t_tiles = max_tiles;
+  return prefill_tm(X, ldx, W, w_rows, ldw, p, gated, 0, st);
 }

@@ -142,9 +142,13 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const PlanParams p) {
   const int E = p.e1 - p.e0, n = p.T * p.k;
   for (int i = threadIdx.x; i < E; i += blockDim.x) { cnt[i] = 0; cur[i] = 0; }
   __syncthreads();
-  for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    const int e = p.idx[i] - p.e0;
-    if (e >= 0 && e < E) atomicAdd(&cnt[e], 1);
+  // eight pairs per thread and round: their loads are in flight together
+  for (int i0 = threadIdx.x; i0 < n; i0 += 8 * blockDim.x) {
+    int e[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) { const int i = i0 + j * blockDim.x; e[j] = i < n ? p.idx[i] - p.e0 : -1; }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) if (e[j] >= 0 && e[j] < E) atomicAdd(&cnt[e[j]], 1);
   }
   __syncthreads();
   if (threadIdx.x == 0) {
@@ -166,14 +170,25 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const PlanParams p) {
       if (ti < p.max_tiles) p.tiles[ti] = make_int4(e, off[e] + j * p.bn, min(p.bn, cnt[e] - j * p.bn), 0);
     }
   }
-  for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    const int e = p.idx[i] - p.e0;
-    int r = -1;
-    if (e >= 0 && e < E) {
-      r = off[e] + atomicAdd(&cur[e], 1);
-      if (r < p.max_rows) { p.src_tok[r] = i / p.k; p.row_w[r] = p.w[i]; } else r = -1;
+  for (int i0 = threadIdx.x; i0 < n; i0 += 8 * blockDim.x) {
+    int e[8], r[8];
+    float w[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int i = i0 + j * blockDim.x;
+      e[j] = i < n ? p.idx[i] - p.e0 : -1;
+      w[j] = i < n ? p.w[i] : 0.f;
     }
-    p.pos[i] = r;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) r[j] = e[j] >= 0 && e[j] < E ? off[e[j]] + atomicAdd(&cur[e[j]], 1) : -1;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int i = i0 + j * blockDim.x;
+      if (i >= n) break;
+      if (r[j] >= p.max_rows) r[j] = -1;
+      if (r[j] >= 0) { p.src_tok[r[j]] = i / p.k; p.row_w[r[j]] = w[j]; }
+      p.pos[i] = r[j];
+    }
   }
 }
 
@@ -189,23 +204,69 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const bf16* __restrict_
   for (int i = threadIdx.x; i < H / 8; i += 128) d[i] = s[i];
 }
 
-// y[t] = sum_s ys[pos[t,s]] (already scaled by the routing weight) + add1[t] + add2[t]   (fp32 sum, bf16 out)
-__global__ void __launch_bounds__(256) moe_combine_kernel(const float* __restrict__ ys, const int* __restrict__ pos, int k,
-                                                          const float* __restrict__ add1, const bf16* __restrict__ add2,
-                                                          int ld2, bf16* __restrict__ y, float* __restrict__ y32, int H) {
+__device__ __forceinline__ void moe_load(const float* p, float (&v)[1]) { v[0] = p[0]; }
+__device__ __forceinline__ void moe_load(const bf16* p, float (&v)[1]) { v[0] = __bfloat162float(p[0]); }
+__device__ __forceinline__ void moe_load(const float* p, float (&v)[4]) {
+  const float4 f = *reinterpret_cast<const float4*>(p);
+  v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+}
+__device__ __forceinline__ void moe_load(const bf16* p, float (&v)[4]) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+}
+
+// y[t] = sum_s w[t,s] ys[pos[t,s]] + add1[t] + add2[t]   (fp32 sum, bf16 or fp32 out).  w null: the rows of ys carry their
+// weight already.  VEC: four columns per thread (H and ld2 multiples of 4).  A row's positions are read first, so that all
+// its loads are in flight together.
+template <typename YT, bool VEC>
+__global__ void __launch_bounds__(256) moe_combine_kernel(const YT* __restrict__ ys, const int* __restrict__ pos,
+                                                          const float* __restrict__ w, int k, const float* __restrict__ add1,
+                                                          const bf16* __restrict__ add2, int ld2, bf16* __restrict__ y,
+                                                          float* __restrict__ y32, int H) {
+  constexpr int V = VEC ? 4 : 1;
   grid_dep_launch();
   grid_dep_wait();
   const int t = blockIdx.x;
-  for (int i = threadIdx.x; i < H; i += 256) {
-    float a = 0.f;
-    for (int s = 0; s < k; ++s) {
-      const int r = pos[t * k + s];
-      if (r >= 0) a += ys[(size_t)r * H + i];
+  const int i = (blockIdx.y * 256 + threadIdx.x) * V;
+  if (i >= H) return;
+  float a[V], v[V];
+#pragma unroll
+  for (int c = 0; c < V; ++c) a[c] = 0.f;
+  for (int s0 = 0; s0 < k; s0 += 8) {
+    int r[8];
+    float f[8], x[8][V];
+#pragma unroll
+    for (int s = 0; s < 8; ++s) {
+      r[s] = s0 + s < k ? pos[t * k + s0 + s] : -1;
+      f[s] = w && s0 + s < k ? w[t * k + s0 + s] : 1.f;
     }
-    if (add1) a += add1[(size_t)t * H + i];
-    if (add2) a += __bfloat162float(add2[(size_t)t * ld2 + i]);
-    if (y32) y32[(size_t)t * H + i] = a;
-    else y[(size_t)t * H + i] = __float2bfloat16(a);
+#pragma unroll
+    for (int s = 0; s < 8; ++s)
+      if (r[s] >= 0) moe_load(ys + (size_t)r[s] * H + i, x[s]);
+#pragma unroll
+    for (int s = 0; s < 8; ++s)
+      if (r[s] >= 0)
+#pragma unroll
+        for (int c = 0; c < V; ++c) a[c] += f[s] * x[s][c];
+  }
+  if (add1) {
+    moe_load(add1 + (size_t)t * H + i, v);
+#pragma unroll
+    for (int c = 0; c < V; ++c) a[c] += v[c];
+  }
+  if (add2) {
+    moe_load(add2 + (size_t)t * ld2 + i, v);
+#pragma unroll
+    for (int c = 0; c < V; ++c) a[c] += v[c];
+  }
+  if (y32) {
+    if (VEC) *reinterpret_cast<float4*>(y32 + (size_t)t * H + i) = make_float4(a[0], a[V > 1 ? 1 : 0], a[V > 2 ? 2 : 0], a[V > 3 ? 3 : 0]);
+    else y32[(size_t)t * H + i] = a[0];
+  } else {
+#pragma unroll
+    for (int c = 0; c < V; ++c) y[(size_t)t * H + i + c] = __float2bfloat16(a[c]);
   }
 }
 
@@ -239,10 +300,28 @@ extern "C" int xft_moe_gather(const void* x, int ldx, const int* src_tok, const 
   return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }
 
+template <typename YT>
+static int launch_combine(const YT* ys, const int* pos, const float* w, int k, const float* add1, const bf16* add2, int ld2, void* y,
+                          float* y32, int T, int H, cudaStream_t st) {
+  const bool vec = H % 4 == 0 && (!add2 || ld2 % 4 == 0) &&
+                   ((reinterpret_cast<uintptr_t>(ys) | reinterpret_cast<uintptr_t>(add1) | reinterpret_cast<uintptr_t>(add2) |
+                     reinterpret_cast<uintptr_t>(y32)) & 15) == 0;
+  const int per = vec ? 1024 : 256;
+  const dim3 grid(T, (H + per - 1) / per);
+  cudaError_t e = vec ? launch_pdl(moe_combine_kernel<YT, true>, grid, dim3(256), 0, st, ys, pos, w, k, add1, add2, ld2, (bf16*)y, y32, H)
+                      : launch_pdl(moe_combine_kernel<YT, false>, grid, dim3(256), 0, st, ys, pos, w, k, add1, add2, ld2, (bf16*)y, y32, H);
+  return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
+}
+
 extern "C" int xft_moe_combine(const float* ys, const int* pos, int k, const float* add1, const void* add2, int ld2, void* y,
                                float* y32, int T, int H, cudaStream_t st) {
   if (T <= 0) return 0;
-  cudaError_t e = launch_pdl(moe_combine_kernel, dim3(T), dim3(256), 0, st, ys, pos, k, add1, (const bf16*)add2, ld2, (bf16*)y,
-                             y32, H);
-  return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
+  return launch_combine<float>(ys, pos, nullptr, k, add1, (const bf16*)add2, ld2, y, y32, T, H, st);
+}
+
+// Prompt sizes: bf16 rows, weighted here with w [T, k].
+extern "C" int xft_moe_combine_bf16(const void* ys, const int* pos, const float* w, int k, const float* add1, const void* add2,
+                                    int ld2, void* y, float* y32, int T, int H, cudaStream_t st) {
+  if (T <= 0) return 0;
+  return launch_combine<bf16>((const bf16*)ys, pos, w, k, add1, (const bf16*)add2, ld2, y, y32, T, H, st);
 }

@@ -306,7 +306,9 @@ class LayeredDecoder(Decoder):
         idx, w = ops.route(logits, "deepseek", f.top, norm_topk=True, scoring="softmax")
         shared = None
         if L.shared is not None:
-            shared = ops.linear(ops.linear(h, L.shared[0], act=L.act), L.shared[1], out_dtype=torch.float32)
+            # few rows: the product leaves in fp32; prompts: in the activation type, like the experts' own rows
+            shared = ops.linear(ops.linear(h, L.shared[0], act=L.act), L.shared[1],
+                                out_dtype=torch.float32 if h.shape[0] <= 128 else None)
         out = ops.moe_experts(h, idx, w, L.experts, L.act, L.e0, gated=False, add=shared)
         if self.tp > 1:
             peer = getattr(self.ctx, "peer", None)

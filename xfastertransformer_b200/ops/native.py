@@ -257,6 +257,14 @@ def gemm_bf16(x, w, N, gated=False, dual_off=0, bias=None, act=None, residual=No
         _check(rc, "gemm_bf16_prefill_tm")
         ws.launches += 1
         return out
+    if _ENV().gemm_prefill_tm and T > 128 and fp32 and row_scale is None and residual is None and not gated and K <= 8192 \
+            and out.stride(1) == 1 and force_splits == 0:
+        fn = lib().xft_gemm_bf16_prefill_tm_f32
+        fn.restype = C.c_int
+        _check(fn(_p(x2), ldx, _p(w), w.shape[0], w.stride(0), _p(out), out.stride(0), T, N, K, _p(bias), _ACT[act], _p(ws.status),
+                  _stream()), "gemm_bf16_prefill_tm_f32")
+        ws.launches += 1
+        return out
     if _ENV().gemm_persistent and T > 128 and gated and not fp32 and row_scale is None and out.stride(1) == 1 \
             and residual is None:
         # gated form of the persistent kernel: four 128-column accumulators, act(gate) * up on the way out

@@ -133,7 +133,7 @@ def moe_experts(x, idx, w, experts, act="silu", expert_offset=0, packed=None, ex
     exchange; it only picks the token tile of the grouped GEMMs."""
     pk = packed or pack_experts(experts)
     if add is not None:
-        assert add.dtype == torch.float32 and add.is_contiguous()
+        assert add.dtype in (torch.float32, torch.bfloat16) and add.is_contiguous() and add.shape[-1] == x.shape[-1]
     if x.dtype == torch.float32:
         return _experts_f32(x.reshape(-1, x.shape[-1]), idx.int(), w.contiguous(), pk, act, expert_offset, gated, add)
     x2, ldx = N._rows2d(x)
@@ -157,6 +157,7 @@ def moe_experts(x, idx, w, experts, act="silu", expert_offset=0, packed=None, ex
     N._check(lib.xft_moe_plan(N._p(idx32), N._p(w.contiguous()), T, k, expert_offset, expert_offset + E, bn, N._p(pos),
                               N._p(src), N._p(row_w), N._p(tiles), N._p(meta), max_tiles, max_rows, N._stream()),
              "moe_plan")
+    add32, add16 = (add, None) if add is None or add.dtype == torch.float32 else (None, add)
     xs = torch.empty(max_rows, H, dtype=torch.bfloat16, device=dev)
     N._check(lib.xft_moe_gather(N._p(x2), ldx, N._p(src), N._p(meta), N._p(xs), max_rows, H, N._stream()), "moe_gather")
     h1 = torch.empty(max_rows, I, dtype=torch.bfloat16, device=dev)
@@ -169,8 +170,24 @@ def moe_experts(x, idx, w, experts, act="silu", expert_offset=0, packed=None, ex
                                        N._p(pk["dns"]), pk["dns"].shape[1], N._p(tiles), N._p(meta), max_tiles, min(bn, 128),
                                        N._p(row_w), 0, N._p(ws.status), N._stream()), "grouped fp8 down")
         out = torch.empty(T, H, dtype=torch.float32, device=dev)
-        N._check(lib.xft_moe_combine(N._p(ys), N._p(pos), k, N._p(add), N._p(None), 0, N._p(None), N._p(out), T, H,
-                                     N._stream()), "moe_combine")
+        N._check(lib.xft_moe_combine(N._p(ys), N._p(pos), k, N._p(add32), N._p(add16), H, N._p(None), N._p(out), T, H,
+                                 N._stream()), "moe_combine")
+        ws.launches += 5
+        return out
+    if bn == 128:
+        # prompt sizes: the token-major persistent kernel; rows stay bf16 until the weighted sum
+        y16 = torch.empty(max_rows, H, dtype=torch.bfloat16, device=dev)
+        fn = lib.xft_gemm_bf16_grouped_tm
+        fn.restype = C.c_int
+        N._check(fn(N._p(xs), H, max_rows, N._p(pk["gu"]), E * up, H, N._p(h1), I, I, H, int(gated), I, up, N._p(tiles), N._p(meta),
+                    max_tiles, N._ACT[act], N._p(ws.status), N._stream()), "grouped gate_up")
+        N._check(fn(N._p(h1), I, max_rows, N._p(pk["dn"]), E * H, I, N._p(y16), H, H, I, 0, 0, H, N._p(tiles), N._p(meta), max_tiles,
+                    0, N._p(ws.status), N._stream()), "grouped down")
+        out = torch.empty(T, H, dtype=torch.float32, device=dev)
+        fn = lib.xft_moe_combine_bf16
+        fn.restype = C.c_int
+        N._check(fn(N._p(y16), N._p(pos), N._p(w.contiguous()), k, N._p(add32), N._p(add16), H, N._p(None), N._p(out), T, H,
+                    N._stream()), "moe_combine")
         ws.launches += 5
         return out
     N._check(lib.xft_gemm_bf16_grouped(N._p(xs), H, max_rows, N._p(pk["gu"]), E * up, H, N._p(h1), I, 0, I, H, int(gated), I,
@@ -181,7 +198,7 @@ def moe_experts(x, idx, w, experts, act="silu", expert_offset=0, packed=None, ex
                                        N._p(tiles), N._p(meta), max_tiles, bn, N._p(row_w), 0, N._p(ws.status),
                                        N._stream()), "grouped down")
     out = torch.empty(T, H, dtype=torch.float32, device=dev)
-    N._check(lib.xft_moe_combine(N._p(ys), N._p(pos), k, N._p(add), N._p(None), 0, N._p(None), N._p(out), T, H,
+    N._check(lib.xft_moe_combine(N._p(ys), N._p(pos), k, N._p(add32), N._p(add16), H, N._p(None), N._p(out), T, H,
                                  N._stream()), "moe_combine")
     ws.launches += 5
     return out
