@@ -353,6 +353,12 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
 #pragma unroll 1
         for (int c = 0; c < BN && peers_ok; c += 16) {
           float g[16], u[16];
+          __nv_bfloat16 gt[16];                  // gates of the chunk, requested together and before the accumulator
+          if (p.gate && n_ok) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+              gt[j] = p.gate[(size_t)min(t0 + c + j, p.T - 1) * p.ldg + y_col0 + n];
+          }
           if (!fused_ar) {
             load_acc(c, g, u);
           } else if (!i_reduce) {
@@ -422,7 +428,7 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
                   x = apply_act(x, p.act);
                   if (DUAL && !pair) x *= (u[j] * (rs * ts) + bias_u);
                   if (p.col_scale) x *= p.col_scale[t];
-                  if (p.gate) x = __fdividef(x, 1.f + __expf(-__bfloat162float(p.gate[(size_t)t * p.ldg + y_col0 + n])));
+                  if (p.gate) x = __fdividef(x, 1.f + __expf(-__bfloat162float(gt[j])));
                   if (p.residual) x += p.res_scale * __bfloat162float(p.residual[(size_t)t * p.ldr + n]);
                   g[j] = x;                     // kept for the two-shot broadcast below
                 }

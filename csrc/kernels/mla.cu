@@ -11,9 +11,9 @@
 //
 // One lane of the ninth warp feeds a ring of 64-key tiles (a cache block, or a part of one) with TMA, 64 columns per box.
 // Warps 0-7: warp w computes the partial scores of keys 16 (w / 2) .. + 15 over one half of the dimensions, with that half
-// of Q in its registers for the whole kernel; the partial scores meet in shared memory, where every warp does the (small)
-// online softmax of the tile for itself; then warp w adds P C for its eighth of the value columns.  Long contexts are split
-// over the CTAs of a cluster, which merge through distributed shared memory, each a part of the columns.
+// of Q in its registers for the whole kernel; the partial scores meet in shared memory, where warp w does the online softmax
+// of rows 2w and 2w + 1 and leaves their weights as bf16; then warp w adds P C for its eighth of the value columns.  Long
+// contexts are split over the CTAs of a cluster, which merge through distributed shared memory, each a part of the columns.
 //
 // A sliding window restricts the tiles to those that hold a visible key.
 #include "ptx.cuh"
@@ -71,7 +71,7 @@ template <int LAT>
 struct MlaCfg {
   static constexpr int DK = LAT + ROPE;
   static constexpr int STAGE_BYTES = MKT * DK * 2;
-  static constexpr int SX_BYTES = 2 * 2 * 16 * kMlaSx * 4;             // [tile parity][half of the dimensions][row][key]
+  static constexpr int SX_BYTES = 2 * 16 * kMlaSx * 4 + 16 * MKT * 2;  // scores [half of the dimensions][row][key], weights
   static constexpr int FIXED = 16 * DK * 2 + SX_BYTES + 1024;
   static constexpr int STAGES = (225 * 1024 - FIXED) / STAGE_BYTES < 6 ? (225 * 1024 - FIXED) / STAGE_BYTES : 6;
   static constexpr int SMEM = FIXED + STAGES * STAGE_BYTES;
@@ -89,8 +89,9 @@ __global__ void __launch_bounds__(384, 1) mla_attn_kernel(const __grid_constant_
   bf16* ring = reinterpret_cast<bf16*>(base);                          // [STAGES][DK / 64][64][64]
   bf16* qs = reinterpret_cast<bf16*>(base + STAGES * Cfg::STAGE_BYTES);
   float* sx = reinterpret_cast<float*>(qs + 16 * DK);
+  bf16* ps = reinterpret_cast<bf16*>(sx + 2 * 16 * kMlaSx);
   __shared__ uint64_t full_bar[STAGES], empty_bar[STAGES];
-  __shared__ float s_ml[16][2], s_fac[16][8];
+  __shared__ float s_ml[16][2], s_fac[16][8], s_corr[16];
   static_assert(16 * PITCH * 4 <= STAGES * Cfg::STAGE_BYTES, "the merge buffer lies over the ring");
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   if (tid == 0) {
@@ -176,7 +177,6 @@ __global__ void __launch_bounds__(384, 1) mla_attn_kernel(const __grid_constant_
       const int st = n % STAGES;
       const bool ok = mbar_wait(&full_bar[st], (n / STAGES) & 1, p.status, XFT_ERR_WAIT_FULL);
       bf16* kt = ring + (size_t)st * (Cfg::STAGE_BYTES / 2);
-      float* sb = sx + (n & 1) * (2 * 16 * kMlaSx);
       {
         float s[4][4];                                                 // two 8-key tiles, even and odd steps
 #pragma unroll
@@ -188,7 +188,7 @@ __global__ void __launch_bounds__(384, 1) mla_attn_kernel(const __grid_constant_
           mla_mma(s[(ks & 1) * 2], qa[ks], bb[0], bb[1]);
           mla_mma(s[(ks & 1) * 2 + 1], qa[ks], bb[2], bb[3]);
         }
-        float* sd = sb + dh * (16 * kMlaSx) + kg * 16 + qc;
+        float* sd = sx + dh * (16 * kMlaSx) + kg * 16 + qc;
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
           *reinterpret_cast<float2*>(sd + r0 * kMlaSx + j * 8) = make_float2(s[j][0] + s[j + 2][0], s[j][1] + s[j + 2][1]);
@@ -196,58 +196,37 @@ __global__ void __launch_bounds__(384, 1) mla_attn_kernel(const __grid_constant_
         }
       }
       if (named_bar_or(1, 256, !ok)) break;                            // scores complete (or all warps give up together)
-      // ---- online softmax of the tile (every warp keeps identical m, l) ----
-      float pv[2][16];                                                 // [row r0 / r1][step(4) x {2q, 2q+1, 2q+8, 2q+9}]
-      float mx[2] = {-INFINITY, -INFINITY};
-      const int k0 = (t_begin + n) * MKT;
-      const bool part = k0 + MKT > n_keys || k0 < key_lo;
-#pragma unroll
-      for (int ks = 0; ks < 4; ++ks)
-#pragma unroll
-        for (int e = 0; e < 2; ++e)
-#pragma unroll
-          for (int r = 0; r < 2; ++r) {
-            const float* a = sb + (r ? r1 : r0) * kMlaSx + ks * 16 + e * 8 + qc;
-            const float2 x = *reinterpret_cast<const float2*>(a), y = *reinterpret_cast<const float2*>(a + 16 * kMlaSx);
-            float v0 = (x.x + y.x) * p.scale, v1 = (x.y + y.y) * p.scale;
-            if (part) {
-              const int key = k0 + ks * 16 + e * 8 + qc;
-              if (key >= n_keys || key < key_lo) v0 = -INFINITY;
-              if (key + 1 >= n_keys || key + 1 < key_lo) v1 = -INFINITY;
-            }
-            pv[r][ks * 4 + e * 2] = v0;
-            pv[r][ks * 4 + e * 2 + 1] = v1;
-            mx[r] = fmaxf(mx[r], fmaxf(v0, v1));
-          }
-      float cf[2];
+      // ---- online softmax of this warp's two rows: two keys per lane ----
+      const int k0 = (t_begin + n) * MKT, key = k0 + 2 * lane;
+      const bool see0 = key < n_keys && key >= key_lo, see1 = key + 1 < n_keys && key + 1 >= key_lo;
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
-        mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
-        mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
-        const float mn = fmaxf(m[r], mx[r]);
-        cf[r] = mn == -INFINITY ? 1.f : __expf(m[r] - mn);
+        const int row = 2 * warp + r;
+        const float* a = sx + row * kMlaSx + 2 * lane;
+        const float2 x = *reinterpret_cast<const float2*>(a), y = *reinterpret_cast<const float2*>(a + 16 * kMlaSx);
+        const float v0 = see0 ? (x.x + y.x) * p.scale : -INFINITY, v1 = see1 ? (x.y + y.y) * p.scale : -INFINITY;
+        float mx = fmaxf(v0, v1);
+#pragma unroll
+        for (int i = 16; i > 0; i >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, i));
+        const float mn = fmaxf(m[r], mx);                              // finite: every visited tile holds a visible key
+        const float c = __expf(m[r] - mn), p0 = __expf(v0 - mn), p1 = __expf(v1 - mn);
         m[r] = mn;
-        float sum = 0.f;
-#pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          pv[r][i] = pv[r][i] == -INFINITY ? 0.f : __expf(pv[r][i] - mn);
-          sum += pv[r][i];
-        }
-        l[r] = l[r] * cf[r] + sum;                                     // per-lane partial row sums
+        l[r] = l[r] * c + p0 + p1;                                     // per-lane partial sums
+        if (lane == 0) s_corr[row] = c;
+        *reinterpret_cast<uint32_t*>(mla_ptr<16>(ps, row, lane >> 2) + 2 * (lane & 3)) = mla_pack(p0, p1);
       }
+      named_bar_sync(1, 256);
       if (has_cols) {
-        if (__any_sync(0xffffffffu, cf[0] != 1.f || cf[1] != 1.f)) {
+        const float c0 = s_corr[r0], c1 = s_corr[r1];
+        if (__any_sync(0xffffffffu, c0 != 1.f || c1 != 1.f)) {
 #pragma unroll
-          for (int i = 0; i < NT; ++i) { o[i][0] *= cf[0]; o[i][1] *= cf[0]; o[i][2] *= cf[1]; o[i][3] *= cf[1]; }
+          for (int i = 0; i < NT; ++i) { o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1; }
         }
         // ---- O[:, this warp's columns] += P · C ----
 #pragma unroll
         for (int ks = 0; ks < 4; ++ks) {
           uint32_t a[4];
-          a[0] = mla_pack(pv[0][ks * 4 + 0], pv[0][ks * 4 + 1]);
-          a[1] = mla_pack(pv[1][ks * 4 + 0], pv[1][ks * 4 + 1]);
-          a[2] = mla_pack(pv[0][ks * 4 + 2], pv[0][ks * 4 + 3]);
-          a[3] = mla_pack(pv[1][ks * 4 + 2], pv[1][ks * 4 + 3]);
+          mla_ldsm(a, mla_ptr<16>(ps, (lane & 7) + ((lane >> 3) & 1) * 8, ks * 2 + (lane >> 4)));
 #pragma unroll
           for (int j = 0; j < NT; j += 2) {
             uint32_t bb[4];
@@ -262,8 +241,9 @@ __global__ void __launch_bounds__(384, 1) mla_attn_kernel(const __grid_constant_
     }
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
-      l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
-      l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
+#pragma unroll
+      for (int i = 16; i > 0; i >>= 1) l[r] += __shfl_xor_sync(0xffffffffu, l[r], i);
+      if (lane == 0) { s_ml[2 * warp + r][0] = m[r]; s_ml[2 * warp + r][1] = l[r]; }
     }
     named_bar_sync(1, 256);                                            // every issued tile was consumed: the ring is idle
     if (has_cols) {
@@ -274,7 +254,6 @@ __global__ void __launch_bounds__(384, 1) mla_attn_kernel(const __grid_constant_
         *reinterpret_cast<float2*>(mo + r1 * PITCH + d) = make_float2(o[j][2], o[j][3]);
       }
     }
-    if (warp == 0 && (lane & 3) == 0) { s_ml[r0][0] = m[0]; s_ml[r0][1] = l[0]; s_ml[r1][0] = m[1]; s_ml[r1][1] = l[1]; }
   }
   // ---- merge: each CTA of the cluster finishes LAT / nsplit columns ----
   __syncwarp();

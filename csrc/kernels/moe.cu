@@ -135,12 +135,15 @@ struct PlanParams {
   int* pos; int* src_tok; float* row_w; int4* tiles; int* meta; int max_tiles; int max_rows;
 };
 
+// Counters are per warp (and expert), so that pairs only collide with those of their own 32 lanes.
 __global__ void __launch_bounds__(1024) moe_plan_kernel(const PlanParams p) {
-  __shared__ int cnt[256], off[257], cur[256], toff[257];
+  extern __shared__ int cur[];                  // [32 warps][E]: counts, then the warp's next row of each expert
+  __shared__ int cnt[256], off[257], toff[257];
   grid_dep_launch();
   grid_dep_wait();
   const int E = p.e1 - p.e0, n = p.T * p.k;
-  for (int i = threadIdx.x; i < E; i += blockDim.x) { cnt[i] = 0; cur[i] = 0; }
+  int* mine = cur + (threadIdx.x >> 5) * E;
+  for (int i = threadIdx.x; i < 32 * E; i += blockDim.x) cur[i] = 0;
   __syncthreads();
   // eight pairs per thread and round: their loads are in flight together
   for (int i0 = threadIdx.x; i0 < n; i0 += 8 * blockDim.x) {
@@ -148,7 +151,13 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const PlanParams p) {
 #pragma unroll
     for (int j = 0; j < 8; ++j) { const int i = i0 + j * blockDim.x; e[j] = i < n ? p.idx[i] - p.e0 : -1; }
 #pragma unroll
-    for (int j = 0; j < 8; ++j) if (e[j] >= 0 && e[j] < E) atomicAdd(&cnt[e[j]], 1);
+    for (int j = 0; j < 8; ++j) if (e[j] >= 0 && e[j] < E) atomicAdd(&mine[e[j]], 1);
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < E; e += blockDim.x) {      // counts of the warps -> where each one's rows start
+    int o = 0;
+    for (int w = 0; w < 32; ++w) { const int c = cur[w * E + e]; cur[w * E + e] = o; o += c; }
+    cnt[e] = o;
   }
   __syncthreads();
   if (threadIdx.x == 0) {
@@ -180,7 +189,7 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const PlanParams p) {
       w[j] = i < n ? p.w[i] : 0.f;
     }
 #pragma unroll
-    for (int j = 0; j < 8; ++j) r[j] = e[j] >= 0 && e[j] < E ? off[e[j]] + atomicAdd(&cur[e[j]], 1) : -1;
+    for (int j = 0; j < 8; ++j) r[j] = e[j] >= 0 && e[j] < E ? off[e[j]] + atomicAdd(&mine[e[j]], 1) : -1;
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       const int i = i0 + j * blockDim.x;
@@ -288,7 +297,7 @@ extern "C" int xft_moe_plan(const int* idx, const float* w, int T, int k, int e0
                             float* row_w, void* tiles, int* meta, int max_tiles, int max_rows, cudaStream_t st) {
   if (e1 - e0 > 256 || e1 <= e0) return -1;
   PlanParams p{idx, w, T, k, e0, e1, bn, pos, src_tok, row_w, reinterpret_cast<int4*>(tiles), meta, max_tiles, max_rows};
-  cudaError_t e = launch_pdl(moe_plan_kernel, dim3(1), dim3(1024), 0, st, p);
+  cudaError_t e = launch_pdl(moe_plan_kernel, dim3(1), dim3(1024), (size_t)32 * (e1 - e0) * sizeof(int), st, p);
   return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }
 

@@ -157,11 +157,15 @@ def flat_attention(x, d, kv, flat, sp, h0, n, scale, window, out):
     ws.launches += 1
 
 
+# clusters of n CTAs (one CTA per SM) that B200 holds at a time: its GPCs have 16 to 20 SMs
+CLUSTERS = {2: 74, 4: 33, 8: 15}
+
+
 def mla_splits(units: int, keys: int) -> int:
-    """CTAs per (token, 16 heads) of the absorbed kernel: as many as there are SMs, at least two
-    64-key tiles for every one, a power of two up to the portable cluster size."""
-    room, tiles, n = 148, (keys + 63) // 64, 1
-    while n < 8 and units * n * 2 <= room and tiles >= 4 * n:
+    """CTAs per (token, 16 heads) of the absorbed kernel, which form a cluster: as many as run in one wave, with at least two
+    64-key tiles each."""
+    tiles, n = (keys + 63) // 64, 1
+    while n < 8 and units <= CLUSTERS[2 * n] and tiles >= 4 * n:
         n *= 2
     return n
 
