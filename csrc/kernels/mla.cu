@@ -9,11 +9,14 @@
 // SAME latent rows (multi-query attention with a LAT + 64 wide key and a LAT wide value), so a CTA takes 16 heads of one
 // query token as its 16 MMA rows and streams the sequence's latent tiles once.
 //
-// One lane of the ninth warp feeds a ring of 64-key tiles (a cache block, or a part of one) with TMA, 64 columns per box.
+// One lane of the ninth warp feeds a ring of 32-key half tiles with TMA, 64 columns per box; the other eight warps work on
+// 64-key tiles (a cache block, or a part of one).
 // Warps 0-7: warp w computes the partial scores of keys 16 (w / 2) .. + 15 over one half of the dimensions, with that half
 // of Q in its registers for the whole kernel; the partial scores meet in shared memory, where warp w does the online softmax
 // of rows 2w and 2w + 1 and leaves their weights as bf16; then warp w adds P C for its eighth of the value columns.  Long
-// contexts are split over the CTAs of a cluster, which merge through distributed shared memory, each a part of the columns.
+// contexts are split over the CTAs of a cluster, which merge through distributed shared memory, each a part of the columns;
+// when that leaves SMs idle, over several clusters, whose parts meet in global scratch (the CTA that arrives last on a part
+// of the columns finishes it; nobody waits).
 //
 // A sliding window restricts the tiles to those that hold a visible key.
 #include "ptx.cuh"
@@ -37,7 +40,8 @@ struct MlaParams {
   int B, T, hl, bs, num_blocks;
   float scale;
   int window;                                    // keys within `window` positions are visible (2^30: all)
-  int nsplit;                                    // CTAs per (token, 16 heads) = cluster size
+  int nsplit, groups;                            // cluster size; clusters per (token, 16 heads)
+  float* part_o; float* part_ml; int* counters;  // groups > 1: [unit][group][16][LAT], [unit][group][rank][16][2], [unit][rank]
   int* status;
 };
 
@@ -70,14 +74,14 @@ __device__ __forceinline__ bf16* mla_ptr(bf16* base, int row, int chunk) {
 template <int LAT>
 struct MlaCfg {
   static constexpr int DK = LAT + ROPE;
-  static constexpr int STAGE_BYTES = MKT * DK * 2;
+  static constexpr int STAGE_BYTES = MKT / 2 * DK * 2;                 // half a tile
   static constexpr int SX_BYTES = 2 * 16 * kMlaSx * 4 + 16 * MKT * 2;  // scores [half of the dimensions][row][key], weights
   static constexpr int FIXED = 16 * DK * 2 + SX_BYTES + 1024;
-  static constexpr int STAGES = (225 * 1024 - FIXED) / STAGE_BYTES < 6 ? (225 * 1024 - FIXED) / STAGE_BYTES : 6;
+  static constexpr int STAGES = (225 * 1024 - FIXED) / STAGE_BYTES < 12 ? (225 * 1024 - FIXED) / STAGE_BYTES : 12;
   static constexpr int SMEM = FIXED + STAGES * STAGE_BYTES;
 };
 
-// grid (tokens * head_chunks, nsplit), clusters of (1, nsplit); 384 threads
+// grid (tokens * head_chunks, nsplit * groups), clusters of (1, nsplit); 384 threads
 template <int LAT>
 __global__ void __launch_bounds__(384, 1) mla_attn_kernel(const __grid_constant__ CUtensorMap tmC, const MlaParams p) {
   using Cfg = MlaCfg<LAT>;
@@ -86,12 +90,13 @@ __global__ void __launch_bounds__(384, 1) mla_attn_kernel(const __grid_constant_
   constexpr int PITCH = LAT + 4;                                       // merge buffer row
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  bf16* ring = reinterpret_cast<bf16*>(base);                          // [STAGES][DK / 64][64][64]
+  bf16* ring = reinterpret_cast<bf16*>(base);                          // [STAGES][DK / 64][32][64]
   bf16* qs = reinterpret_cast<bf16*>(base + STAGES * Cfg::STAGE_BYTES);
   float* sx = reinterpret_cast<float*>(qs + 16 * DK);
   bf16* ps = reinterpret_cast<bf16*>(sx + 2 * 16 * kMlaSx);
   __shared__ uint64_t full_bar[STAGES], empty_bar[STAGES];
-  __shared__ float s_ml[16][2], s_fac[16][8], s_corr[16];
+  __shared__ float s_ml[16][2], s_fac[16][8], s_corr[16], s_top[16][2];
+  __shared__ int s_last;
   static_assert(16 * PITCH * 4 <= STAGES * Cfg::STAGE_BYTES, "the merge buffer lies over the ring");
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   if (tid == 0) {
@@ -115,7 +120,8 @@ __global__ void __launch_bounds__(384, 1) mla_attn_kernel(const __grid_constant_
   const int nq = min(16, p.hl - h0);
   const int key_lo = max(0, n_keys - p.window);                        // and not before the window
   const int t_first = key_lo / MKT, t_all = (n_keys + MKT - 1) / MKT;
-  const int per = (t_all - t_first + p.nsplit - 1) / p.nsplit;
+  const int parts = p.nsplit * p.groups;
+  const int per = (t_all - t_first + parts - 1) / parts;
   const int t_begin = t_first + split * per, t_end = min(t_all, t_begin + per);
   const int nloc = max(0, t_end - t_begin);
 
@@ -126,19 +132,19 @@ __global__ void __launch_bounds__(384, 1) mla_attn_kernel(const __grid_constant_
     if (warp == 8 && lane == 0) {
       const int* bt = p.block_table + (size_t)b * p.bt_stride;
       auto issue = [&](int n) {
-        const int s = n % STAGES, key = (t_begin + n) * MKT;
+        const int s = n % STAGES, key = t_begin * MKT + n * (MKT / 2);
         int blk = bt[key / p.bs];
         if (blk < 0 || blk >= p.num_blocks) { if (p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); blk = 0; }
         mbar_expect_tx(&full_bar[s], Cfg::STAGE_BYTES);
         for (int c = 0; c < DK / 64; ++c)
-          tma_load_2d(reinterpret_cast<uint8_t*>(ring) + s * Cfg::STAGE_BYTES + c * (MKT * 128), &tmC, &full_bar[s], c * 64,
+          tma_load_2d(reinterpret_cast<uint8_t*>(ring) + s * Cfg::STAGE_BYTES + c * (MKT * 64), &tmC, &full_bar[s], c * 64,
                       blk * p.bs + key % p.bs, kEvictNormal);
       };
-      // tiles without a row of this call
-      const int pre = min(min(STAGES, nloc), max(0, past / MKT - t_begin));
+      // half tiles without a row of this call
+      const int halves = 2 * nloc, pre = min(min(STAGES, halves), max(0, past / (MKT / 2) - 2 * t_begin));
       for (int n = 0; n < pre; ++n) issue(n);
       grid_dep_wait();
-      for (int n = pre; n < nloc; ++n) {
+      for (int n = pre; n < halves; ++n) {
         if (!mbar_wait(&empty_bar[n % STAGES], ((n / STAGES) & 1) ^ 1, p.status, XFT_ERR_WAIT_EMPTY)) break;
         issue(n);
       }
@@ -174,9 +180,12 @@ __global__ void __launch_bounds__(384, 1) mla_attn_kernel(const __grid_constant_
     for (int ks = 0; ks < KS; ++ks)
       mla_ldsm(qa[ks], mla_ptr<16>(qs, (lane & 7) + ((lane >> 3) & 1) * 8, (dh * KS + ks) * 2 + (lane >> 4)));
     for (int n = 0; n < nloc; ++n) {
-      const int st = n % STAGES;
-      const bool ok = mbar_wait(&full_bar[st], (n / STAGES) & 1, p.status, XFT_ERR_WAIT_FULL);
-      bf16* kt = ring + (size_t)st * (Cfg::STAGE_BYTES / 2);
+      const int sa = (2 * n) % STAGES, sb = (2 * n + 1) % STAGES;
+      bf16* ka = ring + (size_t)sa * (Cfg::STAGE_BYTES / 2);
+      bf16* kb = ring + (size_t)sb * (Cfg::STAGE_BYTES / 2);
+      bool ok = mbar_wait(&full_bar[sa], ((2 * n) / STAGES) & 1, p.status, XFT_ERR_WAIT_FULL);
+      ok = mbar_wait(&full_bar[sb], ((2 * n + 1) / STAGES) & 1, p.status, XFT_ERR_WAIT_FULL) && ok;
+      bf16* kq = kg < 2 ? ka : kb;                                     // the half with this warp's keys
       {
         float s[4][4];                                                 // two 8-key tiles, even and odd steps
 #pragma unroll
@@ -184,7 +193,7 @@ __global__ void __launch_bounds__(384, 1) mla_attn_kernel(const __grid_constant_
 #pragma unroll
         for (int ks = 0; ks < KS; ++ks) {
           uint32_t bb[4];
-          mla_ldsm(bb, mla_ptr<MKT>(kt, kg * 16 + (lane & 7) + ((lane >> 4) & 1) * 8, (dh * KS + ks) * 2 + ((lane >> 3) & 1)));
+          mla_ldsm(bb, mla_ptr<MKT / 2>(kq, (kg & 1) * 16 + (lane & 7) + ((lane >> 4) & 1) * 8, (dh * KS + ks) * 2 + ((lane >> 3) & 1)));
           mla_mma(s[(ks & 1) * 2], qa[ks], bb[0], bb[1]);
           mla_mma(s[(ks & 1) * 2 + 1], qa[ks], bb[2], bb[3]);
         }
@@ -230,14 +239,14 @@ __global__ void __launch_bounds__(384, 1) mla_attn_kernel(const __grid_constant_
 #pragma unroll
           for (int j = 0; j < NT; j += 2) {
             uint32_t bb[4];
-            mla_ldsm_t(bb, mla_ptr<MKT>(kt, ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, warp * NT + j + (lane >> 4)));
+            mla_ldsm_t(bb, mla_ptr<MKT / 2>(ks < 2 ? ka : kb, (ks & 1) * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, warp * NT + j + (lane >> 4)));
             mla_mma(o[j], a, bb[0], bb[1]);
             mla_mma(o[j + 1], a, bb[2], bb[3]);
           }
         }
       }
       __syncwarp();
-      if (lane == 0) mbar_arrive(&empty_bar[st]);
+      if (lane == 0) { mbar_arrive(&empty_bar[sa]); mbar_arrive(&empty_bar[sb]); }
     }
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
@@ -276,10 +285,13 @@ __global__ void __launch_bounds__(384, 1) mla_attn_kernel(const __grid_constant_
       if (s < ns) { mm[s] = mm[s] == -INFINITY ? 0.f : __expf(mm[s] - top); sum += mm[s] * ll[s]; }
 #pragma unroll
     for (int s = 0; s < 8; ++s)
-      if (s < ns) s_fac[tid][s] = sum > 0.f ? mm[s] / sum : 0.f;
+      if (s < ns) s_fac[tid][s] = p.groups > 1 ? mm[s] : sum > 0.f ? mm[s] / sum : 0.f;
+    if (p.groups > 1) { s_top[tid][0] = top; s_top[tid][1] = sum; }
   }
   __syncthreads();
-  const int cols = LAT / ns, c0 = split * cols;
+  const int rank = split % ns, group = split / ns;
+  const int cols = LAT / ns, c0 = rank * cols;
+  float* po = p.groups > 1 ? p.part_o + ((size_t)blockIdx.x * p.groups + group) * 16 * LAT : nullptr;
   for (int i = tid; i < nq * (cols / 2); i += 384) {
     const int r = i / (cols / 2), d = c0 + 2 * (i % (cols / 2));
     const uint32_t a = smem_u32(mo + r * PITCH + d);
@@ -293,7 +305,38 @@ __global__ void __launch_bounds__(384, 1) mla_attn_kernel(const __grid_constant_
         y += f * (ns > 1 ? ld_dsmem(ra + 4) : mo[r * PITCH + d + 1]);
       }
     }
-    *reinterpret_cast<uint32_t*>(p.out + (h0 + r) * p.o_sh + (long long)t * p.o_st + d) = mla_pack(x, y);
+    if (po) *reinterpret_cast<float2*>(po + r * LAT + d) = make_float2(x, y);
+    else *reinterpret_cast<uint32_t*>(p.out + (h0 + r) * p.o_sh + (long long)t * p.o_st + d) = mla_pack(x, y);
+  }
+  if (po) {
+    // this rank's columns of every group: the last CTA to arrive adds them up
+    auto ml_of = [&](int g) { return p.part_ml + (((size_t)blockIdx.x * p.groups + g) * ns + rank) * 32; };
+    if (tid < 32) ml_of(group)[tid] = s_top[tid >> 1][tid & 1];
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) {
+      int* c = p.counters + (size_t)blockIdx.x * ns + rank;
+      s_last = atomicAdd(c, 1) == p.groups - 1;
+      if (s_last) *c = 0;
+    }
+    __syncthreads();
+    if (s_last) {
+      __threadfence();
+      for (int i = tid; i < nq * (cols / 2); i += 384) {
+        const int r = i / (cols / 2), d = c0 + 2 * (i % (cols / 2));
+        float top = -INFINITY, sum = 0.f, x = 0.f, y = 0.f;
+        for (int g = 0; g < p.groups; ++g) top = fmaxf(top, __ldcg(ml_of(g) + 2 * r));
+        for (int g = 0; g < p.groups; ++g) {
+          const float mg = __ldcg(ml_of(g) + 2 * r), f = mg == -INFINITY ? 0.f : __expf(mg - top);
+          const float2 v = __ldcg(reinterpret_cast<const float2*>(p.part_o + (((size_t)blockIdx.x * p.groups + g) * 16 + r) * LAT + d));
+          sum += f * __ldcg(ml_of(g) + 2 * r + 1);
+          x += f * v.x;
+          y += f * v.y;
+        }
+        const float inv = sum > 0.f ? 1.f / sum : 0.f;
+        *reinterpret_cast<uint32_t*>(p.out + (h0 + r) * p.o_sh + (long long)t * p.o_st + d) = mla_pack(x * inv, y * inv);
+      }
+    }
   }
   if (ns > 1) { cluster_arrive(); cluster_wait(); }                    // a peer may still read this CTA's part
 }
@@ -311,9 +354,9 @@ static int launch_mla(const MlaParams& p, const void* cache, cudaStream_t st) {
     attr = true;
   }
   CUtensorMap tm;
-  if (make_tensor_map(&tm, cache, (uint64_t)p.num_blocks * p.bs, Cfg::DK, Cfg::DK, MKT, 2)) return -4;
+  if (make_tensor_map(&tm, cache, (uint64_t)p.num_blocks * p.bs, Cfg::DK, Cfg::DK, MKT / 2, 2)) return -4;
   cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3(p.T * ((p.hl + 15) / 16), p.nsplit);
+  cfg.gridDim = dim3(p.T * ((p.hl + 15) / 16), p.nsplit * p.groups);
   cfg.blockDim = dim3(384);
   cfg.dynamicSmemBytes = Cfg::SMEM;
   cfg.stream = st;
@@ -329,18 +372,22 @@ static int launch_mla(const MlaParams& p, const void* cache, cudaStream_t st) {
 }
 
 // Sizes of the latent (64, 128, 256 or 512, with 64 rotated key dimensions next to it) and a sliding window: position i
-// sees the keys j <= i with i - j < window (0: all).  nsplit: CTAs per (token, 16 heads), rounded down to 1, 2, 4 or 8.
+// sees the keys j <= i with i - j < window (0: all).  nsplit: CTAs per (token, 16 heads) and
+// cluster, rounded down to 1, 2, 4 or 8; groups: clusters per (token, 16 heads).  With groups > 1 and u = T * ceil(hl / 16):
+// part_o of u * groups * 16 * lat floats, part_ml of u * groups * nsplit * 32, counters of u * nsplit zeros (left as zeros).
 extern "C" int xft_mla_attention_ext(const void* q_abs, long long qa_sh, long long qa_st, const void* q_rope, long long qr_sh,
                                      long long qr_st, void* out, long long o_sh, long long o_st, const void* cache,
                                      const int* block_table, int bt_stride, const int* cu_q, const int* kv_lens, int B, int T,
                                      int hl, int lat, int bs, int num_blocks, float scale, int window, int nsplit,
-                                     int* status, cudaStream_t st) {
+                                     int groups, float* part_o, float* part_ml, int* counters, int* status,
+                                     cudaStream_t st) {
   if (T <= 0 || B <= 0) return 0;
   if (bs <= 0 || bs % MKT) return -2;
   if (window < 0 || hl <= 0) return -1;
   MlaParams p{(const bf16*)q_abs, qa_sh, qa_st, (const bf16*)q_rope, qr_sh, qr_st, (bf16*)out, o_sh, o_st, block_table,
               bt_stride, cu_q, kv_lens, B, T, hl, bs, num_blocks, scale, window > 0 ? min(window, 1 << 30) : 1 << 30,
-              nsplit >= 8 ? 8 : nsplit >= 4 ? 4 : nsplit >= 2 ? 2 : 1, status};
+              nsplit >= 8 ? 8 : nsplit >= 4 ? 4 : nsplit >= 2 ? 2 : 1, groups < 1 ? 1 : groups, part_o, part_ml, counters, status};
+  if (p.groups > 1 && (!part_o || !part_ml || !counters)) return -3;
   switch (lat) {
     case 64: return launch_mla<64>(p, cache, st);
     case 128: return launch_mla<128>(p, cache, st);
@@ -357,5 +404,5 @@ extern "C" int xft_mla_attention(const void* q_abs, long long qa_sh, long long q
                                  int hl, int bs, int num_blocks, float scale, int nsplit, float* /*part_o*/,
                                  float* /*part_ml*/, int* /*counters*/, int* status, cudaStream_t st) {
   return xft_mla_attention_ext(q_abs, qa_sh, qa_st, q_rope, qr_sh, qr_st, out, o_sh, o_st, cache, block_table, bt_stride, cu_q,
-                               kv_lens, B, T, hl, 512, bs, num_blocks, scale, 0, nsplit, status, st);
+                               kv_lens, B, T, hl, 512, bs, num_blocks, scale, 0, nsplit, 1, nullptr, nullptr, nullptr, status, st);
 }

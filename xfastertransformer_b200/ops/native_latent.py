@@ -158,16 +158,27 @@ def flat_attention(x, d, kv, flat, sp, h0, n, scale, window, out):
 
 
 # clusters of n CTAs (one CTA per SM) that B200 holds at a time: its GPCs have 16 to 20 SMs
-CLUSTERS = {2: 74, 4: 33, 8: 15}
+CLUSTERS = {1: 148, 2: 74, 4: 33, 8: 15}
 
 
-def mla_splits(units: int, keys: int) -> int:
-    """CTAs per (token, 16 heads) of the absorbed kernel, which form a cluster: as many as run in one wave, with at least two
-    64-key tiles each."""
-    tiles, n = (keys + 63) // 64, 1
+def mla_splits(units: int, keys: int) -> tuple:
+    """(CTAs per cluster, clusters) that share the keys of a (token, 16 heads) in the absorbed kernel: as many as run in one
+    wave, with at least two 64-key tiles each (eight, where several clusters share them: their merge costs more)."""
+    tiles, n, g = (keys + 63) // 64, 1, 1
     while n < 8 and units <= CLUSTERS[2 * n] and tiles >= 4 * n:
         n *= 2
-    return n
+    while g < 8 and 2 * g * units <= CLUSTERS[n] and tiles >= 16 * n * g:
+        g *= 2
+    return n, g
+
+
+def mla_scratch(ws, units: int, n: int, g: int, rank: int) -> tuple:
+    """(partial outputs, partial maxima and sums, counters) of a launch with `g` clusters per unit."""
+    if g == 1:
+        return None, None, None
+    if units * n > ws.attn_counters.numel():
+        raise N.KernelError("latent attention: more partial results than counters")
+    return (*ws.attn_partials(units * g * 16 * rank, units * g * n * 32), ws.attn_counters)
 
 
 def _absorbed(x, d, cache, block_table, cu_dev, kv_dev, B, max_kv, weights, scale, window, out):
@@ -193,13 +204,15 @@ def _absorbed(x, d, cache, block_table, cu_dev, kv_dev, B, max_kv, weights, scal
     ws = N.Workspace.get(x.device)
     qa, ol = new(T, H * d.rank), new(T, H * d.rank)
     _heads(x, ldx, d.q_width, hd, wk, H, d.rank, d.dim, qa, H * d.rank, d.rank)
-    nsplit = mla_splits(T * ((H + 15) // 16), min(max_kv, window) if window > 0 else max_kv)
+    units = T * ((H + 15) // 16)
+    nsplit, groups = mla_splits(units, min(max_kv, window) if window > 0 else max_kv)
+    po, pm, cnt = mla_scratch(ws, units, nsplit, groups, d.rank)
     nb, _, bs, _ = cache.shape
     LL = C.c_longlong
     qr = x[:, d.dim:]
     N._check(_fn("xft_mla_attention_ext")(
         N._p(qa), LL(d.rank), LL(H * d.rank), N._p(qr), LL(hd), LL(ldx), N._p(ol), LL(d.rank), LL(H * d.rank), N._p(cache),
         N._p(block_table), block_table.stride(0), N._p(cu_dev), N._p(kv_dev), B, T, H, d.rank, bs, nb, C.c_float(scale), window,
-        nsplit, N._p(ws.status), N._stream()), "mla_attention")
+        nsplit, groups, N._p(po), N._p(pm), N._p(cnt), N._p(ws.status), N._stream()), "mla_attention")
     ws.launches += 1
     return _heads(ol, H * d.rank, H * d.rank, d.rank, wv, H, d.vdim, d.rank, out, H * d.vdim, d.vdim, gate, ldx)

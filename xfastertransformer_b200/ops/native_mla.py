@@ -17,7 +17,7 @@ def _lib():
     global _ready
     lib = N.lib()
     if not _ready:
-        lib.xft_mla_attention.restype = C.c_int
+        lib.xft_mla_attention_ext.restype = C.c_int
         lib.xft_gemm_bf16_grouped.restype = C.c_int
         _ready = True
     return lib
@@ -78,14 +78,15 @@ def mla_attention(q_nope, q_rope, latent_cache, block_table, cu_q, kv_lens, w_uk
     o_lat = torch.empty(Hl * T, L, dtype=torch.bfloat16, device=dev)
     nb, _, bs, W = latent_cache.shape
     chunks = (Hl + 15) // 16
-    from .native_latent import mla_splits
-    nsplit = mla_splits(T * chunks, max_kv)
+    from .native_latent import mla_scratch, mla_splits
+    nsplit, groups = mla_splits(T * chunks, max_kv)
+    po, pm, cnt = mla_scratch(ws, T * chunks, nsplit, groups, L)
     q_rope = q_rope.contiguous()
-    rc = _lib().xft_mla_attention(N._p(q_abs), C.c_longlong(T * L), C.c_longlong(L), N._p(q_rope), C.c_longlong(rope),
-                                  C.c_longlong(Hl * rope), N._p(o_lat), C.c_longlong(T * L), C.c_longlong(L),
-                                  N._p(latent_cache), N._p(block_table), block_table.stride(0), N._p(cu_dev),
-                                  N._p(kv_dev), B, T, Hl, bs, nb, C.c_float(scale), nsplit, N._p(None), N._p(None),
-                                  N._p(None), N._p(ws.status), N._stream())
+    LL = C.c_longlong
+    rc = _lib().xft_mla_attention_ext(N._p(q_abs), LL(T * L), LL(L), N._p(q_rope), LL(rope), LL(Hl * rope), N._p(o_lat), LL(T * L),
+                                      LL(L), N._p(latent_cache), N._p(block_table), block_table.stride(0), N._p(cu_dev),
+                                      N._p(kv_dev), B, T, Hl, L, bs, nb, C.c_float(scale), 0, nsplit, groups, N._p(po), N._p(pm),
+                                      N._p(cnt), N._p(ws.status), N._stream())
     N._check(rc, "mla_attention")
     ws.launches += 1
     o = _per_head_gemm(o_lat, wv, Hl, T, vd, L)                      # [Hl*T, vd]
