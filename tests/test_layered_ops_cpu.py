@@ -261,6 +261,21 @@ def test_other_weight_and_cache_types(tmp_path, dtype, kv, tol):
     assert m.generate(torch.tensor([toks]), max_length=50).shape == (1, 50)
 
 
+def test_partial_library_has_what_layered_models_call():
+    """bin/trace_run may build a part of the kernels only: its sources define every entry point the ops look up by name."""
+    import importlib.util
+    import re
+    spec = importlib.util.spec_from_file_location("xft_build", os.path.join(ROOT, "csrc", "build.py"))
+    b = importlib.util.module_from_spec(spec)
+    spec.loader.exec_module(b)
+    text = "".join(open(os.path.join(ROOT, "csrc", "kernels", f)).read() for f in b.LAYERED)
+    defined = set(re.findall(r'extern "C" \w+ (xft_\w+)\(', text))
+    ops_dir = os.path.join(ROOT, "xfastertransformer_b200", "ops")
+    src = {f: open(os.path.join(ops_dir, f)).read() for f in ("native.py", "native_latent.py", "native_moe.py")}
+    wanted = {n for t in src.values() for n in re.findall(r'(?:lib\(\)\.|L\.|lib\.|")(xft_\w+)', t)}
+    assert len(wanted) > 30 and wanted - defined <= {"xft_qgemm_grouped"}, wanted - defined
+
+
 def test_command_line(tmp_path):
     """bin/trace_run as a program: JSON lines in, files of fp32 logits and a line per step out."""
     cfg = O.config([O.attention_layer(), O.attention_layer(kv_from=0, size=7)], vocab=61)

@@ -11,14 +11,16 @@ from . import reference as R
 
 _KIND = {"mixtral": 0, "softmax_topk": 1, "deepseek": 2}
 _ready = False
+# what the bf16 and fp32 experts call (the fp8 product is looked up where it is used: not every library has it)
+ENTRY_POINTS = ("xft_moe_route", "xft_moe_plan", "xft_moe_gather", "xft_moe_combine", "xft_moe_combine_bf16",
+                "xft_gemm_bf16_grouped", "xft_gemm_bf16_grouped_tm", "xft_gemm_f32_grouped")
 
 
 def _lib():
     global _ready
     lib = N.lib()
     if not _ready:
-        for fn in ("xft_moe_route", "xft_moe_plan", "xft_moe_gather", "xft_moe_combine", "xft_gemm_bf16_grouped",
-                   "xft_qgemm_grouped"):
+        for fn in ENTRY_POINTS:
             getattr(lib, fn).restype = C.c_int
         _ready = True
     return lib
@@ -115,7 +117,6 @@ def _experts_f32(x, idx32, w, pk, act, expert_offset, gated, add):
                               N._p(tiles), N._p(meta), tiles_n, n, N._stream()), "moe_plan")
     h1, ys, out = f32(n, I), f32(n, H), f32(T, H)
     fn = lib.xft_gemm_f32_grouped
-    fn.restype = C.c_int
     N._check(fn(N._p(x), x.stride(0) if T > 1 else max(x.stride(0), H), N._p(pk["gu"]), H, N._p(h1), I, I, H, I, N._p(tiles),
                 N._p(meta), tiles_n, N._p(src), N._p(None), N._ACT[act], N._stream()), "grouped fp32 up")
     N._check(fn(N._p(h1), I, N._p(pk["dn"]), I, N._p(ys), H, H, I, H, N._p(tiles), N._p(meta), tiles_n, N._p(None), N._p(row_w), 0,
@@ -178,14 +179,12 @@ def moe_experts(x, idx, w, experts, act="silu", expert_offset=0, packed=None, ex
         # prompt sizes: the token-major persistent kernel; rows stay bf16 until the weighted sum
         y16 = torch.empty(max_rows, H, dtype=torch.bfloat16, device=dev)
         fn = lib.xft_gemm_bf16_grouped_tm
-        fn.restype = C.c_int
         N._check(fn(N._p(xs), H, max_rows, N._p(pk["gu"]), E * up, H, N._p(h1), I, I, H, int(gated), I, up, N._p(tiles), N._p(meta),
                     max_tiles, N._ACT[act], N._p(ws.status), N._stream()), "grouped gate_up")
         N._check(fn(N._p(h1), I, max_rows, N._p(pk["dn"]), E * H, I, N._p(y16), H, H, I, 0, 0, H, N._p(tiles), N._p(meta), max_tiles,
                     0, N._p(ws.status), N._stream()), "grouped down")
         out = torch.empty(T, H, dtype=torch.float32, device=dev)
         fn = lib.xft_moe_combine_bf16
-        fn.restype = C.c_int
         N._check(fn(N._p(y16), N._p(pos), N._p(w.contiguous()), k, N._p(add32), N._p(add16), H, N._p(None), N._p(out), T, H,
                     N._stream()), "moe_combine")
         ws.launches += 5
