@@ -38,3 +38,5 @@ if model.rank == 0:
     torch.save(res, out)
 m._closed = True
 dist.barrier()
+if not torch.cuda.is_available():                   # gloo: no thread of it outlives the interpreter
+    dist.destroy_process_group()

@@ -28,3 +28,5 @@ if model.rank == 0:
                 "microbatches": getattr(m, "pp_microbatches", 0)}, out)
 m._closed = True
 dist.barrier()
+if not torch.cuda.is_available():                   # gloo: no thread of it outlives the interpreter
+    dist.destroy_process_group()

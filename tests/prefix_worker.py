@@ -34,3 +34,5 @@ if model.rank == 0:
     torch.save({"logits": logits, "tokens": tokens, "stats": stats}, out)
 model.model._closed = True
 dist.barrier()
+if not torch.cuda.is_available():                   # gloo: no thread of it outlives the interpreter
+    dist.destroy_process_group()

@@ -29,3 +29,5 @@ if model.rank == 0:
                 "pairs": m.prefill_decoder.pairs_run}, out)
 m._closed = True
 dist.barrier()
+if not torch.cuda.is_available():                   # gloo: no thread of it outlives the interpreter
+    dist.destroy_process_group()
