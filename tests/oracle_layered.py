@@ -1,4 +1,4 @@
-"""A plain, slow implementation of the layered designs (Kafipel, Vepivik), one function per mechanism, for the tests to
+"""A plain, slow implementation of the layered designs (Kafipel, Vepivik, Botusun), one function per mechanism, for the tests to
 compare against.
 
 It works on one whole sequence at a time, without a cache, in the precision of the tensors it is given (tests use fp64
@@ -25,6 +25,17 @@ def rms_norm(x, w, eps):
     return x / torch.sqrt((x * x).sum(-1, keepdim=True) / x.shape[-1] + eps) * w
 
 
+def banded(f, sc):
+    """A frequency scaled by wavelength: short waves keep it, long waves are slowed by the factor, with a ramp between."""
+    wave = 2 * math.pi / f
+    if wave < sc["original"] / sc["high"]:
+        return f
+    if wave > sc["original"] / sc["low"]:
+        return f / sc["factor"]
+    s = (sc["original"] / wave - sc["low"]) / (sc["high"] - sc["low"])
+    return (1 - s) * f / sc["factor"] + s * f
+
+
 def rotary_frequencies(rot):
     """(frequency of each pair, factor on cosine and sine)."""
     n, base = rot["dims"], rot["base"]
@@ -32,6 +43,8 @@ def rotary_frequencies(rot):
     sc = rot.get("scaling")
     if not sc:
         return f, 1.0
+    if "low" in sc:
+        return [banded(fi, sc) for fi in f], 1.0
 
     def dim_of(turns):
         return n * math.log(sc["original"] / (2 * math.pi * turns)) / (2 * math.log(base))
@@ -196,6 +209,115 @@ def experts(h, f, W, prefix):
     return out
 
 
+def grouped_router(z, correction, top, scale, groups=None):
+    """Chosen experts [T, top] (best first) and their weights: sigmoid scores choose with a correction added and weigh
+    without it; with `groups` {count, keep} only experts of the groups with the best sum of two choice scores."""
+    s = 1 / (1 + torch.exp(-z))
+    choice = s + correction
+    T, E = z.shape
+    if groups:
+        n = E // groups["count"]
+        for t in range(T):
+            score = [sum(sorted(choice[t, g * n:(g + 1) * n].tolist())[-2:]) for g in range(groups["count"])]
+            best = sorted(range(groups["count"]), key=lambda g: -score[g])[:groups["keep"]]
+            for e in range(E):
+                if e // n not in best:
+                    choice[t, e] = -math.inf
+    idx = torch.argsort(choice, -1, descending=True)[:, :top]
+    return idx, torch.gather(s, 1, idx) * scale
+
+
+def gated_expert(h, gate, up, down):
+    g = h @ gate.T
+    return (g / (1 + torch.exp(-g)) * (h @ up.T)) @ down.T
+
+
+def grouped_experts(h, f, W, prefix):
+    P, r = prefix + ".mlp.", f["router"]
+    idx, w = grouped_router(h @ W[P + "router"].T, W[P + "correction"], r["top"], r["scale"], r.get("groups"))
+    out = torch.zeros(h.shape[0], W["embed"].shape[1], dtype=h.dtype)
+    for t in range(h.shape[0]):
+        for e, we in zip(idx[t].tolist(), w[t]):
+            out[t] += we * gated_expert(h[t:t + 1], *(W[P + f"e{e}.{n}"] for n in ("gate", "up", "down")))[0]
+    return out
+
+
+def short_conv(u, w):
+    """u [T, C], w [C, taps]: every channel's weighted sum of its last `taps` values, the newest one last."""
+    T, taps = u.shape[0], w.shape[1]
+    y = torch.zeros_like(u)
+    for j in range(taps):
+        back = taps - 1 - j
+        if back < T:
+            y[back:] += w[:, j] * u[:T - back]
+    return y
+
+
+def shared_kv_mixer(h, m, W, prefix, positions, eps):
+    """Attention whose values are its keys: projections with biases, short convolutions, then a norm per head and rotation
+    on queries and keys; the values are the convolved keys.  A sink of score 0 joins the softmax."""
+    T, H, G, d = h.shape[0], m["heads"], m["kv_heads"], m["dim"]
+    P = prefix + ".mix."
+    q, k = h @ W[P + "q"].T + W[P + "q.b"], h @ W[P + "k"].T + W[P + "k.b"]
+    if m.get("conv"):
+        q, k = short_conv(q, W[P + "q.conv"]), short_conv(k, W[P + "k.conv"])
+    q, k = q.view(T, H, d), k.view(T, G, d)
+    v = k
+    q = rotate(rms_norm(q, W[P + "q.norm"], eps), positions, m.get("rot"))
+    k = rotate(rms_norm(k, W[P + "k.norm"], eps), positions, m.get("rot"))
+    a = attention(q, k, v, m["scale"], None, m.get("mask"), torch.zeros(H, dtype=h.dtype))
+    return a.reshape(T, -1) @ W[P + "o"].T
+
+
+def log_decay(z, tau):
+    """log(sigmoid(z)^(1/tau))"""
+    return torch.nn.functional.logsigmoid(z) / tau
+
+
+def gated_linear(q, k, v, decay):
+    """q, k, decay [T, H, d], v [T, H, dv] -> [T, H, dv]: per head S <- diag(decay) S + k v^T, o = S^T q."""
+    T, H, d = q.shape
+    S = torch.zeros(H, d, v.shape[2], dtype=q.dtype)
+    out = []
+    for t in range(T):
+        S = decay[t][:, :, None] * S + k[t][:, :, None] * v[t][:, None, :]
+        out.append((S * q[t][:, :, None]).sum(1))
+    return torch.stack(out)
+
+
+def linear_mixer(h, m, W, prefix, eps):
+    T, H, d, dv = h.shape[0], m["heads"], m["dim"], m["vdim"]
+    P = prefix + ".mix."
+    q = (h @ W[P + "q"].T * d ** -0.5).view(T, H, d)
+    k, v = (h @ W[P + "k"].T).view(T, H, d), (h @ W[P + "v"].T).view(T, H, dv)
+    z = (h @ W[P + "a1"].T) @ W[P + "a2"].T + W[P + "a2.b"]
+    o = gated_linear(q, k, v, torch.exp(log_decay(z, m["tau"])).view(T, H, d))
+    o = rms_norm(o, W[P + "norm"], eps).reshape(T, -1)
+    g = h @ W[P + "g"].T
+    return (o * (g / (1 + torch.exp(-g)))) @ W[P + "o"].T
+
+
+def gelu_tanh(z):
+    return 0.5 * z * (1 + torch.tanh(math.sqrt(2 / math.pi) * (z + 0.044715 * z ** 3)))
+
+
+def token_side(x, tokens, W, i, dim, eps):
+    """What the token's own side embedding adds after layer i."""
+    e = W["side.embed"][torch.tensor(tokens), i * dim:(i + 1) * dim]
+    g = gelu_tanh(x @ W[f"l{i}.side.gate"].T) * e
+    return rms_norm(g @ W[f"l{i}.side.proj"].T, W[f"l{i}.side.norm"], eps)
+
+
+def layer_runs(cfg):
+    """(layer, pass, first layer of a pass) in the order they run: the looped layers several times in a row."""
+    n, loop = len(cfg["layers"]), cfg.get("loop")
+    if not loop:
+        return [(i, 0, False) for i in range(n)]
+    a, b = loop["start"], loop["stop"]
+    return [(i, 0, False) for i in range(a)] + [(i, t, i == a) for t in range(loop["times"]) for i in range(a, b)] + \
+        [(i, 0, False) for i in range(b, n)]
+
+
 def feed_forward(h, W, prefix):
     g, u = h @ W[prefix + ".mlp.gate"].T, h @ W[prefix + ".mlp.up"].T
     return (g / (1 + torch.exp(-g)) * u) @ W[prefix + ".mlp.down"].T
@@ -204,7 +326,7 @@ def feed_forward(h, W, prefix):
 def forward(cfg, W, tokens, layers_out=None, dtype=torch.float64):
     """Logits [T, vocab] of one sequence; `layers_out` (a list) collects the residual stream after every layer."""
     W = {n: (t.to(dtype) if t.is_floating_point() else t) for n, t in W.items()}
-    run = {"Kafipel": _kafipel, "Vepivik": _vepivik}[cfg["architecture"]]
+    run = {"Kafipel": _kafipel, "Vepivik": _vepivik, "Botusun": _botusun}[cfg["architecture"]]
     return run(cfg, W, tokens, [] if layers_out is None else layers_out)
 
 
@@ -238,6 +360,29 @@ def _vepivik(cfg, W, tokens, layers_out):
             x = x + mixer(h, layer["mixer"], W, p, positions, kept)
         if layer.get("mlp"):
             x = x + experts(rms_norm(x, W[p + ".norm2"], eps), layer["mlp"], W, p)
+        layers_out.append(x.clone())
+    return rms_norm(x, W["final.norm"], eps) @ W["embed"].T
+
+
+def _botusun(cfg, W, tokens, layers_out):
+    eps, m = cfg["norm"]["eps"], cfg["residual_mult"]
+    positions = list(range(len(tokens)))
+    x = W["embed"][torch.tensor(tokens)] * cfg["embedding"]["scale"]
+    for i, t, begins in layer_runs(cfg):
+        p, layer = f"l{i}", cfg["layers"][i]
+        if begins:
+            x = x + W["loop.step"][t]
+        h = rms_norm(x, W[p + ".norm1"], eps)
+        if layer["type"] == "gla":
+            x = x + m * linear_mixer(h, layer["mixer"], W, p, eps)
+        else:
+            x = x + m * shared_kv_mixer(h, layer["mixer"], W, p, positions, eps)
+        f = layer.get("mlp")
+        if f:
+            h = rms_norm(x, W[p + ".norm2"], eps)
+            x = x + m * (feed_forward(h, W, p) if f["kind"] == "dense" else grouped_experts(h, f, W, p))
+        if cfg.get("token_side"):
+            x = x + m * token_side(x, tokens, W, i, cfg["token_side"]["dim"], eps)
         layers_out.append(x.clone())
     return rms_norm(x, W["final.norm"], eps) @ W["embed"].T
 

@@ -233,14 +233,14 @@ def test_chatglm_2d_positions_honour_both_mask_tokens(mask_tok):
 
 
 def test_runner_staging_buffer_layout_with_padding_rows():
-    """The decode runner's per-step staging buffer: [ids | positions | slots | kv lengths | cu_q | block table], real rows
-    first, padding rows of the bucket pointing at the runner's scratch block with a context of one token."""
+    """The decode runner's per-step staging buffer: [ids | positions | slots | kv lengths | state slots | cu_q | block table],
+    real rows first, padding rows of the bucket pointing at the runner's scratch block and state with a context of one token."""
     from types import SimpleNamespace
     from xfastertransformer_b200.runtime.cuda_runner import CudaRunner, _Graph
-    cache = PagedKVCache(1, 1, 8, 8, "bf16", torch.device("cpu"), block_size=4)
+    cache = PagedKVCache(1, 1, 8, 8, "bf16", torch.device("cpu"), block_size=4, states=[((2, 3), torch.float32)])
     r = CudaRunner.__new__(CudaRunner)
     r.m = SimpleNamespace(cache=cache)
-    r._scratch_block = None
+    r._scratch_block = r._scratch_state = None
     sb = r._scratch()
     seqs = []
     for sid, past in ((10, 5), (11, 9), (12, 2)):
@@ -251,13 +251,15 @@ def test_runner_staging_buffer_layout_with_padding_rows():
     B, W = 4, 8
     g = _Graph()
     g.B, g.W = B, W
-    o_ids, o_pos, o_slot, o_kv, o_cu, o_bt, total = r._layout(B, W)
+    o_ids, o_pos, o_slot, o_kv, o_st, o_cu, o_bt, total = r._layout(B, W)
     g.host = torch.full((total,), -7, dtype=torch.int32)
     r._fill(g, seqs, slots)
     h = g.host
     assert h[o_ids:o_ids + B].tolist() == [110, 111, 112, 0]
     assert h[o_pos:o_pos + B].tolist() == [5, 9, 2, 0]
     assert h[o_kv:o_kv + B].tolist() == [6, 10, 3, 1]
+    states = [cache.state_slot[s.seq_id] for s in seqs]
+    assert h[o_st:o_st + B].tolist() == states + [r._scratch_state] and len({*states, r._scratch_state}) == 4
     assert h[o_slot:o_slot + B].tolist() == slots + [sb * cache.block]
     for i, s in enumerate(seqs):
         tab = cache.tables[s.seq_id]

@@ -18,17 +18,20 @@ from .runtime.engine import Model
 
 
 class AutoModel:
-    def __init__(self, path, dtype: str = "fp16", kv_cache_dtype: str = "fp16", max_cache_tokens: int = 0):
+    def __init__(self, path, dtype: str = "fp16", kv_cache_dtype: str = "fp16", max_cache_tokens: int = 0,
+                 max_sequences: int = 0):
         if dtype not in WEIGHT_DTYPES:
             raise Exception(f"{self.__class__.__name__} don't support {dtype}.")
         if kv_cache_dtype not in KV_DTYPES:
             raise Exception(f"{self.__class__.__name__} don't support KV cache data type: {kv_cache_dtype}.")
-        self.model = Model(path, dtype, kv_cache_dtype, max_cache_tokens=max_cache_tokens)
+        self.model = Model(path, dtype, kv_cache_dtype, max_cache_tokens=max_cache_tokens, max_sequences=max_sequences)
 
     @classmethod
-    def from_pretrained(cls, path, dtype: str = "fp16", kv_cache_dtype: str = "fp16", max_cache_tokens: int = 0):
-        """``max_cache_tokens`` > 0 (extension): the KV pools are made for that many tokens and never grow."""
-        return cls(path, dtype, kv_cache_dtype, max_cache_tokens)
+    def from_pretrained(cls, path, dtype: str = "fp16", kv_cache_dtype: str = "fp16", max_cache_tokens: int = 0,
+                        max_sequences: int = 0):
+        """``max_cache_tokens`` > 0 (extension): the KV pools are made for that many tokens and never grow;
+        ``max_sequences`` > 0: the same for recurrent states, one slot per sequence."""
+        return cls(path, dtype, kv_cache_dtype, max_cache_tokens, max_sequences)
 
     def __call__(self, inputs, **kwargs):
         """All-position logits [bs, seq, vocab] (torch binding ``forward``, auto_model.h:160-190)."""

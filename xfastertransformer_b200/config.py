@@ -38,7 +38,11 @@ MODEL_TYPES = (
 )
 
 # config.json "architecture" -> model type
-ARCHITECTURES = {"Kafipel": "kafipel", "Vepivik": "vepivik"}
+ARCHITECTURES = {"Kafipel": "kafipel", "Vepivik": "vepivik", "Botusun": "botusun"}
+
+# what a design fixes about its mixers and experts beside what its config.json says
+MIXER_TRAITS = {"botusun": {"attention": dict(values_from_keys=True, qk_bias=True, qk_norm=True, sink=0.0)}}
+MOE_TRAITS = {"botusun": dict(act="silu", gated=True, scoring="sigmoid", renorm=False, correction=True)}
 
 
 def split_hybrid_dtype(dtype: str) -> Tuple[str, str]:
@@ -81,7 +85,9 @@ class RopeConfig:
 @dataclass(frozen=True)
 class RotaryConfig:
     """Rotary positions of one layer: the first `dims` dimensions of each head (of the rotated part, in latent attention),
-    base, optional YaRN scaling; `style` "half" pairs dimension i with i + dims/2, "interleaved" 2i with 2i + 1."""
+    base, optional scaling; `style` "half" pairs dimension i with i + dims/2, "interleaved" 2i with 2i + 1.
+    `scaling` "yarn" uses `fast` and `slow`; "banded" keeps the frequencies of wavelengths below original / `high`, divides
+    those above original / `low` by the factor, with a ramp between them (the scheme of Llama 3.1)."""
     dims: int
     base: float
     factor: float = 0.0               # 0: no scaling
@@ -89,6 +95,9 @@ class RotaryConfig:
     fast: float = 32.0
     slow: float = 1.0
     style: str = "half"
+    scaling: str = "yarn"
+    low: float = 1.0
+    high: float = 4.0
 
 
 @dataclass(frozen=True)
@@ -99,7 +108,15 @@ class MixerConfig:
 
     `kind` "latent": keys and values come from one latent of `kv_rank` values per token, expanded per head to `dim` key and
     `vdim` value dimensions, plus `rot_dim` rotated key dimensions that all heads share (kv_heads is 1: one cache row per
-    token).  `gate`: the concatenated heads are multiplied with sigmoid(W_g h)."""
+    token).  `gate`: the concatenated heads are multiplied with sigmoid(W_g h).
+
+    `conv` > 0: queries and keys go through a causal convolution of that many taps, channel by channel, straight after
+    their projections (`qk_bias`: which have biases).  `values_from_keys`: the values are the keys as they leave it, before
+    norm and rotation.  `qk_norm`: RMS norm per head in front of the rotation.  `sink`: score of a softmax sink that all
+    heads share and that is no tensor.
+
+    `kind` "gla": gated linear attention, heads of `dim` x `vdim` states that decay per key channel by
+    sigmoid(z)^(1 / `tau`); no cache, one fp32 state per sequence."""
     heads: int
     kv_heads: int
     dim: int
@@ -114,6 +131,17 @@ class MixerConfig:
     kv_rank: int = 0
     rot_dim: int = 0
     gate: bool = False
+    conv: int = 0
+    values_from_keys: bool = False
+    qk_bias: bool = False
+    qk_norm: bool = False
+    sink: Optional[float] = None
+    tau: float = 1.0
+
+    @property
+    def has_kv(self) -> bool:
+        """Whether a layer with this mixer keeps keys and values (its own or another layer's)."""
+        return self.kind != "gla"
 
     def kv_shape(self) -> tuple:
         """What two layers must agree on for one to read the other's cache."""
@@ -124,13 +152,23 @@ class MixerConfig:
 
 @dataclass(frozen=True)
 class MoeConfig:
-    """Mixture of experts of one layer: softmax over `experts` router logits, the `top` best with their scores divided by
-    their sum, and (`shared` > 0) one more expert that every token uses.  An expert is down(act(up x))."""
+    """Mixture of experts of one layer: scores from `experts` router logits (`scoring`: softmax over them, or the sigmoid of
+    each), the `top` best, weighted with their scores (`renorm`: divided by their sum) times `scale`, and (`shared` > 0)
+    one more expert that every token uses.  `correction`: a tensor added to the scores for the choice alone.  `groups` > 1:
+    only experts of the `keep_groups` groups with the best sum of two choice scores can be chosen.  An expert is
+    down(act(up x)), or with `gated` down(act(gate x) * up x)."""
     experts: int
     top: int
     ff: int
     shared: int = 0
     act: str = "relu2"
+    gated: bool = False
+    scoring: str = "softmax"
+    renorm: bool = True
+    scale: float = 1.0
+    correction: bool = False
+    groups: int = 1
+    keep_groups: int = 1
 
 
 @dataclass(frozen=True)
@@ -139,6 +177,14 @@ class LayerConfig:
     ff: int = 0                       # width of a dense feed-forward; 0: none
     ff_kind: str = "dense"
     moe: Optional[MoeConfig] = None
+
+
+@dataclass(frozen=True)
+class LoopConfig:
+    """Layers start .. stop - 1 run `times` times in a row; every pass has a cache and states of its own."""
+    start: int
+    stop: int
+    times: int
 
 
 @dataclass
@@ -190,6 +236,9 @@ class ModelConfig:
     # layered designs (config.json): one entry per layer; the scalar sizes above then hold the first layer's
     layers: List[LayerConfig] = field(default_factory=list)
     embed_scale: float = 1.0
+    residual_mult: float = 1.0        # factor of every sublayer's output in the residual sum
+    loop: Optional[LoopConfig] = None
+    side_dim: int = 0                 # > 0: each layer also gets so many values of the token's own side embedding
     # raw key/value pairs (for family-specific look-ups, like DecoderContext::GetAttr)
     raw: Dict[str, str] = field(default_factory=dict)
 
@@ -197,6 +246,14 @@ class ModelConfig:
     @property
     def is_mla(self) -> bool:
         return self.qk_nope_head_dim > 0 and self.qk_rope_head_dim > 0
+
+    def runs(self) -> List[Tuple[int, int]]:
+        """(layer, pass) in the order they run; pass -1: outside the loop."""
+        n, loop = len(self.layers) or self.num_layer, self.loop
+        if loop is None:
+            return [(i, -1) for i in range(n)]
+        return [(i, -1) for i in range(loop.start)] + \
+            [(i, t) for t in range(loop.times) for i in range(loop.start, loop.stop)] + [(i, -1) for i in range(loop.stop, n)]
 
     @property
     def q_size(self) -> int:
@@ -242,7 +299,14 @@ class ModelConfig:
         arch = d.get("architecture")
         if arch not in ARCHITECTURES:
             raise ValueError(f"unsupported architecture {arch!r} in {where}; known: {sorted(ARCHITECTURES)}")
-        layers = [_layer_config(i, e) for i, e in enumerate(d["layers"])]
+        layers = [_layer_config(i, e, ARCHITECTURES[arch]) for i, e in enumerate(d["layers"])]
+        loop = None
+        if d.get("loop"):
+            loop = LoopConfig(*(int(d["loop"][k]) for k in ("start", "stop", "times")))
+            if not 0 <= loop.start < loop.stop <= len(layers) or loop.times < 1:
+                raise ValueError(f"loop {d['loop']} does not fit {len(layers)} layers")
+            if any(l.mixer.kv_from >= 0 for l in layers):
+                raise ValueError("layers that read another layer's keys do not combine with a loop")
         for i, l in enumerate(layers):
             j = l.mixer.kv_from
             if j >= 0:
@@ -256,7 +320,9 @@ class ModelConfig:
                    v_head_dim=m.vdim, hidden_size=int(d["width"]), inter_size=layers[0].ff, num_layer=len(layers),
                    vocab_size=int(d["vocab"]), layernorm_eps=float(d["norm"]["eps"]), start_id=-1, end_id=-1,
                    weight_data_type="bf16", layers=layers, raw=d,
-                   embed_scale=float((d.get("embedding") or {}).get("scale", 1.0)))
+                   embed_scale=float((d.get("embedding") or {}).get("scale", 1.0)),
+                   residual_mult=float(d.get("residual_mult", 1.0)), loop=loop,
+                   side_dim=int((d.get("token_side") or {}).get("dim", 0)))
 
     @classmethod
     def from_ini(cls, path: str) -> "ModelConfig":
@@ -430,19 +496,22 @@ def _rotary(i: int, m: dict, width: int, style: str) -> Optional[RotaryConfig]:
         return None
     r, sc = m["rot"], m["rot"].get("scaling") or {}
     rot = RotaryConfig(int(r["dims"]), float(r["base"]), float(sc.get("factor", 0.0)), float(sc.get("original", 0.0)),
-                       float(sc.get("fast", 32.0)), float(sc.get("slow", 1.0)), style)
+                       float(sc.get("fast", 32.0)), float(sc.get("slow", 1.0)), style, "banded" if "low" in sc else "yarn",
+                       float(sc.get("low", 1.0)), float(sc.get("high", 4.0)))
     if rot.dims % 2 or rot.dims > width:
         raise ValueError(f"layer {i}: rotary dims {rot.dims} do not fit heads of {width}")
     return rot
 
 
-def _layer_config(i: int, e: dict) -> LayerConfig:
+def _layer_config(i: int, e: dict, model_type: str) -> LayerConfig:
     """One entry of config.json's ``layers``."""
     kind, m = e.get("type"), e["mixer"]
     mask = m.get("mask") or {}
-    common = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m.get("vdim", m["dim"])), scale=float(m["scale"]),
+    common = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m.get("vdim", m["dim"])),
+                  scale=float(m["scale"] if kind != "gla" else int(m["dim"]) ** -0.5),
                   window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0),
-                  softcap=float(m.get("softcap") or 0.0), kv_from=-1 if m.get("kv_from") is None else int(m["kv_from"]))
+                  softcap=float(m.get("softcap") or 0.0), kv_from=-1 if m.get("kv_from") is None else int(m["kv_from"]),
+                  conv=int(m.get("conv") or 0), **MIXER_TRAITS.get(model_type, {}).get(kind, {}))
     if kind == "attention":
         mixer = MixerConfig(kv_heads=int(m.get("kv_heads", m["heads"])), rot=_rotary(i, m, int(m["dim"]), "half"), **common)
     elif kind == "latent_attention":
@@ -451,10 +520,16 @@ def _layer_config(i: int, e: dict) -> LayerConfig:
                             gate=True, **common)
         if mixer.keep_first or mixer.softcap:
             raise ValueError(f"layer {i}: latent attention has no kept first keys and no cap on the scores")
+    elif kind == "gla":
+        mixer = MixerConfig(kind="gla", kv_heads=common["heads"], tau=float(m["tau"]), **common)
     else:
         raise ValueError(f"layer {i}: unsupported mixer type {kind!r}")
     if mixer.heads % mixer.kv_heads:
         raise ValueError(f"layer {i}: {mixer.heads} query heads over {mixer.kv_heads} key/value heads")
+    if mixer.values_from_keys and (mixer.dim != mixer.vdim or mixer.kv_from >= 0):
+        raise ValueError(f"layer {i}: values that are keys have the keys' size and a cache of their own")
+    if mixer.conv and not mixer.values_from_keys:
+        raise ValueError(f"layer {i}: a short convolution is for layers whose values are their keys")
     f = e.get("mlp")
     if not f:
         return LayerConfig(mixer)
@@ -462,8 +537,13 @@ def _layer_config(i: int, e: dict) -> LayerConfig:
         return LayerConfig(mixer, int(f["ff"]), "dense")
     if f.get("kind") != "moe":
         raise ValueError(f"layer {i}: unsupported feed-forward {f.get('kind')!r}")
-    moe = MoeConfig(experts=int(f["router"]["experts"]), top=int(f["router"]["top"]), ff=int(f["expert"]["ff"]),
-                    shared=int((f.get("shared") or {}).get("ff", 0)))
-    if not 0 < moe.top <= moe.experts:
-        raise ValueError(f"layer {i}: {moe.top} of {moe.experts} experts")
+    r = f["router"]
+    groups = r.get("groups") or {}
+    moe = MoeConfig(experts=int(r["experts"]), top=int(r["top"]), ff=int(f["expert"]["ff"]),
+                    shared=int((f.get("shared") or {}).get("ff", 0)), scale=float(r.get("scale", 1.0)),
+                    groups=int(groups.get("count", 1)), keep_groups=int(groups.get("keep", 1)), **MOE_TRAITS.get(model_type, {}))
+    if moe.groups < 1 or moe.experts % moe.groups or not 0 < moe.keep_groups <= moe.groups:
+        raise ValueError(f"layer {i}: {moe.keep_groups} of {moe.groups} groups of {moe.experts} experts")
+    if not 0 < moe.top <= moe.experts // moe.groups * moe.keep_groups:
+        raise ValueError(f"layer {i}: {moe.top} of {moe.experts // moe.groups * moe.keep_groups} experts")
     return LayerConfig(mixer, 0, "moe", moe)

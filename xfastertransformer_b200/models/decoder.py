@@ -53,6 +53,7 @@ class Batch:
     is_decode: bool = False
     positions2: Optional[torch.Tensor] = None   # ChatGLM-1 block positions
     prefix_lm_lens: Optional[List[int]] = None
+    state_slots: Optional[torch.Tensor] = None  # [B] int32: each sequence's slot in the state pools
     max_q: int = 0
     max_kv: int = 0
     meta: dict = field(default_factory=dict)    # kernel-side scheduling scratch (native)

@@ -1,4 +1,4 @@
-"""Decoder for designs described layer by layer (``ModelConfig.layers``): Kafipel, Vepivik.
+"""Decoder for designs described layer by layer (``ModelConfig.layers``): Kafipel, Vepivik, Botusun.
 
 It is the generic decoder with sizes, rotation, mask and cache pool taken from each layer's own entry, served by the same
 engine, paged cache, decode runner, sampler and kernels.  What these designs add to it, each as an op with its constants
@@ -12,8 +12,14 @@ as arguments:
 * query/key and value heads of different sizes;
 * latent attention with a window, an output gate and layers that read another layer's latents
   (`ops.latent_prep`, `ops.latent_attention`); its pools have one row per token and no values;
-* mixtures of experts without a gate product (`ops.route`, `ops.moe_experts`), next to a shared expert;
-* a scaled embedding, and logits from the embedding table.
+* attention whose values are its keys, with short convolutions, a norm per head and rotation between the projection and the
+  cache (`ops.head_prep`), the convolutions' last inputs kept as a state;
+* gated linear attention, a recurrent layer with a state instead of a cache (`ops.gated_linear`);
+* mixtures of experts with or without a gate product, chosen by group or among all (`ops.route`, `ops.moe_experts`), next to
+  a shared expert;
+* layers that run several times in a row (`ModelConfig.runs`), each pass with a cache and states of its own;
+* a part of the token's own side embedding after every layer, gated by the residual stream;
+* a scaled embedding, a factor on everything that joins the residual stream, and logits from the embedding table.
 
 Widths that the 16-byte rows of the tensor-core kernels do not allow are padded with zeros at load: the hidden and the
 feed-forward width to a multiple of 8, heads to the next size the attention kernels have, each part of a latent head to a
@@ -22,6 +28,7 @@ to a score or a sum.  The 32-bit path (dtype "fp32") and CPU tensors keep the he
 """
 from __future__ import annotations
 
+import copy
 import math
 from typing import Dict, List, Optional
 
@@ -74,17 +81,30 @@ class LayeredDecoder(Decoder):
         self.has_moe = False
         with TimeLine("Decoder.loadWeights"):
             self._load_ends(embed_from)
-            self.layers: List[Layer] = [self._load_layer(i)
-                                        for i in ProgressBar.wrap(range(self.l0, self.l1), "Loading layers")]
-        # cache pools: one per layer with keys and values of its own
+            # pipeline stages are ranges of runs; a looped layer's weights are loaded once
+            runs = cfg.runs()
+            self.l0, self.l1 = P.pp_layer_range(len(runs), ctx.pp_size, ctx.pp_rank)
+            runs = runs[self.l0:self.l1]
+            loaded = {i: self._load_layer(i) for i in ProgressBar.wrap(sorted({i for i, _ in runs}), "Loading layers")}
+        self.layers: List[Layer] = list(loaded.values())
+        self.runs: List[Layer] = []
+        for i, t in runs:
+            L = copy.copy(loaded[i])
+            L.step = self._step_vector(t) if cfg.loop is not None and i == cfg.loop.start and t >= 0 else None
+            self.runs.append(L)
+        # cache pools: one per run with keys and values of its own; state pools: the ones each run asks for
         self.pools: Dict[int, int] = {}
-        for L in self.layers:
+        self.pool_shapes, self.state_shapes = [], []
+        for L in self.runs:
             if L.own_kv:
-                self.pools[L.idx] = len(self.pools)
-        for L in self.layers:
-            if L.kv_layer not in self.pools:
+                self.pools[L.idx] = len(self.pool_shapes)
+                self.pool_shapes.append((1, L.kd, 0) if L.mix.kind == "latent" else (L.hkv, L.kd, L.vd))
+            L.pool = self.pools.get(L.kv_layer, -1)
+            if L.pool < 0 and L.mix.has_kv:
                 raise ValueError(f"layer {L.idx} reads the keys of layer {L.kv_layer}, which is on another pipeline stage")
-            L.pool = self.pools[L.kv_layer]
+            if L.state_shape is not None:
+                L.state = len(self.state_shapes)
+                self.state_shapes.append(L.state_shape)
         L = self.layers[0]
         self.D, self.hq, self.hkv, self.group, self.scale = L.kd, L.hq, L.hkv, L.group, L.mix.scale
         for L in self.layers:
@@ -99,7 +119,10 @@ class LayeredDecoder(Decoder):
         tab = self._ropes.get(rot)
         if tab is None or tab.shape[0] < positions:
             n = max(_up(positions, 2048), 2 * tab.shape[0] if tab is not None else 0)
-            if rot.factor > 0:
+            if rot.factor > 0 and rot.scaling == "banded":
+                new = R.rope_table(n, rot.dims, rot.base, "banded", rot.factor, rot.original, rot.high, rot.low,
+                                   angle_dtype=torch.float64)
+            elif rot.factor > 0:
                 new = R.rope_table(n, rot.dims, rot.base, "yarn", rot.factor, rot.original, rot.fast, rot.slow,
                                    table_scale=0.1 * math.log(rot.factor) + 1.0, angle_dtype=torch.float64)
             else:
@@ -120,13 +143,23 @@ class LayeredDecoder(Decoder):
     def _gain(self, name: str):
         return self.src.vector(name, self.W, fake_ones=True), None      # (gain, bias)
 
+    def _step_vector(self, t: int) -> torch.Tensor:
+        """What joins the residual stream in front of pass `t` of the looped layers."""
+        return self.src.matrix("loop.step", (self.cfg.loop.times, self.W), rows=(t, t + 1))[0].float().contiguous()
+
     def _load_ends(self, share: Optional["LayeredDecoder"]) -> None:
         c = self.cfg
         self.v0, self.v1 = P.vocab_range(c.vocab_size, self.tp, self.tpr)
         if share is not None:
-            self.wte, self.final, self.lm_head = share.wte, share.final, share.lm_head
+            self.wte, self.final, self.lm_head, self.side_embed = share.wte, share.final, share.lm_head, share.side_embed
             return
-        self.wte = self.final = self.lm_head = None
+        self.wte = self.final = self.lm_head = self.side_embed = None
+        if c.side_dim:
+            # the part of each layer padded to the products' 16-byte rows
+            n, d = len(c.layers), c.side_dim
+            w = self.src.matrix("side.embed", (c.vocab_size, n * d)).view(c.vocab_size, n, d)
+            w = _pad(w, c.vocab_size, n, self._ff_size(d)).reshape(c.vocab_size, -1)
+            self.side_embed = w.to(torch.bfloat16 if self.device.type == "cuda" else w.dtype)
         if self.first_stage:
             self.wte = _pad(self.src.matrix("embed", (c.vocab_size, self.W)).to(torch.bfloat16), c.vocab_size, self.WP)
         if self.last_stage:
@@ -172,12 +205,17 @@ class LayeredDecoder(Decoder):
         L.q_off = qs - ks * L.group
         if L.hq <= 0:
             raise ValueError(f"layer {i}: {m.heads} heads cannot be split over {self.tp} ranks")
-        L.own_kv = m.kv_from < 0
+        L.own_kv = m.has_kv and m.kv_from < 0
+        L.state_shape = None
         L.kv_layer = i if L.own_kv else m.kv_from
         second = self._gain if self.spec.post_norm else lambda name: None
         L.norm1, L.norm1b = self._gain(p + "norm1"), second(p + "norm1b")
         if m.kind == "latent":
             self._load_latent(L, p, (qs, qe))
+        elif m.kind == "gla":
+            self._load_linear(L, p, (qs, qe))
+        elif m.values_from_keys:
+            self._load_shared_kv(L, p, (qs, qe), (ks, ke))
         else:
             self._load_attention(L, p, (qs, qe), (ks, ke))
         L.mlp_kind = "none"
@@ -194,6 +232,14 @@ class LayeredDecoder(Decoder):
             L.gate_up = make_linear(torch.cat([gate, up]), self.kind)
             L.down = make_linear(_pad(self.src.matrix(p + "mlp.down", (self.W, lc.ff), cols=r), self.WP, np_), self.kind)
             L.act = "silu"
+        L.side_gate = None
+        if self.cfg.side_dim:
+            d, kind = self.cfg.side_dim, "fp32" if self.exact or self.device.type == "cpu" else "bf16"
+            n = self._ff_size(d)
+            L.side_gate = make_linear(_pad(self.src.matrix(p + "side.gate", (d, self.W)), n, self.WP), kind)
+            L.side_proj = make_linear(_pad(self.src.matrix(p + "side.proj", (self.W, d)), self.WP, n), kind)
+            L.side_norm = self._gain(p + "side.norm")
+            L.side_at = i * n
         return L
 
     def _ff_size(self, n: int) -> int:
@@ -213,6 +259,45 @@ class LayeredDecoder(Decoder):
         if self.spec.sinks and (self.src.exists(p + "mix.sink") or self.src.fake):
             L.sinks = self.src.vector(p + "mix.sink", m.heads, rng=q).contiguous()
         self._out_rows(L, p, m.heads, q, m.vdim)
+
+    def _load_shared_kv(self, L: Layer, p: str, q, kv) -> None:
+        """Attention whose values are its keys.  Rows leave the projection with the heads' real size; `head_prep` pads them."""
+        m, n = L.mix, (L.hq + L.hkv) * L.mix.dim
+        L.kd = L.vd = self._head_size(m.dim)
+        parts = [(p + "mix.q", m.heads, q), (p + "mix.k", m.kv_heads, kv)]
+        w = torch.cat([self._rows(name, heads, rng, (m.dim, m.dim)) for name, heads, rng in parts])
+        L.qkv = make_linear(_pad(w, self._ff_size(n), self.WP), self.kind)
+        cut = lambda rng: (rng[0] * m.dim, rng[1] * m.dim)
+        L.qkv_b = None
+        if m.qk_bias:
+            b = [self.src.vector(name + ".b", heads * m.dim, rng=cut(rng)) for name, heads, rng in parts]
+            L.qkv_b = _pad(torch.cat(b), L.qkv.out_features).contiguous()
+        conv = None
+        if m.conv:
+            conv = [self.src.matrix(name + ".conv", (heads * m.dim, m.conv), rows=cut(rng)) for name, heads, rng in parts]
+            conv = torch.cat(conv).float().t().contiguous()                # [taps, channels]
+            if m.conv > 1:
+                L.state_shape = ((m.conv - 1, n), self.act_dtype)
+        norms = [self.src.vector(p + f"mix.{x}.norm", m.dim, fake_ones=True).contiguous() if m.qk_norm else None for x in "qk"]
+        L.prep = ops.HeadPrep(L.hq, L.hkv, m.dim, L.kd, conv, *norms)
+        L.sinks = None if m.sink is None else torch.full((L.hq,), m.sink, dtype=torch.float32, device=self.device)
+        self._out_rows(L, p, m.heads, q, m.vdim)
+
+    def _load_linear(self, L: Layer, p: str, rng) -> None:
+        """Gated linear attention: queries, keys, values, output gate and the decay's first product are one projection."""
+        m, gpu = L.mix, self.device.type == "cuda"
+        rank = self.src.shape(p + "mix.a1", (16, self.W))[0]
+        d = L.dims = ops.LinearDims(L.hq, m.dim, m.vdim, rank, 8 if gpu else 1)
+        L.kd, L.vd = m.dim, m.vdim
+        rows = [self._rows(p + "mix." + x, m.heads, rng, (n, n)) for x, n in (("q", m.dim), ("k", m.dim), ("v", m.vdim), ("g", m.vdim))]
+        rows.append(_pad(self.src.matrix(p + "mix.a1", (rank, self.W)), rank, self.WP))
+        L.qkv = make_linear(torch.cat([_pad(r, d.up(r.shape[0]), self.WP) for r in rows]), self.kind)
+        a2 = self.src.matrix(p + "mix.a2", (m.heads * m.dim, rank), rows=(rng[0] * m.dim, rng[1] * m.dim)).to(self.act_dtype)
+        bias = self.src.vector(p + "mix.a2.b", m.heads * m.dim, rng=(rng[0] * m.dim, rng[1] * m.dim))
+        gain = self.src.vector(p + "mix.norm", m.vdim, fake_ones=True)
+        L.decay = ops.LinearWeights(_pad(a2, a2.shape[0], d.up(rank)).contiguous(), bias.contiguous(), m.tau, gain.contiguous())
+        L.state_shape = ((L.hq, m.dim, m.vdim), torch.float32)
+        self._out_rows(L, p, m.heads, rng, m.vdim)
 
     def _load_latent(self, L: Layer, p: str, q) -> None:
         """Latent attention: heads are split over ranks, the latents (one row per token) are on every rank."""
@@ -242,9 +327,13 @@ class LayeredDecoder(Decoder):
         kind = "fp32" if self.exact or self.device.type == "cpu" else "bf16"
         L.router = make_linear(_pad(self.src.matrix(p + "mlp.router", (f.experts, self.W)), f.experts, self.WP), kind)
 
+        L.correction = self.src.vector(p + "mlp.correction", f.experts).contiguous() if f.correction else None
+        first = ("gate", "up") if f.gated else ("up",)
+
         def pair(name, ff, r):
             n = self._ff_size(r[1] - r[0])
-            return (make_linear(_pad(self.src.matrix(p + name + ".up", (ff, self.W), rows=r), n, self.WP), self.kind),
+            w = [_pad(self.src.matrix(f"{p}{name}.{x}", (ff, self.W), rows=r), n, self.WP) for x in first]
+            return (make_linear(torch.cat(w), self.kind),
                     make_linear(_pad(self.src.matrix(p + name + ".down", (self.W, ff), cols=r), self.WP, n), self.kind))
         L.e0, L.e1 = self._local_experts(f.experts)
         r = (0, f.ff) if self.ctx.ep_size > 1 else self._ffn_range(f.ff)
@@ -256,7 +345,8 @@ class LayeredDecoder(Decoder):
     # ------------------------------------------------------------------------------------
     def _mixer(self, L: Layer, h: torch.Tensor, b: Batch, cache: PagedKVCache) -> torch.Tensor:
         """Token-mixing sublayer: normalised input -> output projection (summed over tensor-parallel ranks)."""
-        a = (self._latent if L.mix.kind == "latent" else self._attend)(L, h, b, cache)
+        kind = "shared" if L.mix.values_from_keys else L.mix.kind
+        a = {"latent": self._latent, "gla": self._linear, "shared": self._shared_kv}.get(kind, self._attend)(L, h, b, cache)
         with TimeLine("Output"):
             return self._row_parallel(a, L.o, None, None)
 
@@ -269,6 +359,24 @@ class LayeredDecoder(Decoder):
                             self.eps, pool, b.slots)
         with TimeLine("MHA"):
             return ops.latent_attention(x, L.dims, pool, b.block_table, b.cu_q, b.kv_lens, L.up, m.scale, m.window, meta=b)
+
+    def _linear(self, L: Layer, h: torch.Tensor, b: Batch, cache: PagedKVCache) -> torch.Tensor:
+        with TimeLine("QKV.linear"):
+            x = ops.linear(h, L.qkv)
+        with TimeLine("GLA"):
+            return ops.gated_linear(x, L.dims, L.decay, self.eps, cache.state[L.state], b.state_slots, b.cu_q, b.kv_lens, meta=b)
+
+    def _shared_kv(self, L: Layer, h: torch.Tensor, b: Batch, cache: PagedKVCache) -> torch.Tensor:
+        m, kc, vc = L.mix, cache.k[L.pool], cache.v[L.pool]
+        with TimeLine("QKV.linear"):
+            x = ops.linear(h, L.qkv, L.qkv_b)
+        with TimeLine("QKPO"):
+            q = ops.head_prep(x, L.prep, self.eps, b.positions, self._rope(m.rot, 0), m.rot.dims if m.rot is not None else 0, kc, vc,
+                              b.slots, cache.state[L.state] if m.conv > 1 else None, b.state_slots, b.cu_q, b.kv_lens, meta=b)
+        with TimeLine("MHA"):
+            a = ops.paged_attention(q, kc, vc, b.block_table, b.cu_q, b.kv_lens, m.scale, group=L.group, q_off=L.q_off, meta=b,
+                                    softcap=m.softcap, window=m.window, keep_first=m.keep_first, sinks=L.sinks)
+        return a.reshape(a.shape[0], -1)
 
     def _attend(self, L: Layer, h: torch.Tensor, b: Batch, cache: PagedKVCache) -> torch.Tensor:
         m, li = L.mix, L.pool
@@ -303,13 +411,13 @@ class LayeredDecoder(Decoder):
         """Mixture of experts -> fp32 rows (summed over tensor-parallel ranks)."""
         f = L.moe
         logits = ops.linear(h, L.router, out_dtype=torch.float32)
-        idx, w = ops.route(logits, "deepseek", f.top, norm_topk=True, scoring="softmax")
+        idx, w = ops.route(logits, "deepseek", f.top, L.correction, f.groups, f.keep_groups, f.scale, f.renorm, f.scoring)
         shared = None
         if L.shared is not None:
             # few rows: the product leaves in fp32; prompts: in the activation type, like the experts' own rows
-            shared = ops.linear(ops.linear(h, L.shared[0], act=L.act), L.shared[1],
-                                out_dtype=torch.float32 if h.shape[0] <= 128 else None)
-        out = ops.moe_experts(h, idx, w, L.experts, L.act, L.e0, gated=False, add=shared)
+            u = ops.linear_gated(h, L.shared[0], L.act) if f.gated else ops.linear(h, L.shared[0], act=L.act)
+            shared = ops.linear(u, L.shared[1], out_dtype=torch.float32 if h.shape[0] <= 128 else None)
+        out = ops.moe_experts(h, idx, w, L.experts, L.act, L.e0, gated=f.gated, add=shared)
         if self.tp > 1:
             peer = getattr(self.ctx, "peer", None)
             if peer is not None and out.is_cuda and out.numel() <= peer.slot:
@@ -317,40 +425,52 @@ class LayeredDecoder(Decoder):
             return self.ctx.all_reduce(out)
         return out
 
+    def _side(self, L: Layer, x: torch.Tensor, e: torch.Tensor) -> torch.Tensor:
+        """The token's own side embedding, gated by the residual stream `x` (in the activation type), as wide as it."""
+        with TimeLine("Side"):
+            n = L.side_gate.out_features
+            g = ops.linear(x, L.side_gate, act="gelu_tanh", times=e[:, L.side_at:L.side_at + n])
+            return ops.linear(g, L.side_proj)
+
     def _add_norm(self, x, y, post, nxt, **kw):
-        return ops.residual_norm(x, y, post, nxt, self.eps, self.spec.norm, h_dtype=self.act_dtype, **kw)
+        return ops.residual_norm(x, y, post, nxt, self.eps, self.spec.norm, h_dtype=self.act_dtype, mult=self.cfg.residual_mult, **kw)
 
     def forward(self, b: Batch, cache: PagedKVCache, hidden: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Local logits on the last stage, the residual stream otherwise.  The norm of each sublayer's output, the
-        residual sum and the norm in front of the next sublayer are one launch; so are the embedding and the first norm,
-        and on the last stage the last sum and the final norm, on the rows whose logits are wanted."""
+        residual sum, the vector in front of a pass of looped layers and the norm in front of the next sublayer are one
+        launch; so are the embedding and the first norm, and on the last stage the last sum and the final norm, on the
+        rows whose logits are wanted."""
         self._ensure_positions(b, cache)
         dbg = debugger.enabled()
         step = debugger.next_step() if dbg else 0
         with TimeLine("Decoder.forward"):
-            first = self.layers[0].norm1
+            first = self.runs[0]
             if self.first_stage:
-                x, h = self._add_norm(None, None, None, first, ids=b.ids, table=self.wte, embed_scale=self.cfg.embed_scale)
+                x, h = self._add_norm(None, None, None, first.norm1, ids=b.ids, table=self.wte, embed_scale=self.cfg.embed_scale,
+                                      add=first.step)
             else:
-                x, h = self._add_norm(hidden, None, None, first)
+                x, h = self._add_norm(hidden, None, None, first.norm1, add=first.step)
             if dbg:
                 debugger.dump("embedding", x[:, :self.W], self.ctx.rank, step)
-            for n, L in enumerate(self.layers):
-                last = n + 1 == len(self.layers)
-                after = None if last else self.layers[n + 1].norm1
+            side = ops.embedding(b.ids, self.side_embed, 1.0, self.act_dtype) if self.side_embed is not None else None
+            for n, L in enumerate(self.runs):
+                nxt = self.runs[n + 1] if n + 1 < len(self.runs) else None
                 y, post = self._mixer(L, h, b, cache), L.norm1b
                 if L.mlp_kind != "none":
                     x, h = self._add_norm(x, y, post, L.norm2)
                     if dbg:
                         debugger.dump(f"layer{L.idx}_attn_out", x[:, :self.W], self.ctx.rank, step)
                     y, post = self._ff(L, h), L.norm2b
-                if not last:
-                    x, h = self._add_norm(x, y, post, after)
-                elif dbg or not self.last_stage:
+                if L.side_gate is not None:
+                    x, h = self._add_norm(x, y, post, None, raw=True)
+                    y, post = self._side(L, h, side), L.side_norm
+                if dbg or nxt is None and not self.last_stage:
                     x, _ = self._add_norm(x, y, post, None)
                     y = post = None
                 if dbg:
                     debugger.dump(f"layer{L.idx}_ffn_out", x[:, :self.W], self.ctx.rank, step)
+                if nxt is not None:
+                    x, h = self._add_norm(x, y, post, nxt.norm1, add=nxt.step)
             if not self.last_stage:
                 return x
             if b.logit_rows is not None and b.logit_rows.numel() == 0:
@@ -364,6 +484,6 @@ class LayeredDecoder(Decoder):
         return None                               # windows differ from layer to layer: each launch plans its own split
 
     def kv_geometry(self):
-        own = [L for L in self.layers if L.own_kv]
-        pools = [(1, L.kd, 0) if L.mix.kind == "latent" else (L.hkv, L.kd, L.vd) for L in own]
-        return dict(kv_heads=pools[0][0], k_dim=pools[0][1], v_dim=pools[0][2], latent=False, layers=pools)
+        first = self.pool_shapes[0] if self.pool_shapes else (0, 0, 0)
+        return dict(kv_heads=first[0], k_dim=first[1], v_dim=first[2], latent=False, layers=self.pool_shapes,
+                    states=self.state_shapes)

@@ -56,6 +56,7 @@ FAMILIES: Dict[str, FamilySpec] = {
     "telechat": FamilySpec("telechat", dense_bias=True, telechat_ntk=True),
     "kafipel": FamilySpec("kafipel", norm="layer", layered=True, post_norm=True, sinks=True),
     "vepivik": FamilySpec("vepivik", layered=True, tied_head=True),
+    "botusun": FamilySpec("botusun", layered=True, tied_head=True),
 }
 
 

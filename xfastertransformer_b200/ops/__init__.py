@@ -53,13 +53,13 @@ def layernorm(x, w, b, eps):
 
 
 def residual_norm(x, y, post, nxt, eps, kind="layer", rows=None, h_dtype=torch.bfloat16, ids=None, table=None, keep_x=True,
-                  embed_scale=1.0):
-    """One step of a 32-bit residual stream in one launch: x (or table[ids] * embed_scale) += norm(y) with `post` = (gain, bias or
-    None) (plain y without it), then h = norm(x) with `nxt` for the next product.  Returns (x, h); on a GPU x is updated
-    in place unless `rows` selects rows, and buffers are as wide as x (a multiple of 8, padding zero)."""
-    if _cuda(x if x is not None else table):
-        return _nat().residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids, table, keep_x, embed_scale)
-    return R.residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids, table, keep_x, embed_scale)
+                  embed_scale=1.0, mult=1.0, add=None, raw=False):
+    """One step of a 32-bit residual stream in one launch: x (or table[ids] * embed_scale) += mult * norm(y) with `post` =
+    (gain, bias or None) (plain y without it) + the vector `add`, then h = norm(x) with `nxt` for the next product (`raw`: x
+    itself).  Returns (x, h); on a GPU x is updated in place unless `rows` selects rows, and buffers are as wide as x (a
+    multiple of 8, padding zero)."""
+    impl = _nat().residual_norm if _cuda(x if x is not None else table) else R.residual_norm
+    return impl(x, y, post, nxt, eps, kind, rows, h_dtype, ids, table, keep_x, embed_scale, mult, add, raw)
 
 
 # -- GEMMs ---------------------------------------------------------------------------------
@@ -86,7 +86,10 @@ def _timed(kernel: str, x, W, fn):
     return y
 
 
-def linear(x, W, bias=None, act=None, residual=None, res_scale=1.0, out_dtype=None):
+def linear(x, W, bias=None, act=None, residual=None, res_scale=1.0, out_dtype=None, times=None):
+    """act(x W^T + bias) + res_scale * residual, or with `times` [T, out] act(x W^T + bias) * times."""
+    if times is not None:
+        return (_nat() if _cuda(x) else R).linear_times(x, W, bias, act, times)
     if _verbose():
         name = "gemm" + ("_bias" if bias is not None else "") + (f"_{act}" if act else "") + \
             ("_residual" if residual is not None else "")
@@ -296,6 +299,88 @@ class LatentWeights:
     def __init__(self, uk, uv):
         self.uk, self.uv = uk.contiguous(), uv.contiguous()
         self.cache: dict = {}               # layouts the kernels want, made once
+
+
+# -- attention whose values are its keys ------------------------------------------------------
+@dataclass
+class HeadPrep:
+    """What happens to the heads of a packed row [q: hq x dim | k: hkv x dim] between projection and cache: weights of the
+    short convolution [taps, (hq + hkv) * dim] fp32 (None: none), gains of the norms per head (None: none).  Heads leave
+    `padded` wide, zeros behind `dim`."""
+    hq: int
+    hkv: int
+    dim: int
+    padded: int
+    conv: Optional[torch.Tensor]
+    q_norm: Optional[torch.Tensor]
+    k_norm: Optional[torch.Tensor]
+
+    @property
+    def taps(self) -> int:
+        return 1 if self.conv is None else self.conv.shape[0]
+
+
+def head_prep(x, prep: HeadPrep, eps, positions, table, rot_dims, kc, vc, slots, state, state_slots, cu_q, kv_lens, meta=None):
+    """Causal convolution over time on every channel of q and k, RMS norm per head, rotation of the first `rot_dims`
+    dimensions; appends k to `kc` and the keys as they left the convolution to `vc`, and returns q [T, hq, padded].
+    `state` [slots, taps - 1, channels] holds the last inputs of each sequence's convolution, oldest first, and is moved on
+    to the end of this call's tokens; what lies before a sequence's first token counts as zero."""
+    impl = _native_linear().head_prep if _cuda(x) else R.head_prep
+    return impl(x, prep, eps, positions, table, rot_dims, kc, vc, slots, state, state_slots, cu_q, kv_lens, meta)
+
+
+# -- gated linear attention -------------------------------------------------------------------
+@dataclass(frozen=True)
+class LinearDims:
+    """A packed row of a gated-linear-attention layer: [q: heads x dim | k | v: heads x vdim | g | a1: rank], each part
+    starting at a multiple of `align` values."""
+    heads: int
+    dim: int
+    vdim: int
+    rank: int
+    align: int = 1
+
+    def up(self, n: int) -> int:
+        return (n + self.align - 1) // self.align * self.align
+
+    @property
+    def k_at(self) -> int:
+        return self.up(self.heads * self.dim)
+
+    @property
+    def v_at(self) -> int:
+        return 2 * self.k_at
+
+    @property
+    def g_at(self) -> int:
+        return self.v_at + self.up(self.heads * self.vdim)
+
+    @property
+    def a_at(self) -> int:
+        return self.g_at + self.up(self.heads * self.vdim)
+
+
+@dataclass
+class LinearWeights:
+    """Decay and output norm: the decay's second product a2 [heads * dim, rank (aligned)] and its bias, `tau`, the gain of
+    the norm over a head's vdim outputs."""
+    a2: torch.Tensor
+    bias: torch.Tensor
+    tau: float
+    norm: torch.Tensor
+
+
+def gated_linear(x, dims: LinearDims, w: LinearWeights, eps, state, state_slots, cu_q, kv_lens, meta=None):
+    """Gated linear attention of packed rows x -> [T, heads * vdim].  Per head, with decay = sigmoid(W_a2 a1 + bias)^(1 / tau)
+    per key channel: S <- diag(decay) S + k v^T and o = S^T (q / sqrt(dim)); the result is norm(o) * silu(g).  `state`
+    [slots, heads, dim, vdim] fp32 is carried on; a sequence's first token starts from zero."""
+    impl = _native_linear().gated_linear if _cuda(x) else R.gated_linear
+    return impl(x, dims, w, eps, state, state_slots, cu_q, kv_lens, meta)
+
+
+def _native_linear():
+    from . import native_linear
+    return native_linear
 
 
 # -- MoE -----------------------------------------------------------------------------------

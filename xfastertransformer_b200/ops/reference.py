@@ -72,18 +72,21 @@ def _norm(xf: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor], eps: flo
 
 
 def residual_norm(x, y, post, nxt, eps: float, kind: str = "layer", rows: Optional[torch.Tensor] = None,
-                  h_dtype: torch.dtype = torch.float32, ids=None, table=None, keep_x: bool = True, embed_scale: float = 1.0):
-    """One step of a 32-bit residual stream: x (or table[ids] * embed_scale) plus y — normalised with `post` = (gain, bias) first, when
-    given — and the input of the next sublayer, h = norm(x) with `nxt` = (gain, bias).  `rows` selects rows.  Returns
-    (x or None, h or None)."""
+                  h_dtype: torch.dtype = torch.float32, ids=None, table=None, keep_x: bool = True, embed_scale: float = 1.0,
+                  mult: float = 1.0, add: Optional[torch.Tensor] = None, raw: bool = False):
+    """One step of a 32-bit residual stream: x (or table[ids] * embed_scale) plus mult * y — normalised with `post` = (gain,
+    bias) first, when given — plus the vector `add`, and the input of the next sublayer, h = norm(x) with `nxt` = (gain,
+    bias), or x itself with `raw`.  `rows` selects rows.  Returns (x or None, h or None)."""
     xf = table[ids.long()].float() * embed_scale if ids is not None else x.float()
     yf = None if y is None else y.float()
     if rows is not None:
         xf = xf[rows.long()]
         yf = None if yf is None else yf[rows.long()]
     if yf is not None:
-        xf = xf + (_norm(yf, post[0], post[1], eps, kind) if post is not None else yf)
-    h = None if nxt is None else _norm(xf, nxt[0], nxt[1], eps, kind).to(h_dtype)
+        xf = xf + mult * (_norm(yf, post[0], post[1], eps, kind) if post is not None else yf)
+    if add is not None:
+        xf = xf + add
+    h = xf.to(h_dtype) if raw else None if nxt is None else _norm(xf, nxt[0], nxt[1], eps, kind).to(h_dtype)
     return (xf if keep_x else None), h
 
 
@@ -227,6 +230,11 @@ def gated_act(gu: torch.Tensor, act: str = "silu") -> torch.Tensor:
     return (_act(g, act) * u).to(gu.dtype)
 
 
+def linear_times(x: torch.Tensor, W, bias, act, times: torch.Tensor) -> torch.Tensor:
+    """act(x W^T + bias) * times"""
+    return (linear(x, W, bias, act, out_dtype=torch.float32) * times.float()).to(x.dtype)
+
+
 def linear_gated(x: torch.Tensor, W, act: str = "silu", bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """act(x Wg^T) * (x Wu^T) with W = cat(gate, up) on the out dim; the intermediate is
     kept in fp32 (the fused kernel applies the activation on the TMEM accumulators)."""
@@ -255,11 +263,16 @@ def yarn_mscale(scale: float = 1.0, mscale: float = 1.0) -> float:
 def rope_inv_freq(rot_dim: int, theta: float, scaling_type: str = "", factor: float = 1.0,
                   original_max_pos: int = 2048, beta_fast: float = 32, beta_slow: float = 1,
                   dtype: torch.dtype = torch.float32) -> torch.Tensor:
-    """Frequency of each rotated pair.  YaRN divides the slow ones by `factor`: none of the pairs up to `low`, all from
+    """Frequency of each rotated pair.  "banded" (Llama 3.1): wavelengths below original / beta_fast stay, those above
+    original / beta_slow are divided by `factor`, with a ramp in original / wavelength between.  YaRN divides the slow ones by `factor`: none of the pairs up to `low`, all from
     `high` on, a linear ramp between (a step when the two coincide)."""
     inv = 1.0 / (theta ** (torch.arange(0, rot_dim, 2, dtype=torch.float64) / rot_dim))
     if scaling_type == "linear" and factor != 1.0:
         inv = inv / factor
+    elif scaling_type == "banded":
+        turns = original_max_pos * inv / (2 * math.pi)                     # original / wavelength
+        s = ((turns - beta_slow) / (beta_fast - beta_slow)).clamp(0, 1) if beta_fast != beta_slow else (turns >= beta_slow).double()
+        inv = (1 - s) * inv / factor + s * inv
     elif scaling_type == "yarn" and factor != 1.0:
         low = max(math.floor(_yarn_find_dim(beta_fast, rot_dim, theta, original_max_pos)), 0)
         high = min(math.ceil(_yarn_find_dim(beta_slow, rot_dim, theta, original_max_pos)), rot_dim - 1)
@@ -536,7 +549,7 @@ def route_deepseek(logits: torch.Tensor, bias: Optional[torch.Tensor], top_k: in
     sel = scores + (bias.float() if bias is not None else 0.0)
     if n_group > 1:
         grp = sel.view(T, n_group, E // n_group)
-        gscore = grp.topk(2, dim=-1)[0].sum(-1)
+        gscore = grp.topk(min(2, E // n_group), dim=-1)[0].sum(-1)
         gidx = gscore.topk(topk_group, dim=-1)[1]
         gmask = torch.zeros(T, n_group, device=x.device, dtype=torch.bool).scatter_(1, gidx, True)
         sel = sel.masked_fill(~gmask[:, :, None].expand(T, n_group, E // n_group).reshape(T, E), float("-inf"))
@@ -569,6 +582,61 @@ def moe_experts(x: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, experts, ac
     if out is None:
         out = torch.zeros(T, experts[0][1].out_features, dtype=torch.float32, device=x.device)
     return out
+
+
+# ----------------------------------------------------------------------------------------
+# recurrent mechanisms
+# ----------------------------------------------------------------------------------------
+def head_prep(x, prep, eps, positions, table, rot_dims, kc, vc, slots, state, state_slots, cu_q, kv_lens, meta=None):
+    """See `ops.head_prep`."""
+    n_taps, dim, hq, hkv = prep.taps, prep.dim, prep.hq, prep.hkv
+    C = (hq + hkv) * dim
+    u = x[:, :C].float()
+    if prep.conv is not None:
+        out = torch.empty_like(u)
+        for b in range(len(kv_lens)):
+            a, e = int(cu_q[b]), int(cu_q[b + 1])
+            past = int(kv_lens[b]) - (e - a)
+            before = u.new_zeros(n_taps - 1, C)
+            if n_taps > 1 and past > 0:
+                s = int(state_slots[b])
+                n = min(past, n_taps - 1)
+                before[n_taps - 1 - n:] = state[s, n_taps - 1 - n:].float()
+            seq = torch.cat([before, u[a:e]])
+            out[a:e] = sum(prep.conv[j] * seq[j:j + e - a] for j in range(n_taps))
+            if n_taps > 1:
+                state[int(state_slots[b])] = seq[-(n_taps - 1):].to(state.dtype)
+        u = out
+    q, k = u[:, :hq * dim].reshape(-1, hq, dim), u[:, hq * dim:].reshape(-1, hkv, dim)
+    v = k
+    if prep.q_norm is not None:
+        q, k = rmsnorm(q, prep.q_norm, eps), rmsnorm(k, prep.k_norm, eps)
+    if table is not None and rot_dims > 0:
+        q, k = rope_apply(q, k, positions, table, rot_dims, "half")
+    pad = lambda t: F.pad(t, (0, prep.padded - dim))
+    kv_cache_write(pad(k).to(kc.dtype), pad(v).to(vc.dtype), kc, vc, slots)
+    return pad(q).to(x.dtype)
+
+
+def gated_linear(x, d, w, eps, state, state_slots, cu_q, kv_lens, meta=None):
+    """See `ops.gated_linear`."""
+    T, H = x.shape[0], d.heads
+    f = x.float()
+    q = f[:, :H * d.dim].view(T, H, d.dim) * d.dim ** -0.5
+    k = f[:, d.k_at:d.k_at + H * d.dim].view(T, H, d.dim)
+    v = f[:, d.v_at:d.v_at + H * d.vdim].view(T, H, d.vdim)
+    g = f[:, d.g_at:d.g_at + H * d.vdim]
+    z = f[:, d.a_at:d.a_at + d.rank] @ w.a2[:, :d.rank].float().t() + w.bias
+    decay = torch.exp(F.logsigmoid(z) / w.tau).view(T, H, d.dim)
+    o = torch.empty(T, H, d.vdim)
+    for b in range(len(kv_lens)):
+        a, e, slot = int(cu_q[b]), int(cu_q[b + 1]), int(state_slots[b])
+        S = state[slot].clone() if int(kv_lens[b]) > e - a else torch.zeros_like(state[slot])
+        for t in range(a, e):
+            S = decay[t, :, :, None] * S + k[t, :, :, None] * v[t, :, None, :]
+            o[t] = torch.einsum("hd,hdv->hv", q[t], S)
+        state[slot] = S
+    return (rmsnorm(o, w.norm, eps).reshape(T, -1) * F.silu(g)).to(x.dtype)
 
 
 # ----------------------------------------------------------------------------------------

@@ -7,7 +7,7 @@ flash-decode, the TP reductions), final norm, lm_head, arg-max and the cross-ran
 merge — is captured once and replayed.  Per step the host only
 
   1. appends one cache slot per sequence (block allocator, host side),
-  2. fills ONE pinned int32 staging buffer [ids | positions | slots | kv_lens | block_table],
+  2. fills ONE pinned int32 staging buffer [ids | positions | slots | kv_lens | state slots | block_table],
   3. issues one H2D copy, one graph launch, one D2H copy of the chosen tokens, and waits.
 
 Greedy decoding with no repetition penalty takes this path; anything else (sampling, beams,
@@ -41,7 +41,7 @@ class CudaRunner:
         self.kernel_launches = 0          # kernels of this library launched through replayed graphs / eager steps
         self.timing = False               # record a CUDA-event pair around each step's launch
         self.step_events = []
-        self._scratch_block = None
+        self._scratch_block = self._scratch_state = None
         if self.enabled:
             # taken now, while the pools are empty: a block taken after a request reserved its blocks would leave that
             # request one block short and make the pools grow (and move) in the middle of its decode
@@ -101,11 +101,13 @@ class CudaRunner:
         return self.bucket(len(seqs)), W
 
     def _scratch(self) -> int:
-        """One KV block owned by the runner: padding rows of a bucketed batch write their key/value there and attend
-        to it (a context of one token), so they touch no live sequence."""
+        """One KV block (and state slot) owned by the runner: padding rows of a bucketed batch write their key/value there
+        and attend to it (a context of one token), so they touch no live sequence."""
         if getattr(self, "_scratch_block", None) is None:
             self.m.cache.reserve(1)
             self._scratch_block = self.m.cache.alloc.alloc()
+            if self.m.cache.has_state:
+                self._scratch_state = self.m.cache.take_state()
         return self._scratch_block
 
     def worth_capturing(self, seqs: Sequence) -> bool:
@@ -121,17 +123,18 @@ class CudaRunner:
     # ------------------------------------------------------------------------------------
     def _layout(self, B: int, W: int):
         o_ids, o_pos, o_slot, o_kv = 0, B, 2 * B, 3 * B
-        o_cu = 4 * B
-        o_bt = 5 * B + 1
+        o_st = 4 * B
+        o_cu = 5 * B
+        o_bt = 6 * B + 1
         # keep the block table 16-byte aligned
         o_bt = (o_bt + 3) // 4 * 4
-        return o_ids, o_pos, o_slot, o_kv, o_cu, o_bt, o_bt + B * W
+        return o_ids, o_pos, o_slot, o_kv, o_st, o_cu, o_bt, o_bt + B * W
 
     def _build(self, B: int, W: int, max_kv_hint: int) -> _Graph:
         m = self.m
         g = _Graph()
         g.B, g.W = B, W
-        o_ids, o_pos, o_slot, o_kv, o_cu, o_bt, total = self._layout(B, W)
+        o_ids, o_pos, o_slot, o_kv, o_st, o_cu, o_bt, total = self._layout(B, W)
         g.host = torch.zeros(total, dtype=torch.int32).pin_memory()
         g.dev = torch.zeros(total, dtype=torch.int32, device=self.dev)
         g.tok_dev = torch.zeros(B, dtype=torch.int64, device=self.dev)
@@ -145,6 +148,8 @@ class CudaRunner:
                   logit_rows=None, is_decode=True, max_q=1, max_kv=max_kv_hint)
         b.cu_q_dev = d[o_cu:o_cu + B + 1]
         b.kv_lens_dev = d[o_kv:o_kv + B]
+        if m.cache.has_state:
+            b.state_slots = d[o_st:o_st + B]
         if g.nsplit is not None:
             b.meta["nsplit"] = g.nsplit
         g.batch = b
@@ -173,13 +178,14 @@ class CudaRunner:
     def _fill(self, g: _Graph, seqs, slots: List[int]) -> None:
         m = self.m
         B, W = g.B, g.W
-        o_ids, o_pos, o_slot, o_kv, o_cu, o_bt, total = self._layout(B, W)
+        o_ids, o_pos, o_slot, o_kv, o_st, o_cu, o_bt, total = self._layout(B, W)
         h = g.host
         cache = m.cache
         slots = list(slots)
         ids = [s.pending[0] for s in seqs]
         pos = [s.past_len for s in seqs]
         kvl = [s.past_len + 1 for s in seqs]
+        states = cache.state_slots([s.seq_id for s in seqs]) if cache.has_state else [0] * len(seqs)
         pad = B - len(seqs)
         if pad:                                        # padding rows of the bucket: one token in the scratch block
             sb = self._scratch()
@@ -187,9 +193,10 @@ class CudaRunner:
             pos += [0] * pad
             slots += [sb * cache.block] * pad
             kvl += [1] * pad
-        # ids | positions | slots | kv lengths are adjacent in the staging buffer: one conversion, one copy
-        assert (o_ids, o_pos, o_slot, o_kv) == (0, B, 2 * B, 3 * B)
-        h[0:4 * B] = torch.tensor(ids + pos + slots + kvl, dtype=torch.int32)
+            states += [self._scratch_state or 0] * pad
+        # ids | positions | slots | kv lengths | state slots are adjacent in the staging buffer: one conversion, one copy
+        assert (o_ids, o_pos, o_slot, o_kv, o_st) == (0, B, 2 * B, 3 * B, 4 * B)
+        h[0:5 * B] = torch.tensor(ids + pos + slots + kvl + states, dtype=torch.int32)
         bt = cache.block_table([s.seq_id for s in seqs], W)
         n = len(seqs)
         h[o_bt:o_bt + n * W] = bt.view(-1)

@@ -55,9 +55,10 @@ def _to_lists(ids) -> List[List[int]]:
 
 class Model:
     def __init__(self, path: str, dtype: str = "bf16", kv_cache_dtype: str = "fp16",
-                 ctx: Optional[DistContext] = None, max_cache_tokens: int = 0):
+                 ctx: Optional[DistContext] = None, max_cache_tokens: int = 0, max_sequences: int = 0):
         """`max_cache_tokens` > 0 fixes the size of the KV pools (rounded up to whole blocks): they are made once and
-        never grow, and a request that does not fit raises MemoryError."""
+        never grow, and a request that does not fit raises MemoryError.  `max_sequences` > 0 does the same for the
+        recurrent states of designs that have them."""
         if kv_cache_dtype not in KV_DTYPES:
             raise ValueError(f"don't support KV cache data type: {kv_cache_dtype}.")
         self.ctx = ctx or DistContext.get()
@@ -75,6 +76,8 @@ class Model:
             raise ValueError("XFT_ATTENTION_DP=1 does not run layered designs")
         if layered and kv_cache_dtype == "int8" and any(l.mixer.kind == "latent" for l in self.cfg.layers):
             raise ValueError("latent attention keeps its cache in the activation type: kv_cache_dtype int8 is not for it")
+        if layered and kv_cache_dtype == "int8" and any(l.mixer.values_from_keys for l in self.cfg.layers):
+            raise ValueError("layers whose values are their keys keep them in the activation type: kv_cache_dtype int8 is not for them")
         if self.cfg.model_type == "deepseek_moe" and d_prefill not in ("bf16", "fp8_e4m3"):
             raise ValueError("deepseek_moe supports bf16 and fp8_e4m3 only")      # model_factory.h:105-114
         if d_prefill == "fp8_e4m3" and self.cfg.model_type != "deepseek_moe":
@@ -93,10 +96,14 @@ class Model:
         max_blocks = (max_cache_tokens + blk - 1) // blk + spare if max_cache_tokens > 0 else 0
         self.cache = PagedKVCache(len(self.decoder.layers), geo["kv_heads"], geo["k_dim"], geo["v_dim"],
                                   kv_cache_dtype, self.ctx.device, blk, self.decoder.act_dtype, geo["latent"],
-                                  geo.get("layers"), max_blocks)
+                                  geo.get("layers"), max_blocks, geo.get("states", ()),
+                                  max_sequences + spare if max_sequences > 0 else 0)
         if max_blocks:
             self.cache.ensure_blocks(max_blocks)
-        if self.env.prefix_cache and self.ctx.dp_size == 1:
+        if self.cache.max_states:
+            self.cache.ensure_states(self.cache.max_states)
+        if self.env.prefix_cache and self.ctx.dp_size == 1 and not self.cache.has_state:
+            # (a recurrent state is known only where a sequence stands, not at each block's end)
             # data-parallel attention keeps each sequence's cache on one rank only, while all ranks must agree on how
             # many tokens a prompt still has to run: automatic reuse stays off there
             from .kv_cache import PrefixIndex
@@ -312,6 +319,7 @@ class Model:
     def _spec_ok(self, seqs: Sequence[SequenceMeta], cfg: SamplingMeta) -> bool:
         return (self.env.spec_ngram > 0 and not cfg.do_sample and cfg.num_beams == 1 and cfg.repetition_penalty == 1.0
                 and self.ctx.pp_size == 1 and self.ctx.dp_size == 1 and self.decoder.spec.rope != "2d"
+                and not self.cache.has_state             # rejected drafts cannot be taken back out of a state
                 and all(len(s.pending) == 1 and s.past_len > 0 for s in seqs))
 
     @staticmethod
@@ -752,6 +760,8 @@ class Model:
                   logit_rows=None if every else i32(rows).long() if dev.type == "cpu" else i32(rows),
                   is_decode=decode, max_q=max(cu[i + 1] - cu[i] for i in range(len(seqs))), max_kv=max(kvl))
         b.cu_q_dev, b.kv_lens_dev = i32(cu), i32(kvl)
+        if self.cache.has_state:
+            b.state_slots = i32(self.cache.state_slots([s.seq_id for s in seqs]))
         if self.decoder.spec.rope == "2d":
             self._chatglm_positions(b, seqs)
         return b

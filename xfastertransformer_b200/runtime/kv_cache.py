@@ -12,6 +12,10 @@ reorder and prefix sharing physically copy rows (``kvcache_tensor.h:146-289``,
   ``[num_blocks, 1, block, kv_lora+rope]``.
 * layered designs give every pool its own ``(kv_heads, k_dim, v_dim)``, ``v_dim`` 0 for a latent pool; a layer that reads another layer's keys and
   values has no pool at all (the decoder maps it to the pool it reads);
+* layers that keep a state instead of keys (gated linear attention, the last inputs of short convolutions) have one slot per
+  sequence in a pool ``[slots, ...]`` per layer run; a sequence has the same slot in all of them.  A slot is not cleared: the
+  kernels start from zero at a sequence's first token.  A state has no positions, so it cannot be cut back or adopted block
+  by block; a fork copies it;
 * a sequence is a list of block ids; blocks are reference-counted so a shared prefix or a beam
   fork is a table copy, and beam reorder is a permutation of tables (no data moves unless the
   partially filled tail block must be split — copy-on-write).
@@ -134,7 +138,8 @@ class PrefixIndex:
 class PagedKVCache:
     def __init__(self, num_layers: int, kv_heads: int, k_dim: int, v_dim: int, dtype: str, device: torch.device,
                  block_size: int = 64, act_dtype: torch.dtype = torch.bfloat16, latent: bool = False,
-                 geometry: Optional[Sequence[Tuple[int, int, int]]] = None, max_blocks: int = 0):
+                 geometry: Optional[Sequence[Tuple[int, int, int]]] = None, max_blocks: int = 0,
+                 states: Sequence[Tuple[Tuple[int, ...], torch.dtype]] = (), max_states: int = 0):
         # (kv heads, key size, value size) of every pool
         self.geometry = list(geometry) if geometry is not None else [(kv_heads, k_dim, v_dim)] * num_layers
         self.L = len(self.geometry)
@@ -163,6 +168,49 @@ class PagedKVCache:
         self.lens: Dict[int, int] = {}
         self.version = 0                         # bumped when pools are reallocated
         self.prefix_index: Optional[PrefixIndex] = None      # set by the engine when automatic prefix reuse is on
+        self.state_geometry = list(states)       # (shape of one slot, type) of every state pool
+        self.max_states = max_states             # > 0: the state pools never grow past this many slots
+        self.state: List[torch.Tensor] = []
+        self.state_alloc = BlockAllocator(0)
+        self.state_slot: Dict[int, int] = {}
+
+    # -- states ---------------------------------------------------------------------
+    @property
+    def has_state(self) -> bool:
+        return bool(self.state_geometry)
+
+    def ensure_states(self, total: int) -> None:
+        """Grow the state pools to `total` slots (contents preserved)."""
+        old = self.state_alloc.num_blocks
+        if not self.has_state or total <= old:
+            return
+        if self.max_states and total > self.max_states:
+            raise MemoryError(f"{total} state slots needed, the pools are limited to {self.max_states}")
+        pools = []
+        for i, (shape, dtype) in enumerate(self.state_geometry):
+            t = torch.zeros(total, *shape, dtype=dtype, device=self.device)
+            if old:
+                t[:old] = self.state[i]
+            pools.append(t)
+        self.state = pools
+        self.state_alloc.grow(total)
+        self.version += 1
+
+    def take_state(self) -> int:
+        """A free state slot."""
+        if not self.state_alloc.num_free:
+            n = self.state_alloc.num_blocks
+            grown = max(8, 2 * n)
+            self.ensure_states(max(n + 1, min(grown, self.max_states)) if self.max_states else grown)
+        return self.state_alloc.alloc()
+
+    def state_slots(self, seq_ids: Sequence[int]) -> List[int]:
+        return [self.state_slot[s] for s in seq_ids]
+
+    def _copy_states(self, src: Sequence[int], dst: Sequence[int]) -> None:
+        a, b = (torch.tensor(list(x), dtype=torch.long, device=self.device) for x in (src, dst))
+        for t in self.state:
+            t[b] = t[a]                          # the right side is gathered first
 
     # -- capacity -------------------------------------------------------------------
     def bytes_per_block(self) -> int:
@@ -229,6 +277,8 @@ class PagedKVCache:
     def add_sequence(self, seq_id: int, max_len: int = 0) -> None:
         if seq_id in self.tables:
             raise KeyError(f"sequence {seq_id} already in the cache")
+        if self.has_state:
+            self.state_slot[seq_id] = self.take_state()
         self.tables[seq_id] = []
         self.lens[seq_id] = 0
         if max_len:
@@ -238,18 +288,24 @@ class PagedKVCache:
         for b in self.tables.pop(seq_id, []):
             self.alloc.release(b)
         self.lens.pop(seq_id, None)
+        if seq_id in self.state_slot:
+            self.state_alloc.release(self.state_slot.pop(seq_id))
 
     def adopt(self, seq_id: int, blocks: Sequence[int]) -> int:
         """Start a fresh sequence on shared, full blocks (automatic prefix reuse); returns the tokens they hold."""
         assert not self.tables[seq_id], "adopt() is for a sequence that holds nothing yet"
+        assert not self.has_state, "blocks without the state behind them"
         self.tables[seq_id] = [self.alloc.share(b) for b in blocks]
         self.lens[seq_id] = len(blocks) * self.block
         return self.lens[seq_id]
 
     def fork(self, src: int, dst: int) -> None:
-        """dst shares all of src's blocks (prefix sharing, beam expansion)."""
+        """dst shares all of src's blocks (prefix sharing, beam expansion) and gets a copy of its state."""
         if dst in self.tables:
             self.free_sequence(dst)
+        if self.has_state:
+            self.state_slot[dst] = self.take_state()
+            self._copy_states([self.state_slot[src]], [self.state_slot[dst]])
         self.tables[dst] = [self.alloc.share(b) for b in self.tables[src]]
         self.lens[dst] = self.lens[src]
 
@@ -276,6 +332,8 @@ class PagedKVCache:
         return slots
 
     def truncate(self, seq_id: int, new_len: int) -> None:
+        if self.has_state and 0 < new_len < self.lens[seq_id]:
+            raise RuntimeError(f"sequence {seq_id}: its recurrent state cannot go back from {self.lens[seq_id]} to {new_len} tokens")
         tab = self.tables[seq_id]
         keep = self.blocks_for(new_len)
         for b in tab[keep:]:
@@ -298,6 +356,10 @@ class PagedKVCache:
         for i, s in enumerate(seq_ids):
             self.tables[s] = new[s]
             self.lens[s] = old_lens[seq_ids[src_index[i]]]
+        moved = [(self.state_slot[seq_ids[j]], self.state_slot[s]) for s, j in zip(seq_ids, src_index) if seq_ids[j] != s] \
+            if self.has_state else []
+        if moved:
+            self._copy_states(*zip(*moved))
 
     def _copy_block(self, src: int, dst: int) -> None:
         for l in range(self.L):

@@ -395,6 +395,14 @@ class SafetensorsSource(WeightSource):
     def exists(self, name: str) -> bool:
         return False if self.fake else name in self.file
 
+    def shape(self, name: str, default: Sequence[int]) -> Tuple[int, ...]:
+        """A tensor's shape, for sizes that only the file knows (`default` in fake mode)."""
+        if self.fake:
+            return tuple(default)
+        if name not in self.file:
+            raise KeyError(f"{self.file.path}: no tensor {name}")
+        return tuple(self.file.entries[name]["shape"])
+
     def _take(self, name, shape, rows=None, cols=None) -> torch.Tensor:
         t = self.file.read(name, shape, rows, cols)
         self.loaded_bytes += t.numel() * t.element_size()

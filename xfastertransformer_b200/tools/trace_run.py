@@ -12,7 +12,7 @@ no file).  The cache blocks of the requests in ``end`` are freed once the step h
 
 The tool is a thin client of the continuous-batching API: a request's first entry is admitted with `set_input_cb`, later
 ones continue it (`extend=True`), `forward_cb` runs the step, `free_seqs` ends requests.  Nothing is sampled.  The KV pools
-are made once for ``--max-tokens`` tokens.
+are made once for ``--max-tokens`` tokens, pools of recurrent states for MAX_SEQUENCES requests.
 """
 from __future__ import annotations
 
@@ -22,18 +22,20 @@ import os
 import sys
 from typing import Dict
 
+MAX_SEQUENCES = 4                 # live requests a trace may hold
 DTYPES = {"bfloat16": "bf16", "float32": "fp32"}
 
 
 class TraceRunner:
-    def __init__(self, path: str, dtype: str, max_tokens: int):
+    def __init__(self, path: str, dtype: str, max_tokens: int, max_sequences: int = MAX_SEQUENCES):
         import torch
 
         from ..automodel import AutoModel
         from ..utils.flags import Env
         if not torch.cuda.is_available() and not Env.get().engine.upper().startswith("CPU"):
             raise RuntimeError("no CUDA device (XFT_ENGINE=CPU runs the PyTorch path)")
-        self.model = AutoModel.from_pretrained(path, dtype=dtype, kv_cache_dtype="bf16", max_cache_tokens=max_tokens)
+        self.model = AutoModel.from_pretrained(path, dtype=dtype, kv_cache_dtype="bf16", max_cache_tokens=max_tokens,
+                                               max_sequences=max_sequences)
         self.ids: Dict[str, int] = {}
 
     def step(self, entries, end=()):
