@@ -42,8 +42,14 @@ __device__ __forceinline__ void ll_unpack2(unsigned w, float& lo, float& hi) {
   lo = f.x; hi = f.y;
 }
 
+// An activation code with this bit set: the residual operand multiplies the activated value instead of being added to it.
+constexpr int kActTimes = 16;
+__device__ __forceinline__ float with_residual(float x, float r, float scale, int act) {
+  return act & kActTimes ? x * r : x + scale * r;
+}
+
 __device__ __forceinline__ float apply_act(float x, int act) {
-  switch (act) {
+  switch (act & (kActTimes - 1)) {
     case 1: return fmaxf(x, 0.f);
     case 4: { const float r = fmaxf(x, 0.f); return r * r; }
     case 2: return x / (1.f + __expf(-x));

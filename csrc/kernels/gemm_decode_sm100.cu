@@ -175,7 +175,7 @@ __global__ void __launch_bounds__(192, 2) gemm_sk_kernel(const __grid_constant__
     const float ts = rms ? rsqrtf(ssq / (float)p.K + p.rms_eps) : 1.f;
     float x = apply_act(g * (rs * ts) + (p.bias ? p.bias[n] : 0.f), p.act);
     if constexpr (DUAL) x *= (u * (rs * ts) + (p.bias ? p.bias[p.dual_off + n] : 0.f));
-    if (p.residual) x += p.res_scale * __bfloat162float(p.residual[(size_t)t * p.ldr + n]);
+    if (p.residual) x = with_residual(x, __bfloat162float(p.residual[(size_t)t * p.ldr + n]), p.res_scale, p.act);
     if (p.out_fp32) reinterpret_cast<float*>(p.out)[(size_t)t * p.ldo + n] = x;
     else reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)t * p.ldo + n] = __float2bfloat16(x);
   };
@@ -305,7 +305,7 @@ auto ar_reduce = [&]() {
         const int nn = n + (k >> 1), tt = t + (k & 1);
         float x = f[k] + (p.bias ? p.bias[nn] : 0.f);
         x = apply_act(x, p.act);
-        if (p.residual && tt < p.T) x += p.res_scale * __bfloat162float(p.residual[(size_t)tt * p.ldr + nn]);
+        if (p.residual && tt < p.T) x = with_residual(x, __bfloat162float(p.residual[(size_t)tt * p.ldr + nn]), p.res_scale, p.act);
         f[k] = x;
       }
       if (p.ar.two_shot) {

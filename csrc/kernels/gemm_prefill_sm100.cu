@@ -67,8 +67,14 @@ struct PrefillParams {
   BulkArParams ar;
 };
 
+// An activation code with this bit set: the residual operand multiplies the activated value instead of being added to it.
+constexpr int kPrefillTimes = 16;
+__device__ __forceinline__ float prefill_residual(float x, float r, float scale, int act) {
+  return act & kPrefillTimes ? x * r : x + scale * r;
+}
+
 __device__ __forceinline__ float prefill_act(float x, int act) {
-  switch (act) {
+  switch (act & (kPrefillTimes - 1)) {
     case 1: return fmaxf(x, 0.f);
     case 4: { const float r = fmaxf(x, 0.f); return r * r; }
     case 2: return x / (1.f + __expf(-x));
@@ -351,7 +357,7 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_kernel(const __grid_const
           if (t < p.T) {
             float y = prefill_act(x[j] + bias, p.act);
             if constexpr (DUAL) y *= __uint_as_float(vu[j]) + bias_u;
-            if (p.residual) y += p.res_scale * __bfloat162float(p.residual[(size_t)t * p.ldr + n]);
+            if (p.residual) y = prefill_residual(y, __bfloat162float(p.residual[(size_t)t * p.ldr + n]), p.res_scale, p.act);
             const __nv_bfloat16 yb = __float2bfloat16(y);
             if (wide) {
               s_stage[j * kStageLd + row] = yb;
@@ -628,8 +634,10 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_tm_kernel(const __grid_co
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
               const float2 f0 = __bfloat1622float2(h0[j]), f1 = __bfloat1622float2(h1[j]);
-              x[2 * j] += p.res_scale * f0.x; x[2 * j + 1] += p.res_scale * f0.y;
-              x[8 + 2 * j] += p.res_scale * f1.x; x[8 + 2 * j + 1] += p.res_scale * f1.y;
+              x[2 * j] = prefill_residual(x[2 * j], f0.x, p.res_scale, p.act);
+              x[2 * j + 1] = prefill_residual(x[2 * j + 1], f0.y, p.res_scale, p.act);
+              x[8 + 2 * j] = prefill_residual(x[8 + 2 * j], f1.x, p.res_scale, p.act);
+              x[8 + 2 * j + 1] = prefill_residual(x[8 + 2 * j + 1], f1.y, p.res_scale, p.act);
             }
           }
           uint32_t w[8];
@@ -645,7 +653,7 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_tm_kernel(const __grid_co
           for (int j = 0; j < 16; ++j) {
             if (n0 + j < p.N) {
               float y = x[j];
-              if (rrow) y += p.res_scale * __bfloat162float(rrow[n0 + j]);
+              if (rrow) y = prefill_residual(y, __bfloat162float(rrow[n0 + j]), p.res_scale, p.act);
               orow[n0 + j] = __float2bfloat16(y);
             }
           }

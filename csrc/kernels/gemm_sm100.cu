@@ -429,7 +429,7 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
                   if (DUAL && !pair) x *= (u[j] * (rs * ts) + bias_u);
                   if (p.col_scale) x *= p.col_scale[t];
                   if (p.gate) x = __fdividef(x, 1.f + __expf(-__bfloat162float(gt[j])));
-                  if (p.residual) x += p.res_scale * __bfloat162float(p.residual[(size_t)t * p.ldr + n]);
+                  if (p.residual) x = with_residual(x, __bfloat162float(p.residual[(size_t)t * p.ldr + n]), p.res_scale, p.act);
                   g[j] = x;                     // kept for the two-shot broadcast below
                 }
                 if (p.out_fp32) reinterpret_cast<float*>(p.out)[(size_t)t * p.ldo + y_col0 + n] = x;
@@ -458,7 +458,7 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
               if (t < p.T && c + j < x_rows) {
                 float x = apply_act(u[j] + bias_u, p.act);
                 if (p.col_scale) x *= p.col_scale[t];
-                if (p.residual) x += p.res_scale * __bfloat162float(p.residual[(size_t)t * p.ldr + n2]);
+                if (p.residual) x = with_residual(x, __bfloat162float(p.residual[(size_t)t * p.ldr + n2]), p.res_scale, p.act);
                 if (p.out_fp32) reinterpret_cast<float*>(p.out)[(size_t)t * p.ldo + n2] = x;
                 else reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)t * p.ldo + n2] = __float2bfloat16(x);
               }

@@ -1,0 +1,753 @@
+// Gated linear attention: a recurrent layer whose state per head is a dim x vdim matrix that decays per key channel.
+//
+//   alpha_t = sigmoid(W_a2 a1_t + bias)^(1 / tau)         [dim]
+//   S_t = diag(alpha_t) S_(t-1) + k_t v_t^T                fp32
+//   o_t = S_t^T (q_t / sqrt(dim))                          [vdim]
+//   out = o / sqrt(mean(o^2) + eps) * gain * silu(g_t)
+//
+// Rows of x are packed [q | k | v | g | a1] (queries, keys, values and gate of all heads, the decay's first product).  A
+// sequence's state lives in its slot of a pool [slots, heads, dim, vdim]; its first token starts from zero whatever the slot
+// holds.  Two kernels share a batch, by the length of a sequence's portion:
+//
+// gla_step_kernel (decode, short portions, and everything in fp32): token after token.  The state of a (sequence, head)
+// stays in registers, spread over one CTA or, by columns, over a cluster of up to 8 that exchange the norm's sum of squares
+// through distributed shared memory.  A decode step is bound by reading and writing the state once; the state is fetched
+// before the kernel in front has finished.
+//
+// gla_chunk_kernel (bf16 portions): 64 tokens at a time on the tensor cores.  With b_t the running sum of log(alpha) within
+// the chunk (fp32), its last value b_C and mid = b_C / 2 per channel,
+//
+//   q^_t = q_t exp(b_t - mid),  k^_t = k_t exp(mid - b_t)
+//   O   = q^ (exp(mid) S) + tril(q^ k^^T) V
+//   S  <- exp(mid) (exp(mid) S + k^^T V)
+//
+// which is exact algebra; the exponents stay within +-30 as long as no channel decays by more than e^-60 in a chunk.  A
+// chunk with a faster channel goes in four pieces of 16 tokens, and a piece with such a channel forms its 16 x 16 scores
+// from differences b_t - b_s <= 0, which cannot overflow.  S stays in registers as the accumulator of its product.
+//
+// This file is compiled without fast-math; the chunk kernel asks for the fast exponential and logarithm by name.
+#include "ptx.cuh"
+
+namespace xft {
+
+typedef __nv_bfloat16 bf16;
+
+struct GlaParams {
+  const void* x; int ldx; int k_at, v_at, g_at, a_at;
+  int heads, dim, vdim, rank, rank_ld;     // rank_ld: row stride of a2
+  const void* a2; const float* bias;       // [heads * dim, rank_ld], [heads * dim]
+  float inv_tau, scale, eps;
+  const float* gain;                       // [vdim]
+  float* state; const int* state_slots; int num_states;
+  const int* cu_q; const int* kv_lens; int B;
+  void* out; int ldo;                      // [T, heads * vdim]
+  float* raw;                              // chunk kernel with split columns: o before its norm, fp32 [T, heads * vdim]
+  int min_q, max_q;                        // only sequences with min_q <= tokens in this call < max_q
+  int* status;
+};
+
+template <typename T> __device__ __forceinline__ float gl_f32(T v);
+template <> __device__ __forceinline__ float gl_f32<float>(float v) { return v; }
+template <> __device__ __forceinline__ float gl_f32<bf16>(bf16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T gl_from(float v);
+template <> __device__ __forceinline__ float gl_from<float>(float v) { return v; }
+template <> __device__ __forceinline__ bf16 gl_from<bf16>(float v) { return __float2bfloat16(v); }
+
+__device__ __forceinline__ int gl_slot(const GlaParams& p, int b) {
+  int s = p.state_slots[b];
+  if (s < 0 || s >= p.num_states) { if (threadIdx.x == 0 && p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); s = 0; }
+  return s;
+}
+
+// ------------------------------------------------------------------------------------------ token by token
+constexpr int kStepThreads = 256;
+
+// LC lanes share a row of the state (4 columns each), RPT rows per thread
+template <typename T, int LC, int RPT>
+__global__ void __launch_bounds__(kStepThreads) gla_step_kernel(const GlaParams p) {
+  constexpr int CW = LC * 4, GROUPS = kStepThreads / LC, NW = kStepThreads / 32;
+  extern __shared__ float gs_sm[];
+  float* sq = gs_sm;                       // [dim] each
+  float* sk = sq + p.dim;
+  float* sa = sk + p.dim;
+  float* sr = sa + p.dim;                  // [rank_ld]
+  __shared__ float red[NW][CW];
+  __shared__ float ssq[2][NW];
+  __shared__ float peer_ss[2];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int h = blockIdx.y, b = blockIdx.z, slice = blockIdx.x, nslices = gridDim.x;
+  grid_dep_launch();
+  const int start = p.cu_q[b], n = p.cu_q[b + 1] - start;
+  if (n < p.min_q || n >= p.max_q) { grid_dep_wait(); return; }
+  const int past = p.kv_lens[b] - n;
+  const int lc = tid % LC, grp = tid / LC;
+  const int c0 = slice * CW + lc * 4;                     // this thread's columns c0 .. c0 + 3
+  const bool vec = (p.vdim & 3) == 0;
+  float* st = p.state + ((size_t)gl_slot(p, b) * p.heads + h) * p.dim * p.vdim;
+  float S[RPT][4];
+#pragma unroll
+  for (int r = 0; r < RPT; ++r) {
+    const int d = r * GROUPS + grp;
+    S[r][0] = S[r][1] = S[r][2] = S[r][3] = 0.f;
+    if (past > 0 && d < p.dim) {
+      const float* row = st + (size_t)d * p.vdim + c0;
+      if (vec && c0 < p.vdim) {
+        const float4 v = *reinterpret_cast<const float4*>(row);
+        S[r][0] = v.x; S[r][1] = v.y; S[r][2] = v.z; S[r][3] = v.w;
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) if (c0 + j < p.vdim) S[r][j] = row[j];
+      }
+    }
+  }
+  grid_dep_wait();
+  const T* a2 = reinterpret_cast<const T*>(p.a2) + (size_t)h * p.dim * p.rank_ld;
+  for (int i = 0; i < n; ++i) {
+    const T* row = reinterpret_cast<const T*>(p.x) + (size_t)(start + i) * p.ldx;
+    for (int r = tid; r < p.rank_ld; r += kStepThreads) sr[r] = r < p.rank ? gl_f32<T>(row[p.a_at + r]) : 0.f;
+    float v[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) v[j] = c0 + j < p.vdim ? gl_f32<T>(row[p.v_at + h * p.vdim + c0 + j]) : 0.f;
+    __syncthreads();
+    for (int d = tid; d < p.dim; d += kStepThreads) {
+      float z = p.bias[h * p.dim + d];
+      const T* wr = a2 + (size_t)d * p.rank_ld;
+      for (int r = 0; r < p.rank_ld; r += 8) {            // rows of a2 are multiples of 8 values, zeros behind the rank
+        struct alignas(16) V8 { T e[8]; };
+        const V8 w = *reinterpret_cast<const V8*>(wr + r);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) z = fmaf(gl_f32<T>(w.e[e]), sr[r + e], z);
+      }
+      const float la = (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * p.inv_tau;      // log(sigmoid(z)) / tau
+      sa[d] = expf(la);
+      sq[d] = gl_f32<T>(row[h * p.dim + d]) * p.scale;
+      sk[d] = gl_f32<T>(row[p.k_at + h * p.dim + d]);
+    }
+    __syncthreads();
+    float o[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int r = 0; r < RPT; ++r) {
+      const int d = r * GROUPS + grp;
+      if (d < p.dim) {
+        const float al = sa[d], kk = sk[d], qq = sq[d];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          S[r][j] = fmaf(al, S[r][j], kk * v[j]);
+          o[j] = fmaf(qq, S[r][j], o[j]);
+        }
+      }
+    }
+#pragma unroll
+    for (int m = LC; m < 32; m <<= 1)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) o[j] += __shfl_xor_sync(0xffffffffu, o[j], m);
+    if (lane < LC) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) red[warp][lc * 4 + j] = o[j];
+    }
+    __syncthreads();
+    float y = 0.f;
+    const int col = slice * CW + tid;
+    const bool mine = tid < CW && col < p.vdim;
+    if (tid < CW) {
+#pragma unroll
+      for (int w = 0; w < NW; ++w) y += red[w][tid];
+    }
+    float ss = mine ? y * y : 0.f;
+#pragma unroll
+    for (int m = 16; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+    if (lane == 0) ssq[i & 1][warp] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int w = 0; w < NW; ++w) ss += ssq[i & 1][w];
+    if (nslices > 1) {                                    // the other columns of the head are with the cluster's other CTAs
+      if (tid == 0) peer_ss[i & 1] = ss;
+      cluster_arrive();
+      cluster_wait();
+      ss = 0.f;
+      for (int c = 0; c < nslices; ++c) ss += ld_dsmem(dsmem_addr(smem_u32(&peer_ss[i & 1]), c));
+    }
+    if (mine) {
+      const float g = gl_f32<T>(row[p.g_at + h * p.vdim + col]);
+      const float r = y / sqrtf(ss / (float)p.vdim + p.eps) * p.gain[col] * (g / (1.f + expf(-g)));
+      reinterpret_cast<T*>(p.out)[(size_t)(start + i) * p.ldo + h * p.vdim + col] = gl_from<T>(r);
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < RPT; ++r) {
+    const int d = r * GROUPS + grp;
+    if (d < p.dim) {
+      float* row = st + (size_t)d * p.vdim + c0;
+      if (vec && c0 < p.vdim) *reinterpret_cast<float4*>(row) = make_float4(S[r][0], S[r][1], S[r][2], S[r][3]);
+      else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) if (c0 + j < p.vdim) row[j] = S[r][j];
+      }
+    }
+  }
+  if (nslices > 1) { cluster_arrive(); cluster_wait(); }  // nobody leaves while its shared memory may be read
+}
+
+// ------------------------------------------------------------------------------------------ chunks of 64 tokens
+__device__ __forceinline__ void gl_ldsm(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void gl_ldsm_t(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void gl_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t gl_pack(float lo, float hi) {
+  const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
+__device__ __forceinline__ float2 gl_unpack(uint32_t v) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v)); }
+
+constexpr int kChunk = 64, kPiece = 16;
+constexpr float kMaxDecay = 60.f;
+
+// DP: padded dim, VS: columns of the state per CTA, RP: padded rank
+template <int DP, int VS, int RP>
+struct ChunkCfg {
+  static constexpr int QS = DP + 8, VSS = VS + 8, RS = RP + 8, AS = kChunk + 8;     // row strides (16 bytes of padding)
+  static constexpr int STAGE = kChunk * (2 * QS + VSS + RS);                         // q, k, v, a1 of a chunk, in values
+  static constexpr int STAGES = DP <= 128 ? 2 : 1;
+  static constexpr size_t B16 = (size_t)STAGES * STAGE + kChunk * AS + DP * VSS + DP * RS;
+  static constexpr size_t F32 = (size_t)kChunk * DP + 4 * DP + 3 * DP + DP + 2 * kChunk;
+  static constexpr size_t SMEM = B16 * 2 + F32 * 4;
+};
+
+template <int DP, int VS, int RP>
+__global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
+  using Cfg = ChunkCfg<DP, VS, RP>;
+  constexpr int QS = Cfg::QS, VSS = Cfg::VSS, RS = Cfg::RS, AS = Cfg::AS;
+  constexpr int MW = DP / 16, MPW = MW >= 8 ? MW / 8 : 1, NGRP = MW >= 8 ? 1 : 8 / MW, NPW = VS / 8 / NGRP;
+  extern __shared__ __align__(16) uint8_t gc_raw[];
+  bf16* stage0 = reinterpret_cast<bf16*>(gc_raw);
+  bf16* sA = stage0 + Cfg::STAGES * Cfg::STAGE;           // scores [64][AS]
+  bf16* sS = sA + kChunk * AS;                            // state as an operand [DP][VSS]
+  bf16* sW = sS + DP * VSS;                               // a2 of this head [DP][RS]
+  float* sB = reinterpret_cast<float*>(sW + DP * RS);     // running sums of log(alpha) [64][DP], restarting every 16 rows
+  float* sT = sB + kChunk * DP;                           // their totals [4][DP]
+  float* sPre = sT + 4 * DP;                              // factors of the state's rows: in front of the operand,
+  float* sMid = sPre + DP;                                //   behind it,
+  float* sPost = sMid + DP;                               //   and behind the update
+  float* sBias = sPost + DP;
+  float* sSS = sBias + DP;                                // [2][64] sums of squares of the output rows
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int h = blockIdx.y, b = blockIdx.z, v0 = blockIdx.x * VS;
+  grid_dep_launch();
+  const int start = p.cu_q[b], n = p.cu_q[b + 1] - start;
+  if (n < p.min_q || n >= p.max_q) { grid_dep_wait(); return; }
+  const int past = p.kv_lens[b] - n;
+  const int vw = min(VS, p.vdim - v0);
+  const bool whole8 = (p.dim & 7) == 0 && (p.vdim & 7) == 0 && (p.rank & 7) == 0;
+  float* st = p.state + ((size_t)gl_slot(p, b) * p.heads + h) * p.dim * p.vdim;
+  const bf16* a2 = reinterpret_cast<const bf16*>(p.a2) + (size_t)h * p.dim * p.rank_ld;
+
+  // weights, and zeros where nothing is ever loaded
+  for (int i = tid; i < Cfg::STAGES * Cfg::STAGE / 8; i += 256) reinterpret_cast<uint4*>(stage0)[i] = make_uint4(0, 0, 0, 0);
+  for (int i = tid; i < DP * RP; i += 256) {
+    const int d = i / RP, r = i % RP;
+    sW[d * RS + r] = d < p.dim && r < p.rank ? a2[(size_t)d * p.rank_ld + r] : __float2bfloat16(0.f);
+  }
+  for (int d = tid; d < DP; d += 256) sBias[d] = d < p.dim ? p.bias[h * p.dim + d] : 0.f;
+  // the state: warp tile of MPW x 16 rows and NPW x 8 columns
+  const int sm0 = (MW >= 8 ? warp * MPW : warp % MW) * 16, sn0 = (MW >= 8 ? 0 : warp / MW) * NPW * 8;
+  float S[MPW][NPW][4];
+#pragma unroll
+  for (int m = 0; m < MPW; ++m)
+#pragma unroll
+    for (int j = 0; j < NPW; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int d = sm0 + m * 16 + (lane >> 2) + (e >> 1) * 8, c = sn0 + j * 8 + 2 * (lane & 3) + (e & 1);
+        S[m][j][e] = past > 0 && d < p.dim && c < vw ? st[(size_t)d * p.vdim + v0 + c] : 0.f;
+      }
+  grid_dep_wait();
+  __syncthreads();
+
+  const bf16* x = reinterpret_cast<const bf16*>(p.x) + (size_t)start * p.ldx;
+  auto load = [&](int chunk) {
+    bf16* sq = stage0 + (Cfg::STAGES > 1 ? (chunk & 1) * Cfg::STAGE : 0);
+    bf16* sk = sq + kChunk * QS;
+    bf16* sv = sk + kChunk * QS;
+    bf16* sr = sv + kChunk * VSS;
+    const int t0 = chunk * kChunk, rows = min(kChunk, n - t0);
+    // rows behind the portion's end become zero
+    auto part = [&](bf16* dst, int ld, int at, int width) {
+      if (whole8) {
+        const int per = width >> 3;
+        for (int i = tid; i < kChunk * per; i += 256) {
+          const int r = i / per, c = (i % per) * 8;
+          const bf16* src = x + (size_t)(t0 + min(r, rows - 1)) * p.ldx + at + c;
+          const int bytes = r < rows ? 16 : 0;
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + r * ld + c)), "l"(src), "r"(bytes) : "memory");
+        }
+      } else {
+        for (int i = tid; i < kChunk * width; i += 256) {
+          const int r = i / width, c = i % width;
+          dst[r * ld + c] = r < rows ? x[(size_t)(t0 + r) * p.ldx + at + c] : __float2bfloat16(0.f);
+        }
+      }
+    };
+    part(sq, QS, h * p.dim, p.dim);
+    part(sk, QS, p.k_at + h * p.dim, p.dim);
+    part(sv, VSS, p.v_at + h * p.vdim + v0, vw);
+    part(sr, RS, p.a_at, p.rank);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  const int chunks = (n + kChunk - 1) / kChunk;
+  load(0);
+  for (int ch = 0; ch < chunks; ++ch) {
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    if (Cfg::STAGES > 1 && ch + 1 < chunks) load(ch + 1);
+    bf16* sq = stage0 + (Cfg::STAGES > 1 ? (ch & 1) * Cfg::STAGE : 0);
+    bf16* sk = sq + kChunk * QS;
+    bf16* sv = sk + kChunk * QS;
+    bf16* sr = sv + kChunk * VSS;
+    const int rows = min(kChunk, n - ch * kChunk);
+    const int mt = warp & 3, half = warp >> 2;            // this warp's 16 rows of the chunk, and half of the columns
+
+    // log(alpha) of every row and channel
+    {
+      float z[DP / 16][4];
+#pragma unroll
+      for (int j = 0; j < DP / 16; ++j) z[j][0] = z[j][1] = z[j][2] = z[j][3] = 0.f;
+#pragma unroll
+      for (int ks = 0; ks < RP / 16; ++ks) {
+        uint32_t a[4];
+        gl_ldsm(a, sr + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * RS + ks * 16 + (lane >> 4) * 8);
+#pragma unroll
+        for (int j = 0; j < DP / 16; j += 2) {
+          uint32_t w[4];
+          gl_ldsm(w, sW + (half * (DP / 2) + j * 8 + (lane & 7) + ((lane >> 4) & 1) * 8) * RS + ks * 16 + ((lane >> 3) & 1) * 8);
+          gl_mma(z[j], a, w[0], w[1]);
+          if (j + 1 < DP / 16) gl_mma(z[j + 1 < DP / 16 ? j + 1 : j], a, w[2], w[3]);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < DP / 16; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+          const int r = mt * 16 + (lane >> 2) + (e >> 1) * 8, d = half * (DP / 2) + j * 8 + 2 * (lane & 3);
+          float2 la;
+          float* l = &la.x;
+#pragma unroll
+          for (int k = 0; k < 2; ++k) {
+            const float zz = z[j][e + k] + sBias[d + k];
+            l[k] = r < rows && d + k < p.dim ? (fminf(zz, 0.f) - __logf(1.f + __expf(-fabsf(zz)))) * p.inv_tau : 0.f;
+          }
+          *reinterpret_cast<float2*>(sB + r * DP + d) = la;
+        }
+    }
+    __syncthreads();
+    // running sums within every 16 rows, and their totals
+    for (int it = tid; it < 2 * DP; it += 256) {
+      const int pr = it % (DP / 2), g = it / (DP / 2);
+      float2 c = make_float2(0.f, 0.f);
+      float2 v[kPiece];
+#pragma unroll
+      for (int r = 0; r < kPiece; ++r) v[r] = *reinterpret_cast<const float2*>(sB + (g * kPiece + r) * DP + 2 * pr);
+#pragma unroll
+      for (int r = 0; r < kPiece; ++r) {
+        c.x += v[r].x; c.y += v[r].y;
+        *reinterpret_cast<float2*>(sB + (g * kPiece + r) * DP + 2 * pr) = c;
+      }
+      *reinterpret_cast<float2*>(sT + g * DP + 2 * pr) = c;
+    }
+    __syncthreads();
+    bool ok = true;
+    for (int d = tid; d < DP; d += 256) ok = ok && sT[d] + sT[DP + d] + sT[2 * DP + d] + sT[3 * DP + d] >= -kMaxDecay;
+    const bool one = __syncthreads_and(ok);               // the whole chunk in one piece
+    const int pieces = one ? 1 : (rows + kPiece - 1) / kPiece;
+    float O[VS / 16][4];
+#pragma unroll
+    for (int j = 0; j < VS / 16; ++j) O[j][0] = O[j][1] = O[j][2] = O[j][3] = 0.f;
+    for (int pc = 0; pc < pieces; ++pc) {
+      const int g_lo = one ? 0 : pc, g_hi = one ? 4 : pc + 1;       // groups of 16 rows in this piece
+      bool gentle = true;
+      if (!one) {
+        bool k = true;
+        for (int d = tid; d < DP; d += 256) k = k && sT[pc * DP + d] >= -kMaxDecay;
+        gentle = __syncthreads_and(k);
+        if (!gentle) {
+          // scores of the piece from differences of running sums; 256 pairs of rows, a warp at a time
+          for (int i = warp; i < kPiece * kPiece; i += 8) {
+            const int t = pc * kPiece + i / kPiece, s = pc * kPiece + i % kPiece;
+            float a = 0.f;
+            if (s <= t)
+              for (int d = lane; d < p.dim; d += 32)
+                a += __bfloat162float(sq[t * QS + d]) * __bfloat162float(sk[s * QS + d]) * __expf(sB[t * DP + d] - sB[s * DP + d]);
+#pragma unroll
+            for (int m = 16; m > 0; m >>= 1) a += __shfl_xor_sync(0xffffffffu, a, m);
+            if (lane == 0) sA[t * AS + s] = __float2bfloat16(a * p.scale);
+          }
+          __syncthreads();
+        }
+      }
+      // q^ and k^ in place; the factors of the state's rows
+      for (int it = tid; it < 2 * DP; it += 256) {
+        const int pr = it % (DP / 2), g = it / (DP / 2);
+        if (g < g_lo || g >= g_hi) continue;
+        float2 base = make_float2(0.f, 0.f), tot = make_float2(0.f, 0.f);
+        for (int j = g_lo; j < g_hi; ++j) {
+          const float2 v = *reinterpret_cast<const float2*>(sT + j * DP + 2 * pr);
+          if (j < g) { base.x += v.x; base.y += v.y; }
+          tot.x += v.x; tot.y += v.y;
+        }
+        // q^ = q exp(b - qr), k^ = k exp(kr - b)
+        const float2 qr = gentle ? make_float2(0.5f * tot.x, 0.5f * tot.y) : make_float2(0.f, 0.f);
+        const float2 kr = gentle ? qr : tot;
+        if (g == g_lo) {
+          const float2 e = make_float2(__expf(qr.x), __expf(qr.y));
+          *reinterpret_cast<float2*>(sPre + 2 * pr) = e;
+          *reinterpret_cast<float2*>(sMid + 2 * pr) = gentle ? make_float2(1.f, 1.f) : make_float2(__expf(tot.x), __expf(tot.y));
+          *reinterpret_cast<float2*>(sPost + 2 * pr) = e;
+        }
+#pragma unroll
+        for (int r = 0; r < kPiece; ++r) {
+          const int t = g * kPiece + r;
+          float2 bb = *reinterpret_cast<const float2*>(sB + t * DP + 2 * pr);
+          bb.x += base.x; bb.y += base.y;
+          uint32_t* qp = reinterpret_cast<uint32_t*>(sq + t * QS + 2 * pr);
+          uint32_t* kp = reinterpret_cast<uint32_t*>(sk + t * QS + 2 * pr);
+          const float2 q = gl_unpack(*qp), k = gl_unpack(*kp);
+          *qp = gl_pack(q.x * p.scale * __expf(bb.x - qr.x), q.y * p.scale * __expf(bb.y - qr.y));
+          *kp = gl_pack(k.x * __expf(kr.x - bb.x), k.y * __expf(kr.y - bb.y));
+        }
+      }
+      __syncthreads();
+      // the state as an operand, and the scores
+#pragma unroll
+      for (int m = 0; m < MPW; ++m) {
+        const int d = sm0 + m * 16 + (lane >> 2);
+        const float f0 = sPre[d], f1 = sPre[d + 8], m0 = sMid[d], m1 = sMid[d + 8];
+#pragma unroll
+        for (int j = 0; j < NPW; ++j) {
+          const int c = sn0 + j * 8 + 2 * (lane & 3);
+          S[m][j][0] *= f0; S[m][j][1] *= f0; S[m][j][2] *= f1; S[m][j][3] *= f1;
+          *reinterpret_cast<uint32_t*>(sS + d * VSS + c) = gl_pack(S[m][j][0], S[m][j][1]);
+          *reinterpret_cast<uint32_t*>(sS + (d + 8) * VSS + c) = gl_pack(S[m][j][2], S[m][j][3]);
+          if (!gentle) { S[m][j][0] *= m0; S[m][j][1] *= m0; S[m][j][2] *= m1; S[m][j][3] *= m1; }
+        }
+      }
+      const bool my_rows = mt >= g_lo && mt < g_hi;
+      if (gentle && my_rows) {
+        // columns of this warp: of the whole chunk its half (32), of a piece 8 of its 16
+        if (one) {
+          float A[4][4];
+#pragma unroll
+          for (int j = 0; j < 4; ++j) A[j][0] = A[j][1] = A[j][2] = A[j][3] = 0.f;
+          const int n0 = half * 32;
+          if (n0 <= mt * 16 + 15) {
+#pragma unroll
+            for (int ks = 0; ks < DP / 16; ++ks) {
+              uint32_t a[4];
+              gl_ldsm(a, sq + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * QS + ks * 16 + (lane >> 4) * 8);
+#pragma unroll
+              for (int j = 0; j < 4; j += 2) {
+                uint32_t w[4];
+                gl_ldsm(w, sk + (n0 + j * 8 + (lane & 7) + ((lane >> 4) & 1) * 8) * QS + ks * 16 + ((lane >> 3) & 1) * 8);
+                gl_mma(A[j], a, w[0], w[1]);
+                gl_mma(A[j + 1], a, w[2], w[3]);
+              }
+            }
+          }
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; e += 2) {
+              const int t = mt * 16 + (lane >> 2) + (e >> 1) * 8, s = n0 + j * 8 + 2 * (lane & 3);
+              *reinterpret_cast<uint32_t*>(sA + t * AS + s) = gl_pack(s <= t ? A[j][e] : 0.f, s + 1 <= t ? A[j][e + 1] : 0.f);
+            }
+        } else if (half == 0) {
+          float A[2][4];
+#pragma unroll
+          for (int j = 0; j < 2; ++j) A[j][0] = A[j][1] = A[j][2] = A[j][3] = 0.f;
+#pragma unroll
+          for (int ks = 0; ks < DP / 16; ++ks) {
+            uint32_t a[4], w[4];
+            gl_ldsm(a, sq + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * QS + ks * 16 + (lane >> 4) * 8);
+            gl_ldsm(w, sk + (mt * 16 + (lane & 7) + ((lane >> 4) & 1) * 8) * QS + ks * 16 + ((lane >> 3) & 1) * 8);
+            gl_mma(A[0], a, w[0], w[1]);
+            gl_mma(A[1], a, w[2], w[3]);
+          }
+#pragma unroll
+          for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; e += 2) {
+              const int t = mt * 16 + (lane >> 2) + (e >> 1) * 8, s = mt * 16 + j * 8 + 2 * (lane & 3);
+              *reinterpret_cast<uint32_t*>(sA + t * AS + s) = gl_pack(s <= t ? A[j][e] : 0.f, s + 1 <= t ? A[j][e + 1] : 0.f);
+            }
+        }
+      }
+      __syncthreads();
+      // O = q^ S + A V, rows of this warp, half of the columns
+      if (my_rows) {
+#pragma unroll
+        for (int ks = 0; ks < DP / 16; ++ks) {
+          uint32_t a[4];
+          gl_ldsm(a, sq + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * QS + ks * 16 + (lane >> 4) * 8);
+#pragma unroll
+          for (int j = 0; j < VS / 16; j += 2) {
+            uint32_t w[4];
+            gl_ldsm_t(w, sS + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VSS + half * (VS / 2) + j * 8 + (lane >> 4) * 8);
+            gl_mma(O[j], a, w[0], w[1]);
+            gl_mma(O[j + 1], a, w[2], w[3]);
+          }
+        }
+        for (int ks = g_lo; ks <= mt; ++ks) {              // causal: 16 keys at a time
+          uint32_t a[4];
+          gl_ldsm(a, sA + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * AS + ks * 16 + (lane >> 4) * 8);
+#pragma unroll
+          for (int j = 0; j < VS / 16; j += 2) {
+            uint32_t w[4];
+            gl_ldsm_t(w, sv + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VSS + half * (VS / 2) + j * 8 + (lane >> 4) * 8);
+            gl_mma(O[j], a, w[0], w[1]);
+            gl_mma(O[j + 1], a, w[2], w[3]);
+          }
+        }
+      }
+      // S += k^^T V
+      for (int ks = g_lo; ks < g_hi; ++ks) {
+        uint32_t a[MPW][4];
+#pragma unroll
+        for (int m = 0; m < MPW; ++m)
+          gl_ldsm_t(a[m], sk + (ks * 16 + (lane & 7) + ((lane >> 4) & 1) * 8) * QS + sm0 + m * 16 + ((lane >> 3) & 1) * 8);
+#pragma unroll
+        for (int j = 0; j < NPW; j += 2) {
+          uint32_t w[4];
+          gl_ldsm_t(w, sv + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VSS + sn0 + j * 8 + (lane >> 4) * 8);
+#pragma unroll
+          for (int m = 0; m < MPW; ++m) {
+            gl_mma(S[m][j], a[m], w[0], w[1]);
+            gl_mma(S[m][j + 1], a[m], w[2], w[3]);
+          }
+        }
+      }
+#pragma unroll
+      for (int m = 0; m < MPW; ++m) {
+        const int d = sm0 + m * 16 + (lane >> 2);
+        const float f0 = sPost[d], f1 = sPost[d + 8];
+#pragma unroll
+        for (int j = 0; j < NPW; ++j) { S[m][j][0] *= f0; S[m][j][1] *= f0; S[m][j][2] *= f1; S[m][j][3] *= f1; }
+      }
+      if (pc + 1 < pieces) __syncthreads();               // the next piece writes sS, sA and the factors again
+    }
+    // norm and gate (or the bare output, when other CTAs have the head's other columns)
+    const int r0 = mt * 16 + (lane >> 2), r1 = r0 + 8;
+    if (p.raw) {
+#pragma unroll
+      for (int j = 0; j < VS / 16; ++j) {
+        const int c = half * (VS / 2) + j * 8 + 2 * (lane & 3);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int r = e < 2 ? r0 : r1;
+          if (r < rows && c + (e & 1) < vw)
+            p.raw[(size_t)(start + ch * kChunk + r) * p.heads * p.vdim + h * p.vdim + v0 + c + (e & 1)] = O[j][e];
+        }
+      }
+    } else {
+      float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+      for (int j = 0; j < VS / 16; ++j) {
+        s0 += O[j][0] * O[j][0] + O[j][1] * O[j][1];
+        s1 += O[j][2] * O[j][2] + O[j][3] * O[j][3];
+      }
+#pragma unroll
+      for (int m = 1; m < 4; m <<= 1) {
+        s0 += __shfl_xor_sync(0xffffffffu, s0, m);
+        s1 += __shfl_xor_sync(0xffffffffu, s1, m);
+      }
+      if ((lane & 3) == 0) { sSS[half * kChunk + r0] = s0; sSS[half * kChunk + r1] = s1; }
+      __syncthreads();
+      const float i0 = rsqrtf((sSS[r0] + sSS[kChunk + r0]) / (float)p.vdim + p.eps);
+      const float i1 = rsqrtf((sSS[r1] + sSS[kChunk + r1]) / (float)p.vdim + p.eps);
+      const bool even = (p.vdim & 1) == 0;
+#pragma unroll
+      for (int j = 0; j < VS / 16; ++j) {
+        const int c = half * (VS / 2) + j * 8 + 2 * (lane & 3);
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+          const int r = e ? r1 : r0;
+          if (r >= rows || c >= p.vdim) continue;
+          const float inv = e ? i1 : i0;
+          const bf16* gp = x + (size_t)(ch * kChunk + r) * p.ldx + p.g_at + h * p.vdim + c;
+          bf16* op = reinterpret_cast<bf16*>(p.out) + (size_t)(start + ch * kChunk + r) * p.ldo + h * p.vdim + c;
+          if (even) {
+            const float2 g = gl_unpack(*reinterpret_cast<const uint32_t*>(gp));
+            *reinterpret_cast<uint32_t*>(op) = gl_pack(O[j][e] * inv * p.gain[c] * __fdividef(g.x, 1.f + __expf(-g.x)),
+                                                       O[j][e + 1] * inv * p.gain[c + 1] * __fdividef(g.y, 1.f + __expf(-g.y)));
+          } else {
+#pragma unroll
+            for (int k = 0; k < 2; ++k)
+              if (c + k < p.vdim) {
+                const float g = __bfloat162float(gp[k]);
+                op[k] = __float2bfloat16(O[j][e + k] * inv * p.gain[c + k] * __fdividef(g, 1.f + __expf(-g)));
+              }
+          }
+        }
+      }
+    }
+    __syncthreads();                                       // everything of this chunk has been read
+    if (Cfg::STAGES == 1 && ch + 1 < chunks) load(ch + 1);
+  }
+#pragma unroll
+  for (int m = 0; m < MPW; ++m)
+#pragma unroll
+    for (int j = 0; j < NPW; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int d = sm0 + m * 16 + (lane >> 2) + (e >> 1) * 8, c = sn0 + j * 8 + 2 * (lane & 3) + (e & 1);
+        if (d < p.dim && c < vw) st[(size_t)d * p.vdim + v0 + c] = S[m][j][e];
+      }
+}
+
+// Norm and gate of rows whose columns came from several CTAs: one warp per (token, head) of the sequences in question.
+__global__ void __launch_bounds__(128) gla_norm_kernel(const GlaParams p, int n_tok) {
+  grid_dep_launch();
+  grid_dep_wait();
+  const int lane = threadIdx.x & 31;
+  const long long gw = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+  if (gw >= (long long)n_tok * p.heads) return;
+  const int t = (int)(gw / p.heads), h = (int)(gw % p.heads);
+  int lo = 0, hi = p.B - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (p.cu_q[mid] <= t) lo = mid; else hi = mid - 1;
+  }
+  const int n = p.cu_q[lo + 1] - p.cu_q[lo];
+  if (n < p.min_q || n >= p.max_q) return;
+  const float* o = p.raw + (size_t)t * p.heads * p.vdim + h * p.vdim;
+  float ss = 0.f;
+  for (int c = lane; c < p.vdim; c += 32) ss += o[c] * o[c];
+#pragma unroll
+  for (int m = 16; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+  const float inv = rsqrtf(ss / (float)p.vdim + p.eps);
+  const bf16* gp = reinterpret_cast<const bf16*>(p.x) + (size_t)t * p.ldx + p.g_at + h * p.vdim;
+  bf16* op = reinterpret_cast<bf16*>(p.out) + (size_t)t * p.ldo + h * p.vdim;
+  for (int c = lane; c < p.vdim; c += 32) {
+    const float g = __bfloat162float(gp[c]);
+    op[c] = __float2bfloat16(o[c] * inv * p.gain[c] * __fdividef(g, 1.f + __expf(-g)));
+  }
+}
+
+}  // namespace xft
+
+using namespace xft;
+
+template <typename T, int LC, int RPT>
+static int launch_step(const GlaParams& p, cudaStream_t st) {
+  const int slices = (p.vdim + LC * 4 - 1) / (LC * 4);
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(slices, p.heads, p.B);
+  cfg.blockDim = dim3(kStepThreads);
+  cfg.dynamicSmemBytes = (size_t)(3 * p.dim + p.rank_ld) * sizeof(float);
+  cfg.stream = st;
+  cudaLaunchAttribute at[2];
+  int na = 0;
+  if (slices > 1) {
+    at[na].id = cudaLaunchAttributeClusterDimension;
+    at[na].val.clusterDim.x = slices; at[na].val.clusterDim.y = 1; at[na].val.clusterDim.z = 1;
+    ++na;
+  }
+  if (g_xft_pdl) {
+    at[na].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[na].val.programmaticStreamSerializationAllowed = 1;
+    ++na;
+  }
+  cfg.attrs = at;
+  cfg.numAttrs = na;
+  cudaError_t e = cudaLaunchKernelEx(&cfg, gla_step_kernel<T, LC, RPT>, p);
+  return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
+}
+template <typename T, int LC>
+static int step_rows(const GlaParams& p, cudaStream_t st) {
+  const int rows = (p.dim + kStepThreads / LC - 1) / (kStepThreads / LC);
+  if (rows <= 2) return launch_step<T, LC, 2>(p, st);
+  if (rows <= 4) return launch_step<T, LC, 4>(p, st);
+  if (rows <= 8) return launch_step<T, LC, 8>(p, st);
+  if (rows <= 16) return launch_step<T, LC, 16>(p, st);
+  if (rows <= 32) return launch_step<T, LC, 32>(p, st);
+  return -5;
+}
+template <typename T>
+static int step_columns(const GlaParams& p, int columns, cudaStream_t st) {
+  if (columns == 32) return step_rows<T, 8>(p, st);
+  if (columns == 64) return step_rows<T, 16>(p, st);
+  if (columns == 128) return step_rows<T, 32>(p, st);
+  return -6;
+}
+
+template <int DP, int VS, int RP>
+static int launch_chunk(const GlaParams& p, cudaStream_t st) {
+  using Cfg = ChunkCfg<DP, VS, RP>;
+  static bool attr_set = false;
+  if (!attr_set) {
+    if (cudaFuncSetAttribute(gla_chunk_kernel<DP, VS, RP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM) != cudaSuccess)
+      return 3000 + (int)cudaGetLastError();
+    attr_set = true;
+  }
+  cudaError_t e = launch_pdl(gla_chunk_kernel<DP, VS, RP>, dim3((p.vdim + VS - 1) / VS, p.heads, p.B), dim3(256), Cfg::SMEM, st, p);
+  return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
+}
+template <int DP, int VS>
+static int chunk_rank(const GlaParams& p, cudaStream_t st) {
+  if (p.rank <= 16) return launch_chunk<DP, VS, 16>(p, st);
+  if (p.rank <= 64) return launch_chunk<DP, VS, 64>(p, st);
+  return -7;
+}
+
+// Columns of the state per CTA of the chunk kernel for a key size, 0: it has no instance (the step kernel runs everything).
+extern "C" int xft_gla_chunk_columns(int dim, int vdim, int rank) {
+  if (dim > 256 || rank > (dim > 128 ? 16 : 64) || dim <= 0) return 0;
+  return dim > 128 || vdim <= 64 ? 64 : 128;
+}
+
+// x, a2 and out all fp32 (f32 = 1) or bf16; row strides and offsets as the file comment says, all multiples of 8 (a2's rows
+// too).  Sequences with min_q <= tokens < max_q take part, the others are left alone.  columns: of the state per CTA, 32, 64
+// or 128, at most 8 CTAs per head; rows per CTA: dim <= columns-dependent limit (1024, 512, 256).
+extern "C" int xft_gla_step(const void* x, int ldx, int k_at, int v_at, int g_at, int a_at, int heads, int dim, int vdim, int rank,
+                            int rank_ld, const void* a2, const float* bias, float tau, float scale, float eps, const float* gain,
+                            float* state, const int* state_slots, int num_states, const int* cu_q, const int* kv_lens, int B,
+                            void* out, int ldo, int min_q, int max_q, int columns, int f32, int* status, cudaStream_t st) {
+  if (B <= 0) return 0;
+  if (heads <= 0 || dim <= 0 || vdim <= 0 || rank <= 0 || rank_ld < rank || (rank_ld & 7) || tau <= 0.f || num_states <= 0 ||
+      columns <= 0) return -1;
+  if (heads > 65535 || B > 65535 || (vdim + columns - 1) / columns > 8 || (size_t)(3 * dim + rank_ld) * 4 > 40000) return -2;
+  if (((uintptr_t)a2 | (uintptr_t)state) & 15) return -3;
+  GlaParams p{x, ldx, k_at, v_at, g_at, a_at, heads, dim, vdim, rank, rank_ld, a2, bias, 1.f / tau, scale, eps, gain, state, state_slots,
+              num_states, cu_q, kv_lens, B, out, ldo, nullptr, min_q, max_q, status};
+  return f32 ? step_columns<float>(p, columns, st) : step_columns<bf16>(p, columns, st);
+}
+
+// bf16 portions.  raw: fp32 [T, heads * vdim], needed when a head has more columns than xft_gla_chunk_columns says.
+extern "C" int xft_gla_chunk(const void* x, int ldx, int k_at, int v_at, int g_at, int a_at, int heads, int dim, int vdim, int rank,
+                             int rank_ld, const void* a2, const float* bias, float tau, float scale, float eps, const float* gain,
+                             float* state, const int* state_slots, int num_states, const int* cu_q, const int* kv_lens, int B, int T,
+                             void* out, int ldo, float* raw, int min_q, int max_q, int* status, cudaStream_t st) {
+  if (B <= 0 || T <= 0) return 0;
+  const int cols = xft_gla_chunk_columns(dim, vdim, rank);
+  if (!cols || heads <= 0 || vdim <= 0 || rank <= 0 || rank_ld < rank || tau <= 0.f || num_states <= 0) return -1;
+  if (heads > 65535 || B > 65535 || (vdim > cols && !raw)) return -2;
+  if ((ldx & 7) || (k_at & 7) || (v_at & 7) || (g_at & 7) || (a_at & 7) || ((uintptr_t)x & 15)) return -3;
+  GlaParams p{x, ldx, k_at, v_at, g_at, a_at, heads, dim, vdim, rank, rank_ld, a2, bias, 1.f / tau, scale, eps, gain, state, state_slots,
+              num_states, cu_q, kv_lens, B, out, ldo, vdim > cols ? raw : nullptr, min_q, max_q, status};
+  int r;
+  if (dim > 128) r = launch_chunk<256, 64, 16>(p, st);
+  else if (dim > 64) r = cols == 64 ? chunk_rank<128, 64>(p, st) : chunk_rank<128, 128>(p, st);
+  else if (dim > 32) r = cols == 64 ? chunk_rank<64, 64>(p, st) : chunk_rank<64, 128>(p, st);
+  else r = cols == 64 ? chunk_rank<32, 64>(p, st) : chunk_rank<32, 128>(p, st);
+  if (r || !p.raw) return r;
+  const long long warps = (long long)T * heads;
+  cudaError_t e = launch_pdl(gla_norm_kernel, dim3((unsigned)((warps + 3) / 4)), dim3(128), 0, st, p, T);
+  return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
+}

@@ -1,0 +1,286 @@
+// What happens to the heads of attention whose values are its keys, between the projection and the paged cache, in one
+// launch: a causal convolution over time on every channel of q and k, then on the heads an RMS norm and the rotation of
+// their first dimensions.  The keys as they leave the convolution are the values.
+//
+//   u  rows [T, (hq + hkv) * dim] of the projection (bias included), u_t = 0 before a sequence's first token
+//   y_t = sum_j w[j] u_(t - taps + 1 + j)           per channel
+//   q, k = rotate(y / sqrt(mean(y^2) + eps) * gain)  per head;   v = y of the key heads
+//
+// The last taps - 1 rows of u that a sequence has seen are its state; a portion starts from them and leaves its own.  A
+// state slot is never cleared: rows in front of a sequence's first token are taken as zero by position.
+//
+// One warp per head and run of consecutive tokens: weights, gains and the convolution's window stay in registers, a lane
+// owns two neighbouring channels of every 64.  Heads are stored `padded` wide (zeros behind dim), as the attention kernels
+// take them.  In a decode step the warp that reads a state also moves it on; otherwise a second, small kernel does, after
+// all portions have read theirs.
+#include "ptx.cuh"
+
+namespace xft {
+
+typedef __nv_bfloat16 bf16;
+
+struct HeadPrepParams {
+  const void* x; int ldx; int T, B, hq, hkv, dim, padded, taps;
+  const float* conv;                       // [taps, (hq + hkv) * dim] or null (taps 1)
+  const float* q_norm; const float* k_norm;          // [dim] or null
+  float eps;
+  const int* positions; const float* table; int rot, max_pos;      // table [max_pos, rot]: cosines | sines
+  const int* cu_q; const int* kv_lens;
+  void* state; const int* state_slots; int num_states;             // [slots, taps - 1, (hq + hkv) * dim]
+  void* q_out; void* kc; void* vc; int bs; long long nslots; const int* slots;
+  int run, decode;                         // tokens per warp; decode: one token per sequence, states move on here
+  int* status;
+};
+
+template <typename T> __device__ __forceinline__ float hp_f32(T v);
+template <> __device__ __forceinline__ float hp_f32<float>(float v) { return v; }
+template <> __device__ __forceinline__ float hp_f32<bf16>(bf16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T hp_from(float v);
+template <> __device__ __forceinline__ float hp_from<float>(float v) { return v; }
+template <> __device__ __forceinline__ bf16 hp_from<bf16>(float v) { return __float2bfloat16(v); }
+
+// channels c, c + 1 of a row (n of them exist); `pair`: rows and heads are even, so the two load as one
+template <typename T>
+__device__ __forceinline__ float2 hp_load2(const T* p, int left, bool pair) {
+  float2 r = make_float2(0.f, 0.f);
+  if (pair) {
+    if (left > 0) {
+      struct alignas(2 * sizeof(T)) P2 { T a, b; };
+      const P2 v = *reinterpret_cast<const P2*>(p);
+      r = make_float2(hp_f32<T>(v.a), hp_f32<T>(v.b));
+    }
+  } else {
+    if (left > 0) r.x = hp_f32<T>(p[0]);
+    if (left > 1) r.y = hp_f32<T>(p[1]);
+  }
+  return r;
+}
+template <typename T>
+__device__ __forceinline__ void hp_store2(T* p, float2 v, int left, bool pair) {
+  if (pair) {
+    if (left > 0) {
+      struct alignas(2 * sizeof(T)) P2 { T a, b; };
+      *reinterpret_cast<P2*>(p) = P2{hp_from<T>(v.x), hp_from<T>(v.y)};
+    }
+  } else {
+    if (left > 0) p[0] = hp_from<T>(v.x);
+    if (left > 1) p[1] = hp_from<T>(v.y);
+  }
+}
+
+__device__ __forceinline__ int hp_sequence(const int* cu_q, int B, int t) {       // the sequence that owns token t
+  int lo = 0, hi = B - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (cu_q[mid] <= t) lo = mid; else hi = mid - 1;
+  }
+  return lo;
+}
+
+// NV: pairs of channels per lane (padded <= 64 * NV); TAPS >= taps
+template <typename T, int NV, int TAPS>
+__global__ void __launch_bounds__(128) head_prep_kernel(const HeadPrepParams p) {
+  extern __shared__ float hp_sm[];
+  grid_dep_launch();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int heads = p.hq + p.hkv, C = heads * p.dim;
+  const long long gw = (long long)blockIdx.x * 4 + warp;
+  const int t0 = (int)(gw / heads) * p.run, h = (int)(gw % heads);
+  if (t0 >= p.T) { grid_dep_wait(); return; }
+  const int t1 = min(t0 + p.run, p.T);
+  const bool is_k = h >= p.hq;
+  const bool even = (p.dim & 1) == 0, out_even = (p.padded & 1) == 0;
+  float* row = hp_sm + warp * p.dim;
+  const int skip = TAPS - p.taps;                        // leading taps that do not exist
+  float2 w[TAPS][NV], gain[NV];
+  const float* norm = is_k ? p.k_norm : p.q_norm;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = 2 * lane + 64 * i, left = p.dim - c;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+      w[j][i] = j < skip ? make_float2(0.f, 0.f)
+              : p.conv ? hp_load2<float>(p.conv + (size_t)(j - skip) * C + h * p.dim + c, left, even)
+                       : make_float2(1.f, 1.f);
+    gain[i] = norm ? hp_load2<float>(norm + c, left, even) : make_float2(1.f, 1.f);
+  }
+  grid_dep_wait();
+  const T* x = reinterpret_cast<const T*>(p.x) + h * p.dim;
+  T* state = reinterpret_cast<T*>(p.state);
+  int b = hp_sequence(p.cu_q, p.B, t0);
+  float2 u[TAPS][NV];                                    // the window, newest last
+  bool fresh = true;
+  for (int t = t0; t < t1; ++t) {
+    while (b + 1 < p.B && t >= p.cu_q[b + 1]) { ++b; fresh = true; }
+    const int start = p.cu_q[b], li = t - start;
+    T* st = nullptr;
+    if (p.taps > 1) {
+      int slot = p.state_slots[b];
+      if (slot < 0 || slot >= p.num_states) { if (lane == 0 && p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); slot = 0; }
+      st = state + (size_t)slot * (p.taps - 1) * C + h * p.dim;
+    }
+    if (fresh) {
+      const int past = p.kv_lens[b] - (p.cu_q[b + 1] - start);
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) {
+        const int idx = li - (TAPS - 1) + j;             // place in this portion; negative: before it
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+          const int c = 2 * lane + 64 * i, left = p.dim - c;
+          float2 v = make_float2(0.f, 0.f);
+          if (j >= skip) {
+            if (idx >= 0) v = hp_load2<T>(x + (size_t)(start + idx) * p.ldx + c, left, even);
+            else if (past + idx >= 0) v = hp_load2<T>(st + (size_t)(p.taps - 1 + idx) * C + c, left, even);
+          }
+          u[j][i] = v;
+        }
+      }
+      fresh = false;
+    }
+    float2 y[NV];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = 2 * lane + 64 * i, left = p.dim - c;
+      u[TAPS - 1][i] = hp_load2<T>(x + (size_t)t * p.ldx + c, left, even);
+      float2 a = make_float2(0.f, 0.f);
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) { a.x = fmaf(w[j][i].x, u[j][i].x, a.x); a.y = fmaf(w[j][i].y, u[j][i].y, a.y); }
+      y[i] = a;
+      ss += a.x * a.x + a.y * a.y;
+    }
+    if (p.decode && p.taps > 1) {                        // rows 1 .. taps - 1 of the window are the new state
+#pragma unroll
+      for (int j = 1; j < TAPS; ++j)
+        if (j > skip)
+#pragma unroll
+          for (int i = 0; i < NV; ++i) {
+            const int c = 2 * lane + 64 * i;
+            hp_store2<T>(st + (size_t)(j - 1 - skip) * C + c, u[j][i], p.dim - c, even);
+          }
+    }
+#pragma unroll
+    for (int j = 0; j + 1 < TAPS; ++j)
+#pragma unroll
+      for (int i = 0; i < NV; ++i) u[j][i] = u[j + 1][i];
+    T* dst;
+    if (is_k) {
+      const long long slot = p.slots[t];
+      if (slot < 0 || slot >= p.nslots) { if (lane == 0 && p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); continue; }
+      const size_t at = ((size_t)((slot / p.bs) * p.hkv + (h - p.hq)) * p.bs + slot % p.bs) * p.padded;
+      dst = reinterpret_cast<T*>(p.kc) + at;
+      T* v = reinterpret_cast<T*>(p.vc) + at;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) { const int c = 2 * lane + 64 * i; hp_store2<T>(v + c, y[i], p.padded - c, out_even); }
+    } else {
+      dst = reinterpret_cast<T*>(p.q_out) + ((size_t)t * p.hq + h) * p.padded;
+    }
+    if (norm) {
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      const float inv = 1.f / sqrtf(ss / (float)p.dim + p.eps);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) { y[i].x *= inv * gain[i].x; y[i].y *= inv * gain[i].y; }
+    }
+    if (p.rot > 0) {
+      int pos = p.positions[t];
+      if (pos < 0 || pos >= p.max_pos) { if (lane == 0 && p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); pos = 0; }
+      const float* cs = p.table + (size_t)pos * p.rot;
+      const int half = p.rot >> 1;
+      __syncwarp();
+#pragma unroll
+      for (int i = 0; i < NV; ++i) { const int c = 2 * lane + 64 * i; hp_store2<float>(row + c, y[i], p.dim - c, false); }
+      __syncwarp();
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = 2 * lane + 64 * i;
+        if (c < p.rot) {                                 // rot is even, so both channels turn or neither
+          const bool s0 = c >= half, s1 = c + 1 >= half;
+          const int f0 = s0 ? c - half : c, f1 = s1 ? c + 1 - half : c + 1;
+          const float p0 = row[s0 ? c - half : c + half], p1 = row[s1 ? c + 1 - half : c + 1 + half];
+          y[i].x = y[i].x * cs[f0] + (s0 ? p0 : -p0) * cs[half + f0];
+          y[i].y = y[i].y * cs[f1] + (s1 ? p1 : -p1) * cs[half + f1];
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) { const int c = 2 * lane + 64 * i; hp_store2<T>(dst + c, y[i], p.padded - c, out_even); }
+  }
+}
+
+// States of portions: row r of the new state is the row of u at distance taps - 1 - r from the portion's end.  A thread owns a
+// channel and goes upwards, so the old rows it still needs lie above the ones it has written.
+template <typename T>
+__global__ void __launch_bounds__(256) conv_state_kernel(const T* __restrict__ x, int ldx, int C, int taps, const int* __restrict__ cu_q,
+                                                         const int* __restrict__ kv_lens, T* state, const int* __restrict__ state_slots,
+                                                         int num_states, int* status) {
+  grid_dep_launch();
+  grid_dep_wait();
+  const int b = blockIdx.y, c = blockIdx.x * 256 + threadIdx.x;
+  if (c >= C) return;
+  const int start = cu_q[b], n = cu_q[b + 1] - start, past = kv_lens[b] - n;
+  if (n <= 0) return;
+  const int slot = state_slots[b];
+  if (slot < 0 || slot >= num_states) { if (status) atomicCAS(status, 0, XFT_ERR_BOUNDS); return; }
+  T* st = state + (size_t)slot * (taps - 1) * C + c;
+  for (int r = 0; r < taps - 1; ++r) {
+    const int idx = n - (taps - 1) + r;
+    T v = hp_from<T>(0.f);
+    if (idx >= 0) v = x[(size_t)(start + idx) * ldx + c];
+    else if (past + idx >= 0) v = st[(size_t)(taps - 1 + idx) * C];
+    st[(size_t)r * C] = v;
+  }
+}
+
+}  // namespace xft
+
+using namespace xft;
+
+template <typename T, int NV, int TAPS>
+static cudaError_t launch_head_prep(const HeadPrepParams& p, cudaStream_t st) {
+  const long long warps = (long long)((p.T + p.run - 1) / p.run) * (p.hq + p.hkv);
+  return launch_pdl(head_prep_kernel<T, NV, TAPS>, dim3((unsigned)((warps + 3) / 4)), dim3(128), (size_t)4 * p.dim * sizeof(float), st, p);
+}
+template <typename T, int NV>
+static cudaError_t pick_taps(const HeadPrepParams& p, cudaStream_t st) {
+  if (p.taps <= 1) return launch_head_prep<T, NV, 1>(p, st);
+  if (p.taps <= 2) return launch_head_prep<T, NV, 2>(p, st);
+  if (p.taps <= 4) return launch_head_prep<T, NV, 4>(p, st);
+  return launch_head_prep<T, NV, 8>(p, st);
+}
+template <typename T>
+static cudaError_t pick_width(const HeadPrepParams& p, cudaStream_t st) {
+  if (p.padded <= 64) return pick_taps<T, 1>(p, st);
+  if (p.padded <= 128) return pick_taps<T, 2>(p, st);
+  if (p.padded <= 256) return pick_taps<T, 4>(p, st);
+  return pick_taps<T, 8>(p, st);
+}
+
+// x rows, q_out, caches and state all fp32 (f32 = 1) or bf16.  caches [blocks, hkv, bs, padded].  dim <= padded <= 512, up to 8
+// taps; even dim wants even row strides.  decode: every sequence has one token in this call.
+extern "C" int xft_head_prep(const void* x, int ldx, int T, int B, int hq, int hkv, int dim, int padded, int taps, const float* conv,
+                             const float* q_norm, const float* k_norm, float eps, const int* positions, const float* table, int rot,
+                             int max_pos, const int* cu_q, const int* kv_lens, void* state, const int* state_slots, int num_states,
+                             void* q_out, void* kc, void* vc, int bs, long long nslots, const int* slots, int decode, int f32,
+                             int* status, cudaStream_t st) {
+  if (T <= 0 || B <= 0) return 0;
+  const int C = (hq + hkv) * dim;
+  if (hq <= 0 || hkv <= 0 || dim <= 0 || padded < dim || padded > 512 || taps < 1 || taps > 8 || ldx < C || bs <= 0) return -1;
+  if (rot < 0 || rot > dim || (rot & 1) || (rot > 0 && !table) || (taps > 1 && (!conv || !state || !state_slots || num_states <= 0))) return -2;
+  if ((dim & 1) == 0 && (ldx & 1)) return -3;
+  if (B > 65535) return -4;
+  const int run = decode || T < 2048 ? 1 : 8;
+  HeadPrepParams p{x, ldx, T, B, hq, hkv, dim, padded, taps, conv, q_norm, k_norm, eps, positions, table, rot, max_pos, cu_q, kv_lens,
+                   state, state_slots, num_states, q_out, kc, vc, bs, nslots, slots, run, decode, status};
+  cudaError_t e = f32 ? pick_width<float>(p, st) : pick_width<bf16>(p, st);
+  if (e != cudaSuccess) return (int)e;
+  if (taps > 1 && !decode) {
+    const dim3 grid((C + 255) / 256, B);
+    e = f32 ? launch_pdl(conv_state_kernel<float>, grid, dim3(256), 0, st, (const float*)x, ldx, C, taps, cu_q, kv_lens, (float*)state,
+                         state_slots, num_states, status)
+            : launch_pdl(conv_state_kernel<bf16>, grid, dim3(256), 0, st, (const bf16*)x, ldx, C, taps, cu_q, kv_lens, (bf16*)state,
+                         state_slots, num_states, status);
+    if (e != cudaSuccess) return (int)e;
+  }
+  return (int)cudaGetLastError();
+}

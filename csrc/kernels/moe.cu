@@ -65,7 +65,7 @@ __global__ void __launch_bounds__(128) route_kernel(const RouteParams p) {
         const float v = sel[lane * gsz + i];
         if (v > a) { b = a; a = v; } else if (v > b) b = v;
       }
-      gs[lane] = a + b;
+      gs[lane] = gsz > 1 ? a + b : a;
     }
     __syncwarp();
     if (lane == 0) {                            // keep the topk_group best groups (first wins ties)

@@ -1,7 +1,7 @@
 // Plain kernels for any size: the 32-bit path of the layered decoder (fp32 weights, activations and cache), and what a
 // bf16 model needs when its heads are larger than the tensor-core kernels take.
 //
-//   xft_gemm_f32        Y[T, N] = act(X[T, K] W[N, K]^T) in fp32 (no reduced-precision mode); also one product per head,
+//   xft_gemm_f32        Y[T, N] = act(X[T, K] W[N, K]^T + bias) * times in fp32 (no reduced-precision mode); also one product per head,
 //                       and products of rows grouped by expert
 //   xft_gated_act_f32   act(gate) * up
 //   xft_sigmoid_gate    x * sigmoid(gate)
@@ -29,6 +29,7 @@ struct GemmF32 {
   long long sx, sw, sy;                        // blockIdx.z steps through a batch with these strides
   // grouped form: blockIdx.y is a tile {group, first row, rows, -} of 64 rows; X row r comes from src[r] when given
   const int4* tiles; const int* num_tiles; const int* src; const float* row_w; int group_w_rows;
+  const float* bias; const float* times; int ldt;             // [N] and [T, N], or null
 };
 
 __device__ __forceinline__ float act_f32(float x, int act) {
@@ -84,7 +85,8 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32 p) {
     for (int j = 0; j < 4; ++j) {
       const int r = ty * 4 + i, n = n0 + tx * 4 + j;
       if (r < rows && n < p.N) {
-        float v = act_f32(acc[i][j], p.act);
+        float v = act_f32(acc[i][j] + (p.bias ? p.bias[n] : 0.f), p.act);
+        if (p.times) v *= p.times[(size_t)(t0 + r) * p.ldt + n];
         if (p.row_w) v *= p.row_w[t0 + r];
         Y[(size_t)(t0 + r) * p.ldo + n] = v;
       }
@@ -237,12 +239,13 @@ using namespace xft;
 
 // act: 0 none, 1 relu, 2 silu, 3 gelu (tanh), 4 relu squared
 extern "C" int xft_gemm_f32(const float* X, int ldx, const float* W, int ldw, float* Y, int ldo, int T, int N, int K, int act,
-                            cudaStream_t st) {
+                            const float* bias, const float* times, int ldt, cudaStream_t st) {
   if (T <= 0 || N <= 0) return 0;
-  if (K <= 0 || ldx < K || ldw < K || ldo < N) return -1;
+  if (K <= 0 || ldx < K || ldw < K || ldo < N || (times && ldt < N)) return -1;
   const int ty = (T + 63) / 64;
   if (ty > 65535) return -2;
   GemmF32 p{X, ldx, W, ldw, Y, ldo, T, N, K, act};
+  p.bias = bias; p.times = times; p.ldt = ldt;
   gemm_f32_kernel<<<dim3((N + 63) / 64, ty), 256, 0, st>>>(p);
   return (int)cudaGetLastError();
 }

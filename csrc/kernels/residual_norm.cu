@@ -1,7 +1,9 @@
 // The residual stream kept in 32 bits, with everything that happens to it between two products in one launch:
 //
-//   x <- x + post(y)        y = output of the sublayer just finished; post = a norm with its own gain, or nothing
-//   h <- next(x)            input of the sublayer that follows, for the next product (bf16 or fp32)
+//   x <- x + mult * post(y) + add   y = output of the sublayer just finished; post = a norm with its own gain, or nothing;
+//                                   add = a vector, the same for every row, or nothing
+//   h <- next(x)                    input of the sublayer that follows, for the next product (bf16 or fp32); next = a norm,
+//                                   or x as it is
 //
 // and, for the first layer, x <- table[id] * scale instead of the first line.  The norm is LayerNorm (mean and variance) or
 // RMSNorm, with a gain and an optional bias.  Either half can be left out; `rows` restricts the work to some rows of
@@ -28,7 +30,9 @@ struct ResidualNormParams {
   const int* rows;                                                  // row r of the outputs comes from rows[r], or null
   int n_in;                                                         // rows of x and y
   int H, HP, rms;
-  float eps, embed_scale;
+  float eps, embed_scale, mult;
+  const float* add;                                                 // [H] or null
+  int raw;                                                          // h is x itself
   int* status;
 };
 
@@ -165,7 +169,16 @@ __global__ void __launch_bounds__(NT) residual_norm_kernel(const ResidualNormPar
 #pragma unroll
     for (int c = 0; c < CH; ++c)
 #pragma unroll
+      for (int j = 0; j < 8; ++j) x[c][j] += p.mult * y[c][j];
+  }
+  if (p.add) {
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+      const int i = (threadIdx.x + c * NT) * 8, left = p.H - i;
+      load8(p.add + (left > 0 ? i : 0), left, y[c]);
+#pragma unroll
       for (int j = 0; j < 8; ++j) x[c][j] += y[c][j];
+    }
   }
   if (p.x_out) {
 #pragma unroll
@@ -175,7 +188,7 @@ __global__ void __launch_bounds__(NT) residual_norm_kernel(const ResidualNormPar
     }
   }
   if (p.h) {
-    norm_row<NT, CH, PRE>(x, p, p.next_w, p.next_b, g2, sh[2]);
+    if (!p.raw) norm_row<NT, CH, PRE>(x, p, p.next_w, p.next_b, g2, sh[2]);
 #pragma unroll
     for (int c = 0; c < CH; ++c) {
       const int i = (threadIdx.x + c * NT) * 8;
@@ -192,22 +205,22 @@ __global__ void __launch_bounds__(NT) residual_norm_kernel(const ResidualNormPar
 using namespace xft;
 
 // One launch over n_out rows (see the file comment).  H <= 32768; HP = H rounded up to 8, at most every row stride; row
-// strides multiples of 8, pointers 16-byte aligned (gains and biases too).  kind: 0 LayerNorm, 1 RMSNorm.
+// strides multiples of 8, pointers 16-byte aligned (gains, biases and the added vector too).  kind: 0 LayerNorm, 1 RMSNorm.
 extern "C" int xft_residual_norm(const int* ids, const void* table, int vocab, long long ldt, const float* x, int ldx,
                                  float* x_out, int ldxo, const void* y, int ldy, int y_f32, const float* post_w,
                                  const float* post_b, const float* next_w, const float* next_b, void* h, int ldh, int h_f32,
                                  const int* rows, int n_in, int n_out, int H, int kind, float eps, float embed_scale,
-                                 int* status, cudaStream_t st) {
+                                 float mult, const float* add, int raw, int* status, cudaStream_t st) {
   if (n_out <= 0) return 0;
   const int HP = (H + 7) / 8 * 8;
-  if (H <= 0 || H > 32768 || (!ids && !x) || (h && !next_w) || (!rows && n_out > n_in)) return -1;
+  if (H <= 0 || H > 32768 || (!ids && !x) || (h && !next_w && !raw) || (!rows && n_out > n_in)) return -1;
   if ((ids && ((ldt & 7) || ldt < HP)) || (!ids && ((ldx & 7) || ldx < HP))) return -2;
   if ((x_out && ((ldxo & 7) || ldxo < HP)) || (y && ((ldy & 7) || ldy < HP)) || (h && ((ldh & 7) || ldh < HP))) return -2;
   if (((uintptr_t)table | (uintptr_t)x | (uintptr_t)x_out | (uintptr_t)y | (uintptr_t)post_w | (uintptr_t)post_b |
-       (uintptr_t)next_w | (uintptr_t)next_b | (uintptr_t)h) & 15) return -3;
+       (uintptr_t)next_w | (uintptr_t)next_b | (uintptr_t)h | (uintptr_t)add) & 15) return -3;
   if (rows && x_out == x && x_out) return -4;              // gathered rows cannot be written back in place
   ResidualNormParams p{ids, (const bf16*)table, vocab, ldt, x, ldx, x_out, ldxo, y, ldy, y_f32, post_w, post_b, next_w,
-                       next_b, h, ldh, h_f32, rows, n_in, H, HP, kind, eps, embed_scale, status};
+                       next_b, h, ldh, h_f32, rows, n_in, H, HP, kind, eps, embed_scale, mult, add, raw, status};
   cudaError_t e;
 #define XFT_RN(NT, CH, PRE) e = launch_pdl(residual_norm_kernel<NT, CH, PRE>, dim3(n_out), dim3(NT), 0, st, p)
   const bool few = n_out <= 296;                           // decode: a wide CTA per row, everything in one round of loads

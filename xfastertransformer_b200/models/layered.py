@@ -187,11 +187,11 @@ class LayeredDecoder(Decoder):
             at += a
         return torch.cat(out, 1).reshape(n * padded, self.WP)
 
-    def _out_rows(self, L: Layer, p: str, heads: int, rng, vdim: int) -> None:
-        """The output projection: its columns are heads of `vdim`, padded to L.vd."""
+    def _out_rows(self, L: Layer, p: str, heads: int, rng, vdim: int, width: int = 0) -> None:
+        """The output projection: its columns are heads of `vdim`, padded to L.vd, and all of them to `width`."""
         w = self.src.matrix(p + "mix.o", (self.W, heads * vdim), cols=(rng[0] * vdim, rng[1] * vdim))
-        w = _pad(w.reshape(self.W, L.hq, vdim), self.WP, L.hq, L.vd)
-        L.o = make_linear(w.reshape(self.WP, L.hq * L.vd), self.kind)
+        w = _pad(w.reshape(self.W, L.hq, vdim), self.WP, L.hq, L.vd).reshape(self.WP, L.hq * L.vd)
+        L.o = make_linear(_pad(w, self.WP, max(width, L.hq * L.vd)), self.kind)
 
     def _load_layer(self, i: int) -> Layer:
         lc: LayerConfig = self.cfg.layers[i]
@@ -297,7 +297,7 @@ class LayeredDecoder(Decoder):
         gain = self.src.vector(p + "mix.norm", m.vdim, fake_ones=True)
         L.decay = ops.LinearWeights(_pad(a2, a2.shape[0], d.up(rank)).contiguous(), bias.contiguous(), m.tau, gain.contiguous())
         L.state_shape = ((L.hq, m.dim, m.vdim), torch.float32)
-        self._out_rows(L, p, m.heads, rng, m.vdim)
+        self._out_rows(L, p, m.heads, rng, m.vdim, d.up(L.hq * m.vdim))
 
     def _load_latent(self, L: Layer, p: str, q) -> None:
         """Latent attention: heads are split over ranks, the latents (one row per token) are on every rank."""

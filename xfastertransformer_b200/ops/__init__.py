@@ -371,7 +371,7 @@ class LinearWeights:
 
 
 def gated_linear(x, dims: LinearDims, w: LinearWeights, eps, state, state_slots, cu_q, kv_lens, meta=None):
-    """Gated linear attention of packed rows x -> [T, heads * vdim].  Per head, with decay = sigmoid(W_a2 a1 + bias)^(1 / tau)
+    """Gated linear attention of packed rows x -> [T, heads * vdim (aligned)].  Per head, with decay = sigmoid(W_a2 a1 + bias)^(1 / tau)
     per key channel: S <- diag(decay) S + k v^T and o = S^T (q / sqrt(dim)); the result is norm(o) * silu(g).  `state`
     [slots, heads, dim, vdim] fp32 is carried on; a sequence's first token starts from zero."""
     impl = _native_linear().gated_linear if _cuda(x) else R.gated_linear

@@ -19,6 +19,7 @@ import torch
 _LIB = None
 _ACT = {None: 0, "none": 0, "relu": 1, "silu": 2, "gelu": 3, "gelu_tanh": 3, "gelu_new": 3, "gelu_pytorch_tanh": 3,
         "swiglu": 2, "relu2": 4}
+_ACT.update({(a, "times"): c | 16 for a, c in list(_ACT.items())})       # the residual operand multiplies (kActTimes)
 
 STATUS_TEXT = {0: "ok", 1: "producer timed out waiting for a free stage", 2: "MMA warp timed out waiting for TMA data",
                3: "epilogue timed out waiting for the accumulator", 4: "timed out waiting for a peer flag",
@@ -169,11 +170,11 @@ def layernorm(x, w, b, eps):
 
 
 def residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids=None, table=None, keep_x=True,
-                  embed_scale=1.0):
+                  embed_scale=1.0, mult=1.0, add=None, raw=False):
     """csrc/kernels/residual_norm.cu.  x fp32 [T, HP]; y bf16 or fp32 rows; gains fp32 [H]."""
     dev = (x if x is not None else table).device
     gain = nxt[0] if nxt is not None else post[0] if post is not None else None
-    H = gain.numel() if gain is not None else x.shape[1] if x is not None else table.shape[1]
+    H = gain.numel() if gain is not None else add.numel() if add is not None else x.shape[1] if x is not None else table.shape[1]
     HP = (H + 7) // 8 * 8
     n_in = ids.numel() if ids is not None else x.shape[0]
     n_out = rows.numel() if rows is not None else n_in
@@ -187,7 +188,7 @@ def residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids=None, table=Non
     x_out = None
     if keep_x:
         x_out = x if ids is None and rows is None else torch.empty(n_out, HP, dtype=torch.float32, device=dev)
-    h = torch.empty(n_out, HP, dtype=h_dtype, device=dev) if nxt is not None else None
+    h = torch.empty(n_out, HP, dtype=h_dtype, device=dev) if nxt is not None or raw else None
     rows32 = None if rows is None else rows if rows.dtype == torch.int32 else rows.int()
     ids32 = None if ids is None else ids if ids.dtype == torch.int32 else ids.int()
     ws = Workspace.get(dev)
@@ -200,13 +201,13 @@ def residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids=None, table=Non
               0 if ids is not None else x.stride(0), _p(x_out), 0 if x_out is None else x_out.stride(0), _p(y),
               0 if y is None else y.stride(0), int(y is not None and y.dtype == torch.float32), _p(pw), _p(pb), _p(nw), _p(nb),
               _p(h), HP, int(h_dtype == torch.float32), _p(rows32), n_in, n_out, H, 0 if kind == "layer" else 1,
-              C.c_float(eps), C.c_float(embed_scale), _p(ws.status), _stream()), "residual_norm")
+              C.c_float(eps), C.c_float(embed_scale), C.c_float(mult), _p(add), int(raw), _p(ws.status), _stream()), "residual_norm")
     ws.launches += 1
     return x_out, h
 
 
-def gemm_f32(x, w, N, act=None):
-    """Y[T,N] = act(X[T,K] W[N,K]^T), everything in 32 bits."""
+def gemm_f32(x, w, N, act=None, bias=None, times=None):
+    """Y[T,N] = act(X[T,K] W[N,K]^T + bias) * times[T,N], everything in 32 bits."""
     x2 = x.reshape(-1, x.shape[-1])
     if x2.stride(1) != 1:
         x2 = x2.contiguous()
@@ -216,7 +217,7 @@ def gemm_f32(x, w, N, act=None):
     fn = lib().xft_gemm_f32
     fn.restype = C.c_int
     _check(fn(_p(x2), x2.stride(0) if T > 1 else max(x2.stride(0), K), _p(w), w.stride(0), _p(y), N, T, N, K, _ACT[act],
-              _stream()), "gemm_f32")
+              _p(bias), _p(times), 0 if times is None else times.stride(0), _stream()), "gemm_f32")
     Workspace.get(x.device).launches += 1
     return y
 
@@ -413,13 +414,23 @@ def linear(x, W, bias=None, act=None, residual=None, res_scale=1.0, out_dtype=No
         y = gemm_bf16(x, W.w, W.out_features, bias=bias, act=act, residual=residual, res_scale=res_scale,
                       out_dtype=out_dtype)
     elif W.kind == "fp32":
-        if bias is not None or residual is not None or out_dtype not in (None, torch.float32):
-            raise KernelError("fp32 products have no bias or residual")
-        y = gemm_f32(x, W.w, W.out_features, act)
+        if residual is not None or out_dtype not in (None, torch.float32):
+            raise KernelError("fp32 products have no residual")
+        y = gemm_f32(x, W.w, W.out_features, act, bias)
     else:
         from . import native_quant
         y = native_quant.linear(x, W, bias, act, residual, res_scale, out_dtype)
     return y.view(*lead, W.out_features)
+
+
+def linear_times(x, W, bias, act, times):
+    """act(x W^T + bias) * times, the factor applied in the product's epilogue."""
+    assert times.dim() == 2 and times.stride(1) == 1 and times.shape == (x.shape[0], W.out_features)
+    if W.kind == "fp32":
+        return gemm_f32(x, W.w, W.out_features, act, bias, times)
+    if W.kind != "bf16":
+        raise KernelError(f"no product with a factor for {W.kind} weights")
+    return gemm_bf16(x, W.w, W.out_features, bias=bias, act=(act, "times"), residual=times)
 
 
 def linear_gated(x, W, act="silu", bias=None):

@@ -104,8 +104,6 @@ def _pack_fp8(experts) -> dict:
 
 def _experts_f32(x, idx32, w, pk, act, expert_offset, gated, add):
     """The 32-bit path: rows stay where they are, the first product reads them through the plan."""
-    if gated:
-        raise N.KernelError("fp32 experts have no gate product")
     T, H = x.shape
     k, E, I, dev = idx32.shape[1], pk["E"], pk["I"], x.device
     lib, ws, n = _lib(), N.Workspace.get(dev), T * idx32.shape[1]
@@ -115,10 +113,16 @@ def _experts_f32(x, idx32, w, pk, act, expert_offset, gated, add):
     pos, src, row_w, tiles, meta = i32(n), i32(n), f32(n), i32(tiles_n, 4), i32(2)
     N._check(lib.xft_moe_plan(N._p(idx32), N._p(w), T, k, expert_offset, expert_offset + E, 64, N._p(pos), N._p(src), N._p(row_w),
                               N._p(tiles), N._p(meta), tiles_n, n, N._stream()), "moe_plan")
-    h1, ys, out = f32(n, I), f32(n, H), f32(T, H)
+    up = 2 * I if gated else I
+    h1, ys, out = f32(n, up), f32(n, H), f32(T, H)
     fn = lib.xft_gemm_f32_grouped
-    N._check(fn(N._p(x), x.stride(0) if T > 1 else max(x.stride(0), H), N._p(pk["gu"]), H, N._p(h1), I, I, H, I, N._p(tiles),
-                N._p(meta), tiles_n, N._p(src), N._p(None), N._ACT[act], N._stream()), "grouped fp32 up")
+    N._check(fn(N._p(x), x.stride(0) if T > 1 else max(x.stride(0), H), N._p(pk["gu"]), H, N._p(h1), up, up, H, up, N._p(tiles),
+                N._p(meta), tiles_n, N._p(src), N._p(None), 0 if gated else N._ACT[act], N._stream()), "grouped fp32 up")
+    if gated:
+        gu, h1 = h1, f32(n, I)
+        lib.xft_gated_act_f32.restype = C.c_int
+        N._check(lib.xft_gated_act_f32(N._p(gu), up, N._p(h1), n, I, N._ACT[act], N._stream()), "gated_act_f32")
+        ws.launches += 1
     N._check(fn(N._p(h1), I, N._p(pk["dn"]), I, N._p(ys), H, H, I, H, N._p(tiles), N._p(meta), tiles_n, N._p(None), N._p(row_w), 0,
                 N._stream()), "grouped fp32 down")
     N._check(lib.xft_moe_combine(N._p(ys), N._p(pos), k, N._p(add), N._p(None), 0, N._p(None), N._p(out), T, H, N._stream()),
