@@ -78,6 +78,41 @@ CONFIGS = {
         O.latent_layer(heads=2, dim=208, rot_dim=80, vdim=144, kv_rank=520, size=30, scaling=YARN, mlp=O.moe()),
         O.latent_layer(heads=3, dim=136, rot_dim=24, vdim=72, kv_rank=300, size=41, mlp=O.moe(top=3))], width=64, vocab=83),
 }
+BANDS = {"factor": 5.0, "low": 1.0, "high": 3.0, "original": 80}
+CONFIGS.update({
+    # Botusun: both mixers, unequal sizes, looped layers inside others, a side embedding off the 16-byte rows, experts in groups
+    "recurrent": O.botusun([
+        O.shared_kv_layer(heads=6, kv_heads=3, dim=20, size=17, rot_dims=12, scaling=BANDS, conv=3, mlp=O.dense(70)),
+        O.gla_layer(heads=3, dim=12, vdim=20, tau=4.0, mlp=O.grouped_moe(ff=36, experts=9, top=3, scale=1.7, groups=(3, 2))),
+        O.shared_kv_layer(heads=4, kv_heads=4, dim=48, size=70, rot_dims=48, base=500.0, scale=0.21, conv=1),
+        O.gla_layer(heads=2, dim=40, vdim=24, tau=1.0, mlp=O.dense(44))],
+        width=90, vocab=131, eps=3e-4, scale=1.7, mult=0.35, loop=(1, 3, 3), side=6),
+    # sizes of the kernels without padding; several chunks, a window off the 64-token pages
+    "recurrent128": O.botusun([
+        O.shared_kv_layer(heads=6, kv_heads=2, dim=128, size=100, rot_dims=64, scaling=BANDS, conv=4,
+                          mlp=O.grouped_moe(ff=64, experts=8, top=3, groups=(4, 2))),
+        O.gla_layer(heads=2, dim=128, vdim=128, tau=16.0, mlp=O.grouped_moe(ff=64, experts=5, top=1, scale=2.5)),
+        O.gla_layer(heads=3, dim=64, vdim=64, tau=12.0)], width=160, vocab=300, loop=(0, 2, 2), side=16),
+    # mechanisms left out one by one: no loop, no side embedding, no convolution, window, rotation or scaling, no groups, every
+    # expert chosen, factors of one
+    "recurrent_bare": O.botusun([
+        O.shared_kv_layer(heads=2, kv_heads=1, dim=32, conv=None, mask=False, rot=False, mlp=O.grouped_moe(ff=24, experts=3, top=3, scale=1.0)),
+        O.gla_layer(heads=1, dim=8, vdim=8, tau=1.0),
+        O.shared_kv_layer(heads=3, kv_heads=3, dim=16, size=1, rot_dims=2, conv=2, mlp=O.grouped_moe(ff=16, experts=4, top=1, groups=(4, 1))),
+        O.shared_kv_layer(heads=3, kv_heads=1, dim=64, size=5000, rot_dims=64, conv=4, mlp=O.dense(40))],
+        width=72, vocab=150, scale=1.0, mult=1.0),
+    # larger than the tensor-core kernels take, many taps, output columns over several CTAs; a loop of one pass
+    "recurrent_large": O.botusun([
+        O.shared_kv_layer(heads=2, kv_heads=1, dim=264, size=30, rot_dims=32, conv=7, mlp=O.dense(72)),
+        O.gla_layer(heads=2, dim=200, vdim=144, tau=10.0),
+        O.gla_layer(heads=1, dim=300, vdim=72, tau=6.0, mlp=O.grouped_moe(ff=24, experts=4, top=2, groups=(2, 1)))],
+        width=104, vocab=83, loop=(1, 2, 1), side=24),
+    # decays from none to e^-40 per token: chunks that go in pieces, pieces that go by differences
+    "recurrent_fast": O.botusun([
+        O.gla_layer(heads=2, dim=24, vdim=40, tau=0.2), O.gla_layer(heads=2, dim=72, vdim=80, tau=1.5, mlp=O.dense(40)),
+        O.shared_kv_layer(heads=2, kv_heads=1, dim=36, size=9, rot_dims=20, conv=5)], width=88, vocab=120, mult=0.5, loop=(0, 1, 2)),
+})
+RECURRENT = [n for n in sorted(CONFIGS) if n.startswith("recurrent")]
 LATENT = ["latent", "latent128", "latent_bare", "latent_large"]
 
 TOLERANCE = {"fp32": 3e-5, "bf16": 0.05}
@@ -179,7 +214,9 @@ def mixed_batches(case, dtype, seed=0, lengths=(150, 97, 64, 30, 1, 129), live=3
     pages = lambda n: (n + 63) // 64 * 64
     run = TraceRunner(case.path, dtype, sum(sorted((pages(n) for n in lengths), reverse=True)[:live]))
     cache = run.model.model.cache
-    size = cache.alloc.num_blocks
+    if cache.has_state:                                  # no more slots than live requests need
+        assert cache.max_states - 4 in (0, 1)
+    size, states = cache.alloc.num_blocks, cache.state_alloc.num_blocks
     at, got = {k: 0 for k in toks}, {k: [] for k in toks}
     waiting, alive = list(toks), []
     steps = 0
@@ -206,8 +243,12 @@ def mixed_batches(case, dtype, seed=0, lengths=(150, 97, 64, 30, 1, 129), live=3
                 for t in pool:
                     if t is not None:
                         t[b].fill_(30.0)
+        for s in cache.state_alloc.free:                 # nor what freed states hold
+            for t in cache.state:
+                t[s].fill_(30.0)
         steps += 1
-    assert cache.alloc.num_blocks == size and not cache.tables, "pools grew or requests were left behind"
+    assert (cache.alloc.num_blocks, cache.state_alloc.num_blocks) == (size, states) and not cache.state_slot
+    assert not cache.tables, "requests were left behind"
     for k, rows in got.items():
         check(torch.cat(rows), case.want(toks[k]), dtype, f"{case.name}: request {k} of {len(toks[k])} tokens")
     return steps

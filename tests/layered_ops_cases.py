@@ -331,3 +331,219 @@ def rotation(dev, dtype, rot, d, dv, tol, hq=3, hkv=2, T=90):
     q2 = ops.qkv_rope_cache(qkv[:, :hq * d].contiguous().to(dev), hq, 0, d, torch.tensor(pos, dtype=torch.int32).to(dev),
                             tab.to(dev), rot["dims"], "half", kc, vc, None, None, slots.to(dev), dv=dv)
     assert torch.equal(q2, q), "a layer with queries only rotates them like any other"
+
+
+# ------------------------------------------------------------------------------------------ recurrent mechanisms
+class Portions:
+    """Sequences cut into portions that run in batches: steps() yields (cu_q, kv_lens, which sequence and tokens)."""
+
+    def __init__(self, lengths, sizes, seed=0):
+        g = torch.Generator().manual_seed(seed)
+        self.at, self.n, self.sizes, self.g = [0] * len(lengths), list(lengths), sizes, g
+
+    def steps(self):
+        k = 0
+        while any(a < n for a, n in zip(self.at, self.n)):
+            live = [i for i in range(len(self.n)) if self.at[i] < self.n[i]]
+            if len(live) > 1 and k % 3 == 2:
+                live = live[1:]                           # some sit a step out
+            cu, lens, parts = [0], [], []
+            for i in live:
+                m = min(self.sizes[(k + i) % len(self.sizes)], self.n[i] - self.at[i])
+                parts.append((i, self.at[i], self.at[i] + m))
+                self.at[i] += m
+                cu.append(cu[-1] + m)
+                lens.append(self.at[i])
+            k += 1
+            yield cu, lens, parts
+
+
+def gated_linear(dev, dtype, tol, H, d, dv, rank, tau, lengths, sizes, z_around=1.5, spread=2.0):
+    """Batches of unequal portions over states that start out as garbage, against the recurrence token by token.  In every
+    head one key channel hardly decays and one token's key, 5 places in, owns it: its value must still be there at the end."""
+    g = torch.Generator().manual_seed(d * 7 + dv)
+    r = lambda *s: torch.randn(*s, generator=g).to(dtype).float()
+    gpu = dev.type == "cuda"
+    D = ops.LinearDims(H, d, dv, rank, 8 if gpu else 1)
+    a2 = (r(H * d, rank) * spread / rank ** 0.5).to(dtype).float()
+    bias, gain = z_around + r(H * d), 1 + 0.2 * r(dv)
+    bias[::d] = 14.0                                      # the first channel of every head
+    a2[::d] = 0
+    a2p = torch.zeros(H * d, D.up(rank))
+    a2p[:, :rank] = a2
+    W = ops.LinearWeights(a2p.to(dtype).to(dev).contiguous(), bias.to(dev), tau, gain.to(dev))
+    n = len(lengths)
+    state = torch.full((n + 2, H, d, dv), 50.0, device=dev)
+    slots = torch.randperm(n + 2, generator=g)[:n].int()
+    seqs, want = [], []
+    for T in lengths:
+        q, k, v, gate, a1 = r(T, H, d), r(T, H, d), r(T, H, dv), r(T, H * dv), r(T, rank)
+        k = ((k + q) / d ** 0.25).to(dtype).float()
+        q[:, :, 0], k[:, :, 0] = 4.0, 0.0
+        if T > 5:
+            k[5, :, 0] = 4.0
+        seqs.append((q, k, v, gate, a1))
+        z = a1.double() @ a2.double().T + bias.double()
+        o = O.gated_linear(q.double() * d ** -0.5, k.double(), v.double(), torch.exp(O.log_decay(z, tau)).view(T, H, d))
+        o = O.rms_norm(o, gain.double(), 1e-5).reshape(T, -1)
+        want.append(o * gate.double() * O.output_gate(gate.double(), torch.eye(H * dv, dtype=torch.float64)))
+    got = [torch.zeros(T, H * dv) for T in lengths]
+    for cu, lens, parts in Portions(lengths, sizes).steps():
+        x = torch.full((cu[-1], D.up(D.a_at + rank)), 9.0)
+        x[:, D.a_at:] = 0
+        for (i, a, b), c in zip(parts, cu):
+            q, k, v, gate, a1 = seqs[i]
+            s = slice(c, c + b - a)
+            x[s, :H * d], x[s, D.k_at:D.k_at + H * d] = q[a:b].reshape(b - a, -1), k[a:b].reshape(b - a, -1)
+            x[s, D.v_at:D.v_at + H * dv], x[s, D.g_at:D.g_at + H * dv] = v[a:b].reshape(b - a, -1), gate[a:b]
+            x[s, D.a_at:D.a_at + rank] = a1[a:b]
+        out = ops.gated_linear(x.to(dtype).to(dev), D, W, 1e-5, state, slots[[p[0] for p in parts]].to(dev), cu, lens)
+        out = out.float().cpu()
+        assert bool((out[:, H * dv:] == 0).all())
+        for (i, a, b), c in zip(parts, cu):
+            got[i][a:b] = out[c:c + b - a, :H * dv]
+    if gpu:
+        from xfastertransformer_b200.ops import native
+        native.Workspace.get(dev).check_status()
+    for i, (x, w) in enumerate(zip(got, want)):
+        e = (x.double() - w).abs().amax(-1) / w.abs().max()
+        assert bool((e <= tol).all()), f"sequence {i}: token {int(e.argmax())} of {len(e)} is off by {float(e.max()):.3g}"
+    untouched = [s for s in range(n + 2) if s not in slots.tolist()]
+    assert bool((state[untouched] == 50.0).all())
+
+
+def head_prep(dev, dtype, tol, hq, hkv, d, padded, taps, lengths, sizes, rot=None, norm=True):
+    """Convolution, norm, rotation and append over unequal portions; every tap weighs about as much, so a state that is one
+    token off, or not zero before the first token, shows."""
+    from xfastertransformer_b200.ops import reference as R
+    g = torch.Generator().manual_seed(d * 11 + taps)
+    r = lambda *s: torch.randn(*s, generator=g).to(dtype).float()
+    C = (hq + hkv) * d
+    conv = 0.6 + 0.5 * r(C, taps) if taps else None
+    qn, kn = 1 + 0.3 * r(d), 1 + 0.3 * r(d)
+    prep = ops.HeadPrep(hq, hkv, d, padded, conv.t().contiguous().to(dev) if taps else None, qn.to(dev) if norm else None,
+                        kn.to(dev) if norm else None)
+    tab = None
+    if rot:
+        sc = rot.get("scaling")
+        tab = R.rope_table(600, rot["dims"], rot["base"], "banded", sc["factor"], sc["original"], sc["high"], sc["low"],
+                           angle_dtype=torch.float64) if sc else R.rope_table(600, rot["dims"], rot["base"], angle_dtype=torch.float64)
+        tab = tab.to(dev)
+    n = len(lengths)
+    state = torch.full((n + 1, max(taps - 1, 0), C), 50.0, dtype=dtype, device=dev) if taps > 1 else None
+    slot_of = torch.randperm(n + 1, generator=g)[:n].int()
+    us = [r(T, C) for T in lengths]
+    nb = sum((T + 63) // 64 for T in lengths) + 1
+    place = torch.randperm(nb * 64, generator=g)
+    where = [place[sum(lengths[:i]):sum(lengths[:i + 1])] for i in range(n)]
+    kc, vc = (torch.full((nb, hkv, 64, padded), 7.0, dtype=dtype, device=dev) for _ in range(2))
+    qs = [torch.zeros(T, hq, padded) for T in lengths]
+    for cu, lens, parts in Portions(lengths, sizes).steps():
+        x = torch.cat([us[i][a:b] for i, a, b in parts])
+        wide = C + (-C % 8) + 8
+        x = torch.cat([x, torch.full((x.shape[0], wide - C), 99.0)], 1).to(dtype).to(dev)
+        pos = torch.cat([torch.arange(a, b) for _, a, b in parts]).int().to(dev)
+        slots = torch.cat([where[i][a:b] for i, a, b in parts]).int().to(dev)
+        q = ops.head_prep(x, prep, 1e-4, pos, tab, rot["dims"] if rot else 0, kc, vc, slots, state,
+                          slot_of[[p[0] for p in parts]].to(dev), cu, lens).float().cpu()
+        for (i, a, b), c in zip(parts, cu):
+            qs[i][a:b] = q[c:c + b - a]
+    if dev.type == "cuda":
+        from xfastertransformer_b200.ops import native
+        native.Workspace.get(dev).check_status()
+    for i, T in enumerate(lengths):
+        y = O.short_conv(us[i].double(), conv.double()) if taps else us[i].double()
+        wq, wv = y[:, :hq * d].view(T, hq, d), y[:, hq * d:].view(T, hkv, d)
+        wk = wv
+        if norm:
+            wq, wk = O.rms_norm(wq, qn.double(), 1e-4), O.rms_norm(wv, kn.double(), 1e-4)
+        wq, wk = O.rotate(wq, list(range(T)), rot), O.rotate(wk, list(range(T)), rot)
+        b, o = where[i] // 64, where[i] % 64
+        for got, want, what in ((qs[i], wq, "queries"), (kc.float().cpu()[b, :, o], wk, "keys"), (vc.float().cpu()[b, :, o], wv, "values")):
+            e = (got[..., :d].double() - want).abs().amax(dim=(-1, -2)) / want.abs().max()
+            assert bool((e <= tol).all()), f"{what} of sequence {i}: token {int(e.argmax())} of {T} is off by {float(e.max()):.3g}"
+            assert bool((got[..., d:] == 0).all()), f"{what}: padding"
+        if taps > 1:
+            tail = torch.cat([torch.zeros(taps - 1, C), us[i]])[-(taps - 1):]
+            m = min(taps - 1, T)                          # rows before the first token are never read
+            assert torch.equal(state[int(slot_of[i])].float().cpu()[-m:], tail[-m:]), f"state of sequence {i}"
+
+
+def residual_extras(dev, H, dtype, tol):
+    """The factor on what joins the residual stream, the vector added to every row, and the stream itself as the output."""
+    g = torch.Generator().manual_seed(H)
+    HP = (H + 7) // 8 * 8 if dev.type == "cuda" else H
+    wide = lambda t: torch.cat([t, torch.zeros(*t.shape[:-1], HP - H, dtype=t.dtype)], -1).to(dev).contiguous()
+    x, y, w, v = torch.randn(7, H, generator=g), torch.randn(7, H, generator=g).to(dtype), torch.randn(H, generator=g), torch.randn(H, generator=g)
+    table, ids = torch.randn(11, H, generator=g).bfloat16(), torch.tensor([2, 10, 0], dtype=torch.int32)
+    d = lambda t: t.double()
+    gain = (w.to(dev), None)
+    ht = tol if dtype == torch.float32 else 6e-3
+
+    def close(got, want, t):
+        assert float((got[:, :H].double().cpu() - want).abs().max() / want.abs().max()) <= t
+        assert bool((got[:, H:] == 0).all())
+    a, h = ops.residual_norm(wide(x), wide(y), gain, gain, 1e-3, "rms", h_dtype=dtype, mult=0.3, add=v.to(dev))
+    want = d(x) + 0.3 * O.rms_norm(d(y), d(w), 1e-3) + d(v)
+    close(a, want, tol)
+    close(h, O.rms_norm(want, d(w), 1e-3), ht)
+    a, h = ops.residual_norm(wide(x), wide(y), None, None, 1e-3, "rms", h_dtype=dtype, mult=-1.7, raw=True)
+    close(a, d(x) - 1.7 * d(y), tol)
+    assert torch.equal(h, a.to(dtype))
+    a, h = ops.residual_norm(None, None, None, gain, 1e-3, "rms", h_dtype=dtype, ids=ids.to(dev), table=wide(table), embed_scale=3.0, add=v.to(dev))
+    close(a, d(table)[ids.long()] * 3 + d(v), tol)
+    a, h = ops.residual_norm(wide(x), None, None, gain, 1e-3, "rms", h_dtype=dtype, add=v.to(dev))
+    close(h, O.rms_norm(d(x) + d(v), d(w), 1e-3), ht)
+
+
+def linear_times(dev, dtype, tol, T, K, N):
+    """gelu(x W^T) times rows that are a column range of a wider table."""
+    from xfastertransformer_b200.runtime.loader import make_linear
+    g = torch.Generator().manual_seed(T + N)
+    r = lambda *s: torch.randn(*s, generator=g).to(dtype).float()
+    x, w, e = r(T, K), (r(N, K) * 2 / K ** 0.5).bfloat16().float(), r(T, 3 * N)
+    W = make_linear(w.to(dev), "bf16" if dtype == torch.bfloat16 else "fp32")
+    got = ops.linear(x.to(dtype).to(dev), W, act="gelu_tanh", times=e.to(dtype).to(dev)[:, N:2 * N])
+    want = O.gelu_tanh(x.double() @ w.double().T) * e[:, N:2 * N].double()
+    err = float((got.double().cpu() - want).abs().max() / want.abs().max())
+    assert err <= tol, f"{T} x {K} x {N}: {err:.3g}"
+
+
+def grouped_route(dev, E, top, groups, T=60):
+    """Choice with corrections (also such that choice scores are negative), weights without them and not renormalised; among
+    groups, and among all."""
+    g = torch.Generator().manual_seed(E + top)
+    z = torch.randn(T, E, generator=g) * 3
+    for shift in (0.0, -4.0):
+        c = torch.randn(E, generator=g) * 0.7 + shift
+        wi, ww = O.grouped_router(z.double(), c.double(), top, 1.9, dict(zip(("count", "keep"), groups)) if groups else None)
+        count, keep = groups or (1, 1)
+        idx, w = ops.route(z.to(dev), "deepseek", top, c.to(dev), count, keep, 1.9, False, "sigmoid")
+        order, worder = idx.cpu().long().sort(-1), wi.sort(-1)
+        assert torch.equal(order.values, worder.values), f"{top} of {E} in {groups}, corrections around {shift}"
+        e = (w.cpu().double().gather(1, order.indices) - ww.gather(1, worder.indices)).abs().max()
+        assert float(e) < 1e-5
+
+
+def gated_experts(dev, dtype, tol, T, E, top, ff, width=72, groups=None):
+    """Sigmoid-scored experts with a gate product: router, plan, products and weighted sum."""
+    from xfastertransformer_b200.runtime.loader import make_linear
+    g = torch.Generator().manual_seed(T * 13 + E)
+    r = lambda *s: torch.randn(*s, generator=g).bfloat16().float()
+    h = r(T, width)
+    W = {"embed": torch.zeros(1, width), "l0.mlp.router": (r(E, width) * 2 / width ** 0.5).bfloat16().float(), "l0.mlp.correction": r(E)}
+    for e in range(E):
+        for n, (o, i) in dict(gate=(ff, width), up=(ff, width), down=(width, ff)).items():
+            W[f"l0.mlp.e{e}.{n}"] = (r(o, i) * 1.5 / i ** 0.5).bfloat16().float()
+    f = {"router": {"experts": E, "top": top, "scale": 0.8}}
+    if groups:
+        f["router"]["groups"] = dict(zip(("count", "keep"), groups))
+    want = O.grouped_experts(h.double(), f, {k: v.double() for k, v in W.items()}, "l0")
+    kind = "bf16" if dtype == torch.bfloat16 else "fp32"
+    lin = lambda *n: make_linear(torch.cat([W["l0.mlp." + x] for x in n]).to(dev), kind)
+    x = h.to(dtype).to(dev)
+    idx, w = ops.route(ops.linear(x, lin("router"), out_dtype=torch.float32), "deepseek", top, W["l0.mlp.correction"].to(dev),
+                       *(groups or (1, 1)), 0.8, False, "sigmoid")
+    got = ops.moe_experts(x, idx, w, [(lin(f"e{e}.gate", f"e{e}.up"), lin(f"e{e}.down")) for e in range(E)], "silu", 0, gated=True)
+    e = float((got.double().cpu() - want).abs().max() / want.abs().max())
+    assert e <= tol, f"{T} tokens, {top} of {E}: {e:.3g}"

@@ -439,7 +439,130 @@ def vepivik(layers, width=96, vocab=210, eps=1e-5, scale=2.0):
             "embedding": {"scale": scale}}
 
 
+def botusun(layers, width=96, vocab=210, eps=1e-5, scale=2.0, mult=0.4, loop=None, side=None):
+    """`loop`: (start, stop, times)."""
+    cfg = {"architecture": "Botusun", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width,
+           "embedding": {"scale": scale}, "residual_mult": mult}
+    if loop:
+        cfg["loop"] = dict(zip(("start", "stop", "times"), loop))
+    if side:
+        cfg["token_side"] = {"dim": side}
+    return cfg
+
+
+def shared_kv_layer(heads=4, kv_heads=2, dim=32, size=24, rot_dims=16, base=10000.0, scaling=None, scale=None, conv=4, mlp=None,
+                    mask=True, rot=True):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": scale if scale else dim ** -0.5}
+    if conv:
+        m["conv"] = conv
+    if mask:
+        m["mask"] = {"size": size}
+    if rot:
+        m["rot"] = {"dims": rot_dims, "base": base}
+        if scaling:
+            m["rot"]["scaling"] = scaling
+    return {"type": "attention", "mixer": m, "mlp": mlp}
+
+
+def gla_layer(heads=2, dim=16, vdim=24, tau=8.0, mlp=None):
+    return {"type": "gla", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "tau": tau}, "mlp": mlp}
+
+
+def grouped_moe(ff=40, experts=6, top=2, scale=1.3, groups=None):
+    """`groups`: (count, keep)."""
+    r = {"experts": experts, "top": top, "scale": scale}
+    if groups:
+        r["groups"] = dict(zip(("count", "keep"), groups))
+    return {"kind": "moe", "expert": {"ff": ff}, "router": r}
+
+
+def dense(ff=48):
+    return {"kind": "dense", "ff": ff}
+
+
 def random_weights(cfg, seed=0, gain=1.0):
+    if cfg["architecture"] == "Botusun":
+        return _botusun_weights(cfg, seed)
+    return _weights(cfg, seed, gain)
+
+
+def _botusun_weights(cfg, seed):
+    """As `_weights`.  The code that decides about experts is one per kind of router: a group's levels lie next to each other,
+    so that the groups' order is as clear as the experts'; corrections move single experts to the front or to the back of
+    their group, far enough that it shows."""
+    g = torch.Generator().manual_seed(seed)
+    D, V = cfg["width"], cfg["vocab"]
+
+    def mat(o, i, s=1.0):
+        return (torch.randn(o, i, generator=g) * (s / math.sqrt(i))).bfloat16()
+
+    def vec(n, around=1.0, s=0.2):
+        return (around + s * torch.randn(n, generator=g)).bfloat16()
+    perm = lambda n: torch.randperm(n, generator=g)
+    W = {"embed": (torch.randn(V, D, generator=g) / math.sqrt(D)).bfloat16(), "final.norm": vec(D)}
+    code, used = {}, 0
+    for layer in cfg["layers"]:
+        if (layer.get("mlp") or {}).get("kind") == "moe":
+            r = layer["mlp"]["router"]
+            E, n = r["experts"], (r.get("groups") or {"count": 1})["count"]
+            if (E, n) not in code:
+                levels = ((torch.arange(E) - (E - 1) / 2) * 3.0 / math.sqrt(D)).view(n, E // n)
+                rows = [torch.cat([levels[k][perm(E // n)] for k in perm(n)]) for _ in range(V)]
+                W["embed"][:, used:used + E] = torch.stack(rows).bfloat16()
+                code[E, n] = used
+                used += E
+    if cfg.get("loop"):
+        W["loop.step"] = (torch.randn(cfg["loop"]["times"], D, generator=g) * 0.7 / math.sqrt(D) * cfg["embedding"]["scale"]).bfloat16()
+        W["loop.step"][:, :used] = 0
+    side = (cfg.get("token_side") or {}).get("dim")
+    if side:
+        W["side.embed"] = torch.randn(V, side * len(cfg["layers"]), generator=g).bfloat16()
+    for i, layer in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}", layer["mixer"], layer.get("mlp")
+        H, d, dv = m["heads"], m["dim"], m["vdim"]
+        P = p + ".mix."
+        W[p + ".norm1"] = vec(D)
+        if layer["type"] == "gla":
+            rank = (5, 16, 24, 33)[i % 4] if d <= 128 else 9
+            W[P + "q"], W[P + "v"], W[P + "g"] = mat(H * d, D), mat(H * dv, D), mat(H * dv, D, 2.0)
+            # keys akin to their queries: a first token whose key misses its query has an output of nothing but rounding,
+            # which the norm behind it would blow up
+            W[P + "k"] = (W[P + "q"].float() + 0.7 * mat(H * d, D).float()).bfloat16()
+            W[P + "a1"], W[P + "a2"], W[P + "a2.b"] = mat(rank, D), mat(H * d, rank, 2.0), vec(H * d, 1.0, 2.0)
+            W[P + "norm"] = vec(dv)
+        else:
+            for x, n in (("q", H), ("k", m["kv_heads"])):
+                W[P + x], W[P + x + ".b"], W[P + x + ".norm"] = mat(n * d, D), vec(n * d, 0.0, 0.3), vec(d, 1.3)
+                if m.get("conv"):
+                    W[P + x + ".conv"] = vec(n * d * m["conv"], 0.4, 0.6).view(n * d, m["conv"])
+        W[P + "o"] = mat(D, H * dv, 2.0)
+        if f:
+            W[p + ".norm2"] = vec(D)
+            if f["kind"] == "moe":
+                r = f["router"]
+                E, n = r["experts"], (r.get("groups") or {"count": 1})["count"]
+                at, per = code[E, n], E // n
+                W[p + ".norm2"][at:at + E] = 1.0
+                columns = torch.cat([k * per + perm(per) for k in perm(n)])     # experts of a group read a group of the code
+                w = 0.001 * torch.randn(E, D, generator=g)
+                w[:, at:at + E] = torch.eye(E)[columns]
+                W[p + ".mlp.router"] = w.bfloat16()
+                c = torch.zeros(E)
+                for k in range(n):
+                    c[k * per + int(perm(per)[0])] += 2.0
+                    c[k * per + int(perm(per)[0])] -= 1.0 if per > 2 else 0.0
+                W[p + ".mlp.correction"] = c.bfloat16()
+            for x, ff in [(f".e{e}", f["expert"]["ff"]) for e in range(f["router"]["experts"])] if f["kind"] == "moe" else [("", f["ff"])]:
+                W[p + f".mlp{x}.gate"], W[p + f".mlp{x}.up"], W[p + f".mlp{x}.down"] = mat(ff, D, 2.0), mat(ff, D, 2.0), mat(D, ff, 2.0)
+        if side:
+            W[p + ".side.gate"], W[p + ".side.proj"], W[p + ".side.norm"] = mat(side, D), mat(D, side), vec(D, 0.5)
+    for n, t in W.items():
+        if n.endswith((".mix.o", ".down", ".side.proj")):
+            t[:used] = 0
+    return W
+
+
+def _weights(cfg, seed, gain):
     """bf16-representable weights, scaled so that scores spread over several units and every mechanism matters.
 
     Experts: the first columns of the residual stream hold a code that the embedding alone writes, a permutation of equally

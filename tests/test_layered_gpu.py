@@ -1,4 +1,4 @@
-"""Layered designs (Kafipel, Vepivik) on a GPU: every kernel of the path alone, and whole models in bf16 and in 32 bits, against a
+"""Layered designs (Kafipel, Vepivik, Botusun) on a GPU: every kernel of the path alone, and whole models in bf16 and in 32 bits, against a
 plain implementation of the equations."""
 import os
 import sys
@@ -218,6 +218,85 @@ def test_experts(dtype, tol, T, E, top, ff, shared):
     M.experts(_dev(), dtype, tol, T, E, top, ff, shared)
 
 
+# ------------------------------------------------------------------------------------------ recurrent mechanisms
+KINDS = pytest.mark.parametrize("dtype,tol", [(torch.float32, 1e-5), (torch.bfloat16, 1.5e-2)])
+
+
+@KINDS
+@pytest.mark.parametrize("sizes", [(1000,), (1,), (2,), (1, 40, 3, 17), (64, 200, 16, 65)])
+@pytest.mark.parametrize("H,d,dv,rank,tau", [(3, 12, 20, 5, 4.0), (2, 128, 128, 16, 16.0), (2, 40, 64, 33, 1.0), (2, 72, 80, 24, 9.0)])
+def test_gated_linear(dtype, tol, H, d, dv, rank, tau, sizes):
+    """Token by token, in chunks, and both in one batch."""
+    n = 70 if max(sizes) < 3 else 300
+    M.gated_linear(_dev(), dtype, tol, H, d, dv, rank, tau, (n, 33, 1, 130, 6), sizes)
+
+
+@KINDS
+@pytest.mark.parametrize("H,d,dv,rank", [(1, 200, 144, 16), (2, 256, 64, 9), (1, 300, 72, 9), (2, 33, 21, 7), (1, 8, 8, 1), (1, 64, 520, 64),
+                                         (5, 128, 192, 48), (1, 512, 256, 16)])
+def test_gated_linear_sizes(dtype, tol, H, d, dv, rank):
+    """Columns over several CTAs, sizes without a chunk instance, odd sizes, clusters of many."""
+    M.gated_linear(_dev(), dtype, tol, H, d, dv, rank, 12.0, (100, 20, 3), (1000,))
+    M.gated_linear(_dev(), dtype, tol, H, d, dv, rank, 12.0, (20, 3), (1, 2))
+
+
+@KINDS
+@pytest.mark.parametrize("tau,around,spread", [(0.2, 0.0, 3.0), (1.0, -3.0, 2.0), (0.05, 1.0, 2.0), (2.0, -9.0, 6.0), (16.0, 5.0, 0.5)])
+def test_gated_linear_decays(dtype, tol, tau, around, spread):
+    """Decays from none to all within a token: chunks in one piece, in pieces, and pieces from differences."""
+    M.gated_linear(_dev(), dtype, tol, 2, 64, 64, 16, tau, (200, 65, 17), (1000,), around, spread)
+    M.gated_linear(_dev(), dtype, tol, 1, 136, 40, 16, tau, (90,), (1000,), around, spread)
+
+
+@pytest.mark.parametrize("columns", [32, 64, 128])
+def test_gated_linear_step_columns(monkeypatch, columns):
+    from xfastertransformer_b200.ops import native_linear
+    monkeypatch.setattr(native_linear, "step_columns", lambda *a: columns)
+    M.gated_linear(_dev(), torch.bfloat16, 1.5e-2, 2, 100, 200, 16, 16.0, (40, 9), (1, 3))
+
+
+@pytest.mark.parametrize("dtype,tol", [(torch.float32, 1e-5), (torch.bfloat16, 1e-2)])
+@pytest.mark.parametrize("sizes", [(4000,), (1,), (2,), (1, 40, 3, 17)])
+@pytest.mark.parametrize("hq,hkv,d,padded,taps", [(3, 1, 20, 64, 3), (6, 2, 128, 128, 4), (2, 2, 96, 128, 2), (1, 1, 264, 264, 7), (4, 1, 36, 64, 1),
+                                                  (2, 1, 160, 256, 8), (3, 3, 21, 64, 5), (2, 1, 64, 64, 0)])
+def test_head_prep(dtype, tol, hq, hkv, d, padded, taps, sizes):
+    rot = {"dims": d // 4 * 2, "base": 3000.0, "scaling": dict(factor=6.0, low=1.0, high=4.0, original=50)}
+    padded = d if dtype == torch.float32 else padded
+    lengths = (30, 9, 1) if max(sizes) < 3 else (500, 33, 1, 6)
+    M.head_prep(_dev(), dtype, tol, hq, hkv, d, padded, taps, lengths, sizes, rot)
+    M.head_prep(_dev(), dtype, tol, hq, hkv, d, padded, taps, lengths[1:], sizes, norm=False)
+
+
+def test_head_prep_long():
+    """Runs of tokens per warp that cross from one sequence into the next."""
+    M.head_prep(_dev(), torch.bfloat16, 1e-2, 2, 1, 64, 64, 4, (1500, 3, 500, 1, 99), (4000,), {"dims": 64, "base": 1e4})
+
+
+@pytest.mark.parametrize("H", [72, 100, 256, 1021, 2048, 5120])
+def test_residual_extras(H):
+    M.residual_extras(_dev(), H, torch.bfloat16, 4e-6)
+    M.residual_extras(_dev(), H, torch.float32, 4e-6)
+
+
+@pytest.mark.parametrize("T", [1, 16, 40, 100, 300, 2000])
+@pytest.mark.parametrize("K,N", [(96, 8), (256, 24), (2048, 128), (2048, 256)])
+def test_linear_times(T, K, N):
+    """The factor in the epilogue of every bf16 product kernel: weight stream, tiles, token-major; and in 32 bits."""
+    M.linear_times(_dev(), torch.bfloat16, 8e-3, T, K, N)
+    M.linear_times(_dev(), torch.float32, 1e-5, T, K, N)
+
+
+@pytest.mark.parametrize("E,top,groups", [(12, 3, (4, 2)), (8, 4, (2, 1)), (6, 2, (6, 3)), (9, 9, None), (128, 8, (8, 4)), (62, 5, (31, 7))])
+def test_grouped_route(E, top, groups):
+    M.grouped_route(_dev(), E, top, groups)
+
+
+@pytest.mark.parametrize("T,E,top,ff,groups", [(9, 6, 2, 24, (3, 2)), (1, 4, 4, 8, None), (300, 32, 3, 64, (4, 2)), (200, 2, 1, 136, None)])
+@pytest.mark.parametrize("dtype,tol", [(torch.float32, 3e-6), (torch.bfloat16, 1e-2)])
+def test_gated_experts(dtype, tol, T, E, top, ff, groups):
+    M.gated_experts(_dev(), dtype, tol, T, E, top, ff, groups=groups)
+
+
 # ------------------------------------------------------------------------------------------ whole models
 BOTH = pytest.mark.parametrize("dtype", ["fp32", "bf16"])
 
@@ -229,45 +308,47 @@ def test_whole_prompt(cases, name, dtype):
 
 
 @BOTH
-@pytest.mark.parametrize("name", ["unequal", "heads128", "latent", "latent128"])
+@pytest.mark.parametrize("name", ["unequal", "heads128", "latent", "latent128", "recurrent", "recurrent128", "recurrent_bare"])
 def test_first_tokens(cases, name, dtype):
     C.first_tokens(cases(name), dtype)
 
 
 @BOTH
 @pytest.mark.parametrize("name,start", [("unequal", 1), ("heads128", 40), ("padded", 70), ("shared", 1), ("bare", 100),
-                                        ("latent", 1), ("latent128", 40), ("latent_bare", 30), ("latent_large", 100)])
+                                        ("latent", 1), ("latent128", 40), ("latent_bare", 30), ("latent_large", 100),
+                                        ("recurrent", 1), ("recurrent128", 40), ("recurrent_bare", 30), ("recurrent_fast", 1),
+                                        ("recurrent_large", 100)])
 def test_token_by_token(cases, name, start, dtype):
     C.token_by_token(cases(name), dtype, 140, start)
 
 
 @BOTH
 @pytest.mark.parametrize("sizes", [(2,), (3, 64, 1), (17, 29)])
-@pytest.mark.parametrize("name", ["unequal", "heads128", "latent", "latent128"])
+@pytest.mark.parametrize("name", ["unequal", "heads128", "latent", "latent128", "recurrent", "recurrent128", "recurrent_fast"])
 def test_portions(cases, name, sizes, dtype):
     C.portions(cases(name), dtype, 140, sizes)
 
 
 @BOTH
-@pytest.mark.parametrize("name", ["unequal", "heads128", "shared", "large_heads"] + C.LATENT)
+@pytest.mark.parametrize("name", ["unequal", "heads128", "shared", "large_heads"] + C.LATENT + C.RECURRENT)
 def test_mixed_batches_reuse_pages(cases, name, dtype):
     assert C.mixed_batches(cases(name), dtype) > 8
 
 
 @BOTH
-@pytest.mark.parametrize("name", ["unequal", "heads128", "latent"])
+@pytest.mark.parametrize("name", ["unequal", "heads128", "latent", "recurrent"])
 def test_rows_and_order(cases, name, dtype):
     C.rows_and_order(cases(name), dtype)
 
 
 @BOTH
-@pytest.mark.parametrize("name", ["unequal", "heads128", "padded", "latent", "latent128"])
+@pytest.mark.parametrize("name", ["unequal", "heads128", "padded", "latent", "latent128", "recurrent", "recurrent128"])
 def test_greedy_generation(cases, name, dtype):
     """generate(): the captured decode step (CUDA graph) included."""
     C.greedy(cases(name), dtype, 20, 130)
 
 
-@pytest.mark.parametrize("name", ["heads128", "latent128"])
+@pytest.mark.parametrize("name", ["heads128", "latent128", "recurrent128"])
 def test_graph_and_eager_steps_agree(cases, monkeypatch, name):
     c = cases(name)
     a = C.greedy(c, "bf16", 30, 60)

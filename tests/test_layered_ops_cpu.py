@@ -92,6 +92,116 @@ def _write(tmp_path, cfg, name="m"):
     return O.write_checkpoint(str(tmp_path / name), cfg, O.random_weights(cfg))
 
 
+@pytest.mark.parametrize("sizes", [(1000,), (1,), (2,), (1, 40, 3, 17)])
+@pytest.mark.parametrize("tau", [1.0, 9.0])
+def test_gated_linear(sizes, tau):
+    M.gated_linear(CPU, torch.float32, 2e-5, 2, 12, 20, 5, tau, (70, 33, 1, 6), sizes)
+
+
+@pytest.mark.parametrize("sizes", [(1000,), (1,), (2,), (1, 40, 3, 17)])
+@pytest.mark.parametrize("taps", [0, 1, 2, 4, 7])
+def test_head_prep(sizes, taps):
+    M.head_prep(CPU, torch.float32, 2e-5, 3, 1, 12, 16, taps, (40, 13, 1, 2), sizes, {"dims": 6, "base": 300.0})
+    M.head_prep(CPU, torch.float32, 2e-5, 2, 2, 8, 8, taps, (5, 20), sizes, norm=False)
+
+
+@pytest.mark.parametrize("sc", [dict(factor=8.0, low=1.0, high=4.0, original=100), dict(factor=0.5, low=2.0, high=2.5, original=40),
+                                dict(factor=3.0, low=1.0, high=50.0, original=5000), dict(factor=1.0, low=1.0, high=4.0, original=64)])
+def test_banded_frequencies(sc):
+    """Wavelengths on both sides of the bands and inside the ramp."""
+    M.head_prep(CPU, torch.float32, 3e-5, 2, 1, 40, 40, 3, (500,), (600,), {"dims": 36, "base": 20000.0, "scaling": sc})
+
+
+def test_residual_extras():
+    M.residual_extras(CPU, 77, torch.float32, 2e-6)
+
+
+def test_linear_times():
+    M.linear_times(CPU, torch.float32, 1e-5, 9, 30, 12)
+
+
+@pytest.mark.parametrize("E,top,groups", [(12, 3, (4, 2)), (8, 4, (2, 1)), (6, 2, (6, 3)), (9, 9, None), (5, 1, None), (10, 2, (1, 1))])
+def test_grouped_route(E, top, groups):
+    M.grouped_route(CPU, E, top, groups)
+
+
+@pytest.mark.parametrize("T,E,top,ff,groups", [(9, 6, 2, 24, (3, 2)), (1, 4, 4, 8, None), (30, 8, 1, 16, (2, 1))])
+def test_gated_experts(T, E, top, ff, groups):
+    M.gated_experts(CPU, torch.float32, 1e-5, T, E, top, ff, groups=groups)
+
+
+def test_layer_runs():
+    """The order of looped layers, and what each run owns: a pass has pools and states of its own over shared weights."""
+    import layered_cases as C
+    for name in C.RECURRENT:
+        cfg = C.CONFIGS[name]
+        mine = [(i, max(t, 0)) for i, t in ModelConfig.from_dict(cfg).runs()]
+        assert mine == [(i, t) for i, t, _ in O.layer_runs(cfg)], name
+
+
+def test_recurrent_config_and_pools(tmp_path):
+    import layered_cases as C
+    cfg = C.CONFIGS["recurrent"]
+    p = _write(tmp_path, cfg)
+    c = ModelConfig.load(p)
+    assert c.model_type == "botusun" and c.residual_mult == 0.35 and c.embed_scale == 1.7 and c.side_dim == 6
+    a, g = c.layers[0].mixer, c.layers[1]
+    assert (a.conv, a.values_from_keys, a.qk_norm, a.qk_bias, a.sink, a.rot.scaling) == (3, True, True, True, 0.0, "banded")
+    assert (g.mixer.kind, g.mixer.tau, g.mixer.has_kv) == ("gla", 4.0, False)
+    f = g.moe
+    assert (f.scoring, f.renorm, f.scale, f.groups, f.keep_groups, f.gated, f.correction) == ("sigmoid", False, 1.7, 3, 2, True, True)
+    m = xft.AutoModel.from_pretrained(p, dtype="fp32", max_cache_tokens=130, max_sequences=2)
+    cache = m.model.cache
+    # runs: 0, three times (1, 2), 3: four of them keep keys, four a matrix, one a convolution's inputs (layer 2 has one tap)
+    assert len(cache.k) == 4 and [tuple(t.shape[1:]) for t in cache.state] == [(2, 180)] + [(3, 12, 20)] * 3 + [(2, 40, 24)]
+    assert len(m.model.decoder.layers) == 4 and len(m.model.decoder.runs) == 8
+    for i in range(2):
+        m.set_input_cb([[1, 2, 3]], max_length=10)
+    with pytest.raises(MemoryError, match="state"):
+        m.set_input_cb([[1, 2, 3]], max_length=10)
+    with pytest.raises(ValueError, match="int8"):
+        xft.AutoModel.from_pretrained(p, dtype="bf16", kv_cache_dtype="int8")
+
+
+def test_state_slots():
+    """Slots of the state pools: taken and given back, copied by a fork, permuted by a reorder, kept when the pools grow."""
+    from xfastertransformer_b200.runtime.kv_cache import PagedKVCache
+    c = PagedKVCache(1, 1, 4, 4, "fp32", CPU, block_size=4, states=[((2,), torch.float32), ((3, 1), torch.float32)])
+    for s in (7, 8, 9):
+        c.add_sequence(s)
+        c.append_slots(s, 5)
+        for t in c.state:
+            t[c.state_slot[s]] = s
+    val = lambda s: [float(t[c.state_slot[s]].flatten()[0]) for t in c.state]
+    c.fork(8, 20)
+    assert val(20) == [8, 8] and c.state_slot[20] != c.state_slot[8]
+    c.reorder([7, 8, 9], [1, 0, 0])
+    assert [val(s) for s in (7, 8, 9)] == [[8, 8], [7, 7], [7, 7]]
+    old, version = c.state_alloc.num_blocks, c.version
+    for s in range(100, 100 + old):
+        c.add_sequence(s)
+    assert c.state_alloc.num_blocks > old and c.version > version and val(7) == [8, 8]
+    with pytest.raises(RuntimeError, match="cannot go back"):
+        c.truncate(7, 3)
+    for s in [7, 8, 9, 20] + list(range(100, 100 + old)):
+        c.free_sequence(s)
+    assert c.state_alloc.num_free == c.state_alloc.num_blocks and not c.state_slot
+
+
+@pytest.mark.parametrize("change,match", [
+    (lambda c: c["layers"][0]["mixer"].update(vdim=24), "size"), (lambda c: c["loop"].update(stop=9), "loop"),
+    (lambda c: c["layers"][1]["mlp"]["router"].update(top=7), "experts"),
+    (lambda c: c["layers"][1]["mlp"]["router"]["groups"].update(count=4), "groups")])
+def test_recurrent_config_faults(tmp_path, change, match):
+    import copy
+
+    import layered_cases as C
+    cfg = copy.deepcopy(C.CONFIGS["recurrent"])
+    change(cfg)
+    with pytest.raises(ValueError, match=match):
+        ModelConfig.from_dict(cfg)
+
+
 def test_config_is_read_per_layer(tmp_path):
     sc = {"factor": 2.5, "original": 77, "fast": 9.0, "slow": 0.7}
     cfg = O.config([O.attention_layer(heads=6, kv_heads=3, dim=20, vdim=28, size=11, keep=2, rot_dims=10, scaling=sc, scale=0.3,
@@ -271,7 +381,7 @@ def test_partial_library_has_what_layered_models_call():
     text = "".join(open(os.path.join(ROOT, "csrc", "kernels", f)).read() for f in b.LAYERED)
     defined = set(re.findall(r'extern "C" \w+ (xft_\w+)\(', text))
     ops_dir = os.path.join(ROOT, "xfastertransformer_b200", "ops")
-    src = {f: open(os.path.join(ops_dir, f)).read() for f in ("native.py", "native_latent.py", "native_moe.py")}
+    src = {f: open(os.path.join(ops_dir, f)).read() for f in ("native.py", "native_latent.py", "native_linear.py", "native_moe.py")}
     wanted = {n for t in src.values() for n in re.findall(r'(?:lib\(\)\.|L\.|lib\.|")(xft_\w+)', t)}
     assert len(wanted) > 30 and wanted - defined <= {"xft_qgemm_grouped"}, wanted - defined
 
@@ -298,7 +408,7 @@ def test_command_line(tmp_path):
         assert torch.allclose(got.double(), want, atol=2e-4)
 
 
-@pytest.mark.parametrize("name", ["tiny-kafipel", "tiny-vepivik"])
+@pytest.mark.parametrize("name", ["tiny-kafipel", "tiny-vepivik", "tiny-botusun"])
 def test_synthetic_checkpoint_and_benchmark_tool(tmp_path, monkeypatch, name):
     """The presets write checkpoints that load, and the benchmark tool runs one by name with fake weights."""
     from xfastertransformer_b200.tools.synthetic import preset, write_synthetic_checkpoint

@@ -86,12 +86,36 @@ def vepivik_config(width: int, heads: int, kv_heads: int, layers: int, experts: 
     return {"architecture": "Vepivik", "width": width, "vocab": vocab, "norm": {"eps": eps}, "embedding": {"scale": scale}, "layers": out}
 
 
+def botusun_config(width: int, heads: int, kv_heads: int, layers: int, ff: int, experts: int, top: int, groups: int, keep: int,
+                   vocab: int = 32000, dim: int = 128, window: int = 1024, gla_heads: int = 16, gla_dim: int = 128,
+                   gla_vdim: int = 128, tau: float = 16.0, conv: int = 4, times: int = 1, side: int = 128, gla_every: int = 2,
+                   eps: float = 1e-5, scale: float = 4.0, mult: float = 0.5) -> dict:
+    """config.json of a Botusun model: every `gla_every`-th layer is gated linear attention, the others windowed attention
+    whose values are its keys; the middle half of the layers runs `times` times."""
+    out = []
+    for i in range(layers):
+        mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "scale": 1.0,
+                                                               "groups": {"count": groups, "keep": keep}}}
+        if gla_every and i % gla_every == gla_every - 1:
+            m = {"heads": gla_heads, "dim": gla_dim, "vdim": gla_vdim, "tau": tau}
+            out.append({"type": "gla", "mixer": m, "mlp": mlp})
+        else:
+            m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "conv": conv, "mask": {"size": window},
+                 "rot": {"dims": dim // 2, "base": 500000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+            out.append({"type": "attention", "mixer": m, "mlp": mlp})
+    return {"architecture": "Botusun", "width": width, "vocab": vocab, "norm": {"eps": eps}, "embedding": {"scale": scale}, "layers": out,
+            "residual_mult": mult, "loop": {"start": layers // 4, "stop": layers - layers // 4, "times": times}, "token_side": {"dim": side}}
+
+
 LAYERED_PRESETS: Dict[str, tuple] = {
     "tiny-kafipel": (kafipel_config, dict(width=192, heads=6, kv_heads=2, ff=512, layers=3, vocab=1000, dim=64, window=48)),
     "kafipel-1b": (kafipel_config, dict(width=2048, heads=16, kv_heads=4, ff=5632, layers=16)),
     "kafipel-8b": (kafipel_config, dict(width=4096, heads=32, kv_heads=8, ff=14336, layers=32)),
     "tiny-vepivik": (vepivik_config, dict(width=192, heads=5, kv_heads=1, layers=4, experts=6, top=2, ff=56, shared=72, vocab=1000, dim=40,
                                           rot_dim=24, vdim=32, kv_rank=72, window=48, latent_window=90)),
+    "tiny-botusun": (botusun_config, dict(width=192, heads=6, kv_heads=3, layers=4, ff=40, experts=6, top=2, groups=3, keep=2, vocab=1000,
+                                          dim=40, window=48, gla_heads=3, gla_dim=24, gla_vdim=40, conv=3, times=2, side=20)),
+    "botusun-lite": (botusun_config, dict(width=2048, heads=16, kv_heads=4, layers=16, ff=1408, experts=64, top=6, groups=8, keep=4)),
     "vepivik-lite": (vepivik_config, dict(width=2048, heads=16, kv_heads=4, layers=26, experts=64, top=6, ff=1408, shared=2816)),
 }
 
@@ -121,6 +145,15 @@ def _write_layered(path: str, cfg: ModelConfig, seed: int, std: float) -> str:
             if spec.post_norm:
                 gain(p + n + "b")
         put(p + "mix.q", m.heads * (m.dim + m.rot_dim), W)
+        if m.kind == "gla":
+            rank = 16
+            put(p + "mix.k", m.heads * m.dim, W)
+            put(p + "mix.v", m.heads * m.vdim, W)
+            put(p + "mix.g", m.heads * m.vdim, W)
+            put(p + "mix.a1", rank, W)
+            put(p + "mix.a2", m.heads * m.dim, rank)
+            put(p + "mix.a2.b", m.heads * m.dim, around=2.0)
+            gain(p + "mix.norm", m.vdim)
         if m.kind == "latent":
             if m.kv_from < 0:
                 put(p + "mix.dkv", m.kv_rank + m.rot_dim, W)
@@ -129,7 +162,16 @@ def _write_layered(path: str, cfg: ModelConfig, seed: int, std: float) -> str:
             put(p + "mix.uv", m.heads * m.vdim, m.kv_rank)
             if m.gate:
                 put(p + "mix.g", m.heads * m.vdim, W)
-        elif m.kv_from < 0:
+        elif m.values_from_keys:
+            put(p + "mix.k", m.kv_heads * m.dim, W)
+            for x, n in (("q", m.heads), ("k", m.kv_heads)):
+                if m.qk_bias:
+                    put(p + f"mix.{x}.b", n * m.dim)
+                if m.qk_norm:
+                    gain(p + f"mix.{x}.norm", m.dim)
+                if m.conv:
+                    put(p + f"mix.{x}.conv", n * m.dim, m.conv, around=1.0 / m.conv, s=0.1)
+        elif m.kind != "gla" and m.kv_from < 0:
             put(p + "mix.k", m.kv_heads * m.dim, W)
             put(p + "mix.v", m.kv_heads * m.vdim, W)
         if spec.sinks:
@@ -141,9 +183,20 @@ def _write_layered(path: str, cfg: ModelConfig, seed: int, std: float) -> str:
             put(p + "mlp.down", W, lc.ff)
         if f:
             put(p + "mlp.router", f.experts, W)
+            if f.correction:
+                put(p + "mlp.correction", f.experts)
             for n, ff in [(f"e{e}", f.ff) for e in range(f.experts)] + ([("shared", f.shared)] if f.shared else []):
-                put(p + f"mlp.{n}.up", ff, W)
+                for x in ("gate", "up") if f.gated else ("up",):
+                    put(p + f"mlp.{n}.{x}", ff, W)
                 put(p + f"mlp.{n}.down", W, ff)
+        if cfg.side_dim:
+            put(p + "side.gate", cfg.side_dim, W)
+            put(p + "side.proj", W, cfg.side_dim)
+            gain(p + "side.norm")
+    if cfg.side_dim:
+        put("side.embed", cfg.vocab_size, cfg.side_dim * len(cfg.layers), s=1.0)
+    if cfg.loop:
+        put("loop.step", cfg.loop.times, W)
     write_safetensors(os.path.join(path, "model.safetensors"), t)
     return path
 
