@@ -97,7 +97,7 @@ CONFIGS.update({
     # expert chosen, factors of one
     "recurrent_bare": O.botusun([
         O.shared_kv_layer(heads=2, kv_heads=1, dim=32, conv=None, mask=False, rot=False, mlp=O.grouped_moe(ff=24, experts=3, top=3, scale=1.0)),
-        O.gla_layer(heads=1, dim=8, vdim=8, tau=1.0),
+        O.gla_layer(heads=1, dim=24, vdim=16, tau=1.0),
         O.shared_kv_layer(heads=3, kv_heads=3, dim=16, size=1, rot_dims=2, conv=2, mlp=O.grouped_moe(ff=16, experts=4, top=1, groups=(4, 1))),
         O.shared_kv_layer(heads=3, kv_heads=1, dim=64, size=5000, rot_dims=64, conv=4, mlp=O.dense(40))],
         width=72, vocab=150, scale=1.0, mult=1.0),

@@ -426,8 +426,8 @@ def head_prep(dev, dtype, tol, hq, hkv, d, padded, taps, lengths, sizes, rot=Non
     tab = None
     if rot:
         sc = rot.get("scaling")
-        tab = R.rope_table(600, rot["dims"], rot["base"], "banded", sc["factor"], sc["original"], sc["high"], sc["low"],
-                           angle_dtype=torch.float64) if sc else R.rope_table(600, rot["dims"], rot["base"], angle_dtype=torch.float64)
+        tab = R.rope_table(2000, rot["dims"], rot["base"], "banded", sc["factor"], sc["original"], sc["high"], sc["low"],
+                           angle_dtype=torch.float64) if sc else R.rope_table(2000, rot["dims"], rot["base"], angle_dtype=torch.float64)
         tab = tab.to(dev)
     n = len(lengths)
     state = torch.full((n + 1, max(taps - 1, 0), C), 50.0, dtype=dtype, device=dev) if taps > 1 else None

@@ -219,7 +219,7 @@ def test_experts(dtype, tol, T, E, top, ff, shared):
 
 
 # ------------------------------------------------------------------------------------------ recurrent mechanisms
-KINDS = pytest.mark.parametrize("dtype,tol", [(torch.float32, 1e-5), (torch.bfloat16, 1.5e-2)])
+KINDS = pytest.mark.parametrize("dtype,tol", [(torch.float32, 4e-5), (torch.bfloat16, 1.5e-2)])
 
 
 @KINDS
