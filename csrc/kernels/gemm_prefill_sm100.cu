@@ -571,6 +571,7 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_tm_kernel(const __grid_co
     const int q = warp & 3;
     const int row = q * 32 + lane;
     const bool vec = (p.N % 8 == 0) && (p.ldo % 8 == 0) && (!p.residual || p.ldr % 8 == 0);
+    const bool bias16 = (reinterpret_cast<uintptr_t>(p.bias) & 15) == 0;
     int lt = 0;
     for (int item = blockIdx.x; item < total; item += gridDim.x, ++lt) {
       const Item im = item_of(item);
@@ -602,7 +603,13 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_tm_kernel(const __grid_co
 #pragma unroll
         for (int j = 0; j < 16; ++j) x[j] = __uint_as_float(v[j]);
         const bool full = vec && n0 + 16 <= p.N;
-        if (p.bias) {
+        if (p.bias && full && bias16) {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const float4 v = __ldg(reinterpret_cast<const float4*>(p.bias + n0) + j);
+            x[4 * j] += v.x; x[4 * j + 1] += v.y; x[4 * j + 2] += v.z; x[4 * j + 3] += v.w;
+          }
+        } else if (p.bias) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) if (full || n0 + j < p.N) x[j] += __ldg(p.bias + n0 + j);
         }

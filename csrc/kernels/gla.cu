@@ -24,6 +24,8 @@
 // which is exact algebra; the exponents stay within +-30 as long as no channel decays by more than e^-60 in a chunk.  A
 // chunk with a faster channel goes in four pieces of 16 tokens, and a piece with such a channel forms its 16 x 16 scores
 // from differences b_t - b_s <= 0, which cannot overflow.  S stays in registers as the accumulator of its product.
+// Few sequences: a portion is cut into segments that run side by side.  A first launch carries the state alone through
+// every segment but the last, from zero; in the second each segment starts from the decayed sum of the ones before it.
 //
 // This file is compiled without fast-math; the chunk kernel asks for the fast exponential and logarithm by name.
 #include "ptx.cuh"
@@ -43,6 +45,9 @@ struct GlaParams {
   void* out; int ldo;                      // [T, heads * vdim]
   float* raw;                              // chunk kernel with split columns: o before its norm, fp32 [T, heads * vdim]
   int min_q, max_q;                        // only sequences with min_q <= tokens in this call < max_q
+  int segs, carry;                         // segments per portion; carry: the launch that runs the states alone
+  float* seg_state;                        // [B, heads, segs, dim, vdim]: the initial state, then what segment j - 1 leaves
+  float* seg_decay;                        // [B, heads, segs, dim]: sum of log(alpha) over segment j - 1
   int* status;
 };
 
@@ -219,7 +224,7 @@ struct ChunkCfg {
   static constexpr int STAGE = kChunk * (2 * QS + VSS + RS);                         // q, k, v, a1 of a chunk, in values
   static constexpr int STAGES = DP <= 128 ? 2 : 1;
   static constexpr size_t B16 = (size_t)STAGES * STAGE + kChunk * AS + DP * VSS + DP * RS;
-  static constexpr size_t F32 = (size_t)kChunk * DP + 4 * DP + 3 * DP + DP + 2 * kChunk;
+  static constexpr size_t F32 = (size_t)kChunk * DP + 4 * DP + 3 * DP + DP + 2 * kChunk + VS;
   static constexpr size_t SMEM = B16 * 2 + F32 * 4;
 };
 
@@ -240,13 +245,18 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
   float* sPost = sMid + DP;                               //   and behind the update
   float* sBias = sPost + DP;
   float* sSS = sBias + DP;                                // [2][64] sums of squares of the output rows
+  float* sGain = sSS + 2 * kChunk;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int h = blockIdx.y, b = blockIdx.z, v0 = blockIdx.x * VS;
+  const int h = blockIdx.y, b = blockIdx.z, seg = blockIdx.x % p.segs, v0 = blockIdx.x / p.segs * VS;
   grid_dep_launch();
   const int start = p.cu_q[b], n = p.cu_q[b + 1] - start;
-  if (n < p.min_q || n >= p.max_q) { grid_dep_wait(); return; }
+  const int chunks = (n + kChunk - 1) / kChunk, per_seg = (chunks + p.segs - 1) / p.segs;
+  const int ch0 = seg * per_seg, ch1 = min(ch0 + per_seg, chunks);      // this CTA's chunks
+  if (n < p.min_q || n >= p.max_q || ch0 >= chunks || (p.carry && ch1 == chunks)) { grid_dep_wait(); return; }
   const int past = p.kv_lens[b] - n;
+  const bool alone = per_seg >= chunks;                   // one segment has all of the portion
   const int vw = min(VS, p.vdim - v0);
+  const bool even = (p.vdim & 1) == 0;
   const bool whole8 = (p.dim & 7) == 0 && (p.vdim & 7) == 0 && (p.rank & 7) == 0;
   float* st = p.state + ((size_t)gl_slot(p, b) * p.heads + h) * p.dim * p.vdim;
   const bf16* a2 = reinterpret_cast<const bf16*>(p.a2) + (size_t)h * p.dim * p.rank_ld;
@@ -258,6 +268,7 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
     sW[d * RS + r] = d < p.dim && r < p.rank ? a2[(size_t)d * p.rank_ld + r] : __float2bfloat16(0.f);
   }
   for (int d = tid; d < DP; d += 256) sBias[d] = d < p.dim ? p.bias[h * p.dim + d] : 0.f;
+  for (int c = tid; c < VS; c += 256) sGain[c] = c < vw ? p.gain[v0 + c] : 0.f;
   // the state: warp tile of MPW x 16 rows and NPW x 8 columns
   const int sm0 = (MW >= 8 ? warp * MPW : warp % MW) * 16, sn0 = (MW >= 8 ? 0 : warp / MW) * NPW * 8;
   float S[MPW][NPW][4];
@@ -268,9 +279,40 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int d = sm0 + m * 16 + (lane >> 2) + (e >> 1) * 8, c = sn0 + j * 8 + 2 * (lane & 3) + (e & 1);
-        S[m][j][e] = past > 0 && d < p.dim && c < vw ? st[(size_t)d * p.vdim + v0 + c] : 0.f;
+        S[m][j][e] = past > 0 && seg == 0 && (alone || p.carry) && d < p.dim && c < vw ? st[(size_t)d * p.vdim + v0 + c] : 0.f;
       }
   grid_dep_wait();
+  float* seg_s = p.seg_state + ((size_t)b * p.heads + h) * p.segs * p.dim * p.vdim;
+  float* seg_d = p.seg_decay + ((size_t)b * p.heads + h) * p.segs * p.dim;
+  float carried = 0.f;                                    // carry: sum of log(alpha) of channel tid over the segment
+  if (p.carry && seg == 0) {                // the pool is written while later segments still start: keep a copy
+#pragma unroll
+    for (int m = 0; m < MPW; ++m)
+#pragma unroll
+      for (int j = 0; j < NPW; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int d = sm0 + m * 16 + (lane >> 2) + (e >> 1) * 8, c = sn0 + j * 8 + 2 * (lane & 3) + (e & 1);
+          if (d < p.dim && c < vw) seg_s[(size_t)d * p.vdim + v0 + c] = S[m][j][e];
+        }
+  } else if (!alone && !p.carry) {
+    for (int k = seg == 0 ? 0 : 1; k <= seg; ++k)
+#pragma unroll
+      for (int m = 0; m < MPW; ++m)
+#pragma unroll
+        for (int e2 = 0; e2 < 2; ++e2) {
+          const int d = sm0 + m * 16 + (lane >> 2) + e2 * 8;
+          const float f = k > 1 && d < p.dim ? __expf(seg_d[(size_t)k * p.dim + d]) : 1.f;
+#pragma unroll
+          for (int j = 0; j < NPW; ++j)
+#pragma unroll
+            for (int e = 2 * e2; e < 2 * e2 + 2; ++e) {
+              const int c = sn0 + j * 8 + 2 * (lane & 3) + (e & 1);
+              const float v = d < p.dim && c < vw ? seg_s[((size_t)k * p.dim + d) * p.vdim + v0 + c] : 0.f;
+              S[m][j][e] = fmaf(S[m][j][e], f, v);
+            }
+        }
+  }
   __syncthreads();
 
   const bf16* x = reinterpret_cast<const bf16*>(p.x) + (size_t)start * p.ldx;
@@ -283,12 +325,15 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
     // rows behind the portion's end become zero
     auto part = [&](bf16* dst, int ld, int at, int width) {
       if (whole8) {
-        const int per = width >> 3;
-        for (int i = tid; i < kChunk * per; i += 256) {
-          const int r = i / per, c = (i % per) * 8;
-          const bf16* src = x + (size_t)(t0 + min(r, rows - 1)) * p.ldx + at + c;
+        const int per = width >> 3, dr = 256 / per, dc = 256 % per;
+        int r = tid / per, c = tid % per;
+        while (r < kChunk) {
+          const bf16* src = x + (size_t)(t0 + min(r, rows - 1)) * p.ldx + at + c * 8;
           const int bytes = r < rows ? 16 : 0;
-          asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + r * ld + c)), "l"(src), "r"(bytes) : "memory");
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + r * ld + c * 8)), "l"(src), "r"(bytes) : "memory");
+          r += dr;
+          c += dc;
+          if (c >= per) { c -= per; ++r; }
         }
       } else {
         for (int i = tid; i < kChunk * width; i += 256) {
@@ -297,18 +342,17 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
         }
       }
     };
-    part(sq, QS, h * p.dim, p.dim);
+    if (!p.carry) part(sq, QS, h * p.dim, p.dim);
     part(sk, QS, p.k_at + h * p.dim, p.dim);
     part(sv, VSS, p.v_at + h * p.vdim + v0, vw);
     part(sr, RS, p.a_at, p.rank);
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  const int chunks = (n + kChunk - 1) / kChunk;
-  load(0);
-  for (int ch = 0; ch < chunks; ++ch) {
+  load(ch0);
+  for (int ch = ch0; ch < ch1; ++ch) {
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
-    if (Cfg::STAGES > 1 && ch + 1 < chunks) load(ch + 1);
+    if (Cfg::STAGES > 1 && ch + 1 < ch1) load(ch + 1);
     bf16* sq = stage0 + (Cfg::STAGES > 1 ? (ch & 1) * Cfg::STAGE : 0);
     bf16* sk = sq + kChunk * QS;
     bf16* sv = sk + kChunk * QS;
@@ -364,6 +408,7 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
       *reinterpret_cast<float2*>(sT + g * DP + 2 * pr) = c;
     }
     __syncthreads();
+    if (p.carry && tid < p.dim) carried += sT[tid] + sT[DP + tid] + sT[2 * DP + tid] + sT[3 * DP + tid];
     bool ok = true;
     for (int d = tid; d < DP; d += 256) ok = ok && sT[d] + sT[DP + d] + sT[2 * DP + d] + sT[3 * DP + d] >= -kMaxDecay;
     const bool one = __syncthreads_and(ok);               // the whole chunk in one piece
@@ -371,6 +416,7 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
     float O[VS / 16][4];
 #pragma unroll
     for (int j = 0; j < VS / 16; ++j) O[j][0] = O[j][1] = O[j][2] = O[j][3] = 0.f;
+    uint32_t gate[VS / 16][2];                             // of this warp's output values
     for (int pc = 0; pc < pieces; ++pc) {
       const int g_lo = one ? 0 : pc, g_hi = one ? 4 : pc + 1;       // groups of 16 rows in this piece
       bool gentle = true;
@@ -378,7 +424,7 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
         bool k = true;
         for (int d = tid; d < DP; d += 256) k = k && sT[pc * DP + d] >= -kMaxDecay;
         gentle = __syncthreads_and(k);
-        if (!gentle) {
+        if (!gentle && !p.carry) {
           // scores of the piece from differences of running sums; 256 pairs of rows, a warp at a time
           for (int i = warp; i < kPiece * kPiece; i += 8) {
             const int t = pc * kPiece + i / kPiece, s = pc * kPiece + i % kPiece;
@@ -419,8 +465,11 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
           bb.x += base.x; bb.y += base.y;
           uint32_t* qp = reinterpret_cast<uint32_t*>(sq + t * QS + 2 * pr);
           uint32_t* kp = reinterpret_cast<uint32_t*>(sk + t * QS + 2 * pr);
-          const float2 q = gl_unpack(*qp), k = gl_unpack(*kp);
-          *qp = gl_pack(q.x * p.scale * __expf(bb.x - qr.x), q.y * p.scale * __expf(bb.y - qr.y));
+          const float2 k = gl_unpack(*kp);
+          if (!p.carry) {
+            const float2 q = gl_unpack(*qp);
+            *qp = gl_pack(q.x * p.scale * __expf(bb.x - qr.x), q.y * p.scale * __expf(bb.y - qr.y));
+          }
           *kp = gl_pack(k.x * __expf(kr.x - bb.x), k.y * __expf(kr.y - bb.y));
         }
       }
@@ -434,12 +483,14 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
         for (int j = 0; j < NPW; ++j) {
           const int c = sn0 + j * 8 + 2 * (lane & 3);
           S[m][j][0] *= f0; S[m][j][1] *= f0; S[m][j][2] *= f1; S[m][j][3] *= f1;
-          *reinterpret_cast<uint32_t*>(sS + d * VSS + c) = gl_pack(S[m][j][0], S[m][j][1]);
-          *reinterpret_cast<uint32_t*>(sS + (d + 8) * VSS + c) = gl_pack(S[m][j][2], S[m][j][3]);
+          if (!p.carry) {
+            *reinterpret_cast<uint32_t*>(sS + d * VSS + c) = gl_pack(S[m][j][0], S[m][j][1]);
+            *reinterpret_cast<uint32_t*>(sS + (d + 8) * VSS + c) = gl_pack(S[m][j][2], S[m][j][3]);
+          }
           if (!gentle) { S[m][j][0] *= m0; S[m][j][1] *= m0; S[m][j][2] *= m1; S[m][j][3] *= m1; }
         }
       }
-      const bool my_rows = mt >= g_lo && mt < g_hi;
+      const bool my_rows = mt >= g_lo && mt < g_hi && !p.carry;
       if (gentle && my_rows) {
         // columns of this warp: of the whole chunk its half (32), of a piece 8 of its 16
         if (one) {
@@ -490,6 +541,16 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
         }
       }
       __syncthreads();
+      if (pc == 0 && even && !p.raw && !p.carry) {         // fetched here, used behind the products
+#pragma unroll
+        for (int j = 0; j < VS / 16; ++j)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int c = half * (VS / 2) + j * 8 + 2 * (lane & 3), r = mt * 16 + (lane >> 2) + e * 8;
+            gate[j][e] = r < rows && c < p.vdim ? __ldg(reinterpret_cast<const uint32_t*>(
+                x + (size_t)(ch * kChunk + r) * p.ldx + p.g_at + h * p.vdim + c)) : 0u;
+          }
+      }
       // O = q^ S + A V, rows of this warp, half of the columns
       if (my_rows) {
 #pragma unroll
@@ -542,6 +603,7 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
       }
       if (pc + 1 < pieces) __syncthreads();               // the next piece writes sS, sA and the factors again
     }
+    if (p.carry) { __syncthreads(); if (Cfg::STAGES == 1 && ch + 1 < ch1) load(ch + 1); continue; }
     // norm and gate (or the bare output, when other CTAs have the head's other columns)
     const int r0 = mt * 16 + (lane >> 2), r1 = r0 + 8;
     if (p.raw) {
@@ -571,10 +633,10 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
       __syncthreads();
       const float i0 = rsqrtf((sSS[r0] + sSS[kChunk + r0]) / (float)p.vdim + p.eps);
       const float i1 = rsqrtf((sSS[r1] + sSS[kChunk + r1]) / (float)p.vdim + p.eps);
-      const bool even = (p.vdim & 1) == 0;
 #pragma unroll
       for (int j = 0; j < VS / 16; ++j) {
         const int c = half * (VS / 2) + j * 8 + 2 * (lane & 3);
+        const float w0 = sGain[c], w1 = sGain[c + 1];
 #pragma unroll
         for (int e = 0; e < 4; e += 2) {
           const int r = e ? r1 : r0;
@@ -583,23 +645,27 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
           const bf16* gp = x + (size_t)(ch * kChunk + r) * p.ldx + p.g_at + h * p.vdim + c;
           bf16* op = reinterpret_cast<bf16*>(p.out) + (size_t)(start + ch * kChunk + r) * p.ldo + h * p.vdim + c;
           if (even) {
-            const float2 g = gl_unpack(*reinterpret_cast<const uint32_t*>(gp));
-            *reinterpret_cast<uint32_t*>(op) = gl_pack(O[j][e] * inv * p.gain[c] * __fdividef(g.x, 1.f + __expf(-g.x)),
-                                                       O[j][e + 1] * inv * p.gain[c + 1] * __fdividef(g.y, 1.f + __expf(-g.y)));
+            const float2 g = gl_unpack(gate[j][e >> 1]);
+            *reinterpret_cast<uint32_t*>(op) = gl_pack(O[j][e] * inv * w0 * __fdividef(g.x, 1.f + __expf(-g.x)),
+                                                       O[j][e + 1] * inv * w1 * __fdividef(g.y, 1.f + __expf(-g.y)));
           } else {
 #pragma unroll
             for (int k = 0; k < 2; ++k)
               if (c + k < p.vdim) {
                 const float g = __bfloat162float(gp[k]);
-                op[k] = __float2bfloat16(O[j][e + k] * inv * p.gain[c + k] * __fdividef(g, 1.f + __expf(-g)));
+                op[k] = __float2bfloat16(O[j][e + k] * inv * (k ? w1 : w0) * __fdividef(g, 1.f + __expf(-g)));
               }
           }
         }
       }
     }
     __syncthreads();                                       // everything of this chunk has been read
-    if (Cfg::STAGES == 1 && ch + 1 < chunks) load(ch + 1);
+    if (Cfg::STAGES == 1 && ch + 1 < ch1) load(ch + 1);
   }
+  if (p.carry) {
+    st = seg_s + (size_t)(seg + 1) * p.dim * p.vdim;
+    if (v0 == 0 && tid < p.dim) seg_d[(size_t)(seg + 1) * p.dim + tid] = carried;
+  } else if (ch1 < chunks) return;                         // the last segment leaves the state
 #pragma unroll
   for (int m = 0; m < MPW; ++m)
 #pragma unroll
@@ -696,7 +762,14 @@ static int launch_chunk(const GlaParams& p, cudaStream_t st) {
       return 3000 + (int)cudaGetLastError();
     attr_set = true;
   }
-  cudaError_t e = launch_pdl(gla_chunk_kernel<DP, VS, RP>, dim3((p.vdim + VS - 1) / VS, p.heads, p.B), dim3(256), Cfg::SMEM, st, p);
+  const dim3 grid((p.vdim + VS - 1) / VS * p.segs, p.heads, p.B);
+  cudaError_t e = cudaSuccess;
+  if (p.segs > 1) {
+    GlaParams q = p;
+    q.carry = 1;
+    e = launch_pdl(gla_chunk_kernel<DP, VS, RP>, grid, dim3(256), Cfg::SMEM, st, q);
+  }
+  if (e == cudaSuccess) e = launch_pdl(gla_chunk_kernel<DP, VS, RP>, grid, dim3(256), Cfg::SMEM, st, p);
   return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }
 template <int DP, int VS>
@@ -725,22 +798,26 @@ extern "C" int xft_gla_step(const void* x, int ldx, int k_at, int v_at, int g_at
   if (heads > 65535 || B > 65535 || (vdim + columns - 1) / columns > 8 || (size_t)(3 * dim + rank_ld) * 4 > 40000) return -2;
   if (((uintptr_t)a2 | (uintptr_t)state) & 15) return -3;
   GlaParams p{x, ldx, k_at, v_at, g_at, a_at, heads, dim, vdim, rank, rank_ld, a2, bias, 1.f / tau, scale, eps, gain, state, state_slots,
-              num_states, cu_q, kv_lens, B, out, ldo, nullptr, min_q, max_q, status};
+              num_states, cu_q, kv_lens, B, out, ldo, nullptr, min_q, max_q, 1, 0, nullptr, nullptr, status};
   return f32 ? step_columns<float>(p, columns, st) : step_columns<bf16>(p, columns, st);
 }
 
 // bf16 portions.  raw: fp32 [T, heads * vdim], needed when a head has more columns than xft_gla_chunk_columns says.
+// segs > 1: portions are cut into so many segments (two launches), with scratch seg_state fp32 [B, heads, segs, dim, vdim] and
+// seg_decay fp32 [B, heads, segs, dim].
 extern "C" int xft_gla_chunk(const void* x, int ldx, int k_at, int v_at, int g_at, int a_at, int heads, int dim, int vdim, int rank,
                              int rank_ld, const void* a2, const float* bias, float tau, float scale, float eps, const float* gain,
                              float* state, const int* state_slots, int num_states, const int* cu_q, const int* kv_lens, int B, int T,
-                             void* out, int ldo, float* raw, int min_q, int max_q, int* status, cudaStream_t st) {
+                             void* out, int ldo, float* raw, int min_q, int max_q, int segs, float* seg_state, float* seg_decay,
+                             int* status, cudaStream_t st) {
   if (B <= 0 || T <= 0) return 0;
+  if (segs < 1 || (segs > 1 && (!seg_state || !seg_decay))) return -4;
   const int cols = xft_gla_chunk_columns(dim, vdim, rank);
   if (!cols || heads <= 0 || vdim <= 0 || rank <= 0 || rank_ld < rank || tau <= 0.f || num_states <= 0) return -1;
   if (heads > 65535 || B > 65535 || (vdim > cols && !raw)) return -2;
   if ((ldx & 7) || (k_at & 7) || (v_at & 7) || (g_at & 7) || (a_at & 7) || ((uintptr_t)x & 15)) return -3;
   GlaParams p{x, ldx, k_at, v_at, g_at, a_at, heads, dim, vdim, rank, rank_ld, a2, bias, 1.f / tau, scale, eps, gain, state, state_slots,
-              num_states, cu_q, kv_lens, B, out, ldo, vdim > cols ? raw : nullptr, min_q, max_q, status};
+              num_states, cu_q, kv_lens, B, out, ldo, vdim > cols ? raw : nullptr, min_q, max_q, segs, 0, seg_state, seg_decay, status};
   int r;
   if (dim > 128) r = launch_chunk<256, 64, 16>(p, st);
   else if (dim > 64) r = cols == 64 ? chunk_rank<128, 64>(p, st) : chunk_rank<128, 128>(p, st);

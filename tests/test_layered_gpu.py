@@ -248,6 +248,13 @@ def test_gated_linear_decays(dtype, tol, tau, around, spread):
     M.gated_linear(_dev(), dtype, tol, 1, 136, 40, 16, tau, (90,), (1000,), around, spread)
 
 
+@pytest.mark.parametrize("H,d,dv,tau", [(2, 64, 64, 16.0), (1, 128, 128, 4.0), (1, 136, 100, 16.0), (2, 24, 40, 0.5)])
+@pytest.mark.parametrize("sizes", [(2000,), (900, 1400)])
+def test_gated_linear_segments(H, d, dv, tau, sizes):
+    """Few long portions go in segments that run side by side, beside portions of one chunk and of one token."""
+    M.gated_linear(_dev(), torch.bfloat16, 1.5e-2, H, d, dv, 16, tau, (1500, 70, 1130, 33, 3), sizes)
+
+
 @pytest.mark.parametrize("columns", [32, 64, 128])
 def test_gated_linear_step_columns(monkeypatch, columns):
     from xfastertransformer_b200.ops import native_linear

@@ -55,6 +55,13 @@ def step_columns(units: int, dim: int, vdim: int) -> int:
     return best
 
 
+def segments(units: int, longest: int) -> int:
+    """Segments that run side by side where `units` CTAs alone would leave SMs idle: their two passes over a portion cost about
+    one and a half, so it takes more than two of them, of at least four chunks each."""
+    n = min(SMS // max(units, 1), longest // (4 * 64), 32)
+    return n if n > 1 else 1
+
+
 def gated_linear(x, d, w, eps, state, state_slots, cu_q, kv_lens, meta=None):
     cu, lens, B, decode, _ = N.batch_arrays(cu_q, kv_lens, meta, x.device)
     assert x.dim() == 2 and x.stride(1) == 1 and state.dtype == torch.float32 and state.is_contiguous()
@@ -74,9 +81,13 @@ def gated_linear(x, d, w, eps, state, state_slots, cu_q, kv_lens, meta=None):
         sizes = [cu_q[i + 1] - cu_q[i] for i in range(B)]
         if max(sizes) >= least:
             raw = torch.empty(T, d.heads * d.vdim, dtype=torch.float32, device=x.device) if d.vdim > columns else None
-            N._check(_fn("xft_gla_chunk")(*common, T, N._p(out), out.stride(0), N._p(raw), least, NO_LIMIT, N._p(ws.status),
-                                          N._stream()), "gla_chunk")
-            ws.launches += 1 if raw is None else 2
+            long = sum(n >= least for n in sizes)
+            segs = segments(long * d.heads * ((d.vdim + columns - 1) // columns), max(sizes))
+            ss, sd = (torch.empty(B, d.heads, segs, n, dtype=torch.float32, device=x.device) if segs > 1 else None
+                      for n in (d.dim * d.vdim, d.dim))
+            N._check(_fn("xft_gla_chunk")(*common, T, N._p(out), out.stride(0), N._p(raw), least, NO_LIMIT, segs, N._p(ss), N._p(sd),
+                                          N._p(ws.status), N._stream()), "gla_chunk")
+            ws.launches += 1 + (raw is not None) + (segs > 1)
         if min(sizes) >= least:
             return out
     N._check(_fn("xft_gla_step")(*common, N._p(out), out.stride(0), 1, least, step_columns(B * d.heads, d.dim, d.vdim), int(exact),
