@@ -47,7 +47,7 @@ struct GlaParams {
   int min_q, max_q;                        // only sequences with min_q <= tokens in this call < max_q
   int segs, carry;                         // segments per portion; carry: the launch that runs the states alone
   float* seg_state;                        // [B, heads, segs, dim, vdim]: the initial state, then what segment j - 1 leaves
-  float* seg_decay;                        // [B, heads, segs, dim]: sum of log(alpha) over segment j - 1
+  float* seg_decay;                        // [B, heads, segs, dim]: sum of log2(alpha) over segment j - 1
   int* status;
 };
 
@@ -217,35 +217,49 @@ __device__ __forceinline__ float2 gl_unpack(uint32_t v) { return __bfloat1622flo
 constexpr int kChunk = 64, kPiece = 16;
 constexpr float kMaxDecay = 60.f;
 
-// DP: padded dim, VS: columns of the state per CTA, RP: padded rank
+// approximate instructions of the special-function unit, denormals flushed
+__device__ __forceinline__ float gl_ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+__device__ __forceinline__ float gl_lg2(float x) { float y; asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+__device__ __forceinline__ float gl_rcp(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+constexpr float kLog2e = 1.4426950408889634f;
+// x * sigmoid(x); e^-x past the largest float makes it 0
+__device__ __forceinline__ float gl_silu(float x) { return x * gl_rcp(1.f + gl_ex2(-x * kLog2e)); }
+
+// DP: padded dim, VS: columns of the state per CTA, RP: padded rank.  16 warps: products of rows take 16 rows (of four) and a
+// quarter of the columns per warp, the state is divided by 16 rows and, when they are fewer than 16 x 16, by columns.
+constexpr int kChunkThreads = 512;
 template <int DP, int VS, int RP>
 struct ChunkCfg {
   static constexpr int QS = DP + 8, VSS = VS + 8, RS = RP + 8, AS = kChunk + 8;     // row strides (16 bytes of padding)
+  static constexpr int BS = DP + 8;
   static constexpr int STAGE = kChunk * (2 * QS + VSS + RS);                         // q, k, v, a1 of a chunk, in values
   static constexpr int STAGES = DP <= 128 ? 2 : 1;
   static constexpr size_t B16 = (size_t)STAGES * STAGE + kChunk * AS + DP * VSS + DP * RS;
-  static constexpr size_t F32 = (size_t)kChunk * DP + 4 * DP + 3 * DP + DP + 2 * kChunk + VS;
+  static constexpr size_t F32 = (size_t)kChunk * BS + 8 * DP + 4 * DP + 4 * kChunk + VS;
   static constexpr size_t SMEM = B16 * 2 + F32 * 4;
 };
 
 template <int DP, int VS, int RP>
-__global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
+__global__ void __launch_bounds__(kChunkThreads, 1) gla_chunk_kernel(const GlaParams p) {
   using Cfg = ChunkCfg<DP, VS, RP>;
-  constexpr int QS = Cfg::QS, VSS = Cfg::VSS, RS = Cfg::RS, AS = Cfg::AS;
-  constexpr int MW = DP / 16, MPW = MW >= 8 ? MW / 8 : 1, NGRP = MW >= 8 ? 1 : 8 / MW, NPW = VS / 8 / NGRP;
+  constexpr int NT = kChunkThreads;
+  constexpr int QS = Cfg::QS, VSS = Cfg::VSS, RS = Cfg::RS, AS = Cfg::AS, BS = Cfg::BS;
+  constexpr int MW = DP / 16, NGRP = 16 / MW, NPW = VS / 8 / NGRP;     // state: m-tiles, column groups, n-tiles per warp
+  constexpr int NO = VS / 32, NZ = DP / 32;                            // n-tiles of a quarter of the columns
+  static_assert(MW <= 16 && NPW >= 2 && NPW % 2 == 0 && NO % 2 == 0 && NZ % 2 == 0, "warp tiles");
   extern __shared__ __align__(16) uint8_t gc_raw[];
   bf16* stage0 = reinterpret_cast<bf16*>(gc_raw);
   bf16* sA = stage0 + Cfg::STAGES * Cfg::STAGE;           // scores [64][AS]
   bf16* sS = sA + kChunk * AS;                            // state as an operand [DP][VSS]
   bf16* sW = sS + DP * VSS;                               // a2 of this head [DP][RS]
-  float* sB = reinterpret_cast<float*>(sW + DP * RS);     // running sums of log(alpha) [64][DP], restarting every 16 rows
-  float* sT = sB + kChunk * DP;                           // their totals [4][DP]
-  float* sPre = sT + 4 * DP;                              // factors of the state's rows: in front of the operand,
+  float* sB = reinterpret_cast<float*>(sW + DP * RS);     // running sums of log2(alpha) [64][BS], restarting every 8 rows
+  float* sT = sB + kChunk * BS;                           // their totals [8][DP]
+  float* sPre = sT + 8 * DP;                              // factors of the state's rows: in front of the operand,
   float* sMid = sPre + DP;                                //   behind it,
-  float* sPost = sMid + DP;                               //   and behind the update
+  float* sPost = sMid + DP;                               //   and behind the update (applied with the next sPre)
   float* sBias = sPost + DP;
-  float* sSS = sBias + DP;                                // [2][64] sums of squares of the output rows
-  float* sGain = sSS + 2 * kChunk;
+  float* sSS = sBias + DP;                                // [4][64] sums of squares of the output rows
+  float* sGain = sSS + 4 * kChunk;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int h = blockIdx.y, b = blockIdx.z, seg = blockIdx.x % p.segs, v0 = blockIdx.x / p.segs * VS;
   grid_dep_launch();
@@ -262,56 +276,40 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
   const bf16* a2 = reinterpret_cast<const bf16*>(p.a2) + (size_t)h * p.dim * p.rank_ld;
 
   // weights, and zeros where nothing is ever loaded
-  for (int i = tid; i < Cfg::STAGES * Cfg::STAGE / 8; i += 256) reinterpret_cast<uint4*>(stage0)[i] = make_uint4(0, 0, 0, 0);
-  for (int i = tid; i < DP * RP; i += 256) {
+  for (int i = tid; i < Cfg::STAGES * Cfg::STAGE / 8; i += NT) reinterpret_cast<uint4*>(stage0)[i] = make_uint4(0, 0, 0, 0);
+  for (int i = tid; i < DP * RP; i += NT) {
     const int d = i / RP, r = i % RP;
     sW[d * RS + r] = d < p.dim && r < p.rank ? a2[(size_t)d * p.rank_ld + r] : __float2bfloat16(0.f);
   }
-  for (int d = tid; d < DP; d += 256) sBias[d] = d < p.dim ? p.bias[h * p.dim + d] : 0.f;
-  for (int c = tid; c < VS; c += 256) sGain[c] = c < vw ? p.gain[v0 + c] : 0.f;
-  // the state: warp tile of MPW x 16 rows and NPW x 8 columns
-  const int sm0 = (MW >= 8 ? warp * MPW : warp % MW) * 16, sn0 = (MW >= 8 ? 0 : warp / MW) * NPW * 8;
-  float S[MPW][NPW][4];
-#pragma unroll
-  for (int m = 0; m < MPW; ++m)
+  for (int d = tid; d < DP; d += NT) { sBias[d] = d < p.dim ? p.bias[h * p.dim + d] : 0.f; sPost[d] = 1.f; }
+  for (int c = tid; c < VS; c += NT) sGain[c] = c < vw ? p.gain[v0 + c] : 0.f;
+  // the state: warp tile of 16 rows and NPW x 8 columns
+  const int sd = (warp % MW) * 16 + (lane >> 2), sn0 = warp / MW * NPW * 8, sc = sn0 + 2 * (lane & 3);
+  float S[NPW][4];                                        // element e: row sd + 8 (e >> 1), column sc + 8 j + (e & 1)
+  auto each_state = [&](auto f) {
 #pragma unroll
     for (int j = 0; j < NPW; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int d = sm0 + m * 16 + (lane >> 2) + (e >> 1) * 8, c = sn0 + j * 8 + 2 * (lane & 3) + (e & 1);
-        S[m][j][e] = past > 0 && seg == 0 && (alone || p.carry) && d < p.dim && c < vw ? st[(size_t)d * p.vdim + v0 + c] : 0.f;
+        const int d = sd + (e >> 1) * 8, c = sc + j * 8 + (e & 1);
+        f(S[j][e], (size_t)d * p.vdim + v0 + c, d < p.dim && c < vw, e >> 1);
       }
+  };
+  each_state([&](float& v, size_t at, bool in, int) { v = past > 0 && seg == 0 && (alone || p.carry) && in ? st[at] : 0.f; });
   grid_dep_wait();
   float* seg_s = p.seg_state + ((size_t)b * p.heads + h) * p.segs * p.dim * p.vdim;
   float* seg_d = p.seg_decay + ((size_t)b * p.heads + h) * p.segs * p.dim;
-  float carried = 0.f;                                    // carry: sum of log(alpha) of channel tid over the segment
-  if (p.carry && seg == 0) {                // the pool is written while later segments still start: keep a copy
-#pragma unroll
-    for (int m = 0; m < MPW; ++m)
-#pragma unroll
-      for (int j = 0; j < NPW; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int d = sm0 + m * 16 + (lane >> 2) + (e >> 1) * 8, c = sn0 + j * 8 + 2 * (lane & 3) + (e & 1);
-          if (d < p.dim && c < vw) seg_s[(size_t)d * p.vdim + v0 + c] = S[m][j][e];
-        }
+  float carried = 0.f;                                    // carry: sum of log2(alpha) of channel tid over the segment
+  if (p.carry && seg == 0) {                              // the pool is written while later segments still start: keep a copy
+    each_state([&](float& v, size_t at, bool in, int) { if (in) seg_s[at] = v; });
   } else if (!alone && !p.carry) {
-    for (int k = seg == 0 ? 0 : 1; k <= seg; ++k)
+    for (int k = seg == 0 ? 0 : 1; k <= seg; ++k) {
+      float f[2];
 #pragma unroll
-      for (int m = 0; m < MPW; ++m)
-#pragma unroll
-        for (int e2 = 0; e2 < 2; ++e2) {
-          const int d = sm0 + m * 16 + (lane >> 2) + e2 * 8;
-          const float f = k > 1 && d < p.dim ? __expf(seg_d[(size_t)k * p.dim + d]) : 1.f;
-#pragma unroll
-          for (int j = 0; j < NPW; ++j)
-#pragma unroll
-            for (int e = 2 * e2; e < 2 * e2 + 2; ++e) {
-              const int c = sn0 + j * 8 + 2 * (lane & 3) + (e & 1);
-              const float v = d < p.dim && c < vw ? seg_s[((size_t)k * p.dim + d) * p.vdim + v0 + c] : 0.f;
-              S[m][j][e] = fmaf(S[m][j][e], f, v);
-            }
-        }
+      for (int e = 0; e < 2; ++e) f[e] = k > 1 && sd + e * 8 < p.dim ? gl_ex2(seg_d[(size_t)k * p.dim + sd + e * 8]) : 1.f;
+      const float* from = seg_s + (size_t)k * p.dim * p.vdim;
+      each_state([&](float& v, size_t at, bool in, int e) { v = fmaf(v, f[e], in ? from[at] : 0.f); });
+    }
   }
   __syncthreads();
 
@@ -325,7 +323,7 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
     // rows behind the portion's end become zero
     auto part = [&](bf16* dst, int ld, int at, int width) {
       if (whole8) {
-        const int per = width >> 3, dr = 256 / per, dc = 256 % per;
+        const int per = width >> 3, dr = NT / per, dc = NT % per;
         int r = tid / per, c = tid % per;
         while (r < kChunk) {
           const bf16* src = x + (size_t)(t0 + min(r, rows - 1)) * p.ldx + at + c * 8;
@@ -336,7 +334,7 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
           if (c >= per) { c -= per; ++r; }
         }
       } else {
-        for (int i = tid; i < kChunk * width; i += 256) {
+        for (int i = tid; i < kChunk * width; i += NT) {
           const int r = i / width, c = i % width;
           dst[r * ld + c] = r < rows ? x[(size_t)(t0 + r) * p.ldx + at + c] : __float2bfloat16(0.f);
         }
@@ -348,6 +346,13 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
     part(sr, RS, p.a_at, p.rank);
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
+  // fragment addresses: A (rows x k) and B (columns x k) row-major, B (k x columns) through a transposing load
+  const int fa_r = (lane & 7) + ((lane >> 3) & 1) * 8, fa_c = (lane >> 4) * 8;
+  const int fb_r = (lane & 7) + ((lane >> 4) & 1) * 8, fb_c = ((lane >> 3) & 1) * 8;
+  const int mt = warp & 3, quarter = warp >> 2;           // this warp's 16 rows of the chunk, and its part of the columns
+  const int r0 = mt * 16 + (lane >> 2), cc = 2 * (lane & 3);
+  const float tau2 = p.inv_tau * kLog2e, scale2 = log2f(p.scale);
+
   load(ch0);
   for (int ch = ch0; ch < ch1; ++ch) {
     asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -358,80 +363,90 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
     bf16* sv = sk + kChunk * QS;
     bf16* sr = sv + kChunk * VSS;
     const int rows = min(kChunk, n - ch * kChunk);
-    const int mt = warp & 3, half = warp >> 2;            // this warp's 16 rows of the chunk, and half of the columns
 
-    // log(alpha) of every row and channel
+    // log2(alpha) of every row and channel
     {
-      float z[DP / 16][4];
+      float z[NZ][4];
 #pragma unroll
-      for (int j = 0; j < DP / 16; ++j) z[j][0] = z[j][1] = z[j][2] = z[j][3] = 0.f;
+      for (int j = 0; j < NZ; ++j) z[j][0] = z[j][1] = z[j][2] = z[j][3] = 0.f;
 #pragma unroll
       for (int ks = 0; ks < RP / 16; ++ks) {
         uint32_t a[4];
-        gl_ldsm(a, sr + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * RS + ks * 16 + (lane >> 4) * 8);
+        gl_ldsm(a, sr + (mt * 16 + fa_r) * RS + ks * 16 + fa_c);
 #pragma unroll
-        for (int j = 0; j < DP / 16; j += 2) {
+        for (int j = 0; j < NZ; j += 2) {
           uint32_t w[4];
-          gl_ldsm(w, sW + (half * (DP / 2) + j * 8 + (lane & 7) + ((lane >> 4) & 1) * 8) * RS + ks * 16 + ((lane >> 3) & 1) * 8);
+          gl_ldsm(w, sW + (quarter * (DP / 4) + j * 8 + fb_r) * RS + ks * 16 + fb_c);
           gl_mma(z[j], a, w[0], w[1]);
-          if (j + 1 < DP / 16) gl_mma(z[j + 1 < DP / 16 ? j + 1 : j], a, w[2], w[3]);
+          gl_mma(z[j + 1], a, w[2], w[3]);
         }
       }
 #pragma unroll
-      for (int j = 0; j < DP / 16; ++j)
+      for (int j = 0; j < NZ; ++j) {
+        const int d = quarter * (DP / 4) + j * 8 + cc;
+        const float2 bias = *reinterpret_cast<const float2*>(sBias + d);
 #pragma unroll
-        for (int e = 0; e < 4; e += 2) {
-          const int r = mt * 16 + (lane >> 2) + (e >> 1) * 8, d = half * (DP / 2) + j * 8 + 2 * (lane & 3);
-          float2 la;
-          float* l = &la.x;
+        for (int e = 0; e < 2; ++e) {
+          const int r = r0 + e * 8;
+          float l[2];
 #pragma unroll
           for (int k = 0; k < 2; ++k) {
-            const float zz = z[j][e + k] + sBias[d + k];
-            l[k] = r < rows && d + k < p.dim ? (fminf(zz, 0.f) - __logf(1.f + __expf(-fabsf(zz)))) * p.inv_tau : 0.f;
+            const float zz = z[j][2 * e + k] + (k ? bias.y : bias.x);
+            const float la = fminf(zz, 0.f) * tau2 - gl_lg2(1.f + gl_ex2(-fabsf(zz) * kLog2e)) * p.inv_tau;
+            l[k] = r < rows && d + k < p.dim ? la : 0.f;
           }
-          *reinterpret_cast<float2*>(sB + r * DP + d) = la;
+          *reinterpret_cast<float2*>(sB + r * BS + d) = make_float2(l[0], l[1]);
         }
+      }
     }
     __syncthreads();
-    // running sums within every 16 rows, and their totals
-    for (int it = tid; it < 2 * DP; it += 256) {
+    // running sums within every 8 rows, and their totals
+    for (int it = tid; it < 4 * DP; it += NT) {
       const int pr = it % (DP / 2), g = it / (DP / 2);
-      float2 c = make_float2(0.f, 0.f);
-      float2 v[kPiece];
+      float2* col = reinterpret_cast<float2*>(sB + g * 8 * BS + 2 * pr);
+      float2 c = make_float2(0.f, 0.f), v[8];
 #pragma unroll
-      for (int r = 0; r < kPiece; ++r) v[r] = *reinterpret_cast<const float2*>(sB + (g * kPiece + r) * DP + 2 * pr);
+      for (int r = 0; r < 8; ++r) v[r] = col[r * (BS / 2)];
 #pragma unroll
-      for (int r = 0; r < kPiece; ++r) {
+      for (int r = 0; r < 8; ++r) {
         c.x += v[r].x; c.y += v[r].y;
-        *reinterpret_cast<float2*>(sB + (g * kPiece + r) * DP + 2 * pr) = c;
+        col[r * (BS / 2)] = c;
       }
       *reinterpret_cast<float2*>(sT + g * DP + 2 * pr) = c;
     }
     __syncthreads();
-    if (p.carry && tid < p.dim) carried += sT[tid] + sT[DP + tid] + sT[2 * DP + tid] + sT[3 * DP + tid];
     bool ok = true;
-    for (int d = tid; d < DP; d += 256) ok = ok && sT[d] + sT[DP + d] + sT[2 * DP + d] + sT[3 * DP + d] >= -kMaxDecay;
+    for (int d = tid; d < DP; d += NT) {
+      float t = 0.f;
+#pragma unroll
+      for (int g = 0; g < 8; ++g) t += sT[g * DP + d];
+      carried += t;
+      ok = t >= -kMaxDecay * kLog2e;
+    }
     const bool one = __syncthreads_and(ok);               // the whole chunk in one piece
     const int pieces = one ? 1 : (rows + kPiece - 1) / kPiece;
-    float O[VS / 16][4];
+    float O[NO][4];
 #pragma unroll
-    for (int j = 0; j < VS / 16; ++j) O[j][0] = O[j][1] = O[j][2] = O[j][3] = 0.f;
-    uint32_t gate[VS / 16][2];                             // of this warp's output values
+    for (int j = 0; j < NO; ++j) O[j][0] = O[j][1] = O[j][2] = O[j][3] = 0.f;
+    uint32_t gate[NO][2];                                  // of this warp's output values
     for (int pc = 0; pc < pieces; ++pc) {
       const int g_lo = one ? 0 : pc, g_hi = one ? 4 : pc + 1;       // groups of 16 rows in this piece
       bool gentle = true;
       if (!one) {
         bool k = true;
-        for (int d = tid; d < DP; d += 256) k = k && sT[pc * DP + d] >= -kMaxDecay;
+        for (int d = tid; d < DP; d += NT) k = sT[2 * pc * DP + d] + sT[(2 * pc + 1) * DP + d] >= -kMaxDecay * kLog2e;
         gentle = __syncthreads_and(k);
         if (!gentle && !p.carry) {
           // scores of the piece from differences of running sums; 256 pairs of rows, a warp at a time
-          for (int i = warp; i < kPiece * kPiece; i += 8) {
+          for (int i = warp; i < kPiece * kPiece; i += NT / 32) {
             const int t = pc * kPiece + i / kPiece, s = pc * kPiece + i % kPiece;
             float a = 0.f;
             if (s <= t)
-              for (int d = lane; d < p.dim; d += 32)
-                a += __bfloat162float(sq[t * QS + d]) * __bfloat162float(sk[s * QS + d]) * __expf(sB[t * DP + d] - sB[s * DP + d]);
+              for (int d = lane; d < p.dim; d += 32) {
+                const float between = (t & 8) && !(s & 8) ? sT[2 * pc * DP + d] : 0.f;       // the sums restart between s and t
+                a += __bfloat162float(sq[t * QS + d]) * __bfloat162float(sk[s * QS + d]) *
+                     gl_ex2(sB[t * BS + d] - sB[s * BS + d] + between);
+              }
 #pragma unroll
             for (int m = 16; m > 0; m >>= 1) a += __shfl_xor_sync(0xffffffffu, a, m);
             if (lane == 0) sA[t * AS + s] = __float2bfloat16(a * p.scale);
@@ -440,138 +455,112 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
         }
       }
       // q^ and k^ in place; the factors of the state's rows
-      for (int it = tid; it < 2 * DP; it += 256) {
+      for (int it = tid; it < 4 * DP; it += NT) {
         const int pr = it % (DP / 2), g = it / (DP / 2);
-        if (g < g_lo || g >= g_hi) continue;
+        if (g < 2 * g_lo || g >= 2 * g_hi) continue;
         float2 base = make_float2(0.f, 0.f), tot = make_float2(0.f, 0.f);
-        for (int j = g_lo; j < g_hi; ++j) {
+        for (int j = 2 * g_lo; j < 2 * g_hi; ++j) {
           const float2 v = *reinterpret_cast<const float2*>(sT + j * DP + 2 * pr);
           if (j < g) { base.x += v.x; base.y += v.y; }
           tot.x += v.x; tot.y += v.y;
         }
-        // q^ = q exp(b - qr), k^ = k exp(kr - b)
+        // q^ = q exp2(b - qr), k^ = k exp2(kr - b)
         const float2 qr = gentle ? make_float2(0.5f * tot.x, 0.5f * tot.y) : make_float2(0.f, 0.f);
         const float2 kr = gentle ? qr : tot;
-        if (g == g_lo) {
-          const float2 e = make_float2(__expf(qr.x), __expf(qr.y));
-          *reinterpret_cast<float2*>(sPre + 2 * pr) = e;
-          *reinterpret_cast<float2*>(sMid + 2 * pr) = gentle ? make_float2(1.f, 1.f) : make_float2(__expf(tot.x), __expf(tot.y));
-          *reinterpret_cast<float2*>(sPost + 2 * pr) = e;
+        if (g == 2 * g_lo) {
+          const float2 e = make_float2(gl_ex2(qr.x), gl_ex2(qr.y));
+          float2* post = reinterpret_cast<float2*>(sPost + 2 * pr);
+          *reinterpret_cast<float2*>(sPre + 2 * pr) = make_float2(e.x * post->x, e.y * post->y);
+          if (!gentle) *reinterpret_cast<float2*>(sMid + 2 * pr) = make_float2(gl_ex2(tot.x), gl_ex2(tot.y));
+          *post = e;
         }
+        const float2 qo = make_float2(base.x - qr.x + scale2, base.y - qr.y + scale2), ko = make_float2(kr.x - base.x, kr.y - base.y);
 #pragma unroll
-        for (int r = 0; r < kPiece; ++r) {
-          const int t = g * kPiece + r;
-          float2 bb = *reinterpret_cast<const float2*>(sB + t * DP + 2 * pr);
-          bb.x += base.x; bb.y += base.y;
+        for (int r = 0; r < 8; ++r) {
+          const int t = g * 8 + r;
+          const float2 bb = *reinterpret_cast<const float2*>(sB + t * BS + 2 * pr);
           uint32_t* qp = reinterpret_cast<uint32_t*>(sq + t * QS + 2 * pr);
           uint32_t* kp = reinterpret_cast<uint32_t*>(sk + t * QS + 2 * pr);
           const float2 k = gl_unpack(*kp);
           if (!p.carry) {
             const float2 q = gl_unpack(*qp);
-            *qp = gl_pack(q.x * p.scale * __expf(bb.x - qr.x), q.y * p.scale * __expf(bb.y - qr.y));
+            *qp = gl_pack(q.x * gl_ex2(bb.x + qo.x), q.y * gl_ex2(bb.y + qo.y));
           }
-          *kp = gl_pack(k.x * __expf(kr.x - bb.x), k.y * __expf(kr.y - bb.y));
+          *kp = gl_pack(k.x * gl_ex2(ko.x - bb.x), k.y * gl_ex2(ko.y - bb.y));
         }
       }
       __syncthreads();
       // the state as an operand, and the scores
-#pragma unroll
-      for (int m = 0; m < MPW; ++m) {
-        const int d = sm0 + m * 16 + (lane >> 2);
-        const float f0 = sPre[d], f1 = sPre[d + 8], m0 = sMid[d], m1 = sMid[d + 8];
+      {
+        const float f0 = sPre[sd], f1 = sPre[sd + 8];
 #pragma unroll
         for (int j = 0; j < NPW; ++j) {
-          const int c = sn0 + j * 8 + 2 * (lane & 3);
-          S[m][j][0] *= f0; S[m][j][1] *= f0; S[m][j][2] *= f1; S[m][j][3] *= f1;
+          S[j][0] *= f0; S[j][1] *= f0; S[j][2] *= f1; S[j][3] *= f1;
           if (!p.carry) {
-            *reinterpret_cast<uint32_t*>(sS + d * VSS + c) = gl_pack(S[m][j][0], S[m][j][1]);
-            *reinterpret_cast<uint32_t*>(sS + (d + 8) * VSS + c) = gl_pack(S[m][j][2], S[m][j][3]);
+            *reinterpret_cast<uint32_t*>(sS + sd * VSS + sc + j * 8) = gl_pack(S[j][0], S[j][1]);
+            *reinterpret_cast<uint32_t*>(sS + (sd + 8) * VSS + sc + j * 8) = gl_pack(S[j][2], S[j][3]);
           }
-          if (!gentle) { S[m][j][0] *= m0; S[m][j][1] *= m0; S[m][j][2] *= m1; S[m][j][3] *= m1; }
+        }
+        if (!gentle) {
+          const float m0 = sMid[sd], m1 = sMid[sd + 8];
+#pragma unroll
+          for (int j = 0; j < NPW; ++j) { S[j][0] *= m0; S[j][1] *= m0; S[j][2] *= m1; S[j][3] *= m1; }
         }
       }
       const bool my_rows = mt >= g_lo && mt < g_hi && !p.carry;
-      if (gentle && my_rows) {
-        // columns of this warp: of the whole chunk its half (32), of a piece 8 of its 16
-        if (one) {
-          float A[4][4];
+      const int kt = one ? quarter : mt;                   // the 16 keys of this warp's scores
+      if (gentle && my_rows && kt <= mt && (one || quarter == 0)) {
+        float A[2][4];
 #pragma unroll
-          for (int j = 0; j < 4; ++j) A[j][0] = A[j][1] = A[j][2] = A[j][3] = 0.f;
-          const int n0 = half * 32;
-          if (n0 <= mt * 16 + 15) {
+        for (int j = 0; j < 2; ++j) A[j][0] = A[j][1] = A[j][2] = A[j][3] = 0.f;
 #pragma unroll
-            for (int ks = 0; ks < DP / 16; ++ks) {
-              uint32_t a[4];
-              gl_ldsm(a, sq + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * QS + ks * 16 + (lane >> 4) * 8);
-#pragma unroll
-              for (int j = 0; j < 4; j += 2) {
-                uint32_t w[4];
-                gl_ldsm(w, sk + (n0 + j * 8 + (lane & 7) + ((lane >> 4) & 1) * 8) * QS + ks * 16 + ((lane >> 3) & 1) * 8);
-                gl_mma(A[j], a, w[0], w[1]);
-                gl_mma(A[j + 1], a, w[2], w[3]);
-              }
-            }
-          }
-#pragma unroll
-          for (int j = 0; j < 4; ++j)
-#pragma unroll
-            for (int e = 0; e < 4; e += 2) {
-              const int t = mt * 16 + (lane >> 2) + (e >> 1) * 8, s = n0 + j * 8 + 2 * (lane & 3);
-              *reinterpret_cast<uint32_t*>(sA + t * AS + s) = gl_pack(s <= t ? A[j][e] : 0.f, s + 1 <= t ? A[j][e + 1] : 0.f);
-            }
-        } else if (half == 0) {
-          float A[2][4];
-#pragma unroll
-          for (int j = 0; j < 2; ++j) A[j][0] = A[j][1] = A[j][2] = A[j][3] = 0.f;
-#pragma unroll
-          for (int ks = 0; ks < DP / 16; ++ks) {
-            uint32_t a[4], w[4];
-            gl_ldsm(a, sq + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * QS + ks * 16 + (lane >> 4) * 8);
-            gl_ldsm(w, sk + (mt * 16 + (lane & 7) + ((lane >> 4) & 1) * 8) * QS + ks * 16 + ((lane >> 3) & 1) * 8);
-            gl_mma(A[0], a, w[0], w[1]);
-            gl_mma(A[1], a, w[2], w[3]);
-          }
-#pragma unroll
-          for (int j = 0; j < 2; ++j)
-#pragma unroll
-            for (int e = 0; e < 4; e += 2) {
-              const int t = mt * 16 + (lane >> 2) + (e >> 1) * 8, s = mt * 16 + j * 8 + 2 * (lane & 3);
-              *reinterpret_cast<uint32_t*>(sA + t * AS + s) = gl_pack(s <= t ? A[j][e] : 0.f, s + 1 <= t ? A[j][e + 1] : 0.f);
-            }
+        for (int ks = 0; ks < DP / 16; ++ks) {
+          uint32_t a[4], w[4];
+          gl_ldsm(a, sq + (mt * 16 + fa_r) * QS + ks * 16 + fa_c);
+          gl_ldsm(w, sk + (kt * 16 + fb_r) * QS + ks * 16 + fb_c);
+          gl_mma(A[0], a, w[0], w[1]);
+          gl_mma(A[1], a, w[2], w[3]);
         }
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; e += 2) {
+            const int t = r0 + (e >> 1) * 8, s = kt * 16 + j * 8 + cc;
+            *reinterpret_cast<uint32_t*>(sA + t * AS + s) = gl_pack(s <= t ? A[j][e] : 0.f, s + 1 <= t ? A[j][e + 1] : 0.f);
+          }
       }
-      __syncthreads();
       if (pc == 0 && even && !p.raw && !p.carry) {         // fetched here, used behind the products
 #pragma unroll
-        for (int j = 0; j < VS / 16; ++j)
+        for (int j = 0; j < NO; ++j)
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
-            const int c = half * (VS / 2) + j * 8 + 2 * (lane & 3), r = mt * 16 + (lane >> 2) + e * 8;
+            const int c = quarter * (VS / 4) + j * 8 + cc, r = r0 + e * 8;
             gate[j][e] = r < rows && c < p.vdim ? __ldg(reinterpret_cast<const uint32_t*>(
                 x + (size_t)(ch * kChunk + r) * p.ldx + p.g_at + h * p.vdim + c)) : 0u;
           }
       }
-      // O = q^ S + A V, rows of this warp, half of the columns
+      __syncthreads();
+      // O = q^ S + A V, rows of this warp, a quarter of the columns
       if (my_rows) {
 #pragma unroll
         for (int ks = 0; ks < DP / 16; ++ks) {
           uint32_t a[4];
-          gl_ldsm(a, sq + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * QS + ks * 16 + (lane >> 4) * 8);
+          gl_ldsm(a, sq + (mt * 16 + fa_r) * QS + ks * 16 + fa_c);
 #pragma unroll
-          for (int j = 0; j < VS / 16; j += 2) {
+          for (int j = 0; j < NO; j += 2) {
             uint32_t w[4];
-            gl_ldsm_t(w, sS + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VSS + half * (VS / 2) + j * 8 + (lane >> 4) * 8);
+            gl_ldsm_t(w, sS + (ks * 16 + fa_r) * VSS + quarter * (VS / 4) + j * 8 + fa_c);
             gl_mma(O[j], a, w[0], w[1]);
             gl_mma(O[j + 1], a, w[2], w[3]);
           }
         }
         for (int ks = g_lo; ks <= mt; ++ks) {              // causal: 16 keys at a time
           uint32_t a[4];
-          gl_ldsm(a, sA + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * AS + ks * 16 + (lane >> 4) * 8);
+          gl_ldsm(a, sA + (mt * 16 + fa_r) * AS + ks * 16 + fa_c);
 #pragma unroll
-          for (int j = 0; j < VS / 16; j += 2) {
+          for (int j = 0; j < NO; j += 2) {
             uint32_t w[4];
-            gl_ldsm_t(w, sv + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VSS + half * (VS / 2) + j * 8 + (lane >> 4) * 8);
+            gl_ldsm_t(w, sv + (ks * 16 + fa_r) * VSS + quarter * (VS / 4) + j * 8 + fa_c);
             gl_mma(O[j], a, w[0], w[1]);
             gl_mma(O[j + 1], a, w[2], w[3]);
           }
@@ -579,102 +568,80 @@ __global__ void __launch_bounds__(256, 1) gla_chunk_kernel(const GlaParams p) {
       }
       // S += k^^T V
       for (int ks = g_lo; ks < g_hi; ++ks) {
-        uint32_t a[MPW][4];
-#pragma unroll
-        for (int m = 0; m < MPW; ++m)
-          gl_ldsm_t(a[m], sk + (ks * 16 + (lane & 7) + ((lane >> 4) & 1) * 8) * QS + sm0 + m * 16 + ((lane >> 3) & 1) * 8);
+        uint32_t a[4];
+        gl_ldsm_t(a, sk + (ks * 16 + fb_r) * QS + (warp % MW) * 16 + fb_c);
 #pragma unroll
         for (int j = 0; j < NPW; j += 2) {
           uint32_t w[4];
-          gl_ldsm_t(w, sv + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VSS + sn0 + j * 8 + (lane >> 4) * 8);
-#pragma unroll
-          for (int m = 0; m < MPW; ++m) {
-            gl_mma(S[m][j], a[m], w[0], w[1]);
-            gl_mma(S[m][j + 1], a[m], w[2], w[3]);
-          }
+          gl_ldsm_t(w, sv + (ks * 16 + fa_r) * VSS + sn0 + j * 8 + fa_c);
+          gl_mma(S[j], a, w[0], w[1]);
+          gl_mma(S[j + 1], a, w[2], w[3]);
         }
-      }
-#pragma unroll
-      for (int m = 0; m < MPW; ++m) {
-        const int d = sm0 + m * 16 + (lane >> 2);
-        const float f0 = sPost[d], f1 = sPost[d + 8];
-#pragma unroll
-        for (int j = 0; j < NPW; ++j) { S[m][j][0] *= f0; S[m][j][1] *= f0; S[m][j][2] *= f1; S[m][j][3] *= f1; }
       }
       if (pc + 1 < pieces) __syncthreads();               // the next piece writes sS, sA and the factors again
     }
-    if (p.carry) { __syncthreads(); if (Cfg::STAGES == 1 && ch + 1 < ch1) load(ch + 1); continue; }
     // norm and gate (or the bare output, when other CTAs have the head's other columns)
-    const int r0 = mt * 16 + (lane >> 2), r1 = r0 + 8;
-    if (p.raw) {
+    if (p.carry) {
+    } else if (p.raw) {
 #pragma unroll
-      for (int j = 0; j < VS / 16; ++j) {
-        const int c = half * (VS / 2) + j * 8 + 2 * (lane & 3);
+      for (int j = 0; j < NO; ++j) {
+        const int c = quarter * (VS / 4) + j * 8 + cc;
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int r = e < 2 ? r0 : r1;
+          const int r = r0 + (e >> 1) * 8;
           if (r < rows && c + (e & 1) < vw)
             p.raw[(size_t)(start + ch * kChunk + r) * p.heads * p.vdim + h * p.vdim + v0 + c + (e & 1)] = O[j][e];
         }
       }
     } else {
-      float s0 = 0.f, s1 = 0.f;
+      float ss[2] = {0.f, 0.f};
 #pragma unroll
-      for (int j = 0; j < VS / 16; ++j) {
-        s0 += O[j][0] * O[j][0] + O[j][1] * O[j][1];
-        s1 += O[j][2] * O[j][2] + O[j][3] * O[j][3];
+      for (int j = 0; j < NO; ++j) {
+        ss[0] += O[j][0] * O[j][0] + O[j][1] * O[j][1];
+        ss[1] += O[j][2] * O[j][2] + O[j][3] * O[j][3];
       }
 #pragma unroll
-      for (int m = 1; m < 4; m <<= 1) {
-        s0 += __shfl_xor_sync(0xffffffffu, s0, m);
-        s1 += __shfl_xor_sync(0xffffffffu, s1, m);
+      for (int e = 0; e < 2; ++e) {
+        ss[e] += __shfl_xor_sync(0xffffffffu, ss[e], 1);
+        ss[e] += __shfl_xor_sync(0xffffffffu, ss[e], 2);
+        if ((lane & 3) == 0) sSS[quarter * kChunk + r0 + e * 8] = ss[e];
       }
-      if ((lane & 3) == 0) { sSS[half * kChunk + r0] = s0; sSS[half * kChunk + r1] = s1; }
-      __syncthreads();
-      const float i0 = rsqrtf((sSS[r0] + sSS[kChunk + r0]) / (float)p.vdim + p.eps);
-      const float i1 = rsqrtf((sSS[r1] + sSS[kChunk + r1]) / (float)p.vdim + p.eps);
+      named_bar_sync(1 + mt, 128);                         // the four warps that have these rows
+      const float inv_n = 1.f / (float)p.vdim;
 #pragma unroll
-      for (int j = 0; j < VS / 16; ++j) {
-        const int c = half * (VS / 2) + j * 8 + 2 * (lane & 3);
-        const float w0 = sGain[c], w1 = sGain[c + 1];
+      for (int e = 0; e < 2; ++e) {
+        const int r = r0 + e * 8;
+        const float inv = rsqrtf((sSS[r] + sSS[kChunk + r] + sSS[2 * kChunk + r] + sSS[3 * kChunk + r]) * inv_n + p.eps);
+        const size_t trow = (size_t)(ch * kChunk + r);
+        bf16* orow = reinterpret_cast<bf16*>(p.out) + (start + trow) * p.ldo + h * p.vdim;
+        const bf16* grow = x + trow * p.ldx + p.g_at + h * p.vdim;
 #pragma unroll
-        for (int e = 0; e < 4; e += 2) {
-          const int r = e ? r1 : r0;
+        for (int j = 0; j < NO; ++j) {
+          const int c = quarter * (VS / 4) + j * 8 + cc;
           if (r >= rows || c >= p.vdim) continue;
-          const float inv = e ? i1 : i0;
-          const bf16* gp = x + (size_t)(ch * kChunk + r) * p.ldx + p.g_at + h * p.vdim + c;
-          bf16* op = reinterpret_cast<bf16*>(p.out) + (size_t)(start + ch * kChunk + r) * p.ldo + h * p.vdim + c;
+          const float2 w = *reinterpret_cast<const float2*>(sGain + c);
           if (even) {
-            const float2 g = gl_unpack(gate[j][e >> 1]);
-            *reinterpret_cast<uint32_t*>(op) = gl_pack(O[j][e] * inv * w0 * __fdividef(g.x, 1.f + __expf(-g.x)),
-                                                       O[j][e + 1] * inv * w1 * __fdividef(g.y, 1.f + __expf(-g.y)));
+            const float2 g = gl_unpack(gate[j][e]);
+            *reinterpret_cast<uint32_t*>(orow + c) = gl_pack(O[j][2 * e] * inv * w.x * gl_silu(g.x), O[j][2 * e + 1] * inv * w.y * gl_silu(g.y));
           } else {
-#pragma unroll
-            for (int k = 0; k < 2; ++k)
-              if (c + k < p.vdim) {
-                const float g = __bfloat162float(gp[k]);
-                op[k] = __float2bfloat16(O[j][e + k] * inv * (k ? w1 : w0) * __fdividef(g, 1.f + __expf(-g)));
-              }
+            orow[c] = __float2bfloat16(O[j][2 * e] * inv * w.x * gl_silu(__bfloat162float(grow[c])));
+            if (c + 1 < p.vdim) orow[c + 1] = __float2bfloat16(O[j][2 * e + 1] * inv * w.y * gl_silu(__bfloat162float(grow[c + 1])));
           }
         }
       }
     }
-    __syncthreads();                                       // everything of this chunk has been read
-    if (Cfg::STAGES == 1 && ch + 1 < ch1) load(ch + 1);
+    if (Cfg::STAGES == 1) {
+      __syncthreads();                                     // everything of this chunk has been read
+      if (ch + 1 < ch1) load(ch + 1);
+    }
   }
+  __syncthreads();
   if (p.carry) {
     st = seg_s + (size_t)(seg + 1) * p.dim * p.vdim;
     if (v0 == 0 && tid < p.dim) seg_d[(size_t)(seg + 1) * p.dim + tid] = carried;
   } else if (ch1 < chunks) return;                         // the last segment leaves the state
-#pragma unroll
-  for (int m = 0; m < MPW; ++m)
-#pragma unroll
-    for (int j = 0; j < NPW; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int d = sm0 + m * 16 + (lane >> 2) + (e >> 1) * 8, c = sn0 + j * 8 + 2 * (lane & 3) + (e & 1);
-        if (d < p.dim && c < vw) st[(size_t)d * p.vdim + v0 + c] = S[m][j][e];
-      }
+  const float post[2] = {sPost[sd], sPost[sd + 8]};
+  each_state([&](float& v, size_t at, bool in, int e) { if (in) st[at] = v * post[e]; });
 }
 
 // Norm and gate of rows whose columns came from several CTAs: one warp per (token, head) of the sequences in question.
@@ -767,9 +734,9 @@ static int launch_chunk(const GlaParams& p, cudaStream_t st) {
   if (p.segs > 1) {
     GlaParams q = p;
     q.carry = 1;
-    e = launch_pdl(gla_chunk_kernel<DP, VS, RP>, grid, dim3(256), Cfg::SMEM, st, q);
+    e = launch_pdl(gla_chunk_kernel<DP, VS, RP>, grid, dim3(kChunkThreads), Cfg::SMEM, st, q);
   }
-  if (e == cudaSuccess) e = launch_pdl(gla_chunk_kernel<DP, VS, RP>, grid, dim3(256), Cfg::SMEM, st, p);
+  if (e == cudaSuccess) e = launch_pdl(gla_chunk_kernel<DP, VS, RP>, grid, dim3(kChunkThreads), Cfg::SMEM, st, p);
   return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }
 template <int DP, int VS>
@@ -821,8 +788,7 @@ extern "C" int xft_gla_chunk(const void* x, int ldx, int k_at, int v_at, int g_a
   int r;
   if (dim > 128) r = launch_chunk<256, 64, 16>(p, st);
   else if (dim > 64) r = cols == 64 ? chunk_rank<128, 64>(p, st) : chunk_rank<128, 128>(p, st);
-  else if (dim > 32) r = cols == 64 ? chunk_rank<64, 64>(p, st) : chunk_rank<64, 128>(p, st);
-  else r = cols == 64 ? chunk_rank<32, 64>(p, st) : chunk_rank<32, 128>(p, st);
+  else r = cols == 64 ? chunk_rank<64, 64>(p, st) : chunk_rank<64, 128>(p, st);
   if (r || !p.raw) return r;
   const long long warps = (long long)T * heads;
   cudaError_t e = launch_pdl(gla_norm_kernel, dim3((unsigned)((warps + 3) / 4)), dim3(128), 0, st, p, T);
