@@ -586,38 +586,62 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_tm_kernel(const __grid_co
       __nv_bfloat16* orow = p.out + (size_t)t * p.ldo;
       const __nv_bfloat16* rrow = p.residual ? p.residual + (size_t)t * p.ldr : nullptr;
 #pragma unroll 1
-      for (int c = 0; c < BNF; c += 16) {
-        uint32_t v[16];
-        uint32_t vu[DUAL ? 16 : 1];
-        tmem_ld16(taddr + c, v);
-        if constexpr (DUAL) tmem_ld16(taddr + BNF + c, vu);
+      for (int c = 0; c < BNF; c += 32) {
+        const int n0 = im.nt * BNF + c;
+        const bool full = vec && n0 + 32 <= p.N;
+        uint32_t v[32];
+        uint32_t vu[DUAL ? 32 : 1];
+        tmem_ld32(taddr + c, v);
+        if constexpr (DUAL) tmem_ld32(taddr + BNF + c, reinterpret_cast<uint32_t (&)[32]>(vu));
+        uint4 res[4];
+        const bool take = rrow && full && t_ok && !p.out_fp32;
+        if (take) {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) res[j] = *reinterpret_cast<const uint4*>(rrow + n0 + 8 * j);
+        }
         tmem_ld_wait();
-        if (c + 16 >= BNF) {
+        if (c + 32 >= BNF) {
           tcgen05_fence_before();
           __syncwarp();
           if (lane == 0) mbar_arrive(&tmem_empty[a]);
         }
-        const int n0 = im.nt * BNF + c;
         if (!t_ok || n0 >= p.N) continue;
-        float x[16];
+        float x[32];
 #pragma unroll
-        for (int j = 0; j < 16; ++j) x[j] = __uint_as_float(v[j]);
-        const bool full = vec && n0 + 16 <= p.N;
+        for (int j = 0; j < 32; ++j) x[j] = __uint_as_float(v[j]);
         if (p.bias && full && bias16) {
 #pragma unroll
-          for (int j = 0; j < 4; ++j) {
-            const float4 v = __ldg(reinterpret_cast<const float4*>(p.bias + n0) + j);
-            x[4 * j] += v.x; x[4 * j + 1] += v.y; x[4 * j + 2] += v.z; x[4 * j + 3] += v.w;
+          for (int j = 0; j < 8; ++j) {
+            const float4 w = __ldg(reinterpret_cast<const float4*>(p.bias + n0) + j);
+            x[4 * j] += w.x; x[4 * j + 1] += w.y; x[4 * j + 2] += w.z; x[4 * j + 3] += w.w;
           }
         } else if (p.bias) {
 #pragma unroll
-          for (int j = 0; j < 16; ++j) if (full || n0 + j < p.N) x[j] += __ldg(p.bias + n0 + j);
+          for (int j = 0; j < 32; ++j) if (full || n0 + j < p.N) x[j] += __ldg(p.bias + n0 + j);
         }
+        // one branch for the whole row: a branch per element cost more than the arithmetic
+        switch (p.act & (kPrefillTimes - 1)) {
+          case 1:
 #pragma unroll
-        for (int j = 0; j < 16; ++j) x[j] = prefill_act(x[j], p.act);
+            for (int j = 0; j < 32; ++j) x[j] = prefill_act(x[j], 1);
+            break;
+          case 2:
+#pragma unroll
+            for (int j = 0; j < 32; ++j) x[j] = prefill_act(x[j], 2);
+            break;
+          case 3:
+#pragma unroll
+            for (int j = 0; j < 32; ++j) x[j] = prefill_act(x[j], 3);
+            break;
+          case 4:
+#pragma unroll
+            for (int j = 0; j < 32; ++j) x[j] = prefill_act(x[j], 4);
+            break;
+          default: break;
+        }
         if constexpr (DUAL) {
 #pragma unroll
-          for (int j = 0; j < 16; ++j) {
+          for (int j = 0; j < 32; ++j) {
             float u = __uint_as_float(vu[j]);
             if (p.bias && (full || n0 + j < p.N)) u += __ldg(p.bias + p.dual_off + n0 + j);
             x[j] *= u;
@@ -627,37 +651,42 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_tm_kernel(const __grid_co
           float* frow = reinterpret_cast<float*>(p.out) + (size_t)t * p.ldo + n0;
           if (full) {
 #pragma unroll
-            for (int j = 0; j < 4; ++j)
+            for (int j = 0; j < 8; ++j)
               reinterpret_cast<float4*>(frow)[j] = make_float4(x[4 * j], x[4 * j + 1], x[4 * j + 2], x[4 * j + 3]);
           } else {
 #pragma unroll
-            for (int j = 0; j < 16; ++j) if (n0 + j < p.N) frow[j] = x[j];
+            for (int j = 0; j < 32; ++j) if (n0 + j < p.N) frow[j] = x[j];
           }
         } else if (full) {
-          if (rrow) {
-            const uint4 r0 = *reinterpret_cast<const uint4*>(rrow + n0), r1 = *reinterpret_cast<const uint4*>(rrow + n0 + 8);
-            const __nv_bfloat162* h0 = reinterpret_cast<const __nv_bfloat162*>(&r0);
-            const __nv_bfloat162* h1 = reinterpret_cast<const __nv_bfloat162*>(&r1);
+          if (take) {
+            const __nv_bfloat162* r2 = reinterpret_cast<const __nv_bfloat162*>(res);
+            if (p.act & kPrefillTimes) {
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
-              const float2 f0 = __bfloat1622float2(h0[j]), f1 = __bfloat1622float2(h1[j]);
-              x[2 * j] = prefill_residual(x[2 * j], f0.x, p.res_scale, p.act);
-              x[2 * j + 1] = prefill_residual(x[2 * j + 1], f0.y, p.res_scale, p.act);
-              x[8 + 2 * j] = prefill_residual(x[8 + 2 * j], f1.x, p.res_scale, p.act);
-              x[8 + 2 * j + 1] = prefill_residual(x[8 + 2 * j + 1], f1.y, p.res_scale, p.act);
+              for (int j = 0; j < 16; ++j) {
+                const float2 f = __bfloat1622float2(r2[j]);
+                x[2 * j] *= f.x; x[2 * j + 1] *= f.y;
+              }
+            } else {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) {
+                const float2 f = __bfloat1622float2(r2[j]);
+                x[2 * j] += p.res_scale * f.x; x[2 * j + 1] += p.res_scale * f.y;
+              }
             }
           }
-          uint32_t w[8];
 #pragma unroll
-          for (int j = 0; j < 8; ++j) {
-            const __nv_bfloat162 b = __floats2bfloat162_rn(x[2 * j], x[2 * j + 1]);
-            w[j] = *reinterpret_cast<const uint32_t*>(&b);
+          for (int i = 0; i < 4; ++i) {
+            uint32_t w[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+              const __nv_bfloat162 b = __floats2bfloat162_rn(x[8 * i + 2 * j], x[8 * i + 2 * j + 1]);
+              w[j] = *reinterpret_cast<const uint32_t*>(&b);
+            }
+            *reinterpret_cast<uint4*>(orow + n0 + 8 * i) = make_uint4(w[0], w[1], w[2], w[3]);
           }
-          *reinterpret_cast<uint4*>(orow + n0) = make_uint4(w[0], w[1], w[2], w[3]);
-          *reinterpret_cast<uint4*>(orow + n0 + 8) = make_uint4(w[4], w[5], w[6], w[7]);
         } else {
 #pragma unroll
-          for (int j = 0; j < 16; ++j) {
+          for (int j = 0; j < 32; ++j) {
             if (n0 + j < p.N) {
               float y = x[j];
               if (rrow) y = prefill_residual(y, __bfloat162float(rrow[n0 + j]), p.res_scale, p.act);
