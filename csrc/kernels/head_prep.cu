@@ -10,7 +10,7 @@
 // state slot is never cleared: rows in front of a sequence's first token are taken as zero by position.
 //
 // One warp per head and run of consecutive tokens: weights, gains and the convolution's window stay in registers, a lane
-// owns two neighbouring channels of every 64.  Heads are stored `padded` wide (zeros behind dim), as the attention kernels
+// owns two or four neighbouring channels.  Heads are stored `padded` wide (zeros behind dim), as the attention kernels
 // take them.  In a decode step the warp that reads a state also moves it on; otherwise a second, small kernel does, after
 // all portions have read theirs.
 #include "ptx.cuh"
@@ -39,32 +39,31 @@ template <typename T> __device__ __forceinline__ T hp_from(float v);
 template <> __device__ __forceinline__ float hp_from<float>(float v) { return v; }
 template <> __device__ __forceinline__ bf16 hp_from<bf16>(float v) { return __float2bfloat16(v); }
 
-// channels c, c + 1 of a row (n of them exist); `pair`: rows and heads are even, so the two load as one
-template <typename T>
-__device__ __forceinline__ float2 hp_load2(const T* p, int left, bool pair) {
-  float2 r = make_float2(0.f, 0.f);
-  if (pair) {
-    if (left > 0) {
-      struct alignas(2 * sizeof(T)) P2 { T a, b; };
-      const P2 v = *reinterpret_cast<const P2*>(p);
-      r = make_float2(hp_f32<T>(v.a), hp_f32<T>(v.b));
-    }
+// VEC neighbouring channels of a row, `left` of which exist; whole: they are aligned and exist all or not at all
+template <int VEC, typename T>
+__device__ __forceinline__ void hp_load(const T* p, int left, bool whole, float (&v)[VEC]) {
+  if (whole) {
+    struct alignas(VEC * sizeof(T)) V { T e[VEC]; };
+    V r;
+    if (left > 0) r = *reinterpret_cast<const V*>(p);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) v[k] = left > 0 ? hp_f32<T>(r.e[k]) : 0.f;
   } else {
-    if (left > 0) r.x = hp_f32<T>(p[0]);
-    if (left > 1) r.y = hp_f32<T>(p[1]);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) v[k] = k < left ? hp_f32<T>(p[k]) : 0.f;
   }
-  return r;
 }
-template <typename T>
-__device__ __forceinline__ void hp_store2(T* p, float2 v, int left, bool pair) {
-  if (pair) {
-    if (left > 0) {
-      struct alignas(2 * sizeof(T)) P2 { T a, b; };
-      *reinterpret_cast<P2*>(p) = P2{hp_from<T>(v.x), hp_from<T>(v.y)};
-    }
+template <int VEC, typename T>
+__device__ __forceinline__ void hp_store(T* p, const float (&v)[VEC], int left, bool whole) {
+  if (whole) {
+    struct alignas(VEC * sizeof(T)) V { T e[VEC]; };
+    V r;
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) r.e[k] = hp_from<T>(v[k]);
+    if (left > 0) *reinterpret_cast<V*>(p) = r;
   } else {
-    if (left > 0) p[0] = hp_from<T>(v.x);
-    if (left > 1) p[1] = hp_from<T>(v.y);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) if (k < left) p[k] = hp_from<T>(v[k]);
   }
 }
 
@@ -77,10 +76,11 @@ __device__ __forceinline__ int hp_sequence(const int* cu_q, int B, int t) {     
   return lo;
 }
 
-// NV: pairs of channels per lane (padded <= 64 * NV); TAPS >= taps
-template <typename T, int NV, int TAPS>
+// A lane owns VEC neighbouring channels of every 32 VEC, NV times (padded <= 32 VEC NV); TAPS >= taps.  VEC 4: dim, row
+// strides and half the rotated dimensions are multiples of 4.
+template <typename T, int VEC, int NV, int TAPS>
 __global__ void __launch_bounds__(128) head_prep_kernel(const HeadPrepParams p) {
-  extern __shared__ float hp_sm[];
+  extern __shared__ __align__(16) float hp_sm[];
   grid_dep_launch();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int heads = p.hq + p.hkv, C = heads * p.dim;
@@ -89,32 +89,39 @@ __global__ void __launch_bounds__(128) head_prep_kernel(const HeadPrepParams p) 
   if (t0 >= p.T) { grid_dep_wait(); return; }
   const int t1 = min(t0 + p.run, p.T);
   const bool is_k = h >= p.hq;
-  const bool even = (p.dim & 1) == 0, out_even = (p.padded & 1) == 0;
-  float* row = hp_sm + warp * p.dim;
+  const bool whole = VEC == 4 || (p.dim & 1) == 0, out_whole = VEC == 4 || (p.padded & 1) == 0;
+  float* row = hp_sm + warp * ((p.dim + 3) & ~3);
   const int skip = TAPS - p.taps;                        // leading taps that do not exist
-  float2 w[TAPS][NV], gain[NV];
+  float w[TAPS][NV][VEC], gain[NV][VEC];
   const float* norm = is_k ? p.k_norm : p.q_norm;
+  auto chan = [&](int i) { return VEC * lane + 32 * VEC * i; };
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
-    const int c = 2 * lane + 64 * i, left = p.dim - c;
+    const int c = chan(i), left = p.dim - c;
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j)
-      w[j][i] = j < skip ? make_float2(0.f, 0.f)
-              : p.conv ? hp_load2<float>(p.conv + (size_t)(j - skip) * C + h * p.dim + c, left, even)
-                       : make_float2(1.f, 1.f);
-    gain[i] = norm ? hp_load2<float>(norm + c, left, even) : make_float2(1.f, 1.f);
+    for (int j = 0; j < TAPS; ++j) {
+      if (j >= skip && p.conv) {
+        hp_load<VEC>(p.conv + (size_t)(j - skip) * C + h * p.dim + c, left, whole, w[j][i]);
+      } else {
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) w[j][i][k] = j < skip ? 0.f : 1.f;
+      }
+    }
+    if (norm) hp_load<VEC>(norm + c, left, whole, gain[i]);
   }
   grid_dep_wait();
   const T* x = reinterpret_cast<const T*>(p.x) + h * p.dim;
   T* state = reinterpret_cast<T*>(p.state);
   int b = hp_sequence(p.cu_q, p.B, t0);
-  float2 u[TAPS][NV];                                    // the window, newest last
+  float u[TAPS][NV][VEC], next[NV][VEC];                 // the window, newest last; the row behind it
+#pragma unroll
+  for (int i = 0; i < NV; ++i) hp_load<VEC>(x + (size_t)t0 * p.ldx + chan(i), p.dim - chan(i), whole, next[i]);
   bool fresh = true;
   for (int t = t0; t < t1; ++t) {
     while (b + 1 < p.B && t >= p.cu_q[b + 1]) { ++b; fresh = true; }
     const int start = p.cu_q[b], li = t - start;
     T* st = nullptr;
-    if (p.taps > 1) {
+    if (p.taps > 1 && (fresh || p.decode)) {
       int slot = p.state_slots[b];
       if (slot < 0 || slot >= p.num_states) { if (lane == 0 && p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); slot = 0; }
       st = state + (size_t)slot * (p.taps - 1) * C + h * p.dim;
@@ -126,61 +133,66 @@ __global__ void __launch_bounds__(128) head_prep_kernel(const HeadPrepParams p) 
         const int idx = li - (TAPS - 1) + j;             // place in this portion; negative: before it
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
-          const int c = 2 * lane + 64 * i, left = p.dim - c;
-          float2 v = make_float2(0.f, 0.f);
-          if (j >= skip) {
-            if (idx >= 0) v = hp_load2<T>(x + (size_t)(start + idx) * p.ldx + c, left, even);
-            else if (past + idx >= 0) v = hp_load2<T>(st + (size_t)(p.taps - 1 + idx) * C + c, left, even);
+          const int c = chan(i), left = p.dim - c;
+          if (j >= skip && idx >= 0) hp_load<VEC>(x + (size_t)(start + idx) * p.ldx + c, left, whole, u[j][i]);
+          else if (j >= skip && past + idx >= 0) hp_load<VEC>(st + (size_t)(p.taps - 1 + idx) * C + c, left, whole, u[j][i]);
+          else {
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) u[j][i][k] = 0.f;
           }
-          u[j][i] = v;
         }
       }
       fresh = false;
     }
-    float2 y[NV];
+    float y[NV][VEC];
     float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int c = 2 * lane + 64 * i, left = p.dim - c;
-      u[TAPS - 1][i] = hp_load2<T>(x + (size_t)t * p.ldx + c, left, even);
-      float2 a = make_float2(0.f, 0.f);
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) { a.x = fmaf(w[j][i].x, u[j][i].x, a.x); a.y = fmaf(w[j][i].y, u[j][i].y, a.y); }
-      y[i] = a;
-      ss += a.x * a.x + a.y * a.y;
+      for (int k = 0; k < VEC; ++k) {
+        u[TAPS - 1][i][k] = next[i][k];
+        float a = 0.f;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) a = fmaf(w[j][i][k], u[j][i][k], a);
+        y[i][k] = a;
+        ss = fmaf(a, a, ss);
+      }
+      if (t + 1 < t1) hp_load<VEC>(x + (size_t)(t + 1) * p.ldx + chan(i), p.dim - chan(i), whole, next[i]);
     }
     if (p.decode && p.taps > 1) {                        // rows 1 .. taps - 1 of the window are the new state
 #pragma unroll
       for (int j = 1; j < TAPS; ++j)
         if (j > skip)
 #pragma unroll
-          for (int i = 0; i < NV; ++i) {
-            const int c = 2 * lane + 64 * i;
-            hp_store2<T>(st + (size_t)(j - 1 - skip) * C + c, u[j][i], p.dim - c, even);
-          }
+          for (int i = 0; i < NV; ++i) hp_store<VEC>(st + (size_t)(j - 1 - skip) * C + chan(i), u[j][i], p.dim - chan(i), whole);
     }
 #pragma unroll
     for (int j = 0; j + 1 < TAPS; ++j)
 #pragma unroll
-      for (int i = 0; i < NV; ++i) u[j][i] = u[j + 1][i];
+      for (int i = 0; i < NV; ++i)
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) u[j][i][k] = u[j + 1][i][k];
     T* dst;
     if (is_k) {
       const long long slot = p.slots[t];
       if (slot < 0 || slot >= p.nslots) { if (lane == 0 && p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); continue; }
-      const size_t at = ((size_t)((slot / p.bs) * p.hkv + (h - p.hq)) * p.bs + slot % p.bs) * p.padded;
+      const int blk = (int)(slot / p.bs);
+      const size_t at = ((size_t)(blk * p.hkv + (h - p.hq)) * p.bs + (slot - (long long)blk * p.bs)) * p.padded;
       dst = reinterpret_cast<T*>(p.kc) + at;
       T* v = reinterpret_cast<T*>(p.vc) + at;
 #pragma unroll
-      for (int i = 0; i < NV; ++i) { const int c = 2 * lane + 64 * i; hp_store2<T>(v + c, y[i], p.padded - c, out_even); }
+      for (int i = 0; i < NV; ++i) hp_store<VEC>(v + chan(i), y[i], p.padded - chan(i), out_whole);
     } else {
       dst = reinterpret_cast<T*>(p.q_out) + ((size_t)t * p.hq + h) * p.padded;
     }
     if (norm) {
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-      const float inv = 1.f / sqrtf(ss / (float)p.dim + p.eps);
+      const float inv = rsqrtf(ss / (float)p.dim + p.eps);
 #pragma unroll
-      for (int i = 0; i < NV; ++i) { y[i].x *= inv * gain[i].x; y[i].y *= inv * gain[i].y; }
+      for (int i = 0; i < NV; ++i)
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) y[i][k] *= inv * gain[i][k];
     }
     if (p.rot > 0) {
       int pos = p.positions[t];
@@ -189,22 +201,33 @@ __global__ void __launch_bounds__(128) head_prep_kernel(const HeadPrepParams p) 
       const int half = p.rot >> 1;
       __syncwarp();
 #pragma unroll
-      for (int i = 0; i < NV; ++i) { const int c = 2 * lane + 64 * i; hp_store2<float>(row + c, y[i], p.dim - c, false); }
+      for (int i = 0; i < NV; ++i) hp_store<VEC>(row + chan(i), y[i], p.dim - chan(i), VEC == 4);
       __syncwarp();
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
-        const int c = 2 * lane + 64 * i;
-        if (c < p.rot) {                                 // rot is even, so both channels turn or neither
-          const bool s0 = c >= half, s1 = c + 1 >= half;
-          const int f0 = s0 ? c - half : c, f1 = s1 ? c + 1 - half : c + 1;
-          const float p0 = row[s0 ? c - half : c + half], p1 = row[s1 ? c + 1 - half : c + 1 + half];
-          y[i].x = y[i].x * cs[f0] + (s0 ? p0 : -p0) * cs[half + f0];
-          y[i].y = y[i].y * cs[f1] + (s1 ? p1 : -p1) * cs[half + f1];
+        const int c = chan(i);
+        if (c >= p.rot) continue;                        // rot is a multiple of VEC
+        float other[VEC], cosv[VEC], sinv[VEC];
+        if (VEC == 4) {                                  // all of them in the same half
+          const int f = c >= half ? c - half : c;
+          hp_load<VEC>(row + (c >= half ? f : c + half), VEC, true, other);
+          hp_load<VEC>(cs + f, VEC, true, cosv);
+          hp_load<VEC>(cs + half + f, VEC, true, sinv);
+        } else {
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) {
+            const int f = c + k >= half ? c + k - half : c + k;
+            other[k] = row[c + k >= half ? f : c + k + half];
+            cosv[k] = cs[f];
+            sinv[k] = cs[half + f];
+          }
         }
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) y[i][k] = y[i][k] * cosv[k] + (c + k >= half ? other[k] : -other[k]) * sinv[k];
       }
     }
 #pragma unroll
-    for (int i = 0; i < NV; ++i) { const int c = 2 * lane + 64 * i; hp_store2<T>(dst + c, y[i], p.padded - c, out_even); }
+    for (int i = 0; i < NV; ++i) hp_store<VEC>(dst + chan(i), y[i], p.padded - chan(i), out_whole);
   }
 }
 
@@ -236,24 +259,30 @@ __global__ void __launch_bounds__(256) conv_state_kernel(const T* __restrict__ x
 
 using namespace xft;
 
-template <typename T, int NV, int TAPS>
+template <typename T, int VEC, int NV, int TAPS>
 static cudaError_t launch_head_prep(const HeadPrepParams& p, cudaStream_t st) {
   const long long warps = (long long)((p.T + p.run - 1) / p.run) * (p.hq + p.hkv);
-  return launch_pdl(head_prep_kernel<T, NV, TAPS>, dim3((unsigned)((warps + 3) / 4)), dim3(128), (size_t)4 * p.dim * sizeof(float), st, p);
+  return launch_pdl(head_prep_kernel<T, VEC, NV, TAPS>, dim3((unsigned)((warps + 3) / 4)), dim3(128),
+                    (size_t)4 * ((p.dim + 3) / 4 * 4) * sizeof(float), st, p);
 }
-template <typename T, int NV>
+template <typename T, int VEC, int NV>
 static cudaError_t pick_taps(const HeadPrepParams& p, cudaStream_t st) {
-  if (p.taps <= 1) return launch_head_prep<T, NV, 1>(p, st);
-  if (p.taps <= 2) return launch_head_prep<T, NV, 2>(p, st);
-  if (p.taps <= 4) return launch_head_prep<T, NV, 4>(p, st);
-  return launch_head_prep<T, NV, 8>(p, st);
+  if (p.taps <= 1) return launch_head_prep<T, VEC, NV, 1>(p, st);
+  if (p.taps <= 2) return launch_head_prep<T, VEC, NV, 2>(p, st);
+  if (p.taps <= 4) return launch_head_prep<T, VEC, NV, 4>(p, st);
+  return launch_head_prep<T, VEC, NV, 8>(p, st);
 }
 template <typename T>
 static cudaError_t pick_width(const HeadPrepParams& p, cudaStream_t st) {
-  if (p.padded <= 64) return pick_taps<T, 1>(p, st);
-  if (p.padded <= 128) return pick_taps<T, 2>(p, st);
-  if (p.padded <= 256) return pick_taps<T, 4>(p, st);
-  return pick_taps<T, 8>(p, st);
+  if (p.dim % 4 == 0 && p.padded % 4 == 0 && p.ldx % 4 == 0 && p.rot % 8 == 0) {
+    if (p.padded <= 128) return pick_taps<T, 4, 1>(p, st);
+    if (p.padded <= 256) return pick_taps<T, 4, 2>(p, st);
+    return pick_taps<T, 4, 4>(p, st);
+  }
+  if (p.padded <= 64) return pick_taps<T, 2, 1>(p, st);
+  if (p.padded <= 128) return pick_taps<T, 2, 2>(p, st);
+  if (p.padded <= 256) return pick_taps<T, 2, 4>(p, st);
+  return pick_taps<T, 2, 8>(p, st);
 }
 
 // x rows, q_out, caches and state all fp32 (f32 = 1) or bf16.  caches [blocks, hkv, bs, padded].  dim <= padded <= 512, up to 8

@@ -140,7 +140,7 @@ def test_token_major_prefill_gemm_matches_fp32(T, N, K, gated):
         want = torch.nn.functional.silu(y[:, :N]) * y[:, N:]
     else:
         want = torch.nn.functional.gelu(y, approximate="tanh") + 0.5 * res.float()
-    N_._ENV().gemm_prefill_tm, N_._ENV().gemm_prefill_tm_all = True, True      # every shape through the token-major kernel
+    N_._ENV().gemm_prefill_tm = True      # every shape through the token-major kernel
     got = N_.gemm_bf16(x, w, N, gated=gated, dual_off=N if gated else 0, bias=bias, act="silu" if gated else "gelu",
                        residual=res, res_scale=0.5)
     torch.cuda.synchronize()

@@ -243,11 +243,8 @@ def gemm_bf16(x, w, N, gated=False, dual_off=0, bias=None, act=None, residual=No
     if T <= SK_MAX_TOKENS and force_splits == 0 and _sk_choice(T, N, K, gated):
         _gemm_sk(x2, ldx, w, out, T, N, K, gated, dual_off, bias, r2, ldr, res_scale, act, row_scale, None, None, None)
         return out
-    # measured on B200 (benchmarks/bench_gemm.py --shapes prefill): the token-major kernel wins wherever the epilogue
-    # weighs (reductions up to 8192, ungated); long reductions and the gated form stay on the tile-per-CTA kernel, whose
-    # paired 256 x 256 tiles read fewer operand bytes per FLOP
     if _ENV().gemm_prefill_tm and T > 128 and not fp32 and row_scale is None and out.stride(1) == 1 \
-            and out.dtype == torch.bfloat16 and (K <= 8192 and not gated or _ENV().gemm_prefill_tm_all):
+            and out.dtype == torch.bfloat16 and not (gated and _ENV().gemm_persistent):
         # prompt sizes: persistent token-major kernel (tokens are the MMA rows, so bias / residual / output move as
         # 16-byte vectors along a token's features; two TMEM accumulators overlap the epilogue with the next tile)
         L = lib()
@@ -258,7 +255,7 @@ def gemm_bf16(x, w, N, gated=False, dual_off=0, bias=None, act=None, residual=No
         _check(rc, "gemm_bf16_prefill_tm")
         ws.launches += 1
         return out
-    if _ENV().gemm_prefill_tm and T > 128 and fp32 and row_scale is None and residual is None and not gated and K <= 8192 \
+    if _ENV().gemm_prefill_tm and T > 128 and fp32 and row_scale is None and residual is None and not gated \
             and out.stride(1) == 1 and force_splits == 0:
         fn = lib().xft_gemm_bf16_prefill_tm_f32
         fn.restype = C.c_int
