@@ -15,6 +15,8 @@ penalties, prefill, pipeline stages) runs the eager path in `engine.Model`.
 """
 from __future__ import annotations
 
+import contextlib
+import gc
 from typing import Dict, List, Sequence
 
 import torch
@@ -22,6 +24,20 @@ import torch
 from ..models.decoder import Batch
 from ..utils import trace
 from . import sampler as S
+
+
+@contextlib.contextmanager
+def _capture(graph, stream):
+    """torch.cuda.graph without the garbage collector: a collection in the middle of a capture may destroy the graphs of a
+    model that has gone out of use, which a capturing stream does not permit."""
+    was = gc.isenabled()
+    gc.disable()
+    try:
+        with torch.cuda.graph(graph, stream=stream):
+            yield
+    finally:
+        if was:
+            gc.enable()
 
 
 class _Graph:
@@ -243,7 +259,7 @@ class CudaRunner:
                 g = _Graph()
                 g.version = -1
                 graph = torch.cuda.CUDAGraph()
-                with torch.cuda.graph(graph, stream=st):
+                with _capture(graph, st):
                     self.m.decoder.forward_idle()
                 g.graph = graph
                 self.graphs["idle"] = g
@@ -279,7 +295,7 @@ class CudaRunner:
                 ws = N.Workspace.get(self.dev)
                 n0 = ws.launches
                 graph = torch.cuda.CUDAGraph()
-                with torch.cuda.graph(graph, stream=st):
+                with _capture(graph, st):
                     self._step_body(g)
                 g.graph = graph
                 g.kernels = ws.launches - n0
