@@ -234,9 +234,12 @@ struct ChunkCfg {
   static constexpr int BS = DP + 8;
   static constexpr int STAGE = kChunk * (2 * QS + VSS + RS);                         // q, k, v, a1 of a chunk, in values
   static constexpr int STAGES = DP <= 128 ? 2 : 1;
-  static constexpr size_t B16 = (size_t)STAGES * STAGE + kChunk * AS + DP * VSS + DP * RS;
-  static constexpr size_t F32 = (size_t)kChunk * BS + 8 * DP + 4 * DP + 4 * kChunk + VS;
-  static constexpr size_t SMEM = B16 * 2 + F32 * 4;
+  // the running sums are done with when the state is written as an operand: one place for both
+  static constexpr size_t SHARED = (size_t)kChunk * BS * 4 > (size_t)DP * VSS * 2 ? (size_t)kChunk * BS * 4 : (size_t)DP * VSS * 2;
+  static constexpr size_t B16 = (size_t)STAGES * STAGE + kChunk * AS + DP * RS;
+  static constexpr size_t F32 = 8 * DP + 4 * 2 * DP + DP + 4 * kChunk + VS;
+  static constexpr size_t SMEM = B16 * 2 + SHARED + F32 * 4;
+  static_assert(SMEM <= 227 * 1024, "shared memory");
 };
 
 template <int DP, int VS, int RP>
@@ -250,14 +253,13 @@ __global__ void __launch_bounds__(kChunkThreads, 1) gla_chunk_kernel(const GlaPa
   extern __shared__ __align__(16) uint8_t gc_raw[];
   bf16* stage0 = reinterpret_cast<bf16*>(gc_raw);
   bf16* sA = stage0 + Cfg::STAGES * Cfg::STAGE;           // scores [64][AS]
-  bf16* sS = sA + kChunk * AS;                            // state as an operand [DP][VSS]
-  bf16* sW = sS + DP * VSS;                               // a2 of this head [DP][RS]
+  bf16* sW = sA + kChunk * AS;                            // a2 of this head [DP][RS]
   float* sB = reinterpret_cast<float*>(sW + DP * RS);     // running sums of log2(alpha) [64][BS], restarting every 8 rows
-  float* sT = sB + kChunk * BS;                           // their totals [8][DP]
-  float* sPre = sT + 8 * DP;                              // factors of the state's rows: in front of the operand,
-  float* sMid = sPre + DP;                                //   behind it,
-  float* sPost = sMid + DP;                               //   and behind the update (applied with the next sPre)
-  float* sBias = sPost + DP;
+  bf16* sS = reinterpret_cast<bf16*>(sB);                 // then the state as an operand [DP][VSS]
+  float* sT = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(sB) + Cfg::SHARED);     // totals of the sums [8][DP]
+  float* sPre = sT + 8 * DP;                              // [4][DP] factors of the state's rows, per piece: in front of the operand
+  float* sMid = sPre + 4 * DP;                            // [4][DP] and behind it
+  float* sBias = sMid + 4 * DP;
   float* sSS = sBias + DP;                                // [4][64] sums of squares of the output rows
   float* sGain = sSS + 4 * kChunk;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -281,10 +283,11 @@ __global__ void __launch_bounds__(kChunkThreads, 1) gla_chunk_kernel(const GlaPa
     const int d = i / RP, r = i % RP;
     sW[d * RS + r] = d < p.dim && r < p.rank ? a2[(size_t)d * p.rank_ld + r] : __float2bfloat16(0.f);
   }
-  for (int d = tid; d < DP; d += NT) { sBias[d] = d < p.dim ? p.bias[h * p.dim + d] : 0.f; sPost[d] = 1.f; }
+  for (int d = tid; d < DP; d += NT) { sBias[d] = d < p.dim ? p.bias[h * p.dim + d] : 0.f; }
   for (int c = tid; c < VS; c += NT) sGain[c] = c < vw ? p.gain[v0 + c] : 0.f;
   // the state: warp tile of 16 rows and NPW x 8 columns
   const int sd = (warp % MW) * 16 + (lane >> 2), sn0 = warp / MW * NPW * 8, sc = sn0 + 2 * (lane & 3);
+  float post0 = 1.f, post1 = 1.f;                         // factors of the two rows still to come
   float S[NPW][4];                                        // element e: row sd + 8 (e >> 1), column sc + 8 j + (e & 1)
   auto each_state = [&](auto f) {
 #pragma unroll
@@ -429,70 +432,77 @@ __global__ void __launch_bounds__(kChunkThreads, 1) gla_chunk_kernel(const GlaPa
 #pragma unroll
     for (int j = 0; j < NO; ++j) O[j][0] = O[j][1] = O[j][2] = O[j][3] = 0.f;
     uint32_t gate[NO][2];                                  // of this warp's output values
+    // which pieces (groups of 16 rows) have a channel too fast for factors
+    uint32_t harsh = 0;
+    if (!one) {
+      uint32_t mine = 0;
+      for (int d = tid; d < DP; d += NT)
+#pragma unroll
+        for (int g = 0; g < 4; ++g) mine |= (sT[2 * g * DP + d] + sT[(2 * g + 1) * DP + d] < -kMaxDecay * kLog2e ? 1u : 0u) << g;
+#pragma unroll
+      for (int g = 0; g < 4; ++g) harsh |= (__syncthreads_or(mine >> g & 1) ? 1u : 0u) << g;
+      if (harsh && !p.carry) {
+        // their scores from differences of running sums: 256 pairs of rows each, a warp at a time
+        for (int i = warp; i < 4 * kPiece * kPiece; i += NT / 32) {
+          const int g = i / (kPiece * kPiece), t = g * kPiece + i / kPiece % kPiece, s = g * kPiece + i % kPiece;
+          if (!(harsh >> g & 1)) continue;
+          float a = 0.f;
+          if (s <= t)
+            for (int d = lane; d < p.dim; d += 32) {
+              const float between = (t & 8) && !(s & 8) ? sT[2 * g * DP + d] : 0.f;       // the sums restart between s and t
+              a += __bfloat162float(sq[t * QS + d]) * __bfloat162float(sk[s * QS + d]) * gl_ex2(sB[t * BS + d] - sB[s * BS + d] + between);
+            }
+#pragma unroll
+          for (int m = 16; m > 0; m >>= 1) a += __shfl_xor_sync(0xffffffffu, a, m);
+          if (lane == 0) sA[t * AS + s] = __float2bfloat16(a * p.scale);
+        }
+        __syncthreads();
+      }
+    }
+    // q^ and k^ in place; the factors of the state's rows
+    for (int it = tid; it < 4 * DP; it += NT) {
+      const int pr = it % (DP / 2), g = it / (DP / 2);
+      const int lo = one ? 0 : g & ~1, hi = one ? 8 : lo + 2;        // the piece's groups of 8 rows
+      float2 base = make_float2(0.f, 0.f), tot = make_float2(0.f, 0.f);
+      for (int j = lo; j < hi; ++j) {
+        const float2 v = *reinterpret_cast<const float2*>(sT + j * DP + 2 * pr);
+        if (j < g) { base.x += v.x; base.y += v.y; }
+        tot.x += v.x; tot.y += v.y;
+      }
+      // q^ = q exp2(b - qr), k^ = k exp2(kr - b)
+      const bool gentle = !(harsh >> (g >> 1) & 1);
+      const float2 qr = gentle ? make_float2(0.5f * tot.x, 0.5f * tot.y) : make_float2(0.f, 0.f);
+      const float2 kr = gentle ? qr : tot;
+      if (g == lo) {
+        const float2 e = make_float2(gl_ex2(qr.x), gl_ex2(qr.y));
+        *reinterpret_cast<float2*>(sMid + (lo >> 1) * DP + 2 * pr) = gentle ? make_float2(1.f, 1.f) : make_float2(gl_ex2(tot.x), gl_ex2(tot.y));
+        *reinterpret_cast<float2*>(sPre + (lo >> 1) * DP + 2 * pr) = e;
+      }
+      const float2 qo = make_float2(base.x - qr.x + scale2, base.y - qr.y + scale2), ko = make_float2(kr.x - base.x, kr.y - base.y);
+#pragma unroll
+      for (int r = 0; r < 8; ++r) {
+        const int t = g * 8 + r;
+        const float2 bb = *reinterpret_cast<const float2*>(sB + t * BS + 2 * pr);
+        uint32_t* qp = reinterpret_cast<uint32_t*>(sq + t * QS + 2 * pr);
+        uint32_t* kp = reinterpret_cast<uint32_t*>(sk + t * QS + 2 * pr);
+        const float2 k = gl_unpack(*kp);
+        if (!p.carry) {
+          const float2 q = gl_unpack(*qp);
+          *qp = gl_pack(q.x * gl_ex2(bb.x + qo.x), q.y * gl_ex2(bb.y + qo.y));
+        }
+        *kp = gl_pack(k.x * gl_ex2(ko.x - bb.x), k.y * gl_ex2(ko.y - bb.y));
+      }
+    }
+    __syncthreads();
     for (int pc = 0; pc < pieces; ++pc) {
       const int g_lo = one ? 0 : pc, g_hi = one ? 4 : pc + 1;       // groups of 16 rows in this piece
-      bool gentle = true;
-      if (!one) {
-        bool k = true;
-        for (int d = tid; d < DP; d += NT) k = sT[2 * pc * DP + d] + sT[(2 * pc + 1) * DP + d] >= -kMaxDecay * kLog2e;
-        gentle = __syncthreads_and(k);
-        if (!gentle && !p.carry) {
-          // scores of the piece from differences of running sums; 256 pairs of rows, a warp at a time
-          for (int i = warp; i < kPiece * kPiece; i += NT / 32) {
-            const int t = pc * kPiece + i / kPiece, s = pc * kPiece + i % kPiece;
-            float a = 0.f;
-            if (s <= t)
-              for (int d = lane; d < p.dim; d += 32) {
-                const float between = (t & 8) && !(s & 8) ? sT[2 * pc * DP + d] : 0.f;       // the sums restart between s and t
-                a += __bfloat162float(sq[t * QS + d]) * __bfloat162float(sk[s * QS + d]) *
-                     gl_ex2(sB[t * BS + d] - sB[s * BS + d] + between);
-              }
-#pragma unroll
-            for (int m = 16; m > 0; m >>= 1) a += __shfl_xor_sync(0xffffffffu, a, m);
-            if (lane == 0) sA[t * AS + s] = __float2bfloat16(a * p.scale);
-          }
-          __syncthreads();
-        }
-      }
-      // q^ and k^ in place; the factors of the state's rows
-      for (int it = tid; it < 4 * DP; it += NT) {
-        const int pr = it % (DP / 2), g = it / (DP / 2);
-        if (g < 2 * g_lo || g >= 2 * g_hi) continue;
-        float2 base = make_float2(0.f, 0.f), tot = make_float2(0.f, 0.f);
-        for (int j = 2 * g_lo; j < 2 * g_hi; ++j) {
-          const float2 v = *reinterpret_cast<const float2*>(sT + j * DP + 2 * pr);
-          if (j < g) { base.x += v.x; base.y += v.y; }
-          tot.x += v.x; tot.y += v.y;
-        }
-        // q^ = q exp2(b - qr), k^ = k exp2(kr - b)
-        const float2 qr = gentle ? make_float2(0.5f * tot.x, 0.5f * tot.y) : make_float2(0.f, 0.f);
-        const float2 kr = gentle ? qr : tot;
-        if (g == 2 * g_lo) {
-          const float2 e = make_float2(gl_ex2(qr.x), gl_ex2(qr.y));
-          float2* post = reinterpret_cast<float2*>(sPost + 2 * pr);
-          *reinterpret_cast<float2*>(sPre + 2 * pr) = make_float2(e.x * post->x, e.y * post->y);
-          if (!gentle) *reinterpret_cast<float2*>(sMid + 2 * pr) = make_float2(gl_ex2(tot.x), gl_ex2(tot.y));
-          *post = e;
-        }
-        const float2 qo = make_float2(base.x - qr.x + scale2, base.y - qr.y + scale2), ko = make_float2(kr.x - base.x, kr.y - base.y);
-#pragma unroll
-        for (int r = 0; r < 8; ++r) {
-          const int t = g * 8 + r;
-          const float2 bb = *reinterpret_cast<const float2*>(sB + t * BS + 2 * pr);
-          uint32_t* qp = reinterpret_cast<uint32_t*>(sq + t * QS + 2 * pr);
-          uint32_t* kp = reinterpret_cast<uint32_t*>(sk + t * QS + 2 * pr);
-          const float2 k = gl_unpack(*kp);
-          if (!p.carry) {
-            const float2 q = gl_unpack(*qp);
-            *qp = gl_pack(q.x * gl_ex2(bb.x + qo.x), q.y * gl_ex2(bb.y + qo.y));
-          }
-          *kp = gl_pack(k.x * gl_ex2(ko.x - bb.x), k.y * gl_ex2(ko.y - bb.y));
-        }
-      }
-      __syncthreads();
+      const bool gentle = !(harsh >> pc & 1);
       // the state as an operand, and the scores
       {
-        const float f0 = sPre[sd], f1 = sPre[sd + 8];
+        // the factor behind the last update and the one in front of the operand; the same one follows this update
+        const float e0 = sPre[pc * DP + sd], e1 = sPre[pc * DP + sd + 8], f0 = post0 * e0, f1 = post1 * e1;
+        post0 = e0;
+        post1 = e1;
 #pragma unroll
         for (int j = 0; j < NPW; ++j) {
           S[j][0] *= f0; S[j][1] *= f0; S[j][2] *= f1; S[j][3] *= f1;
@@ -502,7 +512,7 @@ __global__ void __launch_bounds__(kChunkThreads, 1) gla_chunk_kernel(const GlaPa
           }
         }
         if (!gentle) {
-          const float m0 = sMid[sd], m1 = sMid[sd + 8];
+          const float m0 = sMid[pc * DP + sd], m1 = sMid[pc * DP + sd + 8];
 #pragma unroll
           for (int j = 0; j < NPW; ++j) { S[j][0] *= m0; S[j][1] *= m0; S[j][2] *= m1; S[j][3] *= m1; }
         }
@@ -640,8 +650,7 @@ __global__ void __launch_bounds__(kChunkThreads, 1) gla_chunk_kernel(const GlaPa
     st = seg_s + (size_t)(seg + 1) * p.dim * p.vdim;
     if (v0 == 0 && tid < p.dim) seg_d[(size_t)(seg + 1) * p.dim + tid] = carried;
   } else if (ch1 < chunks) return;                         // the last segment leaves the state
-  const float post[2] = {sPost[sd], sPost[sd + 8]};
-  each_state([&](float& v, size_t at, bool in, int e) { if (in) st[at] = v * post[e]; });
+  each_state([&](float& v, size_t at, bool in, int e) { if (in) st[at] = v * (e ? post1 : post0); });
 }
 
 // Norm and gate of rows whose columns came from several CTAs: one warp per (token, head) of the sequences in question.
@@ -749,7 +758,7 @@ static int chunk_rank(const GlaParams& p, cudaStream_t st) {
 // Columns of the state per CTA of the chunk kernel for a key size, 0: it has no instance (the step kernel runs everything).
 extern "C" int xft_gla_chunk_columns(int dim, int vdim, int rank) {
   if (dim > 256 || rank > (dim > 128 ? 16 : 64) || dim <= 0) return 0;
-  return dim > 128 || vdim <= 64 ? 64 : 128;
+  return vdim <= 64 ? 64 : 128;
 }
 
 // x, a2 and out all fp32 (f32 = 1) or bf16; row strides and offsets as the file comment says, all multiples of 8 (a2's rows
@@ -786,7 +795,7 @@ extern "C" int xft_gla_chunk(const void* x, int ldx, int k_at, int v_at, int g_a
   GlaParams p{x, ldx, k_at, v_at, g_at, a_at, heads, dim, vdim, rank, rank_ld, a2, bias, 1.f / tau, scale, eps, gain, state, state_slots,
               num_states, cu_q, kv_lens, B, out, ldo, vdim > cols ? raw : nullptr, min_q, max_q, segs, 0, seg_state, seg_decay, status};
   int r;
-  if (dim > 128) r = launch_chunk<256, 64, 16>(p, st);
+  if (dim > 128) r = cols == 64 ? launch_chunk<256, 64, 16>(p, st) : launch_chunk<256, 128, 16>(p, st);
   else if (dim > 64) r = cols == 64 ? chunk_rank<128, 64>(p, st) : chunk_rank<128, 128>(p, st);
   else r = cols == 64 ? chunk_rank<64, 64>(p, st) : chunk_rank<64, 128>(p, st);
   if (r || !p.raw) return r;
