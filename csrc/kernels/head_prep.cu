@@ -39,6 +39,21 @@ template <typename T> __device__ __forceinline__ T hp_from(float v);
 template <> __device__ __forceinline__ float hp_from<float>(float v) { return v; }
 template <> __device__ __forceinline__ bf16 hp_from<bf16>(float v) { return __float2bfloat16(v); }
 
+template <int VEC>
+__device__ __forceinline__ void hp_pack(float (&e)[VEC], const float (&v)[VEC]) {
+#pragma unroll
+  for (int k = 0; k < VEC; ++k) e[k] = v[k];
+}
+template <int VEC>
+__device__ __forceinline__ void hp_pack(bf16 (&e)[VEC], const float (&v)[VEC]) {
+#pragma unroll
+  for (int k = 0; k < VEC; k += 2) {
+    const __nv_bfloat162 b = __floats2bfloat162_rn(v[k], v[k + 1]);
+    e[k] = b.x;
+    e[k + 1] = b.y;
+  }
+}
+
 // VEC neighbouring channels of a row, `left` of which exist; whole: they are aligned and exist all or not at all
 template <int VEC, typename T>
 __device__ __forceinline__ void hp_load(const T* p, int left, bool whole, float (&v)[VEC]) {
@@ -58,8 +73,7 @@ __device__ __forceinline__ void hp_store(T* p, const float (&v)[VEC], int left, 
   if (whole) {
     struct alignas(VEC * sizeof(T)) V { T e[VEC]; };
     V r;
-#pragma unroll
-    for (int k = 0; k < VEC; ++k) r.e[k] = hp_from<T>(v[k]);
+    hp_pack<VEC>(r.e, v);
     if (left > 0) *reinterpret_cast<V*>(p) = r;
   } else {
 #pragma unroll
@@ -79,7 +93,7 @@ __device__ __forceinline__ int hp_sequence(const int* cu_q, int B, int t) {     
 // A lane owns VEC neighbouring channels of every 32 VEC, NV times (padded <= 32 VEC NV); TAPS >= taps.  VEC 4: dim, row
 // strides and half the rotated dimensions are multiples of 4.
 template <typename T, int VEC, int NV, int TAPS>
-__global__ void __launch_bounds__(128) head_prep_kernel(const HeadPrepParams p) {
+__global__ void __launch_bounds__(128, TAPS * NV * VEC <= 16 ? 6 : 1) head_prep_kernel(const HeadPrepParams p) {
   extern __shared__ __align__(16) float hp_sm[];
   grid_dep_launch();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -116,18 +130,51 @@ __global__ void __launch_bounds__(128) head_prep_kernel(const HeadPrepParams p) 
   float u[TAPS][NV][VEC], next[NV][VEC];                 // the window, newest last; the row behind it
 #pragma unroll
   for (int i = 0; i < NV; ++i) hp_load<VEC>(x + (size_t)t0 * p.ldx + chan(i), p.dim - chan(i), whole, next[i]);
+  int start = p.cu_q[b], end = p.cu_q[b + 1];
+  int next_pos = p.rot > 0 ? p.positions[t0] : 0, next_slot = is_k ? p.slots[t0] : 0;
+  const float inv_dim = 1.f / (float)p.dim;
+  const int half = p.rot >> 1;
   bool fresh = true;
   for (int t = t0; t < t1; ++t) {
-    while (b + 1 < p.B && t >= p.cu_q[b + 1]) { ++b; fresh = true; }
-    const int start = p.cu_q[b], li = t - start;
+    while (b + 1 < p.B && t >= end) { ++b; start = end; end = p.cu_q[b + 1]; fresh = true; }
+    const int li = t - start;
+    // rotation: the angles' cosines and sines are on their way while the convolution runs
+    float cosv[NV][VEC], sinv[NV][VEC];
+    const int slot = next_slot;
+    if (p.rot > 0) {
+      int pos = next_pos;
+      if (pos < 0 || pos >= p.max_pos) { if (lane == 0 && p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); pos = 0; }
+      const float* cs = p.table + (size_t)pos * p.rot;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = chan(i);
+        if (c >= p.rot) continue;                        // rot is a multiple of VEC
+        if (VEC == 4) {                                  // all of them in the same half
+          const int f = c >= half ? c - half : c;
+          hp_load<VEC>(cs + f, VEC, true, cosv[i]);
+          hp_load<VEC>(cs + half + f, VEC, true, sinv[i]);
+        } else {
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) {
+            const int f = c + k >= half ? c + k - half : c + k;
+            cosv[i][k] = cs[f];
+            sinv[i][k] = cs[half + f];
+          }
+        }
+      }
+    }
+    if (t + 1 < t1) {
+      if (p.rot > 0) next_pos = p.positions[t + 1];
+      if (is_k) next_slot = p.slots[t + 1];
+    }
     T* st = nullptr;
     if (p.taps > 1 && (fresh || p.decode)) {
-      int slot = p.state_slots[b];
-      if (slot < 0 || slot >= p.num_states) { if (lane == 0 && p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); slot = 0; }
-      st = state + (size_t)slot * (p.taps - 1) * C + h * p.dim;
+      int s = p.state_slots[b];
+      if (s < 0 || s >= p.num_states) { if (lane == 0 && p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); s = 0; }
+      st = state + (size_t)s * (p.taps - 1) * C + h * p.dim;
     }
     if (fresh) {
-      const int past = p.kv_lens[b] - (p.cu_q[b + 1] - start);
+      const int past = p.kv_lens[b] - (end - start);
 #pragma unroll
       for (int j = 0; j < TAPS - 1; ++j) {
         const int idx = li - (TAPS - 1) + j;             // place in this portion; negative: before it
@@ -174,10 +221,9 @@ __global__ void __launch_bounds__(128) head_prep_kernel(const HeadPrepParams p) 
         for (int k = 0; k < VEC; ++k) u[j][i][k] = u[j + 1][i][k];
     T* dst;
     if (is_k) {
-      const long long slot = p.slots[t];
       if (slot < 0 || slot >= p.nslots) { if (lane == 0 && p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); continue; }
-      const int blk = (int)(slot / p.bs);
-      const size_t at = ((size_t)(blk * p.hkv + (h - p.hq)) * p.bs + (slot - (long long)blk * p.bs)) * p.padded;
+      const int blk = slot / p.bs;
+      const size_t at = ((size_t)(blk * p.hkv + (h - p.hq)) * p.bs + (slot - blk * p.bs)) * p.padded;
       dst = reinterpret_cast<T*>(p.kc) + at;
       T* v = reinterpret_cast<T*>(p.vc) + at;
 #pragma unroll
@@ -188,17 +234,13 @@ __global__ void __launch_bounds__(128) head_prep_kernel(const HeadPrepParams p) 
     if (norm) {
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-      const float inv = rsqrtf(ss / (float)p.dim + p.eps);
+      const float inv = rsqrtf(ss * inv_dim + p.eps);
 #pragma unroll
       for (int i = 0; i < NV; ++i)
 #pragma unroll
         for (int k = 0; k < VEC; ++k) y[i][k] *= inv * gain[i][k];
     }
     if (p.rot > 0) {
-      int pos = p.positions[t];
-      if (pos < 0 || pos >= p.max_pos) { if (lane == 0 && p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); pos = 0; }
-      const float* cs = p.table + (size_t)pos * p.rot;
-      const int half = p.rot >> 1;
       __syncwarp();
 #pragma unroll
       for (int i = 0; i < NV; ++i) hp_store<VEC>(row + chan(i), y[i], p.dim - chan(i), VEC == 4);
@@ -206,24 +248,16 @@ __global__ void __launch_bounds__(128) head_prep_kernel(const HeadPrepParams p) 
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         const int c = chan(i);
-        if (c >= p.rot) continue;                        // rot is a multiple of VEC
-        float other[VEC], cosv[VEC], sinv[VEC];
-        if (VEC == 4) {                                  // all of them in the same half
-          const int f = c >= half ? c - half : c;
-          hp_load<VEC>(row + (c >= half ? f : c + half), VEC, true, other);
-          hp_load<VEC>(cs + f, VEC, true, cosv);
-          hp_load<VEC>(cs + half + f, VEC, true, sinv);
+        if (c >= p.rot) continue;
+        float other[VEC];
+        if (VEC == 4) {
+          hp_load<VEC>(row + (c >= half ? c - half : c + half), VEC, true, other);
         } else {
 #pragma unroll
-          for (int k = 0; k < VEC; ++k) {
-            const int f = c + k >= half ? c + k - half : c + k;
-            other[k] = row[c + k >= half ? f : c + k + half];
-            cosv[k] = cs[f];
-            sinv[k] = cs[half + f];
-          }
+          for (int k = 0; k < VEC; ++k) other[k] = row[c + k >= half ? c + k - half : c + k + half];
         }
 #pragma unroll
-        for (int k = 0; k < VEC; ++k) y[i][k] = y[i][k] * cosv[k] + (c + k >= half ? other[k] : -other[k]) * sinv[k];
+        for (int k = 0; k < VEC; ++k) y[i][k] = y[i][k] * cosv[i][k] + (c + k >= half ? other[k] : -other[k]) * sinv[i][k];
       }
     }
 #pragma unroll
@@ -298,7 +332,7 @@ extern "C" int xft_head_prep(const void* x, int ldx, int T, int B, int hq, int h
   if (rot < 0 || rot > dim || (rot & 1) || (rot > 0 && !table) || (taps > 1 && (!conv || !state || !state_slots || num_states <= 0))) return -2;
   if ((dim & 1) == 0 && (ldx & 1)) return -3;
   if (B > 65535) return -4;
-  const int run = decode || T < 2048 ? 1 : 8;
+  const int run = decode || T < 2048 ? 1 : T < 8192 ? 8 : 16;
   HeadPrepParams p{x, ldx, T, B, hq, hkv, dim, padded, taps, conv, q_norm, k_norm, eps, positions, table, rot, max_pos, cu_q, kv_lens,
                    state, state_slots, num_states, q_out, kc, vc, bs, nslots, slots, run, decode, status};
   cudaError_t e = f32 ? pick_width<float>(p, st) : pick_width<bf16>(p, st);
