@@ -93,7 +93,7 @@ __device__ __forceinline__ int hp_sequence(const int* cu_q, int B, int t) {     
 // A lane owns VEC neighbouring channels of every 32 VEC, NV times (padded <= 32 VEC NV); TAPS >= taps.  VEC 4: dim, row
 // strides and half the rotated dimensions are multiples of 4.
 template <typename T, int VEC, int NV, int TAPS>
-__global__ void __launch_bounds__(128, TAPS * NV * VEC <= 16 ? 6 : 1) head_prep_kernel(const HeadPrepParams p) {
+__global__ void __launch_bounds__(128, (TAPS + 3) * NV * VEC <= 28 ? 6 : 1) head_prep_kernel(const HeadPrepParams p) {
   extern __shared__ __align__(16) float hp_sm[];
   grid_dep_launch();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
