@@ -69,9 +69,10 @@ def test_rows_and_order(cases, name):
     C.rows_and_order(cases(name), "fp32")
 
 
-def test_long_decoding(cases):
-    """Generation across several pages, far past every window."""
-    C.greedy(cases("large_heads"), "fp32", 5, 140)
+@pytest.mark.parametrize("name", ["large_heads", "recurrent", "recurrent_fast"])
+def test_long_decoding(cases, name):
+    """Generation across several pages, far past every window, over states that have long forgotten the prompt or never do."""
+    C.greedy(cases(name), "fp32", 5, 140)
 
 
 @pytest.mark.parametrize("name", ["shared", "latent", "recurrent"])
