@@ -1,4 +1,4 @@
-"""A plain, slow implementation of the layered designs (Kafipel, Vepivik, Botusun), one function per mechanism, for the tests to
+"""A plain, slow implementation of the layered designs (Kafipel, Vepivik, Botusun, Dagezen), one function per mechanism, for the tests to
 compare against.
 
 It works on one whole sequence at a time, without a cache, in the precision of the tensors it is given (tests use fp64
@@ -326,7 +326,7 @@ def feed_forward(h, W, prefix):
 def forward(cfg, W, tokens, layers_out=None, dtype=torch.float64):
     """Logits [T, vocab] of one sequence; `layers_out` (a list) collects the residual stream after every layer."""
     W = {n: (t.to(dtype) if t.is_floating_point() else t) for n, t in W.items()}
-    run = {"Kafipel": _kafipel, "Vepivik": _vepivik, "Botusun": _botusun}[cfg["architecture"]]
+    run = {"Kafipel": _kafipel, "Vepivik": _vepivik, "Botusun": _botusun, "Dagezen": _dagezen}[cfg["architecture"]]
     return run(cfg, W, tokens, [] if layers_out is None else layers_out)
 
 
@@ -385,6 +385,188 @@ def _botusun(cfg, W, tokens, layers_out):
             x = x + m * token_side(x, tokens, W, i, cfg["token_side"]["dim"], eps)
         layers_out.append(x.clone())
     return rms_norm(x, W["final.norm"], eps) @ W["embed"].T
+
+
+# ------------------------------------------------------------------------------------------ Dagezen
+def layer_norm_bias(x, w, b, eps):
+    return layer_norm(x, w, eps) + b
+
+
+def silu(z):
+    return z / (1 + torch.exp(-z))
+
+
+def softplus(z):
+    return torch.log1p(torch.exp(-z.abs())) + torch.clamp(z, min=0)
+
+
+def state_space(x, B, C, dt, A_log, D):
+    """x [T, H, P], B and C [T, G, N], dt [T, H] (after the softplus) -> [T, H, P]: per head
+    S <- exp(-exp(A_log) dt) S + dt B x^T,  y = S^T C + D x."""
+    T, H, P = x.shape
+    G, N = B.shape[1:]
+    S = torch.zeros(H, N, P, dtype=x.dtype)
+    group = [h // (H // G) for h in range(H)]
+    out = []
+    for t in range(T):
+        keep = torch.exp(-torch.exp(A_log) * dt[t])
+        S = keep[:, None, None] * S + (dt[t][:, None] * B[t][group])[:, :, None] * x[t][:, None, :]
+        out.append((S * C[t][group][:, :, None]).sum(1) + D[:, None] * x[t])
+    return torch.stack(out)
+
+
+def grouped_rms(y, w, n, eps):
+    """RMS norm of every row in `n` equal parts."""
+    T = y.shape[0]
+    parts = y.view(T, n, -1)
+    return (parts / torch.sqrt((parts * parts).mean(-1, keepdim=True) + eps)).reshape(T, -1) * w
+
+
+def mamba_mixer(h, m, W, prefix, eps):
+    T, H, P, N, G = h.shape[0], m["heads"], m["vdim"], m["state"], m["groups"]
+    Q, inner = prefix + ".mix.", m["heads"] * m["vdim"]
+    z, u, dt = torch.split(h @ W[Q + "in"].T, [inner, inner + 2 * G * N, H], 1)
+    u = silu(short_conv(u, W[Q + "conv"]) + W[Q + "conv.b"])
+    x, B, C = torch.split(u, [inner, G * N, G * N], 1)
+    dt = softplus(dt + W[Q + "dt_bias"])
+    y = state_space(x.view(T, H, P), B.view(T, G, N), C.view(T, G, N), dt, W[Q + "A_log"], W[Q + "D"]).reshape(T, -1)
+    return grouped_rms(y * silu(z), W[Q + "norm"], m["norm_groups"], eps) @ W[Q + "o"].T
+
+
+def sink_softmax(s, sink):
+    """Weights of the visible keys of one head with a score that has no key; s [T, T]."""
+    vis = visible(s.shape[-1], None)
+    s = torch.where(vis, s, torch.full_like(s, -math.inf))
+    top = torch.clamp(s.max(-1, keepdim=True).values, min=float(sink))
+    e = torch.exp(s - top)
+    return e / (e.sum(-1, keepdim=True) + torch.exp(sink - top))
+
+
+def latent_sink_mixer(h, m, W, prefix, positions, eps):
+    """Latent attention with a sink per head and one gate value per head."""
+    T, H, d, rd, R = h.shape[0], m["heads"], m["dim"], m["rot_dim"], m["kv_rank"]
+    P = prefix + ".mix."
+    q = (h @ W[P + "q"].T).view(T, H, d + rd).clone()
+    q[:, :, d:] = rotate(q[:, :, d:], positions, m["rot"], interleaved=True)
+    kv = h @ W[P + "dkv"].T
+    c = rms_norm(kv[:, :R], W[P + "dkv.norm"], eps)
+    kr = rotate(kv[:, None, R:], positions, m["rot"], interleaved=True)[:, 0]
+    s, v = latent_scores_and_values(q, c, kr, W[P + "uk"].view(H, d, R), W[P + "uv"].view(H, m["vdim"], R), m["scale"], rd)
+    a = torch.stack([sink_softmax(s[n], W[P + "sink"][n]) @ v[:, n] for n in range(H)], 1)
+    a = a * output_gate(h, W[P + "g"])[:, :, None]
+    return a.reshape(T, -1) @ W[P + "o"].T
+
+
+def distance_scores(q, k, scale, r1, r2):
+    """Scores of one head with the bias r1 ln(1 + r2 distance) taken off (keys behind the query: no meaning)."""
+    T = q.shape[0]
+    i = torch.arange(T, dtype=q.dtype)
+    return (q @ k.T) * scale - r1 * torch.log(1 + r2 * torch.clamp(i[:, None] - i[None, :], min=0))
+
+
+def talking_heads(w, T_):
+    """w [H, T, T] weights: head h gets sum_g T_[h, g] w[g]."""
+    return torch.einsum("hg,gij->hij", T_, w)
+
+
+def talking_mixer(h, m, W, P, eps):
+    """Attention whose values are its keys (before the norm), normalised over the whole projection, with a distance bias and
+    weights mixed between the heads.  -> before the output projection: [T, H * dim], gated."""
+    T, H, G, d = h.shape[0], m["heads"], m["kv_heads"], m["dim"]
+    q, k = h @ W[P + "q"].T, h @ W[P + "k"].T
+    v = k.view(T, G, d)
+    q, k = rms_norm(q, W[P + "q.norm"], eps).view(T, H, d), rms_norm(k, W[P + "k.norm"], eps).view(T, G, d)
+    own = [n // (H // G) for n in range(H)]
+    w = torch.stack([masked_softmax(distance_scores(q[:, n], k[:, own[n]], m["scale"], W[P + "r1"][n], W[P + "r2"][n]), m.get("mask"))
+                     for n in range(H)])
+    w = talking_heads(w, W[P + "talk"])
+    a = torch.stack([w[n] @ v[:, own[n]] for n in range(H)], 1).reshape(T, -1)
+    return (a * output_gate(h, W[P + "g"])) @ W[P + "o"].T
+
+
+def shifted(h):
+    """The previous token's row (zeros for the first)."""
+    return torch.cat([torch.zeros_like(h[:1]), h[:-1]])
+
+
+def time_mix(r, k, v, w, u):
+    """r, k, w [T, H, d], v [T, H, d], u [H, d]: o = (S + diag(u) k v^T)^T r, then S <- diag(w) S + k v^T."""
+    T, H, d = r.shape
+    S = torch.zeros(H, d, v.shape[2], dtype=r.dtype)
+    out = []
+    for t in range(T):
+        kv = k[t][:, :, None] * v[t][:, None, :]
+        out.append(((S + u[:, :, None] * kv) * r[t][:, :, None]).sum(1))
+        S = w[t][:, :, None] * S + kv
+    return torch.stack(out)
+
+
+def time_mixer(h, m, W, P, eps):
+    T, H, d = h.shape[0], m["heads"], m["dim"]
+    mix = {n: h + (shifted(h) - h) * W[P + "mu." + n] for n in "rkvgw"}
+    r, k, v = ((mix[n] @ W[P + n].T).view(T, H, d) for n in "rkv")
+    gate = silu(mix["g"] @ W[P + "g"].T)
+    w = torch.exp(-torch.exp(torch.tanh(mix["w"] @ W[P + "w1"].T) @ W[P + "w2"].T + W[P + "w0"]))
+    o = time_mix(r, k, v, w.view(T, H, d), W[P + "u"])
+    o = (o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps)).reshape(T, -1)
+    return (o * W[P + "norm"] * gate) @ W[P + "o"].T
+
+
+def parallel_mixer(h, m, W, prefix, eps):
+    P = prefix + ".mix."
+    return m["left_scale"] * talking_mixer(h, m["left"], W, P + "left.", eps) + \
+        m["right_scale"] * time_mixer(h, m["right"], W, P + "right.", eps)
+
+
+def clamped_feed_forward(h, f, W, prefix):
+    P, lim = prefix + ".mlp.", f["limit"]
+    g = torch.clamp(h @ W[P + "gate"].T + W[P + "gate.b"], max=lim)
+    u = torch.clamp(h @ W[P + "up"].T + W[P + "up.b"], min=-lim, max=lim)
+    return (g / (1 + torch.exp(-1.702 * g)) * (u + 1)) @ W[P + "down"].T + W[P + "down.b"]
+
+
+def gelu(z):
+    return 0.5 * z * (1 + torch.erf(z / math.sqrt(2)))
+
+
+def chosen_softmax(z, top):
+    """Chosen experts [T, top] (best first) and the softmax over their logits alone."""
+    idx = torch.argsort(z, -1, descending=True)[:, :top]
+    e = torch.exp(torch.gather(z, 1, idx) - z.max(-1, keepdim=True).values)
+    return idx, e / e.sum(-1, keepdim=True)
+
+
+def gelu_experts(h, f, W, prefix):
+    P = prefix + ".mlp."
+    idx, w = chosen_softmax(h @ W[P + "router"].T + W[P + "router.b"], f["router"]["top"])
+    out = torch.zeros(h.shape[0], W["embed"].shape[1], dtype=h.dtype)
+    for e in range(f["router"]["experts"]):
+        y = gelu(h @ W[P + f"e{e}.up"].T) @ W[P + f"e{e}.down"].T
+        out = out + y * torch.where(idx == e, w, torch.zeros_like(w)).sum(-1, keepdim=True)
+    return out
+
+
+def _dagezen(cfg, W, tokens, layers_out):
+    eps, alpha = cfg["norm"]["eps"], cfg["postln_alpha"]
+    positions = list(range(len(tokens)))
+    x = W["embed"][torch.tensor(tokens)]
+    norm = lambda v, n: layer_norm_bias(v, W[n], W[n + ".b"], eps)
+    for i, layer in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}", layer["mixer"], layer.get("mlp")
+        if layer["type"] == "mamba2":
+            y = mamba_mixer(x, m, W, p, eps)
+        elif layer["type"] == "latent_attention":
+            y = latent_sink_mixer(x, m, W, p, positions, eps)
+        else:
+            y = parallel_mixer(x, m, W, p, eps)
+        x = norm(alpha * x + y, p + ".norm1")
+        if f:
+            y = clamped_feed_forward(x, f, W, p) if f["kind"] == "dense" else gelu_experts(x, f, W, p)
+            x = norm(alpha * x + y, p + ".norm2")
+        layers_out.append(x.clone())
+    z = norm(x, "final.norm") @ W["embed"].T
+    cap = cfg.get("logit_softcap")
+    return cap * torch.tanh(z / cap) if cap else z
 
 
 # ------------------------------------------------------------------------------------------ small checkpoints

@@ -38,11 +38,14 @@ MODEL_TYPES = (
 )
 
 # config.json "architecture" -> model type
-ARCHITECTURES = {"Kafipel": "kafipel", "Vepivik": "vepivik", "Botusun": "botusun"}
+ARCHITECTURES = {"Kafipel": "kafipel", "Vepivik": "vepivik", "Botusun": "botusun", "Dagezen": "dagezen"}
 
 # what a design fixes about its mixers and experts beside what its config.json says
-MIXER_TRAITS = {"botusun": {"attention": dict(values_from_keys=True, qk_bias=True, qk_norm=True, sink=0.0)}}
-MOE_TRAITS = {"botusun": dict(act="silu", gated=True, scoring="sigmoid", renorm=False, correction=True)}
+MIXER_TRAITS = {"botusun": {"attention": dict(values_from_keys=True, qk_bias=True, qk_norm=True, sink=0.0)},
+                "dagezen": {"latent_attention": dict(gate="head", sinks=True)}}
+MOE_TRAITS = {"botusun": dict(act="silu", gated=True, scoring="sigmoid", renorm=False, correction=True),
+              "dagezen": dict(act="gelu_erf", scoring="chosen", router_bias=True)}
+DENSE_TRAITS = {"dagezen": dict(act="clamped", ff_bias=True)}
 
 
 def split_hybrid_dtype(dtype: str) -> Tuple[str, str]:
@@ -108,7 +111,8 @@ class MixerConfig:
 
     `kind` "latent": keys and values come from one latent of `kv_rank` values per token, expanded per head to `dim` key and
     `vdim` value dimensions, plus `rot_dim` rotated key dimensions that all heads share (kv_heads is 1: one cache row per
-    token).  `gate`: the concatenated heads are multiplied with sigmoid(W_g h).
+    token).  `gate` "value": the concatenated heads are multiplied with sigmoid(W_g h); "head": each head with one such value.
+    `sinks`: a learned sink per head joins the softmax.
 
     `conv` > 0: queries and keys go through a causal convolution of that many taps, channel by channel, straight after
     their projections (`qk_bias`: which have biases).  `values_from_keys`: the values are the keys as they leave it, before
@@ -116,7 +120,19 @@ class MixerConfig:
     heads share and that is no tensor.
 
     `kind` "gla": gated linear attention, heads of `dim` x `vdim` states that decay per key channel by
-    sigmoid(z)^(1 / `tau`); no cache, one fp32 state per sequence."""
+    sigmoid(z)^(1 / `tau`); no cache, one fp32 state per sequence.
+
+    `kind` "time_mix": a recurrence of the same shape over mixes of each token's input with the previous one's, with decays
+    exp(-exp(z)) and a bonus for the current token.
+
+    `kind` "ssd": a state-space recurrence (Mamba-2), heads of `dim` x `vdim` states with one decay per head and token; keys
+    and queries are shared by the heads of each of `groups`, inputs pass a convolution of `conv` taps, and outputs a norm in
+    `norm_groups` parts.
+
+    `kind` "talking": attention whose values are its keys, with norms over whole projections, a logarithmic distance bias and
+    weights that are mixed between the heads.
+
+    `kind` "parallel": the `parts`, side by side on the same input, their outputs summed with the factors `part_scales`."""
     heads: int
     kv_heads: int
     dim: int
@@ -130,18 +146,23 @@ class MixerConfig:
     kv_from: int = -1
     kv_rank: int = 0
     rot_dim: int = 0
-    gate: bool = False
+    gate: str = ""
+    sinks: bool = False
     conv: int = 0
     values_from_keys: bool = False
     qk_bias: bool = False
     qk_norm: bool = False
     sink: Optional[float] = None
     tau: float = 1.0
+    groups: int = 1
+    norm_groups: int = 1
+    parts: Tuple["MixerConfig", ...] = ()
+    part_scales: Tuple[float, ...] = ()
 
     @property
     def has_kv(self) -> bool:
         """Whether a layer with this mixer keeps keys and values (its own or another layer's)."""
-        return self.kind != "gla"
+        return self.kind not in ("gla", "time_mix", "ssd") and (not self.parts or any(p.has_kv for p in self.parts))
 
     def kv_shape(self) -> tuple:
         """What two layers must agree on for one to read the other's cache."""
@@ -153,7 +174,7 @@ class MixerConfig:
 @dataclass(frozen=True)
 class MoeConfig:
     """Mixture of experts of one layer: scores from `experts` router logits (`scoring`: softmax over them, or the sigmoid of
-    each), the `top` best, weighted with their scores (`renorm`: divided by their sum) times `scale`, and (`shared` > 0)
+    each; "chosen": softmax over the chosen ones' logits alone), the `top` best, weighted with their scores (`renorm`: divided by their sum) times `scale`, and (`shared` > 0)
     one more expert that every token uses.  `correction`: a tensor added to the scores for the choice alone.  `groups` > 1:
     only experts of the `keep_groups` groups with the best sum of two choice scores can be chosen.  An expert is
     down(act(up x)), or with `gated` down(act(gate x) * up x)."""
@@ -169,6 +190,7 @@ class MoeConfig:
     correction: bool = False
     groups: int = 1
     keep_groups: int = 1
+    router_bias: bool = False
 
 
 @dataclass(frozen=True)
@@ -177,6 +199,9 @@ class LayerConfig:
     ff: int = 0                       # width of a dense feed-forward; 0: none
     ff_kind: str = "dense"
     moe: Optional[MoeConfig] = None
+    act: str = "silu"                 # of the dense feed-forward's gate; "clamped" takes `limit` (see ops.linear_gated)
+    limit: float = 0.0
+    ff_bias: bool = False
 
 
 @dataclass(frozen=True)
@@ -237,6 +262,8 @@ class ModelConfig:
     layers: List[LayerConfig] = field(default_factory=list)
     embed_scale: float = 1.0
     residual_mult: float = 1.0        # factor of every sublayer's output in the residual sum
+    residual_carry: float = 1.0       # factor of the stream itself in the residual sum
+    logit_softcap: float = 0.0        # > 0: logits become cap * tanh(logits / cap)
     loop: Optional[LoopConfig] = None
     side_dim: int = 0                 # > 0: each layer also gets so many values of the token's own side embedding
     # raw key/value pairs (for family-specific look-ups, like DecoderContext::GetAttr)
@@ -321,7 +348,8 @@ class ModelConfig:
                    vocab_size=int(d["vocab"]), layernorm_eps=float(d["norm"]["eps"]), start_id=-1, end_id=-1,
                    weight_data_type="bf16", layers=layers, raw=d,
                    embed_scale=float((d.get("embedding") or {}).get("scale", 1.0)),
-                   residual_mult=float(d.get("residual_mult", 1.0)), loop=loop,
+                   residual_mult=float(d.get("residual_mult", 1.0)), residual_carry=float(d.get("postln_alpha", 1.0)),
+                   logit_softcap=float(d.get("logit_softcap") or 0.0), loop=loop,
                    side_dim=int((d.get("token_side") or {}).get("dim", 0)))
 
     @classmethod
@@ -503,38 +531,71 @@ def _rotary(i: int, m: dict, width: int, style: str) -> Optional[RotaryConfig]:
     return rot
 
 
-def _layer_config(i: int, e: dict, model_type: str) -> LayerConfig:
-    """One entry of config.json's ``layers``."""
-    kind, m = e.get("type"), e["mixer"]
+def _mixer_config(i: int, kind: str, m: dict, model_type: str) -> MixerConfig:
+    if kind == "parallel":
+        parts = tuple(_mixer_config(i, k, m[name], model_type) for name, k in PARALLEL_PARTS)
+        q = parts[0]
+        return MixerConfig(kind="parallel", heads=q.heads, kv_heads=q.kv_heads, dim=q.dim, vdim=q.vdim, scale=q.scale, window=q.window,
+                           parts=parts, part_scales=tuple(float(m.get(name + "_scale", 1.0)) for name, _ in PARALLEL_PARTS))
+    if kind not in ("attention", "latent_attention", "gla", "time_mix", "mamba2", "talking"):
+        raise ValueError(f"layer {i}: unsupported mixer type {kind!r}")
     mask = m.get("mask") or {}
-    common = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m.get("vdim", m["dim"])),
-                  scale=float(m["scale"] if kind != "gla" else int(m["dim"]) ** -0.5),
+    dim = int(m["state"] if kind == "mamba2" else m["dim"])
+    scale = {"gla": dim ** -0.5, "mamba2": 1.0, "time_mix": 1.0}.get(kind)
+    common = dict(heads=int(m["heads"]), dim=dim, vdim=int(m.get("vdim", dim)),
+                  scale=float(m["scale"]) if scale is None else scale,
                   window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0),
                   softcap=float(m.get("softcap") or 0.0), kv_from=-1 if m.get("kv_from") is None else int(m["kv_from"]),
                   conv=int(m.get("conv") or 0), **MIXER_TRAITS.get(model_type, {}).get(kind, {}))
     if kind == "attention":
-        mixer = MixerConfig(kv_heads=int(m.get("kv_heads", m["heads"])), rot=_rotary(i, m, int(m["dim"]), "half"), **common)
-    elif kind == "latent_attention":
+        return MixerConfig(kv_heads=int(m.get("kv_heads", m["heads"])), rot=_rotary(i, m, dim, "half"), **common)
+    if kind == "latent_attention":
         rd = int(m["rot_dim"])
         mixer = MixerConfig(kind="latent", kv_heads=1, rot=_rotary(i, m, rd, "interleaved"), kv_rank=int(m["kv_rank"]), rot_dim=rd,
-                            gate=True, **common)
+                            **{"gate": "value", **common})
         if mixer.keep_first or mixer.softcap:
             raise ValueError(f"layer {i}: latent attention has no kept first keys and no cap on the scores")
-    elif kind == "gla":
-        mixer = MixerConfig(kind="gla", kv_heads=common["heads"], tau=float(m["tau"]), **common)
-    else:
-        raise ValueError(f"layer {i}: unsupported mixer type {kind!r}")
+        return mixer
+    if kind == "gla":
+        return MixerConfig(kind="gla", kv_heads=common["heads"], tau=float(m["tau"]), **common)
+    if kind == "time_mix":
+        return MixerConfig(kind="time_mix", kv_heads=common["heads"], **common)
+    if kind == "mamba2":
+        mixer = MixerConfig(kind="ssd", kv_heads=common["heads"], groups=int(m["groups"]), norm_groups=int(m["norm_groups"]), **common)
+        if mixer.groups < 1 or mixer.heads % mixer.groups or mixer.norm_groups < 1 or mixer.heads * mixer.vdim % mixer.norm_groups:
+            raise ValueError(f"layer {i}: {mixer.heads} heads of {mixer.vdim} in {mixer.groups} groups, normalised in {mixer.norm_groups}")
+        return mixer
+    return MixerConfig(kind="talking", kv_heads=int(m.get("kv_heads", m["heads"])), values_from_keys=True, **common)
+
+
+# what a parallel mixer consists of: (key in its entry and prefix of its tensors, mixer type)
+PARALLEL_PARTS = (("left", "talking"), ("right", "time_mix"))
+
+
+def _check_mixer(i: int, mixer: MixerConfig) -> None:
     if mixer.heads % mixer.kv_heads:
         raise ValueError(f"layer {i}: {mixer.heads} query heads over {mixer.kv_heads} key/value heads")
     if mixer.values_from_keys and (mixer.dim != mixer.vdim or mixer.kv_from >= 0):
         raise ValueError(f"layer {i}: values that are keys have the keys' size and a cache of their own")
-    if mixer.conv and not mixer.values_from_keys:
-        raise ValueError(f"layer {i}: a short convolution is for layers whose values are their keys")
+    if mixer.conv and not mixer.values_from_keys and mixer.kind != "ssd":
+        raise ValueError(f"layer {i}: a short convolution is for layers whose values are their keys and for state-space layers")
+    if mixer.kind == "talking" and (mixer.keep_first or mixer.softcap or mixer.conv):
+        raise ValueError(f"layer {i}: mixed heads have no kept first keys, no cap and no convolution")
+    if mixer.kind == "time_mix" and mixer.dim != mixer.vdim:
+        raise ValueError(f"layer {i}: time mixing has values of the keys' size")
+    for p in mixer.parts:
+        _check_mixer(i, p)
+
+
+def _layer_config(i: int, e: dict, model_type: str) -> LayerConfig:
+    """One entry of config.json's ``layers``."""
+    mixer = _mixer_config(i, e.get("type"), e["mixer"], model_type)
+    _check_mixer(i, mixer)
     f = e.get("mlp")
     if not f:
         return LayerConfig(mixer)
     if f.get("kind") == "dense":
-        return LayerConfig(mixer, int(f["ff"]), "dense")
+        return LayerConfig(mixer, int(f["ff"]), "dense", limit=float(f.get("limit") or 0.0), **DENSE_TRAITS.get(model_type, {}))
     if f.get("kind") != "moe":
         raise ValueError(f"layer {i}: unsupported feed-forward {f.get('kind')!r}")
     r = f["router"]

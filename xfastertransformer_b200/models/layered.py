@@ -1,4 +1,4 @@
-"""Decoder for designs described layer by layer (``ModelConfig.layers``): Kafipel, Vepivik, Botusun.
+"""Decoder for designs described layer by layer (``ModelConfig.layers``): Kafipel, Vepivik, Botusun, Dagezen.
 
 It is the generic decoder with sizes, rotation, mask and cache pool taken from each layer's own entry, served by the same
 engine, paged cache, decode runner, sampler and kernels.  What these designs add to it, each as an op with its constants
@@ -17,6 +17,14 @@ as arguments:
 * gated linear attention, a recurrent layer with a state instead of a cache (`ops.gated_linear`);
 * mixtures of experts with or without a gate product, chosen by group or among all (`ops.route`, `ops.moe_experts`), next to
   a shared expert;
+* a residual stream that is the norm of alpha * x + sublayer(x), the sublayers reading the stream itself
+  (`FamilySpec.sum_norm`);
+* state-space layers (`ops.state_space`): convolution, recurrence and grouped norm between their two projections;
+* mixers side by side on the same input (`MixerConfig.parts`), with one output projection over all of their heads: attention
+  with mixed heads (`ops.talking_prep`, `ops.talking_attention`) and time mixing (`ops.token_shift`, `ops.gated_linear` with a
+  bonus);
+* dense feed-forwards with a clamped gate and biases, experts weighted by the softmax over the chosen ones, a tanh cap on the
+  logits;
 * layers that run several times in a row (`ModelConfig.runs`), each pass with a cache and states of its own;
 * a part of the token's own side embedding after every layer, gated by the residual stream;
 * a scaled embedding, a factor on everything that joins the residual stream, and logits from the embedding table.
@@ -35,7 +43,7 @@ from typing import Dict, List, Optional
 import torch
 
 from .. import ops
-from ..config import LayerConfig, ModelConfig, MoeConfig, RotaryConfig
+from ..config import PARALLEL_PARTS, LayerConfig, MixerConfig, ModelConfig, MoeConfig, RotaryConfig
 from ..ops import reference as R
 from ..parallel import partition as P
 from ..parallel.dist import DistContext
@@ -90,22 +98,23 @@ class LayeredDecoder(Decoder):
         self.runs: List[Layer] = []
         for i, t in runs:
             L = copy.copy(loaded[i])
+            L.parts = [copy.copy(q) for q in L.parts]
             L.step = self._step_vector(t) if cfg.loop is not None and i == cfg.loop.start and t >= 0 else None
             self.runs.append(L)
         # cache pools: one per run with keys and values of its own; state pools: the ones each run asks for
         self.pools: Dict[int, int] = {}
         self.pool_shapes, self.state_shapes = [], []
         for L in self.runs:
-            if L.own_kv:
-                self.pools[L.idx] = len(self.pool_shapes)
-                self.pool_shapes.append((1, L.kd, 0) if L.mix.kind == "latent" else (L.hkv, L.kd, L.vd))
-            L.pool = self.pools.get(L.kv_layer, -1)
-            if L.pool < 0 and L.mix.has_kv:
-                raise ValueError(f"layer {L.idx} reads the keys of layer {L.kv_layer}, which is on another pipeline stage")
-            if L.state_shape is not None:
-                L.state = len(self.state_shapes)
-                self.state_shapes.append(L.state_shape)
-        L = self.layers[0]
+            for q in L.parts or [L]:
+                if q.own_kv:
+                    self.pools[L.idx] = len(self.pool_shapes)
+                    self.pool_shapes.append((1, q.kd, 0) if q.mix.kind == "latent" else (q.hkv, q.kd, q.vd))
+                q.pool = self.pools.get(q.kv_layer, -1)
+                if q.pool < 0 and q.mix.has_kv:
+                    raise ValueError(f"layer {L.idx} reads the keys of layer {q.kv_layer}, which is on another pipeline stage")
+                q.state = list(range(len(self.state_shapes), len(self.state_shapes) + len(q.state_shapes)))
+                self.state_shapes.extend(q.state_shapes)
+        L = (self.layers[0].parts or self.layers)[0]
         self.D, self.hq, self.hkv, self.group, self.scale = L.kd, L.hq, L.hkv, L.group, L.mix.scale
         for L in self.layers:
             self._rope(L.mix.rot, 2048)
@@ -141,7 +150,8 @@ class LayeredDecoder(Decoder):
     # weights
     # ------------------------------------------------------------------------------------
     def _gain(self, name: str):
-        return self.src.vector(name, self.W, fake_ones=True), None      # (gain, bias)
+        bias = self.src.vector(name + ".b", self.W) if self.spec.norm_bias else None
+        return self.src.vector(name, self.W, fake_ones=True), bias
 
     def _step_vector(self, t: int) -> torch.Tensor:
         """What joins the residual stream in front of pass `t` of the looped layers."""
@@ -189,49 +199,54 @@ class LayeredDecoder(Decoder):
 
     def _out_rows(self, L: Layer, p: str, heads: int, rng, vdim: int, width: int = 0) -> None:
         """The output projection: its columns are heads of `vdim`, padded to L.vd, and all of them to `width`."""
-        w = self.src.matrix(p + "mix.o", (self.W, heads * vdim), cols=(rng[0] * vdim, rng[1] * vdim))
+        w = self.src.matrix(p + "o", (self.W, heads * vdim), cols=(rng[0] * vdim, rng[1] * vdim))
         w = _pad(w.reshape(self.W, L.hq, vdim), self.WP, L.hq, L.vd).reshape(self.WP, L.hq * L.vd)
-        L.o = make_linear(_pad(w, self.WP, max(width, L.hq * L.vd)), self.kind)
+        L.o_rows = _pad(w, self.WP, max(width, L.hq * L.vd))
 
     def _load_layer(self, i: int) -> Layer:
         lc: LayerConfig = self.cfg.layers[i]
         m = lc.mixer
-        L = Layer()
-        L.idx, L.mix, L.ff = i, m, lc.ff
         p = f"l{i}."
-        # this rank's heads; query head h reads key/value head h // (heads / kv_heads)
-        (qs, qe), (ks, ke) = P.head_range(m.heads, m.kv_heads, self.tp, self.tpr)
-        L.hq, L.hkv, L.group = qe - qs, ke - ks, m.heads // m.kv_heads
-        L.q_off = qs - ks * L.group
-        if L.hq <= 0:
-            raise ValueError(f"layer {i}: {m.heads} heads cannot be split over {self.tp} ranks")
-        L.own_kv = m.has_kv and m.kv_from < 0
-        L.state_shape = None
-        L.kv_layer = i if L.own_kv else m.kv_from
+        L = Layer()
+        L.idx, L.ff = i, lc.ff
         second = self._gain if self.spec.post_norm else lambda name: None
         L.norm1, L.norm1b = self._gain(p + "norm1"), second(p + "norm1b")
-        if m.kind == "latent":
-            self._load_latent(L, p, (qs, qe))
-        elif m.kind == "gla":
-            self._load_linear(L, p, (qs, qe))
-        elif m.values_from_keys:
-            self._load_shared_kv(L, p, (qs, qe), (ks, ke))
+        L.parts = []
+        if m.parts:
+            L.mix, L.own_kv, L.state_shapes = m, False, []
+            for (name, _), q, mult in zip(PARALLEL_PARTS, m.parts, m.part_scales):
+                Q = Layer()
+                Q.idx, Q.mult = i, mult
+                self._load_mixer(Q, f"{p}mix.{name}.", q)
+                Q.width = Q.o_rows.shape[1]
+                L.parts.append(Q)
+            # one output projection over all parts' heads
+            L.o = make_linear(torch.cat([q.o_rows for q in L.parts], 1), self.kind)
+            for q in L.parts:
+                del q.o_rows
         else:
-            self._load_attention(L, p, (qs, qe), (ks, ke))
+            L.mult = 1.0
+            self._load_mixer(L, p + "mix.", m)
+            L.o = make_linear(L.o_rows, self.kind)
+            del L.o_rows
         L.mlp_kind = "none"
         if lc.ff_kind == "moe" or lc.ff:
             L.norm2, L.norm2b = self._gain(p + "norm2"), second(p + "norm2b")
         if lc.ff_kind == "moe":
             self._load_experts(L, p, lc.moe)
         elif lc.ff:
-            L.mlp_kind = "llama"
+            L.mlp_kind, gpu = "llama", self.device.type == "cuda"
             r = self._ffn_range(lc.ff)
             n = r[1] - r[0]
             np_ = self._ff_size(n)
             gate, up = (_pad(self.src.matrix(p + "mlp." + x, (lc.ff, self.W), rows=r), np_, self.WP) for x in ("gate", "up"))
-            L.gate_up = make_linear(torch.cat([gate, up]), self.kind)
+            kind = "bf16" if gpu and lc.act == "clamped" and not self.exact else self.kind       # not in the quantised products
+            L.gate_up = make_linear(torch.cat([gate, up]), kind)
             L.down = make_linear(_pad(self.src.matrix(p + "mlp.down", (self.W, lc.ff), cols=r), self.WP, np_), self.kind)
-            L.act = "silu"
+            L.act, L.limit, L.gate_up_b, L.down_b = lc.act, lc.limit, None, None
+            if lc.ff_bias:
+                L.gate_up_b = torch.cat([_pad(self.src.vector(f"{p}mlp.{x}.b", lc.ff, rng=r), np_) for x in ("gate", "up")]).contiguous()
+                L.down_b = _pad(self.src.vector(p + "mlp.down.b", self.W), self.WP).contiguous()
         L.side_gate = None
         if self.cfg.side_dim:
             d, kind = self.cfg.side_dim, "fp32" if self.exact or self.device.type == "cpu" else "bf16"
@@ -242,6 +257,35 @@ class LayeredDecoder(Decoder):
             L.side_at = i * n
         return L
 
+    def _load_mixer(self, L: Layer, p: str, m: MixerConfig) -> None:
+        """Weights of one mixer, the tensors `p`*; leaves its output projection in L.o_rows."""
+        L.mix = m
+        L.replicated = m.kind in ("ssd", "talking", "time_mix")      # norms, groups and mixes go across heads: on every rank
+        tp, tpr = (1, 0) if L.replicated else (self.tp, self.tpr)
+        # this rank's heads; query head h reads key/value head h // (heads / kv_heads)
+        (qs, qe), (ks, ke) = P.head_range(m.heads, m.kv_heads, tp, tpr)
+        L.hq, L.hkv, L.group = qe - qs, ke - ks, m.heads // m.kv_heads
+        L.q_off = qs - ks * L.group
+        if L.hq <= 0:
+            raise ValueError(f"layer {L.idx}: {m.heads} heads cannot be split over {tp} ranks")
+        L.own_kv = m.has_kv and m.kv_from < 0
+        L.state_shapes = []
+        L.kv_layer = L.idx if L.own_kv else m.kv_from
+        if m.kind == "latent":
+            self._load_latent(L, p, (qs, qe))
+        elif m.kind == "gla":
+            self._load_linear(L, p, (qs, qe))
+        elif m.kind == "ssd":
+            self._load_state_space(L, p)
+        elif m.kind == "talking":
+            self._load_talking(L, p)
+        elif m.kind == "time_mix":
+            self._load_time_mix(L, p)
+        elif m.values_from_keys:
+            self._load_shared_kv(L, p, (qs, qe), (ks, ke))
+        else:
+            self._load_attention(L, p, (qs, qe), (ks, ke))
+
     def _ff_size(self, n: int) -> int:
         return _up(n, 8) if self.device.type == "cuda" else n
 
@@ -250,21 +294,21 @@ class LayeredDecoder(Decoder):
         L.kd, L.vd = self._head_size(m.dim), self._head_size(m.vdim)
         if self.pad_heads:
             L.kd = L.vd = max(L.kd, L.vd)         # the tensor-core kernels have one size for keys and values
-        parts = [self._rows(p + "mix.q", m.heads, q, (m.dim, L.kd))]
+        parts = [self._rows(p + "q", m.heads, q, (m.dim, L.kd))]
         if L.own_kv:
-            parts.append(self._rows(p + "mix.k", m.kv_heads, kv, (m.dim, L.kd)))
-            parts.append(self._rows(p + "mix.v", m.kv_heads, kv, (m.vdim, L.vd)))
+            parts.append(self._rows(p + "k", m.kv_heads, kv, (m.dim, L.kd)))
+            parts.append(self._rows(p + "v", m.kv_heads, kv, (m.vdim, L.vd)))
         L.qkv = make_linear(torch.cat(parts), self.kind)
         L.sinks = None
-        if self.spec.sinks and (self.src.exists(p + "mix.sink") or self.src.fake):
-            L.sinks = self.src.vector(p + "mix.sink", m.heads, rng=q).contiguous()
+        if self.spec.sinks and (self.src.exists(p + "sink") or self.src.fake):
+            L.sinks = self.src.vector(p + "sink", m.heads, rng=q).contiguous()
         self._out_rows(L, p, m.heads, q, m.vdim)
 
     def _load_shared_kv(self, L: Layer, p: str, q, kv) -> None:
         """Attention whose values are its keys.  Rows leave the projection with the heads' real size; `head_prep` pads them."""
         m, n = L.mix, (L.hq + L.hkv) * L.mix.dim
         L.kd = L.vd = self._head_size(m.dim)
-        parts = [(p + "mix.q", m.heads, q), (p + "mix.k", m.kv_heads, kv)]
+        parts = [(p + "q", m.heads, q), (p + "k", m.kv_heads, kv)]
         w = torch.cat([self._rows(name, heads, rng, (m.dim, m.dim)) for name, heads, rng in parts])
         L.qkv = make_linear(_pad(w, self._ff_size(n), self.WP), self.kind)
         cut = lambda rng: (rng[0] * m.dim, rng[1] * m.dim)
@@ -277,8 +321,8 @@ class LayeredDecoder(Decoder):
             conv = [self.src.matrix(name + ".conv", (heads * m.dim, m.conv), rows=cut(rng)) for name, heads, rng in parts]
             conv = torch.cat(conv).float().t().contiguous()                # [taps, channels]
             if m.conv > 1:
-                L.state_shape = ((m.conv - 1, n), self.act_dtype)
-        norms = [self.src.vector(p + f"mix.{x}.norm", m.dim, fake_ones=True).contiguous() if m.qk_norm else None for x in "qk"]
+                L.state_shapes.append(((m.conv - 1, n), self.act_dtype))
+        norms = [self.src.vector(p + f"{x}.norm", m.dim, fake_ones=True).contiguous() if m.qk_norm else None for x in "qk"]
         L.prep = ops.HeadPrep(L.hq, L.hkv, m.dim, L.kd, conv, *norms)
         L.sinks = None if m.sink is None else torch.full((L.hq,), m.sink, dtype=torch.float32, device=self.device)
         self._out_rows(L, p, m.heads, q, m.vdim)
@@ -286,39 +330,94 @@ class LayeredDecoder(Decoder):
     def _load_linear(self, L: Layer, p: str, rng) -> None:
         """Gated linear attention: queries, keys, values, output gate and the decay's first product are one projection."""
         m, gpu = L.mix, self.device.type == "cuda"
-        rank = self.src.shape(p + "mix.a1", (16, self.W))[0]
+        rank = self.src.shape(p + "a1", (16, self.W))[0]
         d = L.dims = ops.LinearDims(L.hq, m.dim, m.vdim, rank, 8 if gpu else 1)
         L.kd, L.vd = m.dim, m.vdim
-        rows = [self._rows(p + "mix." + x, m.heads, rng, (n, n)) for x, n in (("q", m.dim), ("k", m.dim), ("v", m.vdim), ("g", m.vdim))]
-        rows.append(_pad(self.src.matrix(p + "mix.a1", (rank, self.W)), rank, self.WP))
+        rows = [self._rows(p + "" + x, m.heads, rng, (n, n)) for x, n in (("q", m.dim), ("k", m.dim), ("v", m.vdim), ("g", m.vdim))]
+        rows.append(_pad(self.src.matrix(p + "a1", (rank, self.W)), rank, self.WP))
         L.qkv = make_linear(torch.cat([_pad(r, d.up(r.shape[0]), self.WP) for r in rows]), self.kind)
-        a2 = self.src.matrix(p + "mix.a2", (m.heads * m.dim, rank), rows=(rng[0] * m.dim, rng[1] * m.dim)).to(self.act_dtype)
-        bias = self.src.vector(p + "mix.a2.b", m.heads * m.dim, rng=(rng[0] * m.dim, rng[1] * m.dim))
-        gain = self.src.vector(p + "mix.norm", m.vdim, fake_ones=True)
+        a2 = self.src.matrix(p + "a2", (m.heads * m.dim, rank), rows=(rng[0] * m.dim, rng[1] * m.dim)).to(self.act_dtype)
+        bias = self.src.vector(p + "a2.b", m.heads * m.dim, rng=(rng[0] * m.dim, rng[1] * m.dim))
+        gain = self.src.vector(p + "norm", m.vdim, fake_ones=True)
         L.decay = ops.LinearWeights(_pad(a2, a2.shape[0], d.up(rank)).contiguous(), bias.contiguous(), m.tau, gain.contiguous())
-        L.state_shape = ((L.hq, m.dim, m.vdim), torch.float32)
+        L.state_shapes.append(((L.hq, m.dim, m.vdim), torch.float32))
         self._out_rows(L, p, m.heads, rng, m.vdim, d.up(L.hq * m.vdim))
+
+    def _load_state_space(self, L: Layer, p: str) -> None:
+        """Mamba-2: gate, convolved channels and step sizes are one projection."""
+        m, gpu = L.mix, self.device.type == "cuda"
+        H, n = m.heads, m.heads * m.vdim
+        d = L.dims = ops.StateDims(H, m.dim, m.vdim, m.groups, m.norm_groups, max(m.conv, 1), 8 if gpu else 1)
+        L.kd, L.vd = m.dim, m.vdim
+        w = self.src.matrix(p + "in", (n + d.channels + H, self.W))
+        rows = [w[:n], w[n:n + d.channels], w[n + d.channels:]]
+        L.qkv = make_linear(torch.cat([_pad(r, d.up(r.shape[0]), self.WP) for r in rows]), self.kind)
+        f32 = lambda name, k: self.src.vector(p + name, k).contiguous()
+        conv = self.src.matrix(p + "conv", (d.channels, d.taps)).float().t().contiguous()              # [taps, channels]
+        L.ssm = ops.StateWeights(conv, f32("conv.b", d.channels), f32("dt_bias", H), torch.exp(f32("A_log", H)), f32("D", H),
+                                 self.src.vector(p + "norm", n, fake_ones=True).contiguous())
+        L.state_shapes.append(((H, m.dim, m.vdim), torch.float32))
+        if d.taps > 1:
+            L.state_shapes.append(((d.taps - 1, d.channels), self.act_dtype))
+        self._out_rows(L, p, H, (0, H), m.vdim, d.up(n))
+
+    def _load_talking(self, L: Layer, p: str) -> None:
+        """Attention with mixed heads: queries, keys and gate are one projection; heads are padded behind the norms."""
+        m, gpu = L.mix, self.device.type == "cuda"
+        L.kd = L.vd = self._head_size(m.dim)
+        f32 = lambda name, k, ones=False: self.src.vector(p + name, k, fake_ones=ones).contiguous()
+        talk = self.src.matrix(p + "talk", (m.heads, m.heads)).float().contiguous()
+        d = L.talk = ops.TalkingHeads(m.heads, m.kv_heads, m.dim, L.kd, f32("q.norm", m.heads * m.dim, True),
+                                      f32("k.norm", m.kv_heads * m.dim, True), f32("r1", m.heads), f32("r2", m.heads), talk,
+                                      L.mult, 8 if gpu else 1)
+        rows = [self._rows(p + "q", m.heads, (0, m.heads), (m.dim, m.dim)),
+                self._rows(p + "k", m.kv_heads, (0, m.kv_heads), (m.dim, m.dim)),
+                self._rows(p + "g", m.heads, (0, m.heads), (m.vdim, L.vd))]
+        L.qkv = make_linear(torch.cat([_pad(r, d.up(r.shape[0]), self.WP) for r in rows]), self.kind)
+        self._out_rows(L, p, m.heads, (0, m.heads), m.vdim)
+
+    def _load_time_mix(self, L: Layer, p: str) -> None:
+        """Time mixing: four products of one size on four mixes of the input, and the decay's two."""
+        m, gpu = L.mix, self.device.type == "cuda"
+        n, rank = m.heads * m.dim, self.src.shape(p + "w1", (32, self.W))[0]
+        d = L.dims = ops.LinearDims(m.heads, m.dim, m.vdim, rank, 8 if gpu else 1)
+        L.kd, L.vd = m.dim, m.vdim
+        L.mu = torch.stack([_pad(self.src.vector(p + "mu." + x, self.W), self.WP) for x in "rkvgw"]).contiguous()
+        rows = [self._rows(p + x, m.heads, (0, m.heads), (m.dim, m.dim)) for x in "rkvg"]
+        kind = "fp32" if self.exact or self.device.type == "cpu" else "bf16"
+        L.rkvg = make_linear(torch.cat([_pad(r, d.up(n), self.WP) for r in rows]), kind)
+        L.w1 = make_linear(_pad(self.src.matrix(p + "w1", (rank, self.W)), d.up(rank), self.WP), kind)
+        a2 = self.src.matrix(p + "w2", (n, rank)).to(self.act_dtype)
+        L.decay = ops.LinearWeights(_pad(a2, n, d.up(rank)).contiguous(), self.src.vector(p + "w0", n).contiguous(), 1.0,
+                                    self.src.vector(p + "norm", n, fake_ones=True).contiguous(), 1.0,
+                                    self.src.matrix(p + "u", (m.heads, m.dim)).float().contiguous(), L.mult)
+        L.state_shapes.append(((m.heads, m.dim, m.vdim), torch.float32))
+        L.state_shapes.append(((self.WP,), torch.float32))
+        self._out_rows(L, p, m.heads, (0, m.heads), m.vdim, d.up(n))
 
     def _load_latent(self, L: Layer, p: str, q) -> None:
         """Latent attention: heads are split over ranks, the latents (one row per token) are on every rank."""
         m = L.mix
         size = (lambda n: _up(n, 64)) if self.pad_heads else (lambda n: n)
         rank = next((r for r in LATENTS if m.kv_rank <= r), size(m.kv_rank)) if self.pad_heads else m.kv_rank
-        d = L.dims = ops.LatentDims(L.hq, size(m.dim), size(m.rot_dim), rank, size(m.vdim), L.own_kv, m.gate, m.kv_rank)
+        d = L.dims = ops.LatentDims(L.hq, size(m.dim), size(m.rot_dim), rank, size(m.vdim), L.own_kv, bool(m.gate), m.kv_rank,
+                                  m.gate == "head", 8 if self.device.type == "cuda" else 1)
         L.kd, L.vd = d.rank + d.rot, d.vdim
-        parts = [self._rows(p + "mix.q", m.heads, q, (m.dim, d.dim), (m.rot_dim, d.rot))]
+        parts = [self._rows(p + "q", m.heads, q, (m.dim, d.dim), (m.rot_dim, d.rot))]
         L.latent_norm = None
         if L.own_kv:
-            parts.append(self._rows(p + "mix.dkv", 1, (0, 1), (m.kv_rank, d.rank), (m.rot_dim, d.rot)))
-            L.latent_norm = _pad(self.src.vector(p + "mix.dkv.norm", m.kv_rank, fake_ones=True), d.rank)
+            parts.append(self._rows(p + "dkv", 1, (0, 1), (m.kv_rank, d.rank), (m.rot_dim, d.rot)))
+            L.latent_norm = _pad(self.src.vector(p + "dkv.norm", m.kv_rank, fake_ones=True), d.rank)
         if d.gate:
-            parts.append(self._rows(p + "mix.g", m.heads, q, (m.vdim, d.vdim)))
-        L.qkv = make_linear(torch.cat(parts), self.kind)
+            parts.append(self._rows(p + "g", m.heads, q, (1, 1) if d.head_gate else (m.vdim, d.vdim)))
+        w = torch.cat(parts)
+        L.qkv = make_linear(_pad(w, d.row, self.WP), self.kind)
+        L.sinks = self.src.vector(p + "sink", m.heads, rng=q).contiguous() if m.sinks else None
 
         def per_head(name, n, padded):
             w = self.src.matrix(p + name, (m.heads * n, m.kv_rank), rows=(q[0] * n, q[1] * n))
             return _pad(w.view(L.hq, n, m.kv_rank), L.hq, padded, d.rank).to(self.act_dtype)
-        L.up = ops.LatentWeights(per_head("mix.uk", m.dim, d.dim), per_head("mix.uv", m.vdim, d.vdim))
+        L.up = ops.LatentWeights(per_head("uk", m.dim, d.dim), per_head("uv", m.vdim, d.vdim))
         self._out_rows(L, p, m.heads, q, m.vdim)
 
     def _load_experts(self, L: Layer, p: str, f: MoeConfig) -> None:
@@ -327,6 +426,7 @@ class LayeredDecoder(Decoder):
         kind = "fp32" if self.exact or self.device.type == "cpu" else "bf16"
         L.router = make_linear(_pad(self.src.matrix(p + "mlp.router", (f.experts, self.W)), f.experts, self.WP), kind)
 
+        L.router_b = self.src.vector(p + "mlp.router.b", f.experts).contiguous() if f.router_bias else None
         L.correction = self.src.vector(p + "mlp.correction", f.experts).contiguous() if f.correction else None
         first = ("gate", "up") if f.gated else ("up",)
 
@@ -343,12 +443,60 @@ class LayeredDecoder(Decoder):
     # ------------------------------------------------------------------------------------
     # forward
     # ------------------------------------------------------------------------------------
-    def _mixer(self, L: Layer, h: torch.Tensor, b: Batch, cache: PagedKVCache) -> torch.Tensor:
-        """Token-mixing sublayer: normalised input -> output projection (summed over tensor-parallel ranks)."""
-        kind = "shared" if L.mix.values_from_keys else L.mix.kind
-        a = {"latent": self._latent, "gla": self._linear, "shared": self._shared_kv}.get(kind, self._attend)(L, h, b, cache)
+    def _mixer(self, L: Layer, h: torch.Tensor, b: Batch, cache: PagedKVCache, x: torch.Tensor) -> torch.Tensor:
+        """Token-mixing sublayer: its input `h` (the stream itself is `x`) -> output projection (summed over tensor-parallel ranks)."""
+        if L.parts:
+            a = torch.empty(h.shape[0], L.o.in_features, dtype=h.dtype, device=h.device)
+            at = 0
+            for q in L.parts:
+                n = q.width
+                self._heads(q, h, b, cache, x, a[:, at:at + n])
+                at += n
+        else:
+            a = self._heads(L, h, b, cache, x)
         with TimeLine("Output"):
+            if (L.parts or [L])[0].replicated:
+                return ops.linear(a, L.o)
             return self._row_parallel(a, L.o, None, None)
+
+    def _heads(self, L: Layer, h, b: Batch, cache: PagedKVCache, x, out=None) -> torch.Tensor:
+        """A mixer without its output projection."""
+        kind = L.mix.kind
+        if kind == "talking":
+            return self._talking(L, h, b, cache, out)
+        if kind == "time_mix":
+            return self._time_mix(L, x, b, cache, out)
+        if kind == "attention" and L.mix.values_from_keys:
+            return self._shared_kv(L, h, b, cache)
+        return {"latent": self._latent, "gla": self._linear, "ssd": self._state_space}.get(kind, self._attend)(L, h, b, cache)
+
+    def _state_space(self, L: Layer, h: torch.Tensor, b: Batch, cache: PagedKVCache) -> torch.Tensor:
+        with TimeLine("QKV.linear"):
+            x = ops.linear(h, L.qkv)
+        with TimeLine("SSD"):
+            states = [cache.state[i] for i in L.state]
+            return ops.state_space(x, L.dims, L.ssm, self.eps, states[0], states[1] if len(states) > 1 else None, b.state_slots, b.cu_q,
+                                   b.kv_lens, meta=b)
+
+    def _talking(self, L: Layer, h, b: Batch, cache: PagedKVCache, out) -> torch.Tensor:
+        kc, vc = cache.k[L.pool], cache.v[L.pool]
+        with TimeLine("QKV.linear"):
+            x = ops.linear(h, L.qkv)
+        with TimeLine("QKPO"):
+            q = ops.talking_prep(x, L.talk, self.eps, kc, vc, b.slots)
+        with TimeLine("MHA"):
+            return ops.talking_attention(q, x, L.talk, kc, vc, b.block_table, b.cu_q, b.kv_lens, L.mix.scale, L.mix.window, meta=b, out=out)
+
+    def _time_mix(self, L: Layer, x, b: Batch, cache: PagedKVCache, out) -> torch.Tensor:
+        d, W = L.dims, L.mu.shape[1]
+        with TimeLine("Shift"):
+            mix = ops.token_shift(x, L.mu, cache.state[L.state[1]], b.state_slots, b.cu_q, b.kv_lens, self.act_dtype, meta=b)
+        with TimeLine("QKV.linear"):
+            rows = torch.empty(x.shape[0], d.a_at + d.up(d.rank), dtype=self.act_dtype, device=x.device)
+            ops.linear_parts(mix[:, :4 * W], L.rkvg, 4, rows)
+            ops.linear(mix[:, 4 * W:], L.w1, act="tanh", out=rows[:, d.a_at:])
+        with TimeLine("GLA"):
+            return ops.gated_linear(rows, d, L.decay, self.eps, cache.state[L.state[0]], b.state_slots, b.cu_q, b.kv_lens, meta=b, out=out)
 
     def _latent(self, L: Layer, h: torch.Tensor, b: Batch, cache: PagedKVCache) -> torch.Tensor:
         m, pool = L.mix, cache.k[L.pool]
@@ -358,13 +506,13 @@ class LayeredDecoder(Decoder):
             ops.latent_prep(x, L.dims, b.positions, self._rope(m.rot, 0), m.rot.dims if m.rot is not None else 0, L.latent_norm,
                             self.eps, pool, b.slots)
         with TimeLine("MHA"):
-            return ops.latent_attention(x, L.dims, pool, b.block_table, b.cu_q, b.kv_lens, L.up, m.scale, m.window, meta=b)
+            return ops.latent_attention(x, L.dims, pool, b.block_table, b.cu_q, b.kv_lens, L.up, m.scale, m.window, meta=b, sinks=L.sinks)
 
     def _linear(self, L: Layer, h: torch.Tensor, b: Batch, cache: PagedKVCache) -> torch.Tensor:
         with TimeLine("QKV.linear"):
             x = ops.linear(h, L.qkv)
         with TimeLine("GLA"):
-            return ops.gated_linear(x, L.dims, L.decay, self.eps, cache.state[L.state], b.state_slots, b.cu_q, b.kv_lens, meta=b)
+            return ops.gated_linear(x, L.dims, L.decay, self.eps, cache.state[L.state[0]], b.state_slots, b.cu_q, b.kv_lens, meta=b)
 
     def _shared_kv(self, L: Layer, h: torch.Tensor, b: Batch, cache: PagedKVCache) -> torch.Tensor:
         m, kc, vc = L.mix, cache.k[L.pool], cache.v[L.pool]
@@ -372,7 +520,7 @@ class LayeredDecoder(Decoder):
             x = ops.linear(h, L.qkv, L.qkv_b)
         with TimeLine("QKPO"):
             q = ops.head_prep(x, L.prep, self.eps, b.positions, self._rope(m.rot, 0), m.rot.dims if m.rot is not None else 0, kc, vc,
-                              b.slots, cache.state[L.state] if m.conv > 1 else None, b.state_slots, b.cu_q, b.kv_lens, meta=b)
+                              b.slots, cache.state[L.state[0]] if m.conv > 1 else None, b.state_slots, b.cu_q, b.kv_lens, meta=b)
         with TimeLine("MHA"):
             a = ops.paged_attention(q, kc, vc, b.block_table, b.cu_q, b.kv_lens, m.scale, group=L.group, q_off=L.q_off, meta=b,
                                     softcap=m.softcap, window=m.window, keep_first=m.keep_first, sinks=L.sinks)
@@ -405,13 +553,16 @@ class LayeredDecoder(Decoder):
             with TimeLine("MoE"):
                 return self._experts(L, h)
         with TimeLine("LlamaMLP"):
-            return self._row_parallel(ops.linear_gated(h, L.gate_up, L.act), L.down, None, None)
+            return self._row_parallel(ops.linear_gated(h, L.gate_up, L.act, L.gate_up_b, L.limit), L.down, L.down_b, None)
 
     def _experts(self, L: Layer, h: torch.Tensor) -> torch.Tensor:
         """Mixture of experts -> fp32 rows (summed over tensor-parallel ranks)."""
         f = L.moe
-        logits = ops.linear(h, L.router, out_dtype=torch.float32)
-        idx, w = ops.route(logits, "deepseek", f.top, L.correction, f.groups, f.keep_groups, f.scale, f.renorm, f.scoring)
+        logits = ops.linear(h, L.router, L.router_b, out_dtype=torch.float32)
+        if f.scoring == "chosen":
+            idx, w = ops.route(logits, "mixtral", f.top)
+        else:
+            idx, w = ops.route(logits, "deepseek", f.top, L.correction, f.groups, f.keep_groups, f.scale, f.renorm, f.scoring)
         shared = None
         if L.shared is not None:
             # few rows: the product leaves in fp32; prompts: in the activation type, like the experts' own rows
@@ -435,6 +586,45 @@ class LayeredDecoder(Decoder):
     def _add_norm(self, x, y, post, nxt, **kw):
         return ops.residual_norm(x, y, post, nxt, self.eps, self.spec.norm, h_dtype=self.act_dtype, mult=self.cfg.residual_mult, **kw)
 
+    def _sum_norm(self, x, y, post, nxt=None, **kw):
+        """x = norm(alpha * x + y), and the same in the activation type or, with `nxt`, one more norm of it."""
+        return self._add_norm(x, y, post, nxt, raw=nxt is None, carry=self.cfg.residual_carry, post_sum=True, **kw)
+
+    def _logits(self, h):
+        with TimeLine("DistLinear.forward"):
+            cap = self.cfg.logit_softcap
+            if cap > 0:
+                return ops.linear(h, self.lm_head, act="softcap", res_scale=cap, out_dtype=torch.float32)
+            return ops.linear(h, self.lm_head, out_dtype=torch.float32)
+
+    def _forward_sum_norm(self, b: Batch, cache: PagedKVCache, hidden, step) -> torch.Tensor:
+        """The stream is the norm of the residual sum: one launch behind each sublayer makes the sum, its norm, the stream and the
+        next product's input; the last one makes the final norm too, on the rows whose logits are wanted."""
+        dump = (lambda name, x: debugger.dump(name, x[:, :self.W], self.ctx.rank, step)) if debugger.enabled() else lambda name, x: None
+        kw = dict(ids=b.ids, table=self.wte, embed_scale=self.cfg.embed_scale) if self.first_stage else {}
+        x, h = self._add_norm(None if self.first_stage else hidden, None, None, None, raw=True, **kw)
+        dump("embedding", x)
+        for n, L in enumerate(self.runs):
+            last = n + 1 == len(self.runs) and self.last_stage
+            y, post = self._mixer(L, h, b, cache, x), L.norm1
+            if L.mlp_kind != "none":
+                x, h = self._sum_norm(x, y, post)
+                dump(f"layer{L.idx}_attn_out", x)
+                y, post = self._ff(L, h), L.norm2
+            if last and not debugger.enabled():
+                break
+            x, h = self._sum_norm(x, y, post)
+            dump(f"layer{L.idx}_ffn_out", x)
+        if not self.last_stage:
+            return x
+        if b.logit_rows is not None and b.logit_rows.numel() == 0:
+            return torch.empty(0, self.v1 - self.v0, dtype=torch.float32, device=x.device)
+        if debugger.enabled():
+            _, h = self._add_norm(x, None, None, self.final, rows=b.logit_rows, keep_x=False)
+        else:
+            _, h = self._sum_norm(x, y, post, self.final, rows=b.logit_rows, keep_x=False)
+        return self._logits(h)
+
     def forward(self, b: Batch, cache: PagedKVCache, hidden: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Local logits on the last stage, the residual stream otherwise.  The norm of each sublayer's output, the
         residual sum, the vector in front of a pass of looped layers and the norm in front of the next sublayer are one
@@ -444,6 +634,8 @@ class LayeredDecoder(Decoder):
         dbg = debugger.enabled()
         step = debugger.next_step() if dbg else 0
         with TimeLine("Decoder.forward"):
+            if self.spec.sum_norm:
+                return self._forward_sum_norm(b, cache, hidden, step)
             first = self.runs[0]
             if self.first_stage:
                 x, h = self._add_norm(None, None, None, first.norm1, ids=b.ids, table=self.wte, embed_scale=self.cfg.embed_scale,
@@ -455,7 +647,7 @@ class LayeredDecoder(Decoder):
             side = ops.embedding(b.ids, self.side_embed, 1.0, self.act_dtype) if self.side_embed is not None else None
             for n, L in enumerate(self.runs):
                 nxt = self.runs[n + 1] if n + 1 < len(self.runs) else None
-                y, post = self._mixer(L, h, b, cache), L.norm1b
+                y, post = self._mixer(L, h, b, cache, x), L.norm1b
                 if L.mlp_kind != "none":
                     x, h = self._add_norm(x, y, post, L.norm2)
                     if dbg:
@@ -476,8 +668,7 @@ class LayeredDecoder(Decoder):
             if b.logit_rows is not None and b.logit_rows.numel() == 0:
                 return torch.empty(0, self.v1 - self.v0, dtype=torch.float32, device=x.device)
             _, h = self._add_norm(x, y, post, self.final, rows=b.logit_rows, keep_x=False)
-            with TimeLine("DistLinear.forward"):
-                return ops.linear(h, self.lm_head, out_dtype=torch.float32)
+            return self._logits(h)
 
     # -- sizes ------------------------------------------------------------------------------
     def plan_splits(self, B: int, max_kv: int, int8: bool) -> Optional[int]:

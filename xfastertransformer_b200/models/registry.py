@@ -34,6 +34,8 @@ class FamilySpec:
     post_norm: bool = False         # a second norm after each sublayer, before the residual sum
     sinks: bool = False             # one softmax sink per attention head
     tied_head: bool = False         # logits are products with the embedding table
+    norm_bias: bool = False         # layered: norms have a bias beside their gain
+    sum_norm: bool = False          # layered: the norm is taken of the residual sum, and its output is the stream
 
 
 FAMILIES: Dict[str, FamilySpec] = {
@@ -57,6 +59,7 @@ FAMILIES: Dict[str, FamilySpec] = {
     "kafipel": FamilySpec("kafipel", norm="layer", layered=True, post_norm=True, sinks=True),
     "vepivik": FamilySpec("vepivik", layered=True, tied_head=True),
     "botusun": FamilySpec("botusun", layered=True, tied_head=True),
+    "dagezen": FamilySpec("dagezen", norm="layer", layered=True, tied_head=True, norm_bias=True, sum_norm=True),
 }
 
 

@@ -53,13 +53,13 @@ def layernorm(x, w, b, eps):
 
 
 def residual_norm(x, y, post, nxt, eps, kind="layer", rows=None, h_dtype=torch.bfloat16, ids=None, table=None, keep_x=True,
-                  embed_scale=1.0, mult=1.0, add=None, raw=False):
-    """One step of a 32-bit residual stream in one launch: x (or table[ids] * embed_scale) += mult * norm(y) with `post` =
-    (gain, bias or None) (plain y without it) + the vector `add`, then h = norm(x) with `nxt` for the next product (`raw`: x
-    itself).  Returns (x, h); on a GPU x is updated in place unless `rows` selects rows, and buffers are as wide as x (a
+                  embed_scale=1.0, mult=1.0, add=None, raw=False, carry=1.0, post_sum=False):
+    """One step of a 32-bit residual stream in one launch: x (or table[ids] * embed_scale) = carry * x + mult * norm(y) with
+    `post` = (gain, bias or None) (plain y without it) + the vector `add`, then h = norm(x) with `nxt` for the next product
+    (`raw`: x itself).  `post_sum`: `post` normalises the sum instead of y, and its output is the stream.  Returns (x, h); on a GPU x is updated in place unless `rows` selects rows, and buffers are as wide as x (a
     multiple of 8, padding zero)."""
     impl = _nat().residual_norm if _cuda(x if x is not None else table) else R.residual_norm
-    return impl(x, y, post, nxt, eps, kind, rows, h_dtype, ids, table, keep_x, embed_scale, mult, add, raw)
+    return impl(x, y, post, nxt, eps, kind, rows, h_dtype, ids, table, keep_x, embed_scale, mult, add, raw, carry, post_sum)
 
 
 # -- GEMMs ---------------------------------------------------------------------------------
@@ -86,8 +86,12 @@ def _timed(kernel: str, x, W, fn):
     return y
 
 
-def linear(x, W, bias=None, act=None, residual=None, res_scale=1.0, out_dtype=None, times=None):
-    """act(x W^T + bias) + res_scale * residual, or with `times` [T, out] act(x W^T + bias) * times."""
+def linear(x, W, bias=None, act=None, residual=None, res_scale=1.0, out_dtype=None, times=None, out=None):
+    """act(x W^T + bias) + res_scale * residual, or with `times` [T, out] act(x W^T + bias) * times.  `out`: rows to write
+    into.  act "softcap": res_scale * tanh(. / res_scale)."""
+    if out is not None:
+        assert residual is None and times is None
+        return (_nat() if _cuda(x) else R).linear_into(x, W, bias, act, out)
     if times is not None:
         return (_nat() if _cuda(x) else R).linear_times(x, W, bias, act, times)
     if _verbose():
@@ -115,13 +119,19 @@ def linear_rms(x, W, eps, bias=None, act=None, gated=False, out_dtype=None):
     return _linear_rms(x, W, eps, bias, act, gated, out_dtype)
 
 
-def linear_gated(x, W, act="silu", bias=None):
+def linear_gated(x, W, act="silu", bias=None, limit=0.0):
+    """act(g) * u with (g | u) = x W^T + bias; act "clamped": g = min(g, limit), u = u clamped to +-limit, and the result is
+    g sigmoid(1.702 g) (u + 1)."""
+    impl = _nat().linear_gated if _cuda(x) else R.linear_gated
     if _verbose():
-        impl = _nat().linear_gated if _cuda(x) else R.linear_gated
-        return _timed(f"gemm_gated_{act}", x, W, lambda: impl(x, W, act, bias))
-    if _cuda(x):
-        return _nat().linear_gated(x, W, act, bias)
-    return R.linear_gated(x, W, act, bias)
+        return _timed(f"gemm_gated_{act}", x, W, lambda: impl(x, W, act, bias, limit))
+    return impl(x, W, act, bias, limit)
+
+
+def linear_parts(x, W, n, out):
+    """`n` products side by side: part i of x's columns with rows i of W's n equal parts, into part i of `out`'s columns."""
+    impl = _native_linear().linear_parts if _cuda(x) else R.linear_parts
+    return impl(x, W, n, out)
 
 
 def gated_act(gu, act="silu"):
@@ -238,7 +248,8 @@ def mla_prep(q, kv, Hl, nope, rope, kvl, positions, table, kv_norm_w, eps, cache
 @dataclass(frozen=True)
 class LatentDims:
     """Sizes of a latent-attention layer as its kernels see them (heads of this rank; sizes possibly padded with zeros).
-    A packed row is [q: heads x (dim + rot) | latent: rank + rot (unless the layer reads another's) | gate: heads x vdim]."""
+    A packed row is [q: heads x (dim + rot) | latent: rank + rot (unless the layer reads another's) | gate: heads x vdim], or
+    with `head_gate` one gate value per head, in a row of a multiple of `align` values."""
     heads: int
     dim: int                    # unrotated query/key dimensions per head
     rot: int                    # rotated dimensions per head
@@ -247,6 +258,8 @@ class LatentDims:
     own_kv: bool
     gate: bool
     rank_real: int              # values of the latent that are not padding (the norm's count)
+    head_gate: bool = False
+    align: int = 1
 
     @property
     def q_width(self) -> int:
@@ -258,7 +271,8 @@ class LatentDims:
 
     @property
     def row(self) -> int:
-        return self.gate_at + (self.heads * self.vdim if self.gate else 0)
+        n = self.gate_at + (0 if not self.gate else self.heads if self.head_gate else self.heads * self.vdim)
+        return (n + self.align - 1) // self.align * self.align
 
 
 def latent_prep(x, dims: LatentDims, positions, table, rot_dims, norm_w, eps, cache, slots):
@@ -279,16 +293,19 @@ def latent_prep(x, dims: LatentDims, positions, table, rot_dims, norm_w, eps, ca
         latent_cache_write(torch.cat([n.to(x.dtype), kr.reshape(T, d.rot)], -1), cache, slots)
 
 
-def latent_attention(x, dims: LatentDims, cache, block_table, cu_q, kv_lens, weights, scale, window=0, meta=None):
+def latent_attention(x, dims: LatentDims, cache, block_table, cu_q, kv_lens, weights, scale, window=0, meta=None, sinks=None):
     """Attention of the packed rows x (after `latent_prep`) over a latent cache -> [T, heads * vdim], multiplied with the
-    sigmoid of the rows' gate.  `weights`: `LatentWeights`.  `window` as in `paged_attention`."""
+    sigmoid of the rows' gate.  `weights`: `LatentWeights`.  `window` and `sinks` as in `paged_attention`."""
     if _cuda(x):
-        return _nat_latent().latent_attention(x, dims, cache, block_table, cu_q, kv_lens, weights, scale, window, meta)
+        return _nat_latent().latent_attention(x, dims, cache, block_table, cu_q, kv_lens, weights, scale, window, meta, sinks)
     d, T = dims, x.shape[0]
     q = x[:, :d.q_width].view(T, d.heads, d.dim + d.rot)
     a = R.mla_attention(q[..., :d.dim], q[..., d.dim:], cache, block_table, cu_q, kv_lens, weights.uk, weights.uv, scale,
-                        max(cu_q[i + 1] - cu_q[i] for i in range(len(kv_lens))) == 1, window).reshape(T, -1)
-    if d.gate:
+                        max(cu_q[i + 1] - cu_q[i] for i in range(len(kv_lens))) == 1, window, sinks).reshape(T, -1)
+    if d.gate and d.head_gate:
+        g = torch.sigmoid(x[:, d.gate_at:d.gate_at + d.heads].float())[:, :, None]
+        a = (a.view(T, d.heads, d.vdim).float() * g).to(a.dtype).reshape(T, -1)
+    elif d.gate:
         a = (a.float() * torch.sigmoid(x[:, d.gate_at:d.gate_at + d.heads * d.vdim].float())).to(a.dtype)
     return a
 
@@ -363,19 +380,144 @@ class LinearDims:
 @dataclass
 class LinearWeights:
     """Decay and output norm: the decay's second product a2 [heads * dim, rank (aligned)] and its bias, `tau`, the gain of
-    the norm over a head's vdim outputs."""
+    the norm over a head's vdim outputs ([vdim], or [heads * vdim]).  `scale` of the queries (None: 1 / sqrt(dim)).  `bonus`
+    [heads, dim]: the current token is read with this factor on its key instead of through the state, and decays are
+    exp(-exp(z)).  `mult`: a factor of the result."""
     a2: torch.Tensor
     bias: torch.Tensor
     tau: float
     norm: torch.Tensor
+    scale: Optional[float] = None
+    bonus: Optional[torch.Tensor] = None
+    mult: float = 1.0
 
 
-def gated_linear(x, dims: LinearDims, w: LinearWeights, eps, state, state_slots, cu_q, kv_lens, meta=None):
-    """Gated linear attention of packed rows x -> [T, heads * vdim (aligned)].  Per head, with decay = sigmoid(W_a2 a1 + bias)^(1 / tau)
-    per key channel: S <- diag(decay) S + k v^T and o = S^T (q / sqrt(dim)); the result is norm(o) * silu(g).  `state`
-    [slots, heads, dim, vdim] fp32 is carried on; a sequence's first token starts from zero."""
+def gated_linear(x, dims: LinearDims, w: LinearWeights, eps, state, state_slots, cu_q, kv_lens, meta=None, out=None):
+    """Gated linear attention of packed rows x -> [T, heads * vdim (aligned)] (into `out` when given).  Per head, with z = W_a2 a1
+    + bias and decay = sigmoid(z)^(1 / tau) per key channel: S <- diag(decay) S + k v^T and o = S^T (q * scale); the result is
+    norm(o) * silu(g).  With a bonus u: decay = exp(-exp(z)), and o = (S + diag(u) k v^T)^T q is read before S moves on.
+    `state` [slots, heads, dim, vdim] fp32 is carried on; a sequence's first token starts from zero."""
     impl = _native_linear().gated_linear if _cuda(x) else R.gated_linear
-    return impl(x, dims, w, eps, state, state_slots, cu_q, kv_lens, meta)
+    return impl(x, dims, w, eps, state, state_slots, cu_q, kv_lens, meta, out)
+
+
+def token_shift(x, mu, state, state_slots, cu_q, kv_lens, dtype, meta=None):
+    """Mixes of every row with the row of the token before it: column part i of the result [T, n * width] is
+    x + (previous x - x) * mu[i] (mu [n, width] fp32), the arithmetic in fp32.  `state` [slots, width] fp32 holds the last row of
+    each sequence and is moved on; in front of a sequence's first token are zeros."""
+    impl = _native_linear().token_shift if _cuda(x) else R.token_shift
+    return impl(x, mu, state, state_slots, cu_q, kv_lens, dtype, meta)
+
+
+# -- state-space recurrence ---------------------------------------------------------------------
+@dataclass(frozen=True)
+class StateDims:
+    """A packed row of a state-space layer: [z: heads x vdim | x: heads x vdim, B, C: groups x state each | dt: heads]; the three
+    parts start at multiples of `align` values, and x, B, C are one run of channels."""
+    heads: int
+    state: int
+    vdim: int
+    groups: int
+    norm_groups: int
+    taps: int
+    align: int = 1
+
+    def up(self, n: int) -> int:
+        return (n + self.align - 1) // self.align * self.align
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def channels(self) -> int:
+        return self.inner + 2 * self.groups * self.state
+
+    @property
+    def x_at(self) -> int:
+        return self.up(self.inner)
+
+    @property
+    def dt_at(self) -> int:
+        return self.x_at + self.up(self.channels)
+
+    @property
+    def row(self) -> int:
+        return self.dt_at + self.up(self.heads)
+
+
+@dataclass
+class StateWeights:
+    """fp32: the convolution [taps, channels] and its bias, per head dt_bias, the decay's rate exp(A_log) and the skip's factor D,
+    the gain of the output norm [heads * vdim]."""
+    conv: torch.Tensor
+    conv_bias: torch.Tensor
+    dt_bias: torch.Tensor
+    rate: torch.Tensor
+    skip: torch.Tensor
+    norm: torch.Tensor
+
+
+def state_space(x, dims: StateDims, w: StateWeights, eps, state, conv_state, state_slots, cu_q, kv_lens, meta=None):
+    """The mixer of a state-space layer between its two projections, packed rows x -> [T, heads * vdim (aligned)]: x, B and C
+    through a causal convolution and silu, dt through softplus, then per head S <- exp(-rate dt) S + dt B x^T and
+    y = S^T C + D x; y * silu(z) is normalised in `norm_groups` parts.  `state` [slots, heads, state, vdim] fp32 and `conv_state`
+    [slots, taps - 1, channels] (None for one tap) are carried on; a sequence's first token starts from zero."""
+    impl = _native_linear().state_space if _cuda(x) else R.state_space
+    return impl(x, dims, w, eps, state, conv_state, state_slots, cu_q, kv_lens, meta)
+
+
+# -- attention with mixed heads -----------------------------------------------------------------
+@dataclass
+class TalkingHeads:
+    """Attention whose heads' weights are mixed.  A packed row is [q: hq x dim | k: hkv x dim | gate: hq x padded], each part starting
+    at a multiple of `align` values; heads leave `padded` wide.  Gains of the norms over the whole projections [hq * dim] and
+    [hkv * dim], the distance bias r1, r2 [hq], the mixing matrix talk [hq, hq], all fp32.  `mult`: a factor of the result."""
+    hq: int
+    hkv: int
+    dim: int
+    padded: int
+    q_norm: torch.Tensor
+    k_norm: torch.Tensor
+    r1: torch.Tensor
+    r2: torch.Tensor
+    talk: torch.Tensor
+    mult: float = 1.0
+    align: int = 1
+
+    def up(self, n: int) -> int:
+        return (n + self.align - 1) // self.align * self.align
+
+    @property
+    def k_at(self) -> int:
+        return self.up(self.hq * self.dim)
+
+    @property
+    def gate_at(self) -> int:
+        return self.k_at + self.up(self.hkv * self.dim)
+
+    @property
+    def row(self) -> int:
+        return self.gate_at + self.up(self.hq * self.padded)
+
+
+def talking_prep(x, d: TalkingHeads, eps, kc, vc, slots):
+    """RMS norms over all of a row's q and over all of its k; appends k to `kc` and k as it was before its norm to `vc`, and
+    returns q [T, hq, padded]."""
+    return (_native_talking() if _cuda(x) else R).talking_prep(x, d, eps, kc, vc, slots)
+
+
+def talking_attention(q, x, d: TalkingHeads, kc, vc, block_table, cu_q, kv_lens, scale, window=0, meta=None, out=None):
+    """Attention with scores q . k * scale - r1 ln(1 + r2 (i - j)) over the keys that `window` leaves, a softmax per head, the heads'
+    weights mixed by `talk` (head h applies sum_g talk[h, g] weight_g to the values of its own key/value head), and the gate of
+    the packed rows x: -> [T, hq * padded] (into `out` when given)."""
+    impl = (_native_talking() if _cuda(q) else R).talking_attention
+    return impl(q, x, d, kc, vc, block_table, cu_q, kv_lens, scale, window, meta, out)
+
+
+def _native_talking():
+    from . import native_talking
+    return native_talking
 
 
 def _native_linear():

@@ -73,19 +73,24 @@ def _norm(xf: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor], eps: flo
 
 def residual_norm(x, y, post, nxt, eps: float, kind: str = "layer", rows: Optional[torch.Tensor] = None,
                   h_dtype: torch.dtype = torch.float32, ids=None, table=None, keep_x: bool = True, embed_scale: float = 1.0,
-                  mult: float = 1.0, add: Optional[torch.Tensor] = None, raw: bool = False):
-    """One step of a 32-bit residual stream: x (or table[ids] * embed_scale) plus mult * y — normalised with `post` = (gain,
+                  mult: float = 1.0, add: Optional[torch.Tensor] = None, raw: bool = False, carry: float = 1.0,
+                  post_sum: bool = False):
+    """One step of a 32-bit residual stream: carry * x (or table[ids] * embed_scale) plus mult * y — normalised with `post` = (gain,
     bias) first, when given — plus the vector `add`, and the input of the next sublayer, h = norm(x) with `nxt` = (gain,
-    bias), or x itself with `raw`.  `rows` selects rows.  Returns (x or None, h or None)."""
+    bias), or x itself with `raw`.  `post_sum`: `post` normalises the sum.  `rows` selects rows.  Returns (x or None, h or None)."""
     xf = table[ids.long()].float() * embed_scale if ids is not None else x.float()
     yf = None if y is None else y.float()
     if rows is not None:
         xf = xf[rows.long()]
         yf = None if yf is None else yf[rows.long()]
+    if carry != 1.0:
+        xf = carry * xf
     if yf is not None:
-        xf = xf + mult * (_norm(yf, post[0], post[1], eps, kind) if post is not None else yf)
+        xf = xf + mult * (_norm(yf, post[0], post[1], eps, kind) if post is not None and not post_sum else yf)
     if add is not None:
         xf = xf + add
+    if post_sum:
+        xf = _norm(xf, post[0], post[1], eps, kind)
     h = xf.to(h_dtype) if raw else None if nxt is None else _norm(xf, nxt[0], nxt[1], eps, kind).to(h_dtype)
     return (xf if keep_x else None), h
 
@@ -199,6 +204,8 @@ def _act(y: torch.Tensor, act: Optional[str]) -> torch.Tensor:
         return F.relu(y).square()
     if act == "gelu_erf":
         return F.gelu(y)
+    if act == "tanh":
+        return torch.tanh(y)
     raise ValueError(act)
 
 
@@ -217,6 +224,8 @@ def linear(x: torch.Tensor, W, bias: Optional[torch.Tensor] = None, act: Optiona
     y = xf @ dequant_weight(W).t()
     if bias is not None:
         y = y + bias.float()
+    if act == "softcap":
+        return (res_scale * torch.tanh(y / res_scale)).to(out_dtype)
     y = _act(y, act)
     if residual is not None:
         y = y + res_scale * residual.float()
@@ -235,7 +244,20 @@ def linear_times(x: torch.Tensor, W, bias, act, times: torch.Tensor) -> torch.Te
     return (linear(x, W, bias, act, out_dtype=torch.float32) * times.float()).to(x.dtype)
 
 
-def linear_gated(x: torch.Tensor, W, act: str = "silu", bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+def linear_into(x, W, bias, act, out):
+    out[:, :W.out_features] = linear(x, W, bias, act)
+    return out
+
+
+def linear_parts(x, W, n, out):
+    k, m = x.shape[1] // n, W.out_features // n
+    w = dequant_weight(W)
+    for i in range(n):
+        out[:, i * m:(i + 1) * m] = (x[:, i * k:(i + 1) * k].float() @ w[i * m:(i + 1) * m].t()).to(out.dtype)
+    return out
+
+
+def linear_gated(x: torch.Tensor, W, act: str = "silu", bias: Optional[torch.Tensor] = None, limit: float = 0.0) -> torch.Tensor:
     """act(x Wg^T) * (x Wu^T) with W = cat(gate, up) on the out dim; the intermediate is
     kept in fp32 (the fused kernel applies the activation on the TMEM accumulators)."""
     xf = x.float()
@@ -246,6 +268,9 @@ def linear_gated(x: torch.Tensor, W, act: str = "silu", bias: Optional[torch.Ten
     if bias is not None:
         y = y + bias.float()
     i = y.shape[-1] // 2
+    if act == "clamped":
+        g, u = y[..., :i].clamp(max=limit), y[..., i:].clamp(-limit, limit)
+        return (g * torch.sigmoid(1.702 * g) * (u + 1)).to(x.dtype)
     return (_act(y[..., :i], act) * y[..., i:]).to(x.dtype)
 
 
@@ -472,13 +497,13 @@ def paged_attention(q: torch.Tensor, kc: torch.Tensor, vc: torch.Tensor, block_t
 # ----------------------------------------------------------------------------------------
 def mla_attention(q_nope: torch.Tensor, q_rope: torch.Tensor, latent_cache: torch.Tensor,
                   block_table: torch.Tensor, cu_q, kv_lens, w_uk: torch.Tensor, w_uv: torch.Tensor,
-                  scale: float, absorbed: bool = True, window: int = 0) -> torch.Tensor:
+                  scale: float, absorbed: bool = True, window: int = 0, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """DeepSeek MLA over the latent cache (c_kv[kv_lora] ‖ k_rope[rope] per token).
 
     q_nope [T,H,nope], q_rope [T,H,rope]; w_uk [H,nope,kv_lora], w_uv [H,v,kv_lora].
     absorbed:   S = (q_nope·W_uk)·c_kvᵀ + q_rope·k_ropeᵀ ; O = (softmax(S)·c_kv)·W_uvᵀ
     otherwise:  K_nope = c_kv·W_ukᵀ, V = c_kv·W_uvᵀ are materialised (prefill form).
-    `window` > 0: position i sees the keys j <= i with i - j < window.
+    `window` > 0: position i sees the keys j <= i with i - j < window.  `sinks` [H] as in `paged_attention`.
     Reference: crossAttnByHead_DS (attention_kernels.h:1132-1281), selfAttention_MLA (:569-766).
     """
     T, H, nope = q_nope.shape
@@ -507,7 +532,9 @@ def mla_attention(q_nope: torch.Tensor, q_rope: torch.Tensor, latent_cache: torc
         if window > 0:
             mask = mask | (qpos[:, None] - kpos[None, :] >= window)
         s = s.masked_fill(mask[None], float("-inf"))
-        p = torch.softmax(s, -1)
+        if sinks is not None:
+            s = torch.cat([s, sinks.float()[:, None, None].expand(H, ql, 1)], dim=-1)
+        p = torch.softmax(s, -1)[..., :n]
         if absorbed:
             o = torch.matmul(torch.matmul(p, ckv), w_uv.float().transpose(1, 2))   # [H,ql,v]
         else:
@@ -618,25 +645,115 @@ def head_prep(x, prep, eps, positions, table, rot_dims, kc, vc, slots, state, st
     return pad(q).to(x.dtype)
 
 
-def gated_linear(x, d, w, eps, state, state_slots, cu_q, kv_lens, meta=None):
+def gated_linear(x, d, w, eps, state, state_slots, cu_q, kv_lens, meta=None, out=None):
     """See `ops.gated_linear`."""
     T, H = x.shape[0], d.heads
     f = x.float()
-    q = f[:, :H * d.dim].view(T, H, d.dim) * d.dim ** -0.5
+    q = f[:, :H * d.dim].view(T, H, d.dim) * (d.dim ** -0.5 if w.scale is None else w.scale)
     k = f[:, d.k_at:d.k_at + H * d.dim].view(T, H, d.dim)
     v = f[:, d.v_at:d.v_at + H * d.vdim].view(T, H, d.vdim)
     g = f[:, d.g_at:d.g_at + H * d.vdim]
     z = f[:, d.a_at:d.a_at + d.rank] @ w.a2[:, :d.rank].float().t() + w.bias
-    decay = torch.exp(F.logsigmoid(z) / w.tau).view(T, H, d.dim)
+    decay = (torch.exp(F.logsigmoid(z) / w.tau) if w.bonus is None else torch.exp(-torch.exp(z))).view(T, H, d.dim)
     o = torch.empty(T, H, d.vdim)
     for b in range(len(kv_lens)):
         a, e, slot = int(cu_q[b]), int(cu_q[b + 1]), int(state_slots[b])
         S = state[slot].clone() if int(kv_lens[b]) > e - a else torch.zeros_like(state[slot])
         for t in range(a, e):
-            S = decay[t, :, :, None] * S + k[t, :, :, None] * v[t, :, None, :]
-            o[t] = torch.einsum("hd,hdv->hv", q[t], S)
+            kv = k[t, :, :, None] * v[t, :, None, :]
+            if w.bonus is not None:
+                o[t] = torch.einsum("hd,hdv->hv", q[t], S + w.bonus[:, :, None] * kv)
+            S = decay[t, :, :, None] * S + kv
+            if w.bonus is None:
+                o[t] = torch.einsum("hd,hdv->hv", q[t], S)
         state[slot] = S
-    return (rmsnorm(o, w.norm, eps).reshape(T, -1) * F.silu(g)).to(x.dtype)
+    y = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
+    y = ((y.reshape(T, -1) * w.norm if w.norm.numel() == H * d.vdim else (y * w.norm).reshape(T, -1)) * F.silu(g) * w.mult).to(x.dtype)
+    if out is None:
+        return y
+    out[:, :y.shape[1]] = y
+    return out
+
+
+def token_shift(x, mu, state, state_slots, cu_q, kv_lens, dtype, meta=None):
+    """See `ops.token_shift`."""
+    before = torch.empty_like(x)
+    for b in range(len(kv_lens)):
+        a, e, slot = int(cu_q[b]), int(cu_q[b + 1]), int(state_slots[b])
+        if e == a:
+            continue
+        before[a] = state[slot] if int(kv_lens[b]) > e - a else 0.0
+        before[a + 1:e] = x[a:e - 1]
+        state[slot] = x[e - 1]
+    return (x[:, None] + (before - x)[:, None] * mu[None]).reshape(x.shape[0], -1).to(dtype)
+
+
+def state_space(x, d, w, eps, state, conv_state, state_slots, cu_q, kv_lens, meta=None):
+    """See `ops.state_space`."""
+    T, H, N, P, G = x.shape[0], d.heads, d.state, d.vdim, d.groups
+    f, n_in = x.float(), d.inner
+    u, z = f[:, d.x_at:d.x_at + d.channels], f[:, :n_in]
+    dt = F.softplus(f[:, d.dt_at:d.dt_at + H] + w.dt_bias, threshold=1e9)
+    keep = torch.exp(-w.rate * dt)
+    group = torch.arange(H) // (H // G)
+    y = torch.empty(T, H, P)
+    for b in range(len(kv_lens)):
+        a, e, slot = int(cu_q[b]), int(cu_q[b + 1]), int(state_slots[b])
+        past = int(kv_lens[b]) - (e - a)
+        before = u.new_zeros(d.taps - 1, d.channels)
+        n = min(past, d.taps - 1)
+        if n > 0:
+            before[d.taps - 1 - n:] = conv_state[slot, d.taps - 1 - n:].float()
+        seq = torch.cat([before, u[a:e]])
+        c = F.silu(sum(w.conv[j] * seq[j:j + e - a] for j in range(d.taps)) + w.conv_bias).to(x.dtype).float()
+        if d.taps > 1:
+            conv_state[slot] = seq[-(d.taps - 1):].to(conv_state.dtype)
+        xs, B, C = c[:, :n_in].view(-1, H, P), c[:, n_in:n_in + G * N].view(-1, G, N), c[:, n_in + G * N:].view(-1, G, N)
+        S = state[slot].clone() if past > 0 else torch.zeros_like(state[slot])
+        for i in range(e - a):
+            t = a + i
+            S = keep[t, :, None, None] * S + (dt[t, :, None] * B[i, group])[:, :, None] * xs[i][:, None, :]
+            y[t] = torch.einsum("hnp,hn->hp", S, C[i, group]) + w.skip[:, None] * xs[i]
+        state[slot] = S
+    y = (y.reshape(T, -1) * F.silu(z)).view(T, d.norm_groups, -1)
+    y = (y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps)).reshape(T, -1) * w.norm
+    return F.pad(y, (0, d.up(n_in) - n_in)).to(x.dtype)
+
+
+# ----------------------------------------------------------------------------------------
+# attention with mixed heads
+# ----------------------------------------------------------------------------------------
+def talking_prep(x, d, eps, kc, vc, slots):
+    """See `ops.talking_prep`."""
+    T = x.shape[0]
+    q, k = x[:, :d.hq * d.dim].float(), x[:, d.k_at:d.k_at + d.hkv * d.dim].float()
+    pad = lambda t, h: F.pad(t.reshape(T, h, d.dim), (0, d.padded - d.dim))
+    kv_cache_write(pad(rmsnorm(k, d.k_norm, eps), d.hkv).to(kc.dtype), pad(k, d.hkv).to(vc.dtype), kc, vc, slots)
+    return pad(rmsnorm(q, d.q_norm, eps), d.hq).to(x.dtype)
+
+
+def talking_attention(q, x, d, kc, vc, block_table, cu_q, kv_lens, scale, window=0, meta=None, out=None):
+    """See `ops.talking_attention`."""
+    T, H, D = q.shape
+    own = torch.arange(H) // (H // kc.shape[1])
+    y = torch.empty(T, H, D)
+    for b in range(len(kv_lens)):
+        a, e, n = int(cu_q[b]), int(cu_q[b + 1]), int(kv_lens[b])
+        if e == a:
+            continue
+        K, V = (_gather_kv(c, None, block_table[b], n)[own] for c in (kc, vc))
+        far = (torch.arange(n - (e - a), n)[:, None] - torch.arange(n)[None, :]).float()
+        s = torch.matmul(q[a:e].float().permute(1, 0, 2), K.transpose(1, 2)) * scale
+        s = s - d.r1[:, None, None] * torch.log1p(d.r2[:, None, None] * far.clamp(min=0)[None])
+        hidden = far < 0 if window <= 0 else (far < 0) | (far >= window)
+        w = torch.softmax(s.masked_fill(hidden[None], float("-inf")), -1)
+        y[a:e] = torch.matmul(torch.einsum("hg,gij->hij", d.talk, w), V).permute(1, 0, 2)
+    g = torch.sigmoid(x[:, d.gate_at:d.gate_at + H * D].float())
+    y = (y.reshape(T, -1) * g * d.mult).to(x.dtype)
+    if out is None:
+        return y
+    out[:, :y.shape[1]] = y
+    return out
 
 
 # ----------------------------------------------------------------------------------------

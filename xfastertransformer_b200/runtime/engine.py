@@ -76,7 +76,7 @@ class Model:
             raise ValueError("XFT_ATTENTION_DP=1 does not run layered designs")
         if layered and kv_cache_dtype == "int8" and any(l.mixer.kind == "latent" for l in self.cfg.layers):
             raise ValueError("latent attention keeps its cache in the activation type: kv_cache_dtype int8 is not for it")
-        if layered and kv_cache_dtype == "int8" and any(l.mixer.values_from_keys for l in self.cfg.layers):
+        if layered and kv_cache_dtype == "int8" and any(m.values_from_keys for l in self.cfg.layers for m in (l.mixer, *l.mixer.parts)):
             raise ValueError("layers whose values are their keys keep them in the activation type: kv_cache_dtype int8 is not for them")
         if self.cfg.model_type == "deepseek_moe" and d_prefill not in ("bf16", "fp8_e4m3"):
             raise ValueError("deepseek_moe supports bf16 and fp8_e4m3 only")      # model_factory.h:105-114
