@@ -1,4 +1,4 @@
-// Definitions shared by the GEMM kernels of this library (gemm_sm100.cu, gemm_decode_sm100.cu): the peer-memory
+// Definitions shared by the GEMM kernels of this library (gemm_sm100.cu, gemm_decode_sm100.cu, gemm_prefill_sm100.cu): the peer-memory
 // description of the fused all-reduce, the 8-byte transport word, activation functions, the tensor-map helper.
 #pragma once
 #include "ptx.cuh"
@@ -48,8 +48,24 @@ __device__ __forceinline__ float with_residual(float x, float r, float scale, in
   return act & kActTimes ? x * r : x + scale * r;
 }
 
-__device__ __forceinline__ float apply_act(float x, int act) {
+// tanh from one exponential: accurate to a few units of 2^-24 of one, also where the compiler's tanh is the approximate one
+__device__ __forceinline__ float tanh_exp(float x) { return 1.f - __fdividef(2.f, 1.f + __expf(2.f * fminf(x, 40.f))); }
+
+// Codes of activations; `param`: the cap of kActSoftcap.
+constexpr int kActGeluErf = 5, kActClamped = 6, kActTanh = 7, kActSoftcap = 8;
+__device__ __forceinline__ float gelu_erf(float x) { return 0.5f * x * (1.f + erff(x * 0.7071067811865476f)); }
+
+// kActClamped, of a gate and an up value: the gate bounded above and the other on both sides by `limit`
+__device__ __forceinline__ float clamped_glu(float g, float u, float limit) {
+  g = fminf(g, limit);
+  return __fdividef(g, 1.f + __expf(-1.702f * g)) * (fminf(fmaxf(u, -limit), limit) + 1.f);
+}
+
+__device__ __forceinline__ float apply_act(float x, int act, float param = 1.f) {
   switch (act & (kActTimes - 1)) {
+    case kActGeluErf: return gelu_erf(x);
+    case kActTanh: return tanh_exp(x);
+    case kActSoftcap: return param * tanh_exp(__fdividef(x, param));
     case 1: return fmaxf(x, 0.f);
     case 4: { const float r = fmaxf(x, 0.f); return r * r; }
     case 2: return x / (1.f + __expf(-x));
@@ -60,6 +76,10 @@ __device__ __forceinline__ float apply_act(float x, int act) {
     }
     default: return x;
   }
+}
+// act(g) * u, or kActClamped of the two
+__device__ __forceinline__ float apply_gated(float g, float u, int act, float param) {
+  return act == kActClamped ? clamped_glu(g, u, param) : apply_act(g, act) * u;
 }
 
 // K-major matrix [rows, cols] with row stride `ld` elements; box = 128 bytes x box_rows, 128B swizzle (gemm_sm100.cu).

@@ -173,8 +173,9 @@ __global__ void __launch_bounds__(192, 2) gemm_sk_kernel(const __grid_constant__
   auto store_plain = [&](int n, int t, float g, float u, float ssq) {
     const float rs = p.row_scale ? p.row_scale[n] : 1.f;
     const float ts = rms ? rsqrtf(ssq / (float)p.K + p.rms_eps) : 1.f;
-    float x = apply_act(g * (rs * ts) + (p.bias ? p.bias[n] : 0.f), p.act);
-    if constexpr (DUAL) x *= (u * (rs * ts) + (p.bias ? p.bias[p.dual_off + n] : 0.f));
+    float x = g * (rs * ts) + (p.bias ? p.bias[n] : 0.f);
+    if constexpr (DUAL) x = apply_gated(x, u * (rs * ts) + (p.bias ? p.bias[p.dual_off + n] : 0.f), p.act, p.res_scale);
+    else x = apply_act(x, p.act, p.res_scale);
     if (p.residual) x = with_residual(x, __bfloat162float(p.residual[(size_t)t * p.ldr + n]), p.res_scale, p.act);
     if (p.out_fp32) reinterpret_cast<float*>(p.out)[(size_t)t * p.ldo + n] = x;
     else reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)t * p.ldo + n] = __float2bfloat16(x);
@@ -304,7 +305,7 @@ auto ar_reduce = [&]() {
       for (int k = 0; k < 4; ++k) {
         const int nn = n + (k >> 1), tt = t + (k & 1);
         float x = f[k] + (p.bias ? p.bias[nn] : 0.f);
-        x = apply_act(x, p.act);
+        x = apply_act(x, p.act, p.res_scale);
         if (p.residual && tt < p.T) x = with_residual(x, __bfloat162float(p.residual[(size_t)tt * p.ldr + nn]), p.res_scale, p.act);
         f[k] = x;
       }

@@ -23,7 +23,7 @@
 // then one st.release.sys of the flag; the consumer polls with ld.acquire.sys.  Every wait is bounded and reports
 // through the status word.  With world == 1 the same kernel is a plain persistent GEMM with a double-buffered
 // accumulator.
-#include "ptx.cuh"
+#include "gemm_common.cuh"
 
 #include <cstdlib>
 
@@ -73,19 +73,6 @@ __device__ __forceinline__ float prefill_residual(float x, float r, float scale,
   return act & kPrefillTimes ? x * r : x + scale * r;
 }
 
-__device__ __forceinline__ float prefill_act(float x, int act) {
-  switch (act & (kPrefillTimes - 1)) {
-    case 1: return fmaxf(x, 0.f);
-    case 4: { const float r = fmaxf(x, 0.f); return r * r; }
-    case 2: return x / (1.f + __expf(-x));
-    case 3: {
-      const float c = 0.7978845608028654f;
-      const float u = c * (x + 0.044715f * x * x * x);
-      return 0.5f * x * (1.f + tanhf(u));
-    }
-    default: return x;
-  }
-}
 
 __device__ __forceinline__ unsigned ld_acquire_sys(const unsigned* p) {
   unsigned v;
@@ -355,8 +342,9 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_kernel(const __grid_const
         for (int j = 0; j < 16; ++j) {
           const int t = t0 + c + j;
           if (t < p.T) {
-            float y = prefill_act(x[j] + bias, p.act);
-            if constexpr (DUAL) y *= __uint_as_float(vu[j]) + bias_u;
+            float y = x[j] + bias;
+            if constexpr (DUAL) y = apply_gated(y, __uint_as_float(vu[j]) + bias_u, p.act, p.res_scale);
+            else y = apply_act(y, p.act, p.res_scale);
             if (p.residual) y = prefill_residual(y, __bfloat162float(p.residual[(size_t)t * p.ldr + n]), p.res_scale, p.act);
             const __nv_bfloat16 yb = __float2bfloat16(y);
             if (wide) {
@@ -623,19 +611,28 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_tm_kernel(const __grid_co
         switch (p.act & (kPrefillTimes - 1)) {
           case 1:
 #pragma unroll
-            for (int j = 0; j < 32; ++j) x[j] = prefill_act(x[j], 1);
+            for (int j = 0; j < 32; ++j) x[j] = apply_act(x[j], 1);
             break;
           case 2:
 #pragma unroll
-            for (int j = 0; j < 32; ++j) x[j] = prefill_act(x[j], 2);
+            for (int j = 0; j < 32; ++j) x[j] = apply_act(x[j], 2);
             break;
           case 3:
 #pragma unroll
-            for (int j = 0; j < 32; ++j) x[j] = prefill_act(x[j], 3);
+            for (int j = 0; j < 32; ++j) x[j] = apply_act(x[j], 3);
             break;
           case 4:
 #pragma unroll
-            for (int j = 0; j < 32; ++j) x[j] = prefill_act(x[j], 4);
+            for (int j = 0; j < 32; ++j) x[j] = apply_act(x[j], 4);
+            break;
+          case kActGeluErf:
+#pragma unroll
+            for (int j = 0; j < 32; ++j) x[j] = gelu_erf(x[j]);
+            break;
+          case kActTanh:
+          case kActSoftcap:
+#pragma unroll
+            for (int j = 0; j < 32; ++j) x[j] = apply_act(x[j], p.act, p.res_scale);
             break;
           default: break;
         }
@@ -644,7 +641,7 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_tm_kernel(const __grid_co
           for (int j = 0; j < 32; ++j) {
             float u = __uint_as_float(vu[j]);
             if (p.bias && (full || n0 + j < p.N)) u += __ldg(p.bias + p.dual_off + n0 + j);
-            x[j] *= u;
+            x[j] = p.act == kActClamped ? clamped_glu(x[j], u, p.res_scale) : x[j] * u;
           }
         }
         if (p.out_fp32) {
@@ -887,11 +884,11 @@ extern "C" int xft_gemm_bf16_prefill_tm(const void* X, int ldx, const void* W, i
 
 // The same with fp32 rows: Y[T, N] = act(X W^T + bias).
 extern "C" int xft_gemm_bf16_prefill_tm_f32(const void* X, int ldx, const void* W, int w_rows, int ldw, float* Y, int ldo, int T,
-                                            int N, int K, const float* bias, int act, int* status, cudaStream_t st) {
+                                            int N, int K, const float* bias, int act, float param, int* status, cudaStream_t st) {
   if (T <= 0 || N <= 0 || K <= 0) return 0;
   if ((K & 7) || (ldx & 7) || (ldw & 7)) return -2;
   PrefillParams p{};
-  p.N = N; p.T = T; p.K = K; p.out = reinterpret_cast<__nv_bfloat16*>(Y); p.ldo = ldo; p.bias = bias; p.res_scale = 1.f; p.act = act;
+  p.N = N; p.T = T; p.K = K; p.out = reinterpret_cast<__nv_bfloat16*>(Y); p.ldo = ldo; p.bias = bias; p.res_scale = param; p.act = act;
   p.status = status; p.out_fp32 = 1;
   p.t_tiles = (T + 127) / 128;
   return prefill_tm(X, ldx, W, w_rows, ldw, p, 0, 0, st);

@@ -59,8 +59,10 @@ struct GemmParams {
   // column range starting at group * x_col_stride of X; the group's weight rows start at group * group_w_rows and its
   // results go to columns group * y_col_stride ...  `gate` (same column layout): results are multiplied with its sigmoid.
   int batch_tiles, x_col_stride, y_col_stride;
+  // (head_gate: one gate value per group instead)
   const __nv_bfloat16* gate;
   int ldg;
+  int head_gate;
   // pair != 0 (DUAL instantiation, no gating): the two accumulators are two independent 128-feature tiles
   // (rows n and n + 128 of W) sharing one token tile — 256 x BN of output per CTA, which halves the
   // operand bytes per FLOP of the compute-bound (prefill) shapes.
@@ -357,7 +359,7 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
           if (p.gate && n_ok) {
 #pragma unroll
             for (int j = 0; j < 16; ++j)
-              gt[j] = p.gate[(size_t)min(t0 + c + j, p.T - 1) * p.ldg + y_col0 + n];
+              gt[j] = p.gate[(size_t)min(t0 + c + j, p.T - 1) * p.ldg + (p.head_gate ? y_col0 / p.y_col_stride : y_col0 + n)];
           }
           if (!fused_ar) {
             load_acc(c, g, u);
@@ -425,8 +427,8 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
                 } else {
                   const float ts = (BN <= 64 && rms) ? rsqrtf(s_ssq[(c + j) & 63] / (float)p.K + p.rms_eps) : 1.f;
                   x = fused_ar ? g[j] + bias_g : g[j] * (rs * ts) + bias_g;
-                  x = apply_act(x, p.act);
-                  if (DUAL && !pair) x *= (u[j] * (rs * ts) + bias_u);
+                  if (DUAL && !pair) x = apply_gated(x, u[j] * (rs * ts) + bias_u, p.act, p.res_scale);
+                  else x = apply_act(x, p.act, p.res_scale);
                   if (p.col_scale) x *= p.col_scale[t];
                   if (p.gate) x = __fdividef(x, 1.f + __expf(-__bfloat162float(gt[j])));
                   if (p.residual) x = with_residual(x, __bfloat162float(p.residual[(size_t)t * p.ldr + n]), p.res_scale, p.act);
@@ -456,7 +458,7 @@ __global__ void __launch_bounds__(192) gemm_bf16_kernel(const __grid_constant__ 
             for (int j = 0; j < 16; ++j) {
               const int t = t0 + c + j;
               if (t < p.T && c + j < x_rows) {
-                float x = apply_act(u[j] + bias_u, p.act);
+                float x = apply_act(u[j] + bias_u, p.act, p.res_scale);
                 if (p.col_scale) x *= p.col_scale[t];
                 if (p.residual) x = with_residual(x, __bfloat162float(p.residual[(size_t)t * p.ldr + n2]), p.res_scale, p.act);
                 if (p.out_fp32) reinterpret_cast<float*>(p.out)[(size_t)t * p.ldo + n2] = x;
@@ -755,16 +757,18 @@ extern "C" int xft_gemm_bf16_grouped(const void* X, int ldx, int x_rows, const v
 }
 
 // One product per head: Y[:, h * ys + n] = sum_k X[:, h * xs + k] W[h * N + n, k] for h < heads, n < N, k < K; W is
-// [heads * N, K].  gate (bf16 [T, ldg], columns laid out as Y's) or null: results are multiplied with sigmoid(gate).
+// [heads * N, K].  gate (bf16 [T, ldg], columns laid out as Y's, or with head_gate one per head) or null: results are multiplied
+// with sigmoid(gate).
 // xs and K multiples of 8; columns of X from h * xs + K up to the next multiple of 64 are read (times zero).
 extern "C" int xft_gemm_bf16_heads(const void* X, int ldx, int x_cols, int xs, const void* W, int ldw, void* Y, int ldo, int ys,
-                                   int heads, int T, int N, int K, const void* gate, int ldg, int* status, cudaStream_t st) {
+                                   int heads, int T, int N, int K, const void* gate, int ldg, int head_gate, int* status,
+                                   cudaStream_t st) {
   if (T <= 0 || N <= 0 || K <= 0 || heads <= 0) return 0;
   if ((xs & 7) || (K & 7) || (heads - 1) * xs + K > x_cols || x_cols > ldx || (heads - 1) * ys + N > ldo) return -1;
   GemmParams p{};
   p.N = N; p.T = T; p.K = K; p.out = Y; p.ldo = ldo; p.res_scale = 1.f; p.status = status;
   p.group_w_rows = N; p.x_col_stride = xs; p.y_col_stride = ys;
-  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate); p.ldg = ldg;
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate); p.ldg = ldg; p.head_gate = head_gate;
   const int bn = min(pick_bn(T), 128);
   p.batch_tiles = (T + bn - 1) / bn;
   p.n_tiles = (N + 127) / 128;

@@ -5,6 +5,13 @@
 //   o_t = S_t^T (q_t / sqrt(dim))                          [vdim]
 //   out = o / sqrt(mean(o^2) + eps) * gain * silu(g_t)
 //
+// and two relatives of it in the same kernels:
+//
+//   time mixing    alpha_t = exp(-exp(W_a2 a1_t + bias)), o_t = (S_(t-1) + diag(u) k_t v_t^T)^T (q_t scale): the state is read
+//                  before it moves on, and the current token counts with a bonus u per channel
+//   state space    (step kernel) one decay exp(-rate dt) per head and token, k scaled by dt = softplus(raw + bias), q and k shared by
+//                  groups of heads; what leaves is o + D v in fp32, its gate and norm follow in a kernel of their own
+//
 // Rows of x are packed [q | k | v | g | a1] (queries, keys, values and gate of all heads, the decay's first product).  A
 // sequence's state lives in its slot of a pool [slots, heads, dim, vdim]; its first token starts from zero whatever the slot
 // holds.  Two kernels share a batch, by the length of a sequence's portion:
@@ -28,7 +35,7 @@
 // every segment but the last, from zero; in the second each segment starts from the decayed sum of the ones before it.
 //
 // This file is compiled without fast-math; the chunk kernel asks for the fast exponential and logarithm by name.
-#include "ptx.cuh"
+#include "mma_sync.cuh"
 
 namespace xft {
 
@@ -49,7 +56,13 @@ struct GlaParams {
   float* seg_state;                        // [B, heads, segs, dim, vdim]: the initial state, then what segment j - 1 leaves
   float* seg_decay;                        // [B, heads, segs, dim]: sum of log2(alpha) over segment j - 1
   int* status;
+  const float* bonus;                      // [heads, dim] (time mixing)
+  int gain_ld; float mult;                 // gain of head h at h * gain_ld; a factor of the result
+  // state space: q columns start at q_at, heads_per_group heads share q and k, raw step sizes [T, ld_dt], fp32 vectors [heads]
+  int q_at, heads_per_group;
+  const void* dt; int ld_dt; const float* dt_bias; const float* rate; const float* skip;
 };
+enum GlaMode { kGla = 0, kTimeMix = 1, kStateSpace = 2 };
 
 template <typename T> __device__ __forceinline__ float gl_f32(T v);
 template <> __device__ __forceinline__ float gl_f32<float>(float v) { return v; }
@@ -68,14 +81,15 @@ __device__ __forceinline__ int gl_slot(const GlaParams& p, int b) {
 constexpr int kStepThreads = 256;
 
 // LC lanes share a row of the state (4 columns each), RPT rows per thread
-template <typename T, int LC, int RPT>
+template <typename T, int LC, int RPT, int MODE>
 __global__ void __launch_bounds__(kStepThreads) gla_step_kernel(const GlaParams p) {
   constexpr int CW = LC * 4, GROUPS = kStepThreads / LC, NW = kStepThreads / 32;
   extern __shared__ float gs_sm[];
   float* sq = gs_sm;                       // [dim] each
   float* sk = sq + p.dim;
   float* sa = sk + p.dim;
-  float* sr = sa + p.dim;                  // [rank_ld]
+  float* sb = sa + p.dim;                  // time mixing: the bonus' scores
+  float* sr = sb + (MODE == kTimeMix ? p.dim : 0);        // [rank_ld]
   __shared__ float red[NW][CW];
   __shared__ float ssq[2][NW];
   __shared__ float peer_ss[2];
@@ -107,14 +121,27 @@ __global__ void __launch_bounds__(kStepThreads) gla_step_kernel(const GlaParams 
   }
   grid_dep_wait();
   const T* a2 = reinterpret_cast<const T*>(p.a2) + (size_t)h * p.dim * p.rank_ld;
+  const int kh = MODE == kStateSpace ? h / p.heads_per_group : h;                      // the head of q and k
   for (int i = 0; i < n; ++i) {
     const T* row = reinterpret_cast<const T*>(p.x) + (size_t)(start + i) * p.ldx;
+    if (MODE != kStateSpace)
     for (int r = tid; r < p.rank_ld; r += kStepThreads) sr[r] = r < p.rank ? gl_f32<T>(row[p.a_at + r]) : 0.f;
     float v[4];
 #pragma unroll
     for (int j = 0; j < 4; ++j) v[j] = c0 + j < p.vdim ? gl_f32<T>(row[p.v_at + h * p.vdim + c0 + j]) : 0.f;
+    float keep = 0.f, dt = 1.f;
+    if (MODE == kStateSpace) {
+      const float z = gl_f32<T>(reinterpret_cast<const T*>(p.dt)[(size_t)(start + i) * p.ld_dt + h]) + p.dt_bias[h];
+      dt = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
+      keep = expf(-p.rate[h] * dt);
+    }
     __syncthreads();
     for (int d = tid; d < p.dim; d += kStepThreads) {
+      if (MODE == kStateSpace) {
+        sq[d] = gl_f32<T>(row[p.q_at + kh * p.dim + d]);
+        sk[d] = gl_f32<T>(row[p.k_at + kh * p.dim + d]) * dt;
+        continue;
+      }
       float z = p.bias[h * p.dim + d];
       const T* wr = a2 + (size_t)d * p.rank_ld;
       for (int r = 0; r < p.rank_ld; r += 8) {            // rows of a2 are multiples of 8 values, zeros behind the rank
@@ -123,10 +150,12 @@ __global__ void __launch_bounds__(kStepThreads) gla_step_kernel(const GlaParams 
 #pragma unroll
         for (int e = 0; e < 8; ++e) z = fmaf(gl_f32<T>(w.e[e]), sr[r + e], z);
       }
-      const float la = (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * p.inv_tau;      // log(sigmoid(z)) / tau
+      // log(sigmoid(z)) / tau, or -exp(z)
+      const float la = MODE == kTimeMix ? -expf(z) : (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * p.inv_tau;
       sa[d] = expf(la);
       sq[d] = gl_f32<T>(row[h * p.dim + d]) * p.scale;
       sk[d] = gl_f32<T>(row[p.k_at + h * p.dim + d]);
+      if (MODE == kTimeMix) sb[d] = sq[d] * sk[d] * p.bonus[h * p.dim + d];
     }
     __syncthreads();
     float o[4] = {0.f, 0.f, 0.f, 0.f};
@@ -134,11 +163,13 @@ __global__ void __launch_bounds__(kStepThreads) gla_step_kernel(const GlaParams 
     for (int r = 0; r < RPT; ++r) {
       const int d = r * GROUPS + grp;
       if (d < p.dim) {
-        const float al = sa[d], kk = sk[d], qq = sq[d];
+        const float al = MODE == kStateSpace ? keep : sa[d], kk = sk[d], qq = sq[d];
+        const float bb = MODE == kTimeMix ? sb[d] : 0.f;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
+          if (MODE == kTimeMix) o[j] = fmaf(qq, S[r][j], fmaf(bb, v[j], o[j]));
           S[r][j] = fmaf(al, S[r][j], kk * v[j]);
-          o[j] = fmaf(qq, S[r][j], o[j]);
+          if (MODE != kTimeMix) o[j] = fmaf(qq, S[r][j], o[j]);
         }
       }
     }
@@ -158,6 +189,11 @@ __global__ void __launch_bounds__(kStepThreads) gla_step_kernel(const GlaParams 
 #pragma unroll
       for (int w = 0; w < NW; ++w) y += red[w][tid];
     }
+    if (MODE == kStateSpace) {
+      if (mine)
+        p.raw[(size_t)(start + i) * p.heads * p.vdim + h * p.vdim + col] = fmaf(p.skip[h], gl_f32<T>(row[p.v_at + h * p.vdim + col]), y);
+      continue;
+    }
     float ss = mine ? y * y : 0.f;
 #pragma unroll
     for (int m = 16; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
@@ -175,7 +211,7 @@ __global__ void __launch_bounds__(kStepThreads) gla_step_kernel(const GlaParams 
     }
     if (mine) {
       const float g = gl_f32<T>(row[p.g_at + h * p.vdim + col]);
-      const float r = y / sqrtf(ss / (float)p.vdim + p.eps) * p.gain[col] * (g / (1.f + expf(-g)));
+      const float r = y / sqrtf(ss / (float)p.vdim + p.eps) * p.gain[h * p.gain_ld + col] * (g / (1.f + expf(-g))) * p.mult;
       reinterpret_cast<T*>(p.out)[(size_t)(start + i) * p.ldo + h * p.vdim + col] = gl_from<T>(r);
     }
   }
@@ -191,37 +227,13 @@ __global__ void __launch_bounds__(kStepThreads) gla_step_kernel(const GlaParams 
       }
     }
   }
-  if (nslices > 1) { cluster_arrive(); cluster_wait(); }  // nobody leaves while its shared memory may be read
+  if (MODE != kStateSpace && nslices > 1) { cluster_arrive(); cluster_wait(); }  // nobody leaves while its shared memory may be read
 }
 
 // ------------------------------------------------------------------------------------------ chunks of 64 tokens
-__device__ __forceinline__ void gl_ldsm(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void gl_ldsm_t(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void gl_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t gl_pack(float lo, float hi) {
-  const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-  return *reinterpret_cast<const uint32_t*>(&v);
-}
-__device__ __forceinline__ float2 gl_unpack(uint32_t v) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v)); }
-
 constexpr int kChunk = 64, kPiece = 16;
 constexpr float kMaxDecay = 60.f;
 
-// approximate instructions of the special-function unit, denormals flushed
-__device__ __forceinline__ float gl_ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
-__device__ __forceinline__ float gl_lg2(float x) { float y; asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
-__device__ __forceinline__ float gl_rcp(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
-constexpr float kLog2e = 1.4426950408889634f;
 // x * sigmoid(x); e^-x past the largest float makes it 0
 __device__ __forceinline__ float gl_silu(float x) { return x * gl_rcp(1.f + gl_ex2(-x * kLog2e)); }
 
@@ -237,12 +249,12 @@ struct ChunkCfg {
   // the running sums are done with when the state is written as an operand: one place for both
   static constexpr size_t SHARED = (size_t)kChunk * BS * 4 > (size_t)DP * VSS * 2 ? (size_t)kChunk * BS * 4 : (size_t)DP * VSS * 2;
   static constexpr size_t B16 = (size_t)STAGES * STAGE + kChunk * AS + DP * RS;
-  static constexpr size_t F32 = 8 * DP + 4 * 2 * DP + DP + 4 * kChunk + VS;
+  static constexpr size_t F32 = 8 * DP + 4 * 2 * DP + 2 * DP + 5 * kChunk + VS;
   static constexpr size_t SMEM = B16 * 2 + SHARED + F32 * 4;
   static_assert(SMEM <= 227 * 1024, "shared memory");
 };
 
-template <int DP, int VS, int RP>
+template <int DP, int VS, int RP, bool BONUS>
 __global__ void __launch_bounds__(kChunkThreads, 1) gla_chunk_kernel(const GlaParams p) {
   using Cfg = ChunkCfg<DP, VS, RP>;
   constexpr int NT = kChunkThreads;
@@ -262,6 +274,8 @@ __global__ void __launch_bounds__(kChunkThreads, 1) gla_chunk_kernel(const GlaPa
   float* sBias = sMid + 4 * DP;
   float* sSS = sBias + DP;                                // [4][64] sums of squares of the output rows
   float* sGain = sSS + 4 * kChunk;
+  float* sU = sGain + VS;                                 // the bonus [DP], and the scores it gives the rows [64]
+  float* sDiag = sU + DP;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int h = blockIdx.y, b = blockIdx.z, seg = blockIdx.x % p.segs, v0 = blockIdx.x / p.segs * VS;
   grid_dep_launch();
@@ -283,8 +297,11 @@ __global__ void __launch_bounds__(kChunkThreads, 1) gla_chunk_kernel(const GlaPa
     const int d = i / RP, r = i % RP;
     sW[d * RS + r] = d < p.dim && r < p.rank ? a2[(size_t)d * p.rank_ld + r] : __float2bfloat16(0.f);
   }
-  for (int d = tid; d < DP; d += NT) { sBias[d] = d < p.dim ? p.bias[h * p.dim + d] : 0.f; }
-  for (int c = tid; c < VS; c += NT) sGain[c] = c < vw ? p.gain[v0 + c] : 0.f;
+  for (int d = tid; d < DP; d += NT) {
+    sBias[d] = d < p.dim ? p.bias[h * p.dim + d] : 0.f;
+    if (BONUS) sU[d] = d < p.dim ? p.bonus[h * p.dim + d] * p.scale : 0.f;
+  }
+  for (int c = tid; c < VS; c += NT) sGain[c] = c < vw ? p.gain[h * p.gain_ld + v0 + c] * p.mult : 0.f;
   // the state: warp tile of 16 rows and NPW x 8 columns
   const int sd = (warp % MW) * 16 + (lane >> 2), sn0 = warp / MW * NPW * 8, sc = sn0 + 2 * (lane & 3);
   float post0 = 1.f, post1 = 1.f;                         // factors of the two rows still to come
@@ -395,7 +412,9 @@ __global__ void __launch_bounds__(kChunkThreads, 1) gla_chunk_kernel(const GlaPa
 #pragma unroll
           for (int k = 0; k < 2; ++k) {
             const float zz = z[j][2 * e + k] + (k ? bias.y : bias.x);
-            const float la = fminf(zz, 0.f) * tau2 - gl_lg2(1.f + gl_ex2(-fabsf(zz) * kLog2e)) * p.inv_tau;
+            // (a decay of 2^-200 is none that fp32 could tell from zero)
+            const float la = BONUS ? fmaxf(-kLog2e * gl_ex2(zz * kLog2e), -200.f)
+                                   : fminf(zz, 0.f) * tau2 - gl_lg2(1.f + gl_ex2(-fabsf(zz) * kLog2e)) * p.inv_tau;
             l[k] = r < rows && d + k < p.dim ? la : 0.f;
           }
           *reinterpret_cast<float2*>(sB + r * BS + d) = make_float2(l[0], l[1]);
@@ -418,6 +437,19 @@ __global__ void __launch_bounds__(kChunkThreads, 1) gla_chunk_kernel(const GlaPa
       *reinterpret_cast<float2*>(sT + g * DP + 2 * pr) = c;
     }
     __syncthreads();
+    if (BONUS && !p.carry) {                               // the rows' scores with themselves, from q and k as they came
+#pragma unroll
+      for (int r = warp * 4; r < warp * 4 + 4; ++r) {
+        float a = 0.f;
+        for (int d = 2 * lane; d < DP; d += 64) {
+          const float2 q = gl_unpack(*reinterpret_cast<const uint32_t*>(sq + r * QS + d)), k = gl_unpack(*reinterpret_cast<const uint32_t*>(sk + r * QS + d));
+          a += q.x * k.x * sU[d] + q.y * k.y * sU[d + 1];
+        }
+#pragma unroll
+        for (int m = 16; m > 0; m >>= 1) a += __shfl_xor_sync(0xffffffffu, a, m);
+        if (lane == 0) sDiag[r] = a;
+      }
+    }
     bool ok = true;
     for (int d = tid; d < DP; d += NT) {
       float t = 0.f;
@@ -447,14 +479,15 @@ __global__ void __launch_bounds__(kChunkThreads, 1) gla_chunk_kernel(const GlaPa
           const int g = i / (kPiece * kPiece), t = g * kPiece + i / kPiece % kPiece, s = g * kPiece + i % kPiece;
           if (!(harsh >> g & 1)) continue;
           float a = 0.f;
-          if (s <= t)
+          if (BONUS ? s < t : s <= t)
             for (int d = lane; d < p.dim; d += 32) {
               const float between = (t & 8) && !(s & 8) ? sT[2 * g * DP + d] : 0.f;       // the sums restart between s and t
-              a += __bfloat162float(sq[t * QS + d]) * __bfloat162float(sk[s * QS + d]) * gl_ex2(sB[t * BS + d] - sB[s * BS + d] + between);
+              const float bt = !BONUS ? sB[t * BS + d] : t & 7 ? sB[(t - 1) * BS + d] : 0.f;
+              a += __bfloat162float(sq[t * QS + d]) * __bfloat162float(sk[s * QS + d]) * gl_ex2(bt - sB[s * BS + d] + between);
             }
 #pragma unroll
           for (int m = 16; m > 0; m >>= 1) a += __shfl_xor_sync(0xffffffffu, a, m);
-          if (lane == 0) sA[t * AS + s] = __float2bfloat16(a * p.scale);
+          if (lane == 0) sA[t * AS + s] = __float2bfloat16(BONUS && s == t ? sDiag[t] : a * p.scale);
         }
         __syncthreads();
       }
@@ -479,16 +512,19 @@ __global__ void __launch_bounds__(kChunkThreads, 1) gla_chunk_kernel(const GlaPa
         *reinterpret_cast<float2*>(sPre + (lo >> 1) * DP + 2 * pr) = e;
       }
       const float2 qo = make_float2(base.x - qr.x + scale2, base.y - qr.y + scale2), ko = make_float2(kr.x - base.x, kr.y - base.y);
+      float2 before = make_float2(0.f, 0.f);
 #pragma unroll
       for (int r = 0; r < 8; ++r) {
         const int t = g * 8 + r;
         const float2 bb = *reinterpret_cast<const float2*>(sB + t * BS + 2 * pr);
+        const float2 bq = BONUS ? before : bb;             // the state is read before this token's decay
+        before = bb;
         uint32_t* qp = reinterpret_cast<uint32_t*>(sq + t * QS + 2 * pr);
         uint32_t* kp = reinterpret_cast<uint32_t*>(sk + t * QS + 2 * pr);
         const float2 k = gl_unpack(*kp);
         if (!p.carry) {
           const float2 q = gl_unpack(*qp);
-          *qp = gl_pack(q.x * gl_ex2(bb.x + qo.x), q.y * gl_ex2(bb.y + qo.y));
+          *qp = gl_pack(q.x * gl_ex2(bq.x + qo.x), q.y * gl_ex2(bq.y + qo.y));
         }
         *kp = gl_pack(k.x * gl_ex2(ko.x - bb.x), k.y * gl_ex2(ko.y - bb.y));
       }
@@ -536,7 +572,10 @@ __global__ void __launch_bounds__(kChunkThreads, 1) gla_chunk_kernel(const GlaPa
 #pragma unroll
           for (int e = 0; e < 4; e += 2) {
             const int t = r0 + (e >> 1) * 8, s = kt * 16 + j * 8 + cc;
-            *reinterpret_cast<uint32_t*>(sA + t * AS + s) = gl_pack(s <= t ? A[j][e] : 0.f, s + 1 <= t ? A[j][e + 1] : 0.f);
+            float a0 = s <= t ? A[j][e] : 0.f, a1 = s + 1 <= t ? A[j][e + 1] : 0.f;
+            if (BONUS && s == t) a0 = sDiag[t];
+            if (BONUS && s + 1 == t) a1 = sDiag[t];
+            *reinterpret_cast<uint32_t*>(sA + t * AS + s) = gl_pack(a0, a1);
           }
       }
       if (pc == 0 && even && !p.raw && !p.carry) {         // fetched here, used behind the products
@@ -678,7 +717,7 @@ __global__ void __launch_bounds__(128) gla_norm_kernel(const GlaParams p, int n_
   bf16* op = reinterpret_cast<bf16*>(p.out) + (size_t)t * p.ldo + h * p.vdim;
   for (int c = lane; c < p.vdim; c += 32) {
     const float g = __bfloat162float(gp[c]);
-    op[c] = __float2bfloat16(o[c] * inv * p.gain[c] * __fdividef(g, 1.f + __expf(-g)));
+    op[c] = __float2bfloat16(o[c] * inv * p.gain[h * p.gain_ld + c] * p.mult * __fdividef(g, 1.f + __expf(-g)));
   }
 }
 
@@ -686,17 +725,17 @@ __global__ void __launch_bounds__(128) gla_norm_kernel(const GlaParams p, int n_
 
 using namespace xft;
 
-template <typename T, int LC, int RPT>
+template <typename T, int LC, int RPT, int MODE>
 static int launch_step(const GlaParams& p, cudaStream_t st) {
   const int slices = (p.vdim + LC * 4 - 1) / (LC * 4);
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(slices, p.heads, p.B);
   cfg.blockDim = dim3(kStepThreads);
-  cfg.dynamicSmemBytes = (size_t)(3 * p.dim + p.rank_ld) * sizeof(float);
+  cfg.dynamicSmemBytes = (size_t)((MODE == kTimeMix ? 4 : 3) * p.dim + p.rank_ld) * sizeof(float);
   cfg.stream = st;
   cudaLaunchAttribute at[2];
   int na = 0;
-  if (slices > 1) {
+  if (slices > 1 && MODE != kStateSpace) {
     at[na].id = cudaLaunchAttributeClusterDimension;
     at[na].val.clusterDim.x = slices; at[na].val.clusterDim.y = 1; at[na].val.clusterDim.z = 1;
     ++na;
@@ -708,33 +747,33 @@ static int launch_step(const GlaParams& p, cudaStream_t st) {
   }
   cfg.attrs = at;
   cfg.numAttrs = na;
-  cudaError_t e = cudaLaunchKernelEx(&cfg, gla_step_kernel<T, LC, RPT>, p);
+  cudaError_t e = cudaLaunchKernelEx(&cfg, gla_step_kernel<T, LC, RPT, MODE>, p);
   return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }
-template <typename T, int LC>
+template <typename T, int LC, int MODE>
 static int step_rows(const GlaParams& p, cudaStream_t st) {
   const int rows = (p.dim + kStepThreads / LC - 1) / (kStepThreads / LC);
-  if (rows <= 2) return launch_step<T, LC, 2>(p, st);
-  if (rows <= 4) return launch_step<T, LC, 4>(p, st);
-  if (rows <= 8) return launch_step<T, LC, 8>(p, st);
-  if (rows <= 16) return launch_step<T, LC, 16>(p, st);
-  if (rows <= 32) return launch_step<T, LC, 32>(p, st);
+  if (rows <= 2) return launch_step<T, LC, 2, MODE>(p, st);
+  if (rows <= 4) return launch_step<T, LC, 4, MODE>(p, st);
+  if (rows <= 8) return launch_step<T, LC, 8, MODE>(p, st);
+  if (rows <= 16) return launch_step<T, LC, 16, MODE>(p, st);
+  if (rows <= 32) return launch_step<T, LC, 32, MODE>(p, st);
   return -5;
 }
-template <typename T>
+template <typename T, int MODE>
 static int step_columns(const GlaParams& p, int columns, cudaStream_t st) {
-  if (columns == 32) return step_rows<T, 8>(p, st);
-  if (columns == 64) return step_rows<T, 16>(p, st);
-  if (columns == 128) return step_rows<T, 32>(p, st);
+  if (columns == 32) return step_rows<T, 8, MODE>(p, st);
+  if (columns == 64) return step_rows<T, 16, MODE>(p, st);
+  if (columns == 128) return step_rows<T, 32, MODE>(p, st);
   return -6;
 }
 
-template <int DP, int VS, int RP>
-static int launch_chunk(const GlaParams& p, cudaStream_t st) {
+template <int DP, int VS, int RP, bool BONUS>
+static int launch_chunk_mode(const GlaParams& p, cudaStream_t st) {
   using Cfg = ChunkCfg<DP, VS, RP>;
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(gla_chunk_kernel<DP, VS, RP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM) != cudaSuccess)
+    if (cudaFuncSetAttribute(gla_chunk_kernel<DP, VS, RP, BONUS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM) != cudaSuccess)
       return 3000 + (int)cudaGetLastError();
     attr_set = true;
   }
@@ -743,10 +782,14 @@ static int launch_chunk(const GlaParams& p, cudaStream_t st) {
   if (p.segs > 1) {
     GlaParams q = p;
     q.carry = 1;
-    e = launch_pdl(gla_chunk_kernel<DP, VS, RP>, grid, dim3(kChunkThreads), Cfg::SMEM, st, q);
+    e = launch_pdl(gla_chunk_kernel<DP, VS, RP, BONUS>, grid, dim3(kChunkThreads), Cfg::SMEM, st, q);
   }
-  if (e == cudaSuccess) e = launch_pdl(gla_chunk_kernel<DP, VS, RP>, grid, dim3(kChunkThreads), Cfg::SMEM, st, p);
+  if (e == cudaSuccess) e = launch_pdl(gla_chunk_kernel<DP, VS, RP, BONUS>, grid, dim3(kChunkThreads), Cfg::SMEM, st, p);
   return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
+}
+template <int DP, int VS, int RP>
+static int launch_chunk(const GlaParams& p, cudaStream_t st) {
+  return p.bonus ? launch_chunk_mode<DP, VS, RP, true>(p, st) : launch_chunk_mode<DP, VS, RP, false>(p, st);
 }
 template <int DP, int VS>
 static int chunk_rank(const GlaParams& p, cudaStream_t st) {
@@ -763,26 +806,46 @@ extern "C" int xft_gla_chunk_columns(int dim, int vdim, int rank) {
 
 // x, a2 and out all fp32 (f32 = 1) or bf16; row strides and offsets as the file comment says, all multiples of 8 (a2's rows
 // too).  Sequences with min_q <= tokens < max_q take part, the others are left alone.  columns: of the state per CTA, 32, 64
-// or 128, at most 8 CTAs per head; rows per CTA: dim <= columns-dependent limit (1024, 512, 256).
+// or 128, at most 8 CTAs per head; rows per CTA: dim <= columns-dependent limit (1024, 512, 256).  bonus [heads, dim] (fp32): time
+// mixing, null: gated linear attention.  gain [vdim] (gain_ld 0) or [heads, gain_ld].
 extern "C" int xft_gla_step(const void* x, int ldx, int k_at, int v_at, int g_at, int a_at, int heads, int dim, int vdim, int rank,
-                            int rank_ld, const void* a2, const float* bias, float tau, float scale, float eps, const float* gain,
+                            int rank_ld, const void* a2, const float* bias, float tau, float scale, float eps, const float* bonus, int gain_ld, float mult, const float* gain,
                             float* state, const int* state_slots, int num_states, const int* cu_q, const int* kv_lens, int B,
                             void* out, int ldo, int min_q, int max_q, int columns, int f32, int* status, cudaStream_t st) {
   if (B <= 0) return 0;
   if (heads <= 0 || dim <= 0 || vdim <= 0 || rank <= 0 || rank_ld < rank || (rank_ld & 7) || tau <= 0.f || num_states <= 0 ||
       columns <= 0) return -1;
-  if (heads > 65535 || B > 65535 || (vdim + columns - 1) / columns > 8 || (size_t)(3 * dim + rank_ld) * 4 > 40000) return -2;
+  if (heads > 65535 || B > 65535 || (vdim + columns - 1) / columns > 8 || (size_t)(4 * dim + rank_ld) * 4 > 40000) return -2;
   if (((uintptr_t)a2 | (uintptr_t)state) & 15) return -3;
   GlaParams p{x, ldx, k_at, v_at, g_at, a_at, heads, dim, vdim, rank, rank_ld, a2, bias, 1.f / tau, scale, eps, gain, state, state_slots,
               num_states, cu_q, kv_lens, B, out, ldo, nullptr, min_q, max_q, 1, 0, nullptr, nullptr, status};
-  return f32 ? step_columns<float>(p, columns, st) : step_columns<bf16>(p, columns, st);
+  p.bonus = bonus; p.gain_ld = gain_ld; p.mult = mult;
+  if (bonus) return f32 ? step_columns<float, kTimeMix>(p, columns, st) : step_columns<bf16, kTimeMix>(p, columns, st);
+  return f32 ? step_columns<float, kGla>(p, columns, st) : step_columns<bf16, kGla>(p, columns, st);
+}
+
+// The recurrence of a state-space layer, token by token: x rows hold q, k (groups x dim each) and v (heads x vdim) from columns q_at,
+// k_at and v_at; dt [T, ld_dt] raw step sizes of the rows' type; dt_bias, rate, skip fp32 [heads]; raw fp32 [T, heads * vdim] out.
+extern "C" int xft_ssd_step(const void* x, int ldx, int q_at, int k_at, int v_at, int heads, int heads_per_group, int dim, int vdim,
+                            const void* dt, int ld_dt, const float* dt_bias, const float* rate, const float* skip, float* state,
+                            const int* state_slots, int num_states, const int* cu_q, const int* kv_lens, int B, float* raw, int min_q,
+                            int max_q, int columns, int f32, int* status, cudaStream_t st) {
+  if (B <= 0) return 0;
+  if (heads <= 0 || dim <= 0 || vdim <= 0 || heads_per_group <= 0 || heads % heads_per_group || num_states <= 0 || columns <= 0) return -1;
+  if (heads > 65535 || B > 65535 || (size_t)3 * dim * 4 > 40000 || ((uintptr_t)state & 15)) return -2;
+  GlaParams p{};
+  p.x = x; p.ldx = ldx; p.q_at = q_at; p.k_at = k_at; p.v_at = v_at; p.heads = heads; p.heads_per_group = heads_per_group;
+  p.dim = dim; p.vdim = vdim; p.dt = dt; p.ld_dt = ld_dt; p.dt_bias = dt_bias; p.rate = rate; p.skip = skip;
+  p.state = state; p.state_slots = state_slots; p.num_states = num_states; p.cu_q = cu_q; p.kv_lens = kv_lens; p.B = B;
+  p.raw = raw; p.min_q = min_q; p.max_q = max_q; p.segs = 1; p.status = status;
+  return f32 ? step_columns<float, kStateSpace>(p, columns, st) : step_columns<bf16, kStateSpace>(p, columns, st);
 }
 
 // bf16 portions.  raw: fp32 [T, heads * vdim], needed when a head has more columns than xft_gla_chunk_columns says.
 // segs > 1: portions are cut into so many segments (two launches), with scratch seg_state fp32 [B, heads, segs, dim, vdim] and
 // seg_decay fp32 [B, heads, segs, dim].
 extern "C" int xft_gla_chunk(const void* x, int ldx, int k_at, int v_at, int g_at, int a_at, int heads, int dim, int vdim, int rank,
-                             int rank_ld, const void* a2, const float* bias, float tau, float scale, float eps, const float* gain,
+                             int rank_ld, const void* a2, const float* bias, float tau, float scale, float eps, const float* bonus, int gain_ld, float mult, const float* gain,
                              float* state, const int* state_slots, int num_states, const int* cu_q, const int* kv_lens, int B, int T,
                              void* out, int ldo, float* raw, int min_q, int max_q, int segs, float* seg_state, float* seg_decay,
                              int* status, cudaStream_t st) {
@@ -794,6 +857,7 @@ extern "C" int xft_gla_chunk(const void* x, int ldx, int k_at, int v_at, int g_a
   if ((ldx & 7) || (k_at & 7) || (v_at & 7) || (g_at & 7) || (a_at & 7) || ((uintptr_t)x & 15)) return -3;
   GlaParams p{x, ldx, k_at, v_at, g_at, a_at, heads, dim, vdim, rank, rank_ld, a2, bias, 1.f / tau, scale, eps, gain, state, state_slots,
               num_states, cu_q, kv_lens, B, out, ldo, vdim > cols ? raw : nullptr, min_q, max_q, segs, 0, seg_state, seg_decay, status};
+  p.bonus = bonus; p.gain_ld = gain_ld; p.mult = mult;
   int r;
   if (dim > 128) r = cols == 64 ? launch_chunk<256, 64, 16>(p, st) : launch_chunk<256, 128, 16>(p, st);
   else if (dim > 64) r = cols == 64 ? chunk_rank<128, 64>(p, st) : chunk_rank<128, 128>(p, st);

@@ -319,6 +319,17 @@ static cudaError_t pick_width(const HeadPrepParams& p, cudaStream_t st) {
   return pick_taps<T, 2, 8>(p, st);
 }
 
+// The convolution's state [slots, taps - 1, C] behind a call's portions, from its input rows x [T, ldx] and the old state.
+extern "C" int xft_conv_state(const void* x, int ldx, int C, int taps, const int* cu_q, const int* kv_lens, int B, void* state,
+                              const int* state_slots, int num_states, int f32, int* status, cudaStream_t st) {
+  const dim3 grid((C + 255) / 256, B);
+  cudaError_t e = f32 ? launch_pdl(conv_state_kernel<float>, grid, dim3(256), 0, st, (const float*)x, ldx, C, taps, cu_q, kv_lens,
+                                   (float*)state, state_slots, num_states, status)
+                      : launch_pdl(conv_state_kernel<bf16>, grid, dim3(256), 0, st, (const bf16*)x, ldx, C, taps, cu_q, kv_lens,
+                                   (bf16*)state, state_slots, num_states, status);
+  return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
+}
+
 // x rows, q_out, caches and state all fp32 (f32 = 1) or bf16.  caches [blocks, hkv, bs, padded].  dim <= padded <= 512, up to 8
 // taps; even dim wants even row strides.  decode: every sequence has one token in this call.
 extern "C" int xft_head_prep(const void* x, int ldx, int T, int B, int hq, int hkv, int dim, int padded, int taps, const float* conv,
@@ -337,13 +348,6 @@ extern "C" int xft_head_prep(const void* x, int ldx, int T, int B, int hq, int h
                    state, state_slots, num_states, q_out, kc, vc, bs, nslots, slots, run, decode, status};
   cudaError_t e = f32 ? pick_width<float>(p, st) : pick_width<bf16>(p, st);
   if (e != cudaSuccess) return (int)e;
-  if (taps > 1 && !decode) {
-    const dim3 grid((C + 255) / 256, B);
-    e = f32 ? launch_pdl(conv_state_kernel<float>, grid, dim3(256), 0, st, (const float*)x, ldx, C, taps, cu_q, kv_lens, (float*)state,
-                         state_slots, num_states, status)
-            : launch_pdl(conv_state_kernel<bf16>, grid, dim3(256), 0, st, (const bf16*)x, ldx, C, taps, cu_q, kv_lens, (bf16*)state,
-                         state_slots, num_states, status);
-    if (e != cudaSuccess) return (int)e;
-  }
+  if (taps > 1 && !decode) return xft_conv_state(x, ldx, C, taps, cu_q, kv_lens, B, state, state_slots, num_states, f32, status, st);
   return (int)cudaGetLastError();
 }

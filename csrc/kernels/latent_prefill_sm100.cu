@@ -33,6 +33,8 @@ int make_tensor_map(CUtensorMap* out, const void* ptr, uint64_t rows, uint64_t c
 struct FlatAttnParams {
   __nv_bfloat16* out; int ldo;               // row t, head h: columns h * 64 nv ...
   const __nv_bfloat16* gate; int ldg;        // same layout, or null
+  int head_gate;                             // the gate has one column per head instead
+  const float* sinks;                        // [heads] a score without a key per head (of all launches), or null
   const int* q_start; const int* q_len;      // [B] first row and number of rows of a sequence's queries
   const int* kv_len;                         // [B] keys visible after this call's append
   const int* span_lo; const int* span_row;   // [B] first key that lies in the flat arrays, and its row there
@@ -186,6 +188,7 @@ __global__ void __launch_bounds__(384, 1) attn_flat_tc_kernel(const __grid_const
       const uint32_t lane_addr = tmem + (uint32_t(qd * 32) << 16);
       const uint32_t sa = lane_addr + i * 128, oa = lane_addr + 256 + i * 128;
       float m = -INFINITY, l = 0.f;
+      if (p.sinks) { m = p.sinks[p.head0 + hl] * 1.4426950408889634f; l = 1.f; }
       bool ok = true;
       for (int j = 0; j < n_tiles; ++j) {
         if (!mbar_wait(&s_full[i], j & 1, p.status, XFT_ERR_WAIT_TMEM)) { ok = false; break; }
@@ -254,7 +257,8 @@ __global__ void __launch_bounds__(384, 1) attn_flat_tc_kernel(const __grid_const
         const float inv = l > 0.f ? 1.f / l : 0.f;
         const size_t col = (size_t)(p.head0 + hl) * p.nv * 64;
         __nv_bfloat16* dst = p.out + (size_t)(q0 + qrow) * p.ldo + col;
-        const __nv_bfloat16* gt = p.gate ? p.gate + (size_t)(q0 + qrow) * p.ldg + col : nullptr;
+        const __nv_bfloat16* gt = p.gate ? p.gate + (size_t)(q0 + qrow) * p.ldg + (p.head_gate ? p.head0 + hl : col) : nullptr;
+        const float hg = gt && p.head_gate && qrow < q_len ? __fdividef(inv, 1.f + __expf(-__bfloat162float(*gt))) : inv;
         for (int c = 0; c < p.nv * 64; c += 32) {
           uint32_t o[32];
           tmem_ld32(oa + c, o);
@@ -264,8 +268,8 @@ __global__ void __launch_bounds__(384, 1) attn_flat_tc_kernel(const __grid_const
             for (int g = 0; g < 4; ++g) {
               float x[8];
 #pragma unroll
-              for (int e = 0; e < 8; ++e) x[e] = __uint_as_float(o[g * 8 + e]) * inv;
-              if (gt) {
+              for (int e = 0; e < 8; ++e) x[e] = __uint_as_float(o[g * 8 + e]) * hg;
+              if (gt && !p.head_gate) {
                 const uint4 u = *reinterpret_cast<const uint4*>(gt + c + g * 8);
                 const __nv_bfloat162* hb = reinterpret_cast<const __nv_bfloat162*>(&u);
 #pragma unroll
@@ -303,12 +307,12 @@ using namespace xft;
 // Causal attention of prompt rows over flat keys (see the file comment).  Q [T, ldq] (head h at columns h * q_head: nc1 + nc2
 // chunks of 64); kv [rows, ldkv]: per head of this launch nc1 * 64 key columns, then, from v_col0 on, nv * 64 value columns;
 // shared [rows, lds]: the shared key part at columns r_col0 ...; out [T, ldo] and gate [T, ldg] (or null): head h at columns
-// h * nv * 64.  Heads head0 .. head0 + heads - 1.  Per sequence of B: q_start, q_len, kv_len, span_lo, span_row.
+// h * nv * 64 (head_gate: column h of the gate).  sinks [all heads] or null.  Heads head0 .. head0 + heads - 1.  Per sequence of B: q_start, q_len, kv_len, span_lo, span_row.
 // Returns 0, -1 for sizes it does not have, or a CUDA / tensor-map error.
 extern "C" int xft_attn_flat_tc(const void* q, int ldq, int q_cols, int q_head, const void* kv, int ldkv, int v_col0,
-                                const void* shared, int lds, int r_col0, int rows, void* out, int ldo, const void* gate, int ldg,
+                                const void* shared, int lds, int r_col0, int rows, void* out, int ldo, const void* gate, int ldg, int head_gate,
                                 const int* q_start, const int* q_len, const int* kv_len, const int* span_lo, const int* span_row,
-                                int B, int T, int max_q, int head0, int heads, int nc1, int nc2, int nv, float scale, int window,
+                                int B, int T, int max_q, int head0, int heads, int nc1, int nc2, int nv, float scale, const float* sinks, int window,
                                 int* status, cudaStream_t st) {
   if (B <= 0 || T <= 0 || max_q <= 0 || heads <= 0) return 0;
   const int nq = nc1 + nc2;
@@ -317,8 +321,9 @@ extern "C" int xft_attn_flat_tc(const void* q, int ldq, int q_cols, int q_head, 
       heads * nc1 * 64 > v_col0 || r_col0 + nc2 * 64 > lds || (head0 + heads - 1) * q_head + nq * 64 > q_cols || q_cols > ldq ||
       (head0 + heads) * nv * 64 > ldo)
     return -2;
-  if (((uintptr_t)out | (uintptr_t)gate) & 15) return -3;
+  if (((uintptr_t)out | (head_gate ? 0 : (uintptr_t)gate)) & 15) return -3;
   FlatAttnParams p{};
+  p.head_gate = head_gate; p.sinks = sinks;
   p.out = (__nv_bfloat16*)out; p.ldo = ldo; p.gate = (const __nv_bfloat16*)gate; p.ldg = ldg;
   p.q_start = q_start; p.q_len = q_len; p.kv_len = kv_len; p.span_lo = span_lo; p.span_row = span_row;
   p.q_head = q_head; p.head0 = head0; p.nc1 = nc1; p.nc2 = nc2; p.nv = nv; p.v_col0 = v_col0; p.r_col0 = r_col0;

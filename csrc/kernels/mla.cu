@@ -18,7 +18,7 @@
 // when that leaves SMs idle, over several clusters, whose parts meet in global scratch (the CTA that arrives last on a part
 // of the columns finishes it; nobody waits).
 //
-// A sliding window restricts the tiles to those that hold a visible key.
+// A sliding window restricts the tiles to those that hold a visible key.  A sink starts a head's online softmax in the first part.
 #include "ptx.cuh"
 
 namespace xft {
@@ -39,6 +39,7 @@ struct MlaParams {
   const int* cu_q; const int* kv_lens;
   int B, T, hl, bs, num_blocks;
   float scale;
+  const float* sinks;                            // [hl] a score without a key per head, or null
   int window;                                    // keys within `window` positions are visible (2^30: all)
   int nsplit, groups;                            // cluster size; clusters per (token, 16 heads)
   float* part_o; float* part_ml; int* counters;  // groups > 1: [unit][group][16][LAT], [unit][group][rank][16][2], [unit][rank]
@@ -155,6 +156,11 @@ __global__ void __launch_bounds__(384, 1) mla_attn_kernel(const __grid_constant_
     asm volatile("setmaxnreg.inc.sync.aligned.u32 232;");
     grid_dep_wait();
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    if (p.sinks && split == 0) {                                       // it counts once: in the first part
+#pragma unroll
+      for (int r = 0; r < 2; ++r)
+        if (2 * warp + r < nq) { m[r] = p.sinks[h0 + 2 * warp + r]; l[r] = lane == 0 ? 1.f : 0.f; }
+    }
     float o[NT][4];
 #pragma unroll
     for (int i = 0; i < NT; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
@@ -372,20 +378,20 @@ static int launch_mla(const MlaParams& p, const void* cache, cudaStream_t st) {
 }
 
 // Sizes of the latent (64, 128, 256 or 512, with 64 rotated key dimensions next to it) and a sliding window: position i
-// sees the keys j <= i with i - j < window (0: all).  nsplit: CTAs per (token, 16 heads) and
+// sees the keys j <= i with i - j < window (0: all).  sinks [hl] or null.  nsplit: CTAs per (token, 16 heads) and
 // cluster, rounded down to 1, 2, 4 or 8; groups: clusters per (token, 16 heads).  With groups > 1 and u = T * ceil(hl / 16):
 // part_o of u * groups * 16 * lat floats, part_ml of u * groups * nsplit * 32, counters of u * nsplit zeros (left as zeros).
 extern "C" int xft_mla_attention_ext(const void* q_abs, long long qa_sh, long long qa_st, const void* q_rope, long long qr_sh,
                                      long long qr_st, void* out, long long o_sh, long long o_st, const void* cache,
                                      const int* block_table, int bt_stride, const int* cu_q, const int* kv_lens, int B, int T,
-                                     int hl, int lat, int bs, int num_blocks, float scale, int window, int nsplit,
-                                     int groups, float* part_o, float* part_ml, int* counters, int* status,
+                                     int hl, int lat, int bs, int num_blocks, float scale, const float* sinks, int window,
+                                     int nsplit, int groups, float* part_o, float* part_ml, int* counters, int* status,
                                      cudaStream_t st) {
   if (T <= 0 || B <= 0) return 0;
   if (bs <= 0 || bs % MKT) return -2;
   if (window < 0 || hl <= 0) return -1;
   MlaParams p{(const bf16*)q_abs, qa_sh, qa_st, (const bf16*)q_rope, qr_sh, qr_st, (bf16*)out, o_sh, o_st, block_table,
-              bt_stride, cu_q, kv_lens, B, T, hl, bs, num_blocks, scale, window > 0 ? min(window, 1 << 30) : 1 << 30,
+              bt_stride, cu_q, kv_lens, B, T, hl, bs, num_blocks, scale, sinks, window > 0 ? min(window, 1 << 30) : 1 << 30,
               nsplit >= 8 ? 8 : nsplit >= 4 ? 4 : nsplit >= 2 ? 2 : 1, groups < 1 ? 1 : groups, part_o, part_ml, counters, status};
   if (p.groups > 1 && (!part_o || !part_ml || !counters)) return -3;
   switch (lat) {
@@ -404,5 +410,5 @@ extern "C" int xft_mla_attention(const void* q_abs, long long qa_sh, long long q
                                  int hl, int bs, int num_blocks, float scale, int nsplit, float* /*part_o*/,
                                  float* /*part_ml*/, int* /*counters*/, int* status, cudaStream_t st) {
   return xft_mla_attention_ext(q_abs, qa_sh, qa_st, q_rope, qr_sh, qr_st, out, o_sh, o_st, cache, block_table, bt_stride, cu_q,
-                               kv_lens, B, T, hl, 512, bs, num_blocks, scale, 0, nsplit, 1, nullptr, nullptr, nullptr, status, st);
+                               kv_lens, B, T, hl, 512, bs, num_blocks, scale, nullptr, 0, nsplit, 1, nullptr, nullptr, nullptr, status, st);
 }

@@ -30,13 +30,17 @@ struct GemmF32 {
   // grouped form: blockIdx.y is a tile {group, first row, rows, -} of 64 rows; X row r comes from src[r] when given
   const int4* tiles; const int* num_tiles; const int* src; const float* row_w; int group_w_rows;
   const float* bias; const float* times; int ldt;             // [N] and [T, N], or null
+  float param;                                 // of the activation
 };
 
-__device__ __forceinline__ float act_f32(float x, int act) {
+__device__ __forceinline__ float act_f32(float x, int act, float param = 1.f) {
   if (act == 1) return fmaxf(x, 0.f);
   if (act == 2) return x / (1.f + expf(-x));
   if (act == 3) return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
   if (act == 4) { const float r = fmaxf(x, 0.f); return r * r; }
+  if (act == 5) return 0.5f * x * (1.f + erff(x * 0.70710678118654752f));
+  if (act == 7) return tanhf(x);
+  if (act == 8) return param * tanhf(x / param);
   return x;
 }
 
@@ -85,7 +89,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32 p) {
     for (int j = 0; j < 4; ++j) {
       const int r = ty * 4 + i, n = n0 + tx * 4 + j;
       if (r < rows && n < p.N) {
-        float v = act_f32(acc[i][j] + (p.bias ? p.bias[n] : 0.f), p.act);
+        float v = act_f32(acc[i][j] + (p.bias ? p.bias[n] : 0.f), p.act, p.param);
         if (p.times) v *= p.times[(size_t)(t0 + r) * p.ldt + n];
         if (p.row_w) v *= p.row_w[t0 + r];
         Y[(size_t)(t0 + r) * p.ldo + n] = v;
@@ -93,22 +97,25 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32 p) {
     }
 }
 
-__global__ void gated_act_f32_kernel(const float* __restrict__ gu, int ld, float* __restrict__ out, int T, int I, int act) {
+__global__ void gated_act_f32_kernel(const float* __restrict__ gu, int ld, float* __restrict__ out, int T, int I, int act, float limit) {
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= (size_t)T * I) return;
   const int t = (int)(i / I), c = (int)(i % I);
   const float g = gu[(size_t)t * ld + c], u = gu[(size_t)t * ld + I + c];
-  out[i] = act_f32(g, act) * u;
+  if (act == 6) {                                        // gate bounded above, the other on both sides
+    const float c = fminf(g, limit);
+    out[i] = c / (1.f + expf(-1.702f * c)) * (fminf(fmaxf(u, -limit), limit) + 1.f);
+  } else out[i] = act_f32(g, act) * u;
 }
 
-// out[t, c] = x[t, c] * sigmoid(gate[t, c])
+// out[t, c] = x[t, c] * sigmoid(gate[t, c / per])
 template <typename T>
 __global__ void sigmoid_gate_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ gate, int ldg, T* __restrict__ out,
-                                    int ldo, int n_tok, int n) {
+                                    int ldo, int n_tok, int n, int per) {
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= (size_t)n_tok * n) return;
   const int t = (int)(i / n), c = (int)(i % n);
-  const float g = to_f32<T>(gate[(size_t)t * ldg + c]);
+  const float g = to_f32<T>(gate[(size_t)t * ldg + c / per]);
   out[(size_t)t * ldo + c] = from_f32<T>(to_f32<T>(x[(size_t)t * ldx + c]) / (1.f + expf(-g)));
 }
 
@@ -237,15 +244,15 @@ __global__ void __launch_bounds__(128) attention_plain_kernel(const T* __restric
 
 using namespace xft;
 
-// act: 0 none, 1 relu, 2 silu, 3 gelu (tanh), 4 relu squared
+// act: 0 none, 1 relu, 2 silu, 3 gelu (tanh), 4 relu squared, 5 gelu (erf), 7 tanh, 8 param * tanh(. / param)
 extern "C" int xft_gemm_f32(const float* X, int ldx, const float* W, int ldw, float* Y, int ldo, int T, int N, int K, int act,
-                            const float* bias, const float* times, int ldt, cudaStream_t st) {
+                            const float* bias, const float* times, int ldt, float param, cudaStream_t st) {
   if (T <= 0 || N <= 0) return 0;
   if (K <= 0 || ldx < K || ldw < K || ldo < N || (times && ldt < N)) return -1;
   const int ty = (T + 63) / 64;
   if (ty > 65535) return -2;
   GemmF32 p{X, ldx, W, ldw, Y, ldo, T, N, K, act};
-  p.bias = bias; p.times = times; p.ldt = ldt;
+  p.bias = bias; p.times = times; p.ldt = ldt; p.param = param;
   gemm_f32_kernel<<<dim3((N + 63) / 64, ty), 256, 0, st>>>(p);
   return (int)cudaGetLastError();
 }
@@ -274,22 +281,24 @@ extern "C" int xft_gemm_f32_grouped(const float* X, int ldx, const float* W, int
   return (int)cudaGetLastError();
 }
 
-extern "C" int xft_sigmoid_gate(const void* x, int ldx, const void* gate, int ldg, void* out, int ldo, int T, int n, int f32,
+// per: columns that share a gate value
+extern "C" int xft_sigmoid_gate(const void* x, int ldx, const void* gate, int ldg, void* out, int ldo, int T, int n, int per, int f32,
                                 cudaStream_t st) {
   const size_t m = (size_t)T * n;
   if (!m) return 0;
-  if (ldx < n || ldg < n || ldo < n) return -1;
+  if (per < 1 || ldx < n || ldg < (n + per - 1) / per || ldo < n) return -1;
   const unsigned grid = (unsigned)((m + 255) / 256);
-  if (f32) sigmoid_gate_kernel<float><<<grid, 256, 0, st>>>((const float*)x, ldx, (const float*)gate, ldg, (float*)out, ldo, T, n);
-  else sigmoid_gate_kernel<bf16><<<grid, 256, 0, st>>>((const bf16*)x, ldx, (const bf16*)gate, ldg, (bf16*)out, ldo, T, n);
+  if (f32) sigmoid_gate_kernel<float><<<grid, 256, 0, st>>>((const float*)x, ldx, (const float*)gate, ldg, (float*)out, ldo, T, n, per);
+  else sigmoid_gate_kernel<bf16><<<grid, 256, 0, st>>>((const bf16*)x, ldx, (const bf16*)gate, ldg, (bf16*)out, ldo, T, n, per);
   return (int)cudaGetLastError();
 }
 
-extern "C" int xft_gated_act_f32(const float* gu, int ld, float* out, int T, int I, int act, cudaStream_t st) {
+// act 6: see ops.linear_gated ("clamped")
+extern "C" int xft_gated_act_f32(const float* gu, int ld, float* out, int T, int I, int act, float limit, cudaStream_t st) {
   const size_t n = (size_t)T * I;
   if (!n) return 0;
   if (ld < 2 * I) return -1;
-  gated_act_f32_kernel<<<(unsigned)((n + 255) / 256), 256, 0, st>>>(gu, ld, out, T, I, act);
+  gated_act_f32_kernel<<<(unsigned)((n + 255) / 256), 256, 0, st>>>(gu, ld, out, T, I, act, limit);
   return (int)cudaGetLastError();
 }
 

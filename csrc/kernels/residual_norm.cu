@@ -1,7 +1,8 @@
 // The residual stream kept in 32 bits, with everything that happens to it between two products in one launch:
 //
-//   x <- x + mult * post(y) + add   y = output of the sublayer just finished; post = a norm with its own gain, or nothing;
-//                                   add = a vector, the same for every row, or nothing
+//   x <- carry * x + mult * post(y) + add   y = output of the sublayer just finished; post = a norm with its own gain, or
+//                                   nothing; add = a vector, the same for every row, or nothing
+//   or x <- post(carry * x + mult * y + add), the norm of the sum being the stream
 //   h <- next(x)                    input of the sublayer that follows, for the next product (bf16 or fp32); next = a norm,
 //                                   or x as it is
 //
@@ -33,6 +34,7 @@ struct ResidualNormParams {
   float eps, embed_scale, mult;
   const float* add;                                                 // [H] or null
   int raw;                                                          // h is x itself
+  float carry; int post_sum;                                        // factor of x; the norm `post` is that of the sum
   int* status;
 };
 
@@ -164,8 +166,14 @@ __global__ void __launch_bounds__(NT) residual_norm_kernel(const ResidualNormPar
       else load8(reinterpret_cast<const bf16*>(p.y) + (size_t)src * p.ldy + (left > 0 ? i : 0), left, y[c]);
     }
   }
+  if (p.carry != 1.f) {
+#pragma unroll
+    for (int c = 0; c < CH; ++c)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) x[c][j] *= p.carry;
+  }
   if (p.y) {
-    if (p.post_w) norm_row<NT, CH, PRE>(y, p, p.post_w, p.post_b, g1, sh[0]);
+    if (p.post_w && !p.post_sum) norm_row<NT, CH, PRE>(y, p, p.post_w, p.post_b, g1, sh[0]);
 #pragma unroll
     for (int c = 0; c < CH; ++c)
 #pragma unroll
@@ -180,6 +188,7 @@ __global__ void __launch_bounds__(NT) residual_norm_kernel(const ResidualNormPar
       for (int j = 0; j < 8; ++j) x[c][j] += y[c][j];
     }
   }
+  if (p.post_sum) norm_row<NT, CH, PRE>(x, p, p.post_w, p.post_b, g1, sh[0]);
   if (p.x_out) {
 #pragma unroll
     for (int c = 0; c < CH; ++c) {
@@ -210,17 +219,17 @@ extern "C" int xft_residual_norm(const int* ids, const void* table, int vocab, l
                                  float* x_out, int ldxo, const void* y, int ldy, int y_f32, const float* post_w,
                                  const float* post_b, const float* next_w, const float* next_b, void* h, int ldh, int h_f32,
                                  const int* rows, int n_in, int n_out, int H, int kind, float eps, float embed_scale,
-                                 float mult, const float* add, int raw, int* status, cudaStream_t st) {
+                                 float mult, const float* add, int raw, float carry, int post_sum, int* status, cudaStream_t st) {
   if (n_out <= 0) return 0;
   const int HP = (H + 7) / 8 * 8;
-  if (H <= 0 || H > 32768 || (!ids && !x) || (h && !next_w && !raw) || (!rows && n_out > n_in)) return -1;
+  if (H <= 0 || H > 32768 || (!ids && !x) || (h && !next_w && !raw) || (post_sum && !post_w) || (!rows && n_out > n_in)) return -1;
   if ((ids && ((ldt & 7) || ldt < HP)) || (!ids && ((ldx & 7) || ldx < HP))) return -2;
   if ((x_out && ((ldxo & 7) || ldxo < HP)) || (y && ((ldy & 7) || ldy < HP)) || (h && ((ldh & 7) || ldh < HP))) return -2;
   if (((uintptr_t)table | (uintptr_t)x | (uintptr_t)x_out | (uintptr_t)y | (uintptr_t)post_w | (uintptr_t)post_b |
        (uintptr_t)next_w | (uintptr_t)next_b | (uintptr_t)h | (uintptr_t)add) & 15) return -3;
   if (rows && x_out == x && x_out) return -4;              // gathered rows cannot be written back in place
   ResidualNormParams p{ids, (const bf16*)table, vocab, ldt, x, ldx, x_out, ldxo, y, ldy, y_f32, post_w, post_b, next_w,
-                       next_b, h, ldh, h_f32, rows, n_in, H, HP, kind, eps, embed_scale, mult, add, raw, status};
+                       next_b, h, ldh, h_f32, rows, n_in, H, HP, kind, eps, embed_scale, mult, add, raw, carry, post_sum, status};
   cudaError_t e;
 #define XFT_RN(NT, CH, PRE) e = launch_pdl(residual_norm_kernel<NT, CH, PRE>, dim3(n_out), dim3(NT), 0, st, p)
   const bool few = n_out <= 296;                           // decode: a wide CTA per row, everything in one round of loads

@@ -18,7 +18,7 @@ import torch
 
 _LIB = None
 _ACT = {None: 0, "none": 0, "relu": 1, "silu": 2, "gelu": 3, "gelu_tanh": 3, "gelu_new": 3, "gelu_pytorch_tanh": 3,
-        "swiglu": 2, "relu2": 4}
+        "swiglu": 2, "relu2": 4, "gelu_erf": 5, "clamped": 6, "tanh": 7, "softcap": 8}
 _ACT.update({(a, "times"): c | 16 for a, c in list(_ACT.items())})       # the residual operand multiplies (kActTimes)
 
 STATUS_TEXT = {0: "ok", 1: "producer timed out waiting for a free stage", 2: "MMA warp timed out waiting for TMA data",
@@ -170,7 +170,7 @@ def layernorm(x, w, b, eps):
 
 
 def residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids=None, table=None, keep_x=True,
-                  embed_scale=1.0, mult=1.0, add=None, raw=False):
+                  embed_scale=1.0, mult=1.0, add=None, raw=False, carry=1.0, post_sum=False):
     """csrc/kernels/residual_norm.cu.  x fp32 [T, HP]; y bf16 or fp32 rows; gains fp32 [H]."""
     dev = (x if x is not None else table).device
     gain = nxt[0] if nxt is not None else post[0] if post is not None else None
@@ -201,23 +201,24 @@ def residual_norm(x, y, post, nxt, eps, kind, rows, h_dtype, ids=None, table=Non
               0 if ids is not None else x.stride(0), _p(x_out), 0 if x_out is None else x_out.stride(0), _p(y),
               0 if y is None else y.stride(0), int(y is not None and y.dtype == torch.float32), _p(pw), _p(pb), _p(nw), _p(nb),
               _p(h), HP, int(h_dtype == torch.float32), _p(rows32), n_in, n_out, H, 0 if kind == "layer" else 1,
-              C.c_float(eps), C.c_float(embed_scale), C.c_float(mult), _p(add), int(raw), _p(ws.status), _stream()), "residual_norm")
+              C.c_float(eps), C.c_float(embed_scale), C.c_float(mult), _p(add), int(raw), C.c_float(carry), int(post_sum), _p(ws.status), _stream()), "residual_norm")
     ws.launches += 1
     return x_out, h
 
 
-def gemm_f32(x, w, N, act=None, bias=None, times=None):
-    """Y[T,N] = act(X[T,K] W[N,K]^T + bias) * times[T,N], everything in 32 bits."""
+def gemm_f32(x, w, N, act=None, bias=None, times=None, param=1.0, out=None):
+    """Y[T,N] = act(X[T,K] W[N,K]^T + bias) * times[T,N], everything in 32 bits.  `param`: of the activation."""
     x2 = x.reshape(-1, x.shape[-1])
     if x2.stride(1) != 1:
         x2 = x2.contiguous()
     T, K = x2.shape
     assert x2.dtype == torch.float32 and w.dtype == torch.float32 and w.stride(1) == 1 and w.shape[1] == K
-    y = torch.empty(T, N, dtype=torch.float32, device=x.device)
+    y = torch.empty(T, N, dtype=torch.float32, device=x.device) if out is None else out
+    assert y.dtype == torch.float32 and y.stride(1) == 1
     fn = lib().xft_gemm_f32
     fn.restype = C.c_int
-    _check(fn(_p(x2), x2.stride(0) if T > 1 else max(x2.stride(0), K), _p(w), w.stride(0), _p(y), N, T, N, K, _ACT[act],
-              _p(bias), _p(times), 0 if times is None else times.stride(0), _stream()), "gemm_f32")
+    _check(fn(_p(x2), x2.stride(0) if T > 1 else max(x2.stride(0), K), _p(w), w.stride(0), _p(y), max(y.stride(0), N), T, N, K, _ACT[act],
+              _p(bias), _p(times), 0 if times is None else times.stride(0), C.c_float(param), _stream()), "gemm_f32")
     Workspace.get(x.device).launches += 1
     return y
 
@@ -259,8 +260,8 @@ def gemm_bf16(x, w, N, gated=False, dual_off=0, bias=None, act=None, residual=No
             and out.stride(1) == 1 and force_splits == 0:
         fn = lib().xft_gemm_bf16_prefill_tm_f32
         fn.restype = C.c_int
-        _check(fn(_p(x2), ldx, _p(w), w.shape[0], w.stride(0), _p(out), out.stride(0), T, N, K, _p(bias), _ACT[act], _p(ws.status),
-                  _stream()), "gemm_bf16_prefill_tm_f32")
+        _check(fn(_p(x2), ldx, _p(w), w.shape[0], w.stride(0), _p(out), out.stride(0), T, N, K, _p(bias), _ACT[act],
+                  C.c_float(res_scale), _p(ws.status), _stream()), "gemm_bf16_prefill_tm_f32")
         ws.launches += 1
         return out
     if _ENV().gemm_persistent and T > 128 and gated and not fp32 and row_scale is None and out.stride(1) == 1 \
@@ -413,11 +414,21 @@ def linear(x, W, bias=None, act=None, residual=None, res_scale=1.0, out_dtype=No
     elif W.kind == "fp32":
         if residual is not None or out_dtype not in (None, torch.float32):
             raise KernelError("fp32 products have no residual")
-        y = gemm_f32(x, W.w, W.out_features, act, bias)
+        y = gemm_f32(x, W.w, W.out_features, act, bias, param=res_scale)
     else:
         from . import native_quant
         y = native_quant.linear(x, W, bias, act, residual, res_scale, out_dtype)
     return y.view(*lead, W.out_features)
+
+
+def linear_into(x, W, bias, act, out):
+    """act(x W^T + bias) into the first columns of the rows `out`."""
+    assert x.dim() == 2 and out.shape[0] == x.shape[0] and out.shape[1] >= W.out_features and out.stride(1) == 1
+    if W.kind == "fp32":
+        return gemm_f32(x, W.w, W.out_features, act, bias, out=out)
+    if W.kind != "bf16" or out.dtype != torch.bfloat16:
+        raise KernelError(f"no product of {W.kind} weights into {out.dtype} rows")
+    return gemm_bf16(x, W.w, W.out_features, bias=bias, act=act, out=out)
 
 
 def linear_times(x, W, bias, act, times):
@@ -430,19 +441,17 @@ def linear_times(x, W, bias, act, times):
     return gemm_bf16(x, W.w, W.out_features, bias=bias, act=(act, "times"), residual=times)
 
 
-def linear_gated(x, W, act="silu", bias=None):
+def linear_gated(x, W, act="silu", bias=None, limit=0.0):
     lead = x.shape[:-1]
     I = W.out_features // 2
     if W.kind == "bf16":
-        y = gemm_bf16(x, W.w, I, gated=True, dual_off=I, bias=bias, act=act)
+        y = gemm_bf16(x, W.w, I, gated=True, dual_off=I, bias=bias, act=act, res_scale=limit if act == "clamped" else 1.0)
     elif W.kind == "fp32":
-        if bias is not None:
-            raise KernelError("fp32 products have no epilogue")
-        gu = gemm_f32(x, W.w, 2 * I)
+        gu = gemm_f32(x, W.w, 2 * I, bias=bias)
         y = torch.empty(gu.shape[0], I, dtype=torch.float32, device=x.device)
         fn = lib().xft_gated_act_f32
         fn.restype = C.c_int
-        _check(fn(_p(gu), 2 * I, _p(y), gu.shape[0], I, _ACT[act], _stream()), "gated_act_f32")
+        _check(fn(_p(gu), 2 * I, _p(y), gu.shape[0], I, _ACT[act], C.c_float(limit), _stream()), "gated_act_f32")
         Workspace.get(x.device).launches += 1
     else:
         from . import native_quant

@@ -46,7 +46,7 @@ def _stacked(w, name, make):
     return w.cache[name]
 
 
-def _heads(x, ldx, x_cols, xs, w, heads, n_out, k, out, ldo, ys, gate=None, ldg=0):
+def _heads(x, ldx, x_cols, xs, w, heads, n_out, k, out, ldo, ys, gate=None, ldg=0, head_gate=False):
     """One product per head (w [heads * n_out, k]) on column ranges of x and out."""
     ws = N.Workspace.get(w.device)
     T = out.shape[0]
@@ -55,7 +55,7 @@ def _heads(x, ldx, x_cols, xs, w, heads, n_out, k, out, ldo, ys, gate=None, ldg=
         rc = _fn("xft_gemm_f32_heads")(N._p(x), ldx, xs, N._p(w), N._p(out), ldo, ys, heads, T, n_out, k, N._stream())
     else:
         rc = _fn("xft_gemm_bf16_heads")(N._p(x), ldx, x_cols, xs, N._p(w), k, N._p(out), ldo, ys, heads, T, n_out, k, N._p(gate), ldg,
-                                        N._p(ws.status), N._stream())
+                                        int(head_gate), N._p(ws.status), N._stream())
     N._check(rc, "per-head product")
     ws.launches += 1
     return out
@@ -99,11 +99,11 @@ class _Spans:
             self.part = rows, seqs, cu_dev, kv, len(self.short), max(kv_lens[i] for i in self.short)
 
 
-def latent_attention(x, d, cache, block_table, cu_q, kv_lens, weights, scale, window=0, meta=None):
+def latent_attention(x, d, cache, block_table, cu_q, kv_lens, weights, scale, window=0, meta=None, sinks=None):
     cu_dev, kv_dev, B, decode, max_kv = N.batch_arrays(cu_q, kv_lens, meta, x.device)
     out = torch.empty(x.shape[0], d.heads * d.vdim, dtype=x.dtype, device=x.device)
     if decode or x.dtype == torch.float32 or not can_expand(d, scale):
-        return _absorbed(x, d, cache, block_table, cu_dev, kv_dev, B, max_kv, weights, scale, window, out)
+        return _absorbed(x, d, cache, block_table, cu_dev, kv_dev, B, max_kv, weights, scale, window, sinks, out)
     least = N._ENV().latent_expand_min_q
     kept = meta.meta if meta is not None else {}
     key = ("latent spans", window, least)
@@ -111,18 +111,18 @@ def latent_attention(x, d, cache, block_table, cu_q, kv_lens, weights, scale, wi
     if sp is None:
         sp = kept[key] = _Spans(cu_q, kv_lens, window, least, x.device)
     if not sp.long:
-        return _absorbed(x, d, cache, block_table, cu_dev, kv_dev, B, max_kv, weights, scale, window, out)
-    _expanded(x, d, cache, block_table, sp, weights, scale, window, out)
+        return _absorbed(x, d, cache, block_table, cu_dev, kv_dev, B, max_kv, weights, scale, window, sinks, out)
+    _expanded(x, d, cache, block_table, sp, weights, scale, window, sinks, out)
     if sp.part is not None:
         rows, seqs, cu, kv, n, longest = sp.part
         xs = x.index_select(0, rows)
         a = torch.empty(xs.shape[0], d.heads * d.vdim, dtype=x.dtype, device=x.device)
         out.index_copy_(0, rows.long(), _absorbed(xs, d, cache, block_table.index_select(0, seqs), cu, kv, n, longest, weights, scale,
-                                                  window, a))
+                                                  window, sinks, a))
     return out
 
 
-def _expanded(x, d, cache, block_table, sp, weights, scale, window, out):
+def _expanded(x, d, cache, block_table, sp, weights, scale, window, sinks, out):
     """Prompt portions `sp.long` of the rows x into `out`."""
     ws, H, W = N.Workspace.get(x.device), d.heads, d.rank + d.rot
     nb, _, bs, _ = cache.shape
@@ -140,10 +140,10 @@ def _expanded(x, d, cache, block_table, sp, weights, scale, window, out):
             kv = torch.empty(sp.rows, n * (d.dim + d.vdim), dtype=x.dtype, device=x.device)
             N.gemm_bf16(flat[:, :d.rank], w[h0 * d.dim:(h0 + n) * d.dim], n * d.dim, out=kv[:, :n * d.dim])
             N.gemm_bf16(flat[:, :d.rank], w[H * d.dim + h0 * d.vdim:H * d.dim + (h0 + n) * d.vdim], n * d.vdim, out=kv[:, n * d.dim:])
-        flat_attention(x, d, kv, flat, sp, h0, n, scale, window, out)
+        flat_attention(x, d, kv, flat, sp, h0, n, scale, window, out, sinks)
 
 
-def flat_attention(x, d, kv, flat, sp, h0, n, scale, window, out):
+def flat_attention(x, d, kv, flat, sp, h0, n, scale, window, out, sinks=None):
     """Heads h0 .. h0 + n - 1 of the packed rows x over expanded keys and values `kv` [rows, n * (dim + vdim)] and the gathered
     cache rows `flat`, which hold the shared key part (csrc/kernels/latent_prefill_sm100.cu)."""
     ws = N.Workspace.get(x.device)
@@ -151,8 +151,8 @@ def flat_attention(x, d, kv, flat, sp, h0, n, scale, window, out):
     gate = x[:, d.gate_at:] if d.gate else None
     N._check(_fn("xft_attn_flat_tc")(
         N._p(x), ldx, d.q_width, d.dim + d.rot, N._p(kv), kv.shape[1], n * d.dim, N._p(flat), flat.shape[1], d.rank, sp.rows,
-        N._p(out), out.stride(0), N._p(gate), ldx if d.gate else 0, N._p(sp.q_start), N._p(sp.q_len), N._p(sp.kv_len), N._p(sp.lo),
-        N._p(sp.row), len(sp.long), x.shape[0], sp.max_q, h0, n, d.dim // 64, d.rot // 64, d.vdim // 64, C.c_float(scale), window,
+        N._p(out), out.stride(0), N._p(gate), ldx if d.gate else 0, int(d.head_gate), N._p(sp.q_start), N._p(sp.q_len), N._p(sp.kv_len), N._p(sp.lo),
+        N._p(sp.row), len(sp.long), x.shape[0], sp.max_q, h0, n, d.dim // 64, d.rot // 64, d.vdim // 64, C.c_float(scale), N._p(sinks), window,
         N._p(ws.status), N._stream()), "attn_flat_tc")
     ws.launches += 1
 
@@ -181,7 +181,7 @@ def mla_scratch(ws, units: int, n: int, g: int, rank: int) -> tuple:
     return (*ws.attn_partials(units * g * 16 * rank, units * g * n * 32), ws.attn_counters)
 
 
-def _absorbed(x, d, cache, block_table, cu_dev, kv_dev, B, max_kv, weights, scale, window, out):
+def _absorbed(x, d, cache, block_table, cu_dev, kv_dev, B, max_kv, weights, scale, window, sinks, out):
     T, ldx, H, hd = x.shape[0], max(x.stride(0), x.shape[1]), d.heads, d.dim + d.rot
     exact = x.dtype == torch.float32
     wk = _stacked(weights, "uk", lambda: weights.uk.transpose(1, 2).reshape(H * d.rank, d.dim))       # [H * rank, dim]
@@ -192,13 +192,13 @@ def _absorbed(x, d, cache, block_table, cu_dev, kv_dev, B, max_kv, weights, scal
         q = new(T, H, d.rank + d.rot)
         _heads(x, ldx, d.q_width, hd, wk, H, d.rank, d.dim, q, H * (d.rank + d.rot), d.rank + d.rot)
         q[:, :, d.rank:] = x[:, :d.q_width].view(T, H, hd)[:, :, d.dim:]
-        o = N.attention_plain(q, cache, cache, d.rank, block_table, cu_dev, kv_dev, B, scale, H, window=window)
+        o = N.attention_plain(q, cache, cache, d.rank, block_table, cu_dev, kv_dev, B, scale, H, window=window, sinks=sinks)
         if not exact:
-            return _heads(o, H * d.rank, H * d.rank, d.rank, wv, H, d.vdim, d.rank, out, H * d.vdim, d.vdim, gate, ldx)
+            return _heads(o, H * d.rank, H * d.rank, d.rank, wv, H, d.vdim, d.rank, out, H * d.vdim, d.vdim, gate, ldx, d.head_gate)
         _heads(o, H * d.rank, H * d.rank, d.rank, wv, H, d.vdim, d.rank, out, H * d.vdim, d.vdim)
         if d.gate:
-            N._check(_fn("xft_sigmoid_gate")(N._p(out), H * d.vdim, N._p(gate), ldx, N._p(out), H * d.vdim, T, H * d.vdim, 1,
-                                             N._stream()), "sigmoid_gate")
+            N._check(_fn("xft_sigmoid_gate")(N._p(out), H * d.vdim, N._p(gate), ldx, N._p(out), H * d.vdim, T, H * d.vdim,
+                                             d.vdim if d.head_gate else 1, 1, N._stream()), "sigmoid_gate")
             N.Workspace.get(x.device).launches += 1
         return out
     ws = N.Workspace.get(x.device)
@@ -212,7 +212,7 @@ def _absorbed(x, d, cache, block_table, cu_dev, kv_dev, B, max_kv, weights, scal
     qr = x[:, d.dim:]
     N._check(_fn("xft_mla_attention_ext")(
         N._p(qa), LL(d.rank), LL(H * d.rank), N._p(qr), LL(hd), LL(ldx), N._p(ol), LL(d.rank), LL(H * d.rank), N._p(cache),
-        N._p(block_table), block_table.stride(0), N._p(cu_dev), N._p(kv_dev), B, T, H, d.rank, bs, nb, C.c_float(scale), window,
+        N._p(block_table), block_table.stride(0), N._p(cu_dev), N._p(kv_dev), B, T, H, d.rank, bs, nb, C.c_float(scale), N._p(sinks), window,
         nsplit, groups, N._p(po), N._p(pm), N._p(cnt), N._p(ws.status), N._stream()), "mla_attention")
     ws.launches += 1
-    return _heads(ol, H * d.rank, H * d.rank, d.rank, wv, H, d.vdim, d.rank, out, H * d.vdim, d.vdim, gate, ldx)
+    return _heads(ol, H * d.rank, H * d.rank, d.rank, wv, H, d.vdim, d.rank, out, H * d.vdim, d.vdim, gate, ldx, d.head_gate)

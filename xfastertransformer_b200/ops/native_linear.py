@@ -1,5 +1,5 @@
-"""Recurrent mechanisms on the GPU: the heads of attention whose values are its keys (csrc/kernels/head_prep.cu), and gated
-linear attention (csrc/kernels/gla.cu).
+"""Recurrent mechanisms on the GPU: the heads of attention whose values are its keys (csrc/kernels/head_prep.cu), gated linear
+attention and time mixing (csrc/kernels/gla.cu), and state-space layers (gla.cu and csrc/kernels/ssd.cu).
 
 Gated linear attention has two kernels.  Portions of at least XFT_GLA_CHUNK_MIN_Q tokens go through the tensor cores in chunks
 of 64; shorter ones, decode steps, the 32-bit path and sizes without a chunk instance go token by token.  A batch may hold
@@ -62,17 +62,22 @@ def segments(units: int, longest: int) -> int:
     return n if n > 1 else 1
 
 
-def gated_linear(x, d, w, eps, state, state_slots, cu_q, kv_lens, meta=None):
+def gated_linear(x, d, w, eps, state, state_slots, cu_q, kv_lens, meta=None, out=None):
     cu, lens, B, decode, _ = N.batch_arrays(cu_q, kv_lens, meta, x.device)
     assert x.dim() == 2 and x.stride(1) == 1 and state.dtype == torch.float32 and state.is_contiguous()
     assert tuple(state.shape[1:]) == (d.heads, d.dim, d.vdim) and w.a2.dtype == x.dtype and w.a2.is_contiguous()
     T, exact = x.shape[0], x.dtype == torch.float32
     width = d.up(d.heads * d.vdim)                       # the rows of the product that follows
-    out = (torch.empty if width == d.heads * d.vdim else torch.zeros)(T, width, dtype=x.dtype, device=x.device)
+    whole = width == d.heads * d.vdim
+    if out is None:
+        out = (torch.empty if whole else torch.zeros)(T, width, dtype=x.dtype, device=x.device)
+    elif not whole:
+        out[:, d.heads * d.vdim:width].zero_()
     ws = N.Workspace.get(x.device)
     f = C.c_float
     common = (N._p(x), max(x.stride(0), x.shape[1]), d.k_at, d.v_at, d.g_at, d.a_at, d.heads, d.dim, d.vdim, d.rank, w.a2.shape[1],
-              N._p(w.a2), N._p(w.bias), f(w.tau), f(d.dim ** -0.5), f(eps), N._p(w.norm), N._p(state), N._p(state_slots),
+              N._p(w.a2), N._p(w.bias), f(w.tau), f(d.dim ** -0.5 if w.scale is None else w.scale),
+              f(eps), N._p(w.bonus), 0 if w.norm.numel() == d.vdim else d.vdim, f(w.mult), N._p(w.norm), N._p(state), N._p(state_slots),
               state.shape[0], N._p(cu), N._p(lens), B)
     columns = 0 if decode or exact else _fn("xft_gla_chunk_columns")(d.dim, d.vdim, d.rank)
     least = NO_LIMIT
@@ -92,5 +97,89 @@ def gated_linear(x, d, w, eps, state, state_slots, cu_q, kv_lens, meta=None):
             return out
     N._check(_fn("xft_gla_step")(*common, N._p(out), out.stride(0), 1, least, step_columns(B * d.heads, d.dim, d.vdim), int(exact),
                                  N._p(ws.status), N._stream()), "gla_step")
+    ws.launches += 1
+    return out
+
+
+def token_shift(x, mu, state, state_slots, cu_q, kv_lens, dtype, meta=None):
+    cu, lens, B, _, _ = N.batch_arrays(cu_q, kv_lens, meta, x.device)
+    n, W = mu.shape
+    assert x.dtype == torch.float32 and x.shape[1] == W and x.stride(1) == 1 and tuple(state.shape[1:]) == (W,)
+    T = x.shape[0]
+    out = torch.empty(T, n * W, dtype=dtype, device=x.device)
+    ws = N.Workspace.get(x.device)
+    N._check(_fn("xft_token_shift")(N._p(x), max(x.stride(0), W), T, n, W, N._p(mu), N._p(cu), N._p(lens), B, N._p(state), N._p(state_slots),
+                                    state.shape[0], N._p(out), int(dtype == torch.float32), N._p(ws.status), N._stream()), "token_shift")
+    ws.launches += 1
+    return out
+
+
+def linear_parts(x, W, n, out):
+    k, m, T = x.shape[1] // n, W.out_features // n, x.shape[0]
+    ldx, ldo = max(x.stride(0), x.shape[1]), max(out.stride(0), out.shape[1])
+    ws = N.Workspace.get(x.device)
+    assert W.in_features == k and x.dtype == out.dtype and x.stride(1) == out.stride(1) == 1
+    if W.kind == "fp32":
+        rc = _fn("xft_gemm_f32_heads")(N._p(x), ldx, k, N._p(W.w), N._p(out), ldo, m, n, T, m, k, N._stream())
+    elif W.kind != "bf16":
+        raise N.KernelError(f"no products side by side for {W.kind} weights")
+    elif T > 128:                                        # prompt sizes: the token-major kernel, part by part
+        for i in range(n):
+            N.gemm_bf16(x[:, i * k:(i + 1) * k], W.w[i * m:(i + 1) * m], m, out=out[:, i * m:(i + 1) * m])
+        return out
+    else:
+        rc = _fn("xft_gemm_bf16_heads")(N._p(x), ldx, x.shape[1], k, N._p(W.w), k, N._p(out), ldo, m, n, T, m, k, N._p(None), 0, 0,
+                                        N._p(ws.status), N._stream())
+    N._check(rc, "products side by side")
+    ws.launches += 1
+    return out
+
+
+def ssd_columns(units: int, state: int, vdim: int) -> int:
+    """As `step_columns`, for a kernel whose CTAs of a head need not meet."""
+    fits = [c for c in (128, 64, 32) if state <= 32 * 1024 // c]
+    if not fits:
+        raise N.KernelError(f"state space: no kernel for states of {state} x {vdim}")
+    best = fits[0]
+    for c in fits[1:]:
+        if units * ((vdim + best - 1) // best) < 2 * SMS or best >= 2 * vdim or state * best > 16 * 1024:
+            best = c
+    return best
+
+
+def state_space(x, d, w, eps, state, conv_state, state_slots, cu_q, kv_lens, meta=None):
+    cu, lens, B, decode, _ = N.batch_arrays(cu_q, kv_lens, meta, x.device)
+    assert x.dim() == 2 and x.stride(1) == 1 and state.dtype == torch.float32 and state.is_contiguous()
+    assert tuple(state.shape[1:]) == (d.heads, d.state, d.vdim)
+    assert d.taps == 1 or conv_state.dtype == x.dtype and tuple(conv_state.shape[1:]) == (d.taps - 1, d.channels)
+    T, exact, dev = x.shape[0], x.dtype == torch.float32, x.device
+    ldx, slots, ns = max(x.stride(0), x.shape[1]), N._p(state_slots), state.shape[0]
+    ws = N.Workspace.get(dev)
+    f32 = int(exact)
+    u = torch.empty(T, d.up(d.channels), dtype=x.dtype, device=dev)
+    N._check(_fn("xft_channel_conv")(N._p(x[:, d.x_at:]), ldx, T, B, d.channels, d.taps, N._p(w.conv), N._p(w.conv_bias), N._p(cu), N._p(lens),
+                                     N._p(conv_state), slots, ns, N._p(u), u.shape[1], int(decode), f32, N._p(ws.status), N._stream()),
+             f"channel_conv ({d.taps} taps)")
+    ws.launches += 1 if decode or d.taps == 1 else 2
+    y = torch.empty(T, d.inner, dtype=torch.float32, device=dev)
+    b_at, c_at, per = d.inner, d.inner + d.groups * d.state, d.heads // d.groups
+    dt, vectors = x[:, d.dt_at:], (N._p(w.dt_bias), N._p(w.rate), N._p(w.skip))
+    least = NO_LIMIT
+    if not decode and not exact and _fn("xft_ssd_has_chunk")(d.state):
+        least = max(1, N._ENV().ssd_chunk_min_q)
+        sizes = [cu_q[i + 1] - cu_q[i] for i in range(B)]
+        if max(sizes) >= least:
+            N._check(_fn("xft_ssd_chunk")(N._p(u), u.shape[1], b_at, c_at, N._p(dt), ldx, *vectors, d.heads, per, d.state, d.vdim, N._p(state),
+                                          slots, ns, N._p(cu), N._p(lens), B, N._p(y), least, N._p(ws.status), N._stream()), "ssd_chunk")
+            ws.launches += 1
+    if least == NO_LIMIT or min(sizes) < least:
+        N._check(_fn("xft_ssd_step")(N._p(u), u.shape[1], c_at, b_at, 0, d.heads, per, d.state, d.vdim, N._p(dt), ldx, *vectors, N._p(state),
+                                     slots, ns, N._p(cu), N._p(lens), B, N._p(y), 1, least, ssd_columns(B * d.heads, d.state, d.vdim), f32,
+                                     N._p(ws.status), N._stream()), "ssd_step")
+        ws.launches += 1
+    width = d.up(d.inner)
+    out = (torch.empty if width == d.inner else torch.zeros)(T, width, dtype=x.dtype, device=dev)
+    N._check(_fn("xft_gated_norm")(N._p(y), d.inner, N._p(x), ldx, N._p(w.norm), N._p(out), width, T, d.norm_groups, d.inner // d.norm_groups,
+                                   C.c_float(eps), f32, N._stream()), "gated_norm")
     ws.launches += 1
     return out

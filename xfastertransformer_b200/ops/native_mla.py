@@ -85,7 +85,7 @@ def mla_attention(q_nope, q_rope, latent_cache, block_table, cu_q, kv_lens, w_uk
     LL = C.c_longlong
     rc = _lib().xft_mla_attention_ext(N._p(q_abs), LL(T * L), LL(L), N._p(q_rope), LL(rope), LL(Hl * rope), N._p(o_lat), LL(T * L),
                                       LL(L), N._p(latent_cache), N._p(block_table), block_table.stride(0), N._p(cu_dev),
-                                      N._p(kv_dev), B, T, Hl, L, bs, nb, C.c_float(scale), 0, nsplit, groups, N._p(po), N._p(pm),
+                                      N._p(kv_dev), B, T, Hl, L, bs, nb, C.c_float(scale), N._p(None), 0, nsplit, groups, N._p(po), N._p(pm),
                                       N._p(cnt), N._p(ws.status), N._stream())
     N._check(rc, "mla_attention")
     ws.launches += 1

@@ -121,7 +121,7 @@ def _experts_f32(x, idx32, w, pk, act, expert_offset, gated, add):
     if gated:
         gu, h1 = h1, f32(n, I)
         lib.xft_gated_act_f32.restype = C.c_int
-        N._check(lib.xft_gated_act_f32(N._p(gu), up, N._p(h1), n, I, N._ACT[act], N._stream()), "gated_act_f32")
+        N._check(lib.xft_gated_act_f32(N._p(gu), up, N._p(h1), n, I, N._ACT[act], C.c_float(0.0), N._stream()), "gated_act_f32")
         ws.launches += 1
     N._check(fn(N._p(h1), I, N._p(pk["dn"]), I, N._p(ys), H, H, I, H, N._p(tiles), N._p(meta), tiles_n, N._p(None), N._p(row_w), 0,
                 N._stream()), "grouped fp32 down")
