@@ -112,6 +112,36 @@ CONFIGS.update({
         O.gla_layer(heads=2, dim=24, vdim=40, tau=0.2), O.gla_layer(heads=2, dim=72, vdim=80, tau=1.5, mlp=O.dense(40)),
         O.shared_kv_layer(heads=2, kv_heads=1, dim=36, size=9, rot_dims=20, conv=5)], width=88, vocab=120, mult=0.5, loop=(0, 1, 2)),
 })
+CONFIGS.update({
+    # Dagezen: all mixers, unequal sizes, a layer without feed-forward, widths off the 16-byte rows
+    "mixed_heads": O.dagezen([
+        O.mamba_layer(heads=6, vdim=12, state=20, groups=3, norm_groups=2, conv=3, mlp=O.chosen_moe(ff=36, experts=7, top=3)),
+        O.sink_latent_layer(heads=3, dim=24, rot_dim=12, vdim=20, kv_rank=28, base=900.0, mlp=O.clamped(70, 0.8)),
+        O.parallel_layer(heads=6, kv_heads=3, dim=20, size=17, right_heads=2, right_dim=24, scales=(0.5, 1.7)),
+        O.parallel_layer(heads=4, kv_heads=1, dim=36, size=70, right_heads=3, right_dim=12, mlp=O.chosen_moe(ff=20, experts=5, top=1))],
+        width=90, vocab=131, eps=3e-4, alpha=1.6, cap=11.0),
+    # sizes of the kernels without padding; several chunks, a window off the 64-token pages, 16 heads
+    "mixed_heads128": O.dagezen([
+        O.parallel_layer(heads=16, kv_heads=4, dim=128, size=100, right_heads=2, right_dim=128, mlp=O.clamped(64, 2.0)),
+        O.mamba_layer(heads=4, vdim=64, state=128, groups=1, norm_groups=1, conv=4, mlp=O.clamped(128, 1.2)),
+        O.sink_latent_layer(heads=18, dim=128, rot_dim=64, vdim=128, kv_rank=128, mlp=O.chosen_moe(ff=64, experts=6, top=2)),
+        O.parallel_layer(heads=8, kv_heads=8, dim=64, size=65, right_heads=3, right_dim=64)], width=160, vocab=300),
+    # mechanisms at their least: one head, one group, one tap, one expert, no cap, factors of one, a window of one, one past the end
+    "mixed_heads_bare": O.dagezen([
+        O.parallel_layer(heads=1, kv_heads=1, dim=16, size=1, right_heads=1, right_dim=8, scales=(1.0, 1.0), mlp=O.chosen_moe(ff=8, experts=1, top=1)),
+        O.mamba_layer(heads=2, vdim=8, state=8, groups=1, norm_groups=1, conv=1),
+        O.sink_latent_layer(heads=1, dim=16, rot_dim=2, vdim=8, kv_rank=12, scale=0.11, mlp=O.chosen_moe(ff=16, experts=4, top=4)),
+        O.parallel_layer(heads=3, kv_heads=3, dim=64, size=5000, right_heads=1, right_dim=64, mlp=O.clamped(40, 100.0))],
+        width=72, vocab=150, alpha=1.0, cap=None),
+    # larger than the tensor-core kernels take, many heads, many taps, norm parts that cut through heads
+    "mixed_heads_large": O.dagezen([
+        O.parallel_layer(heads=2, kv_heads=1, dim=264, size=30, right_heads=1, right_dim=200, mlp=O.clamped(72)),
+        O.mamba_layer(heads=5, vdim=136, state=264, groups=5, norm_groups=4, conv=7),
+        O.sink_latent_layer(heads=2, dim=208, rot_dim=80, vdim=144, kv_rank=520, mlp=O.clamped(24)),
+        O.parallel_layer(heads=24, kv_heads=2, dim=24, size=66, right_heads=2, right_dim=300),
+        O.mamba_layer(heads=3, vdim=72, state=130, groups=1, norm_groups=3, conv=2)], width=104, vocab=83, alpha=3.0),
+})
+MIXED_HEADS = ["mixed_heads", "mixed_heads128", "mixed_heads_bare", "mixed_heads_large"]
 RECURRENT = [n for n in sorted(CONFIGS) if n.startswith("recurrent")]
 LATENT = ["latent", "latent128", "latent_bare", "latent_large"]
 

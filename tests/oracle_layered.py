@@ -662,9 +662,43 @@ def dense(ff=48):
     return {"kind": "dense", "ff": ff}
 
 
+def mamba_layer(heads=4, vdim=16, state=24, groups=2, norm_groups=2, conv=4, mlp=None):
+    return {"type": "mamba2", "mlp": mlp, "mixer": {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "norm_groups": norm_groups,
+                                                    "conv": conv}}
+
+
+def sink_latent_layer(heads=4, dim=32, rot_dim=16, vdim=24, kv_rank=40, base=10000.0, scale=None, mlp=None):
+    m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank,
+         "scale": scale if scale else (dim + rot_dim) ** -0.5, "rot": {"dims": rot_dim, "base": base}}
+    return {"type": "latent_attention", "mixer": m, "mlp": mlp}
+
+
+def parallel_layer(heads=4, kv_heads=2, dim=32, size=24, scale=None, right_heads=3, right_dim=16, scales=(0.7, 1.3), mlp=None):
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": scale if scale else dim ** -0.5, "mask": {"size": size}}
+    return {"type": "parallel", "mlp": mlp, "mixer": {"left": left, "right": {"heads": right_heads, "dim": right_dim},
+                                                      "left_scale": scales[0], "right_scale": scales[1]}}
+
+
+def clamped(ff=48, limit=1.5):
+    return {"kind": "dense", "ff": ff, "limit": limit}
+
+
+def chosen_moe(ff=40, experts=6, top=2):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+
+
+def dagezen(layers, width=96, vocab=210, eps=1e-5, alpha=2.0, cap=20.0):
+    cfg = {"architecture": "Dagezen", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width, "postln_alpha": alpha}
+    if cap:
+        cfg["logit_softcap"] = cap
+    return cfg
+
+
 def random_weights(cfg, seed=0, gain=1.0):
     if cfg["architecture"] == "Botusun":
         return _botusun_weights(cfg, seed)
+    if cfg["architecture"] == "Dagezen":
+        return _dagezen_weights(cfg, seed)
     return _weights(cfg, seed, gain)
 
 
@@ -741,6 +775,82 @@ def _botusun_weights(cfg, seed):
     for n, t in W.items():
         if n.endswith((".mix.o", ".down", ".side.proj")):
             t[:used] = 0
+    return W
+
+
+def _dagezen_weights(cfg, seed):
+    """As `_weights`.  The norms keep the code's order (gain one, no bias there); router biases are a part of its steps, so that
+    they change the weights and no choice."""
+    g = torch.Generator().manual_seed(seed)
+    D, V = cfg["width"], cfg["vocab"]
+
+    def mat(o, i, s=1.0):
+        return (torch.randn(o, i, generator=g) * (s / math.sqrt(i))).bfloat16()
+
+    def vec(n, around=0.0, s=0.2):
+        return (around + s * torch.randn(n, generator=g)).bfloat16()
+    E = max([l["mlp"]["router"]["experts"] for l in cfg["layers"] if (l.get("mlp") or {}).get("kind") == "moe"], default=0)
+    W = {"embed": torch.randn(V, D, generator=g).bfloat16()}
+    if E:
+        levels = (torch.arange(E) - (E - 1) / 2) * (4.0 / E)
+        W["embed"][:, :E] = torch.stack([levels[torch.randperm(E, generator=g)] for _ in range(V)]).bfloat16()
+
+    def norm(name):
+        W[name], W[name + ".b"] = vec(D, 1.0), vec(D, 0.0, 0.3)
+        if not name.startswith("final"):
+            W[name][:E], W[name + ".b"][:E] = 1.0, 0.0
+    norm("final.norm")
+    for i, layer in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}", layer["mixer"], layer.get("mlp")
+        P = p + ".mix."
+        norm(p + ".norm1")
+        if layer["type"] == "mamba2":
+            H, n = m["heads"], m["heads"] * m["vdim"]
+            c = n + 2 * m["groups"] * m["state"]
+            W[P + "in"] = mat(n + c + H, D, 1.3)
+            W[P + "conv"], W[P + "conv.b"] = vec(c * m["conv"], 0.4, 0.5).view(c, m["conv"]), vec(c, 0.2, 0.3)
+            W[P + "dt_bias"], W[P + "A_log"], W[P + "D"], W[P + "norm"] = vec(H, -1.5, 1.5), vec(H, 0.0, 1.2), vec(H, 1.0, 0.5), vec(n, 1.0)
+            W[P + "o"] = mat(D, n, 1.5)
+        elif layer["type"] == "latent_attention":
+            H = m["heads"]
+            W[P + "q"] = mat(H * (m["dim"] + m["rot_dim"]), D, 1.6)
+            W[P + "dkv"], W[P + "dkv.norm"] = mat(m["kv_rank"] + m["rot_dim"], D, 1.3), vec(m["kv_rank"], 1.0)
+            W[P + "uk"], W[P + "uv"] = mat(H * m["dim"], m["kv_rank"], 1.6), mat(H * m["vdim"], m["kv_rank"])
+            W[P + "sink"], W[P + "g"], W[P + "o"] = vec(H, 1.0, 1.0), mat(H, D, 2.0), mat(D, H * m["vdim"], 2.0)
+        else:
+            l, r = m["left"], m["right"]
+            H, d = l["heads"], l["dim"]
+            L = P + "left."
+            W[L + "q"], W[L + "k"], W[L + "g"] = mat(H * d, D), mat(l["kv_heads"] * d, D), mat(H * d, D, 2.0)
+            W[L + "q.norm"], W[L + "k.norm"] = vec(H * d, 1.5), vec(l["kv_heads"] * d, 1.5)
+            W[L + "r1"], W[L + "r2"] = vec(H, 1.0, 0.5).abs(), vec(H, 0.3, 0.2).abs()
+            W[L + "talk"] = (0.8 * torch.eye(H) + 0.4 * torch.randn(H, H, generator=g) / math.sqrt(H)).bfloat16()
+            W[L + "o"] = mat(D, H * d, 2.0)
+            R, H, d, rank = P + "right.", r["heads"], r["dim"], (5, 16, 24, 33)[i % 4] if r["dim"] <= 128 else 9
+            for x in "rkvgw":
+                W[R + "mu." + x] = vec(D, 0.5, 0.2) if x != "k" else (W[R + "mu.r"].float() + 0.05 * torch.randn(D, generator=g)).bfloat16()
+            W[R + "r"], W[R + "v"], W[R + "g"] = mat(H * d, D, 1.5), mat(H * d, D), mat(H * d, D, 2.0)
+            # keys akin to their queries: an output of nothing but rounding would be blown up by the norm behind it
+            W[R + "k"] = (W[R + "r"].float() + 0.7 * mat(H * d, D).float()).bfloat16()
+            W[R + "w1"], W[R + "w2"], W[R + "w0"] = mat(rank, D), mat(H * d, rank, 1.5), vec(H * d, -1.5, 1.5)
+            W[R + "u"], W[R + "norm"], W[R + "o"] = vec(H * d, 1.0, 0.3).abs().view(H, d), vec(H * d, 1.0), mat(D, H * d, 1.5)
+        if not f:
+            continue
+        norm(p + ".norm2")
+        if f["kind"] == "moe":
+            n = f["router"]["experts"]
+            r = 0.001 * torch.randn(n, D, generator=g)
+            r[:, :E] = 2.0 * torch.eye(E)[torch.randperm(E, generator=g)[:n]]
+            W[p + ".mlp.router"] = r.bfloat16()
+            W[p + ".mlp.router.b"] = (0.15 * (4.0 / E) * torch.randn(n, generator=g).clamp(-2, 2)).bfloat16()
+            for e in range(n):
+                W[p + f".mlp.e{e}.up"], W[p + f".mlp.e{e}.down"] = mat(f["expert"]["ff"], D, 1.5), mat(D, f["expert"]["ff"], 1.5)
+        else:
+            for x, (o, k) in dict(gate=(f["ff"], D), up=(f["ff"], D), down=(D, f["ff"])).items():
+                W[p + f".mlp.{x}"], W[p + f".mlp.{x}.b"] = mat(o, k, 1.5), vec(o, 0.0, 0.3)
+    for n, t in W.items():
+        if n.endswith((".o", ".down", ".down.b")):
+            t[:E] = 0
     return W
 
 

@@ -1,4 +1,4 @@
-"""Layered designs (Kafipel, Vepivik, Botusun) on the CPU path: the engine, cache, batching and command-line tool against a plain
+"""Layered designs (Kafipel, Vepivik, Botusun, Dagezen) on the CPU path: the engine, cache, batching and command-line tool against a plain
 implementation of the equations."""
 import os
 import subprocess
@@ -38,44 +38,45 @@ def test_whole_prompt(cases, name):
     C.whole_prompt(cases(name), "fp32", 75)
 
 
-@pytest.mark.parametrize("name", ["unequal", "bare", "latent", "latent_bare", "recurrent", "recurrent_bare"])
+@pytest.mark.parametrize("name", ["unequal", "bare", "latent", "latent_bare", "recurrent", "recurrent_bare", "mixed_heads", "mixed_heads_bare"])
 def test_first_tokens(cases, name):
     C.first_tokens(cases(name), "fp32")
 
 
-@pytest.mark.parametrize("name,n,start", [("unequal", 75, 1), ("shared", 75, 60), ("latent", 75, 1), ("recurrent", 75, 1), ("recurrent_bare", 75, 30)])
+@pytest.mark.parametrize("name,n,start", [("unequal", 75, 1), ("shared", 75, 60), ("latent", 75, 1), ("recurrent", 75, 1), ("recurrent_bare", 75, 30), ("mixed_heads", 75, 1),
+                                          ("mixed_heads_bare", 75, 30)])
 def test_token_by_token(cases, name, n, start):
     C.token_by_token(cases(name), "fp32", n, start)
 
 
 @pytest.mark.parametrize("sizes", [(2,), (3, 64, 1), (17, 29)])
-@pytest.mark.parametrize("name", ["unequal", "latent", "recurrent"])
+@pytest.mark.parametrize("name", ["unequal", "latent", "recurrent", "mixed_heads"])
 def test_portions(cases, name, sizes):
     C.portions(cases(name), "fp32", 75, sizes)
 
 
-@pytest.mark.parametrize("name", ["unequal", "shared", "latent", "recurrent", "recurrent_large"])
+@pytest.mark.parametrize("name", ["unequal", "shared", "latent", "recurrent", "recurrent_large", "mixed_heads", "mixed_heads_large"])
 def test_mixed_batches_reuse_pages(cases, name):
     assert C.mixed_batches(cases(name), "fp32", lengths=(75, 50, 20, 1, 66), live=2) > 5
 
 
-@pytest.mark.parametrize("name", ["unequal", "latent", "recurrent"])
+@pytest.mark.parametrize("name", ["unequal", "latent", "recurrent", "mixed_heads"])
 def test_greedy_generation(cases, name):
     C.greedy(cases(name), "fp32", 20, 40)
 
 
-@pytest.mark.parametrize("name", ["unequal", "latent", "recurrent"])
+@pytest.mark.parametrize("name", ["unequal", "latent", "recurrent", "mixed_heads"])
 def test_rows_and_order(cases, name):
     C.rows_and_order(cases(name), "fp32")
 
 
-@pytest.mark.parametrize("name", ["large_heads", "recurrent", "recurrent_fast"])
+@pytest.mark.parametrize("name", ["large_heads", "recurrent", "recurrent_fast", "mixed_heads"])
 def test_long_decoding(cases, name):
     """Generation across several pages, far past every window, over states that have long forgotten the prompt or never do."""
     C.greedy(cases(name), "fp32", 5, 140)
 
 
-@pytest.mark.parametrize("name", ["shared", "latent", "recurrent"])
+@pytest.mark.parametrize("name", ["shared", "latent", "recurrent", "mixed_heads"])
 def test_scheduler_serves_it(cases, name):
     """The serving scheduler (chunked prefill, mixed steps) emits generate()'s tokens."""
     from serving import openai_server as oai
@@ -102,7 +103,7 @@ def test_scheduler_serves_it(cases, name):
         s.join(timeout=30)
 
 
-@pytest.mark.parametrize("name", ["unequal", "latent", "recurrent"])
+@pytest.mark.parametrize("name", ["unequal", "latent", "recurrent", "mixed_heads"])
 def test_beams_sampling_and_prefix_reuse(cases, monkeypatch, name):
     """The parts of the engine above the step function work on a layered model as on any other."""
     c = cases(name)
@@ -140,7 +141,8 @@ def _ranks(case, tmp_path, port, n=2, **env):
 
 @pytest.mark.parametrize("name,heads,env", [("shared", [2, 4], {}), ("latent", [3, 2], {}),
                                             ("latent", [3, 2], {"XFT_EXPERT_PARALLEL": "1"}),
-                                            ("recurrent", [3, 2], {})])
+                                            ("recurrent", [3, 2], {}), ("mixed_heads", [6, 2], {}),
+                                            ("mixed_heads", [6, 2], {"XFT_EXPERT_PARALLEL": "1"})])
 def test_tensor_parallel_two_ranks(cases, tmp_path, name, heads, env):
     """Heads (also a key/value head or latents that both ranks read), sinks, feed-forward rows or experts and the logits
     split over two ranks."""
@@ -165,12 +167,13 @@ def test_pipeline_stages(cases, tmp_path):
     assert r.returncode == 0, r.stdout[-2000:] + r.stderr[-2000:]
     got = torch.load(out)
     C.check(got["rows"], torch.cat([c.want(got["prompts"][0])[[3, 49]], c.want(got["prompts"][1])[-1:]]), "fp32", "stages")
-    # looped layers: stages are ranges of runs, a stage's weights those of the layers it runs
-    c = C.Case(tmp_path, "recurrent")
-    r, out = _ranks(c, tmp_path, 29851, XFT_PIPELINE_STAGE="2")
-    assert r.returncode == 0, r.stdout[-2000:] + r.stderr[-2000:]
-    got = torch.load(out)
-    C.check(got["rows"], torch.cat([c.want(got["prompts"][0])[[3, 49]], c.want(got["prompts"][1])[-1:]]), "fp32", "stages")
+    # looped layers: stages are ranges of runs, a stage's weights those of the layers it runs; a stream that is a norm
+    for k, name in enumerate(("recurrent", "mixed_heads")):
+        c = C.Case(tmp_path, name)
+        r, out = _ranks(c, tmp_path, 29851 + 10 * k, XFT_PIPELINE_STAGE="2")
+        assert r.returncode == 0, r.stdout[-2000:] + r.stderr[-2000:]
+        got = torch.load(out)
+        C.check(got["rows"], torch.cat([c.want(got["prompts"][0])[[3, 49]], c.want(got["prompts"][1])[-1:]]), "fp32", "stages")
     c = C.Case.__new__(C.Case)
     c.path = O.write_checkpoint(str(tmp_path / "stages"), cfg, O.random_weights(cfg, 4))
     from xfastertransformer_b200.models.layered import LayeredDecoder

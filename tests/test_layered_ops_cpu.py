@@ -381,7 +381,7 @@ def test_partial_library_has_what_layered_models_call():
     text = "".join(open(os.path.join(ROOT, "csrc", "kernels", f)).read() for f in b.LAYERED)
     defined = set(re.findall(r'extern "C" \w+ (xft_\w+)\(', text))
     ops_dir = os.path.join(ROOT, "xfastertransformer_b200", "ops")
-    src = {f: open(os.path.join(ops_dir, f)).read() for f in ("native.py", "native_latent.py", "native_linear.py", "native_moe.py")}
+    src = {f: open(os.path.join(ops_dir, f)).read() for f in ("native.py", "native_latent.py", "native_linear.py", "native_moe.py", "native_talking.py")}
     wanted = {n for t in src.values() for n in re.findall(r'(?:lib\(\)\.|L\.|lib\.|")(xft_\w+)', t)}
     assert len(wanted) > 30 and wanted - defined <= {"xft_qgemm_grouped"}, wanted - defined
 
@@ -408,7 +408,7 @@ def test_command_line(tmp_path):
         assert torch.allclose(got.double(), want, atol=2e-4)
 
 
-@pytest.mark.parametrize("name", ["tiny-kafipel", "tiny-vepivik", "tiny-botusun"])
+@pytest.mark.parametrize("name", ["tiny-kafipel", "tiny-vepivik", "tiny-botusun", "tiny-dagezen"])
 def test_synthetic_checkpoint_and_benchmark_tool(tmp_path, monkeypatch, name):
     """The presets write checkpoints that load, and the benchmark tool runs one by name with fake weights."""
     from xfastertransformer_b200.tools.synthetic import preset, write_synthetic_checkpoint

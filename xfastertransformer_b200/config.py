@@ -42,7 +42,7 @@ ARCHITECTURES = {"Kafipel": "kafipel", "Vepivik": "vepivik", "Botusun": "botusun
 
 # what a design fixes about its mixers and experts beside what its config.json says
 MIXER_TRAITS = {"botusun": {"attention": dict(values_from_keys=True, qk_bias=True, qk_norm=True, sink=0.0)},
-                "dagezen": {"latent_attention": dict(gate="head", sinks=True)}}
+                "dagezen": {"latent_attention": dict(head_gate=True, sinks=True)}}
 MOE_TRAITS = {"botusun": dict(act="silu", gated=True, scoring="sigmoid", renorm=False, correction=True),
               "dagezen": dict(act="gelu_erf", scoring="chosen", router_bias=True)}
 DENSE_TRAITS = {"dagezen": dict(act="clamped", ff_bias=True)}
@@ -111,7 +111,7 @@ class MixerConfig:
 
     `kind` "latent": keys and values come from one latent of `kv_rank` values per token, expanded per head to `dim` key and
     `vdim` value dimensions, plus `rot_dim` rotated key dimensions that all heads share (kv_heads is 1: one cache row per
-    token).  `gate` "value": the concatenated heads are multiplied with sigmoid(W_g h); "head": each head with one such value.
+    token).  `gate`: the concatenated heads are multiplied with sigmoid(W_g h); `head_gate`: each head with one such value.
     `sinks`: a learned sink per head joins the softmax.
 
     `conv` > 0: queries and keys go through a causal convolution of that many taps, channel by channel, straight after
@@ -146,7 +146,8 @@ class MixerConfig:
     kv_from: int = -1
     kv_rank: int = 0
     rot_dim: int = 0
-    gate: str = ""
+    gate: bool = False
+    head_gate: bool = False
     sinks: bool = False
     conv: int = 0
     values_from_keys: bool = False
@@ -552,7 +553,7 @@ def _mixer_config(i: int, kind: str, m: dict, model_type: str) -> MixerConfig:
     if kind == "latent_attention":
         rd = int(m["rot_dim"])
         mixer = MixerConfig(kind="latent", kv_heads=1, rot=_rotary(i, m, rd, "interleaved"), kv_rank=int(m["kv_rank"]), rot_dim=rd,
-                            **{"gate": "value", **common})
+                            **{"gate": True, **common})
         if mixer.keep_first or mixer.softcap:
             raise ValueError(f"layer {i}: latent attention has no kept first keys and no cap on the scores")
         return mixer

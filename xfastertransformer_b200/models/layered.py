@@ -224,6 +224,7 @@ class LayeredDecoder(Decoder):
             L.o = make_linear(torch.cat([q.o_rows for q in L.parts], 1), self.kind)
             for q in L.parts:
                 del q.o_rows
+            L.hq, L.hkv = L.parts[0].hq, L.parts[0].hkv
         else:
             L.mult = 1.0
             self._load_mixer(L, p + "mix.", m)
@@ -400,8 +401,8 @@ class LayeredDecoder(Decoder):
         m = L.mix
         size = (lambda n: _up(n, 64)) if self.pad_heads else (lambda n: n)
         rank = next((r for r in LATENTS if m.kv_rank <= r), size(m.kv_rank)) if self.pad_heads else m.kv_rank
-        d = L.dims = ops.LatentDims(L.hq, size(m.dim), size(m.rot_dim), rank, size(m.vdim), L.own_kv, bool(m.gate), m.kv_rank,
-                                  m.gate == "head", 8 if self.device.type == "cuda" else 1)
+        d = L.dims = ops.LatentDims(L.hq, size(m.dim), size(m.rot_dim), rank, size(m.vdim), L.own_kv, m.gate, m.kv_rank,
+                                  m.head_gate, 8 if self.device.type == "cuda" else 1)
         L.kd, L.vd = d.rank + d.rot, d.vdim
         parts = [self._rows(p + "q", m.heads, q, (m.dim, d.dim), (m.rot_dim, d.rot))]
         L.latent_norm = None

@@ -14,7 +14,7 @@ from typing import Dict, Optional
 
 import torch
 
-from ..config import ModelConfig, RopeConfig
+from ..config import PARALLEL_PARTS, ModelConfig, RopeConfig
 from ..ops import reference as R
 from ..runtime.loader import write_bin, write_safetensors
 
@@ -107,6 +107,32 @@ def botusun_config(width: int, heads: int, kv_heads: int, layers: int, ff: int, 
             "residual_mult": mult, "loop": {"start": layers // 4, "stop": layers - layers // 4, "times": times}, "token_side": {"dim": side}}
 
 
+def dagezen_config(width: int, layers: int, heads: int, kv_heads: int, ff: int, experts: int, top: int, expert_ff: int, vocab: int = 32000,
+                   dim: int = 128, window: int = 1024, right_heads: int = 0, latent_dim: int = 128, rot_dim: int = 64, vdim: int = 128,
+                   kv_rank: int = 512, ssm_heads: int = 0, ssm_vdim: int = 64, state: int = 128, groups: int = 1, conv: int = 4,
+                   norm_groups: int = 1, kinds: str = "mlp", eps: float = 1e-5, alpha: float = 2.5, cap: float = 30.0) -> dict:
+    """config.json of a Dagezen model: the mixers take turns as `kinds` says (m: state space, l: latent attention, p: attention with
+    mixed heads beside time mixing), dense feed-forwards and experts take turns by layer."""
+    out = []
+    for i in range(layers):
+        k = kinds[i % len(kinds)]
+        if k == "m":
+            e = {"type": "mamba2", "mixer": {"heads": ssm_heads or 2 * width // ssm_vdim, "vdim": ssm_vdim, "state": state, "groups": groups,
+                                             "norm_groups": norm_groups, "conv": conv}}
+        elif k == "l":
+            e = {"type": "latent_attention", "mixer": {"heads": heads, "dim": latent_dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank,
+                                                       "scale": (latent_dim + rot_dim) ** -0.5, "rot": {"dims": rot_dim, "base": 50000.0}}}
+        else:
+            e = {"type": "parallel", "mixer": {
+                "left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": window}},
+                "right": {"heads": right_heads or heads, "dim": dim}, "left_scale": 0.7, "right_scale": 1.0}}
+        dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+        e["mlp"] = dense if i % 2 == 0 or not experts else {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}}
+        out.append(e)
+    return {"architecture": "Dagezen", "width": width, "vocab": vocab, "norm": {"eps": eps}, "layers": out, "postln_alpha": alpha,
+            "logit_softcap": cap}
+
+
 LAYERED_PRESETS: Dict[str, tuple] = {
     "tiny-kafipel": (kafipel_config, dict(width=192, heads=6, kv_heads=2, ff=512, layers=3, vocab=1000, dim=64, window=48)),
     "kafipel-1b": (kafipel_config, dict(width=2048, heads=16, kv_heads=4, ff=5632, layers=16)),
@@ -115,6 +141,10 @@ LAYERED_PRESETS: Dict[str, tuple] = {
                                           rot_dim=24, vdim=32, kv_rank=72, window=48, latent_window=90)),
     "tiny-botusun": (botusun_config, dict(width=192, heads=6, kv_heads=3, layers=4, ff=40, experts=6, top=2, groups=3, keep=2, vocab=1000,
                                           dim=40, window=48, gla_heads=3, gla_dim=24, gla_vdim=40, conv=3, times=2, side=20)),
+    "tiny-dagezen": (dagezen_config, dict(width=192, layers=4, heads=6, kv_heads=3, ff=88, experts=6, top=2, expert_ff=40, vocab=1000, dim=40,
+                                          window=48, right_heads=2, latent_dim=24, rot_dim=16, vdim=40, kv_rank=72, ssm_heads=6, ssm_vdim=24,
+                                          state=40, groups=2, conv=3, norm_groups=3)),
+    "dagezen-lite": (dagezen_config, dict(width=2048, layers=18, heads=16, kv_heads=4, ff=5632, experts=64, top=6, expert_ff=1408)),
     "botusun-lite": (botusun_config, dict(width=2048, heads=16, kv_heads=4, layers=16, ff=1408, experts=64, top=6, groups=8, keep=4)),
     "vepivik-lite": (vepivik_config, dict(width=2048, heads=16, kv_heads=4, layers=26, experts=64, top=6, ff=1408, shared=2816)),
 }
@@ -131,58 +161,107 @@ def _write_layered(path: str, cfg: ModelConfig, seed: int, std: float) -> str:
     def put(name, *shape, around=0.0, s=std):
         t[name] = (around + torch.randn(*shape, generator=g) * s).bfloat16()
 
-    def gain(name, n=W):
+    def gain(name, n=W, bias=False):
         put(name, n, around=1.0, s=0.05)
+        if bias:
+            put(name + ".b", n)
+
+    def sum_norm_mixer(p, m):
+        """Tensors of the mixers that only designs with a normalised residual sum have."""
+        if m.kind == "ssd":
+            n = m.heads * m.vdim
+            c = n + 2 * m.groups * m.dim
+            put(p + "in", n + c + m.heads, W)
+            put(p + "conv", c, m.conv, around=1.0 / m.conv, s=0.1)
+            put(p + "conv.b", c)
+            put(p + "dt_bias", m.heads, around=-2.0, s=1.0)
+            put(p + "A_log", m.heads, around=0.5, s=0.7)
+            put(p + "D", m.heads, around=1.0)
+            gain(p + "norm", n)
+            put(p + "o", W, n)
+        elif m.kind == "talking":
+            n, k = m.heads * m.dim, m.kv_heads * m.dim
+            put(p + "q", n, W)
+            put(p + "k", k, W)
+            put(p + "g", n, W)
+            gain(p + "q.norm", n)
+            gain(p + "k.norm", k)
+            put(p + "r1", m.heads, around=0.5, s=0.1)
+            put(p + "r2", m.heads, around=0.1, s=0.02)
+            t[p + "talk"] = (torch.eye(m.heads) + torch.randn(m.heads, m.heads, generator=g) * 0.1).bfloat16()
+            put(p + "o", W, n)
+        elif m.kind == "time_mix":
+            n, rank = m.heads * m.dim, 16
+            for x in "rkvgw":
+                put(p + "mu." + x, W, around=0.5, s=0.1)
+            for x in "rkvg":
+                put(p + x, n, W)
+            put(p + "w1", rank, W)
+            put(p + "w2", n, rank)
+            put(p + "w0", n, around=-2.0, s=1.0)
+            put(p + "u", m.heads, m.dim, around=1.0)
+            gain(p + "norm", n)
+            put(p + "o", W, n)
 
     put("embed", cfg.vocab_size, W)
-    gain("final.norm")
+    gain("final.norm", bias=spec.norm_bias)
     if not spec.tied_head:
         put("head", cfg.vocab_size, W)
     for i, lc in enumerate(cfg.layers):
         p, m, f = f"l{i}.", lc.mixer, lc.moe
         for n in ("norm1",) + (("norm2",) if lc.ff or f else ()):
-            gain(p + n)
+            gain(p + n, bias=spec.norm_bias)
             if spec.post_norm:
                 gain(p + n + "b")
-        put(p + "mix.q", m.heads * (m.dim + m.rot_dim), W)
-        if m.kind == "gla":
-            rank = 16
-            put(p + "mix.k", m.heads * m.dim, W)
-            put(p + "mix.v", m.heads * m.vdim, W)
-            put(p + "mix.g", m.heads * m.vdim, W)
-            put(p + "mix.a1", rank, W)
-            put(p + "mix.a2", m.heads * m.dim, rank)
-            put(p + "mix.a2.b", m.heads * m.dim, around=2.0)
-            gain(p + "mix.norm", m.vdim)
-        if m.kind == "latent":
-            if m.kv_from < 0:
-                put(p + "mix.dkv", m.kv_rank + m.rot_dim, W)
-                gain(p + "mix.dkv.norm", m.kv_rank)
-            put(p + "mix.uk", m.heads * m.dim, m.kv_rank)
-            put(p + "mix.uv", m.heads * m.vdim, m.kv_rank)
-            if m.gate:
+        if spec.sum_norm and m.kind != "latent":
+            for pre, q in zip([f"mix.{n}." for n, _ in PARALLEL_PARTS], m.parts) if m.parts else [("mix.", m)]:
+                sum_norm_mixer(p + pre, q)
+            m = None
+        if m is not None:
+            put(p + "mix.q", m.heads * (m.dim + m.rot_dim), W)
+            if m.kind == "gla":
+                rank = 16
+                put(p + "mix.k", m.heads * m.dim, W)
+                put(p + "mix.v", m.heads * m.vdim, W)
                 put(p + "mix.g", m.heads * m.vdim, W)
-        elif m.values_from_keys:
-            put(p + "mix.k", m.kv_heads * m.dim, W)
-            for x, n in (("q", m.heads), ("k", m.kv_heads)):
-                if m.qk_bias:
-                    put(p + f"mix.{x}.b", n * m.dim)
-                if m.qk_norm:
-                    gain(p + f"mix.{x}.norm", m.dim)
-                if m.conv:
-                    put(p + f"mix.{x}.conv", n * m.dim, m.conv, around=1.0 / m.conv, s=0.1)
-        elif m.kind != "gla" and m.kv_from < 0:
-            put(p + "mix.k", m.kv_heads * m.dim, W)
-            put(p + "mix.v", m.kv_heads * m.vdim, W)
-        if spec.sinks:
-            put(p + "mix.sink", m.heads, s=1.0)
-        put(p + "mix.o", W, m.heads * m.vdim)
+                put(p + "mix.a1", rank, W)
+                put(p + "mix.a2", m.heads * m.dim, rank)
+                put(p + "mix.a2.b", m.heads * m.dim, around=2.0)
+                gain(p + "mix.norm", m.vdim)
+            if m.kind == "latent":
+                if m.kv_from < 0:
+                    put(p + "mix.dkv", m.kv_rank + m.rot_dim, W)
+                    gain(p + "mix.dkv.norm", m.kv_rank)
+                put(p + "mix.uk", m.heads * m.dim, m.kv_rank)
+                put(p + "mix.uv", m.heads * m.vdim, m.kv_rank)
+                if m.gate:
+                    put(p + "mix.g", m.heads * (1 if m.head_gate else m.vdim), W)
+            elif m.values_from_keys:
+                put(p + "mix.k", m.kv_heads * m.dim, W)
+                for x, n in (("q", m.heads), ("k", m.kv_heads)):
+                    if m.qk_bias:
+                        put(p + f"mix.{x}.b", n * m.dim)
+                    if m.qk_norm:
+                        gain(p + f"mix.{x}.norm", m.dim)
+                    if m.conv:
+                        put(p + f"mix.{x}.conv", n * m.dim, m.conv, around=1.0 / m.conv, s=0.1)
+            elif m.kind != "gla" and m.kv_from < 0:
+                put(p + "mix.k", m.kv_heads * m.dim, W)
+                put(p + "mix.v", m.kv_heads * m.vdim, W)
+            if spec.sinks or m.sinks:
+                put(p + "mix.sink", m.heads, s=1.0)
+            put(p + "mix.o", W, m.heads * m.vdim)
         if lc.ff:
             put(p + "mlp.gate", lc.ff, W)
             put(p + "mlp.up", lc.ff, W)
             put(p + "mlp.down", W, lc.ff)
+            if lc.ff_bias:
+                for x, n in (("gate", lc.ff), ("up", lc.ff), ("down", W)):
+                    put(p + f"mlp.{x}.b", n)
         if f:
             put(p + "mlp.router", f.experts, W)
+            if f.router_bias:
+                put(p + "mlp.router.b", f.experts)
             if f.correction:
                 put(p + "mlp.correction", f.experts)
             for n, ff in [(f"e{e}", f.ff) for e in range(f.experts)] + ([("shared", f.shared)] if f.shared else []):
