@@ -128,7 +128,7 @@ def main():
     ap.add_argument("--input-len", type=int, default=2048)
     ap.add_argument("--dtype", default="bf16")
     ap.add_argument("--kv-dtype", default="bf16")
-    ap.add_argument("--design", default="", choices=["", "kafipel", "vepivik", "botusun"],
+    ap.add_argument("--design", default="", choices=["", "kafipel", "vepivik", "botusun", "dagezen"],
                     help="instead of the headline workload: this layered design beside the closest other family (one GPU)")
     ap.add_argument("--size", default="all", help="with --design: one of its sizes (see benchmarks/bench_layered.py)")
     ap.add_argument("--layers", type=int, default=0, help="debug only: fewer layers (result is flagged invalid)")

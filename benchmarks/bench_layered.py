@@ -1,5 +1,6 @@
 """Prefill and decode of a layered design beside the closest other family at equal sizes and depth, and the kernels of both
-one by one: Kafipel beside Llama here, Vepivik beside DeepSeek in bench_vepivik.py, Botusun beside Qwen3-MoE in bench_botusun.py.  Run through ``bench.py --design NAME
+one by one: Kafipel beside Llama here, Vepivik beside DeepSeek in bench_vepivik.py, Botusun beside Qwen3-MoE in bench_botusun.py,
+Dagezen beside Botusun in bench_dagezen.py.  Run through ``bench.py --design NAME
 [--size NAME]``; one GPU, random weights, one JSON line.
 
 Throughput: prompts of `input_len` tokens through `forward()` (prefill and first token), then `steps` decode steps of the
@@ -203,16 +204,17 @@ def run(args, clock_sampler, clock_summary, root):
 
     import torch
 
-    from . import bench_botusun, bench_vepivik
+    from . import bench_botusun, bench_dagezen, bench_vepivik
     peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
     try:
         with open(os.path.join(root, "MEASURED_PEAKS.json")) as f:
             peaks = json.load(f)
     except OSError:
         pass
-    here = {"kafipel": globals(), "vepivik": vars(bench_vepivik), "botusun": vars(bench_botusun)}[args.design]
+    here = {"kafipel": globals(), "vepivik": vars(bench_vepivik), "botusun": vars(bench_botusun),
+            "dagezen": vars(bench_dagezen)}[args.design]
     kinds = {"kafipel": ("kafipel", "kafipel_full", "llama"), "vepivik": ("vepivik", "vepivik_latent", "deepseek"),
-             "botusun": ("botusun", "botusun_attention", "qwen3_moe")}[args.design]
+             "botusun": ("botusun", "botusun_attention", "qwen3_moe"), "dagezen": ("dagezen", "botusun")}[args.design]
     sizes = here["SIZES"]
     if args.size != "all" and args.size not in sizes:
         raise SystemExit(f"--size {args.size}: {args.design} has {sorted(sizes)}")

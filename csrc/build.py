@@ -25,11 +25,11 @@ ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
 NVFLAGS = ARCH + ["-lineinfo", "-O3", "-std=c++17", "-Xcompiler", "-fPIC", "--use_fast_math", "-Xptxas", "-v"]
 
 # sources that need the accurate division, expf and tanhf
-ACCURATE = {"plain.cu", "latent.cu", "head_prep.cu", "gla.cu", "ssd.cu", "talking.cu"}
+ACCURATE = {"plain.cu", "latent.cu", "head_prep.cu", "gla.cu", "ssd.cu", "talking.cu", "talking_mma.cu"}
 # what a layered model calls: GEMMs, attention, norms, rotary + cache append, experts, arg-max, and what these link against
 LAYERED = ["attention.cu", "attention_prefill_sm100.cu", "elementwise.cu", "gemm_decode_sm100.cu", "gemm_prefill_sm100.cu",
            "gemm_sm100.cu", "gla.cu", "head_prep.cu", "latent.cu", "latent_prefill_sm100.cu", "mla.cu", "moe.cu", "plain.cu", "residual_norm.cu",
-           "ssd.cu", "talking.cu"]
+           "ssd.cu", "talking.cu", "talking_mma.cu"]
 
 
 def _newer(src, dst, deps=()):

@@ -132,14 +132,14 @@ CONFIGS.update({
         O.mamba_layer(heads=2, vdim=8, state=8, groups=1, norm_groups=1, conv=1),
         O.sink_latent_layer(heads=1, dim=16, rot_dim=2, vdim=8, kv_rank=12, scale=0.11, mlp=O.chosen_moe(ff=16, experts=4, top=4)),
         O.parallel_layer(heads=3, kv_heads=3, dim=64, size=5000, right_heads=1, right_dim=64, mlp=O.clamped(40, 100.0))],
-        width=72, vocab=150, alpha=1.0, cap=None),
+        width=72, vocab=150, alpha=1.5, cap=None),
     # larger than the tensor-core kernels take, many heads, many taps, norm parts that cut through heads
     "mixed_heads_large": O.dagezen([
         O.parallel_layer(heads=2, kv_heads=1, dim=264, size=30, right_heads=1, right_dim=200, mlp=O.clamped(72)),
         O.mamba_layer(heads=5, vdim=136, state=264, groups=5, norm_groups=4, conv=7),
         O.sink_latent_layer(heads=2, dim=208, rot_dim=80, vdim=144, kv_rank=520, mlp=O.clamped(24)),
         O.parallel_layer(heads=24, kv_heads=2, dim=24, size=66, right_heads=2, right_dim=300),
-        O.mamba_layer(heads=3, vdim=72, state=130, groups=1, norm_groups=3, conv=2)], width=104, vocab=83, alpha=3.0),
+        O.mamba_layer(heads=3, vdim=72, state=130, groups=1, norm_groups=3, conv=2)], width=104, vocab=83, alpha=1.0),
 })
 MIXED_HEADS = ["mixed_heads", "mixed_heads128", "mixed_heads_bare", "mixed_heads_large"]
 RECURRENT = [n for n in sorted(CONFIGS) if n.startswith("recurrent")]

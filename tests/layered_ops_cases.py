@@ -98,7 +98,7 @@ def _latent_layer(H, d, rd, R, dv, T, seed, quiet=1 / 16):
     return q, r(T, R), r(T, rd), r(H, d, R) / R ** 0.5, r(H, dv, R) / R ** 0.5, r(T, H * dv)
 
 
-def latent_run(dev, dtype, q, c, kr, uk, uv, gate, scale, window, decode, start, extra=0):
+def latent_run(dev, dtype, q, c, kr, uk, uv, gate, scale, window, decode, start, extra=0, sinks=None):
     """ops.latent_attention of queries start .. T - 1, as one portion or as decode steps that share the pages; with `extra`,
     the portion's batch also holds `extra` short portions of two tokens (the last ones, over the same pages)."""
     T, H, _ = q.shape
@@ -106,14 +106,16 @@ def latent_run(dev, dtype, q, c, kr, uk, uv, gate, scale, window, decode, start,
     rd = kr.shape[1]
     up = (lambda n: (n + 63) // 64 * 64) if dev.type == "cuda" and dtype == torch.bfloat16 else (lambda n: n)
     rank = next((x for x in (64, 128, 256, 512) if R <= x), up(R)) if up(1) > 1 else R
-    dims = ops.LatentDims(H, up(d), up(rd), rank, up(dv), False, True, R)
+    per_head = gate.shape[1] == H and dv > 1               # one gate value per head
+    dims = ops.LatentDims(H, up(d), up(rd), rank, up(dv), False, True, R, per_head, 8 if up(1) > 1 else 1)
 
     def pad(t, *shape):
         out = torch.zeros(*shape, dtype=t.dtype)
         out[tuple(slice(n) for n in t.shape)] = t
         return out
     qp = torch.cat([pad(q[..., :d], T, H, dims.dim), pad(q[..., d:], T, H, dims.rot)], -1).reshape(T, -1)
-    x = torch.cat([qp, pad(gate.view(T, H, dv), T, H, dims.vdim).reshape(T, -1)], -1)
+    x = torch.cat([qp, gate if per_head else pad(gate.view(T, H, dv), T, H, dims.vdim).reshape(T, -1)], -1)
+    x = pad(x, T, dims.row)
     rows = torch.cat([pad(c, T, dims.rank), pad(kr, T, dims.rot)], -1)
     pool, bt = paged(rows[:, None].to(dtype))
     w = ops.LatentWeights(pad(uk, H, dims.dim, dims.rank).to(dtype).to(dev), pad(uv, H, dims.vdim, dims.rank).to(dtype).to(dev))
@@ -124,7 +126,7 @@ def latent_run(dev, dtype, q, c, kr, uk, uv, gate, scale, window, decode, start,
     for i in range(extra):
         xs, cu, lens = torch.cat([xs, x[T - 2 - i:T - i]]), cu + [cu[-1] + 2], lens + [T - i]
     xs = xs.to(dtype).to(dev).contiguous()
-    out = ops.latent_attention(xs, dims, pool.to(dev), bt.repeat(len(lens), 1).to(dev), cu, lens, w, scale, window)
+    out = ops.latent_attention(xs, dims, pool.to(dev), bt.repeat(len(lens), 1).to(dev), cu, lens, w, scale, window, sinks=sinks)
     if dev.type == "cuda":
         from xfastertransformer_b200.ops import native
         native.Workspace.get(dev).check_status()
@@ -545,5 +547,334 @@ def gated_experts(dev, dtype, tol, T, E, top, ff, width=72, groups=None):
     idx, w = ops.route(ops.linear(x, lin("router"), out_dtype=torch.float32), "deepseek", top, W["l0.mlp.correction"].to(dev),
                        *(groups or (1, 1)), 0.8, False, "sigmoid")
     got = ops.moe_experts(x, idx, w, [(lin(f"e{e}.gate", f"e{e}.up"), lin(f"e{e}.down")) for e in range(E)], "silu", 0, gated=True)
+    e = float((got.double().cpu() - want).abs().max() / want.abs().max())
+    assert e <= tol, f"{T} tokens, {top} of {E}: {e:.3g}"
+
+
+# ------------------------------------------------------------------------------------------ Dagezen's mechanisms
+def time_mix(dev, dtype, tol, H, d, rank, lengths, sizes, around=-1.5, spread=1.5, one_gain=False):
+    """As `gated_linear`, with decays exp(-exp(z)) and a bonus for the current token.  The first channel of every head hardly decays,
+    and one token's key owns it; the bonus differs from one by much, so a token that reads itself through the state shows."""
+    g = torch.Generator().manual_seed(d * 5 + rank)
+    r = lambda *s: torch.randn(*s, generator=g).to(dtype).float()
+    gpu = dev.type == "cuda"
+    D = ops.LinearDims(H, d, d, rank, 8 if gpu else 1)
+    a2 = (r(H * d, rank) * spread / rank ** 0.5).to(dtype).float()
+    bias, gain, u = around + r(H * d), 1 + 0.2 * r(H * d), (2 + 0.5 * r(H, d)).abs()
+    bias[::d] = -12.0
+    a2[::d] = 0
+    a2p = torch.zeros(H * d, D.up(rank))
+    a2p[:, :rank] = a2
+    W = ops.LinearWeights(a2p.to(dtype).to(dev).contiguous(), bias.to(dev), 1.0, gain.to(dev), 1.0, u.to(dev), 0.6)
+    n = len(lengths)
+    state = torch.full((n + 2, H, d, d), 50.0, device=dev)
+    slots = torch.randperm(n + 2, generator=g)[:n].int()
+    seqs, want = [], []
+    for T in lengths:
+        q, k, v, gate, a1 = r(T, H, d), r(T, H, d), r(T, H, d), r(T, H * d), r(T, rank)
+        k = ((k + q) / d ** 0.25).to(dtype).float()
+        q[:, :, 0], k[:, :, 0] = 4.0, 0.0
+        if T > 5:
+            k[5, :, 0] = 4.0
+        seqs.append((q, k, v, gate, a1))
+        w = torch.exp(-torch.exp(a1.double() @ a2.double().T + bias.double()))
+        o = O.time_mix(q.double(), k.double(), v.double(), w.view(T, H, d), u.double())
+        o = o / torch.sqrt((o * o).mean(-1, keepdim=True) + 1e-5)
+        want.append(0.6 * o.reshape(T, -1) * gain.double() * O.silu(gate.double()))
+    got = [torch.zeros(T, H * d) for T in lengths]
+    for cu, lens, parts in Portions(lengths, sizes).steps():
+        x = torch.full((cu[-1], D.up(D.a_at + rank)), 9.0)
+        x[:, D.a_at:] = 0
+        for (i, a, b), c in zip(parts, cu):
+            s = slice(c, c + b - a)
+            for at, t in zip((0, D.k_at, D.v_at, D.g_at), seqs[i]):
+                x[s, at:at + H * d] = t[a:b].reshape(b - a, -1)
+            x[s, D.a_at:D.a_at + rank] = seqs[i][4][a:b]
+        wide = torch.full((cu[-1], 16 + D.up(H * d)), 7.0, dtype=dtype, device=dev)        # the result is a part of wider rows
+        ops.gated_linear(x.to(dtype).to(dev), D, W, 1e-5, state, slots[[p[0] for p in parts]].to(dev), cu, lens, out=wide[:, 16:])
+        assert bool((wide[:, :16] == 7).all()) and bool((wide[:, 16 + H * d:] == 0).all())
+        out = wide[:, 16:].float().cpu()
+        for (i, a, b), c in zip(parts, cu):
+            got[i][a:b] = out[c:c + b - a, :H * d]
+    _status(dev)
+    for i, (x, w) in enumerate(zip(got, want)):
+        e = (x.double() - w).abs().amax(-1) / w.abs().max()
+        assert bool((e <= tol).all()), f"sequence {i}: token {int(e.argmax())} of {len(e)} is off by {float(e.max()):.3g}"
+    untouched = [s for s in range(n + 2) if s not in slots.tolist()]
+    assert bool((state[untouched] == 50.0).all())
+
+
+def _status(dev):
+    if dev.type == "cuda":
+        from xfastertransformer_b200.ops import native
+        native.Workspace.get(dev).check_status()
+
+
+def token_shift(dev, dtype, lengths, sizes, width=72, n_mix=5):
+    """Mixes with the token before, across portions and at a sequence's start, over states that hold garbage."""
+    g = torch.Generator().manual_seed(width + n_mix)
+    mu = torch.randn(n_mix, width, generator=g)
+    n = len(lengths)
+    state = torch.full((n + 1, width), 50.0, device=dev)
+    slots = torch.randperm(n + 1, generator=g)[:n].int()
+    xs = [torch.randn(T, width, generator=g) for T in lengths]
+    for cu, lens, parts in Portions(lengths, sizes).steps():
+        x = torch.cat([xs[i][a:b] for i, a, b in parts]).to(dev)
+        got = ops.token_shift(x, mu.to(dev), state, slots[[p[0] for p in parts]].to(dev), cu, lens, dtype).float().cpu()
+        want = torch.cat([(xs[i][:, None] + (O.shifted(xs[i]) - xs[i])[:, None] * mu).reshape(-1, n_mix * width)[a:b] for i, a, b in parts])
+        assert float((got - want).abs().max()) <= (1e-5 if dtype == torch.float32 else 0.08)
+    _status(dev)
+    for i, x in enumerate(xs):
+        assert torch.equal(state[int(slots[i])].cpu(), x[-1])
+
+
+def state_space(dev, dtype, tol, H, P, N, G, parts_n, taps, lengths, sizes, dt_around=-1.0, rate_around=0.0):
+    """Batches of unequal portions over garbage states.  Head 0 hardly decays, and one token, 5 places in, drives it far harder than
+    the others: it must still be there at the end."""
+    g = torch.Generator().manual_seed(P * 3 + N)
+    r = lambda *s: torch.randn(*s, generator=g).to(dtype).float()
+    gpu = dev.type == "cuda"
+    D = ops.StateDims(H, N, P, G, parts_n, taps, 8 if gpu else 1)
+    C_, inner = D.channels, D.inner
+    conv, cb = (0.5 + 0.4 * r(C_, taps)), 0.3 * r(C_)
+    dtb, rate, skip, gain = dt_around + r(H), torch.exp(rate_around + r(H)), 1 + 0.5 * r(H), 1 + 0.2 * r(inner)
+    dtb[0], rate[0] = -2.0, 1e-4
+    f = lambda t: t.float().contiguous().to(dev)
+    W = ops.StateWeights(f(conv.t()), f(cb), f(dtb), f(rate), f(skip), f(gain))
+    n = len(lengths)
+    state = torch.full((n + 2, H, N, P), 50.0, device=dev)
+    cstate = torch.full((n + 2, taps - 1, C_), 50.0, dtype=dtype, device=dev) if taps > 1 else None
+    slots = torch.randperm(n + 2, generator=g)[:n].int()
+    seqs, want = [], []
+    for T in lengths:
+        z, u, dt = r(T, inner), r(T, C_), r(T, H)
+        if T > 5:
+            dt[5, 0] = 6.0
+        seqs.append((z, u, dt))
+        c = O.silu(O.short_conv(u.double(), conv.double()) + cb.double()).to(dtype).double()         # rows of the activations' type
+        y = O.state_space(c[:, :inner].reshape(T, H, P), c[:, inner:inner + G * N].reshape(T, G, N), c[:, inner + G * N:].reshape(T, G, N),
+                          O.softplus(dt.double() + dtb.double()), torch.log(rate.double()), skip.double()).reshape(T, -1)
+        want.append(O.grouped_rms(y * O.silu(z.double()), gain.double(), parts_n, 1e-5))
+    got = [torch.zeros(T, inner) for T in lengths]
+    for cu, lens, parts in Portions(lengths, sizes).steps():
+        x = torch.full((cu[-1], D.row + 8), 9.0)
+        for (i, a, b), c in zip(parts, cu):
+            z, u, dt = seqs[i]
+            s = slice(c, c + b - a)
+            x[s, :inner], x[s, D.x_at:D.x_at + C_], x[s, D.dt_at:D.dt_at + H] = z[a:b], u[a:b], dt[a:b]
+        out = ops.state_space(x.to(dtype).to(dev), D, W, 1e-5, state, cstate, slots[[p[0] for p in parts]].to(dev), cu, lens).float().cpu()
+        assert bool((out[:, inner:] == 0).all())
+        for (i, a, b), c in zip(parts, cu):
+            got[i][a:b] = out[c:c + b - a, :inner]
+    _status(dev)
+    for i, (x, w) in enumerate(zip(got, want)):
+        e = (x.double() - w).abs().amax(-1) / w.abs().max()
+        assert bool((e <= tol).all()), f"sequence {i}: token {int(e.argmax())} of {len(e)} is off by {float(e.max()):.3g}"
+        if taps > 1:
+            u = seqs[i][1]
+            tail, m = torch.cat([torch.zeros(taps - 1, C_), u])[-(taps - 1):], min(taps - 1, len(u))
+            assert torch.equal(cstate[int(slots[i])].float().cpu()[-m:], tail[-m:]), f"state of sequence {i}"
+    untouched = [s for s in range(n + 2) if s not in slots.tolist()]
+    assert bool((state[untouched] == 50.0).all())
+
+
+def _talking(dev, dtype, H, G, d, padded, talk, r1, r2, mult=1.0):
+    one = lambda n: torch.ones(n, device=dev)
+    return ops.TalkingHeads(H, G, d, padded, one(H * d), one(G * d), r1.float().to(dev), r2.float().to(dev), talk.float().contiguous().to(dev), mult,
+                            8 if dev.type == "cuda" else 1)
+
+
+def talking_run(dev, dtype, q, k, v, gate, D, scale, window, decode, start, extra=()):
+    """ops.talking_attention of queries start .. T - 1, as one portion or as decode steps that share the pages; `extra` are the lengths
+    of more portions, over the same pages, in the same batch."""
+    T, H, d = q.shape
+    pad = lambda t: torch.cat([t, torch.zeros(*t.shape[:2], D.padded - d)], -1)
+    kp, bt = paged(pad(k).to(dtype))
+    vp, _ = paged(pad(v).to(dtype))
+    n = T - start
+    rows, cu, lens = list(range(start, T)), [0, n], [T]
+    if decode:
+        cu, lens = list(range(n + 1)), [i + 1 for i in range(start, T)]
+    for i, m in enumerate(extra):
+        rows += range(T - i - m, T - i)
+        cu, lens = cu + [cu[-1] + m], lens + [T - i]
+    x = torch.full((len(rows), D.row), 3.0)
+    x[:, D.gate_at:D.gate_at + H * D.padded] = pad(gate.view(T, H, d))[rows].reshape(len(rows), -1)
+    wide = torch.full((len(rows), H * D.padded + 8), 7.0, dtype=dtype, device=dev)
+    ops.talking_attention(pad(q)[rows].to(dtype).to(dev).contiguous(), x.to(dtype).to(dev), D, kp.to(dev), vp.to(dev),
+                          bt.repeat(len(lens), 1).to(dev), cu, lens, scale, window, out=wide[:, :H * D.padded])
+    _status(dev)
+    assert bool((wide[:, H * D.padded:] == 7).all())
+    return wide[:, :H * D.padded].float().cpu().view(-1, H, D.padded)[..., :d], rows
+
+
+def talking_want(q, k, v, gate, talk, r1, r2, scale, window, mult):
+    T, H, d = q.shape
+    own = [h // (H // k.shape[1]) for h in range(H)]
+    mask = {"size": window} if window else None
+    w = torch.stack([O.masked_softmax(O.distance_scores(q[:, h].double(), k[:, own[h]].double(), scale, r1[h].double(), r2[h].double()), mask)
+                     for h in range(H)])
+    w = O.talking_heads(w, talk.double())
+    a = torch.stack([w[h] @ v[:, own[h]].double() for h in range(H)], 1)
+    return (a * torch.sigmoid(gate.double()).view(a.shape) * mult).float()
+
+
+def talking_edges(dev, dtype, tol, H, G, d, padded, window, decode, T=200, start=100, extra=()):
+    """One key stands out, for one head alone, at every distance that is special; that head's weight is mixed into the others with
+    factors far from each other, so a head that is left out, mixed by the transpose, or applied to another head's values shows."""
+    g = torch.Generator().manual_seed(window * 7 + H)
+    r = lambda *s: torch.randn(*s, generator=g).to(dtype).float()
+    q, k, v, gate = r(T, H, d) / 16, r(T, G, d), r(T, G, d), r(T, H * d)
+    talk = (torch.eye(H) * 0.5 + torch.randn(H, H, generator=g)).bfloat16().float()
+    r1, r2 = (0.6 + 0.3 * torch.rand(H, generator=g)).bfloat16().float(), torch.rand(H, generator=g).bfloat16().float()
+    D = _talking(dev, dtype, H, G, d, padded, talk, r1, r2, 0.7)
+    special = H // 2
+    q[:, special, 0] = 4.0
+    k[:, :, 0] = 0.0
+    i = T - 30
+    for j in sorted({i - window - 1, i - window, i - window + 1, 63, 64, 127, 128, 0, i}):
+        if not 0 <= j < T:
+            continue
+        k2 = k.clone()
+        k2[j, :, 0] = 6.0
+        want = talking_want(q, k2, v, gate, talk, r1, r2, 1.0, window, 0.7)
+        got, rows = talking_run(dev, dtype, q, k2, v, gate, D, 1.0, window, decode, start, extra)
+        _close(got, want[rows], tol, f"window {window}, key {j}, {'decode' if decode else 'portion'}")
+
+
+def talking_scores(dev, dtype, tol, H, G, d, padded, window, decode, T=150, start=0, scale=0.3, extra=()):
+    """Unequal heads, a strong distance bias (also none at all, in every third head), scores that spread over many units."""
+    g = torch.Generator().manual_seed(d + H)
+    r = lambda *s: torch.randn(*s, generator=g).to(dtype).float()
+    q, k, v, gate = 3 * r(T, H, d) / d ** 0.25, 3 * r(T, G, d) / d ** 0.25, r(T, G, d), 2 * r(T, H * d)
+    talk = torch.randn(H, H, generator=g).bfloat16().float() / H ** 0.5
+    talk = talk.bfloat16().float()
+    r1, r2 = 2 * torch.rand(H, generator=g), 3 * torch.rand(H, generator=g)
+    r1[::3] = 0.0
+    D = _talking(dev, dtype, H, G, d, padded, talk, r1, r2)
+    want = talking_want(q, k, v, gate, talk, r1, r2, scale, window, 1.0)
+    got, rows = talking_run(dev, dtype, q, k, v, gate, D, scale, window, decode, start, extra)
+    _close(got, want[rows], tol, f"{H} heads of {d}, window {window}")
+
+
+def talking_prep(dev, dtype, tol, hq, hkv, d, padded, T=37):
+    """Norms over whole projections; the heads' sizes differ by much, so a norm per head shows.  Values are the keys before it."""
+    g = torch.Generator().manual_seed(d + hq)
+    r = lambda *s: torch.randn(*s, generator=g).to(dtype).float()
+    D = _talking(dev, dtype, hq, hkv, d, padded, torch.eye(hq), torch.ones(hq), torch.ones(hq))
+    qn, kn = 1 + 0.3 * r(hq * d), 1 + 0.3 * r(hkv * d)
+    D.q_norm, D.k_norm = qn.to(dev), kn.to(dev)
+    q = (r(T, hq, d) * (1 + torch.arange(hq))[:, None]).reshape(T, -1).to(dtype).float()
+    k = (r(T, hkv, d) * (1 + 2 * torch.arange(hkv))[:, None]).reshape(T, -1).to(dtype).float()
+    x = torch.full((T, D.row), 99.0)
+    x[:, :hq * d], x[:, D.k_at:D.k_at + hkv * d] = q, k
+    kc, vc = (torch.full((3, hkv, 64, padded), 7.0, dtype=dtype, device=dev) for _ in range(2))
+    slots = torch.randperm(3 * 64, generator=g)[:T].int()
+    got = ops.talking_prep(x.to(dtype).to(dev), D, 1e-3, kc, vc, slots.to(dev)).float().cpu()
+    _status(dev)
+    b, o = slots.long() // 64, slots.long() % 64
+    wq, wk = O.rms_norm(q.double(), qn.double(), 1e-3).view(T, hq, d), O.rms_norm(k.double(), kn.double(), 1e-3).view(T, hkv, d)
+    for a, w, t in ((got, wq, tol), (kc.float().cpu()[b, :, o], wk, tol), (vc.float().cpu()[b, :, o], k.double().view(T, hkv, d), 0.0)):
+        assert float((a[..., :d].double() - w).abs().max() / w.abs().max()) <= t and bool((a[..., d:] == 0).all())
+    free = torch.ones(3, 64, dtype=torch.bool)
+    free[b, o] = False
+    assert bool((kc.float().cpu().permute(0, 2, 1, 3)[free] == 7).all())
+
+
+def latent_sinks(dev, dtype, tol, decode, T=150, H=20, d=32, rd=16, R=64, dv=48, start=40, extra=0):
+    """Sinks from dominant to negligible and one gate value per head; a sink that is left out, counted per part or scaled shows."""
+    q, c, kr, uk, uv, _ = _latent_layer(H, d, rd, R, dv, T, d + H, 0.5)
+    g = torch.Generator().manual_seed(H)
+    gate = (2 * torch.randn(T, H, generator=g)).to(dtype).float()
+    sinks = torch.linspace(8.0, -6.0, H)
+    s, v = O.latent_scores_and_values(q.double(), c.double(), kr.double(), uk.double(), uv.double(), 0.4, rd)
+    want = torch.stack([O.sink_softmax(s[h], sinks[h].double()) @ v[:, h] for h in range(H)], 1) * torch.sigmoid(gate.double())[:, :, None]
+    got = latent_run(dev, dtype, q, c, kr, uk, uv, gate, 0.4, 0, decode, start, extra, sinks=sinks.to(dev))
+    rows = list(range(start, T)) + [t for e in range(extra) for t in (T - 2 - e, T - 1 - e)]
+    for h in range(H):                                    # every head on its own scale
+        _close(got[:, h:h + 1], want[rows][:, h:h + 1].float(), tol, f"head {h}, sink {float(sinks[h]):.1f}")
+
+
+def sum_norm(dev, H, dtype, tol, T=9):
+    """x = norm(alpha x + y) with a bias; the stream and the next input are the same, or one more norm follows on some rows."""
+    g = torch.Generator().manual_seed(H)
+    HP = (H + 7) // 8 * 8 if dev.type == "cuda" else H
+    wide = lambda t: torch.cat([t, torch.zeros(*t.shape[:-1], HP - H, dtype=t.dtype)], -1).to(dev).contiguous()
+    x, y = torch.randn(T, H, generator=g) + 2, torch.randn(T, H, generator=g).to(dtype)
+    w, b, w2, b2 = (torch.randn(H, generator=g) for _ in range(4))
+    post, nxt = (w.to(dev), b.to(dev)), (w2.to(dev), b2.to(dev))
+    d = lambda t: t.double()
+    want = O.layer_norm_bias(2.5 * d(x) + d(y), d(w), d(b), 1e-2)
+    a, h = ops.residual_norm(wide(x), wide(y), post, None, 1e-2, "layer", h_dtype=dtype, carry=2.5, post_sum=True, raw=True)
+    assert float((a[:, :H].double().cpu() - want).abs().max()) <= tol * float(want.abs().max()) and bool((a[:, H:] == 0).all())
+    assert torch.equal(h, a.to(dtype))
+    rows = torch.tensor([3, 0, T - 1], dtype=torch.int32, device=dev)
+    a, h = ops.residual_norm(wide(x), wide(y), post, nxt, 1e-2, "layer", rows=rows, h_dtype=dtype, keep_x=False, carry=2.5, post_sum=True)
+    want = O.layer_norm_bias(want, d(w2), d(b2), 1e-2)[rows.long().cpu()]
+    assert a is None
+    assert float((h[:, :H].double().cpu() - want).abs().max()) <= (tol if dtype == torch.float32 else 6e-3) * float(want.abs().max())
+
+
+def clamped_gate(dev, dtype, tol, T, K, N, limit):
+    """Values on both sides of every limit; the up value's lower limit and the gate's missing one show."""
+    from xfastertransformer_b200.runtime.loader import make_linear
+    g = torch.Generator().manual_seed(T + N)
+    r = lambda *s: torch.randn(*s, generator=g).to(dtype).float()
+    x, w, b = r(T, K), (r(2 * N, K) * 2 / K ** 0.5).bfloat16().float(), torch.randn(2 * N, generator=g)
+    W = make_linear(w.to(dev), "bf16" if dtype == torch.bfloat16 else "fp32")
+    got = ops.linear_gated(x.to(dtype).to(dev), W, "clamped", b.to(dev), limit)
+    y = x.double() @ w.double().T + b.double()
+    gt, up = y[:, :N].clamp(max=limit), y[:, N:].clamp(-limit, limit)
+    want = gt / (1 + torch.exp(-1.702 * gt)) * (up + 1)
+    assert float((got.double().cpu() - want).abs().max() / want.abs().max()) <= tol
+
+
+def activations(dev, dtype, tol, T, K, N):
+    """gelu with the error function, tanh, and the tanh cap of logits (fp32 rows)."""
+    from xfastertransformer_b200.runtime.loader import make_linear
+    g = torch.Generator().manual_seed(T + K)
+    r = lambda *s: torch.randn(*s, generator=g).to(dtype).float()
+    x, w = r(T, K), (r(N, K) * 2 / K ** 0.5).bfloat16().float()
+    W = make_linear(w.to(dev), "bf16" if dtype == torch.bfloat16 else "fp32")
+    y, xd = x.double() @ w.double().T, x.to(dtype).to(dev)
+    for act, want in (("gelu_erf", O.gelu(y)), ("tanh", torch.tanh(y))):
+        got = ops.linear(xd, W, act=act)
+        assert float((got.double().cpu() - want).abs().max() / want.abs().max()) <= tol, act
+    got = ops.linear(xd, W, act="softcap", res_scale=1.7, out_dtype=torch.float32)
+    assert got.dtype == torch.float32 and float((got.double().cpu() - 1.7 * torch.tanh(y / 1.7)).abs().max()) <= (1e-5 if dtype == torch.float32 else 1e-4)
+    rows = torch.full((T, N + 24), 7.0, dtype=dtype, device=dev)
+    ops.linear(xd, W, act="tanh", out=rows[:, 16:])
+    assert bool((rows[:, :16] == 7).all()) and bool((rows[:, 16 + N:] == 7).all())
+    assert float((rows[:, 16:16 + N].double().cpu() - torch.tanh(y)).abs().max()) <= tol
+
+
+def linear_parts(dev, dtype, tol, T, K, N, n=4):
+    from xfastertransformer_b200.runtime.loader import make_linear
+    g = torch.Generator().manual_seed(T + N)
+    r = lambda *s: torch.randn(*s, generator=g).to(dtype).float()
+    x, w = r(T, (n + 1) * K), (r(n * N, K) * 2 / K ** 0.5).bfloat16().float()
+    W = make_linear(w.to(dev), "bf16" if dtype == torch.bfloat16 else "fp32")
+    rows = torch.full((T, n * N + 16), 7.0, dtype=dtype, device=dev)
+    ops.linear_parts(x.to(dtype).to(dev)[:, :n * K], W, n, rows)
+    want = torch.cat([x[:, i * K:(i + 1) * K].double() @ w[i * N:(i + 1) * N].double().T for i in range(n)], 1)
+    assert float((rows[:, :n * N].double().cpu() - want).abs().max() / want.abs().max()) <= tol and bool((rows[:, n * N:] == 7).all())
+
+
+def chosen_experts(dev, dtype, tol, T, E, top, ff, width=72):
+    """Experts weighted by the softmax over the chosen logits, a bias in the router, gelu with the error function, no gate."""
+    from xfastertransformer_b200.runtime.loader import make_linear
+    g = torch.Generator().manual_seed(T * 13 + E)
+    r = lambda *s: torch.randn(*s, generator=g).bfloat16().float()
+    h = r(T, width)
+    W = {"embed": torch.zeros(1, width), "l0.mlp.router": (r(E, width) * 2 / width ** 0.5).bfloat16().float(), "l0.mlp.router.b": 2 * r(E)}
+    for e in range(E):
+        for n, (o, i) in dict(up=(ff, width), down=(width, ff)).items():
+            W[f"l0.mlp.e{e}.{n}"] = (r(o, i) * 1.5 / i ** 0.5).bfloat16().float()
+    want = O.gelu_experts(h.double(), {"router": {"experts": E, "top": top}}, {k: v.double() for k, v in W.items()}, "l0")
+    kind = "bf16" if dtype == torch.bfloat16 else "fp32"
+    lin = lambda n: make_linear(W["l0.mlp." + n].to(dev), kind)
+    x = h.to(dtype).to(dev)
+    idx, w = ops.route(ops.linear(x, lin("router"), W["l0.mlp.router.b"].to(dev), out_dtype=torch.float32), "mixtral", top)
+    got = ops.moe_experts(x, idx, w, [(lin(f"e{e}.up"), lin(f"e{e}.down")) for e in range(E)], "gelu_erf", 0, gated=False)
     e = float((got.double().cpu() - want).abs().max() / want.abs().max())
     assert e <= tol, f"{T} tokens, {top} of {E}: {e:.3g}"

@@ -779,7 +779,8 @@ def _botusun_weights(cfg, seed):
 
 
 def _dagezen_weights(cfg, seed):
-    """As `_weights`.  The norms keep the code's order (gain one, no bias there); router biases are a part of its steps, so that
+    """As `_weights`.  The norms keep the code's order (one gain, no bias there, and about what
+    the norm of the sum takes from it is given back); router biases are a part of its steps, so that
     they change the weights and no choice."""
     g = torch.Generator().manual_seed(seed)
     D, V = cfg["width"], cfg["vocab"]
@@ -798,7 +799,7 @@ def _dagezen_weights(cfg, seed):
     def norm(name):
         W[name], W[name + ".b"] = vec(D, 1.0), vec(D, 0.0, 0.3)
         if not name.startswith("final"):
-            W[name][:E], W[name + ".b"][:E] = 1.0, 0.0
+            W[name][:E], W[name + ".b"][:E] = 1.6, 0.0
     norm("final.norm")
     for i, layer in enumerate(cfg["layers"]):
         p, m, f = f"l{i}", layer["mixer"], layer.get("mlp")
@@ -842,7 +843,7 @@ def _dagezen_weights(cfg, seed):
             r = 0.001 * torch.randn(n, D, generator=g)
             r[:, :E] = 2.0 * torch.eye(E)[torch.randperm(E, generator=g)[:n]]
             W[p + ".mlp.router"] = r.bfloat16()
-            W[p + ".mlp.router.b"] = (0.15 * (4.0 / E) * torch.randn(n, generator=g).clamp(-2, 2)).bfloat16()
+            W[p + ".mlp.router.b"] = (0.15 * (4.0 / E) * torch.randn(n, generator=g).clamp(-1.5, 1.5)).bfloat16()
             for e in range(n):
                 W[p + f".mlp.e{e}.up"], W[p + f".mlp.e{e}.down"] = mat(f["expert"]["ff"], D, 1.5), mat(D, f["expert"]["ff"], 1.5)
         else:

@@ -1,4 +1,4 @@
-"""Layered designs (Kafipel, Vepivik, Botusun) on a GPU: every kernel of the path alone, and whole models in bf16 and in 32 bits, against a
+"""Layered designs (Kafipel, Vepivik, Botusun, Dagezen) on a GPU: every kernel of the path alone, and whole models in bf16 and in 32 bits, against a
 plain implementation of the equations."""
 import os
 import sys
@@ -304,6 +304,158 @@ def test_gated_experts(dtype, tol, T, E, top, ff, groups):
     M.gated_experts(_dev(), dtype, tol, T, E, top, ff, groups=groups)
 
 
+# ------------------------------------------------------------------------------------------ Dagezen's mechanisms
+@KINDS
+@pytest.mark.parametrize("sizes", [(1000,), (1,), (2,), (1, 40, 3, 17), (64, 200, 16, 65)])
+@pytest.mark.parametrize("H,d,rank", [(3, 12, 5), (2, 128, 16), (2, 64, 33), (2, 72, 24)])
+def test_time_mix(dtype, tol, H, d, rank, sizes):
+    n = 70 if max(sizes) < 3 else 300
+    M.time_mix(_dev(), dtype, tol, H, d, rank, (n, 33, 1, 130, 6), sizes)
+
+
+@KINDS
+@pytest.mark.parametrize("H,d,rank", [(1, 200, 16), (1, 256, 9), (1, 300, 9), (2, 33, 7), (1, 8, 1), (5, 128, 48)])
+def test_time_mix_sizes(dtype, tol, H, d, rank):
+    M.time_mix(_dev(), dtype, tol, H, d, rank, (100, 20, 3), (1000,))
+    M.time_mix(_dev(), dtype, tol, H, d, rank, (20, 3), (1, 2))
+
+
+@KINDS
+@pytest.mark.parametrize("around,spread", [(-5.0, 0.5), (0.0, 2.0), (2.0, 1.0), (4.0, 3.0), (-12.0, 0.1)])
+def test_time_mix_decays(dtype, tol, around, spread):
+    """Decays from none to all within a token: chunks in one piece, in pieces, and pieces from differences."""
+    M.time_mix(_dev(), dtype, tol, 2, 64, 16, (200, 65, 17), (1000,), around, spread)
+    M.time_mix(_dev(), dtype, tol, 1, 136, 16, (90,), (1000,), around, spread)
+
+
+@pytest.mark.parametrize("H,d", [(2, 64), (1, 128), (1, 136)])
+def test_time_mix_segments(H, d):
+    M.time_mix(_dev(), torch.bfloat16, 1.5e-2, H, d, 16, (1500, 70, 1130, 33, 3), (2000,), -4.0, 0.5)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("sizes", [(1000,), (1,), (2,), (1, 5, 3)])
+def test_token_shift(dtype, sizes):
+    M.token_shift(_dev(), dtype, (300, 9, 1, 2), sizes)
+    M.token_shift(_dev(), dtype, (30, 9, 1, 2), sizes, 1048, 3)
+
+
+STATES = pytest.mark.parametrize("dtype,tol", [(torch.float32, 4e-5), (torch.bfloat16, 2e-2)])
+
+
+@STATES
+@pytest.mark.parametrize("sizes", [(1000,), (1,), (2,), (1, 40, 3, 17), (64, 200, 16, 65)])
+@pytest.mark.parametrize("H,P,N,G,parts,taps", [(4, 12, 20, 2, 3, 3), (8, 64, 128, 1, 1, 4), (6, 32, 64, 3, 2, 2)])
+def test_state_space(dtype, tol, H, P, N, G, parts, taps, sizes):
+    """Token by token, in chunks, and both in one batch."""
+    n = 70 if max(sizes) < 3 else 300
+    M.state_space(_dev(), dtype, tol, H, P, N, G, parts, taps, (n, 33, 1, 130, 6), sizes)
+
+
+@STATES
+@pytest.mark.parametrize("H,P,N,G,parts,taps", [(1, 200, 256, 1, 1, 8), (2, 136, 300, 2, 4, 5), (3, 21, 33, 1, 3, 1), (2, 128, 96, 2, 1, 4),
+                                                (2, 72, 200, 1, 6, 7), (64, 64, 16, 8, 1, 4)])
+def test_state_space_sizes(dtype, tol, H, P, N, G, parts, taps):
+    """Columns over several CTAs, sizes without a chunk instance, odd sizes, norm parts that cut through heads."""
+    M.state_space(_dev(), dtype, tol, H, P, N, G, parts, taps, (100, 20, 3), (1000,))
+    M.state_space(_dev(), dtype, tol, H, P, N, G, parts, taps, (20, 3), (1, 2))
+
+
+@STATES
+@pytest.mark.parametrize("dt,rate", [(-6.0, -2.0), (2.0, 2.0), (0.0, 4.0), (-3.0, 0.0)])
+def test_state_space_decays(dtype, tol, dt, rate):
+    M.state_space(_dev(), dtype, tol, 4, 64, 64, 1, 1, 4, (200, 65, 17), (1000,), dt, rate)
+
+
+def test_state_space_long():
+    """Runs of tokens per thread of the convolution that cross from one sequence into the next; many chunks."""
+    M.state_space(_dev(), torch.bfloat16, 2e-2, 2, 64, 64, 1, 1, 4, (900, 3, 500, 1, 99), (4000,), -3.0)
+
+
+TALK = [(6, 3, 20, 64), (16, 4, 128, 128), (4, 4, 64, 64), (1, 1, 64, 64), (3, 1, 100, 128), (32, 8, 128, 128), (24, 2, 64, 64), (13, 13, 64, 64)]
+
+
+@pytest.mark.parametrize("window", [40, 64, 1, 129, 0])
+@pytest.mark.parametrize("decode", [False, True])
+@pytest.mark.parametrize("H,G,d,padded", TALK)
+def test_talking_edges(H, G, d, padded, decode, window):
+    """The prompt kernel (units of one head and of two, several blocks of queries) and the decode kernels."""
+    M.talking_edges(_dev(), torch.bfloat16, 1.5e-2, H, G, d, padded, window, decode)
+
+
+@pytest.mark.parametrize("H,G,d,padded", TALK + [(20, 20, 64, 64), (40, 8, 64, 64), (4, 2, 200, 256), (2, 1, 264, 264), (18, 1, 64, 64)])
+def test_talking_sizes(H, G, d, padded):
+    """Also sizes that only the plain kernel has, portions of a few tokens, and portions beside single tokens."""
+    for decode in (False, True):
+        M.talking_scores(_dev(), torch.bfloat16, 1.5e-2, H, G, d, padded, 70, decode)
+    M.talking_scores(_dev(), torch.bfloat16, 1.5e-2, H, G, d, padded, 70, False, start=148)
+    M.talking_scores(_dev(), torch.bfloat16, 1.5e-2, H, G, d, padded, 70, False, extra=(1, 17, 1, 2))
+    M.talking_prep(_dev(), torch.bfloat16, 1e-2, H, G, d, padded)
+
+
+@pytest.mark.parametrize("window", [40, 1, 0])
+@pytest.mark.parametrize("decode", [False, True])
+@pytest.mark.parametrize("dtype,tol", [(torch.float32, 2e-5), (torch.bfloat16, 8e-3)])
+def test_talking_plain_kernel(monkeypatch, dtype, tol, decode, window):
+    from xfastertransformer_b200.utils.flags import Env
+    monkeypatch.setenv("XFT_TALKING_TC", "0")
+    Env.get().reload()
+    M.talking_edges(_dev(), dtype, tol, 6, 3, 20, 20 if dtype == torch.float32 else 64, window, decode)
+    M.talking_scores(_dev(), dtype, tol, 5, 1, 33, 33, window, decode)
+    M.talking_prep(_dev(), dtype, tol, 5, 1, 33, 33)
+
+
+@pytest.mark.parametrize("decode", [False, True])
+def test_talking_far_keys(decode):
+    """A key thousands of positions back, just inside and just outside a wide window; decode steps split over many ranges."""
+    M.talking_edges(_dev(), torch.bfloat16, 1.5e-2, 16, 4, 128, 128, 1900, decode, T=2100, start=2050)
+    M.talking_scores(_dev(), torch.bfloat16, 1.5e-2, 32, 8, 128, 128, 1000, decode, T=1300, start=1240)
+
+
+@FORMS
+@pytest.mark.parametrize("sizes", [dict(), dict(H=2, d=208, rd=80, R=520, dv=144), dict(H=33, d=64, rd=64, R=512, dv=64), dict(H=4, d=16, rd=2, R=12, dv=8)])
+def test_latent_sinks(monkeypatch, form, sizes):
+    decode, extra = _form(monkeypatch, form)
+    M.latent_sinks(_dev(), torch.bfloat16, 1.5e-2, decode, extra=extra, **sizes)
+
+
+def test_latent_sinks_long_context(monkeypatch):
+    """Contexts split over the CTAs of a cluster and over clusters: the sink counts in one of them."""
+    for form in ("decode", "portion"):
+        decode, _ = _form(monkeypatch, form)
+        M.latent_sinks(_dev(), torch.bfloat16, 2e-2, decode, T=2500, H=3, start=2495)
+
+
+@pytest.mark.parametrize("decode", [False, True])
+def test_latent_sinks_fp32(decode):
+    M.latent_sinks(_dev(), torch.float32, 1e-5, decode)
+
+
+@pytest.mark.parametrize("H", [72, 100, 256, 1021, 2048, 5120, 9000])
+def test_sum_norm(H):
+    M.sum_norm(_dev(), H, torch.bfloat16, 4e-6)
+    M.sum_norm(_dev(), H, torch.float32, 4e-6)
+    M.sum_norm(_dev(), H, torch.bfloat16, 4e-6, T=400)
+
+
+@pytest.mark.parametrize("T", [1, 16, 40, 100, 300, 2000])
+@pytest.mark.parametrize("K,N", [(96, 8), (256, 24), (2048, 128), (2048, 256)])
+def test_clamped_gate_and_activations(T, K, N):
+    """The epilogues of every product kernel: weight stream, tiles, token-major; and in 32 bits."""
+    M.clamped_gate(_dev(), torch.bfloat16, 8e-3, T, K, N, 0.7)
+    M.clamped_gate(_dev(), torch.float32, 1e-5, T, K, N, 7.0)
+    M.activations(_dev(), torch.bfloat16, 8e-3, T, K, N)
+    M.activations(_dev(), torch.float32, 1e-5, T, K, N)
+    M.linear_parts(_dev(), torch.bfloat16, 8e-3, T, K, N)
+    M.linear_parts(_dev(), torch.float32, 1e-5, T, K, N)
+
+
+@pytest.mark.parametrize("T,E,top,ff", [(9, 6, 2, 24), (1, 7, 7, 8), (300, 32, 3, 64), (200, 1, 1, 136)])
+@pytest.mark.parametrize("dtype,tol", [(torch.float32, 3e-6), (torch.bfloat16, 1e-2)])
+def test_chosen_experts(dtype, tol, T, E, top, ff):
+    M.chosen_experts(_dev(), dtype, tol, T, E, top, ff)
+
+
 # ------------------------------------------------------------------------------------------ whole models
 BOTH = pytest.mark.parametrize("dtype", ["fp32", "bf16"])
 
@@ -315,7 +467,7 @@ def test_whole_prompt(cases, name, dtype):
 
 
 @BOTH
-@pytest.mark.parametrize("name", ["unequal", "heads128", "latent", "latent128", "recurrent", "recurrent128", "recurrent_bare"])
+@pytest.mark.parametrize("name", ["unequal", "heads128", "latent", "latent128", "recurrent", "recurrent128", "recurrent_bare"] + C.MIXED_HEADS)
 def test_first_tokens(cases, name, dtype):
     C.first_tokens(cases(name), dtype)
 
@@ -324,38 +476,40 @@ def test_first_tokens(cases, name, dtype):
 @pytest.mark.parametrize("name,start", [("unequal", 1), ("heads128", 40), ("padded", 70), ("shared", 1), ("bare", 100),
                                         ("latent", 1), ("latent128", 40), ("latent_bare", 30), ("latent_large", 100),
                                         ("recurrent", 1), ("recurrent128", 40), ("recurrent_bare", 30), ("recurrent_fast", 1),
-                                        ("recurrent_large", 100)])
+                                        ("recurrent_large", 100), ("mixed_heads", 1), ("mixed_heads128", 40),
+                                        ("mixed_heads_bare", 30), ("mixed_heads_large", 100)])
 def test_token_by_token(cases, name, start, dtype):
     C.token_by_token(cases(name), dtype, 140, start)
 
 
 @BOTH
 @pytest.mark.parametrize("sizes", [(2,), (3, 64, 1), (17, 29)])
-@pytest.mark.parametrize("name", ["unequal", "heads128", "latent", "latent128", "recurrent", "recurrent128", "recurrent_fast"])
+@pytest.mark.parametrize("name", ["unequal", "heads128", "latent", "latent128", "recurrent", "recurrent128", "recurrent_fast", "mixed_heads",
+                                  "mixed_heads128", "mixed_heads_large"])
 def test_portions(cases, name, sizes, dtype):
     C.portions(cases(name), dtype, 140, sizes)
 
 
 @BOTH
-@pytest.mark.parametrize("name", ["unequal", "heads128", "shared", "large_heads"] + C.LATENT + C.RECURRENT)
+@pytest.mark.parametrize("name", ["unequal", "heads128", "shared", "large_heads"] + C.LATENT + C.RECURRENT + C.MIXED_HEADS)
 def test_mixed_batches_reuse_pages(cases, name, dtype):
     assert C.mixed_batches(cases(name), dtype) > 8
 
 
 @BOTH
-@pytest.mark.parametrize("name", ["unequal", "heads128", "latent", "recurrent"])
+@pytest.mark.parametrize("name", ["unequal", "heads128", "latent", "recurrent", "mixed_heads"])
 def test_rows_and_order(cases, name, dtype):
     C.rows_and_order(cases(name), dtype)
 
 
 @BOTH
-@pytest.mark.parametrize("name", ["unequal", "heads128", "padded", "latent", "latent128", "recurrent", "recurrent128"])
+@pytest.mark.parametrize("name", ["unequal", "heads128", "padded", "latent", "latent128", "recurrent", "recurrent128", "mixed_heads", "mixed_heads128"])
 def test_greedy_generation(cases, name, dtype):
     """generate(): the captured decode step (CUDA graph) included."""
     C.greedy(cases(name), dtype, 20, 130)
 
 
-@pytest.mark.parametrize("name", ["heads128", "latent128", "recurrent128"])
+@pytest.mark.parametrize("name", ["heads128", "latent128", "recurrent128", "mixed_heads128"])
 def test_graph_and_eager_steps_agree(cases, monkeypatch, name):
     c = cases(name)
     a = C.greedy(c, "bf16", 30, 60)

@@ -317,6 +317,70 @@ def test_safetensors_types_and_odd_offsets(tmp_path):
     assert torch.equal(st.read("a", (2, 3)), a) and torch.equal(st.read("b", (3,)), b) and torch.equal(st.read("c", (5,)), c)
 
 
+# ------------------------------------------------------------------------------------------ Dagezen's mechanisms
+@pytest.mark.parametrize("sizes", [(1000,), (1,), (1, 40, 3, 17)])
+def test_time_mix(sizes):
+    M.time_mix(CPU, torch.float32, 4e-5, 2, 12, 5, (70, 33, 1, 6), sizes)
+
+
+@pytest.mark.parametrize("sizes", [(1000,), (1,), (2,), (1, 5, 3)])
+def test_token_shift(sizes):
+    M.token_shift(CPU, torch.float32, (30, 9, 1, 2), sizes)
+
+
+@pytest.mark.parametrize("sizes", [(1000,), (1,), (1, 40, 3, 17)])
+@pytest.mark.parametrize("H,P,N,G,parts,taps", [(4, 12, 20, 2, 3, 3), (2, 8, 5, 1, 1, 1), (3, 16, 24, 3, 4, 7)])
+def test_state_space(H, P, N, G, parts, taps, sizes):
+    M.state_space(CPU, torch.float32, 4e-5, H, P, N, G, parts, taps, (70, 33, 1, 6), sizes)
+
+
+@pytest.mark.parametrize("window", [40, 64, 1, 129, 0])
+@pytest.mark.parametrize("decode", [False, True])
+def test_talking_edges(window, decode):
+    M.talking_edges(CPU, torch.float32, 2e-5, 6, 3, 20, 20, window, decode)
+
+
+def test_talking_scores_and_prep():
+    M.talking_scores(CPU, torch.float32, 2e-5, 4, 1, 24, 24, 33, False)
+    M.talking_prep(CPU, torch.float32, 1e-5, 5, 1, 20, 20)
+
+
+@pytest.mark.parametrize("decode", [False, True])
+def test_latent_sinks(decode):
+    M.latent_sinks(CPU, torch.float32, 2e-5, decode)
+
+
+def test_sum_norm_gates_and_experts():
+    M.sum_norm(CPU, 90, torch.float32, 4e-6)
+    M.clamped_gate(CPU, torch.float32, 1e-5, 9, 40, 24, 0.7)
+    M.activations(CPU, torch.float32, 1e-5, 9, 40, 24)
+    M.linear_parts(CPU, torch.float32, 1e-5, 9, 40, 24)
+    M.chosen_experts(CPU, torch.float32, 1e-5, 30, 6, 3, 20)
+
+
+def test_dagezen_config_is_read_per_layer(tmp_path):
+    cfg = O.dagezen([O.mamba_layer(heads=6, vdim=10, state=14, groups=3, norm_groups=5, conv=2, mlp=O.clamped(30, 0.25)),
+                     O.sink_latent_layer(heads=5, dim=14, rot_dim=6, vdim=18, kv_rank=22, base=77.0, scale=0.4, mlp=O.chosen_moe(12, 9, 4)),
+                     O.parallel_layer(heads=6, kv_heads=2, dim=20, size=11, scale=0.3, right_heads=7, right_dim=9, scales=(0.2, 3.0))],
+                    eps=2e-3, alpha=1.25, cap=9.5)
+    c = ModelConfig.load(_write(tmp_path, cfg))
+    a, b, p = c.layers
+    assert (c.model_type, c.residual_carry, c.logit_softcap, c.layernorm_eps) == ("dagezen", 1.25, 9.5, 2e-3)
+    m = a.mixer
+    assert (m.kind, m.heads, m.vdim, m.dim, m.groups, m.norm_groups, m.conv, m.has_kv) == ("ssd", 6, 10, 14, 3, 5, 2, False)
+    assert (a.ff, a.act, a.limit, a.ff_bias) == (30, "clamped", 0.25, True)
+    m = b.mixer
+    assert (m.kind, m.gate, m.head_gate, m.sinks, m.window, m.scale, m.rot.style, m.rot.base) == ("latent", True, True, True, 0, 0.4, "interleaved", 77.0)
+    assert (b.moe.act, b.moe.scoring, b.moe.router_bias, b.moe.shared, b.moe.experts, b.moe.top) == ("gelu_erf", "chosen", True, 0, 9, 4)
+    l, r = p.mixer.parts
+    assert p.mixer.part_scales == (0.2, 3.0) and p.mixer.has_kv and (l.kind, l.heads, l.kv_heads, l.dim, l.window, l.scale) == ("talking", 6, 2, 20, 11, 0.3)
+    assert (r.kind, r.heads, r.dim, r.has_kv) == ("time_mix", 7, 9, False) and p.ff == 0 and p.moe is None
+    with pytest.raises(ValueError, match="groups"):
+        ModelConfig.from_dict(O.dagezen([O.mamba_layer(heads=4, groups=3)]))
+    with pytest.raises(ValueError, match="int8"):
+        xft.AutoModel.from_pretrained(str(tmp_path / "m"), dtype="bf16", kv_cache_dtype="int8")
+
+
 # ------------------------------------------------------------------------------------------ limits and refusals
 def test_fixed_pools_refuse_what_does_not_fit(tmp_path):
     cfg = O.config([O.attention_layer(), O.attention_layer(kv_from=0, size=5)])

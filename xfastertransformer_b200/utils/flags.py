@@ -79,6 +79,7 @@ class Env:
         self.latent_expand_min_q = _int("XFT_LATENT_EXPAND_MIN_Q", 16)   # prompt portions from this size on expand their latents
         self.gla_chunk_min_q = _int("XFT_GLA_CHUNK_MIN_Q", 16)    # gated linear attention: portions from this size on go in chunks
         self.ssd_chunk_min_q = _int("XFT_SSD_CHUNK_MIN_Q", 16)    # the same of state-space layers
+        self.talking_tc = _int("XFT_TALKING_TC", 1) != 0          # attention with mixed heads on the tensor cores (0: plain kernel)
         self.gemm_streamk = _int("XFT_GEMM_STREAMK", 1) != 0
         self.fuse_qkv_rope = _int("XFT_FUSE_QKV_ROPE", 1) != 0
         # tensor-parallel prefill: two groups of prompts are interleaved block by block, so that the all-reduce of one
