@@ -550,6 +550,21 @@ int make_tensor_map(CUtensorMap* out, const void* ptr, uint64_t rows, uint64_t c
   return 0;
 }
 
+// bf16 array [groups, rows, cols] without gaps; box = 64 columns x box_rows x box_groups, 128B swizzle.
+int make_tensor_map_groups(CUtensorMap* out, const void* ptr, uint64_t groups, uint64_t rows, uint64_t cols, uint32_t box_groups,
+                           uint32_t box_rows) {
+  EncodeTiledFn enc = get_encode();
+  if (!enc) return -1;
+  if ((reinterpret_cast<uintptr_t>(ptr) & 15) || (cols & 63) || box_groups > 256 || box_rows > 256) return -2;
+  cuuint64_t dims[3] = {cols, rows, groups};
+  cuuint64_t strides[2] = {cols * 2, rows * cols * 2};
+  cuuint32_t box[3] = {64, box_rows, box_groups};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                   CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -3;
+}
+
 template <int BN, bool DUAL>
 static int launch_gemm(const CUtensorMap& tmW, const CUtensorMap& tmX, GemmParams& p, cudaStream_t st) {
   constexpr int STAGE_BYTES = 128 * 64 * 2 * (DUAL ? 2 : 1) + BN * 64 * 2;

@@ -10,7 +10,7 @@
 //   time mixing    alpha_t = exp(-exp(W_a2 a1_t + bias)), o_t = (S_(t-1) + diag(u) k_t v_t^T)^T (q_t scale): the state is read
 //                  before it moves on, and the current token counts with a bonus u per channel
 //   state space    (step kernel) one decay exp(-rate dt) per head and token, k scaled by dt = softplus(raw + bias), q and k shared by
-//                  groups of heads; what leaves is o + D v in fp32, its gate and norm follow in a kernel of their own
+//                  groups of heads; what leaves is o + D v, its gate and norm follow in a kernel of their own
 //
 // Rows of x are packed [q | k | v | g | a1] (queries, keys, values and gate of all heads, the decay's first product).  A
 // sequence's state lives in its slot of a pool [slots, heads, dim, vdim]; its first token starts from zero whatever the slot
@@ -191,7 +191,8 @@ __global__ void __launch_bounds__(kStepThreads) gla_step_kernel(const GlaParams 
     }
     if (MODE == kStateSpace) {
       if (mine)
-        p.raw[(size_t)(start + i) * p.heads * p.vdim + h * p.vdim + col] = fmaf(p.skip[h], gl_f32<T>(row[p.v_at + h * p.vdim + col]), y);
+        reinterpret_cast<T*>(p.out)[(size_t)(start + i) * p.heads * p.vdim + h * p.vdim + col] =
+            gl_from<T>(fmaf(p.skip[h], gl_f32<T>(row[p.v_at + h * p.vdim + col]), y));
       continue;
     }
     float ss = mine ? y * y : 0.f;
@@ -825,10 +826,11 @@ extern "C" int xft_gla_step(const void* x, int ldx, int k_at, int v_at, int g_at
 }
 
 // The recurrence of a state-space layer, token by token: x rows hold q, k (groups x dim each) and v (heads x vdim) from columns q_at,
-// k_at and v_at; dt [T, ld_dt] raw step sizes of the rows' type; dt_bias, rate, skip fp32 [heads]; raw fp32 [T, heads * vdim] out.
+// k_at and v_at; dt [T, ld_dt] raw step sizes of the rows' type; dt_bias, rate, skip fp32 [heads]; out [T, heads * vdim]
+// of the rows' type.
 extern "C" int xft_ssd_step(const void* x, int ldx, int q_at, int k_at, int v_at, int heads, int heads_per_group, int dim, int vdim,
                             const void* dt, int ld_dt, const float* dt_bias, const float* rate, const float* skip, float* state,
-                            const int* state_slots, int num_states, const int* cu_q, const int* kv_lens, int B, float* raw, int min_q,
+                            const int* state_slots, int num_states, const int* cu_q, const int* kv_lens, int B, void* out, int min_q,
                             int max_q, int columns, int f32, int* status, cudaStream_t st) {
   if (B <= 0) return 0;
   if (heads <= 0 || dim <= 0 || vdim <= 0 || heads_per_group <= 0 || heads % heads_per_group || num_states <= 0 || columns <= 0) return -1;
@@ -837,7 +839,7 @@ extern "C" int xft_ssd_step(const void* x, int ldx, int q_at, int k_at, int v_at
   p.x = x; p.ldx = ldx; p.q_at = q_at; p.k_at = k_at; p.v_at = v_at; p.heads = heads; p.heads_per_group = heads_per_group;
   p.dim = dim; p.vdim = vdim; p.dt = dt; p.ld_dt = ld_dt; p.dt_bias = dt_bias; p.rate = rate; p.skip = skip;
   p.state = state; p.state_slots = state_slots; p.num_states = num_states; p.cu_q = cu_q; p.kv_lens = kv_lens; p.B = B;
-  p.raw = raw; p.min_q = min_q; p.max_q = max_q; p.segs = 1; p.status = status;
+  p.out = out; p.min_q = min_q; p.max_q = max_q; p.segs = 1; p.status = status;
   return f32 ? step_columns<float, kStateSpace>(p, columns, st) : step_columns<bf16, kStateSpace>(p, columns, st);
 }
 

@@ -47,6 +47,11 @@ __device__ __forceinline__ int ss_slot(const int* slots, int b, int num, int* st
   return 0;
 }
 
+// x * sigmoid(x): accurate in fp32, with the approximate instructions for bf16 results
+template <typename T> __device__ __forceinline__ float ss_silu(float x);
+template <> __device__ __forceinline__ float ss_silu<float>(float x) { return x / (1.f + expf(-x)); }
+template <> __device__ __forceinline__ float ss_silu<bf16>(float x) { return x * gl_rcp(1.f + gl_ex2(-x * 1.4426950408889634f)); }
+
 // ------------------------------------------------------------------------------------------ convolution over time
 struct ChannelConvParams {
   const void* x; int ldx; int T, B, C, taps;               // x points at the first channel
@@ -83,6 +88,7 @@ __global__ void __launch_bounds__(128) channel_conv_kernel(const ChannelConvPara
   int b = ss_sequence(p.cu_q, p.B, t0), start = p.cu_q[b], end = p.cu_q[b + 1];
   bool fresh = true;
   float u[TAPS][VEC];
+  V next = *reinterpret_cast<const V*>(x + (size_t)t0 * p.ldx);        // the row ahead is on its way while one is summed up
   for (int t = t0; t < t1; ++t) {
     while (b + 1 < p.B && t >= end) { ++b; start = end; end = p.cu_q[b + 1]; fresh = true; }
     const int li = t - start;
@@ -103,14 +109,16 @@ __global__ void __launch_bounds__(128) channel_conv_kernel(const ChannelConvPara
       }
       fresh = false;
     }
-    load(x + (size_t)t * p.ldx, u[TAPS - 1]);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) u[TAPS - 1][k] = ss_f32<T>(next.e[k]);
+    if (t + 1 < t1) next = *reinterpret_cast<const V*>(x + (size_t)(t + 1) * p.ldx);
     V y;
 #pragma unroll
     for (int k = 0; k < VEC; ++k) {
       float a = bias[k];
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) a = fmaf(w[j][k], u[j][k], a);
-      y.e[k] = ss_from<T>(a / (1.f + expf(-a)));
+      y.e[k] = ss_from<T>(ss_silu<T>(a));
     }
     *reinterpret_cast<V*>(reinterpret_cast<T*>(p.out) + (size_t)t * p.ldo + c) = y;
     if (p.decode && p.taps > 1) {                          // rows 1 .. taps - 1 of the window are the new state
@@ -131,20 +139,65 @@ __global__ void __launch_bounds__(128) channel_conv_kernel(const ChannelConvPara
 }
 
 // ------------------------------------------------------------------------------------------ gate and grouped norm
-// One CTA per (token, part).  A thread keeps up to 16 values; wider parts are read again.
+// One CTA per (token, part); a thread has 8 neighbouring values up to twice.
+__global__ void __launch_bounds__(256) gated_norm_vec_kernel(const bf16* __restrict__ y, int ldy, const bf16* __restrict__ z, int ldz,
+                                                             const float* __restrict__ gain, bf16* __restrict__ out, int ldo, int n, float eps) {
+  __shared__ float sh[8];
+  const int t = blockIdx.y, c0 = blockIdx.x * n, nt = blockDim.x;
+  grid_dep_launch();
+  grid_dep_wait();
+  const bf16* yr = y + (size_t)t * ldy + c0;
+  const bf16* zr = z + (size_t)t * ldz + c0;
+  uint4 a[2], b[2];
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    const int i = (threadIdx.x + k * nt) * 8;
+    a[k] = b[k] = make_uint4(0, 0, 0, 0);
+    if (i < n) { a[k] = *reinterpret_cast<const uint4*>(yr + i); b[k] = *reinterpret_cast<const uint4*>(zr + i); }
+  }
+  float v[16], ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < 2; ++k)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 p = gl_unpack(reinterpret_cast<const uint32_t*>(&a[k])[j]), q = gl_unpack(reinterpret_cast<const uint32_t*>(&b[k])[j]);
+      v[k * 8 + 2 * j] = p.x * ss_silu<bf16>(q.x);
+      v[k * 8 + 2 * j + 1] = p.y * ss_silu<bf16>(q.y);
+      ss = fmaf(v[k * 8 + 2 * j], v[k * 8 + 2 * j], fmaf(v[k * 8 + 2 * j + 1], v[k * 8 + 2 * j + 1], ss));
+    }
+#pragma unroll
+  for (int m = 16; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+  if ((threadIdx.x & 31) == 0) sh[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  ss = 0.f;
+  for (int i = 0; i < (nt >> 5); ++i) ss += sh[i];
+  const float inv = rsqrtf(ss / (float)n + eps);
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    const int i = (threadIdx.x + k * nt) * 8;
+    if (i >= n) continue;
+    const float4 g0 = *reinterpret_cast<const float4*>(gain + c0 + i), g1 = *reinterpret_cast<const float4*>(gain + c0 + i + 4);
+    const float* w = v + k * 8;
+    uint4 r;
+    r.x = gl_pack(w[0] * inv * g0.x, w[1] * inv * g0.y);
+    r.y = gl_pack(w[2] * inv * g0.z, w[3] * inv * g0.w);
+    r.z = gl_pack(w[4] * inv * g1.x, w[5] * inv * g1.y);
+    r.w = gl_pack(w[6] * inv * g1.z, w[7] * inv * g1.w);
+    *reinterpret_cast<uint4*>(out + (size_t)t * ldo + c0 + i) = r;
+  }
+}
+
+// Any size: a thread keeps up to 16 values; wider parts are read again.
 template <typename T>
-__global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict__ y, int ldy, const T* __restrict__ z, int ldz,
+__global__ void __launch_bounds__(256) gated_norm_kernel(const T* __restrict__ y, int ldy, const T* __restrict__ z, int ldz,
                                                          const float* __restrict__ gain, T* __restrict__ out, int ldo, int n, float eps) {
   __shared__ float sh[8];
   grid_dep_launch();
   grid_dep_wait();
   const int t = blockIdx.y, c0 = blockIdx.x * n, nt = blockDim.x;
-  const float* yr = y + (size_t)t * ldy + c0;
+  const T* yr = y + (size_t)t * ldy + c0;
   const T* zr = z + (size_t)t * ldz + c0;
-  auto value = [&](int i) {
-    const float g = ss_f32<T>(zr[i]);
-    return yr[i] * (g / (1.f + expf(-g)));
-  };
+  auto value = [&](int i) { return ss_f32<T>(yr[i]) * ss_silu<T>(ss_f32<T>(zr[i])); };
   float v[16], ss = 0.f;
 #pragma unroll
   for (int k = 0; k < 16; ++k) {
@@ -208,42 +261,50 @@ struct SsdChunkParams {
   int heads, per_group, state_n, vdim;
   float* state; const int* state_slots; int num_states;
   const int* cu_q; const int* kv_lens;
-  float* y;                                                // [T, heads * vdim]
+  bf16* y;                                                 // [T, heads * vdim]
   int min_q;
+  int segs, carry;                                         // segments per portion; carry: the launch that runs the states alone
+  float* seg_state;                                        // [B, heads, segs, state, vdim]: the initial state, then what segment j - 1 leaves
+  float* seg_decay;                                        // [B, heads, segs]: sum of log2 of the decays of segment j - 1
   int* status;
 };
 
-constexpr int kSsdChunk = 64, kSsdThreads = 256;
-template <int NP, int VS>
+constexpr int kSsdChunk = 64, kSsdThreads = 256;           // threads per head
+template <int NP, int VS, int HPC>
 struct SsdCfg {
   static constexpr int NS = NP + 8, XS = VS + 8, AS = kSsdChunk + 8;
-  static constexpr int STAGE = kSsdChunk * (2 * NS + XS);                  // C, B, x of a chunk
+  static constexpr int STAGE = kSsdChunk * (2 * NS + HPC * XS);            // C, B, x of every head of a chunk
   static constexpr int STAGES = NP <= 128 ? 2 : 1;
-  static constexpr size_t SMEM = ((size_t)STAGES * STAGE + kSsdChunk * XS + NP * XS + kSsdChunk * AS) * 2 + 2 * kSsdChunk * 4;
+  static constexpr int HEAD = kSsdChunk * XS + NP * XS + kSsdChunk * AS;   // of a head: x with its factor, the state, scores
+  static constexpr size_t SMEM = ((size_t)STAGES * STAGE + HPC * HEAD) * 2 + HPC * 2 * kSsdChunk * 4;
   static_assert(SMEM <= 227 * 1024, "shared memory");
 };
 
-template <int NP, int VS>
-__global__ void __launch_bounds__(kSsdThreads, 1) ssd_chunk_kernel(const SsdChunkParams p) {
-  using Cfg = SsdCfg<NP, VS>;
-  constexpr int NT = kSsdThreads, NS = Cfg::NS, XS = Cfg::XS, AS = Cfg::AS;
+// A CTA takes HPC heads that share B and C, with eight warps each.
+template <int NP, int VS, int HPC>
+__global__ void __launch_bounds__(kSsdThreads * HPC, 1) ssd_chunk_kernel(const SsdChunkParams p) {
+  using Cfg = SsdCfg<NP, VS, HPC>;
+  constexpr int NT = kSsdThreads * HPC, NS = Cfg::NS, XS = Cfg::XS, AS = Cfg::AS;
   constexpr int MT = NP / 16, SPLIT = MT < 8 ? 8 / MT : 1, MPW = MT < 8 ? 1 : MT / 8;    // the state: row tiles, column parts, tiles per warp
   constexpr int NSW = VS / 8 / SPLIT;                      // its 8-column tiles per warp
   constexpr int NO = VS / 16;                              // 8-column tiles of half the output columns
   static_assert(NSW % 2 == 0 && NO % 2 == 0, "warp tiles");
   extern __shared__ __align__(16) uint8_t sc_raw[];
+  const int tid = threadIdx.x, lane = tid & 31, hw = tid / kSsdThreads, ht = tid % kSsdThreads, warp = ht >> 5;
   bf16* stage0 = reinterpret_cast<bf16*>(sc_raw);
-  bf16* sX2 = stage0 + Cfg::STAGES * Cfg::STAGE;           // x with its factor of the state's update
+  bf16* sX2 = stage0 + Cfg::STAGES * Cfg::STAGE + hw * Cfg::HEAD;          // x with its factor of the state's update
   bf16* sS = sX2 + kSsdChunk * XS;                         // the state as an operand [NP][XS]
   bf16* sA = sS + NP * XS;                                 // scores [64][AS]
-  float* sL = reinterpret_cast<float*>(sA + kSsdChunk * AS);          // running sums, base 2
+  float* sL = reinterpret_cast<float*>(stage0 + Cfg::STAGES * Cfg::STAGE + HPC * Cfg::HEAD) + hw * 2 * kSsdChunk;   // running sums, base 2
   float* sDt = sL + kSsdChunk;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int h = blockIdx.y, b = blockIdx.z, v0 = blockIdx.x * VS;
+  const int h = blockIdx.y * HPC + hw, b = blockIdx.z, seg = blockIdx.x % p.segs, v0 = blockIdx.x / p.segs * VS;
   grid_dep_launch();
   const int start = p.cu_q[b], n = p.cu_q[b + 1] - start;
-  if (n < p.min_q || n <= 0) { grid_dep_wait(); return; }
-  const int chunks = (n + kSsdChunk - 1) / kSsdChunk, past = p.kv_lens[b] - n;
+  const int chunks = (n + kSsdChunk - 1) / kSsdChunk, per_seg = (chunks + p.segs - 1) / p.segs;
+  const int ch0 = seg * per_seg, ch1 = min(ch0 + per_seg, chunks);         // this CTA's chunks
+  if (n < p.min_q || n <= 0 || ch0 >= chunks || (p.carry && ch1 == chunks)) { grid_dep_wait(); return; }
+  const bool alone = per_seg >= chunks;                    // one segment has all of the portion
+  const int past = p.kv_lens[b] - n;
   const int N = p.state_n, vw = min(VS, p.vdim - v0);
   const bool whole8 = (N & 7) == 0 && (p.vdim & 7) == 0 && (p.ldu & 7) == 0 && (p.b_at & 7) == 0 && (p.c_at & 7) == 0;
   float* st = p.state + ((size_t)ss_slot(p.state_slots, b, p.num_states, p.status) * p.heads + h) * N * p.vdim;
@@ -251,61 +312,79 @@ __global__ void __launch_bounds__(kSsdThreads, 1) ssd_chunk_kernel(const SsdChun
   // the state: MPW tiles of 16 rows, NSW x 8 columns; element e of tile (m, j): row sd + 128 m + 8 (e >> 1), column sc + 8 j + (e & 1)
   const int sd = (warp % (MT < 8 ? MT : 8)) * 16 + (lane >> 2), sn0 = MT < 8 ? warp / MT * NSW * 8 : 0, sc = sn0 + 2 * (lane & 3);
   float S[MPW][NSW][4];
+  auto each_state = [&](auto f) {
 #pragma unroll
-  for (int m = 0; m < MPW; ++m)
+    for (int m = 0; m < MPW; ++m)
 #pragma unroll
-    for (int j = 0; j < NSW; ++j)
+      for (int j = 0; j < NSW; ++j)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int d = sd + m * 128 + (e >> 1) * 8, c = sc + j * 8 + (e & 1);
-        S[m][j][e] = past > 0 && d < N && c < vw ? st[(size_t)d * p.vdim + v0 + c] : 0.f;
-      }
+        for (int e = 0; e < 4; ++e) {
+          const int d = sd + m * 128 + (e >> 1) * 8, c = sc + j * 8 + (e & 1);
+          f(S[m][j][e], (size_t)d * p.vdim + v0 + c, d < N && c < vw);
+        }
+  };
+  each_state([&](float& v, size_t at, bool in) { v = past > 0 && seg == 0 && (alone || p.carry) && in ? st[at] : 0.f; });
   const float rate2 = p.rate[h] * 1.4426950408889634f, skip = p.skip[h], dtb = p.dt_bias[h];
   grid_dep_wait();
+  float* seg_s = p.seg_state + ((size_t)b * p.heads + h) * p.segs * N * p.vdim;
+  float* seg_d = p.seg_decay + ((size_t)b * p.heads + h) * p.segs;
+  float carried = 0.f;                                     // carry: sum of the logarithms over the segment
+  if (p.carry && seg == 0) {                               // the pool is written while later segments still start: keep a copy
+    each_state([&](float& v, size_t at, bool in) { if (in) seg_s[at] = v; });
+  } else if (!alone && !p.carry) {
+    for (int k = seg == 0 ? 0 : 1; k <= seg; ++k) {
+      const float f = k > 1 ? gl_ex2(seg_d[k]) : 1.f;
+      const float* from = seg_s + (size_t)k * N * p.vdim;
+      each_state([&](float& v, size_t at, bool in) { v = fmaf(v, f, in ? from[at] : 0.f); });
+    }
+  }
   __syncthreads();
   const bf16* u = p.u + (size_t)start * p.ldu;
-  const int kg = h / p.per_group;
+  const int kg = h / p.per_group;                          // the same for all heads of the CTA
   auto load = [&](int ch) {
     bf16* sC = stage0 + (Cfg::STAGES > 1 ? (ch & 1) * Cfg::STAGE : 0);
     bf16* sB = sC + kSsdChunk * NS;
-    bf16* sX = sB + kSsdChunk * NS;
+    bf16* sX = sB + kSsdChunk * NS + hw * kSsdChunk * XS;
     const int t0 = ch * kSsdChunk, rows = min(kSsdChunk, n - t0);
-    auto part = [&](bf16* dst, int ld, int at, int width) {
+    auto part = [&](bf16* dst, int ld, int at, int width, int id, int nt) {
       if (whole8) {
-        const int per = width >> 3;
-        for (int i = tid; i < kSsdChunk * per; i += NT) {
-          const int r = i / per, c = i - r * per;
+        const int per = width >> 3, dr = nt / per, dc = nt % per;
+        int r = id / per, c = id % per;
+        while (r < kSsdChunk) {
           const bf16* src = u + (size_t)(t0 + min(r, rows - 1)) * p.ldu + at + c * 8;
           const int bytes = r < rows ? 16 : 0;
           asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + r * ld + c * 8)), "l"(src), "r"(bytes) : "memory");
+          r += dr;
+          c += dc;
+          if (c >= per) { c -= per; ++r; }
         }
       } else {
-        for (int i = tid; i < kSsdChunk * width; i += NT) {
+        for (int i = id; i < kSsdChunk * width; i += nt) {
           const int r = i / width, c = i - r * width;
           dst[r * ld + c] = r < rows ? u[(size_t)(t0 + r) * p.ldu + at + c] : __float2bfloat16(0.f);
         }
       }
     };
-    part(sC, NS, p.c_at + kg * N, N);
-    part(sB, NS, p.b_at + kg * N, N);
-    part(sX, XS, h * p.vdim + v0, vw);
+    if (!p.carry) part(sC, NS, p.c_at + kg * N, N, tid, NT);
+    part(sB, NS, p.b_at + kg * N, N, tid, NT);
+    part(sX, XS, h * p.vdim + v0, vw, ht, kSsdThreads);
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  auto raw_dt = [&](int ch) {                              // of token tid of a chunk
-    const int t = ch * kSsdChunk + tid;
-    return tid < kSsdChunk && t < n ? __bfloat162float(p.dt[(size_t)(start + t) * p.ld_dt + h]) + dtb : -INFINITY;
+  auto raw_dt = [&](int ch) {                              // of token ht of a chunk
+    const int t = ch * kSsdChunk + ht;
+    return ht < kSsdChunk && t < n ? __bfloat162float(p.dt[(size_t)(start + t) * p.ld_dt + h]) + dtb : -INFINITY;
   };
   const int fa_r = (lane & 7) + ((lane >> 3) & 1) * 8, fa_c = (lane >> 4) * 8;
   const int fb_r = (lane & 7) + ((lane >> 4) & 1) * 8, fb_c = ((lane >> 3) & 1) * 8;
   const int mt = warp & 3, half = warp >> 2, r0 = mt * 16 + (lane >> 2), cc = 2 * (lane & 3);
-  load(0);
-  float z = raw_dt(0);
-  for (int ch = 0; ch < chunks; ++ch) {
+  load(ch0);
+  float z = raw_dt(ch0);
+  for (int ch = ch0; ch < ch1; ++ch) {
     bf16* sC = stage0 + (Cfg::STAGES > 1 ? (ch & 1) * Cfg::STAGE : 0);
     bf16* sB = sC + kSsdChunk * NS;
-    bf16* sX = sB + kSsdChunk * NS;
+    bf16* sX = sB + kSsdChunk * NS + hw * kSsdChunk * XS;
     const int rows = min(kSsdChunk, n - ch * kSsdChunk);
-    // step sizes and running sums: the first two warps, a token per lane
+    // step sizes and running sums: two warps per head, a token per lane
     if (warp < 2) {
       const float dt = z == -INFINITY ? 0.f : fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
       float L = -rate2 * dt;
@@ -314,58 +393,68 @@ __global__ void __launch_bounds__(kSsdThreads, 1) ssd_chunk_kernel(const SsdChun
         const float v = __shfl_up_sync(0xffffffffu, L, o);
         if (lane >= o) L += v;
       }
-      sL[tid] = L;
-      sDt[tid] = dt;
+      sL[ht] = L;
+      sDt[ht] = dt;
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                       // also: everyone is done with the chunk before
-    if (Cfg::STAGES > 1 && ch + 1 < chunks) load(ch + 1);
-    z = ch + 1 < chunks ? raw_dt(ch + 1) : -INFINITY;
+    if (Cfg::STAGES > 1 && ch + 1 < ch1) load(ch + 1);
+    z = ch + 1 < ch1 ? raw_dt(ch + 1) : -INFINITY;
     const float half_sum = sL[31], end_sum = half_sum + sL[63];
+    carried += end_sum;
     auto sum_at = [&](int t) { return sL[t] + (t >= 32 ? half_sum : 0.f); };
     // x with its factor; the state as an operand; the scores
-    for (int i = tid; i < kSsdChunk * VS / 2; i += NT) {
-      const int r = i / (VS / 2), c = i - r * (VS / 2);
-      const float f = sDt[r] * gl_ex2(end_sum - sum_at(r));
-      const float2 x = gl_unpack(*reinterpret_cast<const uint32_t*>(sX + r * XS + 2 * c));
-      *reinterpret_cast<uint32_t*>(sX2 + r * XS + 2 * c) = gl_pack(x.x * f, x.y * f);
+    {
+      const int c = ht % (VS / 2), dr = kSsdThreads / (VS / 2);
+#pragma unroll 4
+      for (int r = ht / (VS / 2); r < kSsdChunk; r += dr) {
+        const float f = sDt[r] * gl_ex2(end_sum - sum_at(r));
+        const float2 x = gl_unpack(*reinterpret_cast<const uint32_t*>(sX + r * XS + 2 * c));
+        *reinterpret_cast<uint32_t*>(sX2 + r * XS + 2 * c) = gl_pack(x.x * f, x.y * f);
+      }
     }
-#pragma unroll
-    for (int m = 0; m < MPW; ++m)
-#pragma unroll
-      for (int j = 0; j < NSW; ++j) {
-        *reinterpret_cast<uint32_t*>(sS + (sd + m * 128) * XS + sc + j * 8) = gl_pack(S[m][j][0], S[m][j][1]);
-        *reinterpret_cast<uint32_t*>(sS + (sd + m * 128 + 8) * XS + sc + j * 8) = gl_pack(S[m][j][2], S[m][j][3]);
-      }
     const float l0 = sum_at(r0), l1 = sum_at(r0 + 8);
-    for (int kt = half; kt <= mt; kt += 2) {
-      float A[2][4];
+    if (!p.carry) {
 #pragma unroll
-      for (int j = 0; j < 2; ++j) A[j][0] = A[j][1] = A[j][2] = A[j][3] = 0.f;
+      for (int m = 0; m < MPW; ++m)
 #pragma unroll
-      for (int ks = 0; ks < NP / 16; ++ks) {
-        uint32_t a[4], w[4];
-        gl_ldsm(a, sC + (mt * 16 + fa_r) * NS + ks * 16 + fa_c);
-        gl_ldsm(w, sB + (kt * 16 + fb_r) * NS + ks * 16 + fb_c);
-        gl_mma(A[0], a, w[0], w[1]);
-        gl_mma(A[1], a, w[2], w[3]);
-      }
+        for (int j = 0; j < NSW; ++j) {
+          *reinterpret_cast<uint32_t*>(sS + (sd + m * 128) * XS + sc + j * 8) = gl_pack(S[m][j][0], S[m][j][1]);
+          *reinterpret_cast<uint32_t*>(sS + (sd + m * 128 + 8) * XS + sc + j * 8) = gl_pack(S[m][j][2], S[m][j][3]);
+        }
+      // the ten tiles of 16 x 16 scores on and below the diagonal
+      for (int i = warp; i < 10; i += 8) {
+        const int qt = i < 1 ? 0 : i < 3 ? 1 : i < 6 ? 2 : 3, kt = i - qt * (qt + 1) / 2;
+        float A[2][4];
 #pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        const int s = kt * 16 + j * 8 + cc;
-        const float ls0 = sum_at(s), ls1 = sum_at(s + 1), d0 = sDt[s], d1 = sDt[s + 1];
+        for (int j = 0; j < 2; ++j) A[j][0] = A[j][1] = A[j][2] = A[j][3] = 0.f;
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int t = r0 + e * 8;
-          const float lt = e ? l1 : l0;
-          const float a0 = s <= t ? A[j][2 * e] * gl_ex2(lt - ls0) * d0 : 0.f, a1 = s + 1 <= t ? A[j][2 * e + 1] * gl_ex2(lt - ls1) * d1 : 0.f;
-          *reinterpret_cast<uint32_t*>(sA + t * AS + s) = gl_pack(a0, a1);
+        for (int ks = 0; ks < NP / 16; ++ks) {
+          uint32_t a[4], w[4];
+          gl_ldsm(a, sC + (qt * 16 + fa_r) * NS + ks * 16 + fa_c);
+          gl_ldsm(w, sB + (kt * 16 + fb_r) * NS + ks * 16 + fb_c);
+          gl_mma(A[0], a, w[0], w[1]);
+          gl_mma(A[1], a, w[2], w[3]);
+        }
+        const int tq = qt * 16 + (lane >> 2);
+        const float lq0 = sum_at(tq), lq1 = sum_at(tq + 8);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          const int s = kt * 16 + j * 8 + cc;
+          const float ls0 = sum_at(s), ls1 = sum_at(s + 1), d0 = sDt[s], d1 = sDt[s + 1];
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int t = tq + e * 8;
+            const float lt = e ? lq1 : lq0;
+            const float a0 = s <= t ? A[j][2 * e] * gl_ex2(lt - ls0) * d0 : 0.f, a1 = s + 1 <= t ? A[j][2 * e + 1] * gl_ex2(lt - ls1) * d1 : 0.f;
+            *reinterpret_cast<uint32_t*>(sA + t * AS + s) = gl_pack(a0, a1);
+          }
         }
       }
     }
     __syncthreads();
     // y = exp(L) C S + A x + D x: rows of this warp, half the columns
-    {
+    if (!p.carry) {
       float O[NO][4];
 #pragma unroll
       for (int j = 0; j < NO; ++j) O[j][0] = O[j][1] = O[j][2] = O[j][3] = 0.f;
@@ -399,15 +488,15 @@ __global__ void __launch_bounds__(kSsdThreads, 1) ssd_chunk_kernel(const SsdChun
       for (int e = 0; e < 2; ++e) {
         const int r = r0 + e * 8;
         if (r >= rows) continue;
-        float* yr = p.y + (size_t)(start + ch * kSsdChunk + r) * p.heads * p.vdim + h * p.vdim + v0;
+        bf16* yr = p.y + (size_t)(start + ch * kSsdChunk + r) * p.heads * p.vdim + h * p.vdim + v0;
 #pragma unroll
         for (int j = 0; j < NO; ++j) {
           const int c = half * (VS / 2) + j * 8 + cc;
           if (c >= vw) continue;
           const float2 x = gl_unpack(*reinterpret_cast<const uint32_t*>(sX + r * XS + c));
           const float2 v = make_float2(fmaf(skip, x.x, O[j][2 * e]), fmaf(skip, x.y, O[j][2 * e + 1]));
-          if ((p.vdim & 1) == 0) *reinterpret_cast<float2*>(yr + c) = v;
-          else { yr[c] = v.x; if (c + 1 < vw) yr[c + 1] = v.y; }
+          if ((p.vdim & 1) == 0) *reinterpret_cast<uint32_t*>(yr + c) = gl_pack(v.x, v.y);
+          else { yr[c] = __float2bfloat16(v.x); if (c + 1 < vw) yr[c + 1] = __float2bfloat16(v.y); }
         }
       }
     }
@@ -431,17 +520,13 @@ __global__ void __launch_bounds__(kSsdThreads, 1) ssd_chunk_kernel(const SsdChun
       }
     }
     __syncthreads();                                       // the sums, and with one stage the tiles, are written again
-    if (Cfg::STAGES == 1 && ch + 1 < chunks) load(ch + 1);
+    if (Cfg::STAGES == 1 && ch + 1 < ch1) load(ch + 1);
   }
-#pragma unroll
-  for (int m = 0; m < MPW; ++m)
-#pragma unroll
-    for (int j = 0; j < NSW; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int d = sd + m * 128 + (e >> 1) * 8, c = sc + j * 8 + (e & 1);
-        if (d < N && c < vw) st[(size_t)d * p.vdim + v0 + c] = S[m][j][e];
-      }
+  if (p.carry) {
+    st = seg_s + (size_t)(seg + 1) * N * p.vdim;
+    if (v0 == 0 && ht == 0) seg_d[seg + 1] = carried;
+  } else if (ch1 < chunks) return;                         // the last segment leaves the state
+  each_state([&](float& v, size_t at, bool in) { if (in) st[at] = v; });
 }
 
 }  // namespace xft
@@ -479,18 +564,21 @@ extern "C" int xft_channel_conv(const void* x, int ldx, int T, int B, int C, int
   return (int)cudaGetLastError();
 }
 
-// y fp32 [T, ldy], z and out [T, ld] fp32 or bf16, `parts` parts of n columns each, gain fp32 [parts * n].
-extern "C" int xft_gated_norm(const float* y, int ldy, const void* z, int ldz, const float* gain, void* out, int ldo, int T, int parts, int n,
+// y, z and out [T, ld], all fp32 (f32 = 1) or bf16, `parts` parts of n columns each, gain fp32 [parts * n].
+extern "C" int xft_gated_norm(const void* y, int ldy, const void* z, int ldz, const float* gain, void* out, int ldo, int T, int parts, int n,
                               float eps, int f32, cudaStream_t st) {
   if (T <= 0) return 0;
-  if (parts <= 0 || n <= 0 || ldy < parts * n || ldz < parts * n || ldo < parts * n || T > 65535 * 16) return -1;
-  const int nt = n <= 512 ? 64 : n <= 2048 ? 128 : 256;
+  if (parts <= 0 || n <= 0 || ldy < parts * n || ldz < parts * n || ldo < parts * n) return -1;
+  const bool vec = !f32 && n <= 4096 && ((n | ldy | ldz | ldo) & 7) == 0 && (((uintptr_t)y | (uintptr_t)z | (uintptr_t)out | (uintptr_t)gain) & 15) == 0;
+  const int nt = vec ? (n <= 512 ? 32 : n <= 1024 ? 64 : n <= 2048 ? 128 : 256) : n <= 512 ? 64 : n <= 2048 ? 128 : 256;
   for (int t0 = 0; t0 < T; t0 += 65535) {                  // the grid's second dimension
-    const int m = T - t0 < 65535 ? T - t0 : 65535;
-    cudaError_t e = f32 ? launch_pdl(gated_norm_kernel<float>, dim3(parts, m), dim3(nt), 0, st, y + (size_t)t0 * ldy, ldy,
-                                     (const float*)z + (size_t)t0 * ldz, ldz, gain, (float*)out + (size_t)t0 * ldo, ldo, n, eps)
-                        : launch_pdl(gated_norm_kernel<bf16>, dim3(parts, m), dim3(nt), 0, st, y + (size_t)t0 * ldy, ldy,
-                                     (const bf16*)z + (size_t)t0 * ldz, ldz, gain, (bf16*)out + (size_t)t0 * ldo, ldo, n, eps);
+    const dim3 grid(parts, T - t0 < 65535 ? T - t0 : 65535);
+    const size_t ay = (size_t)t0 * ldy, az = (size_t)t0 * ldz, ao = (size_t)t0 * ldo;
+    cudaError_t e;
+    if (f32) e = launch_pdl(gated_norm_kernel<float>, grid, dim3(nt), 0, st, (const float*)y + ay, ldy, (const float*)z + az, ldz, gain,
+                            (float*)out + ao, ldo, n, eps);
+    else e = launch_pdl(vec ? gated_norm_vec_kernel : gated_norm_kernel<bf16>, grid, dim3(nt), 0, st, (const bf16*)y + ay, ldy,
+                        (const bf16*)z + az, ldz, gain, (bf16*)out + ao, ldo, n, eps);
     if (e != cudaSuccess) return (int)e;
   }
   return (int)cudaGetLastError();
@@ -510,33 +598,52 @@ extern "C" int xft_token_shift(const float* x, int ldx, int T, int n_mix, int W,
   return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }
 
-template <int NP, int VS>
-static int launch_ssd_chunk(const SsdChunkParams& p, int B, cudaStream_t st) {
-  using Cfg = SsdCfg<NP, VS>;
+template <int NP, int VS, int HPC>
+static int launch_ssd_heads(const SsdChunkParams& p, int B, cudaStream_t st) {
+  using Cfg = SsdCfg<NP, VS, HPC>;
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(ssd_chunk_kernel<NP, VS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM) != cudaSuccess)
+    if (cudaFuncSetAttribute(ssd_chunk_kernel<NP, VS, HPC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM) != cudaSuccess)
       return 3000 + (int)cudaGetLastError();
     attr_set = true;
   }
-  const dim3 grid((p.vdim + VS - 1) / VS, p.heads, B);
-  cudaError_t e = launch_pdl(ssd_chunk_kernel<NP, VS>, grid, dim3(kSsdThreads), Cfg::SMEM, st, p);
+  const dim3 grid((p.vdim + VS - 1) / VS * p.segs, p.heads / HPC, B), block(kSsdThreads * HPC);
+  cudaError_t e = cudaSuccess;
+  if (p.segs > 1) {
+    SsdChunkParams q = p;
+    q.carry = 1;
+    e = launch_pdl(ssd_chunk_kernel<NP, VS, HPC>, grid, block, Cfg::SMEM, st, q);
+  }
+  if (e == cudaSuccess) e = launch_pdl(ssd_chunk_kernel<NP, VS, HPC>, grid, block, Cfg::SMEM, st, p);
   return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }
+template <int NP, int VS>
+static int launch_ssd_chunk(const SsdChunkParams& p, int B, cudaStream_t st) {
+  if (p.per_group % 2 == 0) return launch_ssd_heads<NP, VS, 2>(p, B, st);
+  return launch_ssd_heads<NP, VS, 1>(p, B, st);
+}
 
-// Whether the chunk kernel has an instance for states of so many rows.
-extern "C" int xft_ssd_has_chunk(int state_n) { return state_n > 0 && state_n <= 256; }
+// CTAs that a sequence occupies in the chunk kernel, 0: it has no instance for states of so many rows.
+extern "C" int xft_ssd_chunk_ctas(int heads, int per_group, int state_n, int vdim) {
+  if (state_n <= 0 || state_n > 256 || heads <= 0 || per_group <= 0 || vdim <= 0) return 0;
+  const int cols = state_n > 128 || vdim <= 64 ? 64 : 128;
+  const bool two = per_group % 2 == 0 && !(cols == 128) && state_n <= 128;
+  return heads / (two ? 2 : 1) * ((vdim + cols - 1) / cols);
+}
 
-// bf16 portions of at least min_q tokens (others are left alone): u rows [x | B | C] behind the convolution, dt raw step sizes.
+// bf16 portions of at least min_q tokens (others are left alone): u rows [x | B | C] behind the convolution, dt raw step sizes, y
+// [T, heads * vdim] bf16.  segs > 1: portions are cut into so many segments (two launches), with scratch seg_state fp32 [B, heads, segs,
+// state, vdim] and seg_decay fp32 [B, heads, segs].
 extern "C" int xft_ssd_chunk(const void* u, int ldu, int b_at, int c_at, const void* dt, int ld_dt, const float* dt_bias, const float* rate,
                              const float* skip, int heads, int per_group, int state_n, int vdim, float* state, const int* state_slots,
-                             int num_states, const int* cu_q, const int* kv_lens, int B, float* y, int min_q, int* status, cudaStream_t st) {
+                             int num_states, const int* cu_q, const int* kv_lens, int B, void* y, int min_q, int segs, float* seg_state,
+                             float* seg_decay, int* status, cudaStream_t st) {
   if (B <= 0) return 0;
-  if (!xft_ssd_has_chunk(state_n) || heads <= 0 || per_group <= 0 || heads % per_group || vdim <= 0 || num_states <= 0) return -1;
-  if (heads > 65535 || B > 65535 || ((uintptr_t)u & 15)) return -2;
+  if (!xft_ssd_chunk_ctas(heads, per_group, state_n, vdim) || heads % per_group || num_states <= 0) return -1;
+  if (heads > 65535 || B > 65535 || ((uintptr_t)u & 15) || segs < 1 || (segs > 1 && (!seg_state || !seg_decay))) return -2;
   SsdChunkParams p{(const bf16*)u, ldu, b_at, c_at, (const bf16*)dt, ld_dt, dt_bias, rate, skip, heads, per_group, state_n, vdim, state,
-                   state_slots, num_states, cu_q, kv_lens, y, min_q, status};
-  if (state_n <= 64) return vdim <= 64 ? launch_ssd_chunk<64, 64>(p, B, st) : launch_ssd_chunk<64, 128>(p, B, st);
-  if (state_n <= 128) return vdim <= 64 ? launch_ssd_chunk<128, 64>(p, B, st) : launch_ssd_chunk<128, 128>(p, B, st);
-  return launch_ssd_chunk<256, 64>(p, B, st);
+                   state_slots, num_states, cu_q, kv_lens, (bf16*)y, min_q, segs, 0, seg_state, seg_decay, status};
+  if (state_n <= 64) return vdim <= 64 ? launch_ssd_chunk<64, 64>(p, B, st) : launch_ssd_heads<64, 128, 1>(p, B, st);
+  if (state_n <= 128) return vdim <= 64 ? launch_ssd_chunk<128, 64>(p, B, st) : launch_ssd_heads<128, 128, 1>(p, B, st);
+  return launch_ssd_heads<256, 64, 1>(p, B, st);
 }

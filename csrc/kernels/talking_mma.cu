@@ -2,47 +2,74 @@
 //
 // Prompt portions, talking_prefill_kernel: a CTA takes a tile of queries with all of their heads, since the weights of all heads
 // of a (query, key) pair meet in the mix.  A warp owns a unit of 16 rows: 16 queries of one head, or (more than 16 heads) 8
-// queries of two heads that share keys.  The keys are visited twice.  The first pass carries a running maximum and sum per row.
+// queries of two heads that share keys.  Where the heads of a group allow it a warp has two such units side by side, which halves the
+// operands that it reads from shared memory.  The keys are visited twice.  The first pass carries a running maximum and sum per row.
 // The second forms the scores again, and from them the finished weights; they go to shared memory as two bf16 halves, are
 // multiplied with the mixing matrix there (a product over the heads, both halves with fp32 sums: nothing of their 16 bits of
 // mantissa is lost before the mix), and come back as the operand of the product with the values.
 //
 // Decode steps: talking_scores_kernel writes the scores of a key range of one key/value head with its maxima and sums,
-// talking_values_kernel merges those of all ranges, mixes in fp32 and adds up the values of its range; the CTA that arrives last
-// on a head adds up the ranges and applies the gate.
+// talking_values_kernel merges those of all ranges, mixes in fp32 and adds up the values of its range.  The ranges of a head are a
+// cluster, whose CTAs add up their results through distributed shared memory, each a part of the columns, and apply the gate.
 #include "mma_sync.cuh"
 
 namespace xft {
 
 typedef __nv_bfloat16 bf16;
+int make_tensor_map_groups(CUtensorMap* out, const void* ptr, uint64_t groups, uint64_t rows, uint64_t cols, uint32_t box_groups,
+                           uint32_t box_rows);
 constexpr float kTalkLog2e = 1.4426950408889634f;
 
 // ------------------------------------------------------------------------------------------ prompt portions
 struct TalkPrefillParams {
   const bf16* q; const bf16* gate; int ldg; bf16* out; int ldo;
-  const bf16* kc; const bf16* vc; const int* block_table; int bt_stride;
+  const int* block_table; int bt_stride;
   const int* cu_q; const int* kv_lens;
   int hq, hkv, group, bs, num_blocks, window;
   int units, blocks;                         // units of 16 rows, blocks of queries (units = blocks * hq / heads per unit)
+  int stages;                                // tiles of keys in shared memory, 1 or 2
   float scale2, mult;                        // softmax scale * log2(e)
   const float* r1; const float* r2; const float* talk;
   int* status;
 };
 
-constexpr int kTalkThreads = 512;
+constexpr int kTalkUnits = 16;               // units of 16 rows per CTA at most
+constexpr int kTalkPages = 64;
+constexpr size_t kTalkSmem = 227 * 1024 - 512;          // beside the static part
 
+// Shared memory: `stages` tiles of keys and one of values as TMA leaves them (per 64 columns and head KT rows of 128 bytes, swizzled
+// by row & 7), the queries in the order of their fragments, the mixing matrix, weights (two buffers of the upper halves, which the mixed
+// weights replace, and one of the lower), biases.
 template <int D, int HB, int KT>
-__global__ void __launch_bounds__(kTalkThreads, 1) talking_prefill_kernel(const TalkPrefillParams p) {
-  constexpr int QPB = 16 / HB, HP = HB == 1 ? 16 : 32;                 // queries of a block; heads, padded
-  constexpr int KS = D + 8, QP = KT + 8, PITCH = QPB * QP + 8;         // row strides: keys and values, weights of a query, of a head
-  constexpr int KH = D > 64 || KT < 32 ? 16 : 32;                                // keys whose scores are in registers at a time
-  constexpr int MT = HP / 16, MP = HP + 8;
-  extern __shared__ __align__(16) uint8_t tk_raw[];
-  bf16* sK = reinterpret_cast<bf16*>(tk_raw);                          // [hkv][KT][KS]
-  bf16* sV = sK + (size_t)p.hkv * KT * KS;
-  bf16* sM = sV + (size_t)p.hkv * KT * KS;                             // the mixing matrix [HP][MP]
-  bf16* sP = sM + HP * MP;                                             // [2 halves][blocks][HP][PITCH]
-  const int half_size = p.blocks * HP * PITCH;
+struct TalkCfg {
+  static constexpr int QPB = 16 / HB, HP = HB == 1 ? 16 : 32;          // queries of a block; heads, padded
+  static constexpr int QP = KT + 8, PITCH = QPB * QP + 8, MP = HP + 8;      // row strides: weights of a query, of a head, matrix
+  static constexpr int TAB = KT + QPB;                                 // biases of a head: distances of a tile and a block
+  static size_t bytes(int hkv, int blocks, int stages) {
+    return 1024 + ((size_t)(stages + 1) * hkv * KT * D + HP * MP + (size_t)3 * blocks * HP * PITCH) * 2 +
+           (size_t)kTalkUnits * (HB * TAB * 4 + D / 16 * 512);
+  }
+};
+
+// U: units per warp.  With two their queries stay in registers, with one they are read from shared memory.
+template <int D, int HB, int KT, int U>
+__global__ void __launch_bounds__(kTalkUnits / U * 32, 1) talking_prefill_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const TalkPrefillParams p) {
+  using Cfg = TalkCfg<D, HB, KT>;
+  constexpr int QPB = Cfg::QPB, HP = Cfg::HP, QP = Cfg::QP, PITCH = Cfg::PITCH, MP = Cfg::MP, MT = HP / 16;
+  constexpr int NW = kTalkUnits / U, NT = NW * 32;
+  constexpr int KH = U == 1 ? KT : 16;                                 // keys whose scores are in registers at a time
+  constexpr int BOX = KT * 128;                                        // bytes of a head's 64 columns
+  extern __shared__ uint8_t tk_raw[];
+  __shared__ uint64_t full[4];                                         // one per tile buffer
+  __shared__ int pages[kTalkPages];                                    // the first entries of the block table that matter
+  const int tile_size = p.hkv * KT * D, half_size = p.blocks * HP * PITCH, nbuf = p.stages + 1;
+  // tile buffers; the offset is added to the array itself, so that the compiler sees every address to be one of shared memory
+  bf16* sT = reinterpret_cast<bf16*>(tk_raw + ((1024 - (smem_u32(tk_raw) & 1023)) & 1023));
+  uint4* qa = reinterpret_cast<uint4*>(sT + (size_t)nbuf * tile_size) + (threadIdx.x >> 5) * (U * D / 16 * 32) + (threadIdx.x & 31);   // this lane's
+  bf16* sM = sT + (size_t)nbuf * tile_size + kTalkUnits * D * 16;               // the mixing matrix [HP][MP]
+  bf16* sP = sM + HP * MP;                                             // [2 upper, 1 lower][blocks][HP][PITCH]
+  bf16* sLow = sP + (size_t)2 * half_size;
+  float* tab = reinterpret_cast<float*>(sLow + half_size) + (threadIdx.x >> 5) * U * HB * Cfg::TAB;      // this warp's
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int b = blockIdx.y;
   grid_dep_launch();
@@ -53,215 +80,324 @@ __global__ void __launch_bounds__(kTalkThreads, 1) talking_prefill_kernel(const 
   const int last = min(row0 + QT, q_len) - 1;
   const int k_lo = max(0, past + row0 - p.window + 1) / KT * KT;       // a tile lies in one page
   const int n_tiles = (past + last + 1 - k_lo + KT - 1) / KT;
-  // this warp's unit
-  const int per_block = p.hq / HB, qb = warp / per_block, h0 = (warp % per_block) * HB;
-  const bool active = warp < p.units;
+  // this warp's units, neighbouring heads of one group
+  const int per_block = p.hq / HB, qb = warp * U / per_block, h0 = (warp * U % per_block) * HB;
+  const bool active = warp * U < p.units;
   const int kvh = active ? h0 / p.group : 0;
   const int r = lane >> 2, cc = 2 * (lane & 3);
-  int qi[2], qpos[2], head[2];
-  float r1[2], r2[2];
-#pragma unroll
-  for (int e = 0; e < 2; ++e) {                                        // rows r and r + 8
-    qi[e] = row0 + (active ? qb : 0) * QPB + (HB == 1 ? r + 8 * e : r);
-    head[e] = active ? h0 + (HB == 1 ? 0 : e) : 0;
-    qpos[e] = past + min(qi[e], q_len - 1);                            // rows past the end attend like the last one
-    r1[e] = p.r1[head[e]];
-    r2[e] = p.r2[head[e]];
-  }
+  auto query = [&](int e) { return row0 + (active ? qb : 0) * QPB + (HB == 1 ? r + 8 * e : r); };       // of rows r and r + 8
+  auto head = [&](int u, int e) { return active ? h0 + (HB == 1 ? u : 2 * u + e) : 0; };
   // the mixing matrix as an operand
-  for (int i = tid; i < HP * HP; i += kTalkThreads) {
+  for (int i = tid; i < HP * HP; i += NT) {
     const int h = i / HP, g = i % HP;
     sM[h * MP + g] = __float2bfloat16(h < p.hq && g < p.hq ? p.talk[h * p.hq + g] : 0.f);
   }
-  for (int i = tid; i < half_size / 4; i += kTalkThreads) reinterpret_cast<uint4*>(sP)[i] = make_uint4(0, 0, 0, 0);   // both halves
+  for (int i = tid; i < 3 * half_size / 8; i += NT) reinterpret_cast<uint4*>(sP)[i] = make_uint4(0, 0, 0, 0);
+  if (tid == 0) {
+    for (int i = 0; i < nbuf; ++i) mbar_init(&full[i], 1);
+    fence_barrier_init();
+    tma_prefetch_desc(&tmK);
+    tma_prefetch_desc(&tmV);
+  }
+  __syncthreads();
   grid_dep_wait();
-  uint32_t qa[D / 16][4];
+  uint32_t qr[U == 1 ? 1 : U][U == 1 ? 1 : D / 16][4];
 #pragma unroll
-  for (int ks = 0; ks < D / 16; ++ks)
+  for (int u = 0; u < U; ++u)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int i = e & 1;
-      qa[ks][e] = active && qi[i] < q_len ? *reinterpret_cast<const uint32_t*>(
-          p.q + ((size_t)(q0 + qi[i]) * p.hq + head[i]) * D + ks * 16 + cc + (e >> 1) * 8) : 0u;
+    for (int ks = 0; ks < D / 16; ++ks) {
+      uint32_t v[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int i = e & 1;
+        v[e] = active && query(i) < q_len ? *reinterpret_cast<const uint32_t*>(
+            p.q + ((size_t)(q0 + query(i)) * p.hq + head(u, i)) * D + ks * 16 + cc + (e >> 1) * 8) : 0u;
+        if (U > 1) qr[u % (U == 1 ? 1 : U)][ks % (U == 1 ? 1 : D / 16)][e] = v[e];
+      }
+      if (U == 1) qa[ks * 32] = make_uint4(v[0], v[1], v[2], v[3]);    // read back by the same lane
     }
   const int* bt = p.block_table + (size_t)b * p.bt_stride;
-  auto load = [&](bf16* dst, const bf16* cache, int tile) {
-    const int key = k_lo + tile * KT;
-    int blk = bt[key / p.bs];
-    if (blk < 0 || blk >= p.num_blocks) { if (tid == 0 && p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); blk = 0; }
-    const bf16* src = cache + ((size_t)blk * p.hkv * p.bs + key % p.bs) * D;
-    for (int i = tid; i < p.hkv * KT * (D / 8); i += kTalkThreads) {
-      const int row = i / (D / 8), c = i % (D / 8), g = row / KT, k = row % KT;
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst + (size_t)row * KS + c * 8)),
-                   "l"(src + ((size_t)g * p.bs + k) * D + c * 8) : "memory");
-    }
+  // tile buffers are filled by one thread, behind a barrier that says everyone is done with what was there
+  uint32_t phases = 0;
+  const int page0 = k_lo / p.bs;
+  for (int i = tid; i < kTalkPages && i <= (k_lo + (n_tiles - 1) * KT) / p.bs - page0; i += NT) pages[i] = bt[page0 + i];
+  __syncthreads();
+  auto load = [&](int buf, const CUtensorMap& map, int tile, int by) {
+    if (tile >= n_tiles || tid != by * 32) return;
+    const int page = (k_lo + tile * KT) / p.bs - page0;
+    int blk = page < kTalkPages ? pages[page] : bt[page0 + page];
+    if (blk < 0 || blk >= p.num_blocks) { if (p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); blk = 0; }
+    mbar_expect_tx(&full[buf], tile_size * 2);
+    uint8_t* dst = reinterpret_cast<uint8_t*>(sT + (size_t)buf * tile_size);
+#pragma unroll
+    for (int c = 0; c < D / 64; ++c)
+      tma_load_3d(dst + c * p.hkv * BOX, &map, &full[buf], c * 64, (k_lo + tile * KT) % p.bs, blk * p.hkv, kEvictNormal);
   };
-  auto commit = [] { asm volatile("cp.async.commit_group;" ::: "memory"); };
+  auto arrived = [&](int buf) {                                        // a wait that runs out is reported; what was there is read
+    mbar_wait(&full[buf], phases >> buf & 1, p.status, XFT_ERR_WAIT_FULL);
+    phases ^= 1u << buf;
+  };
   const int fa_r = (lane & 7) + ((lane >> 3) & 1) * 8, fa_c = (lane >> 4) * 8;
-  const int fb_r = (lane & 7) + ((lane >> 4) & 1) * 8, fb_c = ((lane >> 3) & 1) * 8;
-  // scores (base 2) of this warp's rows and KH keys from `k` on of the tile in `s`; -inf where a key is not visible
-  float S[KH / 8][4];
-  auto scores = [&](const bf16* s, int tile, int k) {
+  const int fb_r = (lane & 7) + ((lane >> 4) & 1) * 8;
+  // a lane's 16-byte piece of the first 16 columns, swizzled: keys (two pieces along a row) and values (two along the columns)
+  const int xk = (((lane >> 3) & 1) ^ (lane & 7)) * 16, xv = ((lane >> 4) ^ (lane & 7)) * 16;
+  // The bias of a key depends on its distance alone: -r1 log2(1 + r2 distance), and -inf for one that is not visible.  Entry i of a
+  // head's table belongs to the distance top - i, where `top` is that of the block's last query and the tile's first key.
+  float ra[U * HB], rc[U * HB];
 #pragma unroll
-    for (int j = 0; j < KH / 8; ++j) S[j][0] = S[j][1] = S[j][2] = S[j][3] = 0.f;
-    const bf16* base = s + ((size_t)kvh * KT + k) * KS;
+  for (int e = 0; e < U * HB; ++e) {
+    ra[e] = active ? -p.r1[h0 + e] : 0.f;
+    rc[e] = active ? p.r2[h0 + e] : 0.f;
+  }
+  const int top0 = past + row0 + ((active ? qb : 0) + 1) * QPB - 1 - k_lo;
+  auto biases = [&](int tile) {
+    if (!active || tile >= n_tiles) return;
+    __syncwarp();
 #pragma unroll
-    for (int ks = 0; ks < D / 16; ++ks)
+    for (int e = 0; e < U * HB; ++e)
+#pragma unroll
+      for (int i = 0; i < Cfg::TAB - 1; i += 32) {
+        const int far = top0 - tile * KT - i - lane;
+        const float v = ra[e] * gl_lg2(fmaf(rc[e], (float)far, 1.f));
+        if (i + lane < Cfg::TAB - 1) tab[e * Cfg::TAB + i + lane] = far >= 0 && far < p.window ? v : -INFINITY;
+      }
+    __syncwarp();
+  };
+  const int chunk = p.hkv * BOX;                                       // bytes of 64 columns of all heads
+  const float* my_tab = tab + QPB - 1 - r + cc;
+  // scores (base 2) of this warp's rows and KH keys from `k` on of the tile in `s`
+  float S[U][KH / 8][4];
+  auto scores = [&](const bf16* s, int k) {
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+#pragma unroll
+      for (int j = 0; j < KH / 8; ++j) S[u][j][0] = S[u][j][1] = S[u][j][2] = S[u][j][3] = 0.f;
+    const uint8_t* base = reinterpret_cast<const uint8_t*>(s) + kvh * BOX + (k + fb_r) * 128;
+#pragma unroll
+    for (int ks = 0; ks < D / 16; ++ks) {
+      uint32_t a[U][4];
+      if (U == 1) {
+        const uint4 q = qa[ks * 32];
+        a[0][0] = q.x; a[0][1] = q.y; a[0][2] = q.z; a[0][3] = q.w;
+      } else {
+#pragma unroll
+        for (int u = 0; u < U; ++u)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) a[u][e] = qr[u % (U == 1 ? 1 : U)][ks % (U == 1 ? 1 : D / 16)][e];
+      }
 #pragma unroll
       for (int j = 0; j < KH / 8; j += 2) {
         uint32_t w[4];
-        gl_ldsm(w, base + (j * 8 + fb_r) * KS + ks * 16 + fb_c);
-        gl_mma(S[j], qa[ks], w[0], w[1]);
-        gl_mma(S[j + 1], qa[ks], w[2], w[3]);
-      }
-    const int key0 = k_lo + tile * KT + k + cc;
+        gl_ldsm(w, base + ks / 4 * chunk + j * 1024 + (xk ^ (ks % 4 * 32)));
 #pragma unroll
-    for (int j = 0; j < KH / 8; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int far = qpos[e >> 1] - (key0 + j * 8 + (e & 1));
-        const float v = fmaf(S[j][e], p.scale2, -r1[e >> 1] * gl_lg2(fmaf(r2[e >> 1], (float)max(far, 0), 1.f)));
-        S[j][e] = far >= 0 && far < p.window ? v : -INFINITY;
-      }
-  };
-  // ---- first pass: maxima and sums; both tile buffers hold keys
-  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-  load(sK, p.kc, 0);
-  commit();
-  for (int j = 0; j < n_tiles; ++j) {
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();
-    if (j + 1 < n_tiles) load(j & 1 ? sK : sV, p.kc, j + 1);
-    commit();
-    if (!active) continue;
-#pragma unroll 1
-    for (int k = 0; k < KT; k += KH) {
-      scores(j & 1 ? sV : sK, j, k);
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        float mx = m[e];
-#pragma unroll
-        for (int i = 0; i < KH / 8; ++i) mx = fmaxf(mx, fmaxf(S[i][2 * e], S[i][2 * e + 1]));
-        const float ref = mx == -INFINITY ? 0.f : mx;                  // nothing seen yet: every term is zero
-        float sum = 0.f;
-#pragma unroll
-        for (int i = 0; i < KH / 8; ++i) sum += gl_ex2(S[i][2 * e] - ref) + gl_ex2(S[i][2 * e + 1] - ref);
-        l[e] = fmaf(l[e], gl_ex2(m[e] - ref), sum);                    // this lane's columns alone
-        m[e] = mx;
-      }
-    }
-  }
-#pragma unroll
-  for (int e = 0; e < 2; ++e) {                                        // the four lanes of a row; m becomes log2 of the row's sum
-    float mx = m[e];
-    mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-    mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-    float s = m[e] == -INFINITY ? 0.f : l[e] * gl_ex2(m[e] - mx);
-    s += __shfl_xor_sync(0xffffffffu, s, 1);
-    s += __shfl_xor_sync(0xffffffffu, s, 2);
-    m[e] = mx;
-    l[e] = s > 0.f ? __fdividef(1.f, s) : 0.f;
-  }
-  // ---- second pass
-  float O[D / 8][4];
-#pragma unroll
-  for (int j = 0; j < D / 8; ++j) O[j][0] = O[j][1] = O[j][2] = O[j][3] = 0.f;
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
-  __syncthreads();
-  load(sK, p.kc, 0);
-  commit();
-  bf16* pw = sP + (size_t)(active ? qb : 0) * HP * PITCH;              // this unit's block
-  for (int j = 0; j < n_tiles; ++j) {
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();                                                   // keys are here, everyone is done with the values
-    load(sV, p.vc, j);
-    commit();
-    if (active) {
-#pragma unroll 1
-      for (int k = 0; k < KT; k += KH) {
-        scores(sK, j, k);
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          bf16* dst = pw + (size_t)head[e] * PITCH + (HB == 1 ? r + 8 * e : r) * QP + k + cc;
-#pragma unroll
-          for (int i = 0; i < KH / 8; ++i) {
-            const float a = gl_ex2(S[i][2 * e] - m[e]) * l[e], c = gl_ex2(S[i][2 * e + 1] - m[e]) * l[e];
-            const uint32_t hi = gl_pack(a, c);
-            const float2 f = gl_unpack(hi);
-            *reinterpret_cast<uint32_t*>(dst + i * 8) = hi;
-            *reinterpret_cast<uint32_t*>(dst + half_size + i * 8) = gl_pack(a - f.x, c - f.y);
-          }
+        for (int u = 0; u < U; ++u) {
+          gl_mma(S[u][j], a[u], w[0], w[1]);
+          gl_mma(S[u][j + 1], a[u], w[2], w[3]);
         }
       }
     }
-    __syncthreads();                                                   // weights are here, everyone is done with the keys
-    if (j + 1 < n_tiles) load(sK, p.kc, j + 1);
-    commit();
-    // the mix, in place: 16 keys of a query at a time
-    for (int c = warp; c < p.blocks * QPB * (KT / 16); c += kTalkThreads / 32) {
-      const int qq = c / (KT / 16), k = c % (KT / 16) * 16;
-      bf16* at = sP + (size_t)(qq / QPB) * HP * PITCH + qq % QPB * QP + k;
-      float w[MT][2][4];
 #pragma unroll
-      for (int a = 0; a < MT; ++a)
+    for (int u = 0; u < U; ++u)
 #pragma unroll
-        for (int i = 0; i < 2; ++i) w[a][i][0] = w[a][i][1] = w[a][i][2] = w[a][i][3] = 0.f;
+      for (int j = 0; j < KH / 8; ++j)
 #pragma unroll
-      for (int g = 0; g < MT; ++g)
+        for (int e = 0; e < 4; ++e) {
+          const int at = HB == 1 ? u * Cfg::TAB - (e >> 1) * 8 : (2 * u + (e >> 1)) * Cfg::TAB;
+          S[u][j][e] = fmaf(S[u][j][e], p.scale2, my_tab[at + k + j * 8 + (e & 1)]);
+        }
+  };
+  // ---- first pass: maxima and sums; all buffers take turns with keys
+  float m[U][2], l[U][2];
 #pragma unroll
-        for (int part = 0; part < 2; ++part) {
-          uint32_t x[4];
-          gl_ldsm_t(x, at + (size_t)part * half_size + (g * 16 + fa_r) * PITCH + fa_c);
+  for (int u = 0; u < U; ++u) { m[u][0] = m[u][1] = -INFINITY; l[u][0] = l[u][1] = 0.f; }
+  for (int j = 0; j + 1 < nbuf; ++j) load(j, tmK, j, j);
+  biases(0);
+  for (int j = 0, buf = 0, ahead = nbuf - 1; j < n_tiles; ++j, buf = buf + 1 == nbuf ? 0 : buf + 1, ahead = ahead + 1 == nbuf ? 0 : ahead + 1) {
+    __syncthreads();
+    load(ahead, tmK, j + nbuf - 1, j % NW);
+    arrived(buf);
+    if (!active) continue;
 #pragma unroll
-          for (int a = 0; a < MT; ++a) {
-            uint32_t mix[4];
-            gl_ldsm(mix, sM + (a * 16 + fa_r) * MP + g * 16 + fa_c);
-            gl_mma(w[a][0], mix, x[0], x[1]);
-            gl_mma(w[a][1], mix, x[2], x[3]);
+    for (int k = 0; k < KT; k += KH) {
+      scores(sT + buf * tile_size, k);
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          float mx = m[u][e];
+#pragma unroll
+          for (int i = 0; i < KH / 8; ++i) mx = fmaxf(mx, fmaxf(S[u][i][2 * e], S[u][i][2 * e + 1]));
+          const float ref = mx == -INFINITY ? 0.f : mx;                // nothing seen yet: every term is zero
+          float sum = 0.f;
+#pragma unroll
+          for (int i = 0; i < KH / 8; ++i) sum += gl_ex2(S[u][i][2 * e] - ref) + gl_ex2(S[u][i][2 * e + 1] - ref);
+          l[u][e] = fmaf(l[u][e], gl_ex2(m[u][e] - ref), sum);         // this lane's columns alone
+          m[u][e] = mx;
+        }
+    }
+    biases(j + 1);
+  }
+#pragma unroll
+  for (int u = 0; u < U; ++u)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {                                      // the four lanes of a row
+      float mx = m[u][e];
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+      float s = m[u][e] == -INFINITY ? 0.f : l[u][e] * gl_ex2(m[u][e] - mx);
+      s += __shfl_xor_sync(0xffffffffu, s, 1);
+      s += __shfl_xor_sync(0xffffffffu, s, 2);
+      m[u][e] = s > 0.f ? mx + gl_lg2(s) : INFINITY;                   // log2 of the row's sum
+    }
+  // ---- second pass: the scores of one tile beside the values of the one before
+  float O[U][D / 8][4];
+#pragma unroll
+  for (int u = 0; u < U; ++u)
+#pragma unroll
+    for (int j = 0; j < D / 8; ++j) O[u][j][0] = O[u][j][1] = O[u][j][2] = O[u][j][3] = 0.f;
+  const int block_at = (active ? qb : 0) * HP * PITCH;                 // this unit's block
+  auto weights = [&](int j) {                                          // of tile j, in two halves
+    bf16* dst = sP + (j & 1) * half_size + block_at;
+    const bf16* keys = sT + (p.stages > 1 ? (j & 1) * tile_size : 0);
+#pragma unroll
+    for (int k = 0; k < KT; k += KH) {
+      scores(keys, k);
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int at = head(u, e) * PITCH + (HB == 1 ? r + 8 * e : r) * QP + k + cc;
+#pragma unroll
+          for (int i = 0; i < KH / 8; ++i) {
+            const float a = gl_ex2(S[u][i][2 * e] - m[u][e]), c = gl_ex2(S[u][i][2 * e + 1] - m[u][e]);
+            const uint32_t hi = gl_pack(a, c);
+            const float2 f = gl_unpack(hi);
+            *reinterpret_cast<uint32_t*>(dst + at + i * 8) = hi;
+            *reinterpret_cast<uint32_t*>(sLow + block_at + at + i * 8) = gl_pack(a - f.x, c - f.y);
           }
+        }
+    }
+  };
+  // the mix of tile j, in place: 16 keys of a query at a time, two such pieces side by side
+  const int pieces = p.blocks * QPB * (KT / 16);
+  auto mix = [&](int j) {
+    bf16* upper = sP + (j & 1) * half_size;
+    constexpr int N2 = MT == 1 ? 2 : 1;
+    uint32_t t[MT][MT][4];
+#pragma unroll
+    for (int a = 0; a < MT; ++a)
+#pragma unroll
+      for (int g = 0; g < MT; ++g) gl_ldsm(t[a][g], sM + (a * 16 + fa_r) * MP + g * 16 + fa_c);
+    for (int c0 = warp; c0 < pieces; c0 += N2 * NW) {
+      int at[N2];
+      uint32_t x[N2][2][MT][4];
+#pragma unroll
+      for (int n = 0; n < N2; ++n) {
+        const int c = min(c0 + n * NW, pieces - 1), qq = c / (KT / 16), k = c % (KT / 16) * 16;
+        at[n] = qq / QPB * HP * PITCH + qq % QPB * QP + k;
+#pragma unroll
+        for (int g = 0; g < MT; ++g) {
+          gl_ldsm_t(x[n][0][g], upper + at[n] + (g * 16 + fa_r) * PITCH + fa_c);
+          gl_ldsm_t(x[n][1][g], sLow + at[n] + (g * 16 + fa_r) * PITCH + fa_c);
+        }
+      }
+      float w[N2][MT][2][4];
+#pragma unroll
+      for (int n = 0; n < N2; ++n)
+#pragma unroll
+        for (int a = 0; a < MT; ++a) {
+#pragma unroll
+          for (int i = 0; i < 2; ++i) w[n][a][i][0] = w[n][a][i][1] = w[n][a][i][2] = w[n][a][i][3] = 0.f;
+#pragma unroll
+          for (int g = 0; g < MT; ++g)
+#pragma unroll
+            for (int part = 0; part < 2; ++part) {
+              gl_mma(w[n][a][0], t[a][g], x[n][part][g][0], x[n][part][g][1]);
+              gl_mma(w[n][a][1], t[a][g], x[n][part][g][2], x[n][part][g][3]);
+            }
         }
       __syncwarp();
 #pragma unroll
-      for (int a = 0; a < MT; ++a)
+      for (int n = 0; n < N2; ++n)
+        if (n == 0 || c0 + n * NW < pieces)
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          *reinterpret_cast<uint32_t*>(at + (a * 16 + r) * PITCH + i * 8 + cc) = gl_pack(w[a][i][0], w[a][i][1]);
-          *reinterpret_cast<uint32_t*>(at + (a * 16 + r + 8) * PITCH + i * 8 + cc) = gl_pack(w[a][i][2], w[a][i][3]);
-        }
+          for (int a = 0; a < MT; ++a)
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+              *reinterpret_cast<uint32_t*>(upper + at[n] + (a * 16 + r) * PITCH + i * 8 + cc) = gl_pack(w[n][a][i][0], w[n][a][i][1]);
+              *reinterpret_cast<uint32_t*>(upper + at[n] + (a * 16 + r + 8) * PITCH + i * 8 + cc) = gl_pack(w[n][a][i][2], w[n][a][i][3]);
+            }
     }
-    asm volatile("cp.async.wait_group 1;" ::: "memory");
-    __syncthreads();                                                   // mixed weights and values are here
+  };
+  const bool two = p.stages > 1;
+  auto key_buf = [&](int j) { return two ? j & 1 : 0; };
+  const int value_buf = p.stages;
+  auto load_keys = [&](int j) { load(key_buf(j), tmK, j, j % NW); };
+  auto load_values = [&](int j) { load(value_buf, tmV, j, (j + NW / 2) % NW); };
+  __syncthreads();                                                     // everyone is done with the first pass's tiles
+  load_keys(0);
+  if (two) load_keys(1);
+  load_values(0);
+  biases(0);
+  arrived(key_buf(0));
+  if (active) weights(0);
+  __syncthreads();
+  if (!two) load_keys(1);
+  mix(0);
+  biases(1);
+  __syncthreads();
+  for (int j = 0; j < n_tiles; ++j) {
+    // here: mixed weights of tile j; its values and the keys of tile j + 1 are on their way
+    if (two) load_keys(j + 2);
+    if (j + 1 < n_tiles) {
+      arrived(key_buf(j + 1));
+      if (active) weights(j + 1);
+    }
+    arrived(value_buf);
     if (active) {
-      const bf16* wrow = HB == 1 ? pw + (size_t)h0 * PITCH + fa_r * QP : pw + (size_t)(h0 + ((lane >> 3) & 1)) * PITCH + (lane & 7) * QP;
-      const bf16* vb = sV + (size_t)kvh * KT * KS;
+      const bf16* pw = sP + (j & 1) * half_size + block_at;
+      const bf16* wrow = HB == 1 ? pw + h0 * PITCH + fa_r * QP : pw + (h0 + ((lane >> 3) & 1)) * PITCH + (lane & 7) * QP;
+      const uint8_t* vb = reinterpret_cast<const uint8_t*>(sT + (size_t)value_buf * tile_size) + kvh * BOX + fa_r * 128;
 #pragma unroll
       for (int ks = 0; ks < KT / 16; ++ks) {
-        uint32_t a[4];
-        gl_ldsm(a, wrow + ks * 16 + fa_c);
+        uint32_t a[U][4];
+#pragma unroll
+        for (int u = 0; u < U; ++u) gl_ldsm(a[u], wrow + u * HB * PITCH + ks * 16 + fa_c);
 #pragma unroll
         for (int i = 0; i < D / 8; i += 2) {
           uint32_t w[4];
-          gl_ldsm_t(w, vb + (ks * 16 + fa_r) * KS + i * 8 + fa_c);
-          gl_mma(O[i], a, w[0], w[1]);
-          gl_mma(O[i + 1], a, w[2], w[3]);
+          gl_ldsm_t(w, vb + i / 8 * chunk + ks * 2048 + (xv ^ (i % 8 * 16)));
+#pragma unroll
+          for (int u = 0; u < U; ++u) {
+            gl_mma(O[u][i], a[u], w[0], w[1]);
+            gl_mma(O[u][i + 1], a[u], w[2], w[3]);
+          }
         }
       }
     }
+    __syncthreads();
+    if (!two) load_keys(j + 2);
+    load_values(j + 1);
+    if (j + 1 < n_tiles) mix(j + 1);
+    biases(j + 2);
+    __syncthreads();
   }
   if (!active) return;
 #pragma unroll
-  for (int e = 0; e < 2; ++e) {
-    if (qi[e] >= q_len) continue;
-    const size_t t = q0 + qi[e];
-    const bf16* g = p.gate + t * p.ldg + head[e] * D + cc;
-    bf16* o = p.out + t * p.ldo + head[e] * D + cc;
+  for (int u = 0; u < U; ++u)
 #pragma unroll
-    for (int i = 0; i < D / 8; ++i) {
-      const float2 x = gl_unpack(*reinterpret_cast<const uint32_t*>(g + i * 8));
-      *reinterpret_cast<uint32_t*>(o + i * 8) = gl_pack(O[i][2 * e] * p.mult * gl_rcp(1.f + gl_ex2(-x.x * kTalkLog2e)),
-                                                        O[i][2 * e + 1] * p.mult * gl_rcp(1.f + gl_ex2(-x.y * kTalkLog2e)));
+    for (int e = 0; e < 2; ++e) {
+      if (query(e) >= q_len) continue;
+      const size_t t = q0 + query(e);
+      const bf16* g = p.gate + t * p.ldg + head(u, e) * D + cc;
+      bf16* o = p.out + t * p.ldo + head(u, e) * D + cc;
+#pragma unroll
+      for (int i = 0; i < D / 8; ++i) {
+        const float2 x = gl_unpack(*reinterpret_cast<const uint32_t*>(g + i * 8));
+        *reinterpret_cast<uint32_t*>(o + i * 8) = gl_pack(O[u][i][2 * e] * p.mult * gl_rcp(1.f + gl_ex2(-x.x * kTalkLog2e)),
+                                                          O[u][i][2 * e + 1] * p.mult * gl_rcp(1.f + gl_ex2(-x.y * kTalkLog2e)));
+      }
     }
-  }
 }
 
 // ------------------------------------------------------------------------------------------ decode steps
@@ -275,8 +411,6 @@ struct TalkDecodeParams {
   const float* r1; const float* r2; const float* talk;
   float* scores;                             // [B][hq][span], base 2, from the first visited page's first key on
   float* part_ml;                            // [B][hq][splits][2]
-  float* part_o;                             // [B][hq][splits][D] (splits > 1)
-  int* counters;                             // [B * hkv], zero between launches
   int* status;
 };
 
@@ -378,62 +512,70 @@ __global__ void __launch_bounds__(128) talking_scores_kernel(const TalkDecodePar
   }
 }
 
-// grid (splits, hkv, B), 128 threads: a thread owns four columns of the head and every (512 / D)-th key of a page
+// grid (splits, hkv, B), clusters of (splits), 256 threads: a thread owns four columns of the head and every (1024 / D)-th key of a page
+constexpr int kTalkValues = 256;
 template <int D, int GR>
-__global__ void __launch_bounds__(128) talking_values_kernel(const TalkDecodeParams p) {
-  constexpr int CG = D / 4, KSUB = 128 / CG;
-  extern __shared__ float tv_sm[];
-  const int H = p.hq, tid = threadIdx.x, b = blockIdx.z, kvh = blockIdx.y, h0 = kvh * p.group;
-  float* sp = tv_sm;                         // [H][64] weights
+__global__ void __launch_bounds__(kTalkValues) talking_values_kernel(const TalkDecodeParams p) {
+  constexpr int CG = D / 4, KSUB = kTalkValues / CG, NT = kTalkValues;
+  extern __shared__ __align__(16) float tv_sm[];
+  const int H = p.hq, tid = threadIdx.x, lane = tid & 31, b = blockIdx.z, kvh = blockIdx.y, h0 = kvh * p.group, ns = p.splits;
+  float* so = tv_sm;                         // [GR][D] this range's result, which the cluster reads
+  float* sp = so + GR * D;                   // [H][64] weights
   float* sw = sp + H * 64;                   // [64][GR] mixed
   float* st = sw + 64 * GR;                  // [group][H] mixing matrix
   float* sm = st + p.group * H;              // [H] maxima and inverse sums
   float* si = sm + H;
-  float* so = tv_sm;                         // [KSUB][GR][D] at the end
-  __shared__ int s_last;
+  float* sr = sp;                            // [KSUB][GR][D] at the end
   grid_dep_launch();
   const int n_keys = p.kv_lens[b];
   int first, stop, base;
   talk_pages(p, n_keys, blockIdx.x, first, stop, base);
-  for (int i = tid; i < p.group * H; i += 128) st[i] = p.talk[(size_t)h0 * H + i];
+  for (int i = tid; i < p.group * H; i += NT) st[i] = p.talk[(size_t)h0 * H + i];
+  const int c4 = tid % CG * 4, ksub = tid / CG;
   grid_dep_wait();
-  for (int h = tid; h < H; h += 128) {
-    const float* ml = p.part_ml + ((size_t)b * H + h) * p.splits * 2;
-    float mx = -INFINITY, s = 0.f;
-    for (int i = 0; i < p.splits; ++i) mx = fmaxf(mx, __ldcg(ml + 2 * i));
-    for (int i = 0; i < p.splits; ++i) { const float m = __ldcg(ml + 2 * i); s += m == -INFINITY ? 0.f : __ldcg(ml + 2 * i + 1) * gl_ex2(m - mx); }
-    sm[h] = mx;
-    si[h] = s > 0.f ? 1.f / s : 0.f;
+  for (int h = tid >> 5; h < H; h += NT / 32) {            // a warp per head, a range per lane
+    const float2 ml = lane < ns ? __ldcg(reinterpret_cast<const float2*>(p.part_ml) + ((size_t)b * H + h) * ns + lane) : make_float2(-INFINITY, 0.f);
+    float mx = ml.x;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    float s = ml.x == -INFINITY ? 0.f : ml.y * gl_ex2(ml.x - mx);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+    if (lane == 0) { sm[h] = mx; si[h] = s > 0.f ? 1.f / s : 0.f; }
   }
   float acc[GR][4];
 #pragma unroll
   for (int g = 0; g < GR; ++g) acc[g][0] = acc[g][1] = acc[g][2] = acc[g][3] = 0.f;
-  const int c4 = tid % CG * 4, ksub = tid / CG;
+  constexpr int KN = 64 / KSUB;              // keys of a page per thread
   for (int page = first; page < stop; ++page) {
+    // values on their way while the weights are mixed
+    const bf16* v = talk_page(p, p.vc, b, page, kvh, D) + c4;
+    uint2 u[KN];
+#pragma unroll
+    for (int k = 0; k < KN; ++k) u[k] = *reinterpret_cast<const uint2*>(v + (size_t)(k * KSUB + ksub) * D);
     __syncthreads();
-    for (int i = tid; i < H * 16; i += 128) {
+    for (int i = tid; i < H * 16; i += NT) {
       const int h = i >> 4, k = (i & 15) * 4;
       const float4 s = __ldcg(reinterpret_cast<const float4*>(p.scores + ((size_t)b * H + h) * p.span + page * 64 - base + k));
       const float m = sm[h], f = si[h];
       *reinterpret_cast<float4*>(sp + h * 64 + k) = make_float4(gl_ex2(s.x - m) * f, gl_ex2(s.y - m) * f, gl_ex2(s.z - m) * f, gl_ex2(s.w - m) * f);
     }
     __syncthreads();
-    for (int i = tid; i < 64 * GR; i += 128) {
+    for (int i = tid; i < 64 * GR; i += NT) {
       const int g = i >> 6, k = i & 63;
       float w = 0.f;
       if (g < p.group)
+#pragma unroll 8
         for (int x = 0; x < H; ++x) w = fmaf(st[g * H + x], sp[x * 64 + k], w);
       sw[k * GR + g] = w;
     }
     __syncthreads();
-    const bf16* v = talk_page(p, p.vc, b, page, kvh, D) + c4;
-#pragma unroll 4
-    for (int k = ksub; k < 64; k += KSUB) {
-      const uint2 u = *reinterpret_cast<const uint2*>(v + (size_t)k * D);
-      const float2 a = gl_unpack(u.x), c = gl_unpack(u.y);
+#pragma unroll
+    for (int k = 0; k < KN; ++k) {
+      const float2 a = gl_unpack(u[k].x), c = gl_unpack(u[k].y);
 #pragma unroll
       for (int g = 0; g < GR; ++g) {
-        const float w = sw[k * GR + g];
+        const float w = sw[(k * KSUB + ksub) * GR + g];
         acc[g][0] = fmaf(w, a.x, acc[g][0]); acc[g][1] = fmaf(w, a.y, acc[g][1]);
         acc[g][2] = fmaf(w, c.x, acc[g][2]); acc[g][3] = fmaf(w, c.y, acc[g][3]);
       }
@@ -441,75 +583,81 @@ __global__ void __launch_bounds__(128) talking_values_kernel(const TalkDecodePar
   }
   __syncthreads();
 #pragma unroll
-  for (int g = 0; g < GR; ++g) *reinterpret_cast<float4*>(so + ((size_t)ksub * GR + g) * D + c4) = make_float4(acc[g][0], acc[g][1], acc[g][2], acc[g][3]);
+  for (int g = 0; g < GR; ++g) *reinterpret_cast<float4*>(sr + ((size_t)ksub * GR + g) * D + c4) = make_float4(acc[g][0], acc[g][1], acc[g][2], acc[g][3]);
   __syncthreads();
-  auto finish = [&](int g, int d, float x) {
-    const float y = __bfloat162float(p.gate[(size_t)b * p.ldg + (h0 + g) * D + d]);
-    p.out[(size_t)b * p.ldo + (h0 + g) * D + d] = __float2bfloat16(x * p.mult * gl_rcp(1.f + gl_ex2(-y * kTalkLog2e)));
-  };
-  for (int i = tid; i < p.group * D; i += 128) {
-    const int g = i / D, d = i % D;
+  for (int i = tid; i < GR * D; i += NT) {
     float x = 0.f;
 #pragma unroll
-    for (int k = 0; k < KSUB; ++k) x += so[((size_t)k * GR + g) * D + d];
-    if (p.splits == 1) finish(g, d, x);
-    else p.part_o[(((size_t)b * H + h0 + g) * p.splits + blockIdx.x) * D + d] = x;
+    for (int k = 0; k < KSUB; ++k) x += sr[(size_t)k * GR * D + i];
+    so[i] = x;
   }
-  if (p.splits == 1) return;
-  __threadfence();
-  __syncthreads();
-  if (tid == 0) {
-    int* c = p.counters + b * p.hkv + kvh;
-    s_last = atomicAdd(c, 1) == p.splits - 1;
-    if (s_last) *c = 0;
-  }
-  __syncthreads();
-  if (!s_last) return;
-  __threadfence();
-  for (int i = tid; i < p.group * D; i += 128) {
-    const int g = i / D, d = i % D;
-    const float* o = p.part_o + ((size_t)b * H + h0 + g) * p.splits * D + d;
+  if (ns > 1) { cluster_arrive(); cluster_wait(); } else __syncthreads();
+  // this CTA's part of the columns
+  const int n = p.group * D, per = (n + ns - 1) / ns, i0 = blockIdx.x * per, i1 = min(i0 + per, n);
+  for (int i = i0 + tid; i < i1; i += NT) {
     float x = 0.f;
-    for (int s = 0; s < p.splits; ++s) x += __ldcg(o + (size_t)s * D);
-    finish(g, d, x);
+    if (ns > 1) {
+      const uint32_t a = smem_u32(so + i);
+#pragma unroll 8
+      for (int c = 0; c < ns; ++c) x += ld_dsmem(dsmem_addr(a, c));
+    } else x = so[i];
+    const size_t col = (size_t)h0 * D + i;
+    const float y = __bfloat162float(p.gate[(size_t)b * p.ldg + col]);
+    p.out[(size_t)b * p.ldo + col] = __float2bfloat16(x * p.mult * gl_rcp(1.f + gl_ex2(-y * kTalkLog2e)));
   }
+  if (ns > 1) { cluster_arrive(); cluster_wait(); }        // nobody leaves while its shared memory may be read
 }
 
 }  // namespace xft
 
 using namespace xft;
 
-template <int D, int HB, int KT>
-static int launch_prefill(const TalkPrefillParams& p, int B, int max_q, cudaStream_t st) {
-  constexpr int QPB = 16 / HB, HP = HB == 1 ? 16 : 32;
-  const size_t smem = ((size_t)2 * p.hkv * KT * (D + 8) + HP * (HP + 8) + (size_t)2 * p.blocks * HP * (QPB * (KT + 8) + 8)) * 2;
-  if (smem > 227 * 1024) return -6;
+template <int D, int HB, int KT, int U>
+static int launch_units(const TalkPrefillParams& p, const void* kc, const void* vc, int B, int max_q, cudaStream_t st) {
+  using Cfg = TalkCfg<D, HB, KT>;
+  const size_t smem = Cfg::bytes(p.hkv, p.blocks, p.stages);
+  if (smem > kTalkSmem) return -6;
   static size_t allowed = 0;
   if (smem > allowed) {
-    if (cudaFuncSetAttribute(talking_prefill_kernel<D, HB, KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+    if (cudaFuncSetAttribute(talking_prefill_kernel<D, HB, KT, U>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
       return 3000 + (int)cudaGetLastError();
     allowed = smem;
   }
-  const int qt = p.blocks * QPB;
-  cudaError_t e = launch_pdl(talking_prefill_kernel<D, HB, KT>, dim3((max_q + qt - 1) / qt, B), dim3(kTalkThreads), smem, st, p);
+  const int qt = p.blocks * Cfg::QPB;
+  CUtensorMap tmK, tmV;
+  const uint64_t groups = (uint64_t)p.num_blocks * p.hkv;
+  if (make_tensor_map_groups(&tmK, kc, groups, p.bs, D, p.hkv, KT) || make_tensor_map_groups(&tmV, vc, groups, p.bs, D, p.hkv, KT)) return -4;
+  cudaError_t e = launch_pdl(talking_prefill_kernel<D, HB, KT, U>, dim3((max_q + qt - 1) / qt, B), dim3(kTalkUnits / U * 32), smem, st, tmK, tmV, p);
   return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }
-template <int D, int HB>
-static int prefill_keys(const TalkPrefillParams& p, int keys, int B, int max_q, cudaStream_t st) {
-  if (keys == 64) return launch_prefill<D, HB, 64>(p, B, max_q, st);
-  if (keys == 32) return launch_prefill<D, HB, 32>(p, B, max_q, st);
-  return launch_prefill<D, HB, 16>(p, B, max_q, st);
+
+template <int D, int HB, int KT>
+static int launch_prefill(const TalkPrefillParams& p, const void* kc, const void* vc, int B, int max_q, cudaStream_t st) {
+  if (p.group % (2 * HB) == 0) return launch_units<D, HB, KT, 2>(p, kc, vc, B, max_q, st);
+  return launch_units<D, HB, KT, 1>(p, kc, vc, B, max_q, st);
 }
 
-// Keys per tile of the prompt kernel for these sizes, 0: it has no instance.
+// Keys per tile, stages and blocks of queries of the prompt kernel for these sizes; false: it has no instance.
+template <int D, int HB>
+static bool plan_prefill(int hq, int hkv, int& keys, int& stages, int& blocks) {
+  const int most = 16 * HB / hq > 0 ? 16 * HB / hq : 1;
+  for (int st = 2; st >= 1; --st)
+    for (int kt = 32; kt >= 16; kt /= 2)
+      for (int n = most; n >= (most + 1) / 2; --n) {
+        const size_t b = kt == 32 ? TalkCfg<D, HB, 32>::bytes(hkv, n, st) : TalkCfg<D, HB, 16>::bytes(hkv, n, st);
+        if (b <= kTalkSmem) { keys = kt; stages = st; blocks = n; return true; }
+      }
+  return false;
+}
+static bool plan_prefill(int hq, int hkv, int D, int& keys, int& stages, int& blocks) {
+  if (hq <= 0 || hkv <= 0 || hq % hkv || hq > 32 || (D != 64 && D != 128)) return false;
+  if (hq <= 16) return D == 64 ? plan_prefill<64, 1>(hq, hkv, keys, stages, blocks) : plan_prefill<128, 1>(hq, hkv, keys, stages, blocks);
+  if (hq / hkv % 2) return false;                          // two heads of a unit share their keys
+  return D == 64 ? plan_prefill<64, 2>(hq, hkv, keys, stages, blocks) : plan_prefill<128, 2>(hq, hkv, keys, stages, blocks);
+}
 extern "C" int xft_talking_prefill_keys(int hq, int hkv, int D) {
-  if (hq <= 0 || hkv <= 0 || hq % hkv || hq > 32 || (D != 64 && D != 128)) return 0;
-  const int hb = hq > 16 ? 2 : 1;
-  if (hb == 2 && (hq / hkv) % 2) return 0;                 // two heads of a unit share their keys
-  const int blocks = 16 * hb / hq > 0 ? 16 * hb / hq : 1, hp = hb == 1 ? 16 : 32, qpb = 16 / hb;
-  for (int kt = 64; kt >= 16; kt /= 2)
-    if (((size_t)2 * hkv * kt * (D + 8) + hp * (hp + 8) + (size_t)2 * blocks * hp * (qpb * (kt + 8) + 8)) * 2 <= 227 * 1024) return kt;
-  return 0;
+  int keys, stages, blocks;
+  return plan_prefill(hq, hkv, D, keys, stages, blocks) ? keys : 0;
 }
 
 // bf16: q [T, hq, D], gate and out [T, ld] (head h at columns h * D), caches [num_blocks, hkv, bs, D] with bs a multiple of 64; r1, r2
@@ -519,28 +667,52 @@ extern "C" int xft_talking_prefill(const void* q, const void* gate, int ldg, voi
                                    int hkv, int D, int bs, int num_blocks, float scale, const float* r1, const float* r2, const float* talk,
                                    int window, float mult, int* status, cudaStream_t st) {
   if (B <= 0 || max_q <= 0) return 0;
-  const int keys = xft_talking_prefill_keys(hq, hkv, D);
-  if (!keys || bs <= 0 || bs % 64 || window < 0 || ldg < hq * D || ldo < hq * D || ((ldg | ldo) & 1) || B > 65535) return -1;
+  int keys, stages, blocks;
+  if (!plan_prefill(hq, hkv, D, keys, stages, blocks) || bs <= 0 || bs % 64 || window < 0 || ldg < hq * D || ldo < hq * D || ((ldg | ldo) & 1) ||
+      B > 65535 || (long long)num_blocks * hkv * bs >= (1ll << 31)) return -1;
   if (((uintptr_t)q | (uintptr_t)kc | (uintptr_t)vc) & 15 || ((uintptr_t)gate | (uintptr_t)out) & 3) return -2;
-  const int hb = hq > 16 ? 2 : 1, blocks = 16 * hb / hq > 0 ? 16 * hb / hq : 1;
-  TalkPrefillParams p{(const bf16*)q, (const bf16*)gate, ldg, (bf16*)out, ldo, (const bf16*)kc, (const bf16*)vc, block_table, bt_stride, cu_q,
-                      kv_lens, hq, hkv, hq / hkv, bs, num_blocks, window > 0 ? min(window, 1 << 30) : 1 << 30, blocks * hq / hb, blocks,
+  const int hb = hq > 16 ? 2 : 1;
+  TalkPrefillParams p{(const bf16*)q, (const bf16*)gate, ldg, (bf16*)out, ldo, block_table, bt_stride, cu_q,
+                      kv_lens, hq, hkv, hq / hkv, bs, num_blocks, window > 0 ? min(window, 1 << 30) : 1 << 30, blocks * hq / hb, blocks, stages,
                       scale * kTalkLog2e, mult, r1, r2, talk, status};
-  if (D == 64) return hb == 1 ? prefill_keys<64, 1>(p, keys, B, max_q, st) : prefill_keys<64, 2>(p, keys, B, max_q, st);
-  return hb == 1 ? prefill_keys<128, 1>(p, keys, B, max_q, st) : prefill_keys<128, 2>(p, keys, B, max_q, st);
+  if (D == 64) {
+    if (hb == 1) return keys == 32 ? launch_prefill<64, 1, 32>(p, kc, vc, B, max_q, st) : launch_prefill<64, 1, 16>(p, kc, vc, B, max_q, st);
+    return keys == 32 ? launch_prefill<64, 2, 32>(p, kc, vc, B, max_q, st) : launch_prefill<64, 2, 16>(p, kc, vc, B, max_q, st);
+  }
+  if (hb == 1) return keys == 32 ? launch_prefill<128, 1, 32>(p, kc, vc, B, max_q, st) : launch_prefill<128, 1, 16>(p, kc, vc, B, max_q, st);
+  return keys == 32 ? launch_prefill<128, 2, 32>(p, kc, vc, B, max_q, st) : launch_prefill<128, 2, 16>(p, kc, vc, B, max_q, st);
 }
 
 template <int D, int GR>
 static cudaError_t launch_values(const TalkDecodeParams& p, cudaStream_t st) {
-  const size_t work = (size_t)p.hq * 64 + 64 * GR + p.group * p.hq + 2 * p.hq, end = (size_t)512 / D * GR * D;
-  const size_t smem = (work > end ? work : end) * sizeof(float);
+  const size_t work = (size_t)p.hq * 64 + 64 * GR + p.group * p.hq + 2 * p.hq, end = (size_t)kTalkValues * 4 * GR;
+  const size_t smem = (GR * D + (work > end ? work : end)) * sizeof(float);
   static size_t allowed = 48 * 1024;
   if (smem > allowed) {
     const cudaError_t e = cudaFuncSetAttribute(talking_values_kernel<D, GR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
     allowed = smem;
   }
-  return launch_pdl(talking_values_kernel<D, GR>, dim3(p.splits, p.hkv, p.B), dim3(128), smem, st, p);
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(p.splits, p.hkv, p.B);
+  cfg.blockDim = dim3(kTalkValues);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = st;
+  cudaLaunchAttribute at[2];
+  int na = 0;
+  if (p.splits > 1) {
+    at[na].id = cudaLaunchAttributeClusterDimension;
+    at[na].val.clusterDim.x = p.splits; at[na].val.clusterDim.y = 1; at[na].val.clusterDim.z = 1;
+    ++na;
+  }
+  if (g_xft_pdl) {
+    at[na].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[na].val.programmaticStreamSerializationAllowed = 1;
+    ++na;
+  }
+  cfg.attrs = at;
+  cfg.numAttrs = na;
+  return cudaLaunchKernelEx(&cfg, talking_values_kernel<D, GR>, p);
 }
 template <int D>
 static int launch_decode(const TalkDecodeParams& p, cudaStream_t st) {
@@ -551,22 +723,21 @@ static int launch_decode(const TalkDecodeParams& p, cudaStream_t st) {
   return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }
 
-// One token per sequence: q [B, hq, D] and the rest as above, heads of 64, 128 or 256, up to 16 per key/value head and 128 in all.  Scratch:
-// scores [B * hq * span] with span a multiple of 64, at least 64 * (pages that a window can touch); part_ml [B * hq * splits * 2], part_o
-// [B * hq * splits * D], counters [B * hkv] zeros (left as zeros).
+// One token per sequence: q [B, hq, D] and the rest as above, heads of 64, 128 or 256, up to 16 per key/value head and 128 in all.  splits:
+// key ranges, up to 8.  Scratch: scores [B * hq * span] with span a multiple of 64, at least 64 * (pages that a window can touch); part_ml
+// [B * hq * splits * 2].
 extern "C" int xft_talking_decode(const void* q, const void* gate, int ldg, void* out, int ldo, const void* kc, const void* vc,
                                   const int* block_table, int bt_stride, const int* kv_lens, int B, int hq, int hkv, int D, int bs,
                                   int num_blocks, float scale, const float* r1, const float* r2, const float* talk, int window, float mult,
-                                  int splits, int span, float* scores, float* part_ml, float* part_o, int* counters, int* status,
-                                  cudaStream_t st) {
+                                  int splits, int span, float* scores, float* part_ml, int* status, cudaStream_t st) {
   if (B <= 0) return 0;
-  if (hq <= 0 || hkv <= 0 || hq % hkv || hq / hkv > 16 || hq > 128 || bs <= 0 || bs % 64 || window < 0 || splits < 1 || (span & 63) || span <= 0)
+  if (hq <= 0 || hkv <= 0 || hq % hkv || hq / hkv > 16 || hq > 128 || bs <= 0 || bs % 64 || window < 0 || splits < 1 || splits > 8 || (span & 63) || span <= 0)
     return -1;
   if (ldg < hq * D || ldo < hq * D || B > 65535 || hkv > 65535) return -2;
-  if (((uintptr_t)q | (uintptr_t)kc | (uintptr_t)vc | (uintptr_t)scores) & 15) return -3;
+  if (((uintptr_t)q | (uintptr_t)kc | (uintptr_t)vc | (uintptr_t)scores | (uintptr_t)part_ml) & 15) return -3;
   TalkDecodeParams p{(const bf16*)q, (const bf16*)gate, ldg, (bf16*)out, ldo, (const bf16*)kc, (const bf16*)vc, block_table, bt_stride, kv_lens,
                      B, hq, hkv, hq / hkv, bs, num_blocks, window > 0 ? min(window, 1 << 30) : 1 << 30, splits, span, scale * kTalkLog2e, mult,
-                     r1, r2, talk, scores, part_ml, part_o, counters, status};
+                     r1, r2, talk, scores, part_ml, status};
   if (D == 64) return launch_decode<64>(p, st);
   if (D == 128) return launch_decode<128>(p, st);
   if (D == 256) return launch_decode<256>(p, st);

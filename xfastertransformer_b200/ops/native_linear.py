@@ -161,17 +161,21 @@ def state_space(x, d, w, eps, state, conv_state, state_slots, cu_q, kv_lens, met
                                      N._p(conv_state), slots, ns, N._p(u), u.shape[1], int(decode), f32, N._p(ws.status), N._stream()),
              f"channel_conv ({d.taps} taps)")
     ws.launches += 1 if decode or d.taps == 1 else 2
-    y = torch.empty(T, d.inner, dtype=torch.float32, device=dev)
+    y = torch.empty(T, d.inner, dtype=x.dtype, device=dev)
     b_at, c_at, per = d.inner, d.inner + d.groups * d.state, d.heads // d.groups
     dt, vectors = x[:, d.dt_at:], (N._p(w.dt_bias), N._p(w.rate), N._p(w.skip))
     least = NO_LIMIT
-    if not decode and not exact and _fn("xft_ssd_has_chunk")(d.state):
+    ctas = 0 if decode or exact else _fn("xft_ssd_chunk_ctas")(d.heads, per, d.state, d.vdim)
+    if ctas:
         least = max(1, N._ENV().ssd_chunk_min_q)
         sizes = [cu_q[i + 1] - cu_q[i] for i in range(B)]
         if max(sizes) >= least:
+            segs = segments(sum(n >= least for n in sizes) * ctas, max(sizes))
+            ss, sd = (torch.empty(B, d.heads, segs, n, dtype=torch.float32, device=dev) if segs > 1 else None for n in (d.state * d.vdim, 1))
             N._check(_fn("xft_ssd_chunk")(N._p(u), u.shape[1], b_at, c_at, N._p(dt), ldx, *vectors, d.heads, per, d.state, d.vdim, N._p(state),
-                                          slots, ns, N._p(cu), N._p(lens), B, N._p(y), least, N._p(ws.status), N._stream()), "ssd_chunk")
-            ws.launches += 1
+                                          slots, ns, N._p(cu), N._p(lens), B, N._p(y), least, segs, N._p(ss), N._p(sd), N._p(ws.status),
+                                          N._stream()), "ssd_chunk")
+            ws.launches += 1 + (segs > 1)
     if least == NO_LIMIT or min(sizes) < least:
         N._check(_fn("xft_ssd_step")(N._p(u), u.shape[1], c_at, b_at, 0, d.heads, per, d.state, d.vdim, N._p(dt), ldx, *vectors, N._p(state),
                                      slots, ns, N._p(cu), N._p(lens), B, N._p(y), 1, least, ssd_columns(B * d.heads, d.state, d.vdim), f32,

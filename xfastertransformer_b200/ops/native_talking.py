@@ -55,8 +55,11 @@ def _rows(q, x, d, out):
 
 
 def decode_splits(units: int, pages: int) -> int:
-    """Key ranges of a decode step: enough CTAs of 128 threads for the SMs, at least two pages each."""
-    return max(1, min(6 * 148 // max(units, 1), (pages + 1) // 2, 32))
+    """Key ranges of a decode step, a cluster of CTAs: enough for four per SM, at least two pages each."""
+    n = 1
+    while n < 8 and n * units < 4 * 148 and pages >= 4 * n:
+        n *= 2
+    return n
 
 
 def _decode(q, x, d, kc, vc, block_table, lens, B, max_kv, scale, window, out):
@@ -66,17 +69,14 @@ def _decode(q, x, d, kc, vc, block_table, lens, B, max_kv, scale, window, out):
     pages = (max_kv + 63) // 64
     if window > 0:
         pages = min(pages, (window + 62) // 64 + 1)
-    if B * hkv > ws.attn_counters.numel():
-        raise N.KernelError("mixed heads: more key/value heads in a batch than counters")
     splits = decode_splits(B * hkv, pages)
     f32 = lambda *s: torch.empty(*s, dtype=torch.float32, device=q.device)
     scores, ml = f32(B, H, pages * 64), f32(B, H, splits, 2)
-    po = f32(B, H, splits, D) if splits > 1 else None
     f = C.c_float
     N._check(_fn("xft_talking_decode")(
         *_rows(q, x, d, out), N._p(kc), N._p(vc), N._p(block_table), block_table.stride(0), N._p(lens), B, H, hkv, D, bs, nb, f(scale),
-        N._p(d.r1), N._p(d.r2), N._p(d.talk), window, f(d.mult), splits, pages * 64, N._p(scores), N._p(ml), N._p(po),
-        N._p(ws.attn_counters), N._p(ws.status), N._stream()), "talking_decode")
+        N._p(d.r1), N._p(d.r2), N._p(d.talk), window, f(d.mult), splits, pages * 64, N._p(scores), N._p(ml),
+        N._p(ws.status), N._stream()), "talking_decode")
     ws.launches += 2
     return out
 
