@@ -25,8 +25,9 @@ struct TalkPrefillParams {
   const bf16* q; const bf16* gate; int ldg; bf16* out; int ldo;
   const int* block_table; int bt_stride;
   const int* cu_q; const int* kv_lens;
-  int hq, hkv, group, bs, num_blocks, window;
+  int hq, hkv, group, num_blocks, window;
   int units, blocks;                         // units of 16 rows, blocks of queries (units = blocks * hq / heads per unit)
+  int bs_shift;                              // log2 of the page size
   int stages;                                // tiles of keys in shared memory, 1 or 2
   float scale2, mult;                        // softmax scale * log2(e)
   const float* r1; const float* r2; const float* talk;
@@ -119,19 +120,19 @@ __global__ void __launch_bounds__(kTalkUnits / U * 32, 1) talking_prefill_kernel
   const int* bt = p.block_table + (size_t)b * p.bt_stride;
   // tile buffers are filled by one thread, behind a barrier that says everyone is done with what was there
   uint32_t phases = 0;
-  const int page0 = k_lo / p.bs;
-  for (int i = tid; i < kTalkPages && i <= (k_lo + (n_tiles - 1) * KT) / p.bs - page0; i += NT) pages[i] = bt[page0 + i];
+  const int page0 = k_lo >> p.bs_shift;
+  for (int i = tid; i < kTalkPages && i <= ((k_lo + (n_tiles - 1) * KT) >> p.bs_shift) - page0; i += NT) pages[i] = bt[page0 + i];
   __syncthreads();
   auto load = [&](int buf, const CUtensorMap& map, int tile, int by) {
     if (tile >= n_tiles || tid != by * 32) return;
-    const int page = (k_lo + tile * KT) / p.bs - page0;
+    const int key = k_lo + tile * KT, page = (key >> p.bs_shift) - page0;
     int blk = page < kTalkPages ? pages[page] : bt[page0 + page];
     if (blk < 0 || blk >= p.num_blocks) { if (p.status) atomicCAS(p.status, 0, XFT_ERR_BOUNDS); blk = 0; }
     mbar_expect_tx(&full[buf], tile_size * 2);
     uint8_t* dst = reinterpret_cast<uint8_t*>(sT + (size_t)buf * tile_size);
 #pragma unroll
     for (int c = 0; c < D / 64; ++c)
-      tma_load_3d(dst + c * p.hkv * BOX, &map, &full[buf], c * 64, (k_lo + tile * KT) % p.bs, blk * p.hkv, kEvictNormal);
+      tma_load_3d(dst + c * p.hkv * BOX, &map, &full[buf], c * 64, key & ((1 << p.bs_shift) - 1), blk * p.hkv, kEvictNormal);
   };
   auto arrived = [&](int buf) {                                        // a wait that runs out is reported; what was there is read
     mbar_wait(&full[buf], phases >> buf & 1, p.status, XFT_ERR_WAIT_FULL);
@@ -613,7 +614,7 @@ __global__ void __launch_bounds__(kTalkValues) talking_values_kernel(const TalkD
 using namespace xft;
 
 template <int D, int HB, int KT, int U>
-static int launch_units(const TalkPrefillParams& p, const void* kc, const void* vc, int B, int max_q, cudaStream_t st) {
+static int launch_units(const TalkPrefillParams& p, const void* kc, const void* vc, int bs, int B, int max_q, cudaStream_t st) {
   using Cfg = TalkCfg<D, HB, KT>;
   const size_t smem = Cfg::bytes(p.hkv, p.blocks, p.stages);
   if (smem > kTalkSmem) return -6;
@@ -626,15 +627,15 @@ static int launch_units(const TalkPrefillParams& p, const void* kc, const void* 
   const int qt = p.blocks * Cfg::QPB;
   CUtensorMap tmK, tmV;
   const uint64_t groups = (uint64_t)p.num_blocks * p.hkv;
-  if (make_tensor_map_groups(&tmK, kc, groups, p.bs, D, p.hkv, KT) || make_tensor_map_groups(&tmV, vc, groups, p.bs, D, p.hkv, KT)) return -4;
+  if (make_tensor_map_groups(&tmK, kc, groups, bs, D, p.hkv, KT) || make_tensor_map_groups(&tmV, vc, groups, bs, D, p.hkv, KT)) return -4;
   cudaError_t e = launch_pdl(talking_prefill_kernel<D, HB, KT, U>, dim3((max_q + qt - 1) / qt, B), dim3(kTalkUnits / U * 32), smem, st, tmK, tmV, p);
   return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }
 
 template <int D, int HB, int KT>
-static int launch_prefill(const TalkPrefillParams& p, const void* kc, const void* vc, int B, int max_q, cudaStream_t st) {
-  if (p.group % (2 * HB) == 0) return launch_units<D, HB, KT, 2>(p, kc, vc, B, max_q, st);
-  return launch_units<D, HB, KT, 1>(p, kc, vc, B, max_q, st);
+static int launch_prefill(const TalkPrefillParams& p, const void* kc, const void* vc, int bs, int B, int max_q, cudaStream_t st) {
+  if (p.group % (2 * HB) == 0) return launch_units<D, HB, KT, 2>(p, kc, vc, bs, B, max_q, st);
+  return launch_units<D, HB, KT, 1>(p, kc, vc, bs, B, max_q, st);
 }
 
 // Keys per tile, stages and blocks of queries of the prompt kernel for these sizes; false: it has no instance.
@@ -660,27 +661,29 @@ extern "C" int xft_talking_prefill_keys(int hq, int hkv, int D) {
   return plan_prefill(hq, hkv, D, keys, stages, blocks) ? keys : 0;
 }
 
-// bf16: q [T, hq, D], gate and out [T, ld] (head h at columns h * D), caches [num_blocks, hkv, bs, D] with bs a multiple of 64; r1, r2
-// [hq], talk [hq, hq] fp32 (of bf16 values).  window 0: every earlier key.
+// bf16: q [T, hq, D], gate and out [T, ld] (head h at columns h * D), caches [num_blocks, hkv, bs, D] with bs a power of two, at least 64;
+// r1, r2 [hq], talk [hq, hq] fp32 (of bf16 values).  window 0: every earlier key.
 extern "C" int xft_talking_prefill(const void* q, const void* gate, int ldg, void* out, int ldo, const void* kc, const void* vc,
                                    const int* block_table, int bt_stride, const int* cu_q, const int* kv_lens, int B, int max_q, int hq,
                                    int hkv, int D, int bs, int num_blocks, float scale, const float* r1, const float* r2, const float* talk,
                                    int window, float mult, int* status, cudaStream_t st) {
   if (B <= 0 || max_q <= 0) return 0;
   int keys, stages, blocks;
-  if (!plan_prefill(hq, hkv, D, keys, stages, blocks) || bs <= 0 || bs % 64 || window < 0 || ldg < hq * D || ldo < hq * D || ((ldg | ldo) & 1) ||
+  int shift = 6;
+  while (shift < 20 && (1 << shift) < bs) ++shift;
+  if (!plan_prefill(hq, hkv, D, keys, stages, blocks) || bs != 1 << shift || window < 0 || ldg < hq * D || ldo < hq * D || ((ldg | ldo) & 1) ||
       B > 65535 || (long long)num_blocks * hkv * bs >= (1ll << 31)) return -1;
   if (((uintptr_t)q | (uintptr_t)kc | (uintptr_t)vc) & 15 || ((uintptr_t)gate | (uintptr_t)out) & 3) return -2;
   const int hb = hq > 16 ? 2 : 1;
   TalkPrefillParams p{(const bf16*)q, (const bf16*)gate, ldg, (bf16*)out, ldo, block_table, bt_stride, cu_q,
-                      kv_lens, hq, hkv, hq / hkv, bs, num_blocks, window > 0 ? min(window, 1 << 30) : 1 << 30, blocks * hq / hb, blocks, stages,
+                      kv_lens, hq, hkv, hq / hkv, num_blocks, window > 0 ? min(window, 1 << 30) : 1 << 30, blocks * hq / hb, blocks, shift, stages,
                       scale * kTalkLog2e, mult, r1, r2, talk, status};
   if (D == 64) {
-    if (hb == 1) return keys == 32 ? launch_prefill<64, 1, 32>(p, kc, vc, B, max_q, st) : launch_prefill<64, 1, 16>(p, kc, vc, B, max_q, st);
-    return keys == 32 ? launch_prefill<64, 2, 32>(p, kc, vc, B, max_q, st) : launch_prefill<64, 2, 16>(p, kc, vc, B, max_q, st);
+    if (hb == 1) return keys == 32 ? launch_prefill<64, 1, 32>(p, kc, vc, bs, B, max_q, st) : launch_prefill<64, 1, 16>(p, kc, vc, bs, B, max_q, st);
+    return keys == 32 ? launch_prefill<64, 2, 32>(p, kc, vc, bs, B, max_q, st) : launch_prefill<64, 2, 16>(p, kc, vc, bs, B, max_q, st);
   }
-  if (hb == 1) return keys == 32 ? launch_prefill<128, 1, 32>(p, kc, vc, B, max_q, st) : launch_prefill<128, 1, 16>(p, kc, vc, B, max_q, st);
-  return keys == 32 ? launch_prefill<128, 2, 32>(p, kc, vc, B, max_q, st) : launch_prefill<128, 2, 16>(p, kc, vc, B, max_q, st);
+  if (hb == 1) return keys == 32 ? launch_prefill<128, 1, 32>(p, kc, vc, bs, B, max_q, st) : launch_prefill<128, 1, 16>(p, kc, vc, bs, B, max_q, st);
+  return keys == 32 ? launch_prefill<128, 2, 32>(p, kc, vc, bs, B, max_q, st) : launch_prefill<128, 2, 16>(p, kc, vc, bs, B, max_q, st);
 }
 
 template <int D, int GR>

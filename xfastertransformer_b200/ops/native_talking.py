@@ -39,7 +39,7 @@ def talking_attention(q, x, d, kc, vc, block_table, cu_q, kv_lens, scale, window
     if q.dtype == torch.bfloat16 and kc.shape[2] % 64 == 0 and _ENV().talking_tc:
         if decode and can_decode(H, kc.shape[1], D):
             return _decode(q, x, d, kc, vc, block_table, lens, B, max_kv, scale, window, out)
-        if _fn("xft_talking_prefill_keys")(H, kc.shape[1], D):
+        if kc.shape[2] & (kc.shape[2] - 1) == 0 and _fn("xft_talking_prefill_keys")(H, kc.shape[1], D):
             max_q = meta.max_q if meta is not None and meta.max_q else max(cu_q[i + 1] - cu_q[i] for i in range(B))
             return _prefill(q, x, d, kc, vc, block_table, cu, lens, B, max_q, scale, window, out)
     return _plain(q, x, d, kc, vc, block_table, cu, lens, B, scale, window, out)
