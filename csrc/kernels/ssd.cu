@@ -88,8 +88,12 @@ __global__ void __launch_bounds__(128) channel_conv_kernel(const ChannelConvPara
   int b = ss_sequence(p.cu_q, p.B, t0), start = p.cu_q[b], end = p.cu_q[b + 1];
   bool fresh = true;
   float u[TAPS][VEC];
-  V next = *reinterpret_cast<const V*>(x + (size_t)t0 * p.ldx);        // the row ahead is on its way while one is summed up
-  for (int t = t0; t < t1; ++t) {
+  constexpr int AHEAD = 4;                                 // rows on their way while one is summed up
+  V ahead[AHEAD];
+#pragma unroll
+  for (int s = 0; s < AHEAD; ++s)
+    if (t0 + s < t1) ahead[s] = *reinterpret_cast<const V*>(x + (size_t)(t0 + s) * p.ldx);
+  auto step = [&](int t, V& row) {
     while (b + 1 < p.B && t >= end) { ++b; start = end; end = p.cu_q[b + 1]; fresh = true; }
     const int li = t - start;
     T* st = nullptr;
@@ -110,8 +114,8 @@ __global__ void __launch_bounds__(128) channel_conv_kernel(const ChannelConvPara
       fresh = false;
     }
 #pragma unroll
-    for (int k = 0; k < VEC; ++k) u[TAPS - 1][k] = ss_f32<T>(next.e[k]);
-    if (t + 1 < t1) next = *reinterpret_cast<const V*>(x + (size_t)(t + 1) * p.ldx);
+    for (int k = 0; k < VEC; ++k) u[TAPS - 1][k] = ss_f32<T>(row.e[k]);
+    if (t + AHEAD < t1) row = *reinterpret_cast<const V*>(x + (size_t)(t + AHEAD) * p.ldx);
     V y;
 #pragma unroll
     for (int k = 0; k < VEC; ++k) {
@@ -135,14 +139,18 @@ __global__ void __launch_bounds__(128) channel_conv_kernel(const ChannelConvPara
     for (int j = 0; j + 1 < TAPS; ++j)
 #pragma unroll
       for (int k = 0; k < VEC; ++k) u[j][k] = u[j + 1][k];
-  }
+  };
+  for (int t = t0; t < t1; t += AHEAD)
+#pragma unroll
+    for (int s = 0; s < AHEAD; ++s)
+      if (t + s < t1) step(t + s, ahead[s]);
 }
 
 // ------------------------------------------------------------------------------------------ gate and grouped norm
 // One CTA per (token, part); a thread has 8 neighbouring values up to twice.
-__global__ void __launch_bounds__(256) gated_norm_vec_kernel(const bf16* __restrict__ y, int ldy, const bf16* __restrict__ z, int ldz,
+__global__ void __launch_bounds__(1024) gated_norm_vec_kernel(const bf16* __restrict__ y, int ldy, const bf16* __restrict__ z, int ldz,
                                                              const float* __restrict__ gain, bf16* __restrict__ out, int ldo, int n, float eps) {
-  __shared__ float sh[8];
+  __shared__ float sh[32];
   const int t = blockIdx.y, c0 = blockIdx.x * n, nt = blockDim.x;
   grid_dep_launch();
   grid_dep_wait();
@@ -569,8 +577,8 @@ extern "C" int xft_gated_norm(const void* y, int ldy, const void* z, int ldz, co
                               float eps, int f32, cudaStream_t st) {
   if (T <= 0) return 0;
   if (parts <= 0 || n <= 0 || ldy < parts * n || ldz < parts * n || ldo < parts * n) return -1;
-  const bool vec = !f32 && n <= 4096 && ((n | ldy | ldz | ldo) & 7) == 0 && (((uintptr_t)y | (uintptr_t)z | (uintptr_t)out | (uintptr_t)gain) & 15) == 0;
-  const int nt = vec ? (n <= 512 ? 32 : n <= 1024 ? 64 : n <= 2048 ? 128 : 256) : n <= 512 ? 64 : n <= 2048 ? 128 : 256;
+  const bool vec = !f32 && n <= 16384 && ((n | ldy | ldz | ldo) & 7) == 0 && (((uintptr_t)y | (uintptr_t)z | (uintptr_t)out | (uintptr_t)gain) & 15) == 0;
+  const int nt = vec ? (n <= 512 ? 32 : n <= 1024 ? 64 : n <= 2048 ? 128 : n <= 4096 ? 256 : n <= 8192 ? 512 : 1024) : n <= 512 ? 64 : n <= 2048 ? 128 : 256;
   for (int t0 = 0; t0 < T; t0 += 65535) {                  // the grid's second dimension
     const dim3 grid(parts, T - t0 < 65535 ? T - t0 : 65535);
     const size_t ay = (size_t)t0 * ldy, az = (size_t)t0 * ldz, ao = (size_t)t0 * ldo;

@@ -354,7 +354,8 @@ def test_state_space(dtype, tol, H, P, N, G, parts, taps, sizes):
 
 @STATES
 @pytest.mark.parametrize("H,P,N,G,parts,taps", [(1, 200, 256, 1, 1, 8), (2, 136, 300, 2, 4, 5), (3, 21, 33, 1, 3, 1), (2, 128, 96, 2, 1, 4),
-                                                (2, 72, 200, 1, 6, 7), (64, 64, 16, 8, 1, 4)])
+                                                (2, 72, 200, 1, 6, 7), (64, 64, 16, 8, 1, 4), (80, 64, 16, 8, 1, 4), (72, 128, 8, 1, 1, 2),
+                                                (33, 512, 8, 1, 1, 1)])
 def test_state_space_sizes(dtype, tol, H, P, N, G, parts, taps):
     """Columns over several CTAs, sizes without a chunk instance, odd sizes, norm parts that cut through heads."""
     M.state_space(_dev(), dtype, tol, H, P, N, G, parts, taps, (100, 20, 3), (1000,))
@@ -370,6 +371,7 @@ def test_state_space_decays(dtype, tol, dt, rate):
 def test_state_space_long():
     """Runs of tokens per thread of the convolution that cross from one sequence into the next; many chunks."""
     M.state_space(_dev(), torch.bfloat16, 2e-2, 2, 64, 64, 1, 1, 4, (900, 3, 500, 1, 99), (4000,), -3.0)
+    M.state_space(_dev(), torch.bfloat16, 2e-2, 4, 16, 64, 1, 1, 3, (4101, 2, 4095), (9000,), -3.0)
 
 
 TALK = [(6, 3, 20, 64), (16, 4, 128, 128), (4, 4, 64, 64), (1, 1, 64, 64), (3, 1, 100, 128), (32, 8, 128, 128), (24, 2, 64, 64), (13, 13, 64, 64)]
