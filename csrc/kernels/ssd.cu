@@ -72,11 +72,24 @@ __global__ void __launch_bounds__(128) channel_conv_kernel(const ChannelConvPara
   if (c >= p.C) { grid_dep_wait(); return; }               // C is a multiple of VEC
   const int skip = TAPS - p.taps;
   float w[TAPS][VEC], bias[VEC];
+  auto row_of = [](const float* from, float (&v)[VEC]) {
+    constexpr int N = VEC % 4 ? 1 : 4;
+    struct alignas(4 * N) F { float e[N]; };
 #pragma unroll
-  for (int k = 0; k < VEC; ++k) {
-    bias[k] = p.bias[c + k];
+    for (int k = 0; k < VEC; k += N) {
+      const F r = *reinterpret_cast<const F*>(from + k);
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j) w[j][k] = j < skip ? 0.f : p.w[(size_t)(j - skip) * p.C + c + k];
+      for (int i = 0; i < N; ++i) v[k + i] = r.e[i];
+    }
+  };
+  row_of(p.bias + c, bias);
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) {
+    if (j >= skip) row_of(p.w + (size_t)(j - skip) * p.C + c, w[j]);
+    else {
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) w[j][k] = 0.f;
+    }
   }
   grid_dep_wait();
   const T* x = reinterpret_cast<const T*>(p.x) + c;
@@ -88,7 +101,7 @@ __global__ void __launch_bounds__(128) channel_conv_kernel(const ChannelConvPara
   int b = ss_sequence(p.cu_q, p.B, t0), start = p.cu_q[b], end = p.cu_q[b + 1];
   bool fresh = true;
   float u[TAPS][VEC];
-  constexpr int AHEAD = 4;                                 // rows on their way while one is summed up
+  constexpr int AHEAD = 2;                                 // rows on their way while one is summed up
   V ahead[AHEAD];
 #pragma unroll
   for (int s = 0; s < AHEAD; ++s)
@@ -563,7 +576,7 @@ extern "C" int xft_channel_conv(const void* x, int ldx, int T, int B, int C, int
   const int run = decode || T < 1024 ? 1 : T < 8192 ? 8 : 16;
   if ((T + run - 1) / run > 65535) return -2;
   ChannelConvParams p{x, ldx, T, B, C, taps, w, bias, cu_q, kv_lens, state, state_slots, num_states, out, ldo, run, decode, status};
-  const bool vec = ((C | ldx | ldo) & 7) == 0 && (((uintptr_t)x | (uintptr_t)out | (uintptr_t)state) & 15) == 0;
+  const bool vec = ((C | ldx | ldo) & 7) == 0 && (((uintptr_t)x | (uintptr_t)out | (uintptr_t)state | (uintptr_t)w | (uintptr_t)bias) & 15) == 0;
   cudaError_t e;
   if (f32) e = vec ? launch_conv<float, 4>(p, st) : launch_conv<float, 1>(p, st);
   else e = vec ? launch_conv<bf16, 8>(p, st) : launch_conv<bf16, 1>(p, st);
